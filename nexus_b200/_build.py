@@ -150,6 +150,66 @@ def build_host(force: bool = False, verbose: bool = False) -> Path:
     return out
 
 
+# what `ensure_serving` compiles where nothing has been built: the kernels and host code of the layered decoders
+SERVING_CUDA = ("attention_sm100", "gemm_sm100", "infer_kernels", "mixer_kernels", "paged_window_attention", "recurrent_chunk",
+                "recurrent_step")
+SERVING_HOST = ("cpu_kernels", "kv_sched", "module")
+
+
+def _current(out: Path, sources, header_dir: Path) -> bool:
+    return out.exists() and out.stat().st_mtime >= max([_newest_header([header_dir])] + [s.stat().st_mtime for s in sources])
+
+
+def ensure_serving(verbose: bool = False) -> None:
+    """Makes the native code that serving a decoder needs available in this process.  A complete build that is newer than
+    its sources is used as it is; otherwise the serving subset (`SERVING_CUDA`, `SERVING_HOST`) is compiled into
+    ``lib/serving/`` - a fresh checkout serves a model after compiling only that - and selected through
+    ``NEXUS_B200_CUDA_LIB`` / ``NEXUS_B200_NATIVE``.  Concurrent callers wait for one another on a lock file."""
+    import fcntl
+
+    full_cuda = _current(CUDA_LIB, cuda_sources(), CSRC / "cuda")
+    full_host = _current(native_module_path(), host_sources(), CSRC / "host")
+    if full_cuda and full_host:
+        return
+    out_dir = LIB_DIR / "serving"
+    out_dir.mkdir(parents=True, exist_ok=True)
+    cuda_out, host_out = out_dir / "libnexus_b200_cuda.so", out_dir / native_module_path().name
+    with open(out_dir / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        jobs, links = [], []
+        if not full_cuda:
+            nvcc, hdr, objs = _nvcc(), _newest_header([CSRC / "cuda"]), []
+            for name in SERVING_CUDA:
+                src, obj = CSRC / "cuda" / (name + ".cu"), out_dir / (name + ".o")
+                jobs.append((src, obj, [nvcc, *NVCC_FLAGS, "-I", str(CSRC / "cuda"), "-c", str(src), "-o", str(obj)], hdr))
+                objs.append(obj)
+            links.append((cuda_out, objs, [nvcc, "-shared", "-o", str(cuda_out), *map(str, objs), "-gencode",
+                                           "arch=compute_100a,code=sm_100a", "-cudart", "static"]))
+        if not full_host:
+            import pybind11
+
+            hdr, objs = _newest_header([CSRC / "host"]), []
+            inc = ["-I", pybind11.get_include(), "-I", sysconfig.get_paths()["include"], "-I", str(CSRC / "host")]
+            for name in SERVING_HOST:
+                src, obj = CSRC / "host" / (name + ".cpp"), out_dir / ("host_" + name + ".o")
+                jobs.append((src, obj, ["g++", *CXX_FLAGS, "-DNX_SERVING_ONLY", *inc, "-c", str(src), "-o", str(obj)], hdr))
+                objs.append(obj)
+            links.append((host_out, objs, ["g++", "-shared", "-o", str(host_out), *map(str, objs), "-pthread"]))
+        _compile_many(jobs, False)
+        for out, objs, cmd in links:
+            if not out.exists() or out.stat().st_mtime < max(o.stat().st_mtime for o in objs):
+                _run(cmd)
+                if verbose:
+                    print("linked", out, file=sys.stderr)
+    if not full_cuda:
+        os.environ["NEXUS_B200_CUDA_LIB"] = str(cuda_out)
+    if not full_host:
+        os.environ["NEXUS_B200_NATIVE"] = str(host_out)
+        import nexus_b200
+
+        nexus_b200._load_alternative_native()
+
+
 SANITIZERS = {"asan": ["-fsanitize=address,undefined", "-fno-sanitize-recover=undefined"], "tsan": ["-fsanitize=thread"]}
 
 

@@ -43,6 +43,7 @@ struct AttnDev {
   int items, nqb;      // fwd (persistent): number of work items = nqb * H * B, q blocks per (head, batch)
   float* merge_o;      // fwd: FP32 [B,Tq,H,D] running output of earlier key/value chunks (in/out), or null
   float* merge_lse;    // fwd: FP32 [B,H,Tq] running log-sum-exp (in/out)
+  float out_scale;     // fwd: factor of the written output (`out` only)
   float softcap;       // > 0: scores pass through softcap * tanh(scale * s / softcap)
   const float* alibi;  // [H] slopes or null: slope_h * (key position - query position) is added to the scaled score
   // dq kernel: forward output and its gradient as plain row views; the kernel forms dsum = rowsum(dO * O) itself
@@ -113,7 +114,7 @@ __device__ __forceinline__ float score_ext(const ScoreExt& e, float s, int rel, 
   float z = s * e.scale;
   dfac = 1.0f;
   if (e.cap > 0.0f) {
-    const float t = tanh_approx_f(z * e.inv_cap);
+    const float t = tanh_ex2_f(z * e.inv_cap);
     z = e.cap * t;
     dfac = 1.0f - t * t;
   }
@@ -578,7 +579,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
       }
       softmax_bar();  // every thread has read merge_lse / sX before they are written again
       if (ok && q < p.Tq) {
-        const float inv = l_run > 0.0f ? 1.0f / l_run : 0.0f;
+        const float inv = l_run > 0.0f ? p.out_scale / l_run : 0.0f;
         __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + static_cast<int64_t>(b) * p.o_batch +
                               static_cast<int64_t>(q) * p.o_row + static_cast<int64_t>(h) * p.o_head + half * HH;
 #pragma unroll
@@ -1037,7 +1038,7 @@ attn_fwd2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
           l_run = den > 0.0f ? 1.0f : 0.0f;  // o_acc now holds the normalised merged output
           m_fin = (den > 0.0f ? mm + logf(den) : -INFINITY) * kLog2e;
         }
-        const float inv = l_run > 0.0f ? 1.0f / l_run : 0.0f;
+        const float inv = l_run > 0.0f ? p.out_scale / l_run : 0.0f;
         __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + static_cast<int64_t>(w.b) * p.o_batch +
                               static_cast<int64_t>(q) * p.o_row + static_cast<int64_t>(w.h) * p.o_head;
 #pragma unroll
@@ -1706,6 +1707,7 @@ AttnDev base_params(const NxAttnArgs* a) {
   p.window = a->window;
   p.scale = a->scale;
   p.softcap = a->softcap;
+  p.out_scale = a->out_scale == 0.0f ? 1.0f : a->out_scale;
   p.alibi = a->alibi_slopes;
   p.dropout_p = a->dropout_p;
   p.drop_seed = a->dropout_seed;

@@ -1,0 +1,403 @@
+// Memory-bound building blocks of decoders with heterogeneous layers (see nx_api_mixers.h): the chain "add the normed
+// sublayer output, norm for the next sublayer", rotary embedding fused with the paged cache append, the short causal
+// convolution with its carried tail, gated norms, the per-layer token input, SwiGLU and logit soft-capping.
+// Everything is computed in FP32; activations are read and written in BF16 or FP32.
+#include "common.cuh"
+#include "mixer_common.cuh"
+#include "nx_api_mixers.h"
+
+#include <algorithm>
+
+namespace {
+using namespace nx;
+
+// ------------------------------------------------------------------------------------------------
+// residual chain: one block per row, the row stays in shared memory between the passes
+// ------------------------------------------------------------------------------------------------
+template <typename T, int V>
+__global__ void residual_norm_kernel(const NxResidualNormArgs a) {
+  extern __shared__ __align__(16) float s_row[];
+  __shared__ float s_red[32];
+  const int64_t r = blockIdx.x;
+  const int cols = a.cols;
+  float* xr = a.x + r * cols;
+  const float inv_cols = 1.0f / static_cast<float>(cols);
+  float ss = 0.0f;
+  if (a.table != nullptr) {
+    const T* e = static_cast<const T*>(a.table) + static_cast<int64_t>(a.tokens[r]) * cols;
+    for (int c = threadIdx.x * V; c < cols; c += blockDim.x * V) {
+      float v[V];
+      load_vec<T, V>(e + c, v);
+      store_vec<float, V>(xr + c, v);
+      store_vec<float, V>(s_row + c, v);
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += v[j] * v[j];
+    }
+  } else if (a.y != nullptr) {
+    const T* yr = static_cast<const T*>(a.y) + r * a.ldy;
+    float sy = 0.0f;
+    for (int c = threadIdx.x * V; c < cols; c += blockDim.x * V) {
+      float v[V];
+      load_vec<T, V>(yr + c, v);
+      store_vec<float, V>(s_row + c, v);
+#pragma unroll
+      for (int j = 0; j < V; ++j) sy += v[j] * v[j];
+    }
+    const float inv = 1.0f / sqrtf(block_sum(sy, s_red) * inv_cols + a.eps);
+    for (int c = threadIdx.x * V; c < cols; c += blockDim.x * V) {   // each thread re-reads its own columns
+      float v[V], xv[V], w[V];
+      load_vec<float, V>(s_row + c, v);
+      load_vec<float, V>(xr + c, xv);
+      load_vec<float, V>(a.w_post + c, w);
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        v[j] = xv[j] + v[j] * inv * w[j];
+        ss += v[j] * v[j];
+      }
+      store_vec<float, V>(xr + c, v);
+      store_vec<float, V>(s_row + c, v);
+    }
+  } else {
+    for (int c = threadIdx.x * V; c < cols; c += blockDim.x * V) {
+      float v[V];
+      load_vec<float, V>(xr + c, v);
+      store_vec<float, V>(s_row + c, v);
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += v[j] * v[j];
+    }
+  }
+  if (a.x_cast != nullptr) {
+    T* o = static_cast<T*>(a.x_cast) + r * a.ldh;
+    for (int c = threadIdx.x * V; c < cols; c += blockDim.x * V) {
+      float v[V];
+      load_vec<float, V>(s_row + c, v);
+      store_vec<T, V>(o + c, v);
+    }
+    for (int c = cols + threadIdx.x; c < a.ldh; c += blockDim.x) Num<T>::store(o + c, 0.0f);
+  }
+  if (a.h != nullptr) {
+    const float inv = 1.0f / sqrtf(block_sum(ss, s_red) * inv_cols + a.eps);
+    T* o = static_cast<T*>(a.h) + r * a.ldh;
+    for (int c = threadIdx.x * V; c < cols; c += blockDim.x * V) {
+      float v[V], w[V];
+      load_vec<float, V>(s_row + c, v);
+      load_vec<float, V>(a.w_next + c, w);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] *= inv * w[j];
+      store_vec<T, V>(o + c, v);
+    }
+    for (int c = cols + threadIdx.x; c < a.ldh; c += blockDim.x) Num<T>::store(o + c, 0.0f);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// rotary embedding (rotate-half layout, first rot_dims of a head) + cache append: one block per row
+// ------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void rope_append_kernel(const NxRopeAppendArgs a) {
+  const int64_t r = blockIdx.x;
+  const int half = a.rot_dims / 2;
+  T* row = static_cast<T*>(a.proj) + r * a.ld;
+  const int64_t pos = a.positions[r], slot = a.slots[r];
+  const float* cs = a.cos_t + pos * half;
+  const float* sn = a.sin_t + pos * half;
+  T* kc = static_cast<T*>(a.k_cache) + slot * a.kv_heads * a.dim;
+  T* vc = static_cast<T*>(a.v_cache) + slot * a.kv_heads * a.vdim;
+  const int nq = a.heads * half, nk = a.kv_heads * half;
+  for (int i = threadIdx.x; i < nq + nk; i += blockDim.x) {
+    const bool is_k = i >= nq;
+    const int u = is_k ? i - nq : i;
+    const int h = u / half, j = u % half;
+    T* p = row + (is_k ? a.k_off : a.q_off) + h * a.dim + j;
+    const float x0 = Num<T>::load(p), x1 = Num<T>::load(p + half), c = cs[j], s = sn[j];
+    const float y0 = x0 * c - x1 * s, y1 = x1 * c + x0 * s;
+    Num<T>::store(p, y0);
+    Num<T>::store(p + half, y1);
+    if (is_k && slot >= 0) {
+      Num<T>::store(kc + h * a.dim + j, y0);
+      Num<T>::store(kc + h * a.dim + j + half, y1);
+    }
+  }
+  if (slot < 0) return;
+  const int rest = a.dim - a.rot_dims;
+  for (int i = threadIdx.x; i < a.kv_heads * rest; i += blockDim.x) {
+    const int o = (i / rest) * a.dim + a.rot_dims + i % rest;
+    kc[o] = row[a.k_off + o];
+  }
+  for (int i = threadIdx.x; i < a.kv_heads * a.vdim; i += blockDim.x) vc[i] = row[a.v_off + i];
+}
+
+// ------------------------------------------------------------------------------------------------
+// causal convolution + SiLU.  A thread owns V adjacent channels over one tile of a segment's tokens;
+// the first tile reads the carried tail and is the one that writes the new one, so that no other
+// block touches the tail of this segment.
+// ------------------------------------------------------------------------------------------------
+constexpr int kConvTile = 32;
+
+template <typename T, int TAPS, int V>
+__global__ void conv_silu_kernel(const NxConvArgs a) {
+  const int sg = blockIdx.z;
+  const int len = a.seg.len[sg];
+  const int t0 = blockIdx.y * kConvTile;
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (t0 >= len || c >= a.channels) return;
+  const int64_t row0 = a.seg.row0[sg];
+  constexpr int HIST = TAPS > 1 ? TAPS - 1 : 1;
+  float w[TAPS][V], hist[HIST][V], bias[V];
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) load_vec<float, V>(a.w + static_cast<int64_t>(j) * a.channels + c, w[j]);
+#pragma unroll
+  for (int v = 0; v < V; ++v) bias[v] = a.bias != nullptr ? a.bias[c + v] : 0.0f;
+  const T* x = static_cast<const T*>(a.x) + row0 * a.ldx + c;
+  T* y = static_cast<T*>(a.y) + row0 * a.ldy + c;
+  T* st = static_cast<T*>(a.state) + static_cast<int64_t>(a.seg.seq[sg]) * (TAPS - 1) * a.channels + c;
+  const bool carried = a.seg.pos[sg] > 0;
+#pragma unroll
+  for (int j = 0; j < TAPS - 1; ++j) {
+    const int t = t0 - (TAPS - 1) + j;     // token of the segment this tap's first input is
+    if (t >= 0) {
+      load_vec<T, V>(x + static_cast<int64_t>(t) * a.ldx, hist[j]);
+    } else if (carried) {                  // only in the first tile: kConvTile >= TAPS - 1
+      load_vec<T, V>(st + static_cast<int64_t>(TAPS - 1 + t) * a.channels, hist[j]);
+    } else {
+#pragma unroll
+      for (int v = 0; v < V; ++v) hist[j][v] = 0.0f;
+    }
+  }
+  if (t0 == 0) {
+    float tail[HIST][V];
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) {
+      const int t = len - (TAPS - 1) + j;
+      if (t >= 0) {
+        load_vec<T, V>(x + static_cast<int64_t>(t) * a.ldx, tail[j]);
+      } else {                             // a segment shorter than the tail keeps the newest of the old inputs
+#pragma unroll
+        for (int i = 0; i < TAPS - 1; ++i)
+          if (i == TAPS - 1 + t)
+#pragma unroll
+            for (int v = 0; v < V; ++v) tail[j][v] = hist[i][v];
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) store_vec<T, V>(st + static_cast<int64_t>(j) * a.channels, tail[j]);
+  }
+  const int t1 = min(len, t0 + kConvTile);
+  for (int t = t0; t < t1; ++t) {
+    float cur[V], acc[V];
+    load_vec<T, V>(x + static_cast<int64_t>(t) * a.ldx, cur);
+#pragma unroll
+    for (int v = 0; v < V; ++v) acc[v] = bias[v] + w[TAPS - 1][v] * cur[v];
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+      for (int v = 0; v < V; ++v) acc[v] += w[j][v] * hist[j][v];
+#pragma unroll
+    for (int v = 0; v < V; ++v) acc[v] = silu_exact(acc[v]);
+    store_vec<T, V>(y + static_cast<int64_t>(t) * a.ldy, acc);
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+      for (int v = 0; v < V; ++v) hist[j][v] = j + 1 < TAPS - 1 ? hist[j + 1 < HIST ? j + 1 : j][v] : cur[v];
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// gated norm: a warp (small groups) or a block (large groups) per (row, group)
+// ------------------------------------------------------------------------------------------------
+constexpr int kGatedWarpCols = 512;
+
+template <typename T, bool kWarp>
+__global__ void gated_norm_kernel(const NxGatedNormArgs a) {
+  __shared__ float s_red[32];
+  const int lanes = kWarp ? 32 : blockDim.x;
+  const int64_t item = kWarp ? blockIdx.x * static_cast<int64_t>(blockDim.x >> 5) + (threadIdx.x >> 5) : blockIdx.x;
+  if (item >= static_cast<int64_t>(a.rows) * a.groups) return;   // whole warps (or blocks) leave together
+  const int lane = kWarp ? threadIdx.x & 31 : threadIdx.x;
+  const int64_t r = item / a.groups;
+  const int g = static_cast<int>(item % a.groups), n = a.group_size;
+  const T* y = static_cast<const T*>(a.y) + r * a.ldy + static_cast<int64_t>(g) * n;
+  const T* z = static_cast<const T*>(a.z) + r * a.ldz + static_cast<int64_t>(g) * n;
+  T* o = static_cast<T*>(a.out) + r * a.ldo + static_cast<int64_t>(g) * n;
+  const float* w = a.w + (a.w_shared ? 0 : static_cast<int64_t>(g) * n);
+  float ss = 0.0f;
+  for (int c = lane; c < n; c += lanes) {
+    float v = Num<T>::load(y + c);
+    if (a.gate_first) v *= silu_exact(Num<T>::load(z + c));
+    ss += v * v;
+  }
+  ss = kWarp ? warp_sum(ss) : block_sum(ss, s_red);
+  const float inv = a.out_scale / sqrtf(ss / static_cast<float>(n) + a.eps);
+  for (int c = lane; c < n; c += lanes)
+    Num<T>::store(o + c, Num<T>::load(y + c) * silu_exact(Num<T>::load(z + c)) * inv * w[c]);
+}
+
+// ------------------------------------------------------------------------------------------------
+// elementwise
+// ------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void token_side_kernel(const T* __restrict__ a, int64_t lda, const int32_t* __restrict__ tokens,
+                                  const T* __restrict__ table, int64_t ld_table, int offset, T* __restrict__ out,
+                                  int64_t ldo, int dim) {
+  const int64_t r = blockIdx.x;
+  const T* e = table + static_cast<int64_t>(tokens[r]) * ld_table + offset;
+  for (int j = threadIdx.x; j < ldo; j += blockDim.x) {
+    float v = 0.0f;
+    if (j < dim) v = gelu_tanh_exact(Num<T>::load(a + r * lda + j)) * Num<T>::load(e + j);
+    Num<T>::store(out + r * ldo + j, v);
+  }
+}
+
+template <typename T, int V>
+__global__ void silu_mul_kernel(const T* __restrict__ h, int64_t ldh, T* __restrict__ out, int64_t ldo, int half) {
+  const int64_t r = blockIdx.y;
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (c >= half) return;
+  float g[V], u[V];
+  load_vec<T, V>(h + r * ldh + c, g);
+  load_vec<T, V>(h + r * ldh + half + c, u);
+#pragma unroll
+  for (int j = 0; j < V; ++j) g[j] = silu_exact(g[j]) * u[j];
+  store_vec<T, V>(out + r * ldo + c, g);
+}
+
+__global__ void softcap_kernel(float* __restrict__ x, int64_t ld, int cols, float cap) {
+  float* xr = x + blockIdx.y * ld;
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c < cols) xr[c] = cap * tanhf(xr[c] / cap);
+}
+
+template <typename T, int V>
+int launch_conv(const NxConvArgs* a, cudaStream_t st) {
+  const int threads = 128;
+  dim3 grid((a->channels / V + threads - 1) / threads, (a->seg.max_len + kConvTile - 1) / kConvTile, a->seg.count);
+#define NX_CONV(TAPS_) \
+  case TAPS_: conv_silu_kernel<T, TAPS_, V><<<grid, threads, 0, st>>>(*a); break
+  switch (a->taps) {
+    NX_CONV(1); NX_CONV(2); NX_CONV(3); NX_CONV(4); NX_CONV(5); NX_CONV(6); NX_CONV(7); NX_CONV(8);
+    default: return -1;
+  }
+#undef NX_CONV
+  return launch_status();
+}
+
+template <typename T>
+int launch_residual(const NxResidualNormArgs* a, cudaStream_t st) {
+  const bool vec = a->cols % 4 == 0 && (a->y == nullptr || a->ldy % 4 == 0) && a->ldh % 4 == 0;
+  const int per = vec ? 4 : 1;
+  int threads = ((a->cols / per + 1) / 2 + 31) / 32 * 32;
+  threads = std::max(64, std::min(512, threads));
+  const size_t smem = static_cast<size_t>(a->cols) * sizeof(float);
+  if (smem > 200 * 1024) return -1;
+  if (smem > 48 * 1024) {
+    const cudaError_t e = vec ? cudaFuncSetAttribute(residual_norm_kernel<T, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)
+                              : cudaFuncSetAttribute(residual_norm_kernel<T, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
+    if (e != cudaSuccess) return -2;
+  }
+  if (vec) residual_norm_kernel<T, 4><<<a->rows, threads, smem, st>>>(*a);
+  else residual_norm_kernel<T, 1><<<a->rows, threads, smem, st>>>(*a);
+  return launch_status();
+}
+
+}  // namespace
+
+// ================================================================================================
+extern "C" int nx_residual_norm(const NxResidualNormArgs* a, nx_stream_t stream) {
+  if (a == nullptr || a->cols <= 0 || a->x == nullptr) return -1;
+  if (a->rows <= 0) return 0;
+  if (a->y != nullptr && a->w_post == nullptr) return -1;
+  if (a->h != nullptr && a->w_next == nullptr) return -1;
+  if ((a->h != nullptr || a->x_cast != nullptr) && a->ldh < a->cols) return -1;
+  if (a->table != nullptr && a->tokens == nullptr) return -1;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (a->dtype == NX_BF16) return launch_residual<__nv_bfloat16>(a, st);
+  if (a->dtype == NX_F32) return launch_residual<float>(a, st);
+  return -1;
+}
+
+extern "C" int nx_rope_append(const NxRopeAppendArgs* a, nx_stream_t stream) {
+  if (a == nullptr) return -1;
+  if (a->rows <= 0) return 0;
+  if (a->rot_dims < 0 || (a->rot_dims & 1) || a->rot_dims > a->dim) return -1;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int work = std::max(a->heads * a->rot_dims / 2, a->kv_heads * std::max(a->dim, a->vdim));
+  const int threads = std::max(64, std::min(256, (work + 31) / 32 * 32));
+  if (a->dtype == NX_BF16) rope_append_kernel<__nv_bfloat16><<<a->rows, threads, 0, st>>>(*a);
+  else if (a->dtype == NX_F32) rope_append_kernel<float><<<a->rows, threads, 0, st>>>(*a);
+  else return -1;
+  return launch_status();
+}
+
+extern "C" int nx_conv_silu(const NxConvArgs* a, nx_stream_t stream) {
+  if (a == nullptr || a->channels <= 0 || a->taps < 1 || a->taps > 8) return -1;
+  if (a->seg.count <= 0 || a->seg.max_len <= 0) return 0;
+  if (a->seg.count > 65535 || (a->seg.max_len + kConvTile - 1) / kConvTile > 65535) return -1;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool v2 = a->channels % 2 == 0 && a->ldx % 2 == 0 && a->ldy % 2 == 0 && (reinterpret_cast<uintptr_t>(a->x) & 7) == 0;
+  if (a->dtype == NX_BF16) return v2 ? launch_conv<__nv_bfloat16, 2>(a, st) : launch_conv<__nv_bfloat16, 1>(a, st);
+  if (a->dtype == NX_F32) return v2 ? launch_conv<float, 2>(a, st) : launch_conv<float, 1>(a, st);
+  return -1;
+}
+
+extern "C" int nx_gated_norm(const NxGatedNormArgs* a, nx_stream_t stream) {
+  if (a == nullptr || a->groups <= 0 || a->group_size <= 0) return -1;
+  if (a->rows <= 0) return 0;
+  if (a->dtype != NX_BF16 && a->dtype != NX_F32) return -1;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int64_t items = static_cast<int64_t>(a->rows) * a->groups;
+  if (items > 0x7fffffff) return -1;
+  if (a->group_size <= kGatedWarpCols) {
+    const int blocks = static_cast<int>((items + 7) / 8);
+    if (a->dtype == NX_BF16) gated_norm_kernel<__nv_bfloat16, true><<<blocks, 256, 0, st>>>(*a);
+    else gated_norm_kernel<float, true><<<blocks, 256, 0, st>>>(*a);
+  } else {
+    const int threads = std::min(512, (a->group_size / 4 + 31) / 32 * 32);
+    if (a->dtype == NX_BF16) gated_norm_kernel<__nv_bfloat16, false><<<static_cast<int>(items), threads, 0, st>>>(*a);
+    else gated_norm_kernel<float, false><<<static_cast<int>(items), threads, 0, st>>>(*a);
+  }
+  return launch_status();
+}
+
+extern "C" int nx_token_side_gate(const void* a, int64_t lda, const int32_t* tokens, const void* table, int64_t ld_table,
+                                  int offset, void* out, int64_t ldo, int rows, int dim, int dtype, nx_stream_t stream) {
+  if (dim <= 0 || ldo < dim) return -1;
+  if (rows <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int threads = std::max(32, std::min(256, static_cast<int>((ldo + 31) / 32 * 32)));
+  if (dtype == NX_BF16)
+    token_side_kernel<__nv_bfloat16><<<rows, threads, 0, st>>>((const __nv_bfloat16*)a, lda, tokens, (const __nv_bfloat16*)table,
+                                                               ld_table, offset, (__nv_bfloat16*)out, ldo, dim);
+  else if (dtype == NX_F32)
+    token_side_kernel<float><<<rows, threads, 0, st>>>((const float*)a, lda, tokens, (const float*)table, ld_table, offset,
+                                                       (float*)out, ldo, dim);
+  else
+    return -1;
+  return launch_status();
+}
+
+extern "C" int nx_silu_mul(const void* h, int64_t ldh, void* out, int64_t ldo, int rows, int half, int dtype,
+                           nx_stream_t stream) {
+  if (half <= 0) return -1;
+  if (rows <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool vec = half % 8 == 0 && ldh % 8 == 0 && ldo % 8 == 0;
+  for (int r0 = 0; r0 < rows; r0 += 65535) {
+    const int n = std::min(65535, rows - r0);
+    dim3 grid((half / (vec ? 8 : 1) + 127) / 128, n);
+#define NX_SM(T_, V_) \
+  silu_mul_kernel<T_, V_><<<grid, 128, 0, st>>>((const T_*)h + r0 * ldh, ldh, (T_*)out + r0 * ldo, ldo, half)
+    if (dtype == NX_BF16) { if (vec) NX_SM(__nv_bfloat16, 8); else NX_SM(__nv_bfloat16, 1); }
+    else if (dtype == NX_F32) { if (vec) NX_SM(float, 8); else NX_SM(float, 1); }
+    else return -1;
+#undef NX_SM
+  }
+  return launch_status();
+}
+
+extern "C" int nx_softcap(float* x, int64_t ld, int rows, int cols, float cap, nx_stream_t stream) {
+  if (cap <= 0.0f || rows > 65535) return -1;
+  if (rows <= 0 || cols <= 0) return 0;
+  dim3 grid((cols + 255) / 256, rows);
+  softcap_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(x, ld, cols, cap);
+  return launch_status();
+}

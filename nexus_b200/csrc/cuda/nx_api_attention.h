@@ -36,6 +36,7 @@ typedef struct NxAttnArgs {
   // regenerated in the backward kernels.  Out-of-range values are rejected.
   float dropout_p;
   uint64_t dropout_seed, dropout_offset;
+  float out_scale;              // forward: the written `o` is multiplied by this (0 counts as 1)
 } NxAttnArgs;
 
 int nx_attention_fwd(const NxAttnArgs* args, nx_stream_t stream);

@@ -1,0 +1,158 @@
+// C ABI of the building blocks of decoders with heterogeneous layers: pre / post norms around a sublayer, rotary
+// embedding fused with the cache append, windowed and soft-capped paged attention for any head sizes, the short causal
+// convolution with its carried tail, the Mamba-2 (SSD) and gated-delta-rule recurrences with their carried FP32 state,
+// gated norms, the per-layer token input and soft-capping of logits.
+//
+// Activations are BF16 or FP32 (`dtype`: NX_BF16 / NX_F32); weights of norms, decays and convolutions are FP32.
+//
+// A batch is a packed list of rows (tokens); a segment is the run of consecutive rows that one sequence contributes to
+// the step: seg_row0 (first row), seg_len (rows; 0 marks a padding entry of a captured batch), seg_pos (position of
+// the first row in its sequence) and seg_seq (sequence slot: the row of the block table and of every state tensor).
+// A segment that starts at position 0 starts from a zero state, whatever the slot held before.
+#pragma once
+#include "nx_api.h"
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+typedef struct NxSegments {
+  const int32_t* row0;
+  const int32_t* len;
+  const int32_t* pos;
+  const int32_t* seq;
+  int32_t count;
+  int32_t max_len;    // largest len of the list (host copy)
+  int32_t total_len;  // sum of len (host copy)
+} NxSegments;
+
+typedef struct NxResidualNormArgs {
+  float* x;                // [rows, cols] residual stream, updated in place (written when `table` or `y` is given)
+  const int32_t* tokens;   // with `table`: x = table[tokens[row]]
+  const void* table;       // [vocab, cols] dtype, may be null
+  const void* y;           // [rows, ldy] sublayer output, may be null: x += rms(y) * w_post
+  const float* w_post;
+  const float* w_next;     // may be null; else h = rms(x) * w_next
+  void* h;                 // [rows, ldh]; columns cols..ldh are zeroed
+  void* x_cast;            // [rows, ldh], may be null: x in the activation dtype
+  int64_t ldy, ldh;
+  int32_t rows, cols, dtype;
+  float eps;
+} NxResidualNormArgs;
+int nx_residual_norm(const NxResidualNormArgs* args, nx_stream_t stream);
+
+typedef struct NxRopeAppendArgs {
+  void* proj;              // [rows, ld]; q, k, v of a row start at q_off, k_off, v_off; q and k are rotated in place
+  int64_t ld;
+  int32_t q_off, k_off, v_off;
+  int32_t rows, heads, kv_heads, dim, vdim, rot_dims, dtype;
+  const int32_t* positions;
+  const int32_t* slots;    // cache slot per row, negative: nothing is appended
+  const float* cos_t;      // [max_pos, rot_dims / 2]
+  const float* sin_t;
+  void* k_cache;           // [slots, kv_heads, dim]
+  void* v_cache;           // [slots, kv_heads, vdim]
+} NxRopeAppendArgs;
+int nx_rope_append(const NxRopeAppendArgs* args, nx_stream_t stream);
+
+// y = silu(causal_conv(x) + bias) per channel; state [slots, taps - 1, channels] holds the last taps - 1 inputs.
+typedef struct NxConvArgs {
+  const void* x;           // [rows, ldx]
+  void* y;                 // [rows, ldy]
+  const float* w;          // [taps, channels], last row: the current token
+  const float* bias;       // [channels] or null
+  void* state;             // dtype
+  int64_t ldx, ldy;
+  int32_t channels, taps, dtype;
+  NxSegments seg;
+} NxConvArgs;
+int nx_conv_silu(const NxConvArgs* args, nx_stream_t stream);
+
+// Mamba-2: S = exp(-exp(A_log) dt) S + dt B x^T,  y = S^T C + D x,  dt = softplus(dt_raw + dt_bias).
+typedef struct NxSsdArgs {
+  const void* xbc;         // [rows, ld_xbc]: x (heads * vdim) | B (groups * state) | C (groups * state)
+  const void* dt;          // [rows, ld_dt]: heads raw step sizes
+  void* y;                 // [rows, ldy]: heads * vdim
+  const float* dt_bias;
+  const float* a_log;
+  const float* d_skip;
+  float* state;            // [slots, heads, state, vdim]
+  int64_t ld_xbc, ld_dt, ldy;
+  int32_t heads, groups, n_state, vdim, dtype;
+  NxSegments seg;
+  // Long segments on the tensor cores only: the segment list is cut into `parts` spans of `span` tokens per segment
+  // (span a multiple of 64); part_state [seg.count, parts, heads, state, vdim] and part_decay [seg.count, parts, heads]
+  // are scratch.  parts == 1: no scratch.
+  float* part_state;
+  float* part_decay;
+  int32_t parts, span;
+} NxSsdArgs;
+// token by token, any sizes and both dtypes
+int nx_ssd_step(const NxSsdArgs* args, nx_stream_t stream);
+// chunks of 64 tokens on the tensor cores, BF16 activations, state <= 256, vdim <= 256
+int nx_ssd_chunk(const NxSsdArgs* args, nx_stream_t stream);
+
+// Gated delta rule: S = g S;  u = beta (v - S^T k);  S += k u^T;  o = S^T q, with unit q / k (q also times dim^-1/2),
+// beta = sigmoid(b), g = exp(-exp(A_log) softplus(a + dt_bias)).
+typedef struct NxDeltaArgs {
+  const void* qkv;         // [rows, ld_qkv]: q (kv_heads * dim) | k (kv_heads * dim) | v (heads * vdim)
+  const void* b;           // [rows, ld_ba]: heads
+  const void* a;           // [rows, ld_ba]: heads
+  void* o;                 // [rows, ldo]: heads * vdim
+  const float* dt_bias;
+  const float* a_log;
+  float* state;            // [slots, heads, dim, vdim]
+  int64_t ld_qkv, ld_ba, ldo;
+  int32_t heads, kv_heads, dim, vdim, dtype;
+  float unit_eps, q_scale;
+  NxSegments seg;
+} NxDeltaArgs;
+int nx_delta_step(const NxDeltaArgs* args, nx_stream_t stream);
+int nx_delta_chunk(const NxDeltaArgs* args, nx_stream_t stream);
+
+// gate_first: out = rms(y * silu(z)) * w * out_scale, else out = rms(y) * w * silu(z) * out_scale; statistics over each
+// of `groups` equal parts of a row.  w has groups * group_size entries, or group_size shared by every part (w_shared).
+typedef struct NxGatedNormArgs {
+  const void* y;
+  const void* z;
+  const float* w;
+  void* out;
+  int64_t ldy, ldz, ldo;
+  int32_t rows, groups, group_size, gate_first, w_shared, dtype;
+  float eps, out_scale;
+} NxGatedNormArgs;
+int nx_gated_norm(const NxGatedNormArgs* args, nx_stream_t stream);
+
+// out[r][j] = gelu_tanh(a[r][j]) * table[tokens[r]][offset + j], j < dim; columns dim..ldo are zeroed
+int nx_token_side_gate(const void* a, int64_t lda, const int32_t* tokens, const void* table, int64_t ld_table, int offset,
+                       void* out, int64_t ldo, int rows, int dim, int dtype, nx_stream_t stream);
+// out[r][j] = silu(h[r][j]) * h[r][half + j], j < half
+int nx_silu_mul(const void* h, int64_t ldh, void* out, int64_t ldo, int rows, int half, int dtype, nx_stream_t stream);
+// x = cap * tanh(x / cap) in place on FP32 [rows, ld]
+int nx_softcap(float* x, int64_t ld, int rows, int cols, float cap, nx_stream_t stream);
+
+// Causal attention of packed query rows over a paged cache.  Row at position p sees keys p - window + 1 .. p (window <= 0:
+// 0 .. p); score = scale * q.k, soft-capped when softcap > 0.  The rows' own keys are in the cache already.
+typedef struct NxPagedWindowArgs {
+  const void* q;           // [rows, ldq]: heads * dim
+  const void* k_cache;     // [blocks * block_size, kv_heads, dim]
+  const void* v_cache;     // [blocks * block_size, kv_heads, vdim]
+  const int32_t* block_table;  // [slots, max_blocks]
+  void* out;               // [rows, ldo]: heads * vdim, times out_scale
+  int64_t ldq, ldo;
+  float* part_o;           // decode with splits > 1: [count, heads, splits, vdim]
+  float* part_ml;          // decode with splits > 1: [count, heads, splits, 2]
+  int32_t heads, kv_heads, dim, vdim, block_size, max_blocks, window, splits, dtype;
+  float scale, softcap, out_scale;
+  NxSegments seg;
+} NxPagedWindowArgs;
+// one-row segments, BF16: tensor-core tiles of up to 16 query heads of a KV head against 64 keys, split over the keys
+int nx_paged_window_decode(const NxPagedWindowArgs* args, nx_stream_t stream);
+// longer segments, BF16: 64 (row, head) pairs of one KV head against tiles of 64 keys
+int nx_paged_window_prefill(const NxPagedWindowArgs* args, nx_stream_t stream);
+// any segments, FP32
+int nx_paged_window_f32(const NxPagedWindowArgs* args, nx_stream_t stream);
+
+#ifdef __cplusplus
+}
+#endif

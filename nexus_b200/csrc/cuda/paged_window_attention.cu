@@ -1,0 +1,529 @@
+// Causal attention over a paged cache for any head sizes: sliding window, score soft-capping, grouped query heads,
+// different key and value widths (see nx_api_mixers.h).  The query heads that share a KV head are packed into the rows of
+// one tensor-core tile, so a KV page is read once for all of them: 64 (token, head) rows per block in prompts, up to 16
+// heads of one token in decoding.  Scores, soft-capping and softmax are FP32; only the products take BF16 operands.
+#include "mixer_common.cuh"
+#include "nx_api_mixers.h"
+
+#include <algorithm>
+
+namespace {
+using namespace nx;
+
+constexpr int kKeys = 64;              // keys per shared-memory stage
+constexpr float kLog2e = 1.4426950408889634f;
+
+// scaled, soft-capped score in units of log2
+__device__ __forceinline__ float score_log2(float s, float scale, float cap, float inv_cap) {
+  s *= scale;
+  if (cap > 0.0f) s = cap * (1.0f - __fdividef(2.0f, 1.0f + exp2f(2.0f * kLog2e * s * inv_cap)));
+  return s * kLog2e;
+}
+
+// which segment, and which tile of `per` tokens inside it, flat tile index `tile` is; executed by one full warp
+__device__ __forceinline__ bool find_tile(const NxSegments& s, int per, int tile, int& seg, int& off) {
+  const int lane = threadIdx.x & 31;
+  int base = 0;
+  for (int i0 = 0; i0 < s.count; i0 += 32) {
+    const int i = i0 + lane;
+    const int n = i < s.count ? (s.len[i] + per - 1) / per : 0;
+    int incl = n;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, incl, o);
+      if (lane >= o) incl += v;
+    }
+    const unsigned hit = __ballot_sync(0xffffffffu, base + incl > tile);
+    if (hit) {
+      const int first = __ffs(hit) - 1;
+      seg = i0 + first;
+      off = tile - base - __shfl_sync(0xffffffffu, incl - n, first);
+      return true;
+    }
+    base += __shfl_sync(0xffffffffu, incl, 31);
+  }
+  return false;
+}
+
+// rows of a K or V page range into shared memory [kKeys][DP + 8]; keys past `last` and columns past D become zeros
+template <int DP>
+__device__ __forceinline__ void stage_rows(__nv_bfloat16* dst, const __nv_bfloat16* cache, const int32_t* bt, int block_size,
+                                           int kv_heads, int hk, int D, int k0, int last) {
+  constexpr int CH = DP / 8;
+  const bool vec = (D & 7) == 0;
+  for (int i = threadIdx.x; i < kKeys * CH; i += blockDim.x) {
+    const int key = i / CH, c = (i % CH) * 8, j = k0 + key;
+    __nv_bfloat16* d = dst + key * (DP + 8) + c;
+    if (j <= last && c < D) {
+      const int64_t slot = static_cast<int64_t>(bt[j / block_size]) * block_size + j % block_size;
+      const __nv_bfloat16* s = cache + (slot * kv_heads + hk) * D + c;
+      if (vec) {
+        cp_async16(d, s);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) d[e] = c + e < D ? s[e] : __float2bfloat16_rn(0.0f);
+      }
+    } else {
+      *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// prompts: grid (tiles, kv_heads * head tiles), 4 warps of 16 rows
+// ------------------------------------------------------------------------------------------------
+template <int DP>
+__global__ void __launch_bounds__(128)
+paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) {
+  constexpr int LD = DP + 8;
+  extern __shared__ __align__(16) __nv_bfloat16 sm[];
+  __nv_bfloat16* sQ = sm;                       // [64][LD]
+  __nv_bfloat16* sKV = sQ + 64 * LD;            // [2 stages][K, V][64][LD]
+  __shared__ int s_tile[3];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (warp == 0) {
+    int seg = 0, off = 0;
+    const bool ok = find_tile(a.seg, tq, blockIdx.x, seg, off);
+    if (lane == 0) {
+      s_tile[0] = ok;
+      s_tile[1] = seg;
+      s_tile[2] = off;
+    }
+  }
+  __syncthreads();
+  if (!s_tile[0]) return;
+  const int sg = s_tile[1], t0 = s_tile[2] * tq;
+  const int hk = blockIdx.y / head_tiles, ht = blockIdx.y % head_tiles;
+  const int rep = a.heads / a.kv_heads, h0 = hk * rep + ht * rt, nh = min(rt, rep - ht * rt);
+  const int nt = min(tq, a.seg.len[sg] - t0);
+  const int pos0 = a.seg.pos[sg] + t0;
+  const int64_t row0 = static_cast<int64_t>(a.seg.row0[sg]) + t0;
+  const int32_t* bt = a.block_table + static_cast<int64_t>(a.seg.seq[sg]) * a.max_blocks;
+  const int first = a.window > 0 ? max(0, pos0 - a.window + 1) : 0, last = pos0 + nt - 1;
+  const __nv_bfloat16* kc = static_cast<const __nv_bfloat16*>(a.k_cache);
+  const __nv_bfloat16* vc = static_cast<const __nv_bfloat16*>(a.v_cache);
+  auto stage = [&](int k0, int s) {
+    stage_rows<DP>(sKV + (s * 2) * kKeys * LD, kc, bt, a.block_size, a.kv_heads, hk, a.dim, k0, last);
+    stage_rows<DP>(sKV + (s * 2 + 1) * kKeys * LD, vc, bt, a.block_size, a.kv_heads, hk, a.vdim, k0, last);
+    cp_async_commit();
+  };
+  stage(first, 0);
+  {
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q);
+    for (int i = threadIdx.x; i < 64 * DP; i += 128) {
+      const int m = i / DP, d = i % DP, tok = m / rt, hh = m % rt;
+      sQ[m * LD + d] = (tok < nt && hh < nh && d < a.dim) ? q[(row0 + tok) * a.ldq + static_cast<int64_t>(h0 + hh) * a.dim + d]
+                                                          : __float2bfloat16_rn(0.0f);
+    }
+  }
+  int qpos[2];                                  // position of this thread's two rows, -1: padding row
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int m = warp * 16 + i * 8 + (lane >> 2);
+    qpos[i] = (m / rt < nt && m % rt < nh) ? pos0 + m / rt : -1;
+  }
+  const float inv_cap = a.softcap > 0.0f ? 1.0f / a.softcap : 0.0f;
+  float o[DP / 8][4], mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.0f, 0.0f};
+#pragma unroll
+  for (int i = 0; i < DP / 8; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[i][e] = 0.0f;
+  int s = 0;
+  for (int k0 = first; k0 <= last; k0 += kKeys, s ^= 1) {
+    if (k0 + kKeys <= last) {
+      stage(k0 + kKeys, s ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const __nv_bfloat16* sK = sKV + (s * 2) * kKeys * LD;
+    const __nv_bfloat16* sV = sK + kKeys * LD;
+    float sc[8][4];
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sc[n][e] = 0.0f;
+#pragma unroll
+    for (int kk = 0; kk < DP / 16; ++kk) {
+      uint32_t qa[4];
+      ldmatrix_x4(qa, smem_addr(sQ + (warp * 16 + (lane & 15)) * LD + kk * 16 + (lane >> 4) * 8));
+#pragma unroll
+      for (int n = 0; n < 4; ++n) {
+        uint32_t kb[4];
+        ldmatrix_x4(kb, smem_addr(sK + (n * 16 + (lane & 7) + ((lane >> 4) << 3)) * LD + kk * 16 + ((lane >> 3) & 1) * 8));
+        mma_bf16(sc[2 * n], qa, kb[0], kb[1]);
+        mma_bf16(sc[2 * n + 1], qa, kb[2], kb[3]);
+      }
+    }
+    float tmax[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int j = k0 + n * 8 + (lane & 3) * 2 + (e & 1), qp = qpos[e >> 1];
+        const bool see = j <= qp && (a.window <= 0 || j > qp - a.window);
+        sc[n][e] = see ? score_log2(sc[n][e], a.scale, a.softcap, inv_cap) : -INFINITY;
+        tmax[e >> 1] = fmaxf(tmax[e >> 1], sc[n][e]);
+      }
+    float base[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 1));
+      tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 2));
+      const float nm = fmaxf(mx[i], tmax[i]);
+      base[i] = nm == -INFINITY ? 0.0f : nm;
+      const float alpha = exp2f(mx[i] - base[i]);     // first tile: exp2(-inf) = 0
+      mx[i] = nm;
+      sum[i] *= alpha;
+#pragma unroll
+      for (int n = 0; n < DP / 8; ++n) {
+        o[n][2 * i] *= alpha;
+        o[n][2 * i + 1] *= alpha;
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        sc[n][e] = exp2f(sc[n][e] - base[e >> 1]);
+        sum[e >> 1] += sc[n][e];
+      }
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk) {
+      const uint32_t pa[4] = {bf16_pair(sc[2 * kk][0], sc[2 * kk][1]), bf16_pair(sc[2 * kk][2], sc[2 * kk][3]),
+                              bf16_pair(sc[2 * kk + 1][0], sc[2 * kk + 1][1]), bf16_pair(sc[2 * kk + 1][2], sc[2 * kk + 1][3])};
+#pragma unroll
+      for (int n = 0; n < DP / 16; ++n) {
+        uint32_t vb[4];
+        ldmatrix_x4_trans(vb, smem_addr(sV + (kk * 16 + (lane & 15)) * LD + n * 16 + (lane >> 4) * 8));
+        mma_bf16(o[2 * n], pa, vb[0], vb[1]);
+        mma_bf16(o[2 * n + 1], pa, vb[2], vb[3]);
+      }
+    }
+    __syncthreads();
+  }
+  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out);
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 1);
+    sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 2);
+    if (qpos[i] < 0) continue;
+    const int m = warp * 16 + i * 8 + (lane >> 2);
+    const float inv = a.out_scale / sum[i];
+    __nv_bfloat16* op = out + (row0 + m / rt) * a.ldo + static_cast<int64_t>(h0 + m % rt) * a.vdim;
+#pragma unroll
+    for (int n = 0; n < DP / 8; ++n) {
+      const int d = n * 8 + (lane & 3) * 2;
+      if (d < a.vdim) op[d] = __float2bfloat16_rn(o[n][2 * i] * inv);
+      if (d + 1 < a.vdim) op[d + 1] = __float2bfloat16_rn(o[n][2 * i + 1] * inv);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// decoding: grid (segments, kv_heads * head tiles, splits); the 4 warps take 16 keys each of every
+// 64-key stage, with their own running softmax, and merge at the end
+// ------------------------------------------------------------------------------------------------
+template <int DP>
+__global__ void __launch_bounds__(128)
+paged_decode_mma_kernel(const NxPagedWindowArgs a, int head_tiles) {
+  constexpr int LD = DP + 8;
+  extern __shared__ __align__(16) __nv_bfloat16 sm[];
+  __nv_bfloat16* sQ = sm;                       // [16][LD]
+  __nv_bfloat16* sKV = sQ + 16 * LD;            // [2 stages][K, V][64][LD]; the warps' partial outputs afterwards
+  __shared__ float s_m[4][16], s_l[4][16];
+  const int sg = blockIdx.x;
+  if (a.seg.len[sg] <= 0) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int hk = blockIdx.y / head_tiles, ht = blockIdx.y % head_tiles;
+  const int rep = a.heads / a.kv_heads, h0 = hk * rep + ht * 16, nh = min(16, rep - ht * 16);
+  const int pos = a.seg.pos[sg];
+  const int64_t row = a.seg.row0[sg];
+  const int32_t* bt = a.block_table + static_cast<int64_t>(a.seg.seq[sg]) * a.max_blocks;
+  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int per = ((pos - lo + kKeys) / kKeys + a.splits - 1) / a.splits * kKeys;
+  const int first = lo + static_cast<int>(blockIdx.z) * per, last = min(pos, first + per - 1);
+  const __nv_bfloat16* kc = static_cast<const __nv_bfloat16*>(a.k_cache);
+  const __nv_bfloat16* vc = static_cast<const __nv_bfloat16*>(a.v_cache);
+  auto stage = [&](int k0, int s) {
+    stage_rows<DP>(sKV + (s * 2) * kKeys * LD, kc, bt, a.block_size, a.kv_heads, hk, a.dim, k0, last);
+    stage_rows<DP>(sKV + (s * 2 + 1) * kKeys * LD, vc, bt, a.block_size, a.kv_heads, hk, a.vdim, k0, last);
+    cp_async_commit();
+  };
+  if (first <= last) stage(first, 0);
+  for (int i = threadIdx.x; i < 16 * DP; i += 128) {
+    const int m = i / DP, d = i % DP;
+    sQ[m * LD + d] = (m < nh && d < a.dim)
+                         ? static_cast<const __nv_bfloat16*>(a.q)[row * a.ldq + static_cast<int64_t>(h0 + m) * a.dim + d]
+                         : __float2bfloat16_rn(0.0f);
+  }
+  const float inv_cap = a.softcap > 0.0f ? 1.0f / a.softcap : 0.0f;
+  float o[DP / 8][4], mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.0f, 0.0f};
+#pragma unroll
+  for (int i = 0; i < DP / 8; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[i][e] = 0.0f;
+  int s = 0;
+  for (int k0 = first; k0 <= last; k0 += kKeys, s ^= 1) {
+    if (k0 + kKeys <= last) {
+      stage(k0 + kKeys, s ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    if (k0 + warp * 16 <= last) {
+      const __nv_bfloat16* sK = sKV + ((s * 2) * kKeys + warp * 16) * LD;
+      const __nv_bfloat16* sV = sK + kKeys * LD;
+      float sc[2][4] = {{0.0f, 0.0f, 0.0f, 0.0f}, {0.0f, 0.0f, 0.0f, 0.0f}};
+#pragma unroll
+      for (int kk = 0; kk < DP / 16; ++kk) {
+        uint32_t qa[4], kb[4];
+        ldmatrix_x4(qa, smem_addr(sQ + (lane & 15) * LD + kk * 16 + (lane >> 4) * 8));
+        ldmatrix_x4(kb, smem_addr(sK + ((lane & 7) + ((lane >> 4) << 3)) * LD + kk * 16 + ((lane >> 3) & 1) * 8));
+        mma_bf16(sc[0], qa, kb[0], kb[1]);
+        mma_bf16(sc[1], qa, kb[2], kb[3]);
+      }
+      float tmax[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int j = k0 + warp * 16 + n * 8 + (lane & 3) * 2 + (e & 1);
+          sc[n][e] = j <= last ? score_log2(sc[n][e], a.scale, a.softcap, inv_cap) : -INFINITY;
+          tmax[e >> 1] = fmaxf(tmax[e >> 1], sc[n][e]);
+        }
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 1));
+        tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 2));
+        const float nm = fmaxf(mx[i], tmax[i]);       // at least one key of this warp is in range
+        const float alpha = exp2f(mx[i] - nm);
+        mx[i] = nm;
+        sum[i] *= alpha;
+#pragma unroll
+        for (int n = 0; n < DP / 8; ++n) {
+          o[n][2 * i] *= alpha;
+          o[n][2 * i + 1] *= alpha;
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          sc[n][e] = exp2f(sc[n][e] - mx[e >> 1]);
+          sum[e >> 1] += sc[n][e];
+        }
+      const uint32_t pa[4] = {bf16_pair(sc[0][0], sc[0][1]), bf16_pair(sc[0][2], sc[0][3]), bf16_pair(sc[1][0], sc[1][1]),
+                              bf16_pair(sc[1][2], sc[1][3])};
+#pragma unroll
+      for (int n = 0; n < DP / 16; ++n) {
+        uint32_t vb[4];
+        ldmatrix_x4_trans(vb, smem_addr(sV + (lane & 15) * LD + n * 16 + (lane >> 4) * 8));
+        mma_bf16(o[2 * n], pa, vb[0], vb[1]);
+        mma_bf16(o[2 * n + 1], pa, vb[2], vb[3]);
+      }
+    }
+    __syncthreads();
+  }
+  float* sO = reinterpret_cast<float*>(sKV);    // [4 warps][16][DP]
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 1);
+    sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 2);
+    const int m = i * 8 + (lane >> 2);
+    if ((lane & 3) == 0) {
+      s_m[warp][m] = mx[i];
+      s_l[warp][m] = sum[i];
+    }
+#pragma unroll
+    for (int n = 0; n < DP / 8; ++n) {
+      sO[(warp * 16 + m) * DP + n * 8 + (lane & 3) * 2] = o[n][2 * i];
+      sO[(warp * 16 + m) * DP + n * 8 + (lane & 3) * 2 + 1] = o[n][2 * i + 1];
+    }
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < nh * a.vdim; i += 128) {
+    const int m = i / a.vdim, d = i % a.vdim;
+    float gm = -INFINITY;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) gm = fmaxf(gm, s_m[w][m]);
+    float gl = 0.0f, go = 0.0f;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) {
+      const float f = s_m[w][m] == -INFINITY ? 0.0f : exp2f(s_m[w][m] - gm);
+      gl += s_l[w][m] * f;
+      go += sO[(w * 16 + m) * DP + d] * f;
+    }
+    if (a.splits == 1) {
+      static_cast<__nv_bfloat16*>(a.out)[row * a.ldo + static_cast<int64_t>(h0 + m) * a.vdim + d] =
+          __float2bfloat16_rn(go / gl * a.out_scale);
+    } else {
+      const int64_t pi = (static_cast<int64_t>(sg) * a.heads + h0 + m) * a.splits + blockIdx.z;
+      a.part_o[pi * a.vdim + d] = go;
+      if (d == 0) {
+        a.part_ml[pi * 2] = gm;
+        a.part_ml[pi * 2 + 1] = gl;
+      }
+    }
+  }
+}
+
+__global__ void paged_decode_merge_kernel(const NxPagedWindowArgs a) {
+  const int sg = blockIdx.x, h = blockIdx.y;
+  if (a.seg.len[sg] <= 0) return;
+  const int64_t base = (static_cast<int64_t>(sg) * a.heads + h) * a.splits;
+  float gm = -INFINITY;
+  for (int s = 0; s < a.splits; ++s) gm = fmaxf(gm, a.part_ml[(base + s) * 2]);
+  for (int d = threadIdx.x; d < a.vdim; d += blockDim.x) {
+    float gl = 0.0f, go = 0.0f;
+    for (int s = 0; s < a.splits; ++s) {
+      const float m = a.part_ml[(base + s) * 2];
+      const float w = m == -INFINITY ? 0.0f : exp2f(m - gm);
+      gl += a.part_ml[(base + s) * 2 + 1] * w;
+      go += a.part_o[(base + s) * a.vdim + d] * w;
+    }
+    static_cast<__nv_bfloat16*>(a.out)[static_cast<int64_t>(a.seg.row0[sg]) * a.ldo + static_cast<int64_t>(h) * a.vdim + d] =
+        __float2bfloat16_rn(go / gl * a.out_scale);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// FP32: one block per (row, head), a key per thread for the scores, a value column per thread for the sum
+// ------------------------------------------------------------------------------------------------
+constexpr int kF32Cols = 4;   // value columns per thread: vdim <= 512
+
+__global__ void __launch_bounds__(128) paged_window_f32_kernel(const NxPagedWindowArgs a) {
+  extern __shared__ __align__(16) float sf[];
+  __shared__ float s_red[32];
+  __shared__ int64_t s_slot[128];
+  float* sQ = sf;               // [dim]
+  float* sP = sf + a.dim;       // [128]
+  const int t = blockIdx.x, h = blockIdx.y, sg = blockIdx.z;
+  if (t >= a.seg.len[sg]) return;
+  const int hk = h / (a.heads / a.kv_heads), pos = a.seg.pos[sg] + t, tid = threadIdx.x;
+  const int64_t row = static_cast<int64_t>(a.seg.row0[sg]) + t;
+  const int32_t* bt = a.block_table + static_cast<int64_t>(a.seg.seq[sg]) * a.max_blocks;
+  const float* kc = static_cast<const float*>(a.k_cache);
+  const float* vc = static_cast<const float*>(a.v_cache);
+  for (int d = tid; d < a.dim; d += 128) sQ[d] = static_cast<const float*>(a.q)[row * a.ldq + static_cast<int64_t>(h) * a.dim + d];
+  float acc[kF32Cols] = {0.0f, 0.0f, 0.0f, 0.0f}, mx = -INFINITY, sum = 0.0f;
+  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  for (int k0 = lo; k0 <= pos; k0 += 128) {
+    __syncthreads();
+    const int j = k0 + tid;
+    float sc = -INFINITY;
+    if (j <= pos) {
+      const int64_t slot = static_cast<int64_t>(bt[j / a.block_size]) * a.block_size + j % a.block_size;
+      s_slot[tid] = slot;
+      const float* k = kc + (slot * a.kv_heads + hk) * a.dim;
+      float s = 0.0f;
+      for (int d = 0; d < a.dim; ++d) s += sQ[d] * k[d];
+      sc = s * a.scale;
+      if (a.softcap > 0.0f) sc = a.softcap * tanhf(sc / a.softcap);
+    }
+    const float nm = fmaxf(mx, block_max(sc, s_red));
+    const float p = expf(sc - nm), alpha = expf(mx - nm);
+    mx = nm;
+    sP[tid] = p;
+    sum = sum * alpha + block_sum(p, s_red);     // the barriers inside publish sP and s_slot
+    const int n = min(128, pos - k0 + 1);
+#pragma unroll
+    for (int c = 0; c < kF32Cols; ++c) {
+      const int d = tid + c * 128;
+      if (d < a.vdim) {
+        float v = acc[c] * alpha;
+        for (int i = 0; i < n; ++i) v += sP[i] * vc[(s_slot[i] * a.kv_heads + hk) * a.vdim + d];
+        acc[c] = v;
+      }
+    }
+  }
+  for (int c = 0; c < kF32Cols; ++c) {
+    const int d = tid + c * 128;
+    if (d < a.vdim) static_cast<float*>(a.out)[row * a.ldo + static_cast<int64_t>(h) * a.vdim + d] = acc[c] / sum * a.out_scale;
+  }
+}
+
+int check_paged(const NxPagedWindowArgs* a, int dtype) {
+  if (a == nullptr || a->dtype != dtype || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads) return -1;
+  if (a->dim <= 0 || a->vdim <= 0 || a->block_size <= 0 || a->max_blocks <= 0 || a->seg.count > 65535) return -1;
+  return 0;
+}
+int padded_dim(const NxPagedWindowArgs* a) {
+  const int d = std::max(a->dim, a->vdim);
+  return d <= 32 ? 32 : d <= 64 ? 64 : d <= 128 ? 128 : d <= 256 ? 256 : 0;
+}
+
+template <int DP>
+int launch_prefill(const NxPagedWindowArgs* a, dim3 grid, int rt, int tq, int head_tiles, cudaStream_t st) {
+  constexpr int kSmem = (64 + 4 * kKeys) * (DP + 8) * 2;
+  static bool once = false;
+  if (!once) {
+    if (cudaFuncSetAttribute(paged_prefill_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -2;
+    once = true;
+  }
+  paged_prefill_kernel<DP><<<grid, 128, kSmem, st>>>(*a, rt, tq, head_tiles);
+  return launch_status();
+}
+
+template <int DP>
+int launch_decode(const NxPagedWindowArgs* a, dim3 grid, int head_tiles, cudaStream_t st) {
+  constexpr int kSmem = (16 + 4 * kKeys) * (DP + 8) * 2;
+  static_assert(4 * kKeys * (DP + 8) * 2 >= 4 * 16 * DP * 4, "partial outputs reuse the stages");
+  static bool once = false;
+  if (!once) {
+    if (cudaFuncSetAttribute(paged_decode_mma_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -2;
+    once = true;
+  }
+  paged_decode_mma_kernel<DP><<<grid, 128, kSmem, st>>>(*a, head_tiles);
+  return launch_status();
+}
+
+}  // namespace
+
+extern "C" int nx_paged_window_prefill(const NxPagedWindowArgs* a, nx_stream_t stream) {
+  if (check_paged(a, NX_BF16)) return -1;
+  if (a->seg.count <= 0 || a->seg.total_len <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int rep = a->heads / a->kv_heads;
+  const int rt = std::min(rep, 16), head_tiles = (rep + rt - 1) / rt, tq = 64 / rt;
+  dim3 grid(a->seg.total_len / tq + a->seg.count, a->kv_heads * head_tiles);
+  switch (padded_dim(a)) {
+    case 32: return launch_prefill<32>(a, grid, rt, tq, head_tiles, st);
+    case 64: return launch_prefill<64>(a, grid, rt, tq, head_tiles, st);
+    case 128: return launch_prefill<128>(a, grid, rt, tq, head_tiles, st);
+    case 256: return launch_prefill<256>(a, grid, rt, tq, head_tiles, st);
+    default: return -1;
+  }
+}
+
+extern "C" int nx_paged_window_decode(const NxPagedWindowArgs* a, nx_stream_t stream) {
+  if (check_paged(a, NX_BF16) || a->splits < 1 || a->splits > 65535) return -1;
+  if (a->splits > 1 && (a->part_o == nullptr || a->part_ml == nullptr)) return -1;
+  if (a->seg.count <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int rep = a->heads / a->kv_heads, head_tiles = (rep + 15) / 16;
+  dim3 grid(a->seg.count, a->kv_heads * head_tiles, a->splits);
+  int rc = -1;
+  switch (padded_dim(a)) {
+    case 32: rc = launch_decode<32>(a, grid, head_tiles, st); break;
+    case 64: rc = launch_decode<64>(a, grid, head_tiles, st); break;
+    case 128: rc = launch_decode<128>(a, grid, head_tiles, st); break;
+    case 256: rc = launch_decode<256>(a, grid, head_tiles, st); break;
+    default: return -1;
+  }
+  if (rc == 0 && a->splits > 1) {
+    paged_decode_merge_kernel<<<dim3(a->seg.count, a->heads), std::min(256, (a->vdim + 31) / 32 * 32), 0, st>>>(*a);
+    rc = launch_status();
+  }
+  return rc;
+}
+
+extern "C" int nx_paged_window_f32(const NxPagedWindowArgs* a, nx_stream_t stream) {
+  if (check_paged(a, NX_F32) || a->vdim > 128 * kF32Cols || a->dim > 4096) return -1;
+  if (a->seg.count <= 0 || a->seg.max_len <= 0) return 0;
+  dim3 grid(a->seg.max_len, a->heads, a->seg.count);
+  paged_window_f32_kernel<<<grid, 128, (a->dim + 128) * sizeof(float), static_cast<cudaStream_t>(stream)>>>(*a);
+  return launch_status();
+}

@@ -1,6 +1,8 @@
 // Host bookkeeping of the paged-KV inference engine: block pool with reference counts, per-sequence block lists and
 // token lists, copy-on-write on append to a shared partial block, truncation, and the packing of one step's batch into
-// the six index rows the device kernels read (token, position, cache slot, sequence, context length, logit rows).
+// the six index rows the device kernels read (token, position, cache slot, sequence, context length, logit rows), plus
+// the segment table of models whose layers carry state from token to token: one entry per sequence of the step (first
+// row, rows, position of the first row, sequence), one-token segments first, then short ones, then the rest.
 // The engine calls `plan` with the step's chunks, picks a staging width from the result, and has `write` fill the
 // (pinned) staging rows; block copies for copy-on-write and block-table rows of the sequences that changed are
 // reported back for the engine to issue on the device.
@@ -113,9 +115,17 @@ class KvScheduler {
   }
 
   // One step: chunk i appends counts[i] tokens (taken in order from `flat`) to sequence seqs[i], wants logits for its
-  // last logits[i] rows, and output[i] tells whether its tokens are model output.
+  // last logits[i] rows - or for the rows places[i] (offsets into the chunk, in the order asked for) when `places` is
+  // given and logits[i] is negative - and output[i] tells whether its tokens are model output.
+  // `short_len`: segments of 2 .. short_len tokens are listed apart from longer ones.
   py::dict plan(const std::vector<int>& seqs, const std::vector<int>& counts, const std::vector<int32_t>& flat,
-                const std::vector<int>& logits, const std::vector<int>& output, bool device_tokens, int max_tokens) {
+                const std::vector<int>& logits, const std::vector<int>& output, bool device_tokens, int max_tokens,
+                const std::vector<std::vector<int>>& places, int short_len) {
+    if (!places.empty() && places.size() != seqs.size()) throw std::invalid_argument("plan: chunk arrays differ in length");
+    for (size_t i = 0; i < places.size() && i < counts.size() && i < logits.size(); ++i)
+      if (logits[i] < 0)
+        for (int p : places[i])
+          if (p < 0 || p >= counts[i]) throw std::invalid_argument("plan: a wanted place lies outside its chunk");
     if (seqs.size() != counts.size() || seqs.size() != logits.size() || seqs.size() != output.size())
       throw std::invalid_argument("plan: chunk arrays differ in length");
     // pass 0: everything that can fail is checked before any state changes, so a refused step leaves the sequences,
@@ -159,7 +169,7 @@ class KvScheduler {
       }
       if (need_blocks > static_cast<long>(free_blocks_.size())) throw std::runtime_error("KV cache exhausted");
     }
-    tok_.clear(); pos_.clear(); slot_.clear(); rseq_.clear(); logit_rows_.clear();
+    tok_.clear(); pos_.clear(); slot_.clear(); rseq_.clear(); logit_rows_.clear(); segs_.clear();
     std::vector<int> out_rows, logit_seq, table_changed;
     std::vector<std::pair<int, int>> cows, patches;
     py::list runs;
@@ -223,11 +233,22 @@ class KvScheduler {
         }
         if (s.length == 0 || n > 1) prefill += n; else decode += n;
       }
-      const int k = std::min(logits[i], n);
-      for (int j = n - k; j < n; ++j) {
-        logit_rows_.push_back(r0 + j);
-        logit_seq.push_back(sid);
+      if (logits[i] < 0) {
+        for (int j : places.empty() ? std::vector<int>{} : places[i]) {
+          logit_rows_.push_back(r0 + j);
+          logit_seq.push_back(sid);
+        }
+      } else {
+        const int k = std::min(logits[i], n);
+        for (int j = n - k; j < n; ++j) {
+          logit_rows_.push_back(r0 + j);
+          logit_seq.push_back(sid);
+        }
       }
+      if (!segs_.empty() && segs_.back().seq == sid && segs_.back().row0 + segs_.back().len == r0)
+        segs_.back().len += n;                       // adjacent chunks of one sequence are one segment
+      else
+        segs_.push_back({r0, n, s.length, sid});
       if (!output[i] && s.length == s.n_prompt) s.n_prompt += n;
       if (device_tokens) {
         patches.emplace_back(sid, static_cast<int>(s.tokens.size()));
@@ -239,6 +260,17 @@ class KvScheduler {
       cursor += static_cast<size_t>(n);
     }
     flush_run();
+    int group_count[3] = {0, 0, 0}, group_max[3] = {0, 0, 0}, group_total[3] = {0, 0, 0};
+    {
+      const auto group = [&](const Segment& g) { return g.len == 1 ? 0 : (g.len <= short_len ? 1 : 2); };
+      for (const Segment& g : segs_) {
+        const int k = group(g);
+        ++group_count[k];
+        group_max[k] = std::max(group_max[k], g.len);
+        group_total[k] += g.len;
+      }
+      std::stable_sort(segs_.begin(), segs_.end(), [&](const Segment& x, const Segment& y) { return group(x) < group(y); });
+    }
     py::dict out;
     out["tokens"] = static_cast<int>(tok_.size());
     out["logit_rows"] = static_cast<int>(logit_rows_.size());
@@ -250,7 +282,25 @@ class KvScheduler {
     out["cows"] = cows;
     out["tables"] = table_changed;
     out["patches"] = patches;
+    // (count, longest, total) of the one-token, short and long segments, in the order of the table
+    py::list groups;
+    for (int k = 0; k < 3; ++k) groups.append(py::make_tuple(group_count[k], group_max[k], group_total[k]));
+    out["segments"] = groups;
     return out;
+  }
+
+  // The segment table [4, width] (first row, rows, first position, sequence) from the last plan; padding has 0 rows.
+  void write_segments(uintptr_t ptr, int width) const {
+    const size_t n = segs_.size(), w = static_cast<size_t>(width);
+    if (ptr == 0 || width < 0 || w < n) throw std::invalid_argument("write_segments: staging buffer is too small");
+    int32_t* h = reinterpret_cast<int32_t*>(ptr);
+    for (size_t i = 0; i < w; ++i) {
+      const Segment g = i < n ? segs_[i] : Segment{0, 0, 0, 0};
+      h[0 * w + i] = g.row0;
+      h[1 * w + i] = g.len;
+      h[2 * w + i] = g.pos;
+      h[3 * w + i] = g.seq;
+    }
   }
 
   // Fills the staging rows [6, width] (int32, row-major) from the last plan; columns past the batch are padding.
@@ -291,7 +341,12 @@ class KvScheduler {
     return b;
   }
 
+  struct Segment {
+    int32_t row0, len, pos, seq;
+  };
+
   int bs_, ctx_;
+  std::vector<Segment> segs_;
   std::vector<int> refcount_;
   std::vector<int32_t> free_blocks_;
   std::vector<int> free_ids_;
@@ -320,6 +375,8 @@ void bind_kv_sched(py::module_& m) {
       .def("blocks_needed", &KvScheduler::blocks_needed)
       .def("patch", &KvScheduler::patch)
       .def("plan", &KvScheduler::plan, py::arg("seqs"), py::arg("counts"), py::arg("flat"), py::arg("logits"), py::arg("output"),
-           py::arg("device_tokens"), py::arg("max_tokens"))
-      .def("write", &KvScheduler::write);
+           py::arg("device_tokens"), py::arg("max_tokens"), py::arg("places") = std::vector<std::vector<int>>{},
+           py::arg("short_len") = 16)
+      .def("write", &KvScheduler::write)
+      .def("write_segments", &KvScheduler::write_segments);
 }

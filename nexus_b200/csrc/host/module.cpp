@@ -25,10 +25,12 @@ void bind_tb_events(py::module_& m);
 
 PYBIND11_MODULE(_native, m) {
   m.doc() = "nexus_b200 native host runtime";
+  bind_cpu_kernels(m);
+  bind_kv_sched(m);
+#ifndef NX_SERVING_ONLY   // the subset that serving a model needs (see _build.ensure_serving)
   bind_nxs2(m);
   bind_nxs3(m);
   bind_runtime(m);
-  bind_cpu_kernels(m);
   bind_envs(m);
   bind_device_allocator(m);
   bind_store(m);
@@ -36,11 +38,11 @@ PYBIND11_MODULE(_native, m) {
   bind_estimate(m);
   bind_dlpack(m);
   bind_token_data(m);
-  bind_kv_sched(m);
   bind_lowp(m);
   bind_fused_train_cpu(m);
   bind_moe_route(m);
   bind_pipeline_sched(m);
   bind_rl_core(m);
   bind_tb_events(m);
+#endif
 }

@@ -1,4 +1,4 @@
-"""GPT-2 inference engine with a paged KV cache.
+"""Inference engine with a paged KV cache: the step function every served model shares, and the GPT-2 family.
 
 * KV pool per layer ``[blocks, block_size, heads, head_dim]`` (BF16, INT8 or FP8-E4M3 with one scale
   per (slot, head)); the native host scheduler (`csrc/host/kv_sched.cpp`: block pool with reference counts,
@@ -133,6 +133,8 @@ class EngineConfig:
     cuda_graphs: bool = True
     quant: QuantOptions = field(default_factory=QuantOptions)
     device: str = "cuda"
+    kv_tokens: int = 0           # > 0: the KV pool holds this many tokens (whole blocks) instead of kv_bytes
+    context: int = 0             # longest sequence of a model without a position limit (0: what the KV pool holds)
     decode_splits: int = 0       # 0: chosen per step from the batch size and context length
     tp_graphs: bool = False      # decode CUDA graphs of a tensor-parallel engine (its all-reduces are captured too);
                                  # call Engine.release_graphs() before the process group is destroyed
@@ -158,6 +160,7 @@ class Chunk:
     tokens: Sequence[int] = ()
     logits: int = 1          # logits of the last `logits` tokens are produced (0: none)
     output: bool = False     # tokens are model output (frequency / presence counters)
+    places: Optional[Sequence[int]] = None   # instead of `logits`: the offsets of the tokens whose logits are produced
 
 
 @dataclass
@@ -242,7 +245,14 @@ class _Linear:
 
 # ------------------------------------------------------------------------------------------ engine
 class Engine:
-    def __init__(self, weights: Gpt2Weights, config: Optional[EngineConfig] = None, group=None):
+    """The step function, sequences, cache, sampling and decode graphs of every served model.  This class runs the
+    GPT-2 family; another family subclasses it with its own `_configure`, `_load`, `_alloc_kv` and `_body`
+    (`HybridEngine`), and `infer.registry.create_engine` picks the class from the weights."""
+
+    INDEX_ROWS = 6               # token, position, cache slot, sequence, context length, logit rows
+    SEGMENT_ROWS = 0             # 4: the segment table follows (models that carry state from token to token)
+
+    def __init__(self, weights, config: Optional[EngineConfig] = None, group=None):
         self.cfg = config or EngineConfig()
         cfg = self.cfg
         self.dev = torch.device(cfg.device)
@@ -253,17 +263,7 @@ class Engine:
         self.group = group
         self.tp = group.size() if group is not None else 1
         self.tp_rank = group.rank() if group is not None else 0
-        self.L, self.H, self.d, self.V, self.ctx = weights.layers, weights.heads, weights.d, weights.vocab, weights.ctx
-        self.D = self.d // self.H
-        self.Hp = -(-self.H // self.tp)                    # heads per rank (last rank may hold fewer)
-        self.h0 = min(self.H, self.tp_rank * self.Hp)
-        self.Hl = max(0, min(self.Hp, self.H - self.h0))  # local heads
-        F = 4 * self.d
-        self.Fl = F // self.tp
-        if F % self.tp:
-            raise ValueError("MLP width must divide by the tensor-parallel size")
-        if self.fast and self.D not in (64, 128):
-            raise ValueError("the kernel path supports head_dim 64 and 128")
+        self._configure(weights)
         self.Vp = (self.V + 63) // 64 * 64
         self.wdt = torch.bfloat16 if self.fast else torch.float32
         self._load(weights)
@@ -302,6 +302,20 @@ class Engine:
             raise ValueError("tp_comm must be 'nccl' or 'fused'")
 
     # ----------------------------------------------------------------------------- weights / KV pool
+    def _configure(self, weights: Gpt2Weights) -> None:
+        """Sizes of the model: sets at least L, d, V and ctx."""
+        self.L, self.H, self.d, self.V, self.ctx = weights.layers, weights.heads, weights.d, weights.vocab, weights.ctx
+        self.D = self.d // self.H
+        self.Hp = -(-self.H // self.tp)                    # heads per rank (last rank may hold fewer)
+        self.h0 = min(self.H, self.tp_rank * self.Hp)
+        self.Hl = max(0, min(self.Hp, self.H - self.h0))  # local heads
+        F = 4 * self.d
+        self.Fl = F // self.tp
+        if F % self.tp:
+            raise ValueError("MLP width must divide by the tensor-parallel size")
+        if self.fast and self.D not in (64, 128):
+            raise ValueError("the kernel path supports head_dim 64 and 128")
+
     def _load(self, w: Gpt2Weights) -> None:
         dev, q = self.dev, self.cfg.quant
         fl = torch.float32
@@ -381,7 +395,7 @@ class Engine:
         # blocks (the scheduler runs replicated) even when the heads do not divide evenly or a rank holds none
         per_tok = self.L * 2 * self.Hp * self.D * elem + (self.L * 2 * self.Hp * 4 if self.kv_kind else 0)
         self._kv_tok_bytes = per_tok
-        self.n_blocks = max(2, int(cfg.kv_bytes // max(1, per_tok * cfg.block_size)))
+        self.n_blocks = self._pool_blocks(per_tok)
         self.max_blocks = -(-self.ctx // cfg.block_size)
         bs, Hl, D = cfg.block_size, max(self.Hl, 1), self.D
         dt = self.wdt if self.kv_kind == 0 else (torch.int8 if self.kv_kind == 1 else torch.uint8)
@@ -392,6 +406,12 @@ class Engine:
             self.v_scale = [torch.ones((self.n_blocks * bs, Hl), dtype=torch.float32, device=self.dev) for _ in range(self.L)]
         else:
             self.k_scale = self.v_scale = [None] * self.L
+
+    def _pool_blocks(self, bytes_per_token: int) -> int:
+        cfg = self.cfg
+        if cfg.kv_tokens > 0:
+            return max(1, -(-cfg.kv_tokens // cfg.block_size))
+        return max(2, int(cfg.kv_bytes // max(1, bytes_per_token * cfg.block_size)))
 
     # ----------------------------------------------------------------------------- sequences / blocks
     def add_sequence(self) -> int:
@@ -406,12 +426,20 @@ class Engine:
         self.counts_all[sid].copy_(self.counts_all[src])
         self.counts_out[sid].copy_(self.counts_out[src])
         self._write_table(sid)
+        self._fork_state(src, sid)
         return sid
+
+    def _fork_state(self, src: int, dst: int) -> None:
+        """Whatever a sequence owns beside its cache blocks, from ``src`` to its fork."""
 
     def free_sequence(self, seq: int) -> None:
         self.sched.free(seq)
 
+    def _check_truncate(self, seq: int, length: int) -> None:
+        """Refuses a truncation the model cannot follow."""
+
     def truncate(self, seq: int, length: int) -> None:
+        self._check_truncate(seq, length)
         removed, n_out = self.sched.truncate(seq, length)
         if not removed:
             return
@@ -453,6 +481,8 @@ class Engine:
         """Copy-on-write of a shared partial block: every layer's K and V page (and scales) from ``old`` to ``nb``."""
         bs = self.cfg.block_size
         for l in range(self.L):
+            if self.k_cache[l] is None:       # a layer without attention
+                continue
             self.k_cache[l][nb].copy_(self.k_cache[l][old])
             self.v_cache[l][nb].copy_(self.v_cache[l][old])
             if self.kv_kind:
@@ -543,8 +573,13 @@ class Engine:
                 flat.extend(int(t) for t in c.tokens)
         else:
             flat = [0] * len(live)
-        plan = self.sched.plan([c.seq for c in live], [len(c.tokens) for c in live], flat, [c.logits for c in live],
-                               [int(bool(c.output)) for c in live], device_tokens, cfg.max_tokens)
+        self._check_batch(live)
+        places = [list(c.places) if c.places is not None else [] for c in live] \
+            if any(c.places is not None for c in live) else []
+        plan = self.sched.plan([c.seq for c in live], [len(c.tokens) for c in live], flat,
+                               [-1 if c.places is not None else c.logits for c in live],
+                               [int(bool(c.output)) for c in live], device_tokens, cfg.max_tokens, places, self._short_len)
+        self._segments = plan["segments"]
         for old, nb in plan["cows"]:
             self._copy_block(old, nb)
         for sid in plan["tables"]:
@@ -561,7 +596,8 @@ class Engine:
             self._stats = stats
             return self._logits
         self._skinny = 16
-        decode_only = all(k == "paged" for k, *_ in runs) and N == R == stats.decode_tokens
+        decode_only = all(k == "paged" for k, *_ in runs) and N == R == stats.decode_tokens and \
+            (not self.SEGMENT_ROWS or self._segments[0][0] == N)
         # tensor-parallel ranks run the same schedule, so with tp_graphs every rank captures and replays the same buckets
         # in the same order, the all-reduces of the layer loop captured with the kernels around them
         use_graph = self.fast and cfg.cuda_graphs and decode_only and nl == self.L and (self.tp == 1 or cfg.tp_graphs)
@@ -569,6 +605,9 @@ class Engine:
         # one staging buffer in pinned memory, reused every step, and ONE host-to-device copy for all index arrays
         ints = self._stage(bucket)
         self.sched.write(ints.data_ptr(), bucket)
+        if self.SEGMENT_ROWS:
+            self.sched.write_segments(ints[self.INDEX_ROWS].data_ptr(), bucket)
+            self._host_rows = ints
         if use_graph:
             logits = self._decode_graph(bucket, ints, N if device_tokens else 0)[:R]
             dv = self._static[bucket]["ints"]
@@ -577,7 +616,7 @@ class Engine:
             dv = ints.to(self.dev, non_blocking=True)
             if device_tokens:
                 dv[0, :N] = self._last_tok[dv[3, :N].long()]
-            logits = self._body(dv[0], dv[1], dv[2], dv[3], dv[4], dv[5][:R], runs, nl)
+            logits = self._body_rows(dv, R, runs, nl)
         if self.dev.type == "cuda":
             ev = self._stage_evt.get(bucket)
             if ev is None:
@@ -597,6 +636,15 @@ class Engine:
         stats.ms = (time.perf_counter() - t0) * 1e3
         self._stats = stats
         return logits
+
+    _short_len = 16              # segments of up to this many tokens are listed apart from longer ones
+
+    def _check_batch(self, chunks: Sequence[Chunk]) -> None:
+        """Refuses a step the model cannot run, before anything of it is planned."""
+
+    def _body_rows(self, dv: torch.Tensor, logit_rows: int, runs, nl: int) -> torch.Tensor:
+        """`_body` on the index rows of one step ([INDEX_ROWS + SEGMENT_ROWS, rows], on the device)."""
+        return self._body(dv[0], dv[1], dv[2], dv[3], dv[4], dv[5][:logit_rows], runs, nl)
 
     def _body(self, tok, pos, slot, rseq, ctx_len, logit_rows, runs, nl: int) -> torch.Tensor:
         """Layer loop over device index arrays (also the body of the captured decode graphs)."""
@@ -701,13 +749,13 @@ class Engine:
             att[r] = torch.einsum("hn,nhd->hd", s.softmax(-1), vv).to(att.dtype)
 
     def _stage(self, width: int) -> torch.Tensor:
-        """Host staging tensor [6, width] int32 (pinned on a GPU), one per width, reused by every step."""
+        """Host staging tensor [index rows, width] int32 (pinned on a GPU), one per width, reused by every step."""
         t = self._stage_bufs.get(width)
         ev = self._stage_evt.get(width)
         if ev is not None:
             ev.synchronize()          # the copy that last read this buffer has run
         if t is None:
-            t = torch.zeros((6, width), dtype=torch.int32)
+            t = torch.zeros((self.INDEX_ROWS + self.SEGMENT_ROWS, width), dtype=torch.int32)
             if self.dev.type == "cuda":
                 t = t.pin_memory()
             if len(self._stage_bufs) > 64:
@@ -720,22 +768,22 @@ class Engine:
     def _decode_graph(self, bucket: int, ints: torch.Tensor, device_rows: int = 0) -> torch.Tensor:
         st = self._static.get(bucket)
         if st is None:
-            st = {"ints": torch.zeros((6, bucket), dtype=torch.int32, device=self.dev)}
+            st = {"ints": torch.zeros((self.INDEX_ROWS + self.SEGMENT_ROWS, bucket), dtype=torch.int32, device=self.dev)}
             st["ints"][2].fill_(-1)
             self._static[bucket] = st
             runs = [("paged", 0, bucket, -1)]
             side = torch.cuda.Stream()
             side.wait_stream(torch.cuda.current_stream())
-            with torch.cuda.stream(side):    # warm-up outside capture: lazy allocations, scratch growth
-                st["ints"].copy_(ints, non_blocking=True)
-                i = st["ints"]
-                self._body(i[0], i[1], i[2], i[3], i[4], i[5], runs, self.L)
+            self._segments = [(bucket, 1, bucket), (0, 0, 0), (0, 0, 0)]
+            # warm-up outside capture (lazy allocations, scratch growth) on padding rows: they touch no cache slot and no
+            # state, which matters where running a token twice is not the same as running it once
+            with torch.cuda.stream(side):
+                self._body_rows(st["ints"], bucket, runs, self.L)
             torch.cuda.current_stream().wait_stream(side)
             torch.cuda.synchronize()
             g = torch.cuda.CUDAGraph()
             with torch.cuda.graph(g):
-                i = st["ints"]
-                st["logits"] = self._body(i[0], i[1], i[2], i[3], i[4], i[5], runs, self.L)
+                st["logits"] = self._body_rows(st["ints"], bucket, runs, self.L)
             self._graphs[bucket] = g
         st["ints"].copy_(ints, non_blocking=True)
         if device_rows:   # tokens drawn by the previous step, still only on the device

@@ -1,0 +1,337 @@
+"""Serving decoders with heterogeneous layers (`lm.hybrid`) on the shared engine.
+
+What differs from the GPT-2 family is below `Engine.forward`: the layer loop, and what a sequence owns beside its cache
+pages.  Pages exist for the layers with attention only (keys and values may have different widths); the layers with a
+recurrence keep one slot per sequence: the FP32 state and the last inputs of the short convolution.  A sequence that
+starts over starts from zeros because its first segment starts at position 0, so a slot needs no clearing when it is used
+again.
+
+A step runs every row of the batch through each projection together; the mixers then take the segments of the batch (one
+per sequence) in up to three groups, one-token segments, short ones and long ones, with the kernel that suits each:
+
+* attention: split-key decode kernel | paged prompt kernel | tcgen05 flash kernel (fresh prompts, head sizes 64 / 128)
+* recurrences: token-by-token kernel with the state tile in shared memory | chunked tensor-core kernel
+
+The residual stream is FP32; one kernel adds a normed sublayer output to it and norms it for the next sublayer.  In FP32
+precision the same layer loop runs the kernels' FP32 forms and plain FP32 matrix products.
+"""
+from __future__ import annotations
+
+from typing import Dict, List, Sequence
+
+import torch
+
+from ..lm.hybrid import DeltaSpec, HybridConfig, HybridWeights, ParallelSpec
+from .engine import Chunk, Engine, _Linear
+
+__all__ = ["HybridEngine"]
+
+FLASH_MIN = 128          # fresh prompts from this length on take the tcgen05 flash kernel where the head size allows it
+
+
+def _pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+class HybridEngine(Engine):
+    SEGMENT_ROWS = 4
+
+    # ----------------------------------------------------------------------------- configuration
+    def _configure(self, weights: HybridWeights) -> None:
+        cfg = self.cfg
+        if self.dev.type != "cuda":
+            raise ValueError("this model runs on the CUDA kernels only (device 'cuda')")
+        if self.tp > 1:
+            raise ValueError("this model has no tensor-parallel form")
+        if cfg.quant.weights != "bf16" or cfg.quant.kv != "bf16":
+            raise ValueError("this model has no quantised weights or cache")
+        from ..ops import _cuda as K
+        K.lib()
+        if not self.fast:
+            torch.backends.cuda.matmul.allow_tf32 = False
+        self.model: HybridConfig = weights.config
+        self.L, self.d, self.V = len(self.model.layers), self.model.width, self.model.vocab
+        self.adt = torch.bfloat16 if self.fast else torch.float32
+        self.kv_kind = 0
+        elem = 2 if self.fast else 4
+        self._kv_tok_bytes = max(1, self.model.kv_bytes_per_token(elem))
+        self.n_blocks = self._pool_blocks(self._kv_tok_bytes)
+        self.ctx = cfg.context if cfg.context > 0 else self.n_blocks * cfg.block_size
+        self._rope: Dict[tuple, tuple] = {}
+        self._short_len = 1 << 30
+
+    def _rope_tables(self, dims: int, base: float):
+        """cos / sin [ctx, dims / 2]: angles in double, kept in FP32."""
+        key = (dims, base)
+        if key not in self._rope:
+            half = dims // 2
+            freq = float(base) ** (-2.0 * torch.arange(half, dtype=torch.float64) / max(dims, 1))
+            ang = torch.arange(self.ctx, dtype=torch.float64)[:, None] * freq[None, :]
+            self._rope[key] = tuple(f(ang).float().to(self.dev).contiguous() for f in (torch.cos, torch.sin))
+        return self._rope[key]
+
+    # ----------------------------------------------------------------------------- weights
+    def _pack(self, parts: Sequence[torch.Tensor]):
+        """Stacks projections of one input: rows of each part padded to a multiple of 8, columns padded to a multiple of
+        8.  Returns the linear layer and the first output column of every part."""
+        k = _pad8(parts[0].shape[1])
+        offsets, n = [], 0
+        for p in parts:
+            offsets.append(n)
+            n += _pad8(p.shape[0])
+        w = torch.zeros((n, k))
+        for p, o in zip(parts, offsets):
+            w[o: o + p.shape[0], : p.shape[1]] = p.float()
+        lin = _Linear(w, None, self.dev, self.fast)
+        self.weight_nbytes += lin.nbytes
+        return lin, offsets
+
+    def _f32(self, t: torch.Tensor) -> torch.Tensor:
+        return t.to(self.dev, torch.float32).contiguous()
+
+    def _load(self, weights: HybridWeights) -> None:
+        t, model = weights.tensors, self.model
+        self.weight_nbytes = 0
+        head = torch.zeros((self.Vp, self.d))
+        head[: self.V] = t["head"].float()
+        self.head, _ = self._pack([head])
+        self.embed = t["embed"].to(self.dev, self.adt).contiguous()
+        self.side_embed = t["side.embed"].to(self.dev, self.adt).contiguous()
+        self.weight_nbytes += sum(e.numel() * e.element_size() for e in (self.embed, self.side_embed))
+        self.final_norm = self._f32(t["final.norm"])
+        self.layers: List[dict] = []
+        for i, layer in enumerate(model.layers):
+            p, m = f"l{i}.", layer.mixer
+            out = {n: self._f32(t[p + n]) for n in ("norm1", "norm1b")}
+            if isinstance(m, ParallelSpec):
+                a, r = m.left, m.right
+                w_in = t[p + "mix.right.in"]
+                z, xbc, dt = w_in.split([r.inner, r.channels, r.heads], 0)
+                left = [t[p + f"mix.left.{n}"] for n in ("q", "k", "v")]
+                out["in"], out["off"] = self._pack([*left, z, xbc, dt])
+                # both output projections read one buffer [attention | ssd]
+                na, nr = a.heads * a.vdim, r.inner
+                wo = torch.zeros((_pad8(self.d), _pad8(na) + _pad8(nr)))
+                wo[: self.d, :na] = t[p + "mix.left.o"].float()
+                wo[: self.d, _pad8(na): _pad8(na) + nr] = t[p + "mix.right.o"].float()
+                out["out"] = _Linear(wo, None, self.dev, self.fast)
+                self.weight_nbytes += out["out"].nbytes
+                out["conv"] = self._f32(t[p + "mix.right.conv"].t())
+                out["conv_b"] = self._f32(t[p + "mix.right.conv.b"])
+                for n, key in (("dt_bias", "dt_bias"), ("A_log", "a_log"), ("D", "d_skip"), ("norm", "norm")):
+                    out[key] = self._f32(t[p + "mix.right." + n])
+                out["rope"] = self._rope_tables(a.rope_dims, a.rope_base)
+            else:
+                # q, k and v stay adjacent (they share one convolution); then b, a and the output gate
+                qkv = torch.cat([t[p + f"mix.{n}"] for n in ("q", "k", "v")], 0)
+                out["in"], out["off"] = self._pack([qkv, t[p + "mix.b"], t[p + "mix.a"], t[p + "mix.g"]])
+                out["out"], _ = self._pack([t[p + "mix.o"]])
+                out["conv"] = self._f32(torch.cat([t[p + f"mix.{n}.conv"] for n in ("q", "k", "v")], 0).t())
+                out["conv_b"] = None
+                for n, key in (("dt_bias", "dt_bias"), ("A_log", "a_log"), ("norm", "norm")):
+                    out[key] = self._f32(t[p + "mix." + n])
+            if layer.ff:
+                out["norm2"], out["norm2b"] = self._f32(t[p + "norm2"]), self._f32(t[p + "norm2b"])
+                out["up"], _ = self._pack([t[p + "mlp.gate"], t[p + "mlp.up"]])
+                out["down"], _ = self._pack([t[p + "mlp.down"]])
+            out["side_gate"], _ = self._pack([t[p + "side.gate"]])
+            out["side_proj"], _ = self._pack([t[p + "side.proj"]])
+            out["side_norm"] = self._f32(t[p + "side.norm"])
+            self.layers.append(out)
+
+    # ----------------------------------------------------------------------------- cache pages and state slots
+    def _alloc_kv(self) -> None:
+        cfg = self.cfg
+        self.max_blocks = -(-self.ctx // cfg.block_size)
+        self.k_cache: list = [None] * self.L
+        self.v_cache: list = [None] * self.L
+        self.state: list = [None] * self.L        # FP32 [slots, heads, key size, value size]
+        self.conv_tail: list = [None] * self.L    # [slots, taps - 1, channels]
+        for i, layer in enumerate(self.model.layers):
+            m = layer.mixer
+            if isinstance(m, ParallelSpec):
+                a, r = m.left, m.right
+                self.k_cache[i] = torch.zeros((self.n_blocks, cfg.block_size, a.kv_heads, a.dim), dtype=self.adt, device=self.dev)
+                self.v_cache[i] = torch.zeros((self.n_blocks, cfg.block_size, a.kv_heads, a.vdim), dtype=self.adt, device=self.dev)
+                shape, taps, channels = (r.heads, r.state, r.vdim), r.conv, r.channels
+            else:
+                shape, taps, channels = (m.heads, m.dim, m.vdim), m.conv, m.channels
+            self.state[i] = torch.zeros((cfg.max_seqs, *shape), dtype=torch.float32, device=self.dev)
+            self.conv_tail[i] = torch.zeros((cfg.max_seqs, max(taps - 1, 1), channels), dtype=self.adt, device=self.dev)
+        self.k_scale = self.v_scale = [None] * self.L
+
+    def state_bytes_per_sequence(self) -> int:
+        return sum(t[0].numel() * t.element_size() for t in (*self.state, *self.conv_tail))
+
+    def _fork_state(self, src: int, dst: int) -> None:
+        for t in (*self.state, *self.conv_tail):
+            t[dst].copy_(t[src])
+
+    def _check_truncate(self, seq: int, length: int) -> None:
+        if 0 < length < self.length(seq):
+            raise ValueError("a recurrent state cannot be taken back: truncate to 0, or fork the sequence beforehand")
+
+    def _check_batch(self, chunks: Sequence[Chunk]) -> None:
+        seen, last = set(), None
+        for c in chunks:
+            if c.seq != last and c.seq in seen:
+                raise ValueError("chunks of one sequence must be adjacent in a step")
+            seen.add(c.seq)
+            last = c.seq
+
+    def forward(self, chunks: Sequence[Chunk], layers: int = -1, device_tokens: bool = False) -> torch.Tensor:
+        if 0 <= layers < self.L:
+            raise ValueError("running the first layers only would advance some states and not others")
+        return super().forward(chunks, layers, device_tokens)
+
+    # ----------------------------------------------------------------------------- one step
+    def _body_rows(self, dv: torch.Tensor, logit_rows: int, runs, nl: int) -> torch.Tensor:
+        from ..ops import _mixers as M
+        table = dv[self.INDEX_ROWS:]
+        groups, first = [], 0
+        for count, longest, total in self._segments:
+            groups.append(M.Segments(table, first, count, longest, total))
+            first += count
+        self._groups = groups
+        single, short, long_ = groups
+        self._many = M.Segments(table, single.count, short.count + long_.count, max(short.max_len, long_.max_len),
+                                short.total + long_.total)
+        self._stepped = M.Segments(table, 0, single.count + short.count, max(single.max_len, short.max_len),
+                                   single.total + short.total)
+        return self._body(dv[0], dv[1], dv[2], dv[3], dv[4], dv[5][:logit_rows], runs, nl)
+
+    def _buffer(self, rows: int, cols: int) -> torch.Tensor:
+        """Activation buffer whose pitch the tensor-core GEMM accepts; columns past ``cols`` are zeros."""
+        ld = _pad8(cols)
+        return (torch.zeros if ld != cols else torch.empty)((rows, ld), dtype=self.adt, device=self.dev)
+
+    def _decode_splits(self, a, rows: int) -> int:
+        if self.cfg.decode_splits > 0:
+            return self.cfg.decode_splits
+        keys = min(a.window, self.ctx) if a.window > 0 else self.ctx
+        ctas = rows * a.kv_heads * (-(-(a.heads // a.kv_heads) // 16))
+        return max(1, min(592 // max(ctas, 1), -(-keys // 256), 32))
+
+    def _attention(self, i: int, a, proj, off, out, out_scale: float) -> None:
+        """Rotated queries in ``proj`` against the cache of layer ``i``; ``out``: [rows, heads * vdim] view."""
+        from ..ops import _cuda as K
+        from ..ops import _mixers as M
+        single, short, long_ = self._groups
+        q = proj[:, off: off + a.heads * a.dim]
+        kw = dict(heads=a.heads, block_size=self.cfg.block_size, window=a.window, scale=a.scale, softcap=a.softcap,
+                  out_scale=out_scale)
+        paged = (self.k_cache[i], self.v_cache[i], self.block_table, out)
+        if not self.fast:
+            every = M.Segments(single.table, 0, single.count + short.count, max(single.max_len, short.max_len),
+                               single.total + short.total)
+            M.paged_window_attention(q, *paged, every, **kw)
+            return
+        if single.count:
+            M.paged_window_attention(q, *paged, single, splits=self._decode_splits(a, single.count), **kw)
+        if not self._many.count:
+            return
+        host = self._host_rows[self.INDEX_ROWS:]
+        flash = long_.count > 0 and a.dim == a.vdim and a.dim in (64, 128) and self._many.count <= 64 and all(
+            int(host[1, j]) >= FLASH_MIN and int(host[2, j]) == 0 for j in range(single.count, single.count + self._many.count))
+        if not flash:
+            M.paged_window_attention(q, *paged, self._many, **kw)
+            return
+        _, k0, v0 = self.layers[i]["off"][:3]
+        for j in range(single.count, single.count + self._many.count):
+            r0, n = int(host[0, j]), int(host[1, j])
+            rows = proj[r0: r0 + n]
+            K.attention_fwd(rows[:, off: off + a.heads * a.dim].view(1, n, a.heads, a.dim),
+                            rows[:, k0: k0 + a.kv_heads * a.dim].view(1, n, a.kv_heads, a.dim),
+                            rows[:, v0: v0 + a.kv_heads * a.vdim].view(1, n, a.kv_heads, a.vdim), causal=True,
+                            window=a.window, scale=a.scale, softcap=a.softcap, out_scale=out_scale,
+                            out=out[r0: r0 + n].view(1, n, a.heads, a.vdim))
+
+    def _conv(self, x, w, bias, tail) -> torch.Tensor:
+        from ..ops import _mixers as M
+        y = torch.empty((x.shape[0], w.shape[1]), dtype=self.adt, device=self.dev)
+        for seg in (self._groups[0], self._many):
+            if seg.count:
+                M.conv_silu(x, y, w, bias, tail, seg)
+        return y
+
+    def _parallel_mixer(self, i: int, m: ParallelSpec, lw: dict, h, pos, slot) -> torch.Tensor:
+        from ..ops import _mixers as M
+        a, r, n = m.left, m.right, h.shape[0]
+        proj = self._linear(h, lw["in"])
+        oq, ok, ov, oz, ox, od = lw["off"]
+        M.rope_append(proj, oq, ok, ov, a.heads, a.kv_heads, a.dim, a.vdim, a.rope_dims, pos, slot, *lw["rope"],
+                      self.k_cache[i], self.v_cache[i])
+        na, nr = a.heads * a.vdim, r.inner
+        ka = _pad8(na)
+        both = (torch.empty if ka == na and nr % 8 == 0 else torch.zeros)((n, ka + _pad8(nr)), dtype=self.adt, device=self.dev)
+        self._attention(i, a, proj, oq, both[:, :na], m.left_scale)
+        xbc = self._conv(proj[:, ox: ox + r.channels], lw["conv"], lw["conv_b"], self.conv_tail[i])
+        y = torch.empty((n, nr), dtype=self.adt, device=self.dev)
+        ssd = (xbc, proj[:, od: od + r.heads], y, lw["dt_bias"], lw["a_log"], lw["d_skip"], self.state[i], r.groups)
+        if self._stepped.count:
+            M.ssd(*ssd, self._stepped)
+        if self._groups[2].count:
+            M.ssd(*ssd, self._groups[2], chunked=True, parts=self._ssd_parts(r))
+        M.gated_norm(y, proj[:, oz: oz + nr], lw["norm"], both[:, ka: ka + nr], groups=r.norm_groups, gate_first=True,
+                     eps=self.model.norm_eps, out_scale=m.right_scale)
+        return self._linear(both, lw["out"])
+
+    def _ssd_parts(self, r) -> int:
+        """Spans per long segment: enough (segment, head, span) blocks to fill the GPU, at least 4 chunks each."""
+        seg = self._groups[2]
+        chunks = -(-seg.max_len // 64)
+        return max(1, min(296 // max(1, seg.count * r.heads), chunks // 4))
+
+    def _delta_mixer(self, i: int, m: DeltaSpec, lw: dict, h) -> torch.Tensor:
+        from ..ops import _mixers as M
+        n = h.shape[0]
+        proj = self._linear(h, lw["in"])
+        ox, ob, oa, og = lw["off"]
+        qkv = self._conv(proj[:, ox: ox + m.channels], lw["conv"], lw["conv_b"], self.conv_tail[i])
+        o = torch.empty((n, m.heads * m.vdim), dtype=self.adt, device=self.dev)
+        args = (qkv, proj[:, ob: ob + m.heads], proj[:, oa: oa + m.heads], o, lw["dt_bias"], lw["a_log"], self.state[i], m.kv_heads)
+        kw = dict(unit_eps=m.unit_eps, q_scale=m.dim ** -0.5)
+        if self._stepped.count:
+            M.delta(*args, self._stepped, **kw)
+        if self._groups[2].count:
+            M.delta(*args, self._groups[2], chunked=True, **kw)
+        out = self._buffer(n, m.heads * m.vdim)
+        M.gated_norm(o, proj[:, og: og + m.heads * m.vdim], lw["norm"], out[:, : m.heads * m.vdim], groups=m.heads,
+                     gate_first=False, eps=self.model.norm_eps)
+        return self._linear(out, lw["out"])
+
+    def _body(self, tok, pos, slot, rseq, ctx_len, logit_rows, runs, nl: int) -> torch.Tensor:
+        from ..ops import _mixers as M
+        n, eps, model, cap = tok.shape[0], self.model.norm_eps, self.model, self._capture
+        x = torch.empty((n, self.d), dtype=torch.float32, device=self.dev)
+        h = torch.empty((n, _pad8(self.d)), dtype=self.adt, device=self.dev)
+        M.residual_norm(x, tokens=tok, table=self.embed, w_next=self.layers[0]["norm1"], h=h, eps=eps)
+        for i, (layer, lw) in enumerate(zip(model.layers, self.layers)):
+            m = layer.mixer
+            y = self._parallel_mixer(i, m, lw, h, pos, slot) if isinstance(m, ParallelSpec) else self._delta_mixer(i, m, lw, h)
+            post = lw["norm1b"]
+            if layer.ff:
+                M.residual_norm(x, y=y, w_post=post, w_next=lw["norm2"], h=h, eps=eps)
+                gu = self._linear(h, lw["up"])
+                act = torch.empty((n, gu.shape[1] // 2), dtype=self.adt, device=self.dev)
+                M.silu_mul(gu, act)
+                y, post = self._linear(act, lw["down"]), lw["norm2b"]
+            M.residual_norm(x, y=y, w_post=post, x_cast=h, eps=eps)
+            gate = self._linear(h, lw["side_gate"])
+            side = torch.empty_like(gate)
+            M.token_side_gate(gate, tok, self.side_embed, i * model.token_side, side, model.token_side)
+            y = self._linear(side, lw["side_proj"])
+            last = i + 1 == self.L
+            M.residual_norm(x, y=y, w_post=lw["side_norm"], eps=eps, **({} if last else {
+                "w_next": self.layers[i + 1]["norm1"], "h": h}))
+            if cap is not None:
+                cap.append(x.detach().float().cpu())
+        if logit_rows.shape[0] == 0:
+            return torch.zeros((0, self.Vp), dtype=torch.float32, device=self.dev)
+        xr = x.index_select(0, logit_rows.long())
+        hr = torch.empty((xr.shape[0], _pad8(self.d)), dtype=self.adt, device=self.dev)
+        M.residual_norm(xr, w_next=self.final_norm, h=hr, eps=eps)
+        logits = self._linear(hr, self.head, out_dtype=torch.float32)
+        if model.logit_softcap > 0:
+            M.softcap_(logits, self.V, model.logit_softcap)
+        return logits

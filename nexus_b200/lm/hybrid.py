@@ -1,0 +1,280 @@
+"""Decoders whose layers differ from one another: the layer list, the mixers' sizes and constants, and the weights.
+
+A model is an ordered list of :class:`HybridLayer`; each has one mixer - :class:`AttentionSpec` and :class:`SsdSpec` side
+by side (:class:`ParallelSpec`) or :class:`DeltaSpec` - and optionally a gated feed-forward.  The engine
+(`infer.hybrid.HybridEngine`) builds its cache, its state slots and its kernels' arguments from these specs and reads no
+size from anywhere else, so another order of layers or another combination of constants is another configuration, not
+another class.
+
+`Gugedra` is the design that uses them so far: RMS norms before and after every sublayer, a sliding-window soft-capped
+attention branch beside a Mamba-2 branch in some layers, the gated delta rule in the others, a per-layer token input at
+the end of every layer and soft-capped logits.  :func:`gugedra_config` reads its ``config.json``, and
+:func:`load_gugedra` its ``model.safetensors``.
+"""
+from __future__ import annotations
+
+import json
+import math
+import os
+from dataclasses import dataclass, field
+from typing import Dict, List, Optional, Tuple, Union
+
+import torch
+
+from .config import ConfigError
+
+__all__ = ["AttentionSpec", "SsdSpec", "ParallelSpec", "DeltaSpec", "HybridLayer", "HybridConfig", "HybridWeights",
+           "gugedra_config", "gugedra_tensors", "load_gugedra", "random_gugedra"]
+
+
+def _positive(obj, *names) -> None:
+    for n in names:
+        v = getattr(obj, n)
+        if not isinstance(v, int) or isinstance(v, bool) or v < 1:
+            raise ConfigError(f"{type(obj).__name__}.{n} must be a positive integer, not {v!r}")
+
+
+@dataclass(frozen=True)
+class AttentionSpec:
+    """Causal softmax attention; query head h reads KV head h // (heads / kv_heads)."""
+    heads: int
+    kv_heads: int
+    dim: int                 # query / key size of a head
+    vdim: int                # value size of a head
+    scale: float
+    softcap: float = 0.0     # > 0: score = softcap * tanh(score / softcap)
+    window: int = 0          # > 0: a token sees itself and the window - 1 tokens before it
+    rope_dims: int = 0       # leading dimensions of a head that rotate (rotate-half pairing)
+    rope_base: float = 10000.0
+
+    def __post_init__(self):
+        _positive(self, "heads", "kv_heads", "dim", "vdim")
+        if self.heads % self.kv_heads:
+            raise ConfigError("attention: heads must be a multiple of kv_heads")
+        if self.rope_dims % 2 or not 0 <= self.rope_dims <= self.dim:
+            raise ConfigError("attention: the rotary dimensions must be even and at most the head size")
+        if self.window < 0 or self.softcap < 0:
+            raise ConfigError("attention: window and softcap cannot be negative")
+
+
+@dataclass(frozen=True)
+class SsdSpec:
+    """Mamba-2; head h reads group h // (heads / groups)."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int                # taps of the short convolution
+    norm_groups: int
+
+    def __post_init__(self):
+        _positive(self, "heads", "vdim", "state", "groups", "conv", "norm_groups")
+        if self.heads % self.groups:
+            raise ConfigError("ssd: heads must be a multiple of groups")
+        if self.inner % self.norm_groups:
+            raise ConfigError("ssd: norm_groups must divide heads * vdim")
+        if self.conv > 8:
+            raise ConfigError("ssd: the convolution kernel has at most 8 taps")
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:
+        return self.inner + 2 * self.groups * self.state
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """left_scale * attention + right_scale * ssd, both reading the same input."""
+    left: AttentionSpec
+    right: SsdSpec
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+
+@dataclass(frozen=True)
+class DeltaSpec:
+    """Gated delta rule; head h reads query / key head h // (heads / kv_heads)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+    unit_eps: float = 1e-6   # inside the root of the unit vectors
+
+    def __post_init__(self):
+        _positive(self, "heads", "kv_heads", "dim", "vdim", "conv")
+        if self.heads % self.kv_heads:
+            raise ConfigError("delta: heads must be a multiple of kv_heads")
+        if self.conv > 8:
+            raise ConfigError("delta: the convolution kernel has at most 8 taps")
+
+    @property
+    def channels(self) -> int:
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class HybridLayer:
+    mixer: Union[ParallelSpec, DeltaSpec]
+    ff: int = 0              # width of the SwiGLU feed-forward, 0: none
+
+
+@dataclass
+class HybridConfig:
+    vocab: int
+    width: int
+    layers: List[HybridLayer] = field(default_factory=list)
+    norm_eps: float = 1e-6
+    token_side: int = 0      # width of the per-layer token input
+    logit_softcap: float = 0.0
+    name: str = "hybrid"
+
+    def __post_init__(self):
+        _positive(self, "vocab", "width", "token_side")
+        if not self.layers:
+            raise ConfigError("a model needs at least one layer")
+
+    def kv_bytes_per_token(self, element: int) -> int:
+        return sum(m.left.kv_heads * (m.left.dim + m.left.vdim) * element
+                   for m in (layer.mixer for layer in self.layers) if isinstance(m, ParallelSpec))
+
+
+@dataclass
+class HybridWeights:
+    """A configuration and its tensors (host memory, the design's own names)."""
+    config: HybridConfig
+    tensors: Dict[str, torch.Tensor]
+
+    @property
+    def vocab(self) -> int:
+        return self.config.vocab
+
+    def parameters(self) -> int:
+        return sum(t.numel() for t in self.tensors.values())
+
+
+# ------------------------------------------------------------------------------------------ Gugedra
+def _take(obj: dict, where: str, names: Tuple[str, ...]) -> list:
+    """Exactly these keys: a key nobody reads would be a constant that is silently ignored."""
+    if not isinstance(obj, dict):
+        raise ConfigError(f"{where}: an object is expected")
+    missing, extra = [n for n in names if n not in obj], [k for k in obj if k not in names]
+    if missing or extra:
+        raise ConfigError(f"{where}: " + "; ".join(
+            ([f"missing {', '.join(missing)}"] if missing else []) + ([f"unknown {', '.join(extra)}"] if extra else [])))
+    return [obj[n] for n in names]
+
+
+def _attention(obj: dict, where: str) -> AttentionSpec:
+    heads, kv, dim, vdim, scale, cap, mask, rot = _take(
+        obj, where, ("heads", "kv_heads", "dim", "vdim", "scale", "softcap", "mask", "rot"))
+    (size,) = _take(mask, where + ".mask", ("size",))
+    base, dims = _take(rot, where + ".rot", ("base", "dims"))
+    return AttentionSpec(heads, kv, dim, vdim, float(scale), float(cap), int(size), int(dims), float(base))
+
+
+def gugedra_config(obj: dict) -> HybridConfig:
+    """``config.json`` of a Gugedra model."""
+    _, layers, cap, norm, side, vocab, width = _take(
+        obj, "config", ("architecture", "layers", "logit_softcap", "norm", "token_side", "vocab", "width"))
+    (eps,) = _take(norm, "norm", ("eps",))
+    (side_dim,) = _take(side, "token_side", ("dim",))
+    out = []
+    for i, layer in enumerate(layers):
+        kind, mix, mlp = _take(layer, f"layers[{i}]", ("type", "mixer", "mlp"))
+        where = f"layers[{i}].mixer"
+        if kind == "parallel":
+            left, ls, right, rs = _take(mix, where, ("left", "left_scale", "right", "right_scale"))
+            spec = ParallelSpec(_attention(left, where + ".left"),
+                                SsdSpec(*_take(right, where + ".right", ("heads", "vdim", "state", "groups", "conv", "norm_groups"))),
+                                float(ls), float(rs))
+        elif kind == "delta":
+            spec = DeltaSpec(*_take(mix, where, ("heads", "kv_heads", "dim", "vdim", "conv")))
+        else:
+            raise ConfigError(f"layers[{i}]: unknown mixer {kind!r}")
+        ff = 0
+        if mlp is not None:
+            mlp_kind, ff = _take(mlp, f"layers[{i}].mlp", ("kind", "ff"))
+            if mlp_kind != "dense" or ff < 1:
+                raise ConfigError(f"layers[{i}].mlp: a dense feed-forward is expected")
+        out.append(HybridLayer(spec, ff))
+    return HybridConfig(vocab, width, out, float(eps), side_dim, float(cap), "Gugedra")
+
+
+def gugedra_tensors(cfg: HybridConfig) -> Dict[str, Tuple[int, ...]]:
+    """Name and shape of every tensor."""
+    W = cfg.width
+    t: Dict[str, Tuple[int, ...]] = {"embed": (cfg.vocab, W), "side.embed": (cfg.vocab, cfg.token_side * len(cfg.layers)),
+                                     "final.norm": (W,), "head": (cfg.vocab, W)}
+    for i, layer in enumerate(cfg.layers):
+        p, m = f"l{i}.", layer.mixer
+        t[p + "norm1"] = t[p + "norm1b"] = (W,)
+        if isinstance(m, ParallelSpec):
+            a, r = m.left, m.right
+            t[p + "mix.left.q"], t[p + "mix.left.k"] = (a.heads * a.dim, W), (a.kv_heads * a.dim, W)
+            t[p + "mix.left.v"], t[p + "mix.left.o"] = (a.kv_heads * a.vdim, W), (W, a.heads * a.vdim)
+            t[p + "mix.right.in"] = (r.inner + r.channels + r.heads, W)
+            t[p + "mix.right.conv"], t[p + "mix.right.conv.b"] = (r.channels, r.conv), (r.channels,)
+            for n in ("dt_bias", "A_log", "D"):
+                t[p + "mix.right." + n] = (r.heads,)
+            t[p + "mix.right.norm"], t[p + "mix.right.o"] = (r.inner,), (W, r.inner)
+        else:
+            for n, size in (("q", m.kv_heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.heads * m.vdim)):
+                t[p + "mix." + n], t[p + f"mix.{n}.conv"] = (size, W), (size, m.conv)
+            t[p + "mix.b"] = t[p + "mix.a"] = (m.heads, W)
+            t[p + "mix.A_log"] = t[p + "mix.dt_bias"] = (m.heads,)
+            t[p + "mix.norm"], t[p + "mix.g"], t[p + "mix.o"] = (m.vdim,), (m.heads * m.vdim, W), (W, m.heads * m.vdim)
+        if layer.ff:
+            t[p + "norm2"] = t[p + "norm2b"] = (W,)
+            t[p + "mlp.gate"] = t[p + "mlp.up"] = (layer.ff, W)
+            t[p + "mlp.down"] = (W, layer.ff)
+        t[p + "side.gate"], t[p + "side.proj"], t[p + "side.norm"] = (cfg.token_side, W), (W, cfg.token_side), (W,)
+    return t
+
+
+def check_tensors(cfg: HybridConfig, tensors: Dict[str, torch.Tensor]) -> None:
+    want = gugedra_tensors(cfg)
+    missing, extra = sorted(set(want) - set(tensors)), sorted(set(tensors) - set(want))
+    if missing or extra:
+        raise ConfigError(f"weights do not fit the configuration: missing {missing[:4]}, unknown {extra[:4]}")
+    for n, shape in want.items():
+        if tuple(tensors[n].shape) != shape:
+            raise ConfigError(f"{n}: shape {tuple(tensors[n].shape)}, expected {shape}")
+
+
+def load_gugedra(folder: str) -> HybridWeights:
+    """A folder with ``config.json`` and ``model.safetensors``."""
+    from ..interop.safetensors import load_file
+    with open(os.path.join(folder, "config.json")) as f:
+        cfg = gugedra_config(json.load(f))
+    tensors = load_file(os.path.join(folder, "model.safetensors"))
+    check_tensors(cfg, tensors)
+    return HybridWeights(cfg, tensors)
+
+
+def random_gugedra(cfg: HybridConfig, seed: int = 0) -> HybridWeights:
+    """Random BF16 weights of a configuration (benchmarks, examples): unit-variance activations, decays spread over
+    short and long memories."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for n, shape in gugedra_tensors(cfg).items():
+        leaf = n.rsplit(".", 1)[-1]
+        if leaf.startswith("norm") or leaf == "D":
+            v = torch.ones(shape)
+        elif leaf == "A_log":
+            v = torch.linspace(-1.0, 1.5, shape[0])
+        elif leaf == "dt_bias":
+            v = torch.linspace(-4.0, -1.0, shape[0])
+        elif leaf == "conv":
+            v = torch.randn(shape, generator=g) / math.sqrt(shape[1])
+        elif leaf == "b" and len(shape) == 1:
+            v = torch.zeros(shape)
+        elif leaf == "embed":
+            v = torch.randn(shape, generator=g)
+        else:
+            v = torch.randn(shape, generator=g) / math.sqrt(shape[-1])
+        out[n] = v.to(torch.bfloat16)
+    return HybridWeights(cfg, out)

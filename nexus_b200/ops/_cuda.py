@@ -18,6 +18,7 @@ _LIB_PATH = Path(__file__).resolve().parent.parent / "lib" / "libnexus_b200_cuda
 _lib = None
 _status = {}
 _scratch = {}
+_outgrown = []
 launch_count = 0  # kernels launched through this module (bench.py reports it)
 
 BF16, F32, F16, E4M3, E5M2 = 0, 1, 2, 3, 4
@@ -60,6 +61,7 @@ class AttnArgs(C.Structure):
         ("merge_o", C.c_void_p), ("merge_lse", C.c_void_p),
         ("softcap", C.c_float), ("alibi_slopes", C.c_void_p),
         ("dropout_p", C.c_float), ("dropout_seed", C.c_uint64), ("dropout_offset", C.c_uint64),
+        ("out_scale", C.c_float),
     ]
 
 
@@ -95,12 +97,12 @@ def lib():
                 f"{path} is missing: build it with `python -m nexus_b200._build` "
                 "(the sm_100a kernels are required on a GPU machine; there is no fallback)")
         _lib = C.CDLL(str(path))
-        _lib.nx_gemm_workspace_bytes.restype = C.c_size_t
-        _lib.nx_norm_bwd_scratch_bytes.restype = C.c_size_t
-        _lib.nx_ce_state_bytes.restype = C.c_size_t
-        _lib.nx_colsum_scratch_bytes.restype = C.c_size_t
-        _lib.nx_grad_norm_partials.restype = C.c_int64
-        _lib.nx_grad_norm_partials.argtypes = [C.c_int64]
+        for name in ("nx_gemm_workspace_bytes", "nx_norm_bwd_scratch_bytes", "nx_ce_state_bytes", "nx_colsum_scratch_bytes"):
+            if hasattr(_lib, name):       # the serving subset has no training kernels
+                getattr(_lib, name).restype = C.c_size_t
+        if hasattr(_lib, "nx_grad_norm_partials"):
+            _lib.nx_grad_norm_partials.restype = C.c_int64
+            _lib.nx_grad_norm_partials.argtypes = [C.c_int64]
     return _lib
 
 
@@ -143,11 +145,15 @@ def check_status(device=None) -> None:
 
 
 def scratch(nbytes: int, tag: str = "default", device=None) -> torch.Tensor:
-    """Grow-only per-(device, tag) scratch buffer (uint8)."""
+    """Grow-only per-(device, tag) scratch buffer (uint8).  A buffer that is outgrown stays allocated: a captured CUDA
+    graph may hold its address."""
     dev = torch.device("cuda", torch.cuda.current_device()) if device is None else torch.device(device)
     key = (dev, tag)
     t = _scratch.get(key)
     if t is None or t.numel() < nbytes:
+        if t is not None:
+            _outgrown.append(t)
+            nbytes = max(int(nbytes), 3 * t.numel() // 2)
         t = torch.empty(max(int(nbytes), 1 << 20), dtype=torch.uint8, device=dev)
         _scratch[key] = t
     return t
@@ -477,7 +483,8 @@ def _alibi_ptr(alibi_slopes, heads, device):
 
 
 def attention_fwd(q, k, v, *, causal=True, window=0, scale=None, out=None, merge_o=None, merge_lse=None,
-                  softcap=0.0, alibi_slopes=None, dropout_p=0.0, dropout_seed=0, dropout_offset=0, lse=None):
+                  softcap=0.0, alibi_slopes=None, dropout_p=0.0, dropout_seed=0, dropout_offset=0, lse=None,
+                  out_scale=1.0):
     """q [B,Tq,H,D], k/v [B,Tk,Hkv,D] bf16 (strided views allowed).  Returns (o, lse[B,H,Tq]).
     ``merge_o`` (FP32 [B,Tq,H,D]) / ``merge_lse`` (FP32 [B,H,Tq]): running result of earlier key/value
     chunks; this chunk is merged into them in the kernel's epilogue (ring / chunked attention)."""
@@ -495,6 +502,7 @@ def attention_fwd(q, k, v, *, causal=True, window=0, scale=None, out=None, merge
     a.scale = scale if scale is not None else D ** -0.5
     a.softcap, a.alibi_slopes = float(softcap), _alibi_ptr(alibi_slopes, H, q.device)
     a.dropout_p, a.dropout_seed, a.dropout_offset = float(dropout_p), int(dropout_seed), int(dropout_offset)
+    a.out_scale = float(out_scale)
     if merge_o is not None:
         if not (merge_o.is_contiguous() and merge_lse.is_contiguous() and merge_o.dtype == torch.float32):
             raise ValueError("attention_fwd: merge buffers must be contiguous FP32")

@@ -1,0 +1,194 @@
+"""ctypes bindings of the mixer kernels (``nx_api_mixers.h``): the residual / norm chain, rotary embedding with cache
+append, windowed soft-capped paged attention, the short causal convolution, the SSD and gated-delta recurrences, gated
+norms and the per-layer token input.  BF16 or FP32 activations; every wrapper launches on the current torch stream."""
+from __future__ import annotations
+
+import ctypes as C
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from . import _cuda as K
+
+CHUNK = 64       # tokens per chunk of the tensor-core recurrences
+
+
+class SegmentArgs(C.Structure):
+    _fields_ = [("row0", C.c_void_p), ("len", C.c_void_p), ("pos", C.c_void_p), ("seq", C.c_void_p),
+                ("count", C.c_int32), ("max_len", C.c_int32), ("total_len", C.c_int32)]
+
+
+class ResidualNormArgs(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("tokens", C.c_void_p), ("table", C.c_void_p), ("y", C.c_void_p), ("w_post", C.c_void_p),
+                ("w_next", C.c_void_p), ("h", C.c_void_p), ("x_cast", C.c_void_p), ("ldy", C.c_int64), ("ldh", C.c_int64),
+                ("rows", C.c_int32), ("cols", C.c_int32), ("dtype", C.c_int32), ("eps", C.c_float)]
+
+
+class RopeAppendArgs(C.Structure):
+    _fields_ = [("proj", C.c_void_p), ("ld", C.c_int64), ("q_off", C.c_int32), ("k_off", C.c_int32), ("v_off", C.c_int32),
+                ("rows", C.c_int32), ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32),
+                ("rot_dims", C.c_int32), ("dtype", C.c_int32), ("positions", C.c_void_p), ("slots", C.c_void_p),
+                ("cos_t", C.c_void_p), ("sin_t", C.c_void_p), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p)]
+
+
+class ConvArgs(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("y", C.c_void_p), ("w", C.c_void_p), ("bias", C.c_void_p), ("state", C.c_void_p),
+                ("ldx", C.c_int64), ("ldy", C.c_int64), ("channels", C.c_int32), ("taps", C.c_int32), ("dtype", C.c_int32),
+                ("seg", SegmentArgs)]
+
+
+class SsdArgs(C.Structure):
+    _fields_ = [("xbc", C.c_void_p), ("dt", C.c_void_p), ("y", C.c_void_p), ("dt_bias", C.c_void_p), ("a_log", C.c_void_p),
+                ("d_skip", C.c_void_p), ("state", C.c_void_p), ("ld_xbc", C.c_int64), ("ld_dt", C.c_int64), ("ldy", C.c_int64),
+                ("heads", C.c_int32), ("groups", C.c_int32), ("n_state", C.c_int32), ("vdim", C.c_int32), ("dtype", C.c_int32),
+                ("seg", SegmentArgs), ("part_state", C.c_void_p), ("part_decay", C.c_void_p), ("parts", C.c_int32),
+                ("span", C.c_int32)]
+
+
+class DeltaArgs(C.Structure):
+    _fields_ = [("qkv", C.c_void_p), ("b", C.c_void_p), ("a", C.c_void_p), ("o", C.c_void_p), ("dt_bias", C.c_void_p),
+                ("a_log", C.c_void_p), ("state", C.c_void_p), ("ld_qkv", C.c_int64), ("ld_ba", C.c_int64), ("ldo", C.c_int64),
+                ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("dtype", C.c_int32),
+                ("unit_eps", C.c_float), ("q_scale", C.c_float), ("seg", SegmentArgs)]
+
+
+class GatedNormArgs(C.Structure):
+    _fields_ = [("y", C.c_void_p), ("z", C.c_void_p), ("w", C.c_void_p), ("out", C.c_void_p), ("ldy", C.c_int64),
+                ("ldz", C.c_int64), ("ldo", C.c_int64), ("rows", C.c_int32), ("groups", C.c_int32), ("group_size", C.c_int32),
+                ("gate_first", C.c_int32), ("w_shared", C.c_int32), ("dtype", C.c_int32), ("eps", C.c_float),
+                ("out_scale", C.c_float)]
+
+
+class PagedWindowArgs(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p), ("block_table", C.c_void_p),
+                ("out", C.c_void_p), ("ldq", C.c_int64), ("ldo", C.c_int64), ("part_o", C.c_void_p), ("part_ml", C.c_void_p),
+                ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32),
+                ("block_size", C.c_int32), ("max_blocks", C.c_int32), ("window", C.c_int32), ("splits", C.c_int32),
+                ("dtype", C.c_int32), ("scale", C.c_float), ("softcap", C.c_float), ("out_scale", C.c_float),
+                ("seg", SegmentArgs)]
+
+
+@dataclass
+class Segments:
+    """A range of a device segment table ``[4, width]`` (first row, rows, first position, sequence)."""
+    table: torch.Tensor
+    first: int
+    count: int
+    max_len: int
+    total: int
+
+    def args(self) -> SegmentArgs:
+        t, step = self.table, self.table.stride(0) * 4
+        p = t.data_ptr() + self.first * 4
+        return SegmentArgs(p, p + step, p + 2 * step, p + 3 * step, self.count, self.max_len, self.total)
+
+
+def _dt(t: torch.Tensor) -> int:
+    return K._DT[t.dtype]
+
+
+def _ptr(t: Optional[torch.Tensor]):
+    return None if t is None else t.data_ptr()
+
+
+def residual_norm(x, *, y=None, w_post=None, w_next=None, h=None, x_cast=None, tokens=None, table=None, eps) -> None:
+    """x (FP32) = table[tokens], or x + rms(y) * w_post;  h = rms(x) * w_next;  x_cast = x in the activation dtype."""
+    lead = h if h is not None else x_cast
+    act = lead if lead is not None else (y if y is not None else table)
+    if h is not None and x_cast is not None and h.stride(0) != x_cast.stride(0):
+        raise ValueError("residual_norm: h and x_cast must share one row pitch")
+    a = ResidualNormArgs(_ptr(x), _ptr(tokens), _ptr(table), _ptr(y), _ptr(w_post), _ptr(w_next), _ptr(h), _ptr(x_cast),
+                         y.stride(0) if y is not None else 0, lead.stride(0) if lead is not None else x.shape[1], x.shape[0],
+                         x.shape[1], _dt(act), eps)
+    K._check(K.lib().nx_residual_norm(C.byref(a), K._stream()), "nx_residual_norm")
+
+
+def rope_append(proj, q_off, k_off, v_off, heads, kv_heads, dim, vdim, rot_dims, positions, slots, cos_t, sin_t, k_cache,
+                v_cache) -> None:
+    a = RopeAppendArgs(_ptr(proj), proj.stride(0), q_off, k_off, v_off, proj.shape[0], heads, kv_heads, dim, vdim, rot_dims,
+                       _dt(proj), _ptr(positions), _ptr(slots), _ptr(cos_t), _ptr(sin_t), _ptr(k_cache), _ptr(v_cache))
+    K._check(K.lib().nx_rope_append(C.byref(a), K._stream()), "nx_rope_append")
+
+
+def conv_silu(x, y, w, bias, state, seg: Segments) -> None:
+    """x / y: [rows, channels] views; w: FP32 [taps, channels]; state: [slots, taps - 1, channels]."""
+    a = ConvArgs(_ptr(x), _ptr(y), _ptr(w), _ptr(bias), _ptr(state), x.stride(0), y.stride(0), w.shape[1], w.shape[0], _dt(x),
+                 seg.args())
+    K._check(K.lib().nx_conv_silu(C.byref(a), K._stream()), "nx_conv_silu")
+
+
+def ssd(xbc, dt, y, dt_bias, a_log, d_skip, state, groups, seg: Segments, *, chunked=False, parts=1) -> None:
+    """state: FP32 [slots, heads, N, P].  ``chunked``: the tensor-core form; its segments are cut into ``parts`` spans
+    that run at the same time."""
+    _, H, N, P = state.shape
+    a = SsdArgs(_ptr(xbc), _ptr(dt), _ptr(y), _ptr(dt_bias), _ptr(a_log), _ptr(d_skip), _ptr(state), xbc.stride(0),
+                dt.stride(0), y.stride(0), H, groups, N, P, _dt(xbc), seg.args(), None, None, 1, 0)
+    if not chunked:
+        K._check(K.lib().nx_ssd_step(C.byref(a), K._stream()), "nx_ssd_step")
+        return
+    chunks = -(-seg.max_len // CHUNK)
+    per = -(-chunks // max(1, parts))
+    a.span, a.parts = per * CHUNK, -(-chunks // per)
+    if a.parts > 1:
+        a.part_state = K.scratch(seg.count * a.parts * H * N * P * 4, "ssd_state", xbc.device).data_ptr()
+        a.part_decay = K.scratch(seg.count * a.parts * H * 4, "ssd_decay", xbc.device).data_ptr()
+    K._check(K.lib().nx_ssd_chunk(C.byref(a), K._stream()), "nx_ssd_chunk")
+
+
+def delta(qkv, b, a, o, dt_bias, a_log, state, kv_heads, seg: Segments, *, unit_eps, q_scale, chunked=False) -> None:
+    """state: FP32 [slots, heads, D, Dv]."""
+    _, H, D, Dv = state.shape
+    if b.stride(0) != a.stride(0):
+        raise ValueError("delta: the gate projections must share one row pitch")
+    args = DeltaArgs(_ptr(qkv), _ptr(b), _ptr(a), _ptr(o), _ptr(dt_bias), _ptr(a_log), _ptr(state), qkv.stride(0), b.stride(0),
+                     o.stride(0), H, kv_heads, D, Dv, _dt(qkv), unit_eps, q_scale, seg.args())
+    fn = K.lib().nx_delta_chunk if chunked else K.lib().nx_delta_step
+    K._check(fn(C.byref(args), K._stream()), "nx_delta_chunk" if chunked else "nx_delta_step")
+
+
+def gated_norm(y, z, w, out, *, groups, gate_first, eps, out_scale=1.0) -> None:
+    """y, z, out: [rows, groups * size] views; w: FP32, one entry per column or [size] shared by the groups."""
+    size = y.shape[1] // groups
+    a = GatedNormArgs(_ptr(y), _ptr(z), _ptr(w), _ptr(out), y.stride(0), z.stride(0), out.stride(0), y.shape[0], groups, size,
+                      int(gate_first), int(groups > 1 and w.numel() == size), _dt(y), eps, out_scale)
+    K._check(K.lib().nx_gated_norm(C.byref(a), K._stream()), "nx_gated_norm")
+
+
+def token_side_gate(a, tokens, table, offset, out, dim) -> None:
+    K._check(K.lib().nx_token_side_gate(K._p(a), C.c_int64(a.stride(0)), K._p(tokens), K._p(table), C.c_int64(table.stride(0)),
+                                        C.c_int(offset), K._p(out), C.c_int64(out.stride(0)), C.c_int(a.shape[0]), C.c_int(dim),
+                                        C.c_int(_dt(a)), K._stream()), "nx_token_side_gate")
+
+
+def silu_mul(h, out) -> None:
+    """h: [rows, 2 F] = [gate | up]; out: [rows, F]."""
+    K._check(K.lib().nx_silu_mul(K._p(h), C.c_int64(h.stride(0)), K._p(out), C.c_int64(out.stride(0)), C.c_int(h.shape[0]),
+                                 C.c_int(h.shape[1] // 2), C.c_int(_dt(h)), K._stream()), "nx_silu_mul")
+
+
+def softcap_(x, cols, cap) -> None:
+    for r0 in range(0, x.shape[0], 32768):
+        part = x[r0: r0 + 32768]
+        K._check(K.lib().nx_softcap(K._p(part), C.c_int64(part.stride(0)), C.c_int(part.shape[0]), C.c_int(cols), C.c_float(cap),
+                                    K._stream()), "nx_softcap")
+
+
+def paged_window_attention(q, k_cache, v_cache, block_table, out, seg: Segments, *, heads, block_size, window, scale,
+                           softcap=0.0, out_scale=1.0, splits=1) -> None:
+    """q: [rows, heads * dim] view; caches [blocks, block_size, kv_heads, dim | vdim]; out [rows, heads * vdim] view.
+    One-row segments run the decode kernel, longer ones the prompt kernel (BF16); FP32 has one kernel for both."""
+    G, D, Dv = k_cache.shape[2], k_cache.shape[3], v_cache.shape[3]
+    a = PagedWindowArgs(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(out), q.stride(0), out.stride(0), None,
+                        None, heads, G, D, Dv, block_size, block_table.shape[1], window, 1, _dt(q), scale, softcap, out_scale,
+                        seg.args())
+    if q.dtype == torch.float32:
+        K._check(K.lib().nx_paged_window_f32(C.byref(a), K._stream()), "nx_paged_window_f32")
+    elif seg.max_len == 1:
+        a.splits = splits
+        if splits > 1:
+            a.part_o = K.scratch(seg.count * heads * splits * Dv * 4, "window_o", q.device).data_ptr()
+            a.part_ml = K.scratch(seg.count * heads * splits * 8, "window_ml", q.device).data_ptr()
+        K._check(K.lib().nx_paged_window_decode(C.byref(a), K._stream()), "nx_paged_window_decode")
+    else:
+        K._check(K.lib().nx_paged_window_prefill(C.byref(a), K._stream()), "nx_paged_window_prefill")
