@@ -106,8 +106,12 @@ typedef struct NxDeltaArgs {
   int32_t heads, kv_heads, dim, vdim, dtype;
   float unit_eps, q_scale;
   NxSegments seg;
+  void* scratch;           // chunked form: nx_delta_scratch_bytes
 } NxDeltaArgs;
+// token by token, any sizes and both dtypes
 int nx_delta_step(const NxDeltaArgs* args, nx_stream_t stream);
+// chunks of 64 tokens on the tensor cores, BF16 activations, dim <= 256
+int64_t nx_delta_scratch_bytes(int heads, int segments, int max_len);
 int nx_delta_chunk(const NxDeltaArgs* args, nx_stream_t stream);
 
 // gate_first: out = rms(y * silu(z)) * w * out_scale, else out = rms(y) * w * silu(z) * out_scale; statistics over each

@@ -51,6 +51,10 @@ class HybridEngine(Engine):
             torch.backends.cuda.matmul.allow_tf32 = False
         self.model: HybridConfig = weights.config
         self.L, self.d, self.V = len(self.model.layers), self.model.width, self.model.vocab
+        for i, layer in enumerate(self.model.layers):
+            m = layer.mixer
+            if self.fast and isinstance(m, ParallelSpec) and max(m.left.dim, m.left.vdim) > 256:
+                raise ValueError(f"layer {i}: the BF16 attention kernels take head sizes up to 256")
         self.adt = torch.bfloat16 if self.fast else torch.float32
         self.kv_kind = 0
         elem = 2 if self.fast else 4
@@ -58,7 +62,7 @@ class HybridEngine(Engine):
         self.n_blocks = self._pool_blocks(self._kv_tok_bytes)
         self.ctx = cfg.context if cfg.context > 0 else self.n_blocks * cfg.block_size
         self._rope: Dict[tuple, tuple] = {}
-        self._short_len = 1 << 30
+        self._short_len = 16 if self.fast else 1 << 30
 
     def _rope_tables(self, dims: int, base: float):
         """cos / sin [ctx, dims / 2]: angles in double, kept in FP32."""
@@ -198,6 +202,7 @@ class HybridEngine(Engine):
                                 short.total + long_.total)
         self._stepped = M.Segments(table, 0, single.count + short.count, max(single.max_len, short.max_len),
                                    single.total + short.total)
+        self._every = M.Segments(table, 0, first, max(g.max_len for g in groups), sum(g.total for g in groups))
         return self._body(dv[0], dv[1], dv[2], dv[3], dv[4], dv[5][:logit_rows], runs, nl)
 
     def _buffer(self, rows: int, cols: int) -> torch.Tensor:
@@ -222,9 +227,7 @@ class HybridEngine(Engine):
                   out_scale=out_scale)
         paged = (self.k_cache[i], self.v_cache[i], self.block_table, out)
         if not self.fast:
-            every = M.Segments(single.table, 0, single.count + short.count, max(single.max_len, short.max_len),
-                               single.total + short.total)
-            M.paged_window_attention(q, *paged, every, **kw)
+            M.paged_window_attention(q, *paged, self._every, **kw)
             return
         if single.count:
             M.paged_window_attention(q, *paged, single, splits=self._decode_splits(a, single.count), **kw)
@@ -248,7 +251,7 @@ class HybridEngine(Engine):
 
     def _conv(self, x, w, bias, tail) -> torch.Tensor:
         from ..ops import _mixers as M
-        y = torch.empty((x.shape[0], w.shape[1]), dtype=self.adt, device=self.dev)
+        y = torch.empty((x.shape[0], _pad8(w.shape[1])), dtype=self.adt, device=self.dev)[:, : w.shape[1]]
         for seg in (self._groups[0], self._many):
             if seg.count:
                 M.conv_silu(x, y, w, bias, tail, seg)
@@ -268,13 +271,21 @@ class HybridEngine(Engine):
         xbc = self._conv(proj[:, ox: ox + r.channels], lw["conv"], lw["conv_b"], self.conv_tail[i])
         y = torch.empty((n, nr), dtype=self.adt, device=self.dev)
         ssd = (xbc, proj[:, od: od + r.heads], y, lw["dt_bias"], lw["a_log"], lw["d_skip"], self.state[i], r.groups)
-        if self._stepped.count:
-            M.ssd(*ssd, self._stepped)
-        if self._groups[2].count:
-            M.ssd(*ssd, self._groups[2], chunked=True, parts=self._ssd_parts(r))
+        stepped, chunked = self._recurrence_groups(r.state)
+        if stepped.count:
+            M.ssd(*ssd, stepped)
+        if chunked is not None:
+            M.ssd(*ssd, chunked, chunked=True, parts=self._ssd_parts(r))
         M.gated_norm(y, proj[:, oz: oz + nr], lw["norm"], both[:, ka: ka + nr], groups=r.norm_groups, gate_first=True,
                      eps=self.model.norm_eps, out_scale=m.right_scale)
         return self._linear(both, lw["out"])
+
+    def _recurrence_groups(self, key_size: int):
+        """The segments that run token by token, and those that run in chunks (None: no such segments)."""
+        from ..ops import _mixers as M
+        if self._groups[2].count == 0 or key_size > M.CHUNK_MAX_KEY:
+            return self._every, None
+        return self._stepped, self._groups[2]
 
     def _ssd_parts(self, r) -> int:
         """Spans per long segment: enough (segment, head, span) blocks to fill the GPU, at least 4 chunks each."""
@@ -291,10 +302,11 @@ class HybridEngine(Engine):
         o = torch.empty((n, m.heads * m.vdim), dtype=self.adt, device=self.dev)
         args = (qkv, proj[:, ob: ob + m.heads], proj[:, oa: oa + m.heads], o, lw["dt_bias"], lw["a_log"], self.state[i], m.kv_heads)
         kw = dict(unit_eps=m.unit_eps, q_scale=m.dim ** -0.5)
-        if self._stepped.count:
-            M.delta(*args, self._stepped, **kw)
-        if self._groups[2].count:
-            M.delta(*args, self._groups[2], chunked=True, **kw)
+        stepped, chunked = self._recurrence_groups(m.dim)
+        if stepped.count:
+            M.delta(*args, stepped, **kw)
+        if chunked is not None:
+            M.delta(*args, chunked, chunked=True, **kw)
         out = self._buffer(n, m.heads * m.vdim)
         M.gated_norm(o, proj[:, og: og + m.heads * m.vdim], lw["norm"], out[:, : m.heads * m.vdim], groups=m.heads,
                      gate_first=False, eps=self.model.norm_eps)

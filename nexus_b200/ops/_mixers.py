@@ -11,7 +11,8 @@ import torch
 
 from . import _cuda as K
 
-CHUNK = 64       # tokens per chunk of the tensor-core recurrences
+CHUNK = 64            # tokens per chunk of the tensor-core recurrences
+CHUNK_MAX_KEY = 256   # their largest state size along the key dimension
 
 
 class SegmentArgs(C.Structure):
@@ -50,7 +51,7 @@ class DeltaArgs(C.Structure):
     _fields_ = [("qkv", C.c_void_p), ("b", C.c_void_p), ("a", C.c_void_p), ("o", C.c_void_p), ("dt_bias", C.c_void_p),
                 ("a_log", C.c_void_p), ("state", C.c_void_p), ("ld_qkv", C.c_int64), ("ld_ba", C.c_int64), ("ldo", C.c_int64),
                 ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("dtype", C.c_int32),
-                ("unit_eps", C.c_float), ("q_scale", C.c_float), ("seg", SegmentArgs)]
+                ("unit_eps", C.c_float), ("q_scale", C.c_float), ("seg", SegmentArgs), ("scratch", C.c_void_p)]
 
 
 class GatedNormArgs(C.Structure):
@@ -142,7 +143,11 @@ def delta(qkv, b, a, o, dt_bias, a_log, state, kv_heads, seg: Segments, *, unit_
     if b.stride(0) != a.stride(0):
         raise ValueError("delta: the gate projections must share one row pitch")
     args = DeltaArgs(_ptr(qkv), _ptr(b), _ptr(a), _ptr(o), _ptr(dt_bias), _ptr(a_log), _ptr(state), qkv.stride(0), b.stride(0),
-                     o.stride(0), H, kv_heads, D, Dv, _dt(qkv), unit_eps, q_scale, seg.args())
+                     o.stride(0), H, kv_heads, D, Dv, _dt(qkv), unit_eps, q_scale, seg.args(), None)
+    if chunked:
+        size = K.lib().nx_delta_scratch_bytes
+        size.restype = C.c_int64
+        args.scratch = K.scratch(size(C.c_int(H), C.c_int(seg.count), C.c_int(seg.max_len)), "delta", qkv.device).data_ptr()
     fn = K.lib().nx_delta_chunk if chunked else K.lib().nx_delta_step
     K._check(fn(C.byref(args), K._stream()), "nx_delta_chunk" if chunked else "nx_delta_step")
 
