@@ -236,14 +236,14 @@ __global__ void gated_norm_kernel(const NxGatedNormArgs a) {
 // elementwise
 // ------------------------------------------------------------------------------------------------
 template <typename T>
-__global__ void token_side_kernel(const T* __restrict__ a, int64_t lda, const int32_t* __restrict__ tokens,
+__global__ void token_side_kernel(const float* __restrict__ a, int64_t lda, const int32_t* __restrict__ tokens,
                                   const T* __restrict__ table, int64_t ld_table, int offset, T* __restrict__ out,
                                   int64_t ldo, int dim) {
   const int64_t r = blockIdx.x;
   const T* e = table + static_cast<int64_t>(tokens[r]) * ld_table + offset;
   for (int j = threadIdx.x; j < ldo; j += blockDim.x) {
     float v = 0.0f;
-    if (j < dim) v = gelu_tanh_exact(Num<T>::load(a + r * lda + j)) * Num<T>::load(e + j);
+    if (j < dim) v = gelu_tanh_exact(a[r * lda + j]) * Num<T>::load(e + j);
     Num<T>::store(out + r * ldo + j, v);
   }
 }
@@ -358,17 +358,17 @@ extern "C" int nx_gated_norm(const NxGatedNormArgs* a, nx_stream_t stream) {
   return launch_status();
 }
 
-extern "C" int nx_token_side_gate(const void* a, int64_t lda, const int32_t* tokens, const void* table, int64_t ld_table,
+extern "C" int nx_token_side_gate(const float* a, int64_t lda, const int32_t* tokens, const void* table, int64_t ld_table,
                                   int offset, void* out, int64_t ldo, int rows, int dim, int dtype, nx_stream_t stream) {
   if (dim <= 0 || ldo < dim) return -1;
   if (rows <= 0) return 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int threads = std::max(32, std::min(256, static_cast<int>((ldo + 31) / 32 * 32)));
   if (dtype == NX_BF16)
-    token_side_kernel<__nv_bfloat16><<<rows, threads, 0, st>>>((const __nv_bfloat16*)a, lda, tokens, (const __nv_bfloat16*)table,
+    token_side_kernel<__nv_bfloat16><<<rows, threads, 0, st>>>(a, lda, tokens, (const __nv_bfloat16*)table,
                                                                ld_table, offset, (__nv_bfloat16*)out, ldo, dim);
   else if (dtype == NX_F32)
-    token_side_kernel<float><<<rows, threads, 0, st>>>((const float*)a, lda, tokens, (const float*)table, ld_table, offset,
+    token_side_kernel<float><<<rows, threads, 0, st>>>(a, lda, tokens, (const float*)table, ld_table, offset,
                                                        (float*)out, ldo, dim);
   else
     return -1;

@@ -127,8 +127,9 @@ typedef struct NxGatedNormArgs {
 } NxGatedNormArgs;
 int nx_gated_norm(const NxGatedNormArgs* args, nx_stream_t stream);
 
-// out[r][j] = gelu_tanh(a[r][j]) * table[tokens[r]][offset + j], j < dim; columns dim..ldo are zeroed
-int nx_token_side_gate(const void* a, int64_t lda, const int32_t* tokens, const void* table, int64_t ld_table, int offset,
+// out[r][j] = gelu_tanh(a[r][j]) * table[tokens[r]][offset + j], j < dim; columns dim..ldo are zeroed.  `a` is FP32: far
+// out on the negative side the relative slope of GELU is its argument, so a rounded argument would show in the product.
+int nx_token_side_gate(const float* a, int64_t lda, const int32_t* tokens, const void* table, int64_t ld_table, int offset,
                        void* out, int64_t ldo, int rows, int dim, int dtype, nx_stream_t stream);
 // out[r][j] = silu(h[r][j]) * h[r][half + j], j < half
 int nx_silu_mul(const void* h, int64_t ldh, void* out, int64_t ldo, int rows, int half, int dtype, nx_stream_t stream);

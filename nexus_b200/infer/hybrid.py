@@ -329,8 +329,8 @@ class HybridEngine(Engine):
                 M.silu_mul(gu, act)
                 y, post = self._linear(act, lw["down"]), lw["norm2b"]
             M.residual_norm(x, y=y, w_post=post, x_cast=h, eps=eps)
-            gate = self._linear(h, lw["side_gate"])
-            side = torch.empty_like(gate)
+            gate = self._linear(h, lw["side_gate"], out_dtype=torch.float32)
+            side = torch.empty(gate.shape, dtype=self.adt, device=self.dev)
             M.token_side_gate(gate, tok, self.side_embed, i * model.token_side, side, model.token_side)
             y = self._linear(side, lw["side_proj"])
             last = i + 1 == self.L

@@ -161,9 +161,12 @@ def gated_norm(y, z, w, out, *, groups, gate_first, eps, out_scale=1.0) -> None:
 
 
 def token_side_gate(a, tokens, table, offset, out, dim) -> None:
+    """a: FP32 [rows, >= dim]; table and out in the activation dtype."""
+    if a.dtype != torch.float32:
+        raise ValueError("token_side_gate: the gate is FP32")
     K._check(K.lib().nx_token_side_gate(K._p(a), C.c_int64(a.stride(0)), K._p(tokens), K._p(table), C.c_int64(table.stride(0)),
                                         C.c_int(offset), K._p(out), C.c_int64(out.stride(0)), C.c_int(a.shape[0]), C.c_int(dim),
-                                        C.c_int(_dt(a)), K._stream()), "nx_token_side_gate")
+                                        C.c_int(_dt(out)), K._stream()), "nx_token_side_gate")
 
 
 def silu_mul(h, out) -> None:

@@ -257,7 +257,7 @@ def test_gated_norm(dt, tol, groups, size):
 def test_token_side_silu_mul_softcap(dt, tol):
     M = _m()
     n, dim = 6, 20
-    a, table = _rand((n, 24), 1, dt, 2.0), _rand((9, 3 * dim), 2, dt)
+    a, table = _rand((n, 24), 1, s=2.0), _rand((9, 3 * dim), 2, dt)
     tok = torch.tensor([8, 0, 3, 3, 1, 5], dtype=torch.int32)
     out = torch.full((n, 24), 5.0, dtype=dt, device=DEV)
     M.token_side_gate(a.to(DEV), tok.to(DEV), table.to(DEV), 2 * dim, out, dim)
