@@ -180,7 +180,16 @@ __device__ __forceinline__ void row_limits(const AttnDev& p, int q, int& lo, int
 
 // Forward softmax helpers.  A score row (128 keys) is shared by two threads of different warps: `c0` is
 // the first of the 64 columns this thread owns (0 or 64).
-template <bool kMask, bool kExt>
+// 1 / (1 + e^{2z}) for the soft cap: cap * tanh(z) = cap - 2 cap * this;  mul * s = 2 z log2(e)
+__device__ __forceinline__ float cap_rcp(float s, float mul) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(1.0f + ex2f(mul * s)));
+  return y;
+}
+
+// kMode: 0 plain scores, 1 general (soft-capping, ALiBi, dropout), 2 soft-capping alone.  In mode 2 the cap is monotone, so
+// the maximum is taken over the raw scores and mapped once per row, and the softmax pass folds the cap into its exponent.
+template <bool kMask, int kMode>
 __device__ __forceinline__ float half_row_max(uint32_t taddr, int c0, int k0, int lo, int hi, const ScoreExt& ext,
                                               int qpos) {
   float m0 = -INFINITY, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;
@@ -194,7 +203,7 @@ __device__ __forceinline__ float half_row_max(uint32_t taddr, int c0, int k0, in
     for (int c = 0; c < 32; c += 4) {
       float s0 = __uint_as_float(v[c]), s1 = __uint_as_float(v[c + 1]), s2 = __uint_as_float(v[c + 2]),
             s3 = __uint_as_float(v[c + 3]);
-      if (kExt) {
+      if (kMode == 1) {
         const int rel = k0 + c0 + cc * 32 + c - qpos;
         s0 = score_ext(ext, s0, rel);
         s1 = score_ext(ext, s1, rel + 1);
@@ -217,10 +226,11 @@ __device__ __forceinline__ float half_row_max(uint32_t taddr, int c0, int k0, in
 }
 
 // P = exp2(S*sc - m) for this thread's 64 keys -> BF16 into slab `c0 / 64` of the swizzled [128][128] tile.
-template <bool kMask, bool kExt>
+template <bool kMask, int kMode>
 __device__ __forceinline__ float half_softmax_store(uint32_t taddr, uint8_t* sP, int r, int c0, int k0, int lo, int hi,
                                                     float sc, float m_use, const ScoreExt& ext, int qpos, int qoff) {
   float r0 = 0.0f, r1 = 0.0f, r2 = 0.0f, r3 = 0.0f;
+  const float cap = ext.cap * kLog2e, cap2 = 2.0f * cap, mul = 2.0f * sc * ext.inv_cap;
   uint8_t* slab = sP + (c0 >> 6) * (128 * 128);
 #pragma unroll
   for (int cc = 0; cc < 2; ++cc) {
@@ -235,8 +245,8 @@ __device__ __forceinline__ float half_softmax_store(uint32_t taddr, uint8_t* sP,
       for (int j = 0; j < 8; ++j) {
         const int c = 8 * g + j;
         float sv = __uint_as_float(v[c]);
-        if (kExt) sv = score_ext(ext, sv, k0 + c0 + cc * 32 + c - qpos);
-        float x = ex2f(fmaf(sv, sc, -m_use));
+        if (kMode == 1) sv = score_ext(ext, sv, k0 + c0 + cc * 32 + c - qpos);
+        float x = kMode == 2 ? ex2f(fmaf(-cap2, cap_rcp(sv, mul), cap - m_use)) : ex2f(fmaf(sv, sc, -m_use));
         if (kMask && (c < clo || c > chi)) x = 0.0f;
         e[j] = x;
       }
@@ -244,7 +254,7 @@ __device__ __forceinline__ float half_softmax_store(uint32_t taddr, uint8_t* sP,
       r1 += e[1] + e[5];
       r2 += e[2] + e[6];
       r3 += e[3] + e[7];
-      if (kExt && ext.drop_p > 0.0f) {  // the row sum keeps every probability; the tile that meets V does not
+      if (kMode == 1 && ext.drop_p > 0.0f) {  // the row sum keeps every probability; the tile that meets V does not
 #pragma unroll
         for (int j = 0; j < 8; ++j) e[j] *= drop_scale_qk(ext, qpos - qoff, k0 + c0 + cc * 32 + 8 * g + j);
       }
@@ -299,7 +309,7 @@ __device__ __forceinline__ void fwd_item(const AttnDev& p, int item, int& qb, in
   b = rem / p.H;
 }
 
-template <int HD, bool EXT>  // EXT: soft-capping / ALiBi / dropout row math (a build of its own)
+template <int HD, int EXT>  // row math: 0 plain, 1 soft-capping / ALiBi / dropout, 2 soft-capping alone (builds of their own)
 __global__ void __launch_bounds__(kFwdThreads, (HD == 64 ? 2 : 1))
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                 const __grid_constant__ CUtensorMap tm_v, const AttnDev p) {
@@ -471,8 +481,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
       float m_run = -INFINITY, l_run = 0.0f;  // l_run: partial sum over this thread's columns
       int row_lo, row_hi;
       row_limits(p, q, row_lo, row_hi);
-      constexpr bool ext_on = EXT;
-      const ScoreExt ext = EXT ? make_ext(p, h, b) : ScoreExt{};
+      const ScoreExt ext = EXT != 0 ? make_ext(p, h, b) : ScoreExt{};
       float o_acc[HH];
 #pragma unroll
       for (int c = 0; c < HH; ++c) o_acc[c] = 0.0f;
@@ -490,13 +499,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
                                (p.window > 0 && (k0 < q0 + 127 + off - p.window + 1));
         float mx, rs;
         const int qpos = q + off;
-        if (ext_on) {
-          if (need_mask) mx = half_row_max<true, true>(tmem_s + lane_addr, c0, k0, row_lo, row_hi, ext, qpos);
-          else mx = half_row_max<false, true>(tmem_s + lane_addr, c0, k0, row_lo, row_hi, ext, qpos);
-        } else {
-          if (need_mask) mx = half_row_max<true, false>(tmem_s + lane_addr, c0, k0, row_lo, row_hi, ext, qpos);
-          else mx = half_row_max<false, false>(tmem_s + lane_addr, c0, k0, row_lo, row_hi, ext, qpos);
-        }
+        if (need_mask) mx = half_row_max<true, EXT>(tmem_s + lane_addr, c0, k0, row_lo, row_hi, ext, qpos);
+        else mx = half_row_max<false, EXT>(tmem_s + lane_addr, c0, k0, row_lo, row_hi, ext, qpos);
         // second half publishes, first half combines and publishes the row maximum
         if (half == 1) sX[r] = mx;
         softmax_bar();
@@ -506,16 +510,13 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant_
         }
         softmax_bar();
         if (half == 1) mx = sX[r];
-        const float m_new = fmaxf(m_run, mx * sc);
+        float mx_log2 = mx * sc;
+        if (EXT == 2 && mx != -INFINITY) mx_log2 = ext.cap * kLog2e * (1.0f - 2.0f * cap_rcp(mx, 2.0f * sc * ext.inv_cap));
+        const float m_new = fmaxf(m_run, mx_log2);
         const float m_use = (m_new == -INFINITY) ? 0.0f : m_new;
         const float alpha = ex2f(m_run - m_use);  // m_run == -inf -> 0
-        if (ext_on) {
-          if (need_mask) rs = half_softmax_store<true, true>(tmem_s + lane_addr, sP, r, c0, k0, row_lo, row_hi, sc, m_use, ext, qpos, off);
-          else rs = half_softmax_store<false, true>(tmem_s + lane_addr, sP, r, c0, k0, row_lo, row_hi, sc, m_use, ext, qpos, off);
-        } else {
-          if (need_mask) rs = half_softmax_store<true, false>(tmem_s + lane_addr, sP, r, c0, k0, row_lo, row_hi, sc, m_use, ext, qpos, off);
-          else rs = half_softmax_store<false, false>(tmem_s + lane_addr, sP, r, c0, k0, row_lo, row_hi, sc, m_use, ext, qpos, off);
-        }
+        if (need_mask) rs = half_softmax_store<true, EXT>(tmem_s + lane_addr, sP, r, c0, k0, row_lo, row_hi, sc, m_use, ext, qpos, off);
+        else rs = half_softmax_store<false, EXT>(tmem_s + lane_addr, sP, r, c0, k0, row_lo, row_hi, sc, m_use, ext, qpos, off);
         l_run = l_run * alpha + rs;
         m_run = m_new;
         fence_proxy_async_smem();  // generic-proxy writes of P -> visible to the tensor core's async proxy
@@ -1787,12 +1788,15 @@ extern "C" int nx_attention_fwd(const NxAttnArgs* a, nx_stream_t stream_) {
     }                                                                                               \
     attn_fwd_kernel<HD_, EXT_><<<grid, kFwdThreads, FwdCfg<HD_>::kSmem, st>>>(tq, tk, tv, p);       \
   } while (0)
+  const int mode = !ext ? 0 : (p.alibi == nullptr && p.dropout_p <= 0.0f && p.scale > 0.0f ? 2 : 1);
   if (HD == 64) {
-    if (ext) NX_FWD(64, true);
-    else NX_FWD(64, false);
+    if (mode == 2) NX_FWD(64, 2);
+    else if (mode == 1) NX_FWD(64, 1);
+    else NX_FWD(64, 0);
   } else {
-    if (ext) NX_FWD(128, true);
-    else NX_FWD(128, false);
+    if (mode == 2) NX_FWD(128, 2);
+    else if (mode == 1) NX_FWD(128, 1);
+    else NX_FWD(128, 0);
   }
 #undef NX_FWD
   return cudaGetLastError() == cudaSuccess ? 0 : -2;

@@ -171,18 +171,18 @@ __global__ void conv_silu_kernel(const NxConvArgs a) {
       const int t = len - (TAPS - 1) + j;
       if (t >= 0) {
         load_vec<T, V>(x + static_cast<int64_t>(t) * a.ldx, tail[j]);
-      } else {                             // a segment shorter than the tail keeps the newest of the old inputs
+      } else if (carried) {                // a segment shorter than the tail keeps the newest of the old inputs
+        load_vec<T, V>(st + static_cast<int64_t>(TAPS - 1 + t) * a.channels, tail[j]);
+      } else {
 #pragma unroll
-        for (int i = 0; i < TAPS - 1; ++i)
-          if (i == TAPS - 1 + t)
-#pragma unroll
-            for (int v = 0; v < V; ++v) tail[j][v] = hist[i][v];
+        for (int v = 0; v < V; ++v) tail[j][v] = 0.0f;
       }
     }
 #pragma unroll
     for (int j = 0; j < TAPS - 1; ++j) store_vec<T, V>(st + static_cast<int64_t>(j) * a.channels, tail[j]);
   }
   const int t1 = min(len, t0 + kConvTile);
+#pragma unroll 4
   for (int t = t0; t < t1; ++t) {
     float cur[V], acc[V];
     load_vec<T, V>(x + static_cast<int64_t>(t) * a.ldx, cur);
@@ -193,7 +193,7 @@ __global__ void conv_silu_kernel(const NxConvArgs a) {
 #pragma unroll
       for (int v = 0; v < V; ++v) acc[v] += w[j][v] * hist[j][v];
 #pragma unroll
-    for (int v = 0; v < V; ++v) acc[v] = silu_exact(acc[v]);
+    for (int v = 0; v < V; ++v) acc[v] = sizeof(T) == 4 ? silu_exact(acc[v]) : acc[v] * __fdividef(1.0f, 1.0f + __expf(-acc[v]));
     store_vec<T, V>(y + static_cast<int64_t>(t) * a.ldy, acc);
 #pragma unroll
     for (int j = 0; j < TAPS - 1; ++j)
@@ -232,14 +232,61 @@ __global__ void gated_norm_kernel(const NxGatedNormArgs a) {
     Num<T>::store(o + c, Num<T>::load(y + c) * silu_exact(Num<T>::load(z + c)) * inv * w[c]);
 }
 
+// the same with vector accesses and the gated values kept in registers: groups of up to 16 values per thread
+template <typename T, int V, bool kWarp>
+__global__ void gated_norm_vec_kernel(const NxGatedNormArgs a) {
+  constexpr int kIter = 16 / V;
+  __shared__ float s_red[32];
+  const int lanes = kWarp ? 32 : blockDim.x;
+  const int64_t item = kWarp ? blockIdx.x * static_cast<int64_t>(blockDim.x >> 5) + (threadIdx.x >> 5) : blockIdx.x;
+  if (item >= static_cast<int64_t>(a.rows) * a.groups) return;
+  const int lane = kWarp ? threadIdx.x & 31 : threadIdx.x;
+  const int64_t r = item / a.groups;
+  const int g = static_cast<int>(item % a.groups), n = a.group_size;
+  const T* y = static_cast<const T*>(a.y) + r * a.ldy + static_cast<int64_t>(g) * n;
+  const T* z = static_cast<const T*>(a.z) + r * a.ldz + static_cast<int64_t>(g) * n;
+  T* o = static_cast<T*>(a.out) + r * a.ldo + static_cast<int64_t>(g) * n;
+  const float* w = a.w + (a.w_shared ? 0 : static_cast<int64_t>(g) * n);
+  float v[kIter][V], ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < kIter; ++i) {
+    const int c = (lane + i * lanes) * V;
+    if (c < n) {
+      float zv[V];
+      load_vec<T, V>(y + c, v[i]);
+      load_vec<T, V>(z + c, zv);
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        const float gate = zv[j] * __fdividef(1.0f, 1.0f + __expf(-zv[j])), u = v[i][j] * gate;
+        ss += a.gate_first ? u * u : v[i][j] * v[i][j];
+        v[i][j] = u;
+      }
+    }
+  }
+  ss = kWarp ? warp_sum(ss) : block_sum(ss, s_red);
+  const float inv = a.out_scale / sqrtf(ss / static_cast<float>(n) + a.eps);
+#pragma unroll
+  for (int i = 0; i < kIter; ++i) {
+    const int c = (lane + i * lanes) * V;
+    if (c < n) {
+      float wv[V];
+      load_vec<float, V>(w + c, wv);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[i][j] *= inv * wv[j];
+      store_vec<T, V>(o + c, v[i]);
+    }
+  }
+}
+
 // ------------------------------------------------------------------------------------------------
 // elementwise
 // ------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void token_side_kernel(const float* __restrict__ a, int64_t lda, const int32_t* __restrict__ tokens,
                                   const T* __restrict__ table, int64_t ld_table, int offset, T* __restrict__ out,
-                                  int64_t ldo, int dim) {
-  const int64_t r = blockIdx.x;
+                                  int64_t ldo, int dim, int rows) {
+  const int64_t r = blockIdx.x * static_cast<int64_t>(blockDim.y) + threadIdx.y;
+  if (r >= rows) return;
   const T* e = table + static_cast<int64_t>(tokens[r]) * ld_table + offset;
   for (int j = threadIdx.x; j < ldo; j += blockDim.x) {
     float v = 0.0f;
@@ -257,7 +304,7 @@ __global__ void silu_mul_kernel(const T* __restrict__ h, int64_t ldh, T* __restr
   load_vec<T, V>(h + r * ldh + c, g);
   load_vec<T, V>(h + r * ldh + half + c, u);
 #pragma unroll
-  for (int j = 0; j < V; ++j) g[j] = silu_exact(g[j]) * u[j];
+  for (int j = 0; j < V; ++j) g[j] = (sizeof(T) == 4 ? silu_exact(g[j]) : g[j] * __fdividef(1.0f, 1.0f + __expf(-g[j]))) * u[j];
   store_vec<T, V>(out + r * ldo + c, g);
 }
 
@@ -334,6 +381,9 @@ extern "C" int nx_conv_silu(const NxConvArgs* a, nx_stream_t stream) {
   if (a->seg.count > 65535 || (a->seg.max_len + kConvTile - 1) / kConvTile > 65535) return -1;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const bool v2 = a->channels % 2 == 0 && a->ldx % 2 == 0 && a->ldy % 2 == 0 && (reinterpret_cast<uintptr_t>(a->x) & 7) == 0;
+  const bool v4 = a->channels % 4 == 0 && a->ldx % 4 == 0 && a->ldy % 4 == 0 && (reinterpret_cast<uintptr_t>(a->x) & 7) == 0 &&
+                  (reinterpret_cast<uintptr_t>(a->y) & 7) == 0 && a->taps <= 4;
+  if (a->dtype == NX_BF16 && v4) return launch_conv<__nv_bfloat16, 4>(a, st);
   if (a->dtype == NX_BF16) return v2 ? launch_conv<__nv_bfloat16, 2>(a, st) : launch_conv<__nv_bfloat16, 1>(a, st);
   if (a->dtype == NX_F32) return v2 ? launch_conv<float, 2>(a, st) : launch_conv<float, 1>(a, st);
   return -1;
@@ -346,6 +396,17 @@ extern "C" int nx_gated_norm(const NxGatedNormArgs* a, nx_stream_t stream) {
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int64_t items = static_cast<int64_t>(a->rows) * a->groups;
   if (items > 0x7fffffff) return -1;
+  const auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  if (a->dtype == NX_BF16 && a->group_size % 8 == 0 && a->ldy % 8 == 0 && a->ldz % 8 == 0 && a->ldo % 8 == 0 && al(a->y) && al(a->z) &&
+      al(a->out) && al(a->w) && a->group_size <= 16384) {
+    if (a->group_size <= 512) {
+      gated_norm_vec_kernel<__nv_bfloat16, 8, true><<<static_cast<int>((items + 7) / 8), 256, 0, st>>>(*a);
+    } else {
+      const int threads = std::max(64, (a->group_size / 16 + 31) / 32 * 32);
+      gated_norm_vec_kernel<__nv_bfloat16, 8, false><<<static_cast<int>(items), threads, 0, st>>>(*a);
+    }
+    return launch_status();
+  }
   if (a->group_size <= kGatedWarpCols) {
     const int blocks = static_cast<int>((items + 7) / 8);
     if (a->dtype == NX_BF16) gated_norm_kernel<__nv_bfloat16, true><<<blocks, 256, 0, st>>>(*a);
@@ -363,13 +424,15 @@ extern "C" int nx_token_side_gate(const float* a, int64_t lda, const int32_t* to
   if (dim <= 0 || ldo < dim) return -1;
   if (rows <= 0) return 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const int threads = std::max(32, std::min(256, static_cast<int>((ldo + 31) / 32 * 32)));
+  const int tx = std::max(32, std::min(128, static_cast<int>((ldo + 31) / 32 * 32))), ty = rows >= 1024 ? 512 / tx : 1;
+  const dim3 threads(tx, ty);
+  const int blocks = (rows + ty - 1) / ty;
   if (dtype == NX_BF16)
-    token_side_kernel<__nv_bfloat16><<<rows, threads, 0, st>>>(a, lda, tokens, (const __nv_bfloat16*)table,
-                                                               ld_table, offset, (__nv_bfloat16*)out, ldo, dim);
+    token_side_kernel<__nv_bfloat16><<<blocks, threads, 0, st>>>(a, lda, tokens, (const __nv_bfloat16*)table,
+                                                               ld_table, offset, (__nv_bfloat16*)out, ldo, dim, rows);
   else if (dtype == NX_F32)
-    token_side_kernel<float><<<rows, threads, 0, st>>>(a, lda, tokens, (const float*)table, ld_table, offset,
-                                                       (float*)out, ldo, dim);
+    token_side_kernel<float><<<blocks, threads, 0, st>>>(a, lda, tokens, (const float*)table, ld_table, offset,
+                                                       (float*)out, ldo, dim, rows);
   else
     return -1;
   return launch_status();

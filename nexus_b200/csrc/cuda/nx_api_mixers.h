@@ -153,7 +153,7 @@ typedef struct NxPagedWindowArgs {
 } NxPagedWindowArgs;
 // one-row segments, BF16: tensor-core tiles of up to 16 query heads of a KV head against 64 keys, split over the keys
 int nx_paged_window_decode(const NxPagedWindowArgs* args, nx_stream_t stream);
-// longer segments, BF16: 64 (row, head) pairs of one KV head against tiles of 64 keys
+// longer segments, BF16: 128 (row, head) pairs of one KV head against tiles of 64 keys
 int nx_paged_window_prefill(const NxPagedWindowArgs* args, nx_stream_t stream);
 // any segments, FP32
 int nx_paged_window_f32(const NxPagedWindowArgs* args, nx_stream_t stream);

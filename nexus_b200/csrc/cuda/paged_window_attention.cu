@@ -11,14 +11,30 @@ namespace {
 using namespace nx;
 
 constexpr int kKeys = 64;              // keys per shared-memory stage
+constexpr int kRows = 128;             // (token, head) rows per block in prompts
 constexpr float kLog2e = 1.4426950408889634f;
 
-// scaled, soft-capped score in units of log2
-__device__ __forceinline__ float score_log2(float s, float scale, float cap, float inv_cap) {
-  s *= scale;
-  if (cap > 0.0f) s = cap * (1.0f - __fdividef(2.0f, 1.0f + exp2f(2.0f * kLog2e * s * inv_cap)));
-  return s * kLog2e;
-}
+// Scores in units of log2.  Soft-capping goes through one exponential: cap tanh(z) = cap - 2 cap / (1 + e^{2z}).  It is
+// monotone, so row maxima are taken over the raw products and only the maximum is mapped.
+struct ScoreMap {
+  bool capped;
+  float mul, cap2, cap;      // capped: x -> cap - cap2 / (1 + 2^(mul x)); else x -> mul x
+  __device__ __forceinline__ ScoreMap(float scale, float softcap) {
+    capped = softcap > 0.0f;
+    mul = capped ? 2.0f * kLog2e * scale / softcap : scale * kLog2e;
+    cap = softcap * kLog2e;
+    cap2 = 2.0f * cap;
+  }
+  __device__ __forceinline__ float operator()(float x) const {       // -inf (nothing visible) stays -inf
+    if (!capped || x == -INFINITY) return mul * x;
+    return cap - cap2 * rcp_approx(1.0f + ex2_approx(mul * x));
+  }
+  // 2^(mapped x - base)
+  __device__ __forceinline__ float prob(float x, float base) const {
+    if (!capped) return ex2_approx(fmaf(mul, x, -base));
+    return ex2_approx(fmaf(-cap2, rcp_approx(1.0f + ex2_approx(mul * x)), cap - base));
+  }
+};
 
 // which segment, and which tile of `per` tokens inside it, flat tile index `tile` is; executed by one full warp
 __device__ __forceinline__ bool find_tile(const NxSegments& s, int per, int tile, int& seg, int& off) {
@@ -45,40 +61,56 @@ __device__ __forceinline__ bool find_tile(const NxSegments& s, int per, int tile
   return false;
 }
 
-// rows of a K or V page range into shared memory [kKeys][DP + 8]; keys past `last` and columns past D become zeros
+// One stage of keys and values into shared memory, each [kKeys][DP + 8]; keys past `last` and columns past the head size
+// become zeros.
+__device__ __forceinline__ int log2_of(int n) { return (n & (n - 1)) == 0 ? 31 - __clz(n) : -1; }
+struct KvSource {
+  const __nv_bfloat16 *k, *v;
+  const int32_t* bt;
+  int block_size, shift, kv_heads, hk, dim, vdim;      // shift: log2 of a power-of-two block size, else -1
+  __device__ __forceinline__ KvSource(const NxPagedWindowArgs& a, int seq, int head)
+      : k(static_cast<const __nv_bfloat16*>(a.k_cache)), v(static_cast<const __nv_bfloat16*>(a.v_cache)),
+        bt(a.block_table + static_cast<int64_t>(seq) * a.max_blocks), block_size(a.block_size),
+        shift(log2_of(a.block_size)), kv_heads(a.kv_heads), hk(head), dim(a.dim),
+        vdim(a.vdim) {}
+  __device__ __forceinline__ int64_t slot(int j) const {
+    if (shift >= 0) return (static_cast<int64_t>(bt[j >> shift]) << shift) + (j & (block_size - 1));
+    return static_cast<int64_t>(bt[j / block_size]) * block_size + j % block_size;
+  }
+};
+__device__ __forceinline__ void copy8(__nv_bfloat16* d, const __nv_bfloat16* s, int c, int cols) {   // columns c .. c + 7 of a row
+  if ((cols & 7) == 0) {
+    cp_async16(d, s + c);
+  } else {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) d[e] = c + e < cols ? s[c + e] : __float2bfloat16_rn(0.0f);
+  }
+}
 template <int DP>
-__device__ __forceinline__ void stage_rows(__nv_bfloat16* dst, const __nv_bfloat16* cache, const int32_t* bt, int block_size,
-                                           int kv_heads, int hk, int D, int k0, int last) {
-  constexpr int CH = DP / 8;
-  const bool vec = (D & 7) == 0;
+__device__ __forceinline__ void stage_kv(__nv_bfloat16* dst, const KvSource& src, int k0, int last) {
+  constexpr int CH = DP / 8, LD = DP + 8;
   for (int i = threadIdx.x; i < kKeys * CH; i += blockDim.x) {
     const int key = i / CH, c = (i % CH) * 8, j = k0 + key;
-    __nv_bfloat16* d = dst + key * (DP + 8) + c;
-    if (j <= last && c < D) {
-      const int64_t slot = static_cast<int64_t>(bt[j / block_size]) * block_size + j % block_size;
-      const __nv_bfloat16* s = cache + (slot * kv_heads + hk) * D + c;
-      if (vec) {
-        cp_async16(d, s);
-      } else {
-#pragma unroll
-        for (int e = 0; e < 8; ++e) d[e] = c + e < D ? s[e] : __float2bfloat16_rn(0.0f);
-      }
-    } else {
-      *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
-    }
+    __nv_bfloat16 *dk = dst + key * LD + c, *dv = dk + kKeys * LD;
+    const bool in = j <= last;
+    const int64_t row = in ? src.slot(j) * src.kv_heads + src.hk : 0;
+    if (in && c < src.dim) copy8(dk, src.k + row * src.dim, c, src.dim);
+    else *reinterpret_cast<uint4*>(dk) = make_uint4(0u, 0u, 0u, 0u);
+    if (in && c < src.vdim) copy8(dv, src.v + row * src.vdim, c, src.vdim);
+    else *reinterpret_cast<uint4*>(dv) = make_uint4(0u, 0u, 0u, 0u);
   }
 }
 
 // ------------------------------------------------------------------------------------------------
-// prompts: grid (tiles, kv_heads * head tiles), 4 warps of 16 rows
+// prompts: grid (tiles, kv_heads * head tiles), 8 warps of 16 rows
 // ------------------------------------------------------------------------------------------------
 template <int DP>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kRows * 2)
 paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) {
   constexpr int LD = DP + 8;
   extern __shared__ __align__(16) __nv_bfloat16 sm[];
-  __nv_bfloat16* sQ = sm;                       // [64][LD]
-  __nv_bfloat16* sKV = sQ + 64 * LD;            // [2 stages][K, V][64][LD]
+  __nv_bfloat16* sQ = sm;                       // [kRows][LD]
+  __nv_bfloat16* sKV = sQ + kRows * LD;         // [2 stages][K, V][64][LD]
   __shared__ int s_tile[3];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (warp == 0) {
@@ -98,22 +130,28 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
   const int nt = min(tq, a.seg.len[sg] - t0);
   const int pos0 = a.seg.pos[sg] + t0;
   const int64_t row0 = static_cast<int64_t>(a.seg.row0[sg]) + t0;
-  const int32_t* bt = a.block_table + static_cast<int64_t>(a.seg.seq[sg]) * a.max_blocks;
   const int first = a.window > 0 ? max(0, pos0 - a.window + 1) : 0, last = pos0 + nt - 1;
-  const __nv_bfloat16* kc = static_cast<const __nv_bfloat16*>(a.k_cache);
-  const __nv_bfloat16* vc = static_cast<const __nv_bfloat16*>(a.v_cache);
+  const KvSource src(a, a.seg.seq[sg], hk);
   auto stage = [&](int k0, int s) {
-    stage_rows<DP>(sKV + (s * 2) * kKeys * LD, kc, bt, a.block_size, a.kv_heads, hk, a.dim, k0, last);
-    stage_rows<DP>(sKV + (s * 2 + 1) * kKeys * LD, vc, bt, a.block_size, a.kv_heads, hk, a.vdim, k0, last);
+    stage_kv<DP>(sKV + (s * 2) * kKeys * LD, src, k0, last);
     cp_async_commit();
   };
   stage(first, 0);
   {
     const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q);
-    for (int i = threadIdx.x; i < 64 * DP; i += 128) {
-      const int m = i / DP, d = i % DP, tok = m / rt, hh = m % rt;
-      sQ[m * LD + d] = (tok < nt && hh < nh && d < a.dim) ? q[(row0 + tok) * a.ldq + static_cast<int64_t>(h0 + hh) * a.dim + d]
-                                                          : __float2bfloat16_rn(0.0f);
+    const float sign = a.scale < 0.0f ? -1.0f : 1.0f;      // the score map wants a positive factor
+    const uint32_t flip = a.scale < 0.0f ? 0x80008000u : 0u;
+    const bool pairs = ((a.dim | static_cast<int>(a.ldq)) & 1) == 0 && (reinterpret_cast<uintptr_t>(a.q) & 3) == 0;
+    for (int i = threadIdx.x; i < kRows * DP / 2; i += kRows * 2) {
+      const int m = i / (DP / 2), d = (i % (DP / 2)) * 2, tok = m / rt, hh = m % rt;
+      const bool in = tok < nt && hh < nh;
+      const __nv_bfloat16* qp = q + (row0 + tok) * a.ldq + static_cast<int64_t>(h0 + hh) * a.dim + d;
+      if (pairs) {
+        *reinterpret_cast<uint32_t*>(sQ + m * LD + d) = in && d < a.dim ? *reinterpret_cast<const uint32_t*>(qp) ^ flip : 0u;
+      } else {
+        sQ[m * LD + d] = in && d < a.dim ? __float2bfloat16_rn(sign * __bfloat162float(qp[0])) : __float2bfloat16_rn(0.0f);
+        sQ[m * LD + d + 1] = in && d + 1 < a.dim ? __float2bfloat16_rn(sign * __bfloat162float(qp[1])) : __float2bfloat16_rn(0.0f);
+      }
     }
   }
   int qpos[2];                                  // position of this thread's two rows, -1: padding row
@@ -122,7 +160,10 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
     const int m = warp * 16 + i * 8 + (lane >> 2);
     qpos[i] = (m / rt < nt && m % rt < nh) ? pos0 + m / rt : -1;
   }
-  const float inv_cap = a.softcap > 0.0f ? 1.0f / a.softcap : 0.0f;
+  // lowest and highest position among the warp's 16 rows; -1 with a padding row among them
+  const int warp_lo = __reduce_min_sync(0xffffffffu, min(qpos[0], qpos[1]));
+  const int warp_hi = __reduce_max_sync(0xffffffffu, max(qpos[0], qpos[1]));
+  const ScoreMap map(fabsf(a.scale), a.softcap);
   float o[DP / 8][4], mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.0f, 0.0f};
 #pragma unroll
   for (int i = 0; i < DP / 8; ++i)
@@ -156,24 +197,30 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
         mma_bf16(sc[2 * n + 1], qa, kb[2], kb[3]);
       }
     }
+    // every row of this warp sees the whole stage, unless it reaches past a row's own position or before its window
+    const bool edge = warp_lo < 0 || k0 + kKeys - 1 > warp_lo || (a.window > 0 && k0 <= warp_hi - a.window);
     float tmax[2] = {-INFINITY, -INFINITY};
+    if (edge) {
+#pragma unroll
+      for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int j = k0 + n * 8 + (lane & 3) * 2 + (e & 1), qp = qpos[e >> 1];
+          if (!(j <= qp && (a.window <= 0 || j > qp - a.window))) sc[n][e] = -INFINITY;
+        }
+    }
 #pragma unroll
     for (int n = 0; n < 8; ++n)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int j = k0 + n * 8 + (lane & 3) * 2 + (e & 1), qp = qpos[e >> 1];
-        const bool see = j <= qp && (a.window <= 0 || j > qp - a.window);
-        sc[n][e] = see ? score_log2(sc[n][e], a.scale, a.softcap, inv_cap) : -INFINITY;
-        tmax[e >> 1] = fmaxf(tmax[e >> 1], sc[n][e]);
-      }
+      for (int e = 0; e < 4; ++e) tmax[e >> 1] = fmaxf(tmax[e >> 1], sc[n][e]);
     float base[2];
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 1));
       tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 2));
-      const float nm = fmaxf(mx[i], tmax[i]);
+      const float nm = fmaxf(mx[i], map(tmax[i]));
       base[i] = nm == -INFINITY ? 0.0f : nm;
-      const float alpha = exp2f(mx[i] - base[i]);     // first tile: exp2(-inf) = 0
+      const float alpha = ex2_approx(mx[i] - base[i]);     // first stage: 2^-inf = 0
       mx[i] = nm;
       sum[i] *= alpha;
 #pragma unroll
@@ -186,7 +233,7 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
     for (int n = 0; n < 8; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        sc[n][e] = exp2f(sc[n][e] - base[e >> 1]);
+        sc[n][e] = edge && sc[n][e] == -INFINITY ? 0.0f : map.prob(sc[n][e], base[e >> 1]);
         sum[e >> 1] += sc[n][e];
       }
 #pragma unroll
@@ -240,25 +287,24 @@ paged_decode_mma_kernel(const NxPagedWindowArgs a, int head_tiles) {
   const int rep = a.heads / a.kv_heads, h0 = hk * rep + ht * 16, nh = min(16, rep - ht * 16);
   const int pos = a.seg.pos[sg];
   const int64_t row = a.seg.row0[sg];
-  const int32_t* bt = a.block_table + static_cast<int64_t>(a.seg.seq[sg]) * a.max_blocks;
+  const KvSource src(a, a.seg.seq[sg], hk);
   const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
   const int per = ((pos - lo + kKeys) / kKeys + a.splits - 1) / a.splits * kKeys;
   const int first = lo + static_cast<int>(blockIdx.z) * per, last = min(pos, first + per - 1);
-  const __nv_bfloat16* kc = static_cast<const __nv_bfloat16*>(a.k_cache);
-  const __nv_bfloat16* vc = static_cast<const __nv_bfloat16*>(a.v_cache);
   auto stage = [&](int k0, int s) {
-    stage_rows<DP>(sKV + (s * 2) * kKeys * LD, kc, bt, a.block_size, a.kv_heads, hk, a.dim, k0, last);
-    stage_rows<DP>(sKV + (s * 2 + 1) * kKeys * LD, vc, bt, a.block_size, a.kv_heads, hk, a.vdim, k0, last);
+    stage_kv<DP>(sKV + (s * 2) * kKeys * LD, src, k0, last);
     cp_async_commit();
   };
   if (first <= last) stage(first, 0);
+  const float sign = a.scale < 0.0f ? -1.0f : 1.0f;
   for (int i = threadIdx.x; i < 16 * DP; i += 128) {
     const int m = i / DP, d = i % DP;
     sQ[m * LD + d] = (m < nh && d < a.dim)
-                         ? static_cast<const __nv_bfloat16*>(a.q)[row * a.ldq + static_cast<int64_t>(h0 + m) * a.dim + d]
+                         ? __float2bfloat16_rn(sign * __bfloat162float(static_cast<const __nv_bfloat16*>(
+                               a.q)[row * a.ldq + static_cast<int64_t>(h0 + m) * a.dim + d]))
                          : __float2bfloat16_rn(0.0f);
   }
-  const float inv_cap = a.softcap > 0.0f ? 1.0f / a.softcap : 0.0f;
+  const ScoreMap map(fabsf(a.scale), a.softcap);
   float o[DP / 8][4], mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.0f, 0.0f};
 #pragma unroll
   for (int i = 0; i < DP / 8; ++i)
@@ -291,15 +337,15 @@ paged_decode_mma_kernel(const NxPagedWindowArgs a, int head_tiles) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int j = k0 + warp * 16 + n * 8 + (lane & 3) * 2 + (e & 1);
-          sc[n][e] = j <= last ? score_log2(sc[n][e], a.scale, a.softcap, inv_cap) : -INFINITY;
+          sc[n][e] = j <= last ? sc[n][e] : -INFINITY;
           tmax[e >> 1] = fmaxf(tmax[e >> 1], sc[n][e]);
         }
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
         tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 1));
         tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 2));
-        const float nm = fmaxf(mx[i], tmax[i]);       // at least one key of this warp is in range
-        const float alpha = exp2f(mx[i] - nm);
+        const float nm = fmaxf(mx[i], map(tmax[i]));  // at least one key of this warp is in range
+        const float alpha = ex2_approx(mx[i] - nm);
         mx[i] = nm;
         sum[i] *= alpha;
 #pragma unroll
@@ -312,7 +358,7 @@ paged_decode_mma_kernel(const NxPagedWindowArgs a, int head_tiles) {
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          sc[n][e] = exp2f(sc[n][e] - mx[e >> 1]);
+          sc[n][e] = sc[n][e] == -INFINITY ? 0.0f : map.prob(sc[n][e], mx[e >> 1]);
           sum[e >> 1] += sc[n][e];
         }
       const uint32_t pa[4] = {bf16_pair(sc[0][0], sc[0][1]), bf16_pair(sc[0][2], sc[0][3]), bf16_pair(sc[1][0], sc[1][1]),
@@ -457,13 +503,13 @@ int padded_dim(const NxPagedWindowArgs* a) {
 
 template <int DP>
 int launch_prefill(const NxPagedWindowArgs* a, dim3 grid, int rt, int tq, int head_tiles, cudaStream_t st) {
-  constexpr int kSmem = (64 + 4 * kKeys) * (DP + 8) * 2;
+  constexpr int kSmem = (kRows + 4 * kKeys) * (DP + 8) * 2;
   static bool once = false;
   if (!once) {
     if (cudaFuncSetAttribute(paged_prefill_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -2;
     once = true;
   }
-  paged_prefill_kernel<DP><<<grid, 128, kSmem, st>>>(*a, rt, tq, head_tiles);
+  paged_prefill_kernel<DP><<<grid, kRows * 2, kSmem, st>>>(*a, rt, tq, head_tiles);
   return launch_status();
 }
 
@@ -487,7 +533,7 @@ extern "C" int nx_paged_window_prefill(const NxPagedWindowArgs* a, nx_stream_t s
   if (a->seg.count <= 0 || a->seg.total_len <= 0) return 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int rep = a->heads / a->kv_heads;
-  const int rt = std::min(rep, 16), head_tiles = (rep + rt - 1) / rt, tq = 64 / rt;
+  const int rt = std::min(rep, 16), head_tiles = (rep + rt - 1) / rt, tq = kRows / rt;
   dim3 grid(a->seg.total_len / tq + a->seg.count, a->kv_heads * head_tiles);
   switch (padded_dim(a)) {
     case 32: return launch_prefill<32>(a, grid, rt, tq, head_tiles, st);

@@ -110,8 +110,8 @@ __device__ __forceinline__ void scan64(float& v0, float& v1) {
 }
 
 // ------------------------------------------------------------------------------------------------
-// state-space duality.  grid (heads * column tiles, parts, segments), 4 warps.  Warp w owns token rows
-// 16 w .. 16 w + 15 of the chunk's outputs and NP / 4 rows of the state.
+// state-space duality.  grid (heads * column tiles, parts, segments), 8 warps.  Warp w owns 16 token rows of
+// the chunk's outputs and NP / 4 rows of the state (w mod 4), 32 value columns of both (w / 4).
 // kLocal: only the span's own contribution to the state, from zero, and its decay (for spans that run
 // at the same time); otherwise outputs, from the span's true start state.
 // ------------------------------------------------------------------------------------------------
@@ -124,7 +124,7 @@ struct SsdSmem {
 };
 
 template <int NP, bool kLocal>
-__global__ void __launch_bounds__(128) ssd_chunk_kernel(const NxSsdArgs a, int col_tiles) {
+__global__ void __launch_bounds__(256, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const NxSsdArgs a, int col_tiles) {
   using L = SsdSmem<NP>;
   constexpr int LN = L::LN, LP = L::LP, MT = NP / 64;    // MT: 16-row tiles of the state per warp
   extern __shared__ __align__(16) __nv_bfloat16 sm[];
@@ -135,7 +135,7 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const NxSsdArgs a, int c
   const int len = a.seg.len[sg], t_begin = part * a.span, t_end = min(len, t_begin + a.span);
   if (t_begin >= len || (kLocal && t_end == len)) return;   // the last span's contribution is never needed
   const int N = a.n_state, P = a.vdim, cols = min(kCols, P - p0), inner = a.heads * P, g = h / (a.heads / a.groups);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, qr = lane >> 2, qc = (lane & 3) * 2;
+  const int warp = (threadIdx.x >> 5) & 3, cb = (threadIdx.x >> 7) * 32, lane = threadIdx.x & 31, qr = lane >> 2, qc = (lane & 3) * 2;
   const int64_t row0 = a.seg.row0[sg];
   const __nv_bfloat16* xbc = static_cast<const __nv_bfloat16*>(a.xbc) + row0 * a.ld_xbc;
   const __nv_bfloat16* dtp = static_cast<const __nv_bfloat16*>(a.dt) + row0 * a.ld_dt + h;
@@ -145,16 +145,16 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const NxSsdArgs a, int c
   const int64_t plane = static_cast<int64_t>(N) * P;
   float* pool = a.state + (static_cast<int64_t>(a.seg.seq[sg]) * a.heads + h) * plane;
   float* part_state = a.parts > 1 ? a.part_state + ((static_cast<int64_t>(sg) * a.parts + part) * a.heads + h) * plane : nullptr;
-  float S[MT][8][4];
+  float S[MT][4][4];
   {
     const float* src = kLocal ? nullptr : a.parts > 1 ? part_state : (a.seg.pos[sg] == 0 ? nullptr : pool);
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int n = 0; n < 8; ++n)
+      for (int n = 0; n < 4; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int r = (warp * MT + m) * 16 + (e >> 1) * 8 + qr, c = n * 8 + qc + (e & 1);
+          const int r = (warp * MT + m) * 16 + (e >> 1) * 8 + qr, c = cb + n * 8 + qc + (e & 1);
           S[m][n][e] = (src != nullptr && r < N && c < cols) ? src[static_cast<int64_t>(r) * P + p0 + c] : 0.0f;
         }
   }
@@ -166,7 +166,7 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const NxSsdArgs a, int c
     if (!kLocal) load_tile<NP>(sC, src + inner + (a.groups + g) * N, a.ld_xbc, rows, N, vec_n);
     load_tile<kCols>(sX, src + h * P + p0, a.ld_xbc, rows, cols, vec_p);
     cp_async_commit();
-    if (warp == 0) {
+    if (threadIdx.x < 32) {
       float d[2], c[2];
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
@@ -183,15 +183,15 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const NxSsdArgs a, int c
     }
     if (!kLocal) {
 #pragma unroll
-      for (int m = 0; m < MT; ++m) store_split<8, LP>(sSh, sSl, (warp * MT + m) * 16, S[m]);
+      for (int m = 0; m < MT; ++m) store_split<4, LP>(sSh + cb, sSl + cb, (warp * MT + m) * 16, S[m]);
     }
     cp_async_wait<0>();
     __syncthreads();
     const float c_end = s_c[kQ - 1];
     // x weighted for the state update
-    for (int i = threadIdx.x; i < kQ * (kCols / 2); i += 128) {
+    for (int i = threadIdx.x; i < kQ * (kCols / 2); i += 256) {
       const int t = i / (kCols / 2), o = t * LP + (i % (kCols / 2)) * 2;
-      const float w = exp2f(c_end - s_c[t]) * s_dt[t];
+      const float w = ex2_approx(c_end - s_c[t]) * s_dt[t];
       const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(sX + o);
       uint32_t hi, lo;
       bf16_split(__low2float(x) * w, __high2float(x) * w, hi, lo);
@@ -200,26 +200,26 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const NxSsdArgs a, int c
     }
     if (!kLocal) {
       const float ci[2] = {s_c[warp * 16 + qr], s_c[warp * 16 + 8 + qr]};
-      float y[8][4];
+      float y[4][4];
       zero(y);
 #pragma unroll
       for (int kk = 0; kk < NP / 16; ++kk) {             // C S
         uint32_t ca[4];
         ldmatrix_x4(ca, addr_a<LN>(sC, warp * 16, kk * 16));
 #pragma unroll
-        for (int n = 0; n < 4; ++n) {
+        for (int n = 0; n < 2; ++n) {
           uint32_t b[4];
-          ldmatrix_x4_trans(b, addr_b_t<LP>(sSh, kk * 16, n * 16));
+          ldmatrix_x4_trans(b, addr_b_t<LP>(sSh, kk * 16, cb + n * 16));
           mma_bf16(y[2 * n], ca, b[0], b[1]);
           mma_bf16(y[2 * n + 1], ca, b[2], b[3]);
-          ldmatrix_x4_trans(b, addr_b_t<LP>(sSl, kk * 16, n * 16));
+          ldmatrix_x4_trans(b, addr_b_t<LP>(sSl, kk * 16, cb + n * 16));
           mma_bf16(y[2 * n], ca, b[0], b[1]);
           mma_bf16(y[2 * n + 1], ca, b[2], b[3]);
         }
       }
-      const float e0 = exp2f(ci[0]), e1 = exp2f(ci[1]);
+      const float e0 = ex2_approx(ci[0]), e1 = ex2_approx(ci[1]);
 #pragma unroll
-      for (int n = 0; n < 8; ++n) {
+      for (int n = 0; n < 4; ++n) {
         y[n][0] *= e0;
         y[n][1] *= e0;
         y[n][2] *= e1;
@@ -241,7 +241,7 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const NxSsdArgs a, int c
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int s = j * 16 + n * 8 + qc + (e & 1), t = warp * 16 + (e >> 1) * 8 + qr;
-            gm[n][e] = s <= t ? gm[n][e] * exp2f(ci[e >> 1] - s_c[s]) * s_dt[s] : 0.0f;
+            gm[n][e] = s <= t ? gm[n][e] * ex2_approx(ci[e >> 1] - s_c[s]) * s_dt[s] : 0.0f;
           }
         uint32_t mh[4], ml[4];
         bf16_split(gm[0][0], gm[0][1], mh[0], ml[0]);
@@ -249,9 +249,9 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const NxSsdArgs a, int c
         bf16_split(gm[1][0], gm[1][1], mh[2], ml[2]);
         bf16_split(gm[1][2], gm[1][3], mh[3], ml[3]);
 #pragma unroll
-        for (int n = 0; n < 4; ++n) {
+        for (int n = 0; n < 2; ++n) {
           uint32_t b[4];
-          ldmatrix_x4_trans(b, addr_b_t<LP>(sX, j * 16, n * 16));
+          ldmatrix_x4_trans(b, addr_b_t<LP>(sX, j * 16, cb + n * 16));
           mma_bf16(y[2 * n], mh, b[0], b[1]);
           mma_bf16(y[2 * n + 1], mh, b[2], b[3]);
           mma_bf16(y[2 * n], ml, b[0], b[1]);
@@ -259,27 +259,32 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const NxSsdArgs a, int c
         }
       }
       __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.y) + (row0 + t0) * a.ldy + static_cast<int64_t>(h) * P + p0;
+      const bool pair = ((a.ldy | P) & 1) == 0;
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
         const int t = warp * 16 + i * 8 + qr;
         if (t >= rows) continue;
 #pragma unroll
-        for (int n = 0; n < 8; ++n) {
-          const int c = n * 8 + qc;
+        for (int n = 0; n < 4; ++n) {
+          const int c = cb + n * 8 + qc;
           const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(sX + t * LP + c);
           const float v0 = y[n][2 * i] + skip * __low2float(x), v1 = y[n][2 * i + 1] + skip * __high2float(x);
-          if (c < cols) out[t * a.ldy + c] = __float2bfloat16_rn(v0);
-          if (c + 1 < cols) out[t * a.ldy + c + 1] = __float2bfloat16_rn(v1);
+          if (pair) {
+            if (c < cols) *reinterpret_cast<uint32_t*>(out + t * a.ldy + c) = bf16_pair(v0, v1);
+          } else {
+            if (c < cols) out[t * a.ldy + c] = __float2bfloat16_rn(v0);
+            if (c + 1 < cols) out[t * a.ldy + c + 1] = __float2bfloat16_rn(v1);
+          }
         }
       }
     }
     __syncthreads();                                     // weighted x complete
-    const float dec = exp2f(c_end);
+    const float dec = ex2_approx(c_end);
     total += c_end;
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int n = 0; n < 8; ++n)
+      for (int n = 0; n < 4; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) S[m][n][e] *= dec;
 #pragma unroll
@@ -288,10 +293,10 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const NxSsdArgs a, int c
 #pragma unroll
       for (int m = 0; m < MT; ++m) ldmatrix_x4_trans(ba[m], addr_a_t<LN>(sB, kk * 16, (warp * MT + m) * 16));
 #pragma unroll
-      for (int n = 0; n < 4; ++n) {
+      for (int n = 0; n < 2; ++n) {
         uint32_t bh[4], bl[4];
-        ldmatrix_x4_trans(bh, addr_b_t<LP>(sXh, kk * 16, n * 16));
-        ldmatrix_x4_trans(bl, addr_b_t<LP>(sXl, kk * 16, n * 16));
+        ldmatrix_x4_trans(bh, addr_b_t<LP>(sXh, kk * 16, cb + n * 16));
+        ldmatrix_x4_trans(bl, addr_b_t<LP>(sXl, kk * 16, cb + n * 16));
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           mma_bf16(S[m][2 * n], ba[m], bh[0], bh[1]);
@@ -308,14 +313,14 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(const NxSsdArgs a, int c
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int n = 0; n < 8; ++n)
+      for (int n = 0; n < 4; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int r = (warp * MT + m) * 16 + (e >> 1) * 8 + qr, c = n * 8 + qc + (e & 1);
+          const int r = (warp * MT + m) * 16 + (e >> 1) * 8 + qr, c = cb + n * 8 + qc + (e & 1);
           if (r < N && c < cols) dst[static_cast<int64_t>(r) * P + p0 + c] = S[m][n][e];
         }
     if (kLocal && threadIdx.x == 0 && p0 == 0)
-      a.part_decay[(static_cast<int64_t>(sg) * a.parts + part) * a.heads + h] = exp2f(total);
+      a.part_decay[(static_cast<int64_t>(sg) * a.parts + part) * a.heads + h] = ex2_approx(total);
   }
 }
 
@@ -350,28 +355,66 @@ int launch_ssd(const NxSsdArgs* a, cudaStream_t st) {
   const int col_tiles = (a->vdim + kCols - 1) / kCols;
   dim3 grid(a->heads * col_tiles, a->parts, a->seg.count);
   if (a->parts > 1) {
-    ssd_chunk_kernel<NP, true><<<grid, 128, kBytes, st>>>(*a, col_tiles);
+    ssd_chunk_kernel<NP, true><<<grid, 256, kBytes, st>>>(*a, col_tiles);
     const int plane = a->n_state * a->vdim;
     ssd_span_scan_kernel<<<dim3(a->heads, a->seg.count, (plane + 255) / 256), 256, 0, st>>>(*a);
   }
-  ssd_chunk_kernel<NP, false><<<grid, 128, kBytes, st>>>(*a, col_tiles);
+  ssd_chunk_kernel<NP, false><<<grid, 256, kBytes, st>>>(*a, col_tiles);
   return launch_status();
 }
 
 // ------------------------------------------------------------------------------------------------
 // delta rule, first kernel: everything of a chunk that does not depend on the state.
-// grid (chunks, heads, segments), 4 warps.  Scratch per (segment, chunk, head): T hi | T lo | P hi | P lo, each [64][64]
-// BF16, then FP32 [4][64]: cumulative log2 decay, 1 / |k|, dim^-1/2 / |q|, beta.
+// grid (chunks, heads, segments), 4 warps.  Scratch per (segment, chunk, head): T hi | T lo | P hi | P lo, each 64 x 64 BF16
+// in the order of the A fragments that read them - [row tile][16-column block][lane][8], blocks past the diagonal unused -
+// then FP32 [4][64]: cumulative log2 decay, 1 / |k|, dim^-1/2 / |q|, beta.
 // ------------------------------------------------------------------------------------------------
 constexpr int64_t kDeltaTile = kQ * kQ;
 constexpr int64_t kDeltaUnit = 4 * kDeltaTile + 4 * kQ * 2;   // in BF16 elements
+
+__device__ __forceinline__ uint4* fragment(__nv_bfloat16* tile, int row_tile, int block) {
+  return reinterpret_cast<uint4*>(tile) + (row_tile * (kQ / 16) + block) * 32 + (threadIdx.x & 31);
+}
+__device__ __forceinline__ void store_fragment(__nv_bfloat16* hi, __nv_bfloat16* lo, int row_tile, int block, const float (&v)[2][4]) {
+  uint4 h, l;                          // v: two 16 x 8 accumulator tiles side by side
+  bf16_split(v[0][0], v[0][1], h.x, l.x);
+  bf16_split(v[0][2], v[0][3], h.y, l.y);
+  bf16_split(v[1][0], v[1][1], h.z, l.z);
+  bf16_split(v[1][2], v[1][3], h.w, l.w);
+  *fragment(hi, row_tile, block) = h;
+  *fragment(lo, row_tile, block) = l;
+}
+
+// bytes of the first region of the kernel's shared memory: q and k, later the inverse and its scratch
+template <int DP>
+constexpr int prep_front() {
+  constexpr int qk = 2 * kQ * (DP + 8) * 2, inv = (kQ * (kQ + 4) + 4 * 16 * 17) * 4;
+  return qk > inv ? qk : inv;
+}
+
+// acc[r] += sum_k a[r][k] b[k], 8 rows of `a` (pitch LA, 16-byte aligned) and one column of `b` (pitch LB), n a multiple of 4
+template <int LA, int LB = LA>
+__device__ __forceinline__ void block_product(float (&acc)[8], const float* a, const float* b, int n) {
+  for (int k = 0; k < n; k += 4) {
+    float bv[4];
+#pragma unroll
+    for (int q = 0; q < 4; ++q) bv[q] = b[(k + q) * LB];
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+      const float4 av = *reinterpret_cast<const float4*>(a + r * LA + k);
+      acc[r] += av.x * bv[0] + av.y * bv[1] + av.z * bv[2] + av.w * bv[3];
+    }
+  }
+}
 
 template <int DP>
 __global__ void __launch_bounds__(128) delta_prep_kernel(const NxDeltaArgs a, int chunks) {
   constexpr int LD = DP + 8, LA = kQ + 4;
   extern __shared__ __align__(16) __nv_bfloat16 sm[];
   __nv_bfloat16 *sK = sm, *sQ = sm + kQ * LD;
-  float* sA = reinterpret_cast<float*>(sm + 2 * kQ * LD);     // [64][LA]
+  float* sT = reinterpret_cast<float*>(sm);                   // [64][LA], then [4][16][17]: over q and k, once these are consumed
+  float* sW = sT + kQ * LA;
+  float* sA = sT + prep_front<DP>() / 4;                      // [64][LA]
   __shared__ float s_b[kQ], s_rk[kQ], s_rq[kQ], s_beta[kQ];
   const int ch = blockIdx.x, h = blockIdx.y, sg = blockIdx.z, t0 = ch * kQ;
   const int len = a.seg.len[sg];
@@ -429,67 +472,79 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const NxDeltaArgs a, in
   const float rkt[2] = {s_rk[warp * 16 + qr], s_rk[warp * 16 + 8 + qr]};
   const float rqt[2] = {s_rq[warp * 16 + qr], s_rq[warp * 16 + 8 + qr]};
   const float bet[2] = {s_beta[warp * 16 + qr], s_beta[warp * 16 + 8 + qr]};
-#pragma unroll
-  for (int j = 0; j < kQ / 16; ++j) {
+  for (int j = 0; j <= warp; ++j) {
     float kk[2][4], qk[2][4];
     zero(kk);
     zero(qk);
-    if (j <= warp) {
 #pragma unroll
-      for (int d = 0; d < DP / 16; ++d) {
-        uint32_t ka[4], qa[4], b[4];
-        ldmatrix_x4(ka, addr_a<LD>(sK, warp * 16, d * 16));
-        ldmatrix_x4(qa, addr_a<LD>(sQ, warp * 16, d * 16));
-        ldmatrix_x4(b, addr_b<LD>(sK, j * 16, d * 16));
-        mma_bf16(kk[0], ka, b[0], b[1]);
-        mma_bf16(kk[1], ka, b[2], b[3]);
-        mma_bf16(qk[0], qa, b[0], b[1]);
-        mma_bf16(qk[1], qa, b[2], b[3]);
-      }
+    for (int d = 0; d < DP / 16; ++d) {
+      uint32_t ka[4], qa[4], b[4];
+      ldmatrix_x4(ka, addr_a<LD>(sK, warp * 16, d * 16));
+      ldmatrix_x4(qa, addr_a<LD>(sQ, warp * 16, d * 16));
+      ldmatrix_x4(b, addr_b<LD>(sK, j * 16, d * 16));
+      mma_bf16(kk[0], ka, b[0], b[1]);
+      mma_bf16(kk[1], ka, b[2], b[3]);
+      mma_bf16(qk[0], qa, b[0], b[1]);
+      mma_bf16(qk[1], qa, b[2], b[3]);
     }
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int t = warp * 16 + i * 8 + qr, s = j * 16 + n * 8 + qc;
-        float p[2];
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const float w = s + e <= t ? exp2f(bt[i] - s_b[s + e]) * s_rk[s + e] : 0.0f;
-          p[e] = qk[n][2 * i + e] * w * rqt[i];
-          sA[t * LA + s + e] = s + e < t ? kk[n][2 * i + e] * w * rkt[i] * bet[i] : 0.0f;
-        }
-        uint32_t hi, lo;
-        bf16_split(p[0], p[1], hi, lo);
-        *reinterpret_cast<uint32_t*>(Ph + t * kQ + s) = hi;
-        *reinterpret_cast<uint32_t*>(Pl + t * kQ + s) = lo;
+      for (int e = 0; e < 4; ++e) {
+        const int i = e >> 1, t = warp * 16 + i * 8 + qr, s = j * 16 + n * 8 + qc + (e & 1);
+        const float w = s <= t ? ex2_approx(bt[i] - s_b[s]) * s_rk[s] : 0.0f;
+        qk[n][e] *= w * rqt[i];
+        sA[t * LA + s] = s < t ? kk[n][e] * w * rkt[i] * bet[i] : 0.0f;
       }
+    store_fragment(Ph, Pl, warp, j, qk);
   }
   __syncthreads();
-  if (threadIdx.x < kQ) {                      // column c of (I + A)^-1 by forward substitution, in registers
-    const int c = threadIdx.x;
-    float x[kQ];
+  // T = (I + A)^-1 by 16 x 16 blocks, FP32.  Diagonal blocks: one thread per column, forward substitution in registers.
+  if (threadIdx.x < kQ) {
+    const int blk = threadIdx.x / 16 * 16, c = threadIdx.x % 16;
+    float x[16];
 #pragma unroll
-    for (int i = 0; i < kQ; ++i) {
-      float v0 = i == c ? 1.0f : 0.0f, v1 = 0.0f, v2 = 0.0f, v3 = 0.0f;
+    for (int i = 0; i < 16; ++i) {
+      float v = i == c ? 1.0f : 0.0f;
 #pragma unroll
-      for (int j = 0; j + 3 < i; j += 4) {
-        const float4 r = *reinterpret_cast<const float4*>(sA + i * LA + j);
-        v0 -= r.x * x[j];
-        v1 -= r.y * x[j + 1];
-        v2 -= r.z * x[j + 2];
-        v3 -= r.w * x[j + 3];
+      for (int j = 0; j < i; ++j) v -= sA[(blk + i) * LA + blk + j] * x[j];
+      x[i] = v;
+    }
+#pragma unroll
+    for (int i = 0; i < 16; ++i) sT[(blk + i) * LA + blk + c] = x[i];
+  }
+  // Below the diagonal: T_ij = -T_ii sum_{j <= k < i} A_ik T_kj, one block diagonal after the other, a warp per block.  A lane
+  // has one column and 8 rows.
+  for (int d = 1; d < kQ / 16; ++d) {
+    __syncthreads();
+    const int i = warp + d, j = warp;
+    if (i < kQ / 16) {
+      const int c = lane & 15, r0 = (lane >> 4) * 8;
+      float acc[8] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
+      block_product<LA>(acc, sA + (i * 16 + r0) * LA + j * 16, sT + j * 16 * LA + j * 16 + c, 16 * d);
+      float* w = sW + warp * 16 * 17;
+#pragma unroll
+      for (int r = 0; r < 8; ++r) {
+        w[(r0 + r) * 17 + c] = acc[r];
+        acc[r] = 0.0f;
       }
+      __syncwarp();
+      block_product<LA, 17>(acc, sT + (i * 16 + r0) * LA + i * 16, w + c, 16);
 #pragma unroll
-      for (int j = i / 4 * 4; j < i; ++j) v0 -= sA[i * LA + j] * x[j];
-      x[i] = (v0 + v1) + (v2 + v3);
+      for (int r = 0; r < 8; ++r) sT[(i * 16 + r0 + r) * LA + j * 16 + c] = -acc[r];
     }
+  }
+  __syncthreads();
+  for (int j = 0; j <= warp; ++j) {
+    float v[2][4];
 #pragma unroll
-    for (int i = 0; i < kQ; ++i) {
-      const __nv_bfloat16 hi = __float2bfloat16_rn(x[i]);
-      Th[i * kQ + c] = hi;
-      Tl[i * kQ + c] = __float2bfloat16_rn(x[i] - __bfloat162float(hi));
-    }
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[n][e] = sT[(warp * 16 + (e >> 1) * 8 + qr) * LA + j * 16 + n * 8 + qc + (e & 1)];
+    store_fragment(Th, Tl, warp, j, v);
+  }
+  if (threadIdx.x < kQ) {
+    const int c = threadIdx.x;
     float* sc = reinterpret_cast<float*>(unit + 4 * kDeltaTile);
     sc[c] = s_b[c];
     sc[kQ + c] = s_rk[c];
@@ -500,32 +555,33 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const NxDeltaArgs a, in
 
 // ------------------------------------------------------------------------------------------------
 // delta rule, second kernel: the chunks of a segment in order.  grid (heads * column tiles, segments),
-// 4 warps; warp w owns token rows 16 w .. of U and the outputs, and DP / 4 rows of the state.
+// 8 warps: warp w owns 16 token rows of U and the outputs and DP / 4 rows of the state (w mod 4), 32
+// value columns of both (w / 4).
 // ------------------------------------------------------------------------------------------------
-constexpr int kDeltaCols = 32;
+constexpr int kDeltaCols = 64;
 
 template <int DP>
 struct DeltaSmem {
-  static constexpr int LD = DP + 8, LV = kDeltaCols + 8, LT = kQ + 8;
-  static constexpr int kK = 0, kQq = kK + kQ * LD, kV = kQq + kQ * LD, kTh = kV + kQ * LV, kTl = kTh + kQ * LT,
-                       kPh = kTl + kQ * LT, kPl = kPh + kQ * LT, kRh = kPl + kQ * LT, kRl = kRh + kQ * LV, kUh = kRl + kQ * LV,
+  static constexpr int LD = DP + 8, LV = kDeltaCols + 8;
+  static constexpr int kK = 0, kQq = kK + kQ * LD, kRh = kQq + kQ * LD, kRl = kRh + kQ * LV, kUh = kRl + kQ * LV,
                        kUl = kUh + kQ * LV, kSh = kUl + kQ * LV, kSl = kSh + DP * LV, kEnd = kSl + DP * LV;
   static constexpr int kBytes = kEnd * 2;
 };
 
-// d += (ah + al) (bh + bl) up to the product of the two remainders, over the first `kblocks` blocks of 16
-template <int LT, int LV>
-__device__ __forceinline__ void mma_split(float (&d)[kDeltaCols / 8][4], const __nv_bfloat16* ah, const __nv_bfloat16* al,
-                                          const __nv_bfloat16* bh, const __nv_bfloat16* bl, int row, int kblocks) {
-  for (int kk = 0; kk < kblocks; ++kk) {
-    uint32_t fh[4], fl[4];
-    ldmatrix_x4(fh, addr_a<LT>(ah, row, kk * 16));
-    ldmatrix_x4(fl, addr_a<LT>(al, row, kk * 16));
+// d += (ah + al) (bh + bl) up to the product of the two remainders, over the blocks 0 .. row_tile of a lower-triangular tile
+// pair in fragment order; d covers 32 columns
+template <int LV>
+__device__ __forceinline__ void mma_triangle(float (&d)[4][4], const uint4 (&ah)[kQ / 16], const uint4 (&al)[kQ / 16],
+                                             const __nv_bfloat16* bh, const __nv_bfloat16* bl, int row_tile, int col) {
 #pragma unroll
-    for (int n = 0; n < kDeltaCols / 16; ++n) {
+  for (int kk = 0; kk < kQ / 16; ++kk) {
+    if (kk > row_tile) break;
+    const uint32_t fh[4] = {ah[kk].x, ah[kk].y, ah[kk].z, ah[kk].w}, fl[4] = {al[kk].x, al[kk].y, al[kk].z, al[kk].w};
+#pragma unroll
+    for (int n = 0; n < 2; ++n) {
       uint32_t gh[4], gl[4];
-      ldmatrix_x4_trans(gh, addr_b_t<LV>(bh, kk * 16, n * 16));
-      ldmatrix_x4_trans(gl, addr_b_t<LV>(bl, kk * 16, n * 16));
+      ldmatrix_x4_trans(gh, addr_b_t<LV>(bh, kk * 16, col + n * 16));
+      ldmatrix_x4_trans(gl, addr_b_t<LV>(bl, kk * 16, col + n * 16));
       mma_bf16(d[2 * n], fh, gh[0], gh[1]);
       mma_bf16(d[2 * n + 1], fh, gh[2], gh[3]);
       mma_bf16(d[2 * n], fh, gl[0], gl[1]);
@@ -535,34 +591,42 @@ __device__ __forceinline__ void mma_split(float (&d)[kDeltaCols / 8][4], const _
     }
   }
 }
+__device__ __forceinline__ void load_fragments(uint4 (&hi)[kQ / 16], uint4 (&lo)[kQ / 16], const __nv_bfloat16* tile, int row_tile) {
+#pragma unroll
+  for (int kk = 0; kk < kQ / 16; ++kk) {
+    if (kk > row_tile) break;
+    hi[kk] = *fragment(const_cast<__nv_bfloat16*>(tile), row_tile, kk);
+    lo[kk] = *fragment(const_cast<__nv_bfloat16*>(tile) + kDeltaTile, row_tile, kk);
+  }
+}
 
 template <int DP>
-__global__ void __launch_bounds__(128) delta_chunk_kernel(const NxDeltaArgs a, int chunks, int col_tiles) {
+__global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) delta_chunk_kernel(const NxDeltaArgs a, int chunks, int col_tiles) {
   using L = DeltaSmem<DP>;
-  constexpr int LD = L::LD, LV = L::LV, LT = L::LT, MT = DP / 64, NT = kDeltaCols / 8;
+  constexpr int LD = L::LD, LV = L::LV, MT = DP / 64;
   extern __shared__ __align__(16) __nv_bfloat16 sm[];
-  __nv_bfloat16 *sK = sm + L::kK, *sQ = sm + L::kQq, *sV = sm + L::kV, *sTh = sm + L::kTh, *sTl = sm + L::kTl,
-                *sPh = sm + L::kPh, *sPl = sm + L::kPl, *sRh = sm + L::kRh, *sRl = sm + L::kRl, *sUh = sm + L::kUh,
-                *sUl = sm + L::kUl, *sSh = sm + L::kSh, *sSl = sm + L::kSl;
+  __nv_bfloat16 *sK = sm + L::kK, *sQ = sm + L::kQq, *sRh = sm + L::kRh, *sRl = sm + L::kRl, *sUh = sm + L::kUh, *sUl = sm + L::kUl,
+                *sSh = sm + L::kSh, *sSl = sm + L::kSl;
+  __nv_bfloat16* sV = sUh;             // v is consumed before U is written
   __shared__ __align__(16) float s_sc[4 * kQ];           // cumulative log2 decay | 1/|k| | scaled 1/|q| | beta
   const int h = blockIdx.x / col_tiles, v0 = (blockIdx.x % col_tiles) * kDeltaCols, sg = blockIdx.y;
   const int len = a.seg.len[sg];
   if (len <= 0) return;
   const int D = a.dim, Dv = a.vdim, cols = min(kDeltaCols, Dv - v0), hk = h / (a.heads / a.kv_heads), kcols = a.kv_heads * D;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, qr = lane >> 2, qc = (lane & 3) * 2;
+  const int warp = (threadIdx.x >> 5) & 3, cb = (threadIdx.x >> 7) * 32, lane = threadIdx.x & 31, qr = lane >> 2, qc = (lane & 3) * 2;
   const int64_t row0 = a.seg.row0[sg];
   const bool aligned = (a.ld_qkv & 7) == 0 && (reinterpret_cast<uintptr_t>(a.qkv) & 15) == 0;
   const bool vec_d = aligned && (D & 7) == 0, vec_v = aligned && (Dv & 7) == 0 && ((2 * kcols) & 7) == 0;
   float* pool = a.state + (static_cast<int64_t>(a.seg.seq[sg]) * a.heads + h) * D * Dv;
   const bool fresh = a.seg.pos[sg] == 0;
-  float S[MT][NT][4];
+  float S[MT][4][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int n = 0; n < NT; ++n)
+    for (int n = 0; n < 4; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int r = (warp * MT + m) * 16 + (e >> 1) * 8 + qr, c = n * 8 + qc + (e & 1);
+        const int r = (warp * MT + m) * 16 + (e >> 1) * 8 + qr, c = cb + n * 8 + qc + (e & 1);
         S[m][n][e] = (!fresh && r < D && c < cols) ? pool[static_cast<int64_t>(r) * Dv + v0 + c] : 0.0f;
       }
   for (int ch = 0; ch * kQ < len; ++ch) {
@@ -573,87 +637,96 @@ __global__ void __launch_bounds__(128) delta_chunk_kernel(const NxDeltaArgs a, i
     load_tile<DP>(sQ, src + hk * D, a.ld_qkv, rows, D, vec_d);
     load_tile<DP>(sK, src + kcols + hk * D, a.ld_qkv, rows, D, vec_d);
     load_tile<kDeltaCols>(sV, src + 2 * kcols + h * Dv + v0, a.ld_qkv, rows, cols, vec_v);
-    for (int i = threadIdx.x; i < 4 * kQ * 8; i += 128) {       // T and P tiles, 16 bytes each
-      const int m = i / (kQ * 8), r = (i / 8) % kQ, c = (i % 8) * 8;
-      cp_async16(sTh + m * (kQ * LT) + r * LT + c, unit + m * kDeltaTile + r * kQ + c);
-    }
-    for (int i = threadIdx.x; i < kQ; i += 128)
-      cp_async16(s_sc + i * 4, reinterpret_cast<const float*>(unit + 4 * kDeltaTile) + i * 4);
+    if (threadIdx.x < kQ) cp_async16(s_sc + threadIdx.x * 4, reinterpret_cast<const float*>(unit + 4 * kDeltaTile) + threadIdx.x * 4);
     cp_async_commit();
+    uint4 fh[kQ / 16], fl[kQ / 16];                      // rows of T, later of P
+    load_fragments(fh, fl, unit, warp);
 #pragma unroll
-    for (int m = 0; m < MT; ++m) store_split<NT, LV>(sSh, sSl, (warp * MT + m) * 16, S[m]);
+    for (int m = 0; m < MT; ++m) store_split<4, LV>(sSh + cb, sSl + cb, (warp * MT + m) * 16, S[m]);
     cp_async_wait<0>();
     __syncthreads();
     const float b_end = s_sc[kQ - 1];
-    float eb[2], rk[2], rq[2], beta[2], wk[2];
+    float o[4][4], u[4][4];
+    zero(o);
+    {
+      float ks[4][4];
+      zero(ks);
+#pragma unroll
+      for (int d = 0; d < DP / 16; ++d) {
+        uint32_t ka[4], qa[4];
+        ldmatrix_x4(ka, addr_a<LD>(sK, warp * 16, d * 16));
+        ldmatrix_x4(qa, addr_a<LD>(sQ, warp * 16, d * 16));
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          uint32_t bh[4], bl[4];
+          ldmatrix_x4_trans(bh, addr_b_t<LV>(sSh, d * 16, cb + n * 16));
+          ldmatrix_x4_trans(bl, addr_b_t<LV>(sSl, d * 16, cb + n * 16));
+          mma_bf16(ks[2 * n], ka, bh[0], bh[1]);
+          mma_bf16(ks[2 * n + 1], ka, bh[2], bh[3]);
+          mma_bf16(o[2 * n], qa, bh[0], bh[1]);
+          mma_bf16(o[2 * n + 1], qa, bh[2], bh[3]);
+          mma_bf16(ks[2 * n], ka, bl[0], bl[1]);
+          mma_bf16(ks[2 * n + 1], ka, bl[2], bl[3]);
+          mma_bf16(o[2 * n], qa, bl[0], bl[1]);
+          mma_bf16(o[2 * n + 1], qa, bl[2], bl[3]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int t = warp * 16 + i * 8 + qr;
+        const float eb = ex2_approx(s_sc[t]), fk = eb * s_sc[kQ + t], fq = eb * s_sc[2 * kQ + t], beta = s_sc[3 * kQ + t];
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+          const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(sV + t * LV + cb + n * 8 + qc);
+          ks[n][2 * i] = beta * (__low2float(v) - fk * ks[n][2 * i]);
+          ks[n][2 * i + 1] = beta * (__high2float(v) - fk * ks[n][2 * i + 1]);
+          o[n][2 * i] *= fq;
+          o[n][2 * i + 1] *= fq;
+        }
+      }
+      store_split<4, LV>(sRh + cb, sRl + cb, warp * 16, ks);
+    }
+    __syncthreads();
+    zero(u);
+    mma_triangle<LV>(u, fh, fl, sRh, sRl, warp, cb);
+    load_fragments(fh, fl, unit + 2 * kDeltaTile, warp);
+    store_split<4, LV>(sUh + cb, sUl + cb, warp * 16, u);
+    __syncthreads();                                     // U complete, R no longer read: it takes the weighted U
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const int t = warp * 16 + i * 8 + qr;
-      eb[i] = exp2f(s_sc[t]);
-      rk[i] = s_sc[kQ + t];
-      rq[i] = s_sc[2 * kQ + t];
-      beta[i] = s_sc[3 * kQ + t];
-      wk[i] = exp2f(b_end - s_sc[t]) * rk[i];
-    }
-    float ks[NT][4], o[NT][4];
-    zero(ks);
-    zero(o);
+      const float w = ex2_approx(b_end - s_sc[t]) * s_sc[kQ + t];
 #pragma unroll
-    for (int d = 0; d < DP / 16; ++d) {
-      uint32_t ka[4], qa[4];
-      ldmatrix_x4(ka, addr_a<LD>(sK, warp * 16, d * 16));
-      ldmatrix_x4(qa, addr_a<LD>(sQ, warp * 16, d * 16));
-#pragma unroll
-      for (int n = 0; n < NT / 2; ++n) {
-        uint32_t bh[4], bl[4];
-        ldmatrix_x4_trans(bh, addr_b_t<LV>(sSh, d * 16, n * 16));
-        ldmatrix_x4_trans(bl, addr_b_t<LV>(sSl, d * 16, n * 16));
-        mma_bf16(ks[2 * n], ka, bh[0], bh[1]);
-        mma_bf16(ks[2 * n + 1], ka, bh[2], bh[3]);
-        mma_bf16(o[2 * n], qa, bh[0], bh[1]);
-        mma_bf16(o[2 * n + 1], qa, bh[2], bh[3]);
-        mma_bf16(ks[2 * n], ka, bl[0], bl[1]);
-        mma_bf16(ks[2 * n + 1], ka, bl[2], bl[3]);
-        mma_bf16(o[2 * n], qa, bl[0], bl[1]);
-        mma_bf16(o[2 * n + 1], qa, bl[2], bl[3]);
+      for (int n = 0; n < 4; ++n) {
+        u[n][2 * i] *= w;
+        u[n][2 * i + 1] *= w;
       }
     }
-#pragma unroll
-    for (int n = 0; n < NT; ++n)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int i = e >> 1, t = warp * 16 + i * 8 + qr;
-        const float v = __bfloat162float(sV[t * LV + n * 8 + qc + (e & 1)]);
-        ks[n][e] = beta[i] * (v - eb[i] * rk[i] * ks[n][e]);
-        o[n][e] *= eb[i] * rq[i];
-      }
-    store_split<NT, LV>(sRh, sRl, warp * 16, ks);
-    __syncthreads();
-    float u[NT][4];
-    zero(u);
-    mma_split<LT, LV>(u, sTh, sTl, sRh, sRl, warp * 16, warp + 1);
-    store_split<NT, LV>(sUh, sUl, warp * 16, u);
-    __syncthreads();                                     // U complete, R no longer read: it takes the weighted U
-#pragma unroll
-    for (int n = 0; n < NT; ++n)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) u[n][e] *= wk[e >> 1];
-    store_split<NT, LV>(sRh, sRl, warp * 16, u);
-    mma_split<LT, LV>(o, sPh, sPl, sUh, sUl, warp * 16, warp + 1);
+    store_split<4, LV>(sRh + cb, sRl + cb, warp * 16, u);
+    mma_triangle<LV>(o, fh, fl, sUh, sUl, warp, cb);
     __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.o) + (row0 + t0) * a.ldo + static_cast<int64_t>(h) * Dv + v0;
+    const bool pair = ((a.ldo | Dv) & 1) == 0;
 #pragma unroll
-    for (int n = 0; n < NT; ++n)
+    for (int i = 0; i < 2; ++i) {
+      const int t = warp * 16 + i * 8 + qr;
+      if (t >= rows) continue;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int t = warp * 16 + (e >> 1) * 8 + qr, c = n * 8 + qc + (e & 1);
-        if (t < rows && c < cols) out[t * a.ldo + c] = __float2bfloat16_rn(o[n][e]);
+      for (int n = 0; n < 4; ++n) {
+        const int c = cb + n * 8 + qc;
+        if (pair) {
+          if (c < cols) *reinterpret_cast<uint32_t*>(out + t * a.ldo + c) = bf16_pair(o[n][2 * i], o[n][2 * i + 1]);
+        } else {
+          if (c < cols) out[t * a.ldo + c] = __float2bfloat16_rn(o[n][2 * i]);
+          if (c + 1 < cols) out[t * a.ldo + c + 1] = __float2bfloat16_rn(o[n][2 * i + 1]);
+        }
       }
+    }
     __syncthreads();
-    const float dec = exp2f(b_end);
+    const float dec = ex2_approx(b_end);
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int n = 0; n < NT; ++n)
+      for (int n = 0; n < 4; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) S[m][n][e] *= dec;
 #pragma unroll
@@ -662,10 +735,10 @@ __global__ void __launch_bounds__(128) delta_chunk_kernel(const NxDeltaArgs a, i
 #pragma unroll
       for (int m = 0; m < MT; ++m) ldmatrix_x4_trans(ka[m], addr_a_t<LD>(sK, kk * 16, (warp * MT + m) * 16));
 #pragma unroll
-      for (int n = 0; n < NT / 2; ++n) {
+      for (int n = 0; n < 2; ++n) {
         uint32_t bh[4], bl[4];
-        ldmatrix_x4_trans(bh, addr_b_t<LV>(sRh, kk * 16, n * 16));
-        ldmatrix_x4_trans(bl, addr_b_t<LV>(sRl, kk * 16, n * 16));
+        ldmatrix_x4_trans(bh, addr_b_t<LV>(sRh, kk * 16, cb + n * 16));
+        ldmatrix_x4_trans(bl, addr_b_t<LV>(sRl, kk * 16, cb + n * 16));
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           mma_bf16(S[m][2 * n], ka[m], bh[0], bh[1]);
@@ -680,17 +753,17 @@ __global__ void __launch_bounds__(128) delta_chunk_kernel(const NxDeltaArgs a, i
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int n = 0; n < NT; ++n)
+    for (int n = 0; n < 4; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int r = (warp * MT + m) * 16 + (e >> 1) * 8 + qr, c = n * 8 + qc + (e & 1);
+        const int r = (warp * MT + m) * 16 + (e >> 1) * 8 + qr, c = cb + n * 8 + qc + (e & 1);
         if (r < D && c < cols) pool[static_cast<int64_t>(r) * Dv + v0 + c] = S[m][n][e];
       }
 }
 
 template <int DP>
 int launch_delta(const NxDeltaArgs* a, cudaStream_t st) {
-  constexpr int kBytes = DeltaSmem<DP>::kBytes, kPrep = 2 * kQ * (DP + 8) * 2 + kQ * (kQ + 4) * 4;
+  constexpr int kBytes = DeltaSmem<DP>::kBytes, kPrep = prep_front<DP>() + kQ * (kQ + 4) * 4;
   static bool once = false;
   if (!once) {
     if (cudaFuncSetAttribute(delta_chunk_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, kBytes) != cudaSuccess ||
@@ -700,7 +773,7 @@ int launch_delta(const NxDeltaArgs* a, cudaStream_t st) {
   }
   const int chunks = (a->seg.max_len + kQ - 1) / kQ, col_tiles = (a->vdim + kDeltaCols - 1) / kDeltaCols;
   delta_prep_kernel<DP><<<dim3(chunks, a->heads, a->seg.count), 128, kPrep, st>>>(*a, chunks);
-  delta_chunk_kernel<DP><<<dim3(a->heads * col_tiles, a->seg.count), 128, kBytes, st>>>(*a, chunks, col_tiles);
+  delta_chunk_kernel<DP><<<dim3(a->heads * col_tiles, a->seg.count), 256, kBytes, st>>>(*a, chunks, col_tiles);
   return launch_status();
 }
 

@@ -234,7 +234,7 @@ class HybridEngine(Engine):
         if not self._many.count:
             return
         host = self._host_rows[self.INDEX_ROWS:]
-        flash = long_.count > 0 and a.dim == a.vdim and a.dim in (64, 128) and self._many.count <= 64 and all(
+        flash = long_.count > 0 and a.dim == a.vdim and a.dim in (64, 128) and a.scale > 0 and self._many.count <= 64 and all(
             int(host[1, j]) >= FLASH_MIN and int(host[2, j]) == 0 for j in range(single.count, single.count + self._many.count))
         if not flash:
             M.paged_window_attention(q, *paged, self._many, **kw)
