@@ -130,7 +130,7 @@ __global__ void __launch_bounds__(256, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
   extern __shared__ __align__(16) __nv_bfloat16 sm[];
   __nv_bfloat16 *sB = sm + L::kB, *sC = sm + L::kC, *sX = sm + L::kX, *sXh = sm + L::kXh, *sXl = sm + L::kXl,
                 *sSh = sm + L::kSh, *sSl = sm + L::kSl;
-  __shared__ float s_c[kQ], s_dt[kQ];                    // cumulative log2 decay, step size
+  __shared__ float s_c[kQ], s_dt[kQ], s_w[kQ];           // cumulative log2 decay, step size, weight in the new state
   const int h = blockIdx.x / col_tiles, p0 = (blockIdx.x % col_tiles) * kCols, part = blockIdx.y, sg = blockIdx.z;
   const int len = a.seg.len[sg], t_begin = part * a.span, t_end = min(len, t_begin + a.span);
   if (t_begin >= len || (kLocal && t_end == len)) return;   // the last span's contribution is never needed
@@ -159,28 +159,50 @@ __global__ void __launch_bounds__(256, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
         }
   }
   float total = 0.0f;                                    // log2 decay of the whole span
-  for (int t0 = t_begin; t0 < t_end; t0 += kQ) {
-    const int rows = min(kQ, t_end - t0);
+  auto load_cx = [&](int t0) {
     const __nv_bfloat16* src = xbc + t0 * a.ld_xbc;
-    load_tile<NP>(sB, src + inner + g * N, a.ld_xbc, rows, N, vec_n);
+    const int rows = min(kQ, t_end - t0);
     if (!kLocal) load_tile<NP>(sC, src + inner + (a.groups + g) * N, a.ld_xbc, rows, N, vec_n);
     load_tile<kCols>(sX, src + h * P + p0, a.ld_xbc, rows, cols, vec_p);
-    cp_async_commit();
-    if (threadIdx.x < 32) {
-      float d[2], c[2];
+  };
+  auto load_b = [&](int t0) {
+    load_tile<NP>(sB, xbc + t0 * a.ld_xbc + inner + g * N, a.ld_xbc, min(kQ, t_end - t0), N, vec_n);
+  };
+  float raw[2];                                          // first warp: raw step sizes of the next chunk
+  auto fetch_dt = [&](int t0) {
 #pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int t = lane + 32 * i;
-        d[i] = t < rows ? softplus_exact(__bfloat162float(dtp[(t0 + t) * a.ld_dt]) + dtb) : 0.0f;
-        c[i] = rate * d[i];
-      }
-      scan64(c[0], c[1]);
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        s_dt[lane + 32 * i] = d[i];
-        s_c[lane + 32 * i] = c[i];
-      }
+    for (int i = 0; i < 2; ++i) {
+      const int t = t0 + lane + 32 * i;
+      raw[i] = t < t_end ? __bfloat162float(dtp[t * a.ld_dt]) : -INFINITY;      // softplus(-inf) = 0: no step
     }
+  };
+  auto scan_dt = [&] {
+    float d[2], c[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      d[i] = raw[i] == -INFINITY ? 0.0f : softplus_exact(raw[i] + dtb);
+      c[i] = rate * d[i];
+    }
+    scan64(c[0], c[1]);
+    const float c_last = __shfl_sync(0xffffffffu, c[1], 31);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      s_dt[lane + 32 * i] = d[i];
+      s_c[lane + 32 * i] = c[i];
+      s_w[lane + 32 * i] = ex2_approx(c_last - c[i]) * d[i];
+    }
+  };
+  load_cx(t_begin);
+  load_b(t_begin);
+  cp_async_commit();
+  if (threadIdx.x < 32) {
+    fetch_dt(t_begin);
+    scan_dt();
+    fetch_dt(t_begin + kQ);
+  }
+  for (int t0 = t_begin; t0 < t_end; t0 += kQ) {
+    const int rows = min(kQ, t_end - t0);
+    const bool more = t0 + kQ < t_end;
     if (!kLocal) {
 #pragma unroll
       for (int m = 0; m < MT; ++m) store_split<4, LP>(sSh + cb, sSl + cb, (warp * MT + m) * 16, S[m]);
@@ -191,7 +213,7 @@ __global__ void __launch_bounds__(256, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
     // x weighted for the state update
     for (int i = threadIdx.x; i < kQ * (kCols / 2); i += 256) {
       const int t = i / (kCols / 2), o = t * LP + (i % (kCols / 2)) * 2;
-      const float w = ex2_approx(c_end - s_c[t]) * s_dt[t];
+      const float w = s_w[t];
       const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(sX + o);
       uint32_t hi, lo;
       bf16_split(__low2float(x) * w, __high2float(x) * w, hi, lo);
@@ -278,7 +300,14 @@ __global__ void __launch_bounds__(256, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
         }
       }
     }
-    __syncthreads();                                     // weighted x complete
+    __syncthreads();                                     // weighted x complete; C, x and the step sizes are free again
+    if (more) {
+      load_cx(t0 + kQ);
+      if (threadIdx.x < 32) {
+        scan_dt();
+        fetch_dt(t0 + 2 * kQ);
+      }
+    }
     const float dec = ex2_approx(c_end);
     total += c_end;
 #pragma unroll
@@ -306,7 +335,11 @@ __global__ void __launch_bounds__(256, NP <= 128 ? 2 : 1) ssd_chunk_kernel(const
         }
       }
     }
-    __syncthreads();                                     // before the tiles are loaded over
+    __syncthreads();                                     // B is free
+    if (more) {
+      load_b(t0 + kQ);
+      cp_async_commit();
+    }
   }
   float* dst = kLocal ? part_state : (t_end == len ? pool : nullptr);
   if (dst != nullptr) {
@@ -555,30 +588,28 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const NxDeltaArgs a, in
 
 // ------------------------------------------------------------------------------------------------
 // delta rule, second kernel: the chunks of a segment in order.  grid (heads * column tiles, segments),
-// 8 warps: warp w owns 16 token rows of U and the outputs and DP / 4 rows of the state (w mod 4), 32
-// value columns of both (w / 4).
+// 8 warps: warp w owns 16 token rows of U and the outputs and DP / 4 rows of the state (w mod 4), half
+// of the block's COLS value columns of both (w / 4).
 // ------------------------------------------------------------------------------------------------
-constexpr int kDeltaCols = 64;
-
-template <int DP>
+template <int DP, int COLS>
 struct DeltaSmem {
-  static constexpr int LD = DP + 8, LV = kDeltaCols + 8;
+  static constexpr int LD = DP + 8, LV = COLS + 8;
   static constexpr int kK = 0, kQq = kK + kQ * LD, kRh = kQq + kQ * LD, kRl = kRh + kQ * LV, kUh = kRl + kQ * LV,
                        kUl = kUh + kQ * LV, kSh = kUl + kQ * LV, kSl = kSh + DP * LV, kEnd = kSl + DP * LV;
   static constexpr int kBytes = kEnd * 2;
 };
 
 // d += (ah + al) (bh + bl) up to the product of the two remainders, over the blocks 0 .. row_tile of a lower-triangular tile
-// pair in fragment order; d covers 32 columns
-template <int LV>
-__device__ __forceinline__ void mma_triangle(float (&d)[4][4], const uint4 (&ah)[kQ / 16], const uint4 (&al)[kQ / 16],
+// pair in fragment order; d covers 8 NT columns
+template <int LV, int NT>
+__device__ __forceinline__ void mma_triangle(float (&d)[NT][4], const uint4 (&ah)[kQ / 16], const uint4 (&al)[kQ / 16],
                                              const __nv_bfloat16* bh, const __nv_bfloat16* bl, int row_tile, int col) {
 #pragma unroll
   for (int kk = 0; kk < kQ / 16; ++kk) {
     if (kk > row_tile) break;
     const uint32_t fh[4] = {ah[kk].x, ah[kk].y, ah[kk].z, ah[kk].w}, fl[4] = {al[kk].x, al[kk].y, al[kk].z, al[kk].w};
 #pragma unroll
-    for (int n = 0; n < 2; ++n) {
+    for (int n = 0; n < NT / 2; ++n) {
       uint32_t gh[4], gl[4];
       ldmatrix_x4_trans(gh, addr_b_t<LV>(bh, kk * 16, col + n * 16));
       ldmatrix_x4_trans(gl, addr_b_t<LV>(bl, kk * 16, col + n * 16));
@@ -600,56 +631,57 @@ __device__ __forceinline__ void load_fragments(uint4 (&hi)[kQ / 16], uint4 (&lo)
   }
 }
 
-template <int DP>
+template <int DP, int COLS>
 __global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) delta_chunk_kernel(const NxDeltaArgs a, int chunks, int col_tiles) {
-  using L = DeltaSmem<DP>;
-  constexpr int LD = L::LD, LV = L::LV, MT = DP / 64;
+  using L = DeltaSmem<DP, COLS>;
+  constexpr int LD = L::LD, LV = L::LV, MT = DP / 64, NT = COLS / 16;    // NT: 8-column tiles per warp
   extern __shared__ __align__(16) __nv_bfloat16 sm[];
   __nv_bfloat16 *sK = sm + L::kK, *sQ = sm + L::kQq, *sRh = sm + L::kRh, *sRl = sm + L::kRl, *sUh = sm + L::kUh, *sUl = sm + L::kUl,
                 *sSh = sm + L::kSh, *sSl = sm + L::kSl;
   __nv_bfloat16* sV = sUh;             // v is consumed before U is written
   __shared__ __align__(16) float s_sc[4 * kQ];           // cumulative log2 decay | 1/|k| | scaled 1/|q| | beta
-  const int h = blockIdx.x / col_tiles, v0 = (blockIdx.x % col_tiles) * kDeltaCols, sg = blockIdx.y;
+  const int h = blockIdx.x / col_tiles, v0 = (blockIdx.x % col_tiles) * COLS, sg = blockIdx.y;
   const int len = a.seg.len[sg];
   if (len <= 0) return;
-  const int D = a.dim, Dv = a.vdim, cols = min(kDeltaCols, Dv - v0), hk = h / (a.heads / a.kv_heads), kcols = a.kv_heads * D;
-  const int warp = (threadIdx.x >> 5) & 3, cb = (threadIdx.x >> 7) * 32, lane = threadIdx.x & 31, qr = lane >> 2, qc = (lane & 3) * 2;
+  const int D = a.dim, Dv = a.vdim, cols = min(COLS, Dv - v0), hk = h / (a.heads / a.kv_heads), kcols = a.kv_heads * D;
+  const int warp = (threadIdx.x >> 5) & 3, cb = (threadIdx.x >> 7) * (COLS / 2), lane = threadIdx.x & 31, qr = lane >> 2, qc = (lane & 3) * 2;
   const int64_t row0 = a.seg.row0[sg];
   const bool aligned = (a.ld_qkv & 7) == 0 && (reinterpret_cast<uintptr_t>(a.qkv) & 15) == 0;
   const bool vec_d = aligned && (D & 7) == 0, vec_v = aligned && (Dv & 7) == 0 && ((2 * kcols) & 7) == 0;
   float* pool = a.state + (static_cast<int64_t>(a.seg.seq[sg]) * a.heads + h) * D * Dv;
   const bool fresh = a.seg.pos[sg] == 0;
-  float S[MT][4][4];
+  float S[MT][NT][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int n = 0; n < 4; ++n)
+    for (int n = 0; n < NT; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int r = (warp * MT + m) * 16 + (e >> 1) * 8 + qr, c = cb + n * 8 + qc + (e & 1);
         S[m][n][e] = (!fresh && r < D && c < cols) ? pool[static_cast<int64_t>(r) * Dv + v0 + c] : 0.0f;
       }
+  const __nv_bfloat16* qsrc = static_cast<const __nv_bfloat16*>(a.qkv) + row0 * a.ld_qkv + hk * D;
+  load_tile<DP>(sQ, qsrc, a.ld_qkv, min(kQ, len), D, vec_d);
   for (int ch = 0; ch * kQ < len; ++ch) {
     const int t0 = ch * kQ, rows = min(kQ, len - t0);
     const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(a.qkv) + (row0 + t0) * a.ld_qkv;
     const __nv_bfloat16* unit = static_cast<const __nv_bfloat16*>(a.scratch) +
                                 ((static_cast<int64_t>(sg) * chunks + ch) * a.heads + h) * kDeltaUnit;
-    load_tile<DP>(sQ, src + hk * D, a.ld_qkv, rows, D, vec_d);
     load_tile<DP>(sK, src + kcols + hk * D, a.ld_qkv, rows, D, vec_d);
-    load_tile<kDeltaCols>(sV, src + 2 * kcols + h * Dv + v0, a.ld_qkv, rows, cols, vec_v);
+    load_tile<COLS>(sV, src + 2 * kcols + h * Dv + v0, a.ld_qkv, rows, cols, vec_v);
     if (threadIdx.x < kQ) cp_async16(s_sc + threadIdx.x * 4, reinterpret_cast<const float*>(unit + 4 * kDeltaTile) + threadIdx.x * 4);
     cp_async_commit();
     uint4 fh[kQ / 16], fl[kQ / 16];                      // rows of T, later of P
     load_fragments(fh, fl, unit, warp);
 #pragma unroll
-    for (int m = 0; m < MT; ++m) store_split<4, LV>(sSh + cb, sSl + cb, (warp * MT + m) * 16, S[m]);
+    for (int m = 0; m < MT; ++m) store_split<NT, LV>(sSh + cb, sSl + cb, (warp * MT + m) * 16, S[m]);
     cp_async_wait<0>();
     __syncthreads();
     const float b_end = s_sc[kQ - 1];
-    float o[4][4], u[4][4];
+    float o[NT][4], u[NT][4];
     zero(o);
     {
-      float ks[4][4];
+      float ks[NT][4];
       zero(ks);
 #pragma unroll
       for (int d = 0; d < DP / 16; ++d) {
@@ -657,7 +689,7 @@ __global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) delta_chunk_kernel(con
         ldmatrix_x4(ka, addr_a<LD>(sK, warp * 16, d * 16));
         ldmatrix_x4(qa, addr_a<LD>(sQ, warp * 16, d * 16));
 #pragma unroll
-        for (int n = 0; n < 2; ++n) {
+        for (int n = 0; n < NT / 2; ++n) {
           uint32_t bh[4], bl[4];
           ldmatrix_x4_trans(bh, addr_b_t<LV>(sSh, d * 16, cb + n * 16));
           ldmatrix_x4_trans(bl, addr_b_t<LV>(sSl, d * 16, cb + n * 16));
@@ -676,7 +708,7 @@ __global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) delta_chunk_kernel(con
         const int t = warp * 16 + i * 8 + qr;
         const float eb = ex2_approx(s_sc[t]), fk = eb * s_sc[kQ + t], fq = eb * s_sc[2 * kQ + t], beta = s_sc[3 * kQ + t];
 #pragma unroll
-        for (int n = 0; n < 4; ++n) {
+        for (int n = 0; n < NT; ++n) {
           const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(sV + t * LV + cb + n * 8 + qc);
           ks[n][2 * i] = beta * (__low2float(v) - fk * ks[n][2 * i]);
           ks[n][2 * i + 1] = beta * (__high2float(v) - fk * ks[n][2 * i + 1]);
@@ -684,26 +716,27 @@ __global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) delta_chunk_kernel(con
           o[n][2 * i + 1] *= fq;
         }
       }
-      store_split<4, LV>(sRh + cb, sRl + cb, warp * 16, ks);
+      store_split<NT, LV>(sRh + cb, sRl + cb, warp * 16, ks);
     }
     __syncthreads();
     zero(u);
-    mma_triangle<LV>(u, fh, fl, sRh, sRl, warp, cb);
+    mma_triangle<LV, NT>(u, fh, fl, sRh, sRl, warp, cb);
     load_fragments(fh, fl, unit + 2 * kDeltaTile, warp);
-    store_split<4, LV>(sUh + cb, sUl + cb, warp * 16, u);
+    store_split<NT, LV>(sUh + cb, sUl + cb, warp * 16, u);
     __syncthreads();                                     // U complete, R no longer read: it takes the weighted U
+    if (t0 + kQ < len) load_tile<DP>(sQ, qsrc + (t0 + kQ) * a.ld_qkv, a.ld_qkv, min(kQ, len - t0 - kQ), D, vec_d);
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const int t = warp * 16 + i * 8 + qr;
       const float w = ex2_approx(b_end - s_sc[t]) * s_sc[kQ + t];
 #pragma unroll
-      for (int n = 0; n < 4; ++n) {
+      for (int n = 0; n < NT; ++n) {
         u[n][2 * i] *= w;
         u[n][2 * i + 1] *= w;
       }
     }
-    store_split<4, LV>(sRh + cb, sRl + cb, warp * 16, u);
-    mma_triangle<LV>(o, fh, fl, sUh, sUl, warp, cb);
+    store_split<NT, LV>(sRh + cb, sRl + cb, warp * 16, u);
+    mma_triangle<LV, NT>(o, fh, fl, sUh, sUl, warp, cb);
     __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.o) + (row0 + t0) * a.ldo + static_cast<int64_t>(h) * Dv + v0;
     const bool pair = ((a.ldo | Dv) & 1) == 0;
 #pragma unroll
@@ -711,7 +744,7 @@ __global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) delta_chunk_kernel(con
       const int t = warp * 16 + i * 8 + qr;
       if (t >= rows) continue;
 #pragma unroll
-      for (int n = 0; n < 4; ++n) {
+      for (int n = 0; n < NT; ++n) {
         const int c = cb + n * 8 + qc;
         if (pair) {
           if (c < cols) *reinterpret_cast<uint32_t*>(out + t * a.ldo + c) = bf16_pair(o[n][2 * i], o[n][2 * i + 1]);
@@ -726,7 +759,7 @@ __global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) delta_chunk_kernel(con
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int n = 0; n < 4; ++n)
+      for (int n = 0; n < NT; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) S[m][n][e] *= dec;
 #pragma unroll
@@ -735,7 +768,7 @@ __global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) delta_chunk_kernel(con
 #pragma unroll
       for (int m = 0; m < MT; ++m) ldmatrix_x4_trans(ka[m], addr_a_t<LD>(sK, kk * 16, (warp * MT + m) * 16));
 #pragma unroll
-      for (int n = 0; n < 2; ++n) {
+      for (int n = 0; n < NT / 2; ++n) {
         uint32_t bh[4], bl[4];
         ldmatrix_x4_trans(bh, addr_b_t<LV>(sRh, kk * 16, cb + n * 16));
         ldmatrix_x4_trans(bl, addr_b_t<LV>(sRl, kk * 16, cb + n * 16));
@@ -753,7 +786,7 @@ __global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) delta_chunk_kernel(con
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int n = 0; n < 4; ++n)
+    for (int n = 0; n < NT; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int r = (warp * MT + m) * 16 + (e >> 1) * 8 + qr, c = cb + n * 8 + qc + (e & 1);
@@ -761,20 +794,32 @@ __global__ void __launch_bounds__(256, DP <= 128 ? 2 : 1) delta_chunk_kernel(con
       }
 }
 
-template <int DP>
-int launch_delta(const NxDeltaArgs* a, cudaStream_t st) {
-  constexpr int kBytes = DeltaSmem<DP>::kBytes, kPrep = prep_front<DP>() + kQ * (kQ + 4) * 4;
+template <int DP, int COLS>
+int launch_delta_chunks(const NxDeltaArgs* a, int chunks, cudaStream_t st) {
+  constexpr int kBytes = DeltaSmem<DP, COLS>::kBytes;
   static bool once = false;
   if (!once) {
-    if (cudaFuncSetAttribute(delta_chunk_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, kBytes) != cudaSuccess ||
-        cudaFuncSetAttribute(delta_prep_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPrep) != cudaSuccess)
-      return -2;
+    if (cudaFuncSetAttribute(delta_chunk_kernel<DP, COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, kBytes) != cudaSuccess) return -2;
     once = true;
   }
-  const int chunks = (a->seg.max_len + kQ - 1) / kQ, col_tiles = (a->vdim + kDeltaCols - 1) / kDeltaCols;
-  delta_prep_kernel<DP><<<dim3(chunks, a->heads, a->seg.count), 128, kPrep, st>>>(*a, chunks);
-  delta_chunk_kernel<DP><<<dim3(a->heads * col_tiles, a->seg.count), 256, kBytes, st>>>(*a, chunks, col_tiles);
+  const int col_tiles = (a->vdim + COLS - 1) / COLS;
+  delta_chunk_kernel<DP, COLS><<<dim3(a->heads * col_tiles, a->seg.count), 256, kBytes, st>>>(*a, chunks, col_tiles);
   return launch_status();
+}
+
+template <int DP>
+int launch_delta(const NxDeltaArgs* a, cudaStream_t st) {
+  constexpr int kPrep = prep_front<DP>() + kQ * (kQ + 4) * 4;
+  static bool once = false;
+  if (!once) {
+    if (cudaFuncSetAttribute(delta_prep_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPrep) != cudaSuccess) return -2;
+    once = true;
+  }
+  const int chunks = (a->seg.max_len + kQ - 1) / kQ;
+  delta_prep_kernel<DP><<<dim3(chunks, a->heads, a->seg.count), 128, kPrep, st>>>(*a, chunks);
+  // the chunks of a segment are a chain: while the blocks do not fill the GPU, narrower column tiles shorten every link
+  const int wide = a->heads * ((a->vdim + 63) / 64) * a->seg.count;
+  return wide < kNumSmsB200 && a->vdim > 32 ? launch_delta_chunks<DP, 32>(a, chunks, st) : launch_delta_chunks<DP, 64>(a, chunks, st);
 }
 
 }  // namespace
