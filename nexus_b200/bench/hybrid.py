@@ -102,7 +102,6 @@ def model_lines(sizes, iters=10):
 # ------------------------------------------------------------------------------------------ kernels
 def kernel_cases():
     """name -> (launch, flops, bytes)."""
-    from ..infer.engine import EngineConfig  # noqa: F401
     from ..ops import _cuda as K
     from ..ops import _infer as I
     from ..ops import _mixers as M
