@@ -76,6 +76,8 @@ struct DevParams {
   unsigned int* amax_out;  // max |out| as float bits (may be null)
   int tma_store;           // BF16 out (and aux_out) leave through shared memory and tiled TMA stores
   int n_fastest;           // consecutive work units walk along N (A tile reused from L2) instead of along M
+  const int32_t* row_groups;  // grouped form: which B each block of `group_rows` rows meets (negative: none)
+  int group_rows;
   // All-gather fused into the GEMM (nx_gemm_ag): A is this rank's [M][lda] gather buffer; the last `ag_copiers`
   // CTAs of the grid push this rank's row block into every peer's buffer and raise per-chunk flags there, while
   // the GEMM CTAs start with the local rows and take the other ranks' rows in ring order as their flags come up.
@@ -98,6 +100,7 @@ struct DevParams {
 
 struct Unit {
   int m0, n0, batch, slice, kb_begin, kb_end;
+  int group;  // batch index of B; negative: the unit is skipped
 };
 
 // Operands / output spread over the ranks of a group (peer-mapped memory).  Tiles never straddle a
@@ -141,6 +144,7 @@ __device__ __forceinline__ Unit decode_unit(const DevParams& p, int u) {
     if (w.m0 >= p.m) w.m0 -= p.m;
   }
   w.n0 = tn;  // multiplied by BN by the caller
+  w.group = p.row_groups != nullptr ? __ldg(p.row_groups + w.m0 / p.group_rows) : w.batch;
   w.kb_begin = w.slice * p.kb_per_slice;
   w.kb_end = min(p.kb_total, w.kb_begin + p.kb_per_slice);
   return w;
@@ -507,6 +511,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
       const int ag_epoch = p.ag_ranks > 1 ? *reinterpret_cast<const volatile int*>(p.ag_counter) + 1 : 0;
       for (int u = unit_first; u < p.num_units && ok; u += unit_step) {
         Unit w = decode_unit<kTileM>(p, u);
+        if (w.group < 0) continue;
         w.m0 += m_off;
         const int n0 = w.n0 * BN;
         if (p.ag_ranks > 1 && !ag_wait_rows(p, w.m0, ag_epoch, abort_flag)) {
@@ -543,11 +548,11 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
                 tma_load_3d_pair(sa + j * (64 * kBK * 2), &tmap_a, bar, w.m0 + 64 * j, k0, w.batch);
             }
             if (!B_MN) {
-              tma_load_3d_pair(sb, &tmap_b, bar, k0, bn0, w.batch);
+              tma_load_3d_pair(sb, &tmap_b, bar, k0, bn0, w.group);
             } else {
 #pragma unroll
               for (int j = 0; j < C::kBRows / 64; ++j)
-                tma_load_3d_pair(sb + j * (64 * kBK * 2), &tmap_b, bar, bn0 + 64 * j, k0, w.batch);
+                tma_load_3d_pair(sb + j * (64 * kBK * 2), &tmap_b, bar, bn0 + 64 * j, k0, w.group);
             }
             if (++stage == C::kStages) {
               stage = 0;
@@ -588,11 +593,11 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
               tma_load_3d(sa + j * (64 * kBK * 2), ma, &full_bar[stage], am0 + 64 * j, ak0, w.batch);
           }
           if (!B_MN) {
-            tma_load_3d(sb, mb, &full_bar[stage], bk0, bn0, w.batch);
+            tma_load_3d(sb, mb, &full_bar[stage], bk0, bn0, w.group);
           } else {
 #pragma unroll
             for (int j = 0; j < BN / 64; ++j)
-              tma_load_3d(sb + j * (64 * kBK * 2), mb, &full_bar[stage], bn0 + 64 * j, bk0, w.batch);
+              tma_load_3d(sb + j * (64 * kBK * 2), mb, &full_bar[stage], bn0 + 64 * j, bk0, w.group);
           }
           if (++stage == C::kStages) {
             stage = 0;
@@ -628,6 +633,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
               const long long t_begin = clock64();)
       for (int u = unit_first; u < p.num_units && ok; u += unit_step) {
         Unit w = decode_unit<kTileM>(p, u);
+        if (w.group < 0) continue;
         NX_PROF(const long long c0 = clock64();)
         if (!__all_sync(0xffffffffu, mbar_wait_bounded(&tempty_bar[acc], acc_phase ^ 1u, abort_flag))) {
           if (leader) atomicCAS(p.status, 0, kStatusTimeoutMma);
@@ -707,6 +713,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
       int tile_parity = 0;
       for (int u = unit_first; u < p.num_units; u += unit_step, tile_parity ^= 1) {
         Unit w = decode_unit<kTileM>(p, u);
+        if (w.group < 0) continue;
         w.m0 += m_off;
         const int n0 = w.n0 * BN;
         const int row = w.m0 + quarter * 32 + lane;
@@ -810,6 +817,9 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
           if (p.act == NX_ACT_GELU) {
 #pragma unroll
             for (int j = 0; j < 32; ++j) v[j] = gelu_tanh_f(v[j]);
+          } else if (p.act == NX_ACT_RELU2) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = fmaxf(v[j], 0.0f) * fmaxf(v[j], 0.0f);
           }
           stage_row32_bf16(st_out, lane, v);
           if (++gpos == group || last_chunk) {
@@ -852,6 +862,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
             long long e_bias = 0; long long e_stage = 0; long long e_fence = 0; long long e_issue = 0;)
     for (int u = unit_first; u < p.num_units; u += unit_step) {
       Unit w = decode_unit<kTileM>(p, u);
+      if (w.group < 0) continue;
       w.m0 += m_off;
       const int n0 = w.n0 * BN;
       const int row = w.m0 + quarter * 32 + lane;
@@ -1029,6 +1040,9 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
         } else if (p.act == NX_ACT_SILU) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] = silu_f(v[j]);
+        } else if (p.act == NX_ACT_RELU2) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = fmaxf(v[j], 0.0f) * fmaxf(v[j], 0.0f);
         }
         if (p.residual != nullptr && row_ok) {
           float q[32];
@@ -1207,6 +1221,7 @@ __global__ void splitk_reduce_kernel(const float* __restrict__ ws, void* out, in
     if (act == NX_ACT_GELU) s = gelu_tanh_f(s);
     else if (act == NX_ACT_RELU) s = fmaxf(s, 0.0f);
     else if (act == NX_ACT_SILU) s = silu_f(s);
+    else if (act == NX_ACT_RELU2) s = fmaxf(s, 0.0f) * fmaxf(s, 0.0f);
     const int64_t off = static_cast<int64_t>(r) * ldo + c;
     if (out_dtype == NX_F32) {
       float* o = reinterpret_cast<float*>(out);
@@ -1245,7 +1260,7 @@ extern "C" int nx_splitk_reduce_epilogue(const float* workspace, void* out, int 
                                          nx_stream_t stream) {
   const int64_t total = static_cast<int64_t>(m) * n;
   if (total == 0) return 0;
-  if (act != NX_ACT_NONE && act != NX_ACT_GELU && act != NX_ACT_RELU && act != NX_ACT_SILU) return -1;
+  if (act != NX_ACT_NONE && act != NX_ACT_GELU && act != NX_ACT_RELU && act != NX_ACT_SILU && act != NX_ACT_RELU2) return -1;
   int blocks = static_cast<int>(std::min<int64_t>((total + 255) / 256, 148 * 8));
   splitk_reduce_kernel<<<blocks, 256, 0, static_cast<cudaStream_t>(stream)>>>(workspace, out, out_dtype, ldo, m, n,
                                                                               split_k, accumulate, bias, bias_dtype, act);
@@ -1308,6 +1323,12 @@ int gemm_impl(const NxGemmArgs* a, const NxGemmAg* ag, nx_stream_t stream_, cons
   if (split > 1 && a->accumulate == 2 && a->out_dtype != NX_F32) return -1;
   if (split > 1 && a->accumulate != 2 && a->workspace == nullptr) return -1;
 
+  const bool grouped = a->row_groups != nullptr;
+  if (grouped && (fp8 || a->a_mn_major || split > 1 || ag != nullptr || rs != nullptr ||
+                  (a->group_rows != kBM && a->group_rows != 2 * kBM) || a->m % a->group_rows))
+    return -1;
+  const int batch = grouped ? 1 : a->batch;  // of A and the output; B has a->batch matrices either way
+
   int bn = a->block_n;
   if (bn != 128 && bn != 256) bn = (a->n >= 256) ? 256 : 128;
 
@@ -1315,7 +1336,7 @@ int gemm_impl(const NxGemmArgs* a, const NxGemmAg* ag, nx_stream_t stream_, cons
   static const bool single_only = std::getenv("NX_GEMM_SINGLE_CTA") != nullptr;  // measurement switch
   static bool pair_ok = true;  // cleared when the device cannot place clusters of two
   const bool pair = bn == 256 && !fp8 && a->m >= 2 * kBM && pair_ok && (!single_only || ag != nullptr || rs != nullptr) &&
-                    (a->max_ctas <= 0 || a->max_ctas >= 2);
+                    (a->max_ctas <= 0 || a->max_ctas >= 2) && !(grouped && a->group_rows < 2 * kBM);
   if ((ag != nullptr || rs != nullptr) && !pair) return -3;  // the fused forms run on the CTA-pair kernel only
   const int tile_m = pair ? 2 * kBM : kBM;
 
@@ -1336,11 +1357,13 @@ int gemm_impl(const NxGemmArgs* a, const NxGemmAg* ag, nx_stream_t stream_, cons
   p.ldo = a->ldo;
   p.ld_aux = a->ld_aux;
   p.ld_res = a->ld_res;
-  p.stride_o = a->batch > 1 ? a->stride_o : 0;
+  p.stride_o = batch > 1 ? a->stride_o : 0;
   p.m = a->m;
   p.n = a->n;
   p.k = a->k;
-  p.batch = a->batch;
+  p.batch = batch;
+  p.row_groups = a->row_groups;
+  p.group_rows = grouped ? a->group_rows : 1;
   p.out_dtype = a->out_dtype;
   p.bias_dtype = a->bias_dtype;
   p.res_dtype = a->res_dtype;
@@ -1351,7 +1374,7 @@ int gemm_impl(const NxGemmArgs* a, const NxGemmAg* ag, nx_stream_t stream_, cons
   p.tiles_n = (a->n + bn - 1) / bn;
   p.kb_total = kb_total;
   p.kb_per_slice = kb_per;
-  p.num_units = p.tiles_m * p.tiles_n * split * a->batch;
+  p.num_units = p.tiles_m * p.tiles_n * split * batch;
   p.alpha = a->alpha;
   p.fp8 = fp8 ? 1 : 0;
   p.bk_elems = bk;
@@ -1383,13 +1406,13 @@ int gemm_impl(const NxGemmArgs* a, const NxGemmAg* ag, nx_stream_t stream_, cons
                                                                : CU_TENSOR_MAP_DATA_TYPE_FLOAT16);
   const int eb = fp8 ? 1 : 2;
   CUtensorMap ta, tb;
-  const uint64_t sa = a->batch > 1 ? static_cast<uint64_t>(a->stride_a) : 0;
+  const uint64_t sa = batch > 1 ? static_cast<uint64_t>(a->stride_a) : 0;
   const uint64_t sb = a->batch > 1 ? static_cast<uint64_t>(a->stride_b) : 0;
   int rc;
   if (!a->a_mn_major)
-    rc = nx::make_tensor_map_3d(&ta, dt, eb, a->a, a->k, a->m, a->batch, a->lda, sa, bk, kBM);
+    rc = nx::make_tensor_map_3d(&ta, dt, eb, a->a, a->k, a->m, batch, a->lda, sa, bk, kBM);
   else
-    rc = nx::make_tensor_map_3d(&ta, dt, 2, a->a, a->m, a->k, a->batch, a->lda, sa, 64, kBK);
+    rc = nx::make_tensor_map_3d(&ta, dt, 2, a->a, a->m, a->k, batch, a->lda, sa, 64, kBK);
   if (rc != 0) return rc;
   if (!a->b_mn_major)
     rc = nx::make_tensor_map_3d(&tb, dt, eb, a->b, a->k, a->n, a->batch, a->ldb, sb, bk, pair ? bn / 2 : bn);
@@ -1400,14 +1423,14 @@ int gemm_impl(const NxGemmArgs* a, const NxGemmAg* ag, nx_stream_t stream_, cons
   // BF16 results leave through shared memory and tiled stores (full-line writes) when the layout allows a map
   CUtensorMap to, tx;
   const bool can_tma_out = a->out_dtype == NX_BF16 && split == 1 && a->accumulate == 0 && (a->ldo & 7) == 0 &&
-                           (reinterpret_cast<uintptr_t>(a->out) & 15) == 0 && (a->batch == 1 || (a->stride_o & 7) == 0) &&
+                           (reinterpret_cast<uintptr_t>(a->out) & 15) == 0 && (batch == 1 || (a->stride_o & 7) == 0) &&
                            (a->aux_out == nullptr || ((a->ld_aux & 7) == 0 && (reinterpret_cast<uintptr_t>(a->aux_out) & 15) == 0 &&
-                                                      a->batch == 1));
+                                                      batch == 1));
   p.tma_store = 0;
   static const bool direct_only = std::getenv("NX_GEMM_DIRECT_STORE") != nullptr;  // measurement switch
   if (can_tma_out && !direct_only) {
-    const uint64_t so = a->batch > 1 ? static_cast<uint64_t>(a->stride_o) : 0;
-    rc = nx::make_tensor_map_3d(&to, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a->out, a->n, a->m, a->batch, a->ldo, so, 32, 32,
+    const uint64_t so = batch > 1 ? static_cast<uint64_t>(a->stride_o) : 0;
+    rc = nx::make_tensor_map_3d(&to, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a->out, a->n, a->m, batch, a->ldo, so, 32, 32,
                                 CU_TENSOR_MAP_SWIZZLE_64B);
     if (rc == 0 && a->aux_out != nullptr)
       rc = nx::make_tensor_map_3d(&tx, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a->aux_out, a->n, a->m, 1, a->ld_aux, 0, 32, 32,
@@ -1443,7 +1466,7 @@ int gemm_impl(const NxGemmArgs* a, const NxGemmAg* ag, nx_stream_t stream_, cons
     const bool fast = (rs != nullptr || !generic_only) && p.tma_store && a->residual == nullptr && a->scale_a == nullptr &&
                       a->scale_b == nullptr && a->amax_out == nullptr && (reinterpret_cast<uintptr_t>(a->bias) & 15) == 0 &&
                       (a->aux_in == nullptr || (reinterpret_cast<uintptr_t>(a->aux_in) & 15) == 0) &&
-                      (a->act == NX_ACT_NONE || a->act == NX_ACT_GELU || (a->act == NX_ACT_DGELU && a->aux_in != nullptr));
+                      (a->act == NX_ACT_NONE || a->act == NX_ACT_GELU || a->act == NX_ACT_RELU2 || (a->act == NX_ACT_DGELU && a->aux_in != nullptr));
 #define NX_PAIR(AM_, BM_) \
   rc = fast ? launch_pair<AM_, BM_, true>(ta, tb, p, fmt, sms, stream, po, px) \
             : launch_pair<AM_, BM_, false>(ta, tb, p, fmt, sms, stream, po, px)

@@ -403,6 +403,7 @@ skinny_gemm_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx, const __nv_
       if (act == NX_ACT_GELU) v = gelu_tanh_f(v);
       else if (act == NX_ACT_RELU) v = fmaxf(v, 0.0f);
       else if (act == NX_ACT_SILU) v = silu_f(v);
+      else if (act == NX_ACT_RELU2) v = fmaxf(v, 0.0f) * fmaxf(v, 0.0f);
       if (residual) v += Num<YT>::load(residual + i * ldr + col);
       Num<YT>::store(y + i * ldy + col, v);
     }

@@ -28,22 +28,45 @@ __global__ void residual_norm_kernel(const NxResidualNormArgs a) {
     for (int c = threadIdx.x * V; c < cols; c += blockDim.x * V) {
       float v[V];
       load_vec<T, V>(e + c, v);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] *= a.embed_scale;
       store_vec<float, V>(xr + c, v);
       store_vec<float, V>(s_row + c, v);
 #pragma unroll
       for (int j = 0; j < V; ++j) ss += v[j] * v[j];
     }
-  } else if (a.y != nullptr) {
+  } else if (a.y != nullptr || a.experts != nullptr) {
     const T* yr = static_cast<const T*>(a.y) + r * a.ldy;
+    const float yg = a.y_gate != nullptr ? a.y_gate[r] : 1.0f;
     float sy = 0.0f;
     for (int c = threadIdx.x * V; c < cols; c += blockDim.x * V) {
       float v[V];
-      load_vec<T, V>(yr + c, v);
+      if (a.experts != nullptr) {
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[j] = 0.0f;
+        for (int k = 0; k < a.top; ++k) {
+          float u[V];
+          load_vec<T, V>(static_cast<const T*>(a.experts) + static_cast<int64_t>(a.expert_slots[r * a.top + k]) * a.ld_experts + c, u);
+#pragma unroll
+          for (int j = 0; j < V; ++j) v[j] += u[j];
+        }
+        if (a.y != nullptr) {
+          float u[V];
+          load_vec<T, V>(yr + c, u);
+#pragma unroll
+          for (int j = 0; j < V; ++j) v[j] = v[j] * a.expert_scale + u[j] * yg;
+        } else {
+#pragma unroll
+          for (int j = 0; j < V; ++j) v[j] *= a.expert_scale;
+        }
+      } else {
+        load_vec<T, V>(yr + c, v);
+      }
       store_vec<float, V>(s_row + c, v);
 #pragma unroll
       for (int j = 0; j < V; ++j) sy += v[j] * v[j];
     }
-    const float inv = 1.0f / sqrtf(block_sum(sy, s_red) * inv_cols + a.eps);
+    const float inv = a.res_mult / sqrtf(block_sum(sy, s_red) * inv_cols + a.eps);
     for (int c = threadIdx.x * V; c < cols; c += blockDim.x * V) {   // each thread re-reads its own columns
       float v[V], xv[V], w[V];
       load_vec<float, V>(s_row + c, v);
@@ -74,6 +97,29 @@ __global__ void residual_norm_kernel(const NxResidualNormArgs a) {
       store_vec<T, V>(o + c, v);
     }
     for (int c = cols + threadIdx.x; c < a.ldh; c += blockDim.x) Num<T>::store(o + c, 0.0f);
+  }
+  if (a.scatter != nullptr) {
+    for (int k = 0; k < a.top; ++k) {
+      T* o = static_cast<T*>(a.scatter) + static_cast<int64_t>(a.scatter_slots[r * a.top + k]) * a.ldh;
+      for (int c = threadIdx.x * V; c < cols; c += blockDim.x * V) {
+        float v[V];
+        load_vec<float, V>(s_row + c, v);
+        store_vec<T, V>(o + c, v);
+      }
+      for (int c = cols + threadIdx.x; c < a.ldh; c += blockDim.x) Num<T>::store(o + c, 0.0f);
+    }
+  }
+  if (a.w_dot != nullptr) {
+    float sd = 0.0f;
+    for (int c = threadIdx.x * V; c < cols; c += blockDim.x * V) {
+      float v[V], w[V];
+      load_vec<float, V>(s_row + c, v);
+      load_vec<float, V>(a.w_dot + c, w);
+#pragma unroll
+      for (int j = 0; j < V; ++j) sd += v[j] * w[j];
+    }
+    sd = block_sum(sd, s_red);
+    if (threadIdx.x == 0) a.dot_out[r] = sigmoid_exact(sd);
   }
   if (a.h != nullptr) {
     const float inv = 1.0f / sqrtf(block_sum(ss, s_red) * inv_cols + a.eps);
@@ -125,6 +171,106 @@ __global__ void rope_append_kernel(const NxRopeAppendArgs a) {
     kc[o] = row[a.k_off + o];
   }
   for (int i = threadIdx.x; i < a.kv_heads * a.vdim; i += blockDim.x) vc[i] = row[a.v_off + i];
+}
+
+// ------------------------------------------------------------------------------------------------
+// latent attention: norms of both latents, rotation of the shared key part, cache append, gate; one block per row
+// ------------------------------------------------------------------------------------------------
+template <typename T, int V>
+__device__ __forceinline__ float sum_squares(const T* p, int n) {
+  float ss = 0.0f;
+  for (int c = threadIdx.x * V; c < n; c += blockDim.x * V) {
+    float v[V];
+    load_vec<T, V>(p + c, v);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += v[j] * v[j];
+  }
+  return ss;
+}
+
+template <typename T, int V>
+__global__ void latent_prep_kernel(const NxLatentPrepArgs a) {
+  __shared__ float s_red[32];
+  const int64_t r = blockIdx.x;
+  const T* row = static_cast<const T*>(a.proj) + r * a.ld;
+  const int64_t pos = a.positions[r], slot = a.slots[r];
+  const T *q = row + a.q_off, *k = row + a.c_off;
+  const float inv_q = 1.0f / sqrtf(block_sum(sum_squares<T, V>(q, a.q_rank), s_red) / static_cast<float>(a.q_rank) + a.eps);
+  const float inv_k = 1.0f / sqrtf(block_sum(sum_squares<T, V>(k, a.kv_rank), s_red) / static_cast<float>(a.kv_rank) + a.eps);
+  T* cq = static_cast<T*>(a.cq) + r * a.ldq;
+  for (int c = threadIdx.x * V; c < a.q_rank; c += blockDim.x * V) {
+    float v[V], w[V];
+    load_vec<T, V>(q + c, v);
+    load_vec<float, V>(a.w_q + c, w);
+#pragma unroll
+    for (int j = 0; j < V; ++j) v[j] *= inv_q * w[j];
+    store_vec<T, V>(cq + c, v);
+  }
+  for (int c = a.q_rank + threadIdx.x; c < a.ldq; c += blockDim.x) Num<T>::store(cq + c, 0.0f);
+  T* cache = slot >= 0 ? static_cast<T*>(a.cache) + slot * a.ld_cache : nullptr;
+  T* lat = a.lat != nullptr ? static_cast<T*>(a.lat) + r * a.ld_cache : nullptr;
+  for (int c = threadIdx.x * V; c < a.kv_rank; c += blockDim.x * V) {
+    float v[V], w[V];
+    load_vec<T, V>(k + c, v);
+    load_vec<float, V>(a.w_kv + c, w);
+#pragma unroll
+    for (int j = 0; j < V; ++j) v[j] *= inv_k * w[j];
+    if (cache != nullptr) store_vec<T, V>(cache + c, v);
+    if (lat != nullptr) store_vec<T, V>(lat + c, v);
+  }
+  const int half = a.rot_dims / 2;
+  for (int j = threadIdx.x; j < half; j += blockDim.x) {
+    const float u = Num<T>::load(row + a.r_off + j), v = Num<T>::load(row + a.r_off + half + j);
+    const float c = a.cos_t[pos * half + j], s = a.sin_t[pos * half + j];
+    const float y0 = u * c - v * s, y1 = v * c + u * s;
+    if (cache != nullptr) {
+      Num<T>::store(cache + a.rot_col + j, y0);
+      Num<T>::store(cache + a.rot_col + half + j, y1);
+    }
+    if (lat != nullptr) {
+      Num<T>::store(lat + a.rot_col + j, y0);
+      Num<T>::store(lat + a.rot_col + half + j, y1);
+    }
+  }
+  if (lat != nullptr) {
+    for (int c = a.kv_rank + threadIdx.x; c < a.rot_col; c += blockDim.x) Num<T>::store(lat + c, 0.0f);
+    for (int c = a.rot_col + a.rot_dims + threadIdx.x; c < a.ld_cache; c += blockDim.x) Num<T>::store(lat + c, 0.0f);
+  }
+  for (int h = threadIdx.x; h < a.heads; h += blockDim.x)
+    a.gate[r * a.heads + h] = sigmoid_exact(Num<T>::load(row + a.g_off + h));
+}
+
+// V adjacent pairs per thread; a block takes blockDim.y rows
+template <typename T, int V>
+__global__ void rope_heads_kernel(const T* __restrict__ src, int64_t ld_src, int src_head, int src_off, T* dst, int64_t ld_dst,
+                                  int dst_head, int dst_off, int rows, int heads, int rot_dims, int width,
+                                  const int32_t* __restrict__ positions, const float* __restrict__ cos_t,
+                                  const float* __restrict__ sin_t) {
+  const int64_t r = blockIdx.x * static_cast<int64_t>(blockDim.y) + threadIdx.y;
+  if (r >= rows) return;
+  const int half = rot_dims / 2, per = half / V;
+  const int64_t pos = positions[r];
+  for (int i = threadIdx.x; i < heads * per; i += blockDim.x) {
+    const int h = i / per, j = (i % per) * V;
+    const T* s = src + r * ld_src + static_cast<int64_t>(h) * src_head + src_off + j;
+    T* d = dst + r * ld_dst + static_cast<int64_t>(h) * dst_head + dst_off + j;
+    float u[V], v[V], c[V], sn[V];
+    load_vec<T, V>(s, u);
+    load_vec<T, V>(s + half, v);
+    load_vec<float, V>(cos_t + pos * half + j, c);
+    load_vec<float, V>(sin_t + pos * half + j, sn);
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      const float a = u[k] * c[k] - v[k] * sn[k];
+      v[k] = v[k] * c[k] + u[k] * sn[k];
+      u[k] = a;
+    }
+    store_vec<T, V>(d, u);
+    store_vec<T, V>(d + half, v);
+  }
+  const int rest = width - rot_dims;
+  for (int i = threadIdx.x; i < heads * rest; i += blockDim.x)
+    Num<T>::store(dst + r * ld_dst + static_cast<int64_t>(i / rest) * dst_head + dst_off + rot_dims + i % rest, 0.0f);
 }
 
 // ------------------------------------------------------------------------------------------------
@@ -330,7 +476,8 @@ int launch_conv(const NxConvArgs* a, cudaStream_t st) {
 
 template <typename T>
 int launch_residual(const NxResidualNormArgs* a, cudaStream_t st) {
-  const bool vec = a->cols % 4 == 0 && (a->y == nullptr || a->ldy % 4 == 0) && a->ldh % 4 == 0;
+  const bool vec = a->cols % 4 == 0 && (a->y == nullptr || a->ldy % 4 == 0) && a->ldh % 4 == 0 &&
+                   (a->experts == nullptr || a->ld_experts % 4 == 0);
   const int per = vec ? 4 : 1;
   int threads = ((a->cols / per + 1) / 2 + 31) / 32 * 32;
   threads = std::max(64, std::min(512, threads));
@@ -352,7 +499,10 @@ int launch_residual(const NxResidualNormArgs* a, cudaStream_t st) {
 extern "C" int nx_residual_norm(const NxResidualNormArgs* a, nx_stream_t stream) {
   if (a == nullptr || a->cols <= 0 || a->x == nullptr) return -1;
   if (a->rows <= 0) return 0;
-  if (a->y != nullptr && a->w_post == nullptr) return -1;
+  if ((a->y != nullptr || a->experts != nullptr) && a->w_post == nullptr) return -1;
+  if (a->experts != nullptr && (a->expert_slots == nullptr || a->top < 1)) return -1;
+  if (a->scatter != nullptr && (a->scatter_slots == nullptr || a->top < 1 || a->ldh < a->cols)) return -1;
+  if (a->w_dot != nullptr && a->dot_out == nullptr) return -1;
   if (a->h != nullptr && a->w_next == nullptr) return -1;
   if ((a->h != nullptr || a->x_cast != nullptr) && a->ldh < a->cols) return -1;
   if (a->table != nullptr && a->tokens == nullptr) return -1;
@@ -372,6 +522,51 @@ extern "C" int nx_rope_append(const NxRopeAppendArgs* a, nx_stream_t stream) {
   if (a->dtype == NX_BF16) rope_append_kernel<__nv_bfloat16><<<a->rows, threads, 0, st>>>(*a);
   else if (a->dtype == NX_F32) rope_append_kernel<float><<<a->rows, threads, 0, st>>>(*a);
   else return -1;
+  return launch_status();
+}
+
+extern "C" int nx_latent_prep(const NxLatentPrepArgs* a, nx_stream_t stream) {
+  if (a == nullptr || a->q_rank <= 0 || a->kv_rank <= 0 || a->heads <= 0 || a->rot_dims < 0 || (a->rot_dims & 1)) return -1;
+  if (a->ldq < a->q_rank || a->rot_col < a->kv_rank || a->ld_cache < a->rot_col + a->rot_dims) return -1;
+  if (a->rows <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool vec = ((a->q_rank | a->kv_rank | a->q_off | a->c_off) & 3) == 0 && ((a->ld | a->ldq | a->ld_cache) & 3) == 0 &&
+                   (reinterpret_cast<uintptr_t>(a->proj) & 15) == 0;
+  const int most = std::max(a->q_rank, a->kv_rank) / (vec ? 4 : 1);
+  const int threads = std::max(64, std::min(256, (most + 31) / 32 * 32));
+  if (a->dtype == NX_BF16) {
+    if (vec) latent_prep_kernel<__nv_bfloat16, 4><<<a->rows, threads, 0, st>>>(*a);
+    else latent_prep_kernel<__nv_bfloat16, 1><<<a->rows, threads, 0, st>>>(*a);
+  } else if (a->dtype == NX_F32) {
+    if (vec) latent_prep_kernel<float, 4><<<a->rows, threads, 0, st>>>(*a);
+    else latent_prep_kernel<float, 1><<<a->rows, threads, 0, st>>>(*a);
+  } else {
+    return -1;
+  }
+  return launch_status();
+}
+
+extern "C" int nx_rope_heads(const void* src, int64_t ld_src, int src_head, int src_off, void* dst, int64_t ld_dst,
+                             int dst_head, int dst_off, int rows, int heads, int rot_dims, int width,
+                             const int32_t* positions, const float* cos_t, const float* sin_t, int dtype,
+                             nx_stream_t stream) {
+  if (rot_dims < 0 || (rot_dims & 1) || width < rot_dims || heads <= 0) return -1;
+  if (rows <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int half = rot_dims / 2;
+  const bool vec = half % 8 == 0 && ((ld_src | src_head | src_off | ld_dst | dst_head | dst_off) & 7) == 0 &&
+                   ((reinterpret_cast<uintptr_t>(src) | reinterpret_cast<uintptr_t>(dst)) & 15) == 0;
+  const int work = std::max(heads * half / (vec ? 8 : 1), 32);
+  const int tx = std::min(256, (work + 31) / 32 * 32), ty = 256 / tx;
+  const dim3 block(tx, ty), grid((rows + ty - 1) / ty);
+#define NX_RH(T_, V_)                                                                                                   \
+  rope_heads_kernel<T_, V_><<<grid, block, 0, st>>>(static_cast<const T_*>(src), ld_src, src_head, src_off,             \
+                                                    static_cast<T_*>(dst), ld_dst, dst_head, dst_off, rows, heads,      \
+                                                    rot_dims, width, positions, cos_t, sin_t)
+  if (dtype == NX_BF16) { if (vec) NX_RH(__nv_bfloat16, 8); else NX_RH(__nv_bfloat16, 1); }
+  else if (dtype == NX_F32) { if (vec) NX_RH(float, 8); else NX_RH(float, 1); }
+  else return -1;
+#undef NX_RH
   return launch_status();
 }
 

@@ -5,7 +5,10 @@
 // kernels (which also serve expert parallelism over peer memory); the expert FFN itself is a strided
 // batched tcgen05 GEMM over the padded buffers.
 // Parity: src/moe/moe.cpp (router, capacity, permutation) of the reference, which runs on the CPU.
+// Experts that a table picks by token id need no router: one launch sorts a step's assignments for every layer, and the
+// serving forms of the expert products (few rows per expert; FP32) live here too.
 #include "common.cuh"
+#include "mixer_common.cuh"
 #include "nx_api_moe.h"
 
 namespace {
@@ -174,7 +177,199 @@ __global__ void moe_gate_grad_kernel(const __nv_bfloat16* __restrict__ dy, const
   acc = warp_sum(acc);
   if (lane == 0) dgate[i] = acc;
 }
+
+// ------------------------------------------------------------------------------------------------
+// experts by token id: one block per layer counts, places and scatters its assignments
+// ------------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(1024) moe_table_route_kernel(const __grid_constant__ NxTableRouteArgs a) {
+  extern __shared__ int s_cnt[];               // [experts] counts, then the next free slot
+  __shared__ int s_warp[32], s_total;
+  const NxTableRouteLayer& L = a.layer[blockIdx.x];
+  const int total = a.n * L.top, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  for (int e = tid; e < L.experts; e += blockDim.x) s_cnt[e] = 0;
+  for (int i = tid; i < L.max_slots; i += blockDim.x) L.rows[i] = -1;
+  __syncthreads();
+#pragma unroll 4
+  for (int i = tid; i < total; i += blockDim.x) {
+    const int t = a.tokens[i / L.top];
+    const int e = t >= 0 && t < a.vocab ? L.table[static_cast<int64_t>(t) * L.top + i % L.top] : 0;
+    L.slots[i] = e;                            // the expert for now, read again by this thread
+    atomicAdd(&s_cnt[e], 1);
+  }
+  __syncthreads();
+  int base = 0;
+  for (int e0 = 0; e0 < L.experts; e0 += blockDim.x) {
+    const int e = e0 + tid, n = e < L.experts ? s_cnt[e] : 0, padded = (n + a.align - 1) / a.align * a.align;
+    int incl = padded;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, incl, o);
+      if (lane >= o) incl += v;
+    }
+    if (lane == 31) s_warp[warp] = incl;
+    __syncthreads();
+    int before = base;
+    for (int w = 0; w < warp; ++w) before += s_warp[w];
+    const int first = before + incl - padded;
+    if (e < L.experts) {
+      L.start[e] = first;
+      L.count[e] = n;
+      s_cnt[e] = first;
+      for (int g = first / a.align; g < (first + padded) / a.align; ++g) L.groups[g] = e;
+    }
+    if (tid == static_cast<int>(blockDim.x) - 1) s_total = before + incl;
+    __syncthreads();
+    base = s_total;
+  }
+  for (int g = base / a.align + tid; g < L.max_slots / a.align; g += blockDim.x) L.groups[g] = -1;
+#pragma unroll 4
+  for (int i = tid; i < total; i += blockDim.x) {
+    const int s = atomicAdd(&s_cnt[L.slots[i]], 1);
+    L.slots[i] = s;
+    L.rows[s] = i / L.top;
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// expert product, few rows: a warp owns 16 rows of one expert's weights and streams them once for up to 8 NT tokens.  A
+// thread's 16-byte load covers eight neighbours along K; the sum over K may take them in any order as long as both
+// operands agree, so each load is two k-steps of the tensor-core tile as it is.
+// ------------------------------------------------------------------------------------------------
+template <int NT>
+__device__ __forceinline__ void expert_rows(const NxExpertGemmArgs& a, const __nv_bfloat16* w, int n0, int first, int cnt) {
+  const int lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const __nv_bfloat16 *w0 = w + static_cast<int64_t>(n0 + g) * a.ldw + t * 8, *w1 = w0 + 8 * a.ldw;
+  const bool in0 = n0 + g < a.n, in1 = n0 + g + 8 < a.n;
+  const __nv_bfloat16* x[NT];
+  float acc[NT][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i) {
+    const int s = first + min(i * 8 + g, cnt - 1);           // rows past the last repeat it; they are not stored
+    x[i] = static_cast<const __nv_bfloat16*>(a.x) + static_cast<int64_t>(a.rows != nullptr ? a.rows[s] : s) * a.ldx + t * 8;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[i][e] = 0.0f;
+  }
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll(NT == 1 ? 4 : 2)
+  for (int k0 = 0; k0 < a.k; k0 += 64) {
+    uint4 wa[2], wb[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const bool ink = k0 + h * 32 + t * 8 < a.k;
+      wa[h] = ink && in0 ? __ldg(reinterpret_cast<const uint4*>(w0 + k0 + h * 32)) : zero;
+      wb[h] = ink && in1 ? __ldg(reinterpret_cast<const uint4*>(w1 + k0 + h * 32)) : zero;
+    }
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const uint4 v = k0 + h * 32 + t * 8 < a.k ? __ldg(reinterpret_cast<const uint4*>(x[i] + k0 + h * 32)) : zero;
+        const uint32_t f0[4] = {wa[h].x, wb[h].x, wa[h].y, wb[h].y}, f1[4] = {wa[h].z, wb[h].z, wa[h].w, wb[h].w};
+        mma_bf16(acc[i], f0, v.x, v.y);
+        mma_bf16(acc[i], f1, v.z, v.w);
+      }
+  }
+  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out);
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int s = i * 8 + t * 2 + (e & 1), n = n0 + g + (e >> 1) * 8;
+      float v = acc[i][e];
+      if (a.act == NX_ACT_RELU2) v = fmaxf(v, 0.0f) * fmaxf(v, 0.0f);
+      if (s < cnt && n < a.n) out[static_cast<int64_t>(first + s) * a.ldo + n] = __float2bfloat16_rn(v);
+    }
+}
+
+__global__ void __launch_bounds__(128) expert_skinny_kernel(const NxExpertGemmArgs a) {
+  const int e = blockIdx.y, n0 = (blockIdx.x * 4 + (threadIdx.x >> 5)) * 16;
+  int cnt = a.count[e];
+  if (cnt <= 0 || n0 >= a.n) return;
+  int first = a.start[e];
+  const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(a.w) + static_cast<int64_t>(e) * a.stride_w;
+  for (; cnt > 0; cnt -= 32, first += 32) {
+    if (cnt <= 8) expert_rows<1>(a, w, n0, first, cnt);
+    else if (cnt <= 16) expert_rows<2>(a, w, n0, first, cnt);
+    else expert_rows<4>(a, w, n0, first, min(cnt, 32));
+  }
+}
+
+// FP32: 32 slots x 64 columns per block, 16 x 16 threads of 2 x 4
+__global__ void __launch_bounds__(256) expert_f32_kernel(const NxExpertGemmArgs a) {
+  __shared__ float s_x[16][33], s_w[16][65];
+  const int e = a.groups[blockIdx.y];
+  if (e < 0) return;
+  const int s0 = blockIdx.y * 32, n0 = blockIdx.x * 64, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  const float *x = static_cast<const float*>(a.x), *w = static_cast<const float*>(a.w) + static_cast<int64_t>(e) * a.stride_w;
+  const int last = a.start[e] + a.count[e];
+  float acc[2][4] = {{0.0f, 0.0f, 0.0f, 0.0f}, {0.0f, 0.0f, 0.0f, 0.0f}};
+  for (int k0 = 0; k0 < a.k; k0 += 16) {
+    for (int i = threadIdx.x; i < 32 * 16; i += 256) {
+      const int s = s0 + i / 16, k = k0 + i % 16;
+      const bool in = s < last && k < a.k;
+      const int64_t row = in ? (a.rows != nullptr ? a.rows[s] : s) : 0;
+      s_x[i % 16][i / 16] = in ? x[row * a.ldx + k] : 0.0f;
+    }
+    for (int i = threadIdx.x; i < 64 * 16; i += 256) {
+      const int n = n0 + i / 16, k = k0 + i % 16;
+      s_w[i % 16][i / 16] = n < a.n && k < a.k ? w[static_cast<int64_t>(n) * a.ldw + k] : 0.0f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k)
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(s_x[k][ty * 2 + i], s_w[k][tx * 4 + j], acc[i][j]);
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int s = s0 + ty * 2 + i, n = n0 + tx * 4 + j;
+      float v = acc[i][j];
+      if (a.act == NX_ACT_RELU2) v = fmaxf(v, 0.0f) * fmaxf(v, 0.0f);
+      if (s < last && n < a.n) static_cast<float*>(a.out)[static_cast<int64_t>(s) * a.ldo + n] = v;
+    }
+}
+
+int check_expert(const NxExpertGemmArgs* a) {
+  if (a == nullptr || a->x == nullptr || a->w == nullptr || a->out == nullptr || a->start == nullptr || a->count == nullptr) return -1;
+  if (a->experts <= 0 || a->n <= 0 || a->k <= 0 || (a->act != NX_ACT_NONE && a->act != NX_ACT_RELU2)) return -1;
+  return 0;
+}
 }  // namespace
+
+extern "C" int nx_moe_table_route(const NxTableRouteArgs* a, nx_stream_t stream) {
+  if (a == nullptr || a->layers < 0 || a->layers > NX_TABLE_LAYERS || a->align < 1 || a->vocab < 1) return -1;
+  if (a->layers == 0 || a->n <= 0) return 0;
+  int most = 0;
+  for (int l = 0; l < a->layers; ++l) {
+    const NxTableRouteLayer& L = a->layer[l];
+    if (L.experts < 1 || L.experts > 8192 || L.top < 1 || L.max_slots % a->align) return -1;
+    // every expert that is used leaves fewer than `align` slots empty
+    const int64_t total = static_cast<int64_t>(a->n) * L.top, used = total < L.experts ? total : L.experts;
+    if ((total + used * (a->align - 1)) / a->align * a->align > L.max_slots) return -1;
+    most = most > L.experts ? most : L.experts;
+  }
+  moe_table_route_kernel<<<a->layers, 1024, most * sizeof(int), static_cast<cudaStream_t>(stream)>>>(*a);
+  return launch_status();
+}
+
+extern "C" int nx_expert_skinny(const NxExpertGemmArgs* a, nx_stream_t stream) {
+  if (check_expert(a) || (a->k & 7) || (a->ldx & 7) || (a->ldw & 7) || (a->stride_w & 7) || a->experts > 65535) return -1;
+  if ((reinterpret_cast<uintptr_t>(a->x) & 15) || (reinterpret_cast<uintptr_t>(a->w) & 15)) return -1;
+  expert_skinny_kernel<<<dim3((a->n + 63) / 64, a->experts), 128, 0, static_cast<cudaStream_t>(stream)>>>(*a);
+  return launch_status();
+}
+
+extern "C" int nx_expert_f32(const NxExpertGemmArgs* a, nx_stream_t stream) {
+  if (check_expert(a) || a->groups == nullptr || a->align != 32 || a->tiles < 0 || a->tiles > 65535) return -1;
+  if (a->tiles == 0) return 0;
+  expert_f32_kernel<<<dim3((a->n + 63) / 64, a->tiles), 256, 0, static_cast<cudaStream_t>(stream)>>>(*a);
+  return launch_status();
+}
 
 extern "C" int nx_moe_topk(const float* logits, int tokens, int experts, int k, int32_t* expert, float* gate,
                            nx_stream_t stream) {

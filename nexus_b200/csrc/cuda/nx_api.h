@@ -15,7 +15,8 @@ extern "C" {
 typedef void* nx_stream_t;
 
 enum NxDType { NX_BF16 = 0, NX_F32 = 1, NX_F16 = 2, NX_E4M3 = 3, NX_E5M2 = 4 };
-enum NxAct { NX_ACT_NONE = 0, NX_ACT_GELU = 1, NX_ACT_RELU = 2, NX_ACT_DGELU = 3, NX_ACT_SILU = 4 };
+enum NxAct { NX_ACT_NONE = 0, NX_ACT_GELU = 1, NX_ACT_RELU = 2, NX_ACT_DGELU = 3, NX_ACT_SILU = 4,
+             NX_ACT_RELU2 = 5 /* square of relu */ };
 
 // out[b][m][n] = epilogue( alpha * sum_k A[b][m][k] * B[b][n][k] )
 // Operand memory: a_mn_major == 0 -> A is [M][lda] (K contiguous); 1 -> A is [K][lda] (M contiguous).
@@ -49,6 +50,12 @@ typedef struct NxGemmArgs {
   const float* scale_a;   // [M] per-row dequantisation scale of A, may be null
   const float* scale_b;   // [N] per-row dequantisation scale of B, may be null
   float* amax_out;        // receives max |out| (must be zeroed by the caller), may be null
+  // Grouped form (may be null): A and out are one matrix of M rows, B is [batch][N][ldb], and the row tile
+  // [i * group_rows, (i + 1) * group_rows) is multiplied by B[row_groups[i]]; a negative entry skips the tile (its output
+  // rows are not written).  group_rows is 128 or 256; the entries are read on the device, so they may change under a
+  // captured graph.  No split-K, no FP8.
+  const int32_t* row_groups;
+  int32_t group_rows;
 } NxGemmArgs;
 
 int nx_gemm(const NxGemmArgs* args, nx_stream_t stream);
@@ -56,7 +63,7 @@ int nx_gemm(const NxGemmArgs* args, nx_stream_t stream);
 int nx_splitk_reduce(const float* workspace, void* out, int out_dtype, int64_t ldo, int m, int n, int split_k,
                      int accumulate, nx_stream_t stream);
 // The same, with the epilogue the split GEMM could not apply itself: out = act(sum of slices + bias) (+ out when
-// `accumulate`).  act: NX_ACT_NONE / GELU / RELU / SILU.
+// `accumulate`).  act: NX_ACT_NONE / GELU / RELU / SILU / RELU2.
 int nx_splitk_reduce_epilogue(const float* workspace, void* out, int out_dtype, int64_t ldo, int m, int n, int split_k,
                               int accumulate, const void* bias, int bias_dtype, int act, nx_stream_t stream);
 int nx_sm_count(void);

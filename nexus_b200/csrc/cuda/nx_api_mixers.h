@@ -27,17 +27,31 @@ typedef struct NxSegments {
 } NxSegments;
 
 typedef struct NxResidualNormArgs {
-  float* x;                // [rows, cols] residual stream, updated in place (written when `table` or `y` is given)
-  const int32_t* tokens;   // with `table`: x = table[tokens[row]]
+  float* x;                // [rows, cols] residual stream, updated in place (written when `table`, `y` or `experts` is given)
+  const int32_t* tokens;   // with `table`: x = embed_scale * table[tokens[row]]
   const void* table;       // [vocab, cols] dtype, may be null
-  const void* y;           // [rows, ldy] sublayer output, may be null: x += rms(y) * w_post
+  const void* y;           // [rows, ldy] sublayer output, may be null: x += res_mult * rms(y) * w_post
   const float* w_post;
   const float* w_next;     // may be null; else h = rms(x) * w_next
   void* h;                 // [rows, ldh]; columns cols..ldh are zeroed
   void* x_cast;            // [rows, ldh], may be null: x in the activation dtype
   int64_t ldy, ldh;
   int32_t rows, cols, dtype;
-  float eps;
+  float eps, embed_scale, res_mult;
+  // Sublayer output of a layer of experts, may be null: expert_scale * sum_j experts[expert_slots[row * top + j]], plus
+  // y_gate[row] * y[row] when `y` is given too (y_gate null: plain y).
+  const void* experts;     // [slots, ld_experts]
+  const int32_t* expert_slots;
+  const float* y_gate;
+  int64_t ld_experts;
+  int32_t top;
+  float expert_scale;
+  // dot_out[row] = sigmoid(x . w_dot), may be null
+  const float* w_dot;
+  float* dot_out;
+  // copies of the x_cast row at scatter[scatter_slots[row * top + j]], may be null (pitch ldh)
+  void* scatter;
+  const int32_t* scatter_slots;
 } NxResidualNormArgs;
 int nx_residual_norm(const NxResidualNormArgs* args, nx_stream_t stream);
 
@@ -54,6 +68,36 @@ typedef struct NxRopeAppendArgs {
   void* v_cache;           // [slots, kv_heads, vdim]
 } NxRopeAppendArgs;
 int nx_rope_append(const NxRopeAppendArgs* args, nx_stream_t stream);
+
+// What lies between the down projections of latent attention and its cache: the query latent and the key / value latent
+// are normed, the shared key part is rotated, latent and key part go to the cache (and to `lat`), the output gate's
+// sigmoid is taken.
+typedef struct NxLatentPrepArgs {
+  const void* proj;        // [rows, ld]; the parts of a row start at q_off, c_off, r_off, g_off
+  int64_t ld;
+  int32_t q_off, c_off, r_off, g_off;
+  int32_t rows, q_rank, kv_rank, rot_dims, heads, dtype;
+  float eps;
+  const float* w_q;        // [q_rank]
+  const float* w_kv;       // [kv_rank]
+  const int32_t* positions;
+  const int32_t* slots;    // cache slot per row, negative: nothing is appended
+  const float* cos_t;      // [max_pos, rot_dims / 2]
+  const float* sin_t;
+  void* cq;                // [rows, ldq]: normed query latent, columns q_rank..ldq are zeroed
+  int64_t ldq;
+  void* cache;             // [slots, ld_cache]: latent, at column rot_col the rotated key part; other columns stay as they are
+  int64_t ld_cache;
+  int32_t rot_col;
+  void* lat;               // [rows, ld_cache], may be null: the cache row, its other columns zero
+  float* gate;             // [rows, heads]: sigmoid
+} NxLatentPrepArgs;
+int nx_latent_prep(const NxLatentPrepArgs* args, nx_stream_t stream);
+// Rotates `rot_dims` columns of every head: src [rows, ld_src], head h at h * src_head + src_off; dst likewise (the same
+// place is allowed).  Columns rot_dims..width of dst become zeros.
+int nx_rope_heads(const void* src, int64_t ld_src, int src_head, int src_off, void* dst, int64_t ld_dst, int dst_head,
+                  int dst_off, int rows, int heads, int rot_dims, int width, const int32_t* positions, const float* cos_t,
+                  const float* sin_t, int dtype, nx_stream_t stream);
 
 // y = silu(causal_conv(x) + bias) per channel; state [slots, taps - 1, channels] holds the last taps - 1 inputs.
 typedef struct NxConvArgs {
@@ -150,6 +194,9 @@ typedef struct NxPagedWindowArgs {
   int32_t heads, kv_heads, dim, vdim, block_size, max_blocks, window, splits, dtype;
   float scale, softcap, out_scale;
   NxSegments seg;
+  int64_t k_pitch, v_pitch;  // elements between cache slots: kv_heads * dim and kv_heads * vdim, or the row of a latent cache,
+                             // whose values are the leading columns of its keys
+  const float* gate;         // [rows, heads] factor of the output, may be null
 } NxPagedWindowArgs;
 // one-row segments, BF16: tensor-core tiles of up to 16 query heads of a KV head against 64 keys, split over the keys
 int nx_paged_window_decode(const NxPagedWindowArgs* args, nx_stream_t stream);

@@ -26,6 +26,47 @@ int nx_moe_assign_groups(int32_t* expert, const int32_t* order, int tokens, int 
 int nx_moe_gate_grad(const void* dy, const void* expert_out, const int32_t* expert, const int32_t* slot, float* dgate,
                      int tokens, int k, int d, int capacity, nx_stream_t stream);
 
+
+// Experts by token id, for all layers of a step in one launch.  Layer l: table [vocab, top] gives every token's experts;
+// its assignments (token t, choice j) are sorted by expert, every expert's slots starting at a multiple of `align`:
+//   slots[t * top + j]   slot of the assignment          rows[slot]    its token, -1 between the experts
+//   start[e], count[e]   first slot and number of slots  groups[slot / align]   expert, -1 past the last one
+// The order of one expert's assignments among themselves is not fixed.  max_slots is a multiple of align and at least
+// moe_table_slots(tokens * top, experts, align).
+#define NX_TABLE_LAYERS 32
+typedef struct NxTableRouteLayer {
+  const int32_t* table;
+  int32_t* slots;
+  int32_t* rows;
+  int32_t* start;
+  int32_t* count;
+  int32_t* groups;
+  int32_t experts, top, max_slots;
+} NxTableRouteLayer;
+typedef struct NxTableRouteArgs {
+  const int32_t* tokens;
+  int32_t n, vocab, layers, align;
+  NxTableRouteLayer layer[NX_TABLE_LAYERS];
+} NxTableRouteArgs;
+int nx_moe_table_route(const NxTableRouteArgs* args, nx_stream_t stream);
+
+// out[slot] = act(W[e] x[row of slot]) for every slot of every expert; `rows` null: row = slot.  act: NX_ACT_NONE or RELU2.
+typedef struct NxExpertGemmArgs {
+  const void* x;           // [., ldx]
+  const int32_t* rows;
+  const void* w;           // [experts, n, ldw]
+  void* out;               // [slots, ldo]
+  const int32_t* start;
+  const int32_t* count;
+  const int32_t* groups;   // FP32 form: expert per tile of `align` slots
+  int64_t ldx, ldw, stride_w, ldo;
+  int32_t experts, n, k, act, tiles, align;
+} NxExpertGemmArgs;
+// few rows per expert, BF16: the weights stream through registers once per 32 rows; k, ldx, ldw multiples of 8
+int nx_expert_skinny(const NxExpertGemmArgs* args, nx_stream_t stream);
+// FP32, align 32
+int nx_expert_f32(const NxExpertGemmArgs* args, nx_stream_t stream);
+
 #ifdef __cplusplus
 }
 #endif

@@ -67,12 +67,13 @@ __device__ __forceinline__ int log2_of(int n) { return (n & (n - 1)) == 0 ? 31 -
 struct KvSource {
   const __nv_bfloat16 *k, *v;
   const int32_t* bt;
-  int block_size, shift, kv_heads, hk, dim, vdim;      // shift: log2 of a power-of-two block size, else -1
+  int64_t k_pitch, v_pitch;                            // elements between cache slots
+  int block_size, shift, dim, vdim;                    // shift: log2 of a power-of-two block size, else -1
   __device__ __forceinline__ KvSource(const NxPagedWindowArgs& a, int seq, int head)
-      : k(static_cast<const __nv_bfloat16*>(a.k_cache)), v(static_cast<const __nv_bfloat16*>(a.v_cache)),
-        bt(a.block_table + static_cast<int64_t>(seq) * a.max_blocks), block_size(a.block_size),
-        shift(log2_of(a.block_size)), kv_heads(a.kv_heads), hk(head), dim(a.dim),
-        vdim(a.vdim) {}
+      : k(static_cast<const __nv_bfloat16*>(a.k_cache) + static_cast<int64_t>(head) * a.dim),
+        v(static_cast<const __nv_bfloat16*>(a.v_cache) + static_cast<int64_t>(head) * a.vdim),
+        bt(a.block_table + static_cast<int64_t>(seq) * a.max_blocks), k_pitch(a.k_pitch), v_pitch(a.v_pitch),
+        block_size(a.block_size), shift(log2_of(a.block_size)), dim(a.dim), vdim(a.vdim) {}
   __device__ __forceinline__ int64_t slot(int j) const {
     if (shift >= 0) return (static_cast<int64_t>(bt[j >> shift]) << shift) + (j & (block_size - 1));
     return static_cast<int64_t>(bt[j / block_size]) * block_size + j % block_size;
@@ -93,10 +94,10 @@ __device__ __forceinline__ void stage_kv(__nv_bfloat16* dst, const KvSource& src
     const int key = i / CH, c = (i % CH) * 8, j = k0 + key;
     __nv_bfloat16 *dk = dst + key * LD + c, *dv = dk + kKeys * LD;
     const bool in = j <= last;
-    const int64_t row = in ? src.slot(j) * src.kv_heads + src.hk : 0;
-    if (in && c < src.dim) copy8(dk, src.k + row * src.dim, c, src.dim);
+    const int64_t slot = in ? src.slot(j) : 0;
+    if (in && c < src.dim) copy8(dk, src.k + slot * src.k_pitch, c, src.dim);
     else *reinterpret_cast<uint4*>(dk) = make_uint4(0u, 0u, 0u, 0u);
-    if (in && c < src.vdim) copy8(dv, src.v + row * src.vdim, c, src.vdim);
+    if (in && c < src.vdim) copy8(dv, src.v + slot * src.v_pitch, c, src.vdim);
     else *reinterpret_cast<uint4*>(dv) = make_uint4(0u, 0u, 0u, 0u);
   }
 }
@@ -257,7 +258,8 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
     sum[i] += __shfl_xor_sync(0xffffffffu, sum[i], 2);
     if (qpos[i] < 0) continue;
     const int m = warp * 16 + i * 8 + (lane >> 2);
-    const float inv = a.out_scale / sum[i];
+    const float g = a.gate != nullptr ? a.gate[(row0 + m / rt) * a.heads + h0 + m % rt] : 1.0f;
+    const float inv = a.out_scale * g / sum[i];
     __nv_bfloat16* op = out + (row0 + m / rt) * a.ldo + static_cast<int64_t>(h0 + m % rt) * a.vdim;
 #pragma unroll
     for (int n = 0; n < DP / 8; ++n) {
@@ -403,8 +405,9 @@ paged_decode_mma_kernel(const NxPagedWindowArgs a, int head_tiles) {
       go += sO[(w * 16 + m) * DP + d] * f;
     }
     if (a.splits == 1) {
+      const float g = a.gate != nullptr ? a.gate[row * a.heads + h0 + m] : 1.0f;
       static_cast<__nv_bfloat16*>(a.out)[row * a.ldo + static_cast<int64_t>(h0 + m) * a.vdim + d] =
-          __float2bfloat16_rn(go / gl * a.out_scale);
+          __float2bfloat16_rn(go / gl * a.out_scale * g);
     } else {
       const int64_t pi = (static_cast<int64_t>(sg) * a.heads + h0 + m) * a.splits + blockIdx.z;
       a.part_o[pi * a.vdim + d] = go;
@@ -419,7 +422,8 @@ paged_decode_mma_kernel(const NxPagedWindowArgs a, int head_tiles) {
 __global__ void paged_decode_merge_kernel(const NxPagedWindowArgs a) {
   const int sg = blockIdx.x, h = blockIdx.y;
   if (a.seg.len[sg] <= 0) return;
-  const int64_t base = (static_cast<int64_t>(sg) * a.heads + h) * a.splits;
+  const int64_t base = (static_cast<int64_t>(sg) * a.heads + h) * a.splits, row = a.seg.row0[sg];
+  const float g = a.gate != nullptr ? a.gate[row * a.heads + h] : 1.0f;
   float gm = -INFINITY;
   for (int s = 0; s < a.splits; ++s) gm = fmaxf(gm, a.part_ml[(base + s) * 2]);
   for (int d = threadIdx.x; d < a.vdim; d += blockDim.x) {
@@ -430,15 +434,15 @@ __global__ void paged_decode_merge_kernel(const NxPagedWindowArgs a) {
       gl += a.part_ml[(base + s) * 2 + 1] * w;
       go += a.part_o[(base + s) * a.vdim + d] * w;
     }
-    static_cast<__nv_bfloat16*>(a.out)[static_cast<int64_t>(a.seg.row0[sg]) * a.ldo + static_cast<int64_t>(h) * a.vdim + d] =
-        __float2bfloat16_rn(go / gl * a.out_scale);
+    static_cast<__nv_bfloat16*>(a.out)[row * a.ldo + static_cast<int64_t>(h) * a.vdim + d] =
+        __float2bfloat16_rn(go / gl * a.out_scale * g);
   }
 }
 
 // ------------------------------------------------------------------------------------------------
 // FP32: one block per (row, head), a key per thread for the scores, a value column per thread for the sum
 // ------------------------------------------------------------------------------------------------
-constexpr int kF32Cols = 4;   // value columns per thread: vdim <= 512
+constexpr int kF32Cols = 8;   // value columns per thread: vdim <= 1024
 
 __global__ void __launch_bounds__(128) paged_window_f32_kernel(const NxPagedWindowArgs a) {
   extern __shared__ __align__(16) float sf[];
@@ -454,7 +458,9 @@ __global__ void __launch_bounds__(128) paged_window_f32_kernel(const NxPagedWind
   const float* kc = static_cast<const float*>(a.k_cache);
   const float* vc = static_cast<const float*>(a.v_cache);
   for (int d = tid; d < a.dim; d += 128) sQ[d] = static_cast<const float*>(a.q)[row * a.ldq + static_cast<int64_t>(h) * a.dim + d];
-  float acc[kF32Cols] = {0.0f, 0.0f, 0.0f, 0.0f}, mx = -INFINITY, sum = 0.0f;
+  float acc[kF32Cols], mx = -INFINITY, sum = 0.0f;
+#pragma unroll
+  for (int c = 0; c < kF32Cols; ++c) acc[c] = 0.0f;
   const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
   for (int k0 = lo; k0 <= pos; k0 += 128) {
     __syncthreads();
@@ -463,7 +469,7 @@ __global__ void __launch_bounds__(128) paged_window_f32_kernel(const NxPagedWind
     if (j <= pos) {
       const int64_t slot = static_cast<int64_t>(bt[j / a.block_size]) * a.block_size + j % a.block_size;
       s_slot[tid] = slot;
-      const float* k = kc + (slot * a.kv_heads + hk) * a.dim;
+      const float* k = kc + slot * a.k_pitch + hk * a.dim;
       float s = 0.0f;
       for (int d = 0; d < a.dim; ++d) s += sQ[d] * k[d];
       sc = s * a.scale;
@@ -480,20 +486,22 @@ __global__ void __launch_bounds__(128) paged_window_f32_kernel(const NxPagedWind
       const int d = tid + c * 128;
       if (d < a.vdim) {
         float v = acc[c] * alpha;
-        for (int i = 0; i < n; ++i) v += sP[i] * vc[(s_slot[i] * a.kv_heads + hk) * a.vdim + d];
+        for (int i = 0; i < n; ++i) v += sP[i] * vc[s_slot[i] * a.v_pitch + hk * a.vdim + d];
         acc[c] = v;
       }
     }
   }
+  const float g = a.gate != nullptr ? a.gate[row * a.heads + h] : 1.0f;
   for (int c = 0; c < kF32Cols; ++c) {
     const int d = tid + c * 128;
-    if (d < a.vdim) static_cast<float*>(a.out)[row * a.ldo + static_cast<int64_t>(h) * a.vdim + d] = acc[c] / sum * a.out_scale;
+    if (d < a.vdim) static_cast<float*>(a.out)[row * a.ldo + static_cast<int64_t>(h) * a.vdim + d] = acc[c] / sum * (a.out_scale * g);
   }
 }
 
 int check_paged(const NxPagedWindowArgs* a, int dtype) {
   if (a == nullptr || a->dtype != dtype || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads) return -1;
   if (a->dim <= 0 || a->vdim <= 0 || a->block_size <= 0 || a->max_blocks <= 0 || a->seg.count > 65535) return -1;
+  if (a->k_pitch < static_cast<int64_t>(a->kv_heads) * a->dim || a->v_pitch < static_cast<int64_t>(a->kv_heads) * a->vdim) return -1;
   return 0;
 }
 int padded_dim(const NxPagedWindowArgs* a) {

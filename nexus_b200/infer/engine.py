@@ -484,7 +484,8 @@ class Engine:
             if self.k_cache[l] is None:       # a layer without attention
                 continue
             self.k_cache[l][nb].copy_(self.k_cache[l][old])
-            self.v_cache[l][nb].copy_(self.v_cache[l][old])
+            if self.v_cache[l] is not None:   # a latent cache holds keys and values in one row
+                self.v_cache[l][nb].copy_(self.v_cache[l][old])
             if self.kv_kind:
                 self.k_scale[l][nb * bs: (nb + 1) * bs].copy_(self.k_scale[l][old * bs: (old + 1) * bs])
                 self.v_scale[l][nb * bs: (nb + 1) * bs].copy_(self.v_scale[l][old * bs: (old + 1) * bs])

@@ -11,17 +11,22 @@ per sequence) in up to three groups, one-token segments, short ones and long one
 
 * attention: split-key decode kernel | paged prompt kernel | tcgen05 flash kernel (fresh prompts, head sizes 64 / 128)
 * recurrences: token-by-token kernel with the state tile in shared memory | chunked tensor-core kernel
+* latent attention: `latent`; feed-forwards of experts: `experts`
 
-The residual stream is FP32; one kernel adds a normed sublayer output to it and norms it for the next sublayer.  In FP32
+The residual stream is FP32; one kernel adds a normed sublayer output to it and prepares it for the next sublayer.  In FP32
 precision the same layer loop runs the kernels' FP32 forms and plain FP32 matrix products.
 """
 from __future__ import annotations
 
-from typing import Dict, List, Sequence
+from dataclasses import astuple
+from typing import Dict, List, Optional, Sequence
 
 import torch
 
-from ..lm.hybrid import DeltaSpec, HybridConfig, HybridWeights, ParallelSpec
+from ..lm.config import RopeScaling
+from ..lm.hybrid import DeltaSpec, HybridConfig, HybridWeights, LatentSpec, ParallelSpec
+from ..lm.rope import rope_inv_freq
+from . import experts, latent
 from .engine import Chunk, Engine, _Linear
 
 __all__ = ["HybridEngine"]
@@ -64,14 +69,14 @@ class HybridEngine(Engine):
         self._rope: Dict[tuple, tuple] = {}
         self._short_len = 16 if self.fast else 1 << 30
 
-    def _rope_tables(self, dims: int, base: float):
+    def _rope_tables(self, dims: int, base: float, scaling: Optional[RopeScaling] = None):
         """cos / sin [ctx, dims / 2]: angles in double, kept in FP32."""
-        key = (dims, base)
+        scaling = scaling or RopeScaling()
+        key = (dims, base, astuple(scaling))
         if key not in self._rope:
-            half = dims // 2
-            freq = float(base) ** (-2.0 * torch.arange(half, dtype=torch.float64) / max(dims, 1))
-            ang = torch.arange(self.ctx, dtype=torch.float64)[:, None] * freq[None, :]
-            self._rope[key] = tuple(f(ang).float().to(self.dev).contiguous() for f in (torch.cos, torch.sin))
+            freq, mul = rope_inv_freq(max(dims, 1), base, scaling, self.ctx, dtype=torch.float64)
+            ang = torch.arange(self.ctx, dtype=torch.float64)[:, None] * freq[None, : dims // 2]
+            self._rope[key] = tuple((f(ang) * mul).float().to(self.dev).contiguous() for f in (torch.cos, torch.sin))
         return self._rope[key]
 
     # ----------------------------------------------------------------------------- weights
@@ -100,14 +105,21 @@ class HybridEngine(Engine):
         head[: self.V] = t["head"].float()
         self.head, _ = self._pack([head])
         self.embed = t["embed"].to(self.dev, self.adt).contiguous()
-        self.side_embed = t["side.embed"].to(self.dev, self.adt).contiguous()
-        self.weight_nbytes += sum(e.numel() * e.element_size() for e in (self.embed, self.side_embed))
+        self.side_embed = t["side.embed"].to(self.dev, self.adt).contiguous() if model.token_side else None
+        self.weight_nbytes += sum(e.numel() * e.element_size() for e in (self.embed, self.side_embed) if e is not None)
         self.final_norm = self._f32(t["final.norm"])
         self.layers: List[dict] = []
         for i, layer in enumerate(model.layers):
             p, m = f"l{i}.", layer.mixer
-            out = {n: self._f32(t[p + n]) for n in ("norm1", "norm1b")}
-            if isinstance(m, ParallelSpec):
+            # the norms of the two sublayers: on the input (where the design has it) and on the output
+            out = {}
+            for k, needed in (("1", True), ("2", bool(layer.ff or layer.experts))):
+                if needed:
+                    out["pre" + k] = self._f32(t[p + "norm" + k]) if model.pre_norm else None
+                    out["post" + k] = self._f32(t[p + "norm" + k + ("b" if model.pre_norm else "")])
+            if isinstance(m, LatentSpec):
+                out["mix"] = latent.load(self, m, lambda n: t[p + "mix." + n])
+            elif isinstance(m, ParallelSpec):
                 a, r = m.left, m.right
                 w_in = t[p + "mix.right.in"]
                 z, xbc, dt = w_in.split([r.inner, r.channels, r.heads], 0)
@@ -134,13 +146,15 @@ class HybridEngine(Engine):
                 out["conv_b"] = None
                 for n, key in (("dt_bias", "dt_bias"), ("A_log", "a_log"), ("norm", "norm")):
                     out[key] = self._f32(t[p + "mix." + n])
+            if layer.experts:
+                out["ff"] = experts.load(self, layer.experts, lambda n: t[p + "mlp." + n])
             if layer.ff:
-                out["norm2"], out["norm2b"] = self._f32(t[p + "norm2"]), self._f32(t[p + "norm2b"])
                 out["up"], _ = self._pack([t[p + "mlp.gate"], t[p + "mlp.up"]])
                 out["down"], _ = self._pack([t[p + "mlp.down"]])
-            out["side_gate"], _ = self._pack([t[p + "side.gate"]])
-            out["side_proj"], _ = self._pack([t[p + "side.proj"]])
-            out["side_norm"] = self._f32(t[p + "side.norm"])
+            if model.token_side:
+                out["side_gate"], _ = self._pack([t[p + "side.gate"]])
+                out["side_proj"], _ = self._pack([t[p + "side.proj"]])
+                out["side_norm"] = self._f32(t[p + "side.norm"])
             self.layers.append(out)
 
     # ----------------------------------------------------------------------------- cache pages and state slots
@@ -153,6 +167,10 @@ class HybridEngine(Engine):
         self.conv_tail: list = [None] * self.L    # [slots, taps - 1, channels]
         for i, layer in enumerate(self.model.layers):
             m = layer.mixer
+            if isinstance(m, LatentSpec):     # one row per token, whose leading columns are the values; the padding stays zero
+                row = latent.LatentShape(m).row
+                self.k_cache[i] = torch.zeros((self.n_blocks, cfg.block_size, 1, row), dtype=self.adt, device=self.dev)
+                continue
             if isinstance(m, ParallelSpec):
                 a, r = m.left, m.right
                 self.k_cache[i] = torch.zeros((self.n_blocks, cfg.block_size, a.kv_heads, a.dim), dtype=self.adt, device=self.dev)
@@ -165,14 +183,15 @@ class HybridEngine(Engine):
         self.k_scale = self.v_scale = [None] * self.L
 
     def state_bytes_per_sequence(self) -> int:
-        return sum(t[0].numel() * t.element_size() for t in (*self.state, *self.conv_tail))
+        return sum(t[0].numel() * t.element_size() for t in (*self.state, *self.conv_tail) if t is not None)
 
     def _fork_state(self, src: int, dst: int) -> None:
         for t in (*self.state, *self.conv_tail):
-            t[dst].copy_(t[src])
+            if t is not None:
+                t[dst].copy_(t[src])
 
     def _check_truncate(self, seq: int, length: int) -> None:
-        if 0 < length < self.length(seq):
+        if self.model.recurrent and 0 < length < self.length(seq):
             raise ValueError("a recurrent state cannot be taken back: truncate to 0, or fork the sequence beforehand")
 
     def _check_batch(self, chunks: Sequence[Chunk]) -> None:
@@ -184,7 +203,7 @@ class HybridEngine(Engine):
             last = c.seq
 
     def forward(self, chunks: Sequence[Chunk], layers: int = -1, device_tokens: bool = False) -> torch.Tensor:
-        if 0 <= layers < self.L:
+        if self.model.recurrent and 0 <= layers < self.L:
             raise ValueError("running the first layers only would advance some states and not others")
         return super().forward(chunks, layers, device_tokens)
 
@@ -312,30 +331,55 @@ class HybridEngine(Engine):
                      gate_first=False, eps=self.model.norm_eps)
         return self._linear(out, lw["out"])
 
+    def _mixer(self, i: int, m, lw: dict, h, pos, slot) -> torch.Tensor:
+        if isinstance(m, LatentSpec):
+            return latent.mixer(self, i, m, lw["mix"], h, pos, slot)
+        if isinstance(m, ParallelSpec):
+            return self._parallel_mixer(i, m, lw, h, pos, slot)
+        return self._delta_mixer(i, m, lw, h)
+
     def _body(self, tok, pos, slot, rseq, ctx_len, logit_rows, runs, nl: int) -> torch.Tensor:
         from ..ops import _mixers as M
         n, eps, model, cap = tok.shape[0], self.model.norm_eps, self.model, self._capture
+        mult = model.residual_mult
         x = torch.empty((n, self.d), dtype=torch.float32, device=self.dev)
         h = torch.empty((n, _pad8(self.d)), dtype=self.adt, device=self.dev)
-        M.residual_norm(x, tokens=tok, table=self.embed, w_next=self.layers[0]["norm1"], h=h, eps=eps)
-        for i, (layer, lw) in enumerate(zip(model.layers, self.layers)):
-            m = layer.mixer
-            y = self._parallel_mixer(i, m, lw, h, pos, slot) if isinstance(m, ParallelSpec) else self._delta_mixer(i, m, lw, h)
-            post = lw["norm1b"]
-            if layer.ff:
-                M.residual_norm(x, y=y, w_post=post, w_next=lw["norm2"], h=h, eps=eps)
+        routes = experts.route(self, tok)
+
+        def feed(norm) -> dict:      # what the next sublayer reads
+            return {"w_next": norm, "h": h} if norm is not None else {"x_cast": h}
+        M.residual_norm(x, tokens=tok, table=self.embed, eps=eps, embed_scale=model.embed_scale, **feed(self.layers[0]["pre1"]))
+        for i, (layer, lw) in enumerate(zip(model.layers[:nl], self.layers)):
+            more = feed(self.layers[i + 1]["pre1"]) if i + 1 < nl else {}
+            after = more if not model.token_side else {"x_cast": h}
+            y, add = self._mixer(i, layer.mixer, lw, h, pos, slot), {"w_post": lw["post1"]}
+            if layer.experts:
+                f, ff, r = layer.experts, lw["ff"], routes[i]
+                extra = {}
+                if f.shared:
+                    gate = torch.empty(n, dtype=torch.float32, device=self.dev)
+                    extra.update(w_dot=ff["sg"], dot_out=gate)
+                by_slot = None
+                if r.align >= 128:
+                    by_slot = torch.empty((r.max_slots, h.shape[1]), dtype=self.adt, device=self.dev)
+                    extra.update(scatter=by_slot, slots=r.slots, top=r.top)
+                M.residual_norm(x, y=y, eps=eps, res_mult=mult, **add, **feed(lw["pre2"]), **extra)
+                rows, y = experts.forward(self, f, ff, r, h, by_slot)
+                add = {"w_post": lw["post2"], "experts": rows, "slots": r.slots, "top": r.top,
+                       "y_gate": gate if f.shared else None}
+            elif layer.ff:
+                M.residual_norm(x, y=y, eps=eps, res_mult=mult, **add, **feed(lw["pre2"]))
                 gu = self._linear(h, lw["up"])
                 act = torch.empty((n, gu.shape[1] // 2), dtype=self.adt, device=self.dev)
                 M.silu_mul(gu, act)
-                y, post = self._linear(act, lw["down"]), lw["norm2b"]
-            M.residual_norm(x, y=y, w_post=post, x_cast=h, eps=eps)
-            gate = self._linear(h, lw["side_gate"], out_dtype=torch.float32)
-            side = torch.empty(gate.shape, dtype=self.adt, device=self.dev)
-            M.token_side_gate(gate, tok, self.side_embed, i * model.token_side, side, model.token_side)
-            y = self._linear(side, lw["side_proj"])
-            last = i + 1 == self.L
-            M.residual_norm(x, y=y, w_post=lw["side_norm"], eps=eps, **({} if last else {
-                "w_next": self.layers[i + 1]["norm1"], "h": h}))
+                y, add = self._linear(act, lw["down"]), {"w_post": lw["post2"]}
+            M.residual_norm(x, y=y, eps=eps, res_mult=mult, **add, **after)
+            if model.token_side:
+                gate = self._linear(h, lw["side_gate"], out_dtype=torch.float32)
+                side = torch.empty(gate.shape, dtype=self.adt, device=self.dev)
+                M.token_side_gate(gate, tok, self.side_embed, i * model.token_side, side, model.token_side)
+                y = self._linear(side, lw["side_proj"])
+                M.residual_norm(x, y=y, w_post=lw["side_norm"], eps=eps, res_mult=mult, **more)
             if cap is not None:
                 cap.append(x.detach().float().cpu())
         if logit_rows.shape[0] == 0:

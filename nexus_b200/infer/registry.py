@@ -11,6 +11,7 @@ from dataclasses import dataclass
 from typing import Callable, Dict, Optional
 
 from ..lm.hybrid import HybridWeights, load_gugedra
+from ..lm.makuzen import load_makuzen
 from .engine import Engine, EngineConfig, Gpt2Weights, load_gpt2
 from .hybrid import HybridEngine
 
@@ -66,3 +67,4 @@ def _load_gpt2_folder(path: str) -> Gpt2Weights:
 
 register_family(ModelFamily("GPT2", _load_gpt2_folder, Gpt2Weights, Engine))
 register_family(ModelFamily("Gugedra", load_gugedra, HybridWeights, HybridEngine))
+register_family(ModelFamily("Makuzen", load_makuzen, HybridWeights, HybridEngine))

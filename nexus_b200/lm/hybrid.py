@@ -1,15 +1,15 @@
 """Decoders whose layers differ from one another: the layer list, the mixers' sizes and constants, and the weights.
 
 A model is an ordered list of :class:`HybridLayer`; each has one mixer - :class:`AttentionSpec` and :class:`SsdSpec` side
-by side (:class:`ParallelSpec`) or :class:`DeltaSpec` - and optionally a gated feed-forward.  The engine
-(`infer.hybrid.HybridEngine`) builds its cache, its state slots and its kernels' arguments from these specs and reads no
-size from anywhere else, so another order of layers or another combination of constants is another configuration, not
-another class.
+by side (:class:`ParallelSpec`), :class:`DeltaSpec` or :class:`LatentSpec` - and optionally a feed-forward, gated or of
+experts (:class:`ExpertsSpec`).  The engine (`infer.hybrid.HybridEngine`) builds its cache, its state slots and its
+kernels' arguments from these specs and reads no size from anywhere else, so another order of layers or another
+combination of constants is another configuration, not another class.
 
-`Gugedra` is the design that uses them so far: RMS norms before and after every sublayer, a sliding-window soft-capped
+`Gugedra` is one design that uses them: RMS norms before and after every sublayer, a sliding-window soft-capped
 attention branch beside a Mamba-2 branch in some layers, the gated delta rule in the others, a per-layer token input at
 the end of every layer and soft-capped logits.  :func:`gugedra_config` reads its ``config.json``, and
-:func:`load_gugedra` its ``model.safetensors``.
+:func:`load_gugedra` its ``model.safetensors``.  `Makuzen` (`lm.makuzen`) is another.
 """
 from __future__ import annotations
 
@@ -21,10 +21,10 @@ from typing import Dict, List, Optional, Tuple, Union
 
 import torch
 
-from .config import ConfigError
+from .config import ConfigError, RopeScaling
 
-__all__ = ["AttentionSpec", "SsdSpec", "ParallelSpec", "DeltaSpec", "HybridLayer", "HybridConfig", "HybridWeights",
-           "gugedra_config", "gugedra_tensors", "load_gugedra", "random_gugedra"]
+__all__ = ["AttentionSpec", "SsdSpec", "ParallelSpec", "DeltaSpec", "LatentSpec", "ExpertsSpec", "HybridLayer", "HybridConfig",
+           "HybridWeights", "gugedra_config", "gugedra_tensors", "load_gugedra", "random_gugedra"]
 
 
 def _positive(obj, *names) -> None:
@@ -117,9 +117,51 @@ class DeltaSpec:
 
 
 @dataclass(frozen=True)
+class LatentSpec:
+    """Causal softmax attention whose keys and values are linear in one normed latent per token; a token's cache row is the
+    latent and one rotated key part, both shared by the heads."""
+    heads: int
+    dim: int                 # unrotated query / key size of a head
+    rope_dims: int           # rotated query / key size of a head (rotate-half pairing)
+    vdim: int                # value size of a head
+    q_rank: int              # size of the latent the queries go through
+    kv_rank: int             # size of the cached latent
+    scale: float
+    window: int = 0          # > 0: a token sees itself and the window - 1 tokens before it
+    rope_base: float = 10000.0
+    rope_scaling: Optional[RopeScaling] = None
+
+    def __post_init__(self):
+        _positive(self, "heads", "dim", "rope_dims", "vdim", "q_rank", "kv_rank")
+        if self.rope_dims % 2:
+            raise ConfigError("latent attention: the rotary dimensions must be even")
+        if self.window < 0:
+            raise ConfigError("latent attention: window cannot be negative")
+
+
+@dataclass(frozen=True)
+class ExpertsSpec:
+    """Feed-forward of small experts, W_down act(W_up h) with act = relu squared, of which a token uses ``top`` with equal
+    weights; a table gives every token id its experts.  ``shared``: width of an expert that runs for every token, times
+    one sigmoid per token (0: none)."""
+    experts: int
+    top: int
+    ff: int
+    shared: int = 0
+
+    def __post_init__(self):
+        _positive(self, "experts", "top", "ff")
+        if self.top > self.experts:
+            raise ConfigError("experts: a token cannot use more experts than there are")
+        if self.shared < 0:
+            raise ConfigError("experts: the width of the shared expert cannot be negative")
+
+
+@dataclass(frozen=True)
 class HybridLayer:
-    mixer: Union[ParallelSpec, DeltaSpec]
+    mixer: Union[ParallelSpec, DeltaSpec, LatentSpec]
     ff: int = 0              # width of the SwiGLU feed-forward, 0: none
+    experts: Optional[ExpertsSpec] = None
 
 
 @dataclass
@@ -128,18 +170,33 @@ class HybridConfig:
     width: int
     layers: List[HybridLayer] = field(default_factory=list)
     norm_eps: float = 1e-6
-    token_side: int = 0      # width of the per-layer token input
+    token_side: int = 0      # width of the per-layer token input, 0: none
     logit_softcap: float = 0.0
     name: str = "hybrid"
+    pre_norm: bool = True    # sublayers read the normed residual stream, else the stream itself; their outputs are normed always
+    embed_scale: float = 1.0
+    residual_mult: float = 1.0   # factor of every normed sublayer output
 
     def __post_init__(self):
-        _positive(self, "vocab", "width", "token_side")
+        _positive(self, "vocab", "width")
+        if self.token_side < 0:
+            raise ConfigError("token_side cannot be negative")
         if not self.layers:
             raise ConfigError("a model needs at least one layer")
 
+    @property
+    def recurrent(self) -> bool:
+        """Whether a sequence owns state beside its cache pages."""
+        return any(isinstance(layer.mixer, (ParallelSpec, DeltaSpec)) for layer in self.layers)
+
     def kv_bytes_per_token(self, element: int) -> int:
-        return sum(m.left.kv_heads * (m.left.dim + m.left.vdim) * element
-                   for m in (layer.mixer for layer in self.layers) if isinstance(m, ParallelSpec))
+        n = 0
+        for m in (layer.mixer for layer in self.layers):
+            if isinstance(m, ParallelSpec):
+                n += m.left.kv_heads * (m.left.dim + m.left.vdim) * element
+            elif isinstance(m, LatentSpec):
+                n += (m.kv_rank + m.rope_dims) * element
+        return n
 
 
 @dataclass
@@ -182,6 +239,8 @@ def gugedra_config(obj: dict) -> HybridConfig:
         obj, "config", ("architecture", "layers", "logit_softcap", "norm", "token_side", "vocab", "width"))
     (eps,) = _take(norm, "norm", ("eps",))
     (side_dim,) = _take(side, "token_side", ("dim",))
+    if not isinstance(side_dim, int) or side_dim < 1:
+        raise ConfigError("token_side.dim must be a positive integer")
     out = []
     for i, layer in enumerate(layers):
         kind, mix, mlp = _take(layer, f"layers[{i}]", ("type", "mixer", "mlp"))
@@ -235,8 +294,9 @@ def gugedra_tensors(cfg: HybridConfig) -> Dict[str, Tuple[int, ...]]:
     return t
 
 
-def check_tensors(cfg: HybridConfig, tensors: Dict[str, torch.Tensor]) -> None:
-    want = gugedra_tensors(cfg)
+def check_tensors(cfg: HybridConfig, tensors: Dict[str, torch.Tensor], want: Optional[Dict[str, Tuple[int, ...]]] = None) -> None:
+    """``want``: names and shapes of the design's tensors (default: Gugedra's)."""
+    want = gugedra_tensors(cfg) if want is None else want
     missing, extra = sorted(set(want) - set(tensors)), sorted(set(tensors) - set(want))
     if missing or extra:
         raise ConfigError(f"weights do not fit the configuration: missing {missing[:4]}, unknown {extra[:4]}")

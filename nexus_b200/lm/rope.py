@@ -14,9 +14,9 @@ import torch
 from .config import LmConfig, RopeScaling
 
 
-def rope_inv_freq(rot_dim: int, theta: float, scaling: RopeScaling, max_position: int,
-                  seq_len: int = 0) -> Tuple[torch.Tensor, float]:
-    """Returns (inv_freq [rot_dim/2] float64->float32, attention scaling factor)."""
+def rope_inv_freq(rot_dim: int, theta: float, scaling: RopeScaling, max_position: int, seq_len: int = 0,
+                  dtype: torch.dtype = torch.float32) -> Tuple[torch.Tensor, float]:
+    """Returns (inv_freq [rot_dim/2], formed in float64 and rounded to ``dtype``; attention scaling factor)."""
     half = rot_dim // 2
     idx = torch.arange(0, half, dtype=torch.float64)
     base = float(theta)
@@ -38,9 +38,7 @@ def rope_inv_freq(rot_dim: int, theta: float, scaling: RopeScaling, max_position
             return (rot_dim * math.log(orig / (rot * 2 * math.pi))) / (2 * math.log(base))
         low = max(math.floor(corr_dim(scaling.beta_fast)), 0)
         high = min(math.ceil(corr_dim(scaling.beta_slow)), rot_dim - 1)
-        if low == high:
-            high += 0.001
-        ramp = torch.clamp((torch.arange(half, dtype=torch.float64) - low) / (high - low), 0, 1)
+        ramp = torch.clamp((torch.arange(half, dtype=torch.float64) - low) / max(high - low, 0.001), 0, 1)
         extrap = 1.0 - ramp
         inv = (inv / factor) * (1 - extrap) + inv * extrap
         attn = scaling.attention_factor if scaling.attention_factor > 0 else 0.1 * math.log(factor) + 1.0
@@ -53,7 +51,7 @@ def rope_inv_freq(rot_dim: int, theta: float, scaling: RopeScaling, max_position
         smoothed = (1 - smooth) * inv / factor + smooth * inv
         medium = ~(wavelen < high_wl) & ~(wavelen > low_wl)
         inv = torch.where(medium, smoothed, scaled)
-    return inv.to(torch.float32), float(attn)
+    return inv.to(dtype), float(attn)
 
 
 class RopeCache:

@@ -22,7 +22,7 @@ _outgrown = []
 launch_count = 0  # kernels launched through this module (bench.py reports it)
 
 BF16, F32, F16, E4M3, E5M2 = 0, 1, 2, 3, 4
-ACT = {None: 0, "none": 0, "gelu": 1, "relu": 2, "dgelu": 3, "silu": 4}
+ACT = {None: 0, "none": 0, "gelu": 1, "relu": 2, "dgelu": 3, "silu": 4, "relu2": 5}
 _DT = {torch.bfloat16: BF16, torch.float32: F32, torch.float16: F16}
 if hasattr(torch, "float8_e4m3fn"):
     _DT[torch.float8_e4m3fn] = E4M3
@@ -43,6 +43,7 @@ class GemmArgs(C.Structure):
         ("act", C.c_int32), ("accumulate", C.c_int32), ("split_k", C.c_int32), ("block_n", C.c_int32),
         ("alpha", C.c_float), ("max_ctas", C.c_int32), ("b_dtype_plus1", C.c_int32),
         ("scale_a", C.c_void_p), ("scale_b", C.c_void_p), ("amax_out", C.c_void_p),
+        ("row_groups", C.c_void_p), ("group_rows", C.c_int32),
     ]
 
 
@@ -294,6 +295,30 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
 
 
 # -------------------------------------------------------------------------------------------- norms
+def grouped_gemm(a: torch.Tensor, b: torch.Tensor, groups: torch.Tensor, group_rows: int, *, act: Optional[str] = None,
+                 out: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """Rows ``i * group_rows ..`` of ``a`` [M, K] times ``b[groups[i]]`` ([groups, N, K]); a negative entry skips the rows.
+    ``groups``: int32 on the device, one entry per ``group_rows`` (128 or 256) rows."""
+    m, k = a.shape
+    batch, n, kb = b.shape
+    if k != kb or a.stride(1) != 1 or b.stride(2) != 1 or a.dtype != b.dtype or a.dtype != torch.bfloat16:
+        raise ValueError("grouped_gemm: operands must be BF16 with contiguous rows of one length")
+    if groups.dtype != torch.int32 or groups.numel() * group_rows < m:
+        raise ValueError("grouped_gemm: one int32 group per row tile is expected")
+    if out is None:
+        out = torch.empty((m, n), dtype=out_dtype or a.dtype, device=a.device)
+    g = GemmArgs()
+    g.a, g.b, g.out = a.data_ptr(), b.data_ptr(), out.data_ptr()
+    g.lda, g.ldb, g.ldo, g.stride_b = a.stride(0), b.stride(1), out.stride(0), b.stride(0)
+    g.m, g.n, g.k, g.batch = m, n, k, batch
+    g.in_dtype, g.out_dtype = _DT[a.dtype], _DT[out.dtype]
+    g.act, g.alpha, g.split_k = ACT[act], 1.0, 1
+    g.row_groups, g.group_rows = groups.data_ptr(), group_rows
+    g.status = status_word(a.device).data_ptr()
+    _check(lib().nx_gemm(C.byref(g), _stream()), "nx_gemm")
+    return out
+
+
 def norm_fwd(x, gamma, beta=None, *, rms=False, eps=1e-5, residual=None, sum_out=None, out_dtype=None,
              want_stats=True):
     rows, cols = x.numel() // x.shape[-1], x.shape[-1]

@@ -1,0 +1,94 @@
+"""ctypes bindings of the expert layers a table routes (``nx_api_moe.h``): one launch sorts the assignments of a step for
+every layer, and the products over the sorted rows (tcgen05 grouped GEMM, few-rows BF16 kernel, FP32)."""
+from __future__ import annotations
+
+import ctypes as C
+from dataclasses import dataclass
+from typing import List, Optional, Sequence, Tuple
+
+import torch
+
+from . import _cuda as K
+
+MAX_LAYERS = 32       # layers per routing launch
+F32_ALIGN = 32        # slots per tile of the FP32 product
+
+
+class TableRouteLayer(C.Structure):
+    _fields_ = [("table", C.c_void_p), ("slots", C.c_void_p), ("rows", C.c_void_p), ("start", C.c_void_p), ("count", C.c_void_p),
+                ("groups", C.c_void_p), ("experts", C.c_int32), ("top", C.c_int32), ("max_slots", C.c_int32)]
+
+
+class TableRouteArgs(C.Structure):
+    _fields_ = [("tokens", C.c_void_p), ("n", C.c_int32), ("vocab", C.c_int32), ("layers", C.c_int32), ("align", C.c_int32),
+                ("layer", TableRouteLayer * MAX_LAYERS)]
+
+
+class ExpertGemmArgs(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("rows", C.c_void_p), ("w", C.c_void_p), ("out", C.c_void_p), ("start", C.c_void_p),
+                ("count", C.c_void_p), ("groups", C.c_void_p), ("ldx", C.c_int64), ("ldw", C.c_int64), ("stride_w", C.c_int64),
+                ("ldo", C.c_int64), ("experts", C.c_int32), ("n", C.c_int32), ("k", C.c_int32), ("act", C.c_int32),
+                ("tiles", C.c_int32), ("align", C.c_int32)]
+
+
+@dataclass
+class Route:
+    """The sorted assignments of one layer: slots [n, top], rows [max_slots], start / count [experts], groups [tiles]."""
+    slots: torch.Tensor
+    rows: torch.Tensor
+    start: torch.Tensor
+    count: torch.Tensor
+    groups: torch.Tensor
+    align: int
+    top: int
+
+    @property
+    def max_slots(self) -> int:
+        return self.rows.shape[0]
+
+
+def table_slots(assignments: int, experts: int, align: int) -> int:
+    """Slots that ``assignments`` can take at most: every expert in use leaves up to align - 1 of them empty."""
+    return -(-(assignments + min(assignments, experts) * (align - 1)) // align) * align
+
+
+def table_route(tokens: torch.Tensor, layers: Sequence[Tuple[torch.Tensor, int]], align: int) -> List[Route]:
+    """``layers``: (table [vocab, top] int32, experts) of every layer of experts."""
+    n, dev, out = tokens.shape[0], tokens.device, []
+    sizes = [(t.shape[1], e, table_slots(n * t.shape[1], e, align)) for t, e in layers]
+    buf = torch.empty(sum(n * top + cap + 2 * e + cap // align for top, e, cap in sizes), dtype=torch.int32, device=dev)
+    at = 0
+
+    def take(k):
+        nonlocal at
+        at += k
+        return buf[at - k: at]
+    for top, e, cap in sizes:
+        out.append(Route(take(n * top).view(n, top), take(cap), take(e), take(e), take(cap // align), align, top))
+    for first in range(0, len(layers), MAX_LAYERS):
+        part = layers[first: first + MAX_LAYERS]
+        a = TableRouteArgs(tokens.data_ptr(), n, part[0][0].shape[0], len(part), align)
+        for i, (table, experts) in enumerate(part):
+            r = out[first + i]
+            a.layer[i] = TableRouteLayer(table.data_ptr(), r.slots.data_ptr(), r.rows.data_ptr(), r.start.data_ptr(),
+                                         r.count.data_ptr(), r.groups.data_ptr(), experts, r.top, r.max_slots)
+        K._check(K.lib().nx_moe_table_route(C.byref(a), K._stream()), "nx_moe_table_route")
+    return out
+
+
+def expert_product(x: torch.Tensor, w: torch.Tensor, route: Route, *, gather: bool, act: Optional[str] = None) -> torch.Tensor:
+    """out[slot] = act(w[expert] x[row of slot]), w [experts, n, k].  ``gather``: x has the batch's rows, else the slots'.
+    The product is chosen by dtype and the alignment of the route: 1 few rows (BF16), 32 FP32, 128 / 256 the tcgen05 GEMM
+    (whose x is in slot order)."""
+    E, n, k = w.shape
+    out = torch.empty((route.max_slots, n), dtype=x.dtype, device=x.device)
+    if x.dtype == torch.bfloat16 and route.align >= 128:
+        if gather:
+            raise ValueError("expert_product: the GEMM reads its rows in slot order")
+        return K.grouped_gemm(x, w, route.groups, route.align, act=act, out=out)
+    a = ExpertGemmArgs(x.data_ptr(), route.rows.data_ptr() if gather else None, w.data_ptr(), out.data_ptr(), route.start.data_ptr(),
+                       route.count.data_ptr(), route.groups.data_ptr(), x.stride(0), w.stride(1), w.stride(0), out.stride(0), E, n, k,
+                       K.ACT[act], route.groups.shape[0], route.align)
+    name = "nx_expert_skinny" if x.dtype == torch.bfloat16 else "nx_expert_f32"
+    K._check(getattr(K.lib(), name)(C.byref(a), K._stream()), name)
+    return out

@@ -23,7 +23,19 @@ class SegmentArgs(C.Structure):
 class ResidualNormArgs(C.Structure):
     _fields_ = [("x", C.c_void_p), ("tokens", C.c_void_p), ("table", C.c_void_p), ("y", C.c_void_p), ("w_post", C.c_void_p),
                 ("w_next", C.c_void_p), ("h", C.c_void_p), ("x_cast", C.c_void_p), ("ldy", C.c_int64), ("ldh", C.c_int64),
-                ("rows", C.c_int32), ("cols", C.c_int32), ("dtype", C.c_int32), ("eps", C.c_float)]
+                ("rows", C.c_int32), ("cols", C.c_int32), ("dtype", C.c_int32), ("eps", C.c_float), ("embed_scale", C.c_float),
+                ("res_mult", C.c_float), ("experts", C.c_void_p), ("expert_slots", C.c_void_p), ("y_gate", C.c_void_p),
+                ("ld_experts", C.c_int64), ("top", C.c_int32), ("expert_scale", C.c_float), ("w_dot", C.c_void_p),
+                ("dot_out", C.c_void_p), ("scatter", C.c_void_p), ("scatter_slots", C.c_void_p)]
+
+
+class LatentPrepArgs(C.Structure):
+    _fields_ = [("proj", C.c_void_p), ("ld", C.c_int64), ("q_off", C.c_int32), ("c_off", C.c_int32), ("r_off", C.c_int32),
+                ("g_off", C.c_int32), ("rows", C.c_int32), ("q_rank", C.c_int32), ("kv_rank", C.c_int32), ("rot_dims", C.c_int32),
+                ("heads", C.c_int32), ("dtype", C.c_int32), ("eps", C.c_float), ("w_q", C.c_void_p), ("w_kv", C.c_void_p),
+                ("positions", C.c_void_p), ("slots", C.c_void_p), ("cos_t", C.c_void_p), ("sin_t", C.c_void_p), ("cq", C.c_void_p),
+                ("ldq", C.c_int64), ("cache", C.c_void_p), ("ld_cache", C.c_int64), ("rot_col", C.c_int32), ("lat", C.c_void_p),
+                ("gate", C.c_void_p)]
 
 
 class RopeAppendArgs(C.Structure):
@@ -67,7 +79,7 @@ class PagedWindowArgs(C.Structure):
                 ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32),
                 ("block_size", C.c_int32), ("max_blocks", C.c_int32), ("window", C.c_int32), ("splits", C.c_int32),
                 ("dtype", C.c_int32), ("scale", C.c_float), ("softcap", C.c_float), ("out_scale", C.c_float),
-                ("seg", SegmentArgs)]
+                ("seg", SegmentArgs), ("k_pitch", C.c_int64), ("v_pitch", C.c_int64), ("gate", C.c_void_p)]
 
 
 @dataclass
@@ -93,16 +105,39 @@ def _ptr(t: Optional[torch.Tensor]):
     return None if t is None else t.data_ptr()
 
 
-def residual_norm(x, *, y=None, w_post=None, w_next=None, h=None, x_cast=None, tokens=None, table=None, eps) -> None:
-    """x (FP32) = table[tokens], or x + rms(y) * w_post;  h = rms(x) * w_next;  x_cast = x in the activation dtype."""
-    lead = h if h is not None else x_cast
-    act = lead if lead is not None else (y if y is not None else table)
-    if h is not None and x_cast is not None and h.stride(0) != x_cast.stride(0):
-        raise ValueError("residual_norm: h and x_cast must share one row pitch")
+def residual_norm(x, *, y=None, w_post=None, w_next=None, h=None, x_cast=None, tokens=None, table=None, eps, embed_scale=1.0,
+                  res_mult=1.0, experts=None, slots=None, top=0, y_gate=None, w_dot=None, dot_out=None, scatter=None) -> None:
+    """x (FP32) = embed_scale * table[tokens], or x + res_mult * rms(y) * w_post;  h = rms(x) * w_next;  x_cast = x in the
+    activation dtype.  With ``experts`` the sublayer output is the mean of the rows ``experts[slots[r, :]]`` (+ y_gate[r] *
+    y[r]).  ``dot_out`` = sigmoid(x . w_dot); ``scatter[slots[r, :]]`` = the row of x_cast."""
+    lead = next((t for t in (h, x_cast, scatter) if t is not None), None)
+    act = next(t for t in (lead, y, experts, table) if t is not None)
+    if any(t is not None and t.stride(0) != lead.stride(0) for t in (h, x_cast, scatter)):
+        raise ValueError("residual_norm: h, x_cast and scatter must share one row pitch")
     a = ResidualNormArgs(_ptr(x), _ptr(tokens), _ptr(table), _ptr(y), _ptr(w_post), _ptr(w_next), _ptr(h), _ptr(x_cast),
                          y.stride(0) if y is not None else 0, lead.stride(0) if lead is not None else x.shape[1], x.shape[0],
-                         x.shape[1], _dt(act), eps)
+                         x.shape[1], _dt(act), eps, embed_scale, res_mult, _ptr(experts), _ptr(slots), _ptr(y_gate),
+                         experts.stride(0) if experts is not None else 0, top, 1.0 / top if top else 1.0, _ptr(w_dot),
+                         _ptr(dot_out), _ptr(scatter), _ptr(slots))
     K._check(K.lib().nx_residual_norm(C.byref(a), K._stream()), "nx_residual_norm")
+
+
+def latent_prep(proj, offsets, q_rank, kv_rank, rot_dims, heads, w_q, w_kv, positions, slots, cos_t, sin_t, cq, cache, rot_col,
+                gate, *, eps, lat=None) -> None:
+    """``offsets``: first columns of the query latent, the key / value latent, the shared key part and the gate in ``proj``;
+    cache [blocks, block_size, row], lat [rows, row] or None, gate FP32 [rows, heads]."""
+    a = LatentPrepArgs(_ptr(proj), proj.stride(0), *offsets, proj.shape[0], q_rank, kv_rank, rot_dims, heads, _dt(proj), eps,
+                       _ptr(w_q), _ptr(w_kv), _ptr(positions), _ptr(slots), _ptr(cos_t), _ptr(sin_t), _ptr(cq), cq.stride(0),
+                       _ptr(cache), cache.shape[-1], rot_col, _ptr(lat), _ptr(gate))
+    K._check(K.lib().nx_latent_prep(C.byref(a), K._stream()), "nx_latent_prep")
+
+
+def rope_heads(src, src_head, src_off, dst, dst_head, dst_off, heads, rot_dims, width, positions, cos_t, sin_t) -> None:
+    """Rotates ``rot_dims`` columns of every head of ``src`` [rows, .] into ``dst`` (zeros up to ``width``)."""
+    K._check(K.lib().nx_rope_heads(K._p(src), C.c_int64(src.stride(0)), C.c_int(src_head), C.c_int(src_off), K._p(dst),
+                                   C.c_int64(dst.stride(0)), C.c_int(dst_head), C.c_int(dst_off), C.c_int(src.shape[0]),
+                                   C.c_int(heads), C.c_int(rot_dims), C.c_int(width), K._p(positions), K._p(cos_t), K._p(sin_t),
+                                   C.c_int(_dt(src)), K._stream()), "nx_rope_heads")
 
 
 def rope_append(proj, q_off, k_off, v_off, heads, kv_heads, dim, vdim, rot_dims, positions, slots, cos_t, sin_t, k_cache,
@@ -183,13 +218,20 @@ def softcap_(x, cols, cap) -> None:
 
 
 def paged_window_attention(q, k_cache, v_cache, block_table, out, seg: Segments, *, heads, block_size, window, scale,
-                           softcap=0.0, out_scale=1.0, splits=1) -> None:
+                           softcap=0.0, out_scale=1.0, splits=1, gate=None, vdim=0) -> None:
     """q: [rows, heads * dim] view; caches [blocks, block_size, kv_heads, dim | vdim]; out [rows, heads * vdim] view.
-    One-row segments run the decode kernel, longer ones the prompt kernel (BF16); FP32 has one kernel for both."""
-    G, D, Dv = k_cache.shape[2], k_cache.shape[3], v_cache.shape[3]
+    One-row segments run the decode kernel, longer ones the prompt kernel (BF16); FP32 has one kernel for both.
+    ``vdim`` > 0: a latent cache, the values are the leading ``vdim`` columns of the keys (``v_cache`` is not used).
+    ``gate``: FP32 [rows, heads] factor of the output."""
+    G, D = k_cache.shape[2], k_cache.shape[3]
+    if vdim:
+        v_cache = k_cache
+        if G != 1:
+            raise ValueError("paged_window_attention: a latent cache has one KV head")
+    Dv = vdim or v_cache.shape[3]
     a = PagedWindowArgs(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(out), q.stride(0), out.stride(0), None,
                         None, heads, G, D, Dv, block_size, block_table.shape[1], window, 1, _dt(q), scale, softcap, out_scale,
-                        seg.args())
+                        seg.args(), k_cache.stride(1), v_cache.stride(1), _ptr(gate))
     if q.dtype == torch.float32:
         K._check(K.lib().nx_paged_window_f32(C.byref(a), K._stream()), "nx_paged_window_f32")
     elif seg.max_len == 1:
