@@ -15,6 +15,7 @@
 // Features: causal, sliding window, GQA (H % Hkv == 0), Tq != Tk (bottom-right aligned causal
 // mask), head_dim 64 or 128, softmax scale.  Parity: src/cuda/flash_attention.cu:230-857 and
 // include/nexus/attention/params.hpp:18-46 of the reference (which uses mma.sync m16n8k16).
+#include "flash_common.cuh"
 #include "nx_api_attention.h"
 #include "sm100_ptx.cuh"
 #include "tensor_map.h"
@@ -26,7 +27,6 @@ namespace {
 using namespace nx;
 
 constexpr int kThreads = 192;  // warps 0-3: softmax / row math, warp 4: TMA, warp 5: MMA + TMEM
-constexpr float kLog2e = 1.4426950408889634f;
 
 struct AttnDev {
   void* out;        // fwd: O [B,Tq,H,D] bf16;   dq kernel: dQ;   dkdv kernel: dK
@@ -144,29 +144,6 @@ __device__ __forceinline__ void load_tile(uint8_t* dst, const CUtensorMap* tm, u
     else
       tma_load_4d(dst + s * rows * 128, tm, bar, 64 * s, row0, head, batch);
   }
-}
-
-// K-major operand: address of k-step `ks` (16 elements) in a tile of HD/64 (or cols/64) slabs of `rows` rows.
-__device__ __forceinline__ uint64_t desc_kmajor(uint32_t tile_addr, int rows, int ks) {
-  const uint32_t a = tile_addr + static_cast<uint32_t>((ks >> 2) * rows * 128 + (ks & 3) * 32);
-  return make_smem_desc_sw128(a, 16, 1024);
-}
-// MN-major view of a [k_rows][mn] tile stored as mn/64 slabs of [k_rows][64]: k-step `ks` = 16 rows.
-__device__ __forceinline__ uint64_t desc_mnmajor(uint32_t tile_addr, int k_rows, int ks) {
-  const uint32_t a = tile_addr + static_cast<uint32_t>(ks * 2048);
-  return make_smem_desc_sw128(a, static_cast<uint32_t>(k_rows * 128), 1024);
-}
-
-// what k-step `ks` adds to the address field (bytes >> 4) of a K-major / MN-major descriptor built for k-step 0
-__device__ __forceinline__ uint64_t kstep_kmajor(int rows, int ks) {
-  return static_cast<uint64_t>((ks >> 2) * rows * 8 + (ks & 3) * 2);
-}
-__device__ __forceinline__ uint64_t kstep_mnmajor(int ks) { return static_cast<uint64_t>(ks * 128); }
-
-__device__ __forceinline__ float ex2f(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
 }
 
 // Per-row visible key range [lo, hi] (inclusive) under the causal / window / length masks.
@@ -640,20 +617,6 @@ struct Fwd2Cfg {
   static constexpr int kTmemCols = 512;
 };
 constexpr int kFwd2Threads = 320;  // warps 0-3: softmax A, 4-7: softmax B, 8: TMA, 9: MMA
-constexpr float kRescaleStep = 8.0f;  // log2 of the growth of the row maximum that forces a rescale
-
-// D[tmem] (+)= A[tmem] * B[smem]: the A operand (128 rows on the lanes, two BF16 per column along K) is read from TMEM
-__device__ __forceinline__ void umma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc,
-                                            uint32_t accumulate) {
-  asm volatile(
-      "{\n\t"
-      ".reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t"
-      "}" ::"r"(tmem_d),
-      "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
 
 // Work of one round of the persistent loop: CTA c takes item round * grid + c in even rounds and
 // round * grid + (grid - 1 - c) in odd ones, and the items are sorted by cost (late q blocks first under a causal

@@ -1,0 +1,385 @@
+// Attention over a paged latent cache (see nx_api_mixers.h): all heads share one cache row per token, whose leading columns
+// are the values, so a row is read from memory once for every head and for both products.
+//
+// A block owns 16 MT (token, head) rows of one segment and one span of its keys.  Keys arrive in stages of 32; the pages of a
+// stage come as tiled copies of whole cache rows, split into slabs of 64 columns with the 128-byte swizzle, which the fragment
+// loads undo.  The warps split the keys of a stage for the scores and the latent columns for the weighted sum; row maxima and
+// probabilities cross warps through shared memory.  Scores and softmax are FP32; only the products take BF16 operands.
+#include "mixer_common.cuh"
+#include "nx_api_mixers.h"
+#include "paged_common.cuh"
+#include "sm100_ptx.cuh"
+#include "tensor_map.h"
+
+#include <algorithm>
+
+namespace {
+using namespace nx;
+
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr int kKeys = 32;           // per stage
+constexpr int kKGroups = 4;         // warps along the keys of a stage, eight keys each
+constexpr int kLdP = kKeys + 8;
+constexpr int kSmemMax = 226 * 1024;
+
+template <int MT>
+struct Shape {
+  static constexpr int kRows = 16 * MT;
+  static constexpr int kMGroups = MT == 1 ? 1 : 2;      // warps along the rows
+  static constexpr int kWarps = kKGroups * kMGroups;
+  static constexpr int kMTiles = MT / kMGroups;         // 16-row tiles of a warp
+  // behind the stages and Q: P, maxima per key group, running maximum, rescale factor, row sums, barriers
+  static constexpr int kTail = kRows * kLdP * 2 + kKGroups * kRows * 4 + 3 * kRows * 4 + 64;
+};
+
+// CT: 16-column tiles of the latent per warp.  A box holds `1 << box_shift` keys of one page.
+template <int MT, int CT>
+__global__ void __launch_bounds__(Shape<MT>::kWarps * 32)
+latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArgs a, int rt, int tq, int stages, int box_shift) {
+  using S = Shape<MT>;
+  constexpr int ROWS = S::kRows, WARPS = S::kWarps, THREADS = WARPS * 32;
+  extern __shared__ __align__(1024) uint8_t smem[];
+  const int LD = a.row + 8, slabs = a.row / 64, stage_bytes = kKeys * a.row * 2;
+  uint8_t* sKV = smem;                                                // [stages][boxes][slabs][keys of a box][128 B]
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem + stages * stage_bytes);   // [ROWS][LD]
+  __nv_bfloat16* sP = sQ + ROWS * LD;                                 // [ROWS][kLdP]
+  float* s_part = reinterpret_cast<float*>(sP + ROWS * kLdP);         // [key groups][ROWS] stage maxima, then row sums
+  float* s_max = s_part + kKGroups * ROWS;                            // running maximum of a row (log2 units)
+  float* s_alpha = s_max + ROWS;
+  float* s_sum = s_alpha + ROWS;
+  uint64_t* full = reinterpret_cast<uint64_t*>(s_sum + ROWS);         // [stages]
+  __shared__ int s_tile[3];
+  __shared__ volatile int s_abort;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  if (smem_u32(smem) & 1023u) {   // the swizzle needs a 1 KiB aligned base; uniform early exit
+    if (threadIdx.x == 0) atomicCAS(a.status, 0, kStatusBadArgument);
+    return;
+  }
+  if (warp == 0) {
+    int seg = 0, off = 0;
+    const bool ok = find_tile(a.seg, tq, blockIdx.x, seg, off);
+    if (lane == 0) {
+      s_tile[0] = ok;
+      s_tile[1] = seg;
+      s_tile[2] = off;
+      s_abort = 0;
+      for (int i = 0; i < stages; ++i) mbar_init(&full[i], 1);
+      fence_mbar_init();
+    }
+  }
+  __syncthreads();
+  if (!s_tile[0]) return;
+  const int sg = s_tile[1], t0 = s_tile[2] * tq, h0 = blockIdx.y * rt;
+  const int nh = min(rt, a.heads - h0), nt = min(tq, a.seg.len[sg] - t0), pos0 = a.seg.pos[sg] + t0;
+  const int64_t row0 = static_cast<int64_t>(a.seg.row0[sg]) + t0;
+  const int box = 1 << box_shift;
+  const int hi = pos0 + nt - 1, lo = (a.window > 0 ? max(0, pos0 - a.window + 1) : 0) & ~(box - 1);
+  const int per = ((hi - lo + kKeys) / kKeys + a.splits - 1) / a.splits * kKeys;
+  const int first = lo + static_cast<int>(blockIdx.z) * per, last = min(hi, first + per - 1);
+  const int n_stages = last >= first ? (last - first) / kKeys + 1 : 0;
+  const int32_t* bt = a.block_table + static_cast<int64_t>(a.seg.seq[sg]) * a.max_blocks;
+  const int shift = log2_of(a.block_size);
+  // boxes past the last key repeat the last one (masked below), so that every row of a stage holds finite values
+  auto load = [&](int it) {
+    if (threadIdx.x != 0) return;
+    const int s = it % stages;
+    mbar_arrive_expect_tx(&full[s], static_cast<uint32_t>(stage_bytes));
+    for (int b = 0; b < kKeys >> box_shift; ++b) {
+      const int j = min(first + it * kKeys + (b << box_shift), hi & ~(box - 1));
+      tma_load_3d(sKV + s * stage_bytes + b * (a.row * 2 << box_shift), &tm, &full[s], 0,
+                  static_cast<int>(page_slot(bt, a.block_size, shift, j)), 0);
+    }
+  };
+  for (int it = 0; it < min(stages, n_stages); ++it) load(it);
+  {
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q);
+    const int ch = a.row / 8;
+    for (int m = warp; m < ROWS; m += WARPS) {
+      const int tok = m / rt, hh = m % rt;
+      const bool in = tok < nt && hh < nh;
+      const uint4* src = reinterpret_cast<const uint4*>(q + (row0 + tok) * a.ldq + static_cast<int64_t>(h0 + hh) * a.row);
+      for (int c = lane; c < ch; c += 32)
+        *reinterpret_cast<uint4*>(sQ + m * LD + c * 8) = in ? src[c] : make_uint4(0u, 0u, 0u, 0u);
+    }
+  }
+  for (int m = threadIdx.x; m < ROWS; m += THREADS) s_max[m] = -INFINITY;
+  const int mg = warp % S::kMGroups, kg = warp / S::kMGroups;
+  const float mul = a.scale * kLog2e;
+  int vis[S::kMTiles][2];                           // position of this thread's score rows, -1: padding row
+  float sum[S::kMTiles][2];
+#pragma unroll
+  for (int i = 0; i < S::kMTiles; ++i)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int m = (mg * S::kMTiles + i) * 16 + e * 8 + g;
+      vis[i][e] = m / rt < nt && m % rt < nh ? pos0 + m / rt : -1;
+      sum[i][e] = 0.0f;
+    }
+  float o[MT][CT][2][4];
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int c = 0; c < CT; ++c)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[i][c][0][e] = o[i][c][1][e] = 0.0f;
+  // byte offset of a key row inside a stage (slab 0), and the swizzle of its 16-byte chunks
+  auto key_offset = [&](int key) { return (key >> box_shift) * (a.row * 2 << box_shift) + (key & (box - 1)) * 128; };
+  const int slab_bytes = 128 << box_shift;
+  const uint32_t k_off = key_offset(kg * 8 + (lane & 7)), k_swz = lane & 7;      // boxes hold at least eight keys
+  const uint32_t kc0 = ((lane >> 3) ^ k_swz) << 4, kc1 = ((4 + (lane >> 3)) ^ k_swz) << 4;
+  const uint32_t v_off[2] = {static_cast<uint32_t>(key_offset(lane & 15)), static_cast<uint32_t>(key_offset(16 + (lane & 15)))};
+  const uint32_t q_addr = smem_addr(sQ + (mg * S::kMTiles * 16 + (lane & 15)) * LD + (lane >> 4) * 8);
+  __syncthreads();
+  bool ok = true;
+  for (int it = 0; it < n_stages; ++it) {
+    const int s = it % stages, k0 = first + it * kKeys;
+    ok = ok && mbar_wait_bounded(&full[s], (it / stages) & 1, &s_abort);
+    const uint32_t base = smem_u32(sKV) + s * stage_bytes;
+    float sc[S::kMTiles][4], sd[S::kMTiles][4];     // two chains over the columns
+#pragma unroll
+    for (int i = 0; i < S::kMTiles; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sc[i][e] = sd[i][e] = 0.0f;
+#pragma unroll 2
+    for (int b = 0; b < slabs; ++b) {
+      uint32_t ka[4], kb[4];                        // 32 columns each
+      ldmatrix_x4(ka, base + k_off + b * slab_bytes + kc0);
+      ldmatrix_x4(kb, base + k_off + b * slab_bytes + kc1);
+#pragma unroll
+      for (int i = 0; i < S::kMTiles; ++i) {
+        uint32_t q0[4], q1[4], q2[4], q3[4];
+        const uint32_t qa = q_addr + (i * 16 * LD + b * 64) * 2;
+        ldmatrix_x4(q0, qa);
+        ldmatrix_x4(q1, qa + 32);
+        ldmatrix_x4(q2, qa + 64);
+        ldmatrix_x4(q3, qa + 96);
+        mma_bf16(sc[i], q0, ka[0], ka[1]);
+        mma_bf16(sd[i], q1, ka[2], ka[3]);
+        mma_bf16(sc[i], q2, kb[0], kb[1]);
+        mma_bf16(sd[i], q3, kb[2], kb[3]);
+      }
+    }
+    const int kbase = k0 + kg * 8 + t * 2;
+#pragma unroll
+    for (int i = 0; i < S::kMTiles; ++i) {
+      float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int j = kbase + (e & 1), p = vis[i][e >> 1];
+        const bool see = j <= min(p, last) && (a.window <= 0 || j > p - a.window);
+        sc[i][e] = see ? (sc[i][e] + sd[i][e]) * mul : -INFINITY;
+        mx[e >> 1] = fmaxf(mx[e >> 1], sc[i][e]);
+      }
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
+        mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2));
+        if (t == 0) s_part[kg * ROWS + (mg * S::kMTiles + i) * 16 + e * 8 + g] = mx[e];
+      }
+    }
+    __syncthreads();                                // the previous stage has been consumed by every warp, too
+    if (it > 0 && it - 1 + stages < n_stages) load(it - 1 + stages);
+    if (threadIdx.x < ROWS) {
+      const int m = threadIdx.x;
+      const float old = s_max[m];
+      float nm = old;
+#pragma unroll
+      for (int w = 0; w < kKGroups; ++w) nm = fmaxf(nm, s_part[w * ROWS + m]);
+      s_max[m] = nm;
+      s_alpha[m] = nm == -INFINITY ? 1.0f : ex2_approx(old - nm);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < S::kMTiles; ++i)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int m = (mg * S::kMTiles + i) * 16 + e * 8 + g;
+        const float nm = s_max[m], mb = nm == -INFINITY ? 0.0f : nm;
+        const float p0 = ex2_approx(sc[i][2 * e] - mb), p1 = ex2_approx(sc[i][2 * e + 1] - mb);   // -inf: 0
+        sum[i][e] = sum[i][e] * s_alpha[m] + p0 + p1;
+        *reinterpret_cast<uint32_t*>(sP + m * kLdP + kg * 8 + t * 2) = bf16_pair(p0, p1);
+      }
+#pragma unroll
+    for (int i = 0; i < MT; ++i) {
+      const float f0 = s_alpha[i * 16 + g], f1 = s_alpha[i * 16 + 8 + g];
+      if (__any_sync(0xffffffffu, f0 != 1.0f || f1 != 1.0f)) {
+#pragma unroll
+        for (int c = 0; c < CT; ++c)
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            o[i][c][n][0] *= f0;
+            o[i][c][n][1] *= f0;
+            o[i][c][n][2] *= f1;
+            o[i][c][n][3] *= f1;
+          }
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int kk = 0; kk < kKeys / 16; ++kk) {
+      uint32_t pa[MT][4];
+#pragma unroll
+      for (int i = 0; i < MT; ++i)
+        ldmatrix_x4(pa[i], smem_addr(sP + (i * 16 + (lane & 15)) * kLdP + kk * 16 + (lane >> 4) * 8));
+#pragma unroll
+      for (int c = 0; c < CT; ++c) {
+        const int col = (c * WARPS + warp) * 16;
+        if (col >= a.rank) break;
+        uint32_t vb[4];
+        ldmatrix_x4_trans(vb, base + v_off[kk] + (col >> 6) * slab_bytes + (((((col & 63) >> 3) + (lane >> 4)) ^ (lane & 7)) << 4));
+#pragma unroll
+        for (int i = 0; i < MT; ++i) {
+          mma_bf16(o[i][c][0], pa[i], vb[0], vb[1]);
+          mma_bf16(o[i][c][1], pa[i], vb[2], vb[3]);
+        }
+      }
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < S::kMTiles; ++i)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      sum[i][e] += __shfl_xor_sync(0xffffffffu, sum[i][e], 1);
+      sum[i][e] += __shfl_xor_sync(0xffffffffu, sum[i][e], 2);
+      if (t == 0) s_part[kg * ROWS + (mg * S::kMTiles + i) * 16 + e * 8 + g] = sum[i][e];
+    }
+  __syncthreads();
+  if (threadIdx.x < ROWS) {
+    float l = 0.0f;
+#pragma unroll
+    for (int w = 0; w < kKGroups; ++w) l += s_part[w * ROWS + threadIdx.x];
+    s_sum[threadIdx.x] = l;
+  }
+  __syncthreads();
+  if (!ok) {
+    // a wait ran out: time for copies still in flight to land before the shared memory goes away
+    atomicCAS(a.status, 0, kStatusTimeoutProducer);
+    const uint64_t begin = globaltimer_ns();
+    while (globaltimer_ns() - begin < 2000000ull) __nanosleep(2000);
+  }
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int m = i * 16 + e * 8 + g, tok = m / rt, h = h0 + m % rt;
+      if (tok >= nt || m % rt >= nh) continue;
+      const int64_t r = row0 + tok;
+      if (a.splits == 1) {
+        const float f = (a.gate != nullptr ? a.gate[r * a.heads + h] : 1.0f) / s_sum[m];
+        __nv_bfloat16* op = static_cast<__nv_bfloat16*>(a.out) + r * a.ldo + static_cast<int64_t>(h) * a.rank;
+#pragma unroll
+        for (int c = 0; c < CT; ++c)
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            const int col = (c * WARPS + warp) * 16 + n * 8 + t * 2;
+            if (col < a.rank) *reinterpret_cast<uint32_t*>(op + col) = bf16_pair(o[i][c][n][2 * e] * f, o[i][c][n][2 * e + 1] * f);
+          }
+      } else {
+        const int64_t pi = (r * a.heads + h) * a.splits + blockIdx.z;
+#pragma unroll
+        for (int c = 0; c < CT; ++c)
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            const int col = (c * WARPS + warp) * 16 + n * 8 + t * 2;
+            if (col < a.rank)
+              *reinterpret_cast<float2*>(a.part_o + pi * a.rank + col) = make_float2(o[i][c][n][2 * e], o[i][c][n][2 * e + 1]);
+          }
+        if (warp == 0 && t == 0) {
+          a.part_ml[pi * 2] = s_max[m];
+          a.part_ml[pi * 2 + 1] = s_sum[m];
+        }
+      }
+    }
+}
+
+// one block per (segment row, head): the spans of its keys
+__global__ void latent_merge_kernel(const NxLatentAttnArgs a) {
+  const int sg = blockIdx.z, t = blockIdx.x, h = blockIdx.y;
+  if (t >= a.seg.len[sg]) return;
+  const int64_t r = static_cast<int64_t>(a.seg.row0[sg]) + t, base = (r * a.heads + h) * a.splits;
+  float gm = -INFINITY, gl = 0.0f;
+  for (int s = 0; s < a.splits; ++s) gm = fmaxf(gm, a.part_ml[(base + s) * 2]);
+  for (int s = 0; s < a.splits; ++s) {
+    const float m = a.part_ml[(base + s) * 2];
+    gl += m == -INFINITY ? 0.0f : a.part_ml[(base + s) * 2 + 1] * exp2f(m - gm);
+  }
+  const float f = (a.gate != nullptr ? a.gate[r * a.heads + h] : 1.0f) / gl;
+  for (int d = threadIdx.x * 4; d < a.rank; d += blockDim.x * 4) {
+    float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    for (int s = 0; s < a.splits; ++s) {
+      const float m = a.part_ml[(base + s) * 2], w = m == -INFINITY ? 0.0f : exp2f(m - gm) * f;
+      const float4 p = *reinterpret_cast<const float4*>(a.part_o + (base + s) * a.rank + d);
+      v.x += p.x * w;
+      v.y += p.y * w;
+      v.z += p.z * w;
+      v.w += p.w * w;
+    }
+    *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(a.out) + r * a.ldo + static_cast<int64_t>(h) * a.rank + d) =
+        make_uint2(bf16_pair(v.x, v.y), bf16_pair(v.z, v.w));
+  }
+}
+
+template <int MT, int CT>
+int launch(const CUtensorMap& tm, const NxLatentAttnArgs* a, int box_shift, cudaStream_t st) {
+  using S = Shape<MT>;
+  const int stage = kKeys * a->row * 2, fixed = S::kRows * (a->row + 8) * 2 + S::kTail;
+  // two blocks per SM where two stages fit twice, else one block with a deeper ring
+  const int half = (kSmemMax / 2 - 1024 - fixed) / stage;
+  const int stages = std::min(4, half >= 2 ? half : (kSmemMax - 1024 - fixed) / stage);
+  if (stages < 2) return -1;
+  static bool once = false;
+  if (!once) {
+    if (cudaFuncSetAttribute(latent_attn_kernel<MT, CT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemMax - 1024) != cudaSuccess)
+      return -2;
+    once = true;
+  }
+  const int rt = std::min(a->heads, S::kRows), tq = std::max(1, S::kRows / rt);
+  const dim3 grid(a->seg.total_len / tq + a->seg.count, (a->heads + rt - 1) / rt, a->splits);
+  latent_attn_kernel<MT, CT><<<grid, S::kWarps * 32, fixed + stages * stage, st>>>(tm, *a, rt, tq, stages, box_shift);
+  return launch_status();
+}
+
+template <int MT>
+int launch_rank(const CUtensorMap& tm, const NxLatentAttnArgs* a, int box_shift, cudaStream_t st) {
+  constexpr int kW = Shape<MT>::kWarps;
+  if (a->rank <= 128) return launch<MT, 8 / kW>(tm, a, box_shift, st);
+  if (a->rank <= 256) return launch<MT, 16 / kW>(tm, a, box_shift, st);
+  return launch<MT, 32 / kW>(tm, a, box_shift, st);
+}
+
+}  // namespace
+
+extern "C" int nx_latent_attention(const NxLatentAttnArgs* a, nx_stream_t stream) {
+  if (a == nullptr || a->status == nullptr || a->heads <= 0 || a->rank <= 0 || a->rank > 512 || (a->rank & 15)) return -1;
+  if (a->row < a->rank || (a->row & 63) || a->row > 768 || a->block_size < 8 || (a->block_size & 7)) return -1;
+  if (a->max_blocks <= 0 || a->splits < 1 || a->n_slots <= 0) return -1;
+  if (a->splits > 1 && (a->part_o == nullptr || a->part_ml == nullptr)) return -1;
+  if ((a->ldq & 7) || (a->ldo & 7) || a->seg.count > 65535 || a->splits > 65535) return -1;
+  if ((reinterpret_cast<uintptr_t>(a->q) & 15) || (reinterpret_cast<uintptr_t>(a->cache) & 15)) return -1;
+  if (a->seg.count <= 0 || a->seg.max_len <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  int box_shift = 3;                                        // keys of one page per copy: a power of two up to a stage
+  while (box_shift < 5 && a->block_size % (2 << box_shift) == 0) ++box_shift;
+  CUtensorMap tm;
+  {
+    // {64 columns, cache slots, slabs}: one copy brings whole rows, slab by slab
+    nx::EncodeTiledFn fn = nx::encode_tiled_fn();
+    if (fn == nullptr) return -3;
+    const cuuint32_t slabs = static_cast<cuuint32_t>(a->row / 64);
+    cuuint64_t dims[3] = {64, static_cast<cuuint64_t>(a->n_slots), slabs}, strides[2] = {static_cast<cuuint64_t>(a->row) * 2, 128};
+    cuuint32_t box[3] = {64, 1u << box_shift, slabs}, one[3] = {1, 1, 1};
+    if (fn(&tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(a->cache), dims, strides, box, one,
+           CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
+      return -4;
+  }
+  const int rows = a->seg.max_len > 1 ? 64 : a->heads;      // (token, head) pairs of a block
+  const int rc = rows <= 16 ? launch_rank<1>(tm, a, box_shift, st)
+                            : rows <= 32 ? launch_rank<2>(tm, a, box_shift, st) : launch_rank<4>(tm, a, box_shift, st);
+  if (rc == 0 && a->splits > 1) {
+    latent_merge_kernel<<<dim3(a->seg.max_len, a->heads, a->seg.count), std::min(128, (a->rank / 4 + 31) / 32 * 32), 0, st>>>(*a);
+    return launch_status();
+  }
+  return rc;
+}

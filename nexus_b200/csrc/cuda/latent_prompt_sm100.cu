@@ -1,0 +1,464 @@
+// Attention of prompt segments on tcgen05 where a key is a part of its own head beside a part that all heads share (see
+// nx_api_mixers.h).  Queries, keys and values of all segments lie packed in row buffers; a work item is a block of up to 256
+// query rows of one segment and one head.
+//
+// The pipeline is that of the two-tile flash kernel: one persistent CTA per SM, softmax group A (warps 0-3) on query rows
+// 0-127 of the block, group B (warps 4-7) on rows 128-255, both against the same key tiles; the MMA warp interleaves
+//   PV_A(j-1), QK_A(j), PV_B(j-1), QK_B(j).
+// S and O live in TMEM (S_A 0-127, S_B 128-255, O_A 256.., O_B 384..); the probabilities go back as BF16 into the columns of
+// their score tile and are the A operand of P V from there.  O is rescaled only when a row's maximum has grown by 2^8.
+// Key tiles start at the first key the block can see: with a window no tile is wasted on keys before it.  Keys and values
+// have rings of their own, since a key part of 192 columns leaves room for one stage of values.
+#include "flash_common.cuh"
+#include "nx_api_mixers.h"
+#include "sm100_ptx.cuh"
+#include "tensor_map.h"
+
+#include <algorithm>
+
+namespace {
+using namespace nx;
+
+constexpr int kThreads = 320;   // warps 0-3: softmax A, 4-7: softmax B, 8: TMA, 9: MMA
+constexpr int kSlab = 128 * 128;  // bytes of [128 rows][64 columns]
+
+// ND / NV: 64-column slabs of a head's own key part and of its values; the shared part is one slab
+template <int ND, int NV>
+struct Cfg {
+  static constexpr int kQBytes = (ND + 1) * kSlab;
+  static constexpr int kKBytes = (ND + 1) * kSlab;
+  static constexpr int kVBytes = NV * kSlab;
+  static constexpr int kKStages = 2;
+  static constexpr int kVStages = 2 * kQBytes + 2 * kKBytes + 2 * kVBytes <= 224 * 1024 ? 2 : 1;
+  static constexpr int kSmem = 2 * kQBytes + kKStages * kKBytes + kVStages * kVBytes + 256;
+  static_assert(kSmem <= 227 * 1024, "shared memory");
+};
+
+struct Dev {
+  const int32_t* blocks;     // [n_blocks][4]: first row, rows, position of the first row, buffer row of position 0
+  __nv_bfloat16* out;
+  const float* gate;
+  int* status;
+  int64_t ldo;
+  int items, heads, vdim, window, ksteps, rsteps;   // 16-column steps of the own / shared key part
+  float scale;
+};
+
+struct Work {
+  int h, row0, rows, pos0, kv0, k_lo;
+  int jbA, jeA, jbB, jeB, je;      // key tiles of either query tile; tile j holds keys k_lo + 128 j ..
+};
+// CTA c takes items round * grid + c in even rounds and from the other end in odd ones; blocks are sorted by cost
+__device__ __forceinline__ bool next_work(const Dev& p, int round, Work& w) {
+  const int G = static_cast<int>(gridDim.x), c = static_cast<int>(blockIdx.x);
+  const int item = round * G + ((round & 1) ? (G - 1 - c) : c);
+  if (item >= p.items) return false;
+  const int4 b = __ldg(reinterpret_cast<const int4*>(p.blocks) + item / p.heads);
+  w.h = item % p.heads;
+  w.row0 = b.x;
+  w.rows = b.y;
+  w.pos0 = b.z;
+  w.kv0 = b.w;
+  const int back = p.window > 0 ? p.window - 1 : 0x3fffffff;
+  w.k_lo = max(0, w.pos0 - back);
+  w.jbA = 0;
+  w.jeA = (w.pos0 + min(128, w.rows) - 1 - w.k_lo) / 128 + 1;
+  w.jbB = w.jeB = 0;
+  if (w.rows > 128) {
+    w.jbB = (max(0, w.pos0 + 128 - back) - w.k_lo) / 128;
+    w.jeB = (w.pos0 + w.rows - 1 - w.k_lo) / 128 + 1;
+  }
+  w.je = max(w.jeA, w.jeB);
+  return true;
+}
+
+template <int ND, int NV>
+__global__ void __launch_bounds__(kThreads, 1)
+latent_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_qr,
+                     const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_kr,
+                     const __grid_constant__ CUtensorMap tm_v, const Dev p) {
+  using C = Cfg<ND, NV>;
+  constexpr int KS = C::kKStages, VS = C::kVStages;
+  extern __shared__ __align__(1024) uint8_t smem[];
+  if (smem_u32(smem) & 1023u) {  // the swizzled tiles need a 1 KiB aligned base; uniform early exit
+    if (threadIdx.x == 0) atomicCAS(p.status, 0, kStatusBadArgument);
+    return;
+  }
+  uint8_t* sQ = smem;                              // [2] query tiles
+  uint8_t* sK = sQ + 2 * C::kQBytes;               // [KS]
+  uint8_t* sV = sK + KS * C::kKBytes;              // [VS]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + VS * C::kVBytes);
+  uint64_t *q_full = bars, *q_empty = bars + 2, *k_full = bars + 4, *k_empty = bars + 6, *v_full = bars + 8, *v_empty = bars + 10,
+           *s_full = bars + 12, *p_full = bars + 14, *o_done = bars + 16;      // two each
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 18);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x == 0) {
+    for (int x = 0; x < 2; ++x) {
+      mbar_init(&q_full[x], 1);
+      mbar_init(&q_empty[x], 1);
+      mbar_init(&k_full[x], 1);
+      mbar_init(&k_empty[x], 1);
+      mbar_init(&v_full[x], 1);
+      mbar_init(&v_empty[x], 1);
+      mbar_init(&s_full[x], 1);
+      mbar_init(&p_full[x], 4);  // one arrival per softmax warp of the group
+      mbar_init(&o_done[x], 1);
+    }
+    *abort_flag = 0;
+    fence_mbar_init();
+  }
+  if (warp == 9) {
+    tmem_alloc(tmem_slot, 512);
+    tmem_relinquish();
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem_base = *tmem_slot;
+
+  if (warp == 8) {
+    // ------------------------------------------------------------------ TMA producer
+    if (lane == 0) {
+      int nq[2] = {0, 0}, n_kv = 0;
+      bool ok = true;
+      Work w;
+      auto wait = [&](uint64_t* bar, int parity) {
+        if (mbar_wait_bounded(bar, parity, abort_flag)) return true;
+        atomicCAS(p.status, 0, kStatusTimeoutProducer);
+        return false;
+      };
+      for (int round = 0; ok && next_work(p, round, w); ++round) {
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          if (x == 1 && w.jeB <= w.jbB) continue;
+          ok = ok && wait(&q_empty[x], (nq[x] & 1) ^ 1);   // the previous item's Q K^T are done
+          if (!ok) break;
+          ++nq[x];
+          mbar_arrive_expect_tx(&q_full[x], C::kQBytes);
+          uint8_t* d = sQ + x * C::kQBytes;
+#pragma unroll
+          for (int s = 0; s < ND; ++s) tma_load_3d(d + s * kSlab, &tm_q, &q_full[x], 64 * s, w.h, w.row0 + x * 128);
+          tma_load_3d(d + ND * kSlab, &tm_qr, &q_full[x], 0, w.h, w.row0 + x * 128);
+        }
+        for (int j = 0; ok && j < w.je; ++j, ++n_kv) {
+          const int row = w.kv0 + w.k_lo + j * 128;
+          const int s = n_kv % KS, v = n_kv % VS;
+          ok = wait(&k_empty[s], ((n_kv / KS) & 1) ^ 1);
+          if (!ok) break;
+          mbar_arrive_expect_tx(&k_full[s], C::kKBytes);
+          uint8_t* d = sK + s * C::kKBytes;
+#pragma unroll
+          for (int c = 0; c < ND; ++c) tma_load_3d(d + c * kSlab, &tm_k, &k_full[s], 64 * c, w.h, row);
+          tma_load_3d(d + ND * kSlab, &tm_kr, &k_full[s], 0, 0, row);
+          ok = wait(&v_empty[v], ((n_kv / VS) & 1) ^ 1);
+          if (!ok) break;
+          mbar_arrive_expect_tx(&v_full[v], C::kVBytes);
+#pragma unroll
+          for (int c = 0; c < NV; ++c) tma_load_3d(sV + v * C::kVBytes + c * kSlab, &tm_v, &v_full[v], 64 * c, w.h, row);
+        }
+      }
+    }
+  } else if (warp == 9) {
+    // ------------------------------------------------------------------ MMA issuer: the warp walks, one elected lane issues
+    const bool leader = elect_one();
+    const uint32_t idesc_s = make_idesc(kFmtBF16, kFmtBF16, false, false, 128, 128);
+    const uint32_t idesc_o = make_idesc(kFmtBF16, kFmtBF16, false, true, 128, NV * 64);
+    int nq[2] = {0, 0}, np[2] = {0, 0}, n_kv = 0;
+    bool ok = true;
+    Work w;
+    auto wait = [&](uint64_t* bar, int parity) {
+      if (__all_sync(0xffffffffu, mbar_wait_bounded(bar, parity, abort_flag))) return true;
+      if (leader) atomicCAS(p.status, 0, kStatusTimeoutMma);
+      return false;
+    };
+    for (int round = 0; ok && next_work(p, round, w); ++round) {
+      ok = wait(&q_full[0], nq[0] & 1);
+      ++nq[0];
+      if (ok && w.jeB > w.jbB) {
+        ok = wait(&q_full[1], nq[1] & 1);
+        ++nq[1];
+      }
+      const int kv0 = n_kv;
+      for (int j = 0; ok && j <= w.je; ++j) {
+        const int n = kv0 + j, m = n - 1;          // running numbers of key tiles j and j - 1
+        if (j < w.je) ok = wait(&k_full[n % KS], (n / KS) & 1);
+        if (ok && j > 0) ok = wait(&v_full[m % VS], (m / VS) & 1);
+        if (!ok) break;
+        const uint64_t dK = desc_kmajor(smem_u32(sK + (n % KS) * C::kKBytes), 128, 0);
+        const uint64_t dV = desc_mnmajor(smem_u32(sV + ((m + VS) % VS) * C::kVBytes), 128, 0);
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const int jb = x == 0 ? w.jbA : w.jbB, je = x == 0 ? w.jeA : w.jeB;
+          const uint32_t tmem_s = tmem_base + x * 128, tmem_o = tmem_base + 256 + x * 128;
+          if (ok && j - 1 >= jb && j - 1 < je) {   // P_x(j-1) V(j-1)
+            ok = wait(&p_full[x], np[x] & 1);
+            if (ok) {
+              ++np[x];
+              tc_fence_after_sync();
+              const uint32_t acc0 = j - 1 > jb ? 1u : 0u;
+              if (leader) {
+#pragma unroll
+                for (int ks = 0; ks < 8; ++ks)
+                  umma_f16_ts(tmem_o, tmem_s + ks * 8, dV + kstep_mnmajor(ks), idesc_o, ks > 0 ? 1u : acc0);
+                umma_commit(&o_done[x]);
+              }
+            }
+          }
+          if (ok && j >= jb && j < je) {           // S_x(j) = Q_x K(j)^T, own part then shared part
+            tc_fence_after_sync();
+            const uint64_t dQ = desc_kmajor(smem_u32(sQ + x * C::kQBytes), 128, 0);
+            if (leader) {
+              for (int ks = 0; ks < p.ksteps; ++ks)
+                umma_f16_ss(tmem_s, dQ + kstep_kmajor(128, ks), dK + kstep_kmajor(128, ks), idesc_s, ks > 0 ? 1u : 0u);
+              for (int ks = ND * 4; ks < ND * 4 + p.rsteps; ++ks)
+                umma_f16_ss(tmem_s, dQ + kstep_kmajor(128, ks), dK + kstep_kmajor(128, ks), idesc_s, 1u);
+              umma_commit(&s_full[x]);
+              if (j + 1 == je) umma_commit(&q_empty[x]);
+            }
+          }
+        }
+        if (ok && leader) {
+          if (j < w.je) umma_commit(&k_empty[n % KS]);
+          if (j > 0) umma_commit(&v_empty[m % VS]);
+        }
+        __syncwarp();
+      }
+      n_kv = kv0 + w.je;
+    }
+  } else {
+    // ------------------------------------------------------------------ softmax + output rows
+    const int x = warp >> 2, r = (warp & 3) * 32 + lane;   // query tile of this group; row inside it == TMEM lane
+    const uint32_t lane_addr = static_cast<uint32_t>((warp & 3) * 32) << 16;
+    const uint32_t tmem_s = tmem_base + x * 128 + lane_addr, tmem_o = tmem_base + 256 + x * 128 + lane_addr;
+    const float sc = p.scale * kLog2e;
+    int cnt = 0;   // key tiles this group has processed: phase counter of s_full / o_done
+    bool ok = true;
+    Work w;
+    auto wait = [&](uint64_t* bar, int parity) {
+      if (__all_sync(0xffffffffu, mbar_wait_bounded(bar, parity, abort_flag))) return true;
+      if (lane == 0) atomicCAS(p.status, 0, kStatusTimeoutEpilogue);
+      return false;
+    };
+    for (int round = 0; ok && next_work(p, round, w); ++round) {
+      const int jb = x == 0 ? w.jbA : w.jbB, je = x == 0 ? w.jeA : w.jeB;
+      if (je <= jb) continue;
+      const int p0 = w.pos0 + x * 128, pos = p0 + r;
+      const int row_lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+      float m_ref = -INFINITY, l_run = 0.0f;
+      for (int j = jb; j < je; ++j, ++cnt) {
+        const int k0 = w.k_lo + j * 128;
+        ok = wait(&s_full[x], cnt & 1);
+        if (!ok) break;
+        tc_fence_after_sync();
+        uint32_t sv[4][32];
+#pragma unroll
+        for (int cc = 0; cc < 4; ++cc) tmem_ld_32x32b_x32(tmem_s + cc * 32, sv[cc]);
+        tmem_ld_wait();
+        const bool need_mask = k0 + 127 > p0 || (p.window > 0 && k0 < p0 + 127 - p.window + 1);
+        if (need_mask) {
+          const int clo = row_lo - k0, chi = pos - k0;   // column c is visible iff clo <= c <= chi
+#pragma unroll
+          for (int cc = 0; cc < 4; ++cc)
+#pragma unroll
+            for (int c = 0; c < 32; ++c)
+              if (cc * 32 + c < clo || cc * 32 + c > chi) sv[cc][c] = 0xff800000u;  // -inf
+        }
+        float m0 = -INFINITY, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;
+#pragma unroll
+        for (int cc = 0; cc < 4; ++cc)
+#pragma unroll
+          for (int c = 0; c < 32; c += 4) {
+            m0 = fmaxf(m0, __uint_as_float(sv[cc][c]));
+            m1 = fmaxf(m1, __uint_as_float(sv[cc][c + 1]));
+            m2 = fmaxf(m2, __uint_as_float(sv[cc][c + 2]));
+            m3 = fmaxf(m3, __uint_as_float(sv[cc][c + 3]));
+          }
+        const float m_new = fmaxf(m_ref, fmaxf(fmaxf(m0, m1), fmaxf(m2, m3)) * sc);
+        const bool grow = m_new - kRescaleStep > m_ref;
+        if (__any_sync(0xffffffffu, grow)) {
+          const float alpha = grow ? ex2f(m_ref - m_new) : 1.0f;  // m_ref == -inf -> 0
+          if (grow) {
+            l_run *= alpha;
+            m_ref = m_new;
+          }
+          if (j > jb) {  // the output tile holds the sums of the earlier key tiles
+            ok = wait(&o_done[x], (cnt - 1) & 1);
+            if (!ok) break;
+            tc_fence_after_sync();
+#pragma unroll
+            for (int cc = 0; cc < NV * 2; ++cc) {
+              uint32_t ov[32];
+              tmem_ld_32x32b_x32(tmem_o + cc * 32, ov);
+              tmem_ld_wait();
+#pragma unroll
+              for (int c = 0; c < 32; ++c) ov[c] = __float_as_uint(__uint_as_float(ov[c]) * alpha);
+              tmem_st_32x32b_x32(tmem_o + cc * 32, ov);
+            }
+            tmem_st_wait();
+          }
+        }
+        const float m_use = m_ref == -INFINITY ? 0.0f : m_ref;
+        float r0 = 0.0f, r1 = 0.0f, r2 = 0.0f, r3 = 0.0f;
+#pragma unroll
+        for (int cc = 0; cc < 4; ++cc) {
+          uint32_t pk[16];
+#pragma unroll
+          for (int g = 0; g < 4; ++g) {
+            float e[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) e[i] = ex2f(fmaf(__uint_as_float(sv[cc][8 * g + i]), sc, -m_use));  // -inf -> 0
+            r0 += e[0] + e[4];
+            r1 += e[1] + e[5];
+            r2 += e[2] + e[6];
+            r3 += e[3] + e[7];
+            pk[4 * g + 0] = pack_bf16x2(e[0], e[1]);
+            pk[4 * g + 1] = pack_bf16x2(e[2], e[3]);
+            pk[4 * g + 2] = pack_bf16x2(e[4], e[5]);
+            pk[4 * g + 3] = pack_bf16x2(e[6], e[7]);
+          }
+          tmem_st_32x32b_x16(tmem_s + cc * 16, pk);  // two probabilities per column
+        }
+        l_run += (r0 + r1) + (r2 + r3);
+        tmem_st_wait();
+        tc_fence_before_sync();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&p_full[x]);
+      }
+      if (!ok) break;
+      ok = wait(&o_done[x], (cnt - 1) & 1);        // the last P V has retired
+      if (!ok) break;
+      tc_fence_after_sync();
+      const bool row_ok = x * 128 + r < w.rows;
+      const int64_t row = w.row0 + x * 128 + r;
+      const float inv = row_ok ? (p.gate != nullptr ? p.gate[row * p.heads + w.h] : 1.0f) / l_run : 0.0f;
+      __nv_bfloat16* orow = p.out + row * p.ldo + static_cast<int64_t>(w.h) * p.vdim;
+#pragma unroll
+      for (int cc = 0; cc < NV * 2; ++cc) {
+        uint32_t ov[32];
+        tmem_ld_32x32b_x32(tmem_o + cc * 32, ov);
+        tmem_ld_wait();
+        if (!row_ok) continue;
+#pragma unroll
+        for (int g = 0; g < 4; ++g) {
+          if (cc * 32 + g * 8 >= p.vdim) continue;
+          uint4 wv;
+          wv.x = pack_bf16x2(__uint_as_float(ov[8 * g + 0]) * inv, __uint_as_float(ov[8 * g + 1]) * inv);
+          wv.y = pack_bf16x2(__uint_as_float(ov[8 * g + 2]) * inv, __uint_as_float(ov[8 * g + 3]) * inv);
+          wv.z = pack_bf16x2(__uint_as_float(ov[8 * g + 4]) * inv, __uint_as_float(ov[8 * g + 5]) * inv);
+          wv.w = pack_bf16x2(__uint_as_float(ov[8 * g + 6]) * inv, __uint_as_float(ov[8 * g + 7]) * inv);
+          *reinterpret_cast<uint4*>(orow + cc * 32 + g * 8) = wv;
+        }
+      }
+      tc_fence_before_sync();
+    }
+  }
+
+  tc_fence_before_sync();
+  __syncthreads();
+  if (*abort_flag != 0) {
+    const uint64_t t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 2000000ull) __nanosleep(2000);
+    __syncthreads();
+  }
+  if (warp == 9) {
+    tc_fence_after_sync();
+    tmem_dealloc(tmem_base, 512);
+  }
+}
+
+template <int ND, int NV>
+int launch(const NxLatentPromptArgs* a, const CUtensorMap& tq, const CUtensorMap& tqr, const CUtensorMap& tk, const CUtensorMap& tkr,
+           const CUtensorMap& tv, const Dev& p, int grid, cudaStream_t st) {
+  constexpr int kSmem = Cfg<ND, NV>::kSmem;
+  static bool once = false;
+  if (!once) {
+    if (cudaFuncSetAttribute(latent_prompt_kernel<ND, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -2;
+    once = true;
+  }
+  latent_prompt_kernel<ND, NV><<<grid, kThreads, kSmem, st>>>(tq, tqr, tk, tkr, tv, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+
+// copies the cache rows of a segment list into one packed buffer: keys `base` .. of every segment, 16 bytes per thread
+__global__ void latent_gather_kernel(const uint4* __restrict__ cache, uint4* __restrict__ dst, const int32_t* __restrict__ table,
+                                     const int32_t* __restrict__ list, int n, int max_blocks, int block_size, int chunks) {
+  // list [n][4]: first destination row, rows, first position, sequence
+  const int seg = blockIdx.y, count = list[seg * 4 + 1];
+  const int64_t d0 = list[seg * 4], seq = list[seg * 4 + 3];
+  const int p0 = list[seg * 4 + 2];
+  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < static_cast<int64_t>(count) * chunks;
+       i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int k = static_cast<int>(i / chunks), c = static_cast<int>(i % chunks), j = p0 + k;
+    const int64_t slot = static_cast<int64_t>(table[seq * max_blocks + j / block_size]) * block_size + j % block_size;
+    dst[(d0 + k) * chunks + c] = cache[slot * chunks + c];
+  }
+}
+
+}  // namespace
+
+extern "C" int nx_latent_gather(const void* cache, void* dst, const int32_t* block_table, const int32_t* list, int segments,
+                                int longest, int max_blocks, int block_size, int row, nx_stream_t stream) {
+  if (segments < 0 || segments > 65535 || block_size <= 0 || max_blocks <= 0 || row <= 0 || (row & 7)) return -1;
+  if ((reinterpret_cast<uintptr_t>(cache) & 15) || (reinterpret_cast<uintptr_t>(dst) & 15)) return -1;
+  if (segments == 0 || longest <= 0) return 0;
+  const int64_t work = (static_cast<int64_t>(longest) * (row / 8) + 255) / 256;
+  const dim3 grid(static_cast<unsigned>(std::min<int64_t>(work, 1024)), segments);
+  latent_gather_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(
+      static_cast<const uint4*>(cache), static_cast<uint4*>(dst), block_table, list, segments, max_blocks, block_size, row / 8);
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+
+extern "C" int nx_latent_prompt(const NxLatentPromptArgs* a, nx_stream_t stream) {
+  if (a == nullptr || a->status == nullptr || a->blocks == nullptr || a->heads <= 0 || !(a->scale > 0.0f)) return -1;
+  if (a->dim <= 0 || a->dim > 128 || a->rot <= 0 || a->rot > 64 || a->vdim <= 0 || a->vdim > 128) return -1;
+  if ((a->dim & 15) || (a->rot & 15) || (a->vdim & 7)) return -1;
+  if ((a->ldq | a->ldkv | a->ld_lat | a->ldo | a->q_head) & 7) return -1;
+  for (const void* ptr : {a->q, a->kv, a->lat, static_cast<const void*>(a->out)})
+    if (ptr == nullptr || (reinterpret_cast<uintptr_t>(ptr) & 15)) return -1;
+  if (a->n_blocks <= 0) return 0;
+  CUtensorMap tq, tqr, tk, tkr, tv;
+  const auto bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  const auto* q = static_cast<const __nv_bfloat16*>(a->q);
+  const auto* kv = static_cast<const __nv_bfloat16*>(a->kv);
+  const auto* lat = static_cast<const __nv_bfloat16*>(a->lat);
+  const uint64_t H = static_cast<uint64_t>(a->heads);
+  // {columns, heads, rows}, box {64, 1, 128}: columns past a part's width arrive as zeros
+  const auto map = [&](CUtensorMap* m, const __nv_bfloat16* base, uint64_t cols, uint64_t heads, uint64_t rows, uint64_t head_ld,
+                        uint64_t row_ld) {
+    nx::EncodeTiledFn fn = nx::encode_tiled_fn();
+    if (fn == nullptr) return -3;
+    cuuint64_t dims[3] = {cols, heads, rows}, strides[2] = {head_ld * 2, row_ld * 2};
+    cuuint32_t box[3] = {64, 1, 128}, one[3] = {1, 1, 1};
+    return fn(m, bf, 3, const_cast<__nv_bfloat16*>(base), dims, strides, box, one, CU_TENSOR_MAP_INTERLEAVE_NONE,
+              CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS
+               ? 0
+               : -4;
+  };
+  int rc;
+  if ((rc = map(&tq, q, a->dim, H, a->q_rows, a->q_head, a->ldq))) return rc;
+  if ((rc = map(&tqr, q + a->dim, a->rot, H, a->q_rows, a->q_head, a->ldq))) return rc;
+  if ((rc = map(&tk, kv, a->dim, H, a->kv_rows, a->dim, a->ldkv))) return rc;
+  if ((rc = map(&tv, kv + static_cast<int64_t>(H) * a->dim, a->vdim, H, a->kv_rows, a->vdim, a->ldkv))) return rc;
+  if ((rc = map(&tkr, lat + a->rank, a->rot, 1, a->kv_rows, a->ld_lat, a->ld_lat))) return rc;
+  Dev p{};
+  p.blocks = a->blocks;
+  p.out = static_cast<__nv_bfloat16*>(a->out);
+  p.gate = a->gate;
+  p.status = a->status;
+  p.ldo = a->ldo;
+  p.items = a->n_blocks * a->heads;
+  p.heads = a->heads;
+  p.vdim = a->vdim;
+  p.window = a->window;
+  p.ksteps = a->dim / 16;
+  p.rsteps = a->rot / 16;
+  p.scale = a->scale;
+  int sms = 0, dev = 0;
+  if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) return -2;
+  const int grid = std::min(p.items, sms);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (a->dim <= 64) return a->vdim <= 64 ? launch<1, 1>(a, tq, tqr, tk, tkr, tv, p, grid, st) : launch<1, 2>(a, tq, tqr, tk, tkr, tv, p, grid, st);
+  return a->vdim <= 64 ? launch<2, 1>(a, tq, tqr, tk, tkr, tv, p, grid, st) : launch<2, 2>(a, tq, tqr, tk, tkr, tv, p, grid, st);
+}

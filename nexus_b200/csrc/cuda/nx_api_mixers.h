@@ -205,6 +205,50 @@ int nx_paged_window_prefill(const NxPagedWindowArgs* args, nx_stream_t stream);
 // any segments, FP32
 int nx_paged_window_f32(const NxPagedWindowArgs* args, nx_stream_t stream);
 
+
+// Attention of packed query rows over a latent cache, BF16: every head meets the same cache row [latent (rank) | rotated key
+// part], whose leading `rank` columns are the values.  score = scale * q . row; out = gate * softmax-weighted sum of the
+// latents.  Windows as above.
+typedef struct NxLatentAttnArgs {
+  const void* q;           // [rows, ldq]: heads * row
+  const void* cache;       // [blocks * block_size, row]
+  const int32_t* block_table;  // [slots, max_blocks]
+  void* out;               // [rows, ldo]: heads * rank
+  const float* gate;       // [rows, heads], may be null
+  float* part_o;           // splits > 1: [rows, heads, splits, rank]
+  float* part_ml;          // splits > 1: [rows, heads, splits, 2]
+  int* status;
+  int64_t ldq, ldo;
+  int32_t heads, row, rank, block_size, max_blocks, window, splits;   // row a multiple of 64 up to 768, rank of 16 up to 512,
+  int32_t n_slots;                                                    // block_size of 8; n_slots = blocks * block_size
+  float scale;
+  NxSegments seg;
+} NxLatentAttnArgs;
+int nx_latent_attention(const NxLatentAttnArgs* args, nx_stream_t stream);
+
+// The same attention for prompts, BF16, on keys and values formed from the latents: a head's key is its own part (dim) beside
+// the shared rotated part (rot).  q [q_rows, ldq]: head h at h * q_head, own part then rotated part; kv [kv_rows, ldkv]:
+// heads * dim keys, heads * vdim values; lat [kv_rows, ld_lat]: latent rows, the shared key part at column `rank`.
+// blocks [n_blocks, 4]: first row of q, rows (1..256), position of the first row, row of kv / lat that position 0 would have
+// (rows of positions no row can see need not exist); most expensive blocks first.  out [., ldo]: heads * vdim, times the gate.
+typedef struct NxLatentPromptArgs {
+  const void* q;
+  const void* kv;
+  const void* lat;
+  void* out;
+  const float* gate;       // [rows, heads], may be null
+  const int32_t* blocks;   // 16-byte aligned
+  int* status;
+  int64_t ldq, ldkv, ld_lat, ldo;
+  int32_t n_blocks, q_rows, kv_rows, q_head, rank, heads, dim, rot, vdim, window;  // dim <= 128, rot <= 64: multiples of 16;
+  float scale;                                                                     // vdim <= 128: multiple of 8; scale > 0
+} NxLatentPromptArgs;
+int nx_latent_prompt(const NxLatentPromptArgs* args, nx_stream_t stream);
+// Cache rows of `segments` runs of positions into one packed buffer.  list [segments, 4]: first destination row, rows, first
+// position, sequence; `longest`: most rows of a run.
+int nx_latent_gather(const void* cache, void* dst, const int32_t* block_table, const int32_t* list, int segments, int longest,
+                     int max_blocks, int block_size, int row, nx_stream_t stream);
+
 #ifdef __cplusplus
 }
 #endif

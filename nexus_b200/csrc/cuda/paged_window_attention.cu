@@ -4,6 +4,7 @@
 // heads of one token in decoding.  Scores, soft-capping and softmax are FP32; only the products take BF16 operands.
 #include "mixer_common.cuh"
 #include "nx_api_mixers.h"
+#include "paged_common.cuh"
 
 #include <algorithm>
 
@@ -36,34 +37,8 @@ struct ScoreMap {
   }
 };
 
-// which segment, and which tile of `per` tokens inside it, flat tile index `tile` is; executed by one full warp
-__device__ __forceinline__ bool find_tile(const NxSegments& s, int per, int tile, int& seg, int& off) {
-  const int lane = threadIdx.x & 31;
-  int base = 0;
-  for (int i0 = 0; i0 < s.count; i0 += 32) {
-    const int i = i0 + lane;
-    const int n = i < s.count ? (s.len[i] + per - 1) / per : 0;
-    int incl = n;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const int v = __shfl_up_sync(0xffffffffu, incl, o);
-      if (lane >= o) incl += v;
-    }
-    const unsigned hit = __ballot_sync(0xffffffffu, base + incl > tile);
-    if (hit) {
-      const int first = __ffs(hit) - 1;
-      seg = i0 + first;
-      off = tile - base - __shfl_sync(0xffffffffu, incl - n, first);
-      return true;
-    }
-    base += __shfl_sync(0xffffffffu, incl, 31);
-  }
-  return false;
-}
-
 // One stage of keys and values into shared memory, each [kKeys][DP + 8]; keys past `last` and columns past the head size
 // become zeros.
-__device__ __forceinline__ int log2_of(int n) { return (n & (n - 1)) == 0 ? 31 - __clz(n) : -1; }
 struct KvSource {
   const __nv_bfloat16 *k, *v;
   const int32_t* bt;
@@ -75,8 +50,7 @@ struct KvSource {
         bt(a.block_table + static_cast<int64_t>(seq) * a.max_blocks), k_pitch(a.k_pitch), v_pitch(a.v_pitch),
         block_size(a.block_size), shift(log2_of(a.block_size)), dim(a.dim), vdim(a.vdim) {}
   __device__ __forceinline__ int64_t slot(int j) const {
-    if (shift >= 0) return (static_cast<int64_t>(bt[j >> shift]) << shift) + (j & (block_size - 1));
-    return static_cast<int64_t>(bt[j / block_size]) * block_size + j % block_size;
+    return page_slot(bt, block_size, shift, j);
   }
 };
 __device__ __forceinline__ void copy8(__nv_bfloat16* d, const __nv_bfloat16* s, int c, int cols) {   // columns c .. c + 7 of a row

@@ -60,6 +60,10 @@ class HybridEngine(Engine):
             m = layer.mixer
             if self.fast and isinstance(m, ParallelSpec) and max(m.left.dim, m.left.vdim) > 256:
                 raise ValueError(f"layer {i}: the BF16 attention kernels take head sizes up to 256")
+            if isinstance(m, LatentSpec):
+                latent.check(self, i, m)
+            if layer.experts and layer.experts.shared and self.model.pre_norm:
+                raise ValueError(f"layer {i}: the gate of the shared expert reads the residual stream, which this design norms first")
         self.adt = torch.bfloat16 if self.fast else torch.float32
         self.kv_kind = 0
         elem = 2 if self.fast else 4
@@ -222,6 +226,7 @@ class HybridEngine(Engine):
         self._stepped = M.Segments(table, 0, single.count + short.count, max(single.max_len, short.max_len),
                                    single.total + short.total)
         self._every = M.Segments(table, 0, first, max(g.max_len for g in groups), sum(g.total for g in groups))
+        latent.plan(self)
         return self._body(dv[0], dv[1], dv[2], dv[3], dv[4], dv[5][:logit_rows], runs, nl)
 
     def _buffer(self, rows: int, cols: int) -> torch.Tensor:

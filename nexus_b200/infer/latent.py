@@ -1,6 +1,6 @@
 """Latent attention (`lm.hybrid.LatentSpec`) on the engine: packed weights, the latent cache, and the forms a step can take.
 
-A token's cache row is [latent | rotated key part], each part zero-padded to a multiple of 16 columns, shared by all heads.
+A token's cache row is [latent | rotated key part], zero-padded to a multiple of 64 columns, shared by all heads.
 Queries can meet it in two ways that give the same sums:
 
 * absorbed: W_uk goes to the query side, q_lat = W_uk^T q, and the scores are products with the cache rows themselves; the
@@ -28,7 +28,19 @@ class LatentShape:
         self.dim, self.rot = _pad(m.dim, 16), _pad(m.rope_dims, 16)
         self.vdim, self.rank = _pad(m.vdim, 8), _pad(m.kv_rank, 16)
         self.head = self.dim + self.rot          # columns of a query head
-        self.row = self.rank + self.rot          # columns of a cache row
+        self.row = _pad(self.rank + self.rot, 64)     # columns of a cache row
+
+
+def check(engine, i: int, m: LatentSpec) -> None:
+    from ..ops import _mixers as M
+    s = LatentShape(m)
+    if engine.fast and (s.rank > M.LATENT_MAX_RANK or s.row > M.LATENT_MAX_ROW):
+        raise ValueError(f"layer {i}: the BF16 kernels take latents of up to {M.LATENT_MAX_RANK} columns, cache rows of up to "
+                         f"{M.LATENT_MAX_ROW}")
+    if engine.fast and engine.cfg.block_size % 8:
+        raise ValueError(f"layer {i}: the BF16 kernels take pages of a multiple of 8 tokens")
+    if not engine.fast and s.rank > 1024:
+        raise ValueError(f"layer {i}: the FP32 kernel takes latents of up to 1024 columns")
 
 
 def load(engine, m: LatentSpec, get) -> dict:
@@ -72,34 +84,135 @@ def absorbed(engine, i: int, m: LatentSpec, lw: dict, q, gate, pos, out, groups)
     ql = torch.empty((n, H, s.row), dtype=q.dtype, device=q.device)
     _per_head(engine, q.view(n, H, s.head)[:, :, : s.dim].permute(1, 0, 2), lw["uk"], ql[:, :, : s.rank].permute(1, 0, 2), True)
     ql = ql.view(n, H * s.row)
-    M.rope_heads(q, s.head, s.dim, ql, s.row, s.rank, H, m.rope_dims, s.rot, pos, *lw["rope"])
+    M.rope_heads(q, s.head, s.dim, ql, s.row, s.rank, H, m.rope_dims, s.row - s.rank, pos, *lw["rope"])
     ol = torch.empty((n, H * s.rank), dtype=q.dtype, device=q.device)
     for seg in groups:
         if seg.count:
-            M.paged_window_attention(ql, engine.k_cache[i], None, engine.block_table, ol, seg, heads=H,
-                                     block_size=engine.cfg.block_size, window=m.window, scale=m.scale, gate=gate, vdim=s.rank,
-                                     splits=splits(engine, m, seg.count))
+            if engine.fast:
+                M.latent_attention(ql, engine.k_cache[i], engine.block_table, ol, seg, heads=H, rank=s.rank, window=m.window,
+                                   scale=m.scale, gate=gate, splits=splits(engine, m, seg))
+            else:
+                M.paged_window_attention(ql, engine.k_cache[i], None, engine.block_table, ol, seg, heads=H,
+                                         block_size=engine.cfg.block_size, window=m.window, scale=m.scale, gate=gate, vdim=s.rank)
     _per_head(engine, ol.view(n, H, s.rank).permute(1, 0, 2), lw["uv"], out.view(n, H, s.vdim).permute(1, 0, 2), False)
 
 
-def splits(engine, m: LatentSpec, rows: int) -> int:
+def splits(engine, m: LatentSpec, seg) -> int:
+    """Spans of the keys: enough blocks for every SM, at least 128 keys each."""
+    if seg.max_len > 1:
+        return 1
     if engine.cfg.decode_splits > 0:
         return engine.cfg.decode_splits
     keys = min(m.window, engine.ctx) if m.window > 0 else engine.ctx
-    ctas = rows * (-(-m.heads // 16))
-    return max(1, min(296 // max(ctas, 1), -(-keys // 128), 32))
+    blocks = seg.count * -(-m.heads // 64)
+    return max(1, min(-(-148 // blocks), -(-keys // 128), 32))
+
+
+def expandable(m: LatentSpec) -> bool:
+    s = LatentShape(m)
+    return s.dim <= 128 and s.rot <= 64 and s.vdim <= 128 and m.scale > 0
+
+
+class StepPlan:
+    """How the segments of a step that has long ones are split between the two forms; built on the host once per step.
+
+    ``rows``: the rows of the one-token and short segments, ``groups`` these segments over the compacted rows.  Per window:
+    ``blocks``, query blocks of the long segments in the order of their cost, and ``runs``, what to gather from the cache
+    when a long segment does not start at position 0 (else the keys are the rows of the step)."""
+
+    def __init__(self, engine, windows):
+        from ..ops import _mixers as M
+        single, short, long_ = engine._groups
+        host, n = engine._host_rows[engine.INDEX_ROWS:], single.count + short.count
+        segs = [tuple(int(v) for v in host[:, j]) for j in range(n + long_.count)]
+        data, at = [], {}
+
+        def put(name, values):
+            at[name] = (len(data), len(values))
+            data.extend(values)
+            data.extend([0] * (-len(data) % 4))        # tables start on 16 bytes
+        first, table = 0, [[], [], [], []]
+        for row0, count, pos, seq in segs[:n]:
+            for t, v in zip(table, (first, count, pos, seq)):
+                t.append(v)
+            first += count
+        put("rows", [r for row0, count, _, _ in segs[:n] for r in range(row0, row0 + count)])
+        put("table", [v for t in table for v in t])
+        self.gathered = any(pos > 0 for _, _, pos, _ in segs[n:])
+        self.kv_rows: Dict[int, int] = {}
+        for w in windows:
+            back, blocks, runs, d = w - 1 if w > 0 else 1 << 30, [], [], 0
+            for row0, count, pos, seq in segs[n:]:
+                base = max(0, pos - back) if self.gathered else 0
+                kv0 = d - base if self.gathered else row0
+                runs += [d, pos + count - base, base, seq]
+                d += pos + count - base
+                for b in range(0, count, 256):
+                    rows = min(256, count - b)
+                    blocks.append((min(pos + b, back) + rows, row0 + b, rows, pos + b, kv0))
+            blocks.sort(key=lambda x: -x[0])
+            put(("blocks", w), [v for b in blocks for v in b[1:]])
+            put(("runs", w), runs)
+            self.kv_rows[w] = d
+        dev = torch.tensor(data, dtype=torch.int32).pin_memory().to(engine.dev, non_blocking=True)
+
+        def get(name):
+            return dev[at[name][0]: at[name][0] + at[name][1]]
+        self.blocks = {w: get(("blocks", w)).view(-1, 4) for w in windows}
+        self.runs = {w: get(("runs", w)).view(-1, 4) for w in windows}
+        self.longest = {w: max(pos + count - max(0, pos - (w - 1 if w > 0 else 1 << 30)) for _, count, pos, _ in segs[n:])
+                        for w in windows}
+        self.rows = get("rows").long() if n else None
+        if n:
+            t = get("table").view(4, n)
+            self.groups = [M.Segments(t, 0, single.count, single.max_len, single.total),
+                           M.Segments(t, single.count, short.count, short.max_len, short.total)]
+
+
+def plan(engine) -> None:
+    """Called once per step, before the layers."""
+    engine._latent_plan = None
+    if not engine.fast or engine._groups[2].count == 0:
+        return
+    windows = sorted({x.mixer.window for x in engine.model.layers if isinstance(x.mixer, LatentSpec) and expandable(x.mixer)})
+    if windows:
+        engine._latent_plan = StepPlan(engine, windows)
+
+
+def expanded(engine, i: int, m: LatentSpec, lw: dict, q, lat, gate, pos, out, step: StepPlan) -> None:
+    """The long segments of a step.  ``lat``: latent rows of the step; ``q`` is rotated in place."""
+    from ..ops import _mixers as M
+    s, w = lw["shape"], m.window
+    if step.gathered:
+        lat = torch.empty((step.kv_rows[w], s.row), dtype=engine.adt, device=engine.dev)
+        M.latent_gather(engine.k_cache[i], engine.block_table, step.runs[w], step.longest[w], lat)
+    kv = engine._linear(lat[:, : s.rank], lw["ukv"])
+    M.rope_heads(q, s.head, s.dim, q, s.head, s.dim, m.heads, m.rope_dims, s.rot, pos, *lw["rope"])
+    M.latent_prompt(q, kv, lat, out, step.blocks[w], heads=m.heads, dim=s.dim, rot=s.rot, vdim=s.vdim, rank=s.rank, window=w,
+                    scale=m.scale, gate=gate)
 
 
 def mixer(engine, i: int, m: LatentSpec, lw: dict, h, pos, slot):
     from ..ops import _mixers as M
     s, n = lw["shape"], h.shape[0]
+    step = engine._latent_plan if expandable(m) else None
     proj = engine._linear(h, lw["in"])
     cq = torch.empty((n, _pad(m.q_rank, 8)), dtype=engine.adt, device=engine.dev)
     gate = torch.empty((n, m.heads), dtype=torch.float32, device=engine.dev)
+    lat = torch.empty((n, s.row), dtype=engine.adt, device=engine.dev) if step is not None and not step.gathered else None
     M.latent_prep(proj, lw["off"], m.q_rank, m.kv_rank, m.rope_dims, m.heads, lw["w_q"], lw["w_kv"], pos, slot, *lw["rope"], cq,
-                  engine.k_cache[i], s.rank, gate, eps=engine.model.norm_eps)
+                  engine.k_cache[i], s.rank, gate, eps=engine.model.norm_eps, lat=lat)
     q = engine._linear(cq, lw["uq"])
     out = torch.empty((n, m.heads * s.vdim), dtype=engine.adt, device=engine.dev)
-    groups = [engine._every] if not engine.fast else [engine._groups[0], engine._many]
-    absorbed(engine, i, m, lw, q, gate, pos, out, groups)
+    if step is None:
+        groups = [engine._groups[0], engine._many] if engine.fast else [engine._every]
+        absorbed(engine, i, m, lw, q, gate, pos, out, groups)
+    else:
+        if step.rows is not None:       # before the rotation in place
+            part = torch.empty((step.rows.shape[0], out.shape[1]), dtype=engine.adt, device=engine.dev)
+            absorbed(engine, i, m, lw, q.index_select(0, step.rows), gate.index_select(0, step.rows), pos.index_select(0, step.rows),
+                     part, step.groups)
+        expanded(engine, i, m, lw, q, lat, gate, pos, out, step)
+        if step.rows is not None:
+            out.index_copy_(0, step.rows, part)
     return engine._linear(out, lw["out"])

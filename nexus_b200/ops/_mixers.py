@@ -82,6 +82,24 @@ class PagedWindowArgs(C.Structure):
                 ("seg", SegmentArgs), ("k_pitch", C.c_int64), ("v_pitch", C.c_int64), ("gate", C.c_void_p)]
 
 
+class LatentPromptArgs(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("kv", C.c_void_p), ("lat", C.c_void_p), ("out", C.c_void_p), ("gate", C.c_void_p),
+                ("blocks", C.c_void_p), ("status", C.c_void_p), ("ldq", C.c_int64), ("ldkv", C.c_int64), ("ld_lat", C.c_int64),
+                ("ldo", C.c_int64), ("n_blocks", C.c_int32), ("q_rows", C.c_int32), ("kv_rows", C.c_int32), ("q_head", C.c_int32),
+                ("rank", C.c_int32), ("heads", C.c_int32), ("dim", C.c_int32), ("rot", C.c_int32), ("vdim", C.c_int32),
+                ("window", C.c_int32), ("scale", C.c_float)]
+
+
+class LatentAttnArgs(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("cache", C.c_void_p), ("block_table", C.c_void_p), ("out", C.c_void_p), ("gate", C.c_void_p),
+                ("part_o", C.c_void_p), ("part_ml", C.c_void_p), ("status", C.c_void_p), ("ldq", C.c_int64), ("ldo", C.c_int64),
+                ("heads", C.c_int32), ("row", C.c_int32), ("rank", C.c_int32), ("block_size", C.c_int32), ("max_blocks", C.c_int32),
+                ("window", C.c_int32), ("splits", C.c_int32), ("n_slots", C.c_int32), ("scale", C.c_float), ("seg", SegmentArgs)]
+
+
+LATENT_MAX_RANK, LATENT_MAX_ROW = 512, 768
+
+
 @dataclass
 class Segments:
     """A range of a device segment table ``[4, width]`` (first row, rows, first position, sequence)."""
@@ -242,3 +260,33 @@ def paged_window_attention(q, k_cache, v_cache, block_table, out, seg: Segments,
         K._check(K.lib().nx_paged_window_decode(C.byref(a), K._stream()), "nx_paged_window_decode")
     else:
         K._check(K.lib().nx_paged_window_prefill(C.byref(a), K._stream()), "nx_paged_window_prefill")
+
+
+def latent_attention(q, cache, block_table, out, seg: Segments, *, heads, rank, window, scale, gate=None, splits=1) -> None:
+    """q: BF16 [rows, heads * row]; cache [blocks, block_size, 1, row], the values are its leading ``rank`` columns; out
+    [rows, heads * rank]; ``splits`` spans of the keys run at the same time."""
+    a = LatentAttnArgs(_ptr(q), _ptr(cache), _ptr(block_table), _ptr(out), _ptr(gate), None, None,
+                       K.status_word(q.device).data_ptr(), q.stride(0), out.stride(0), heads, cache.shape[-1], rank, cache.shape[1],
+                       block_table.shape[1], window, splits, cache.shape[0] * cache.shape[1], scale, seg.args())
+    if splits > 1:
+        n = q.shape[0] * heads * splits
+        a.part_o = K.scratch(n * rank * 4, "latent_o", q.device).data_ptr()
+        a.part_ml = K.scratch(n * 8, "latent_ml", q.device).data_ptr()
+    K._check(K.lib().nx_latent_attention(C.byref(a), K._stream()), "nx_latent_attention")
+
+
+def latent_prompt(q, kv, lat, out, blocks, *, heads, dim, rot, vdim, rank, window, scale, gate=None) -> None:
+    """The same attention on formed keys and values (tcgen05).  q [rows, heads * (dim + rot)], kv [kv rows, heads * (dim + vdim)],
+    lat [kv rows, row]: the shared key part at column ``rank``; blocks int32 [n, 4] of up to 256 query rows: first row, rows,
+    position of the first row, kv row of position 0."""
+    a = LatentPromptArgs(_ptr(q), _ptr(kv), _ptr(lat), _ptr(out), _ptr(gate), _ptr(blocks), K.status_word(q.device).data_ptr(),
+                         q.stride(0), kv.stride(0), lat.stride(0), out.stride(0), blocks.shape[0], q.shape[0], kv.shape[0], dim + rot,
+                         rank, heads, dim, rot, vdim, window, scale)
+    K._check(K.lib().nx_latent_prompt(C.byref(a), K._stream()), "nx_latent_prompt")
+
+
+def latent_gather(cache, block_table, runs, longest, dst) -> None:
+    """Cache rows of ``runs`` (int32 [n, 4]: first row of ``dst``, rows, first position, sequence) into ``dst`` [., row]."""
+    K._check(K.lib().nx_latent_gather(K._p(cache), K._p(dst), K._p(block_table), K._p(runs), C.c_int(runs.shape[0]), C.c_int(longest),
+                                      C.c_int(block_table.shape[1]), C.c_int(cache.shape[1]), C.c_int(cache.shape[-1]), K._stream()),
+             "nx_latent_gather")
