@@ -12,6 +12,7 @@
 #include "tensor_map.h"
 
 #include <algorithm>
+#include <type_traits>
 
 namespace {
 using namespace nx;
@@ -34,7 +35,7 @@ struct Shape {
 
 // CT: 16-column tiles of the latent per warp.  A box holds `1 << box_shift` keys of one page.
 template <int MT, int CT>
-__global__ void __launch_bounds__(Shape<MT>::kWarps * 32)
+__global__ void __launch_bounds__(Shape<MT>::kWarps * 32, MT == 1 ? 2 : 1)
 latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArgs a, int rt, int tq, int stages, int box_shift) {
   using S = Shape<MT>;
   constexpr int ROWS = S::kRows, WARPS = S::kWarps, THREADS = WARPS * 32;
@@ -123,11 +124,14 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
 #pragma unroll
       for (int e = 0; e < 4; ++e) o[i][c][0][e] = o[i][c][1][e] = 0.0f;
   // byte offset of a key row inside a stage (slab 0), and the swizzle of its 16-byte chunks
-  auto key_offset = [&](int key) { return (key >> box_shift) * (a.row * 2 << box_shift) + (key & (box - 1)) * 128; };
+  auto key_offset = [&](int key) -> uint32_t { return (key >> box_shift) * (a.row * 2 << box_shift) + (key & (box - 1)) * 128; };
   const int slab_bytes = 128 << box_shift;
   const uint32_t k_off = key_offset(kg * 8 + (lane & 7)), k_swz = lane & 7;      // boxes hold at least eight keys
   const uint32_t kc0 = ((lane >> 3) ^ k_swz) << 4, kc1 = ((4 + (lane >> 3)) ^ k_swz) << 4;
-  const uint32_t v_off[2] = {static_cast<uint32_t>(key_offset(lane & 15)), static_cast<uint32_t>(key_offset(16 + (lane & 15)))};
+  // value fragments: this warp's first 16 columns, their chunks swizzled by the key; a round of the warps is WARPS / 4 slabs
+  const uint32_t v_col = (warp >> 2) * slab_bytes + ((((warp & 3) * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
+  const uint32_t v_off[2] = {key_offset(lane & 15) + v_col, key_offset(16 + (lane & 15)) + v_col};
+  const int rounds = (a.rank + WARPS * 16 - 1) / (WARPS * 16);
   const uint32_t q_addr = smem_addr(sQ + (mg * S::kMTiles * 16 + (lane & 15)) * LD + (lane >> 4) * 8);
   __syncthreads();
   bool ok = true;
@@ -140,23 +144,30 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
     for (int i = 0; i < S::kMTiles; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) sc[i][e] = sd[i][e] = 0.0f;
-#pragma unroll 2
-    for (int b = 0; b < slabs; ++b) {
-      uint32_t ka[4], kb[4];                        // 32 columns each
-      ldmatrix_x4(ka, base + k_off + b * slab_bytes + kc0);
-      ldmatrix_x4(kb, base + k_off + b * slab_bytes + kc1);
+    // the fragments of the next slab are on their way while this one's products run
+    uint32_t kf[2][2][4], qf[2][S::kMTiles][4][4];
+    auto fetch = [&](int b, int u) {
+      ldmatrix_x4(kf[u][0], base + k_off + b * slab_bytes + kc0);
+      ldmatrix_x4(kf[u][1], base + k_off + b * slab_bytes + kc1);
 #pragma unroll
-      for (int i = 0; i < S::kMTiles; ++i) {
-        uint32_t q0[4], q1[4], q2[4], q3[4];
-        const uint32_t qa = q_addr + (i * 16 * LD + b * 64) * 2;
-        ldmatrix_x4(q0, qa);
-        ldmatrix_x4(q1, qa + 32);
-        ldmatrix_x4(q2, qa + 64);
-        ldmatrix_x4(q3, qa + 96);
-        mma_bf16(sc[i], q0, ka[0], ka[1]);
-        mma_bf16(sd[i], q1, ka[2], ka[3]);
-        mma_bf16(sc[i], q2, kb[0], kb[1]);
-        mma_bf16(sd[i], q3, kb[2], kb[3]);
+      for (int i = 0; i < S::kMTiles; ++i)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) ldmatrix_x4(qf[u][i][c], q_addr + (i * 16 * LD + b * 64 + c * 16) * 2);
+    };
+    auto multiply = [&](int u) {
+#pragma unroll
+      for (int c = 0; c < 4; ++c)
+#pragma unroll
+        for (int i = 0; i < S::kMTiles; ++i)
+          mma_bf16((c & 1) ? sd[i] : sc[i], qf[u][i][c], kf[u][c >> 1][(c & 1) * 2], kf[u][c >> 1][(c & 1) * 2 + 1]);
+    };
+    fetch(0, 0);
+    for (int b = 0; b < slabs; b += 2) {
+      if (b + 1 < slabs) fetch(b + 1, 1);
+      multiply(0);
+      if (b + 1 < slabs) {
+        if (b + 2 < slabs) fetch(b + 2, 0);
+        multiply(1);
       }
     }
     const int kbase = k0 + kg * 8 + t * 2;
@@ -215,25 +226,31 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
       }
     }
     __syncthreads();
+    // columns past the latent (a last, partial round of tiles) are multiplied but not stored
+    auto weigh = [&](auto tiles, int n) {
+      constexpr int N = decltype(tiles)::value;
 #pragma unroll
-    for (int kk = 0; kk < kKeys / 16; ++kk) {
-      uint32_t pa[MT][4];
+      for (int kk = 0; kk < kKeys / 16; ++kk) {
+        uint32_t pa[MT][4], vb[N][4];
 #pragma unroll
-      for (int i = 0; i < MT; ++i)
-        ldmatrix_x4(pa[i], smem_addr(sP + (i * 16 + (lane & 15)) * kLdP + kk * 16 + (lane >> 4) * 8));
+        for (int i = 0; i < MT; ++i)
+          ldmatrix_x4(pa[i], smem_addr(sP + (i * 16 + (lane & 15)) * kLdP + kk * 16 + (lane >> 4) * 8));
 #pragma unroll
-      for (int c = 0; c < CT; ++c) {
-        const int col = (c * WARPS + warp) * 16;
-        if (col >= a.rank) break;
-        uint32_t vb[4];
-        ldmatrix_x4_trans(vb, base + v_off[kk] + (col >> 6) * slab_bytes + (((((col & 63) >> 3) + (lane >> 4)) ^ (lane & 7)) << 4));
+        for (int c = 0; c < N; ++c)
+          if (N == CT || c < n) ldmatrix_x4_trans(vb[c], base + v_off[kk] + c * (WARPS / 4) * slab_bytes);
 #pragma unroll
-        for (int i = 0; i < MT; ++i) {
-          mma_bf16(o[i][c][0], pa[i], vb[0], vb[1]);
-          mma_bf16(o[i][c][1], pa[i], vb[2], vb[3]);
-        }
+        for (int c = 0; c < N; ++c)
+          if (N == CT || c < n) {
+#pragma unroll
+            for (int i = 0; i < MT; ++i) {
+              mma_bf16(o[i][c][0], pa[i], vb[c][0], vb[c][1]);
+              mma_bf16(o[i][c][1], pa[i], vb[c][2], vb[c][3]);
+            }
+          }
       }
-    }
+    };
+    if (rounds == CT) weigh(std::integral_constant<int, CT>{}, CT);
+    else if constexpr (CT > 1) weigh(std::integral_constant<int, CT - 1>{}, rounds);
   }
   __syncthreads();
 #pragma unroll
