@@ -77,7 +77,7 @@ def time_engine(weights, prompts=(8, 1024), long_prompt=4096, batch=64, iters=10
     ids = [eng.add_sequence() for _ in range(batch)]
     for i in range(0, batch, 8):
         eng.forward([Chunk(s, toks(1024), 0) for s in ids[i: i + 8]])
-    one = [5] * batch
+    one = toks(batch)
     ms = _step_ms(lambda: eng.forward([Chunk(s, [t], 1, True) for s, t in zip(ids, one)]), 30)
     out["decode_tok_s"], out["decode_ms"] = batch / (ms * 1e-3), ms
     K.check_status()

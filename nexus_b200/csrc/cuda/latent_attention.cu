@@ -5,6 +5,7 @@
 // stage come as tiled copies of whole cache rows, split into slabs of 64 columns with the 128-byte swizzle, which the fragment
 // loads undo.  The warps split the keys of a stage for the scores and the latent columns for the weighted sum; row maxima and
 // probabilities cross warps through shared memory.  Scores and softmax are FP32; only the products take BF16 operands.
+#include "flash_common.cuh"
 #include "mixer_common.cuh"
 #include "nx_api_mixers.h"
 #include "paged_common.cuh"
@@ -17,7 +18,6 @@
 namespace {
 using namespace nx;
 
-constexpr float kLog2e = 1.4426950408889634f;
 constexpr int kKeys = 32;           // per stage
 constexpr int kKGroups = 4;         // warps along the keys of a stage, eight keys each
 constexpr int kLdP = kKeys + 8;
@@ -107,7 +107,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
   const int mg = warp % S::kMGroups, kg = warp / S::kMGroups;
   const float mul = a.scale * kLog2e;
   int vis[S::kMTiles][2];                           // position of this thread's score rows, -1: padding row
-  float sum[S::kMTiles][2];
+  float sum[S::kMTiles][2], ref[S::kMTiles][2];     // ref: what the row's scores are measured against (log2 units)
+  const bool full_tile = nt * rt == ROWS && nh == rt;
 #pragma unroll
   for (int i = 0; i < S::kMTiles; ++i)
 #pragma unroll
@@ -115,6 +116,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
       const int m = (mg * S::kMTiles + i) * 16 + e * 8 + g;
       vis[i][e] = m / rt < nt && m % rt < nh ? pos0 + m / rt : -1;
       sum[i][e] = 0.0f;
+      ref[i][e] = -INFINITY;
     }
   float o[MT][CT][2][4];
 #pragma unroll
@@ -171,49 +173,63 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
       }
     }
     const int kbase = k0 + kg * 8 + t * 2;
+    const bool inside = k0 + kKeys - 1 <= min(pos0, last) && (a.window <= 0 || k0 > hi - a.window) && full_tile;
+    float top[S::kMTiles][2];
+    bool grow = false;
 #pragma unroll
     for (int i = 0; i < S::kMTiles; ++i) {
       float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int j = kbase + (e & 1), p = vis[i][e >> 1];
-        const bool see = j <= min(p, last) && (a.window <= 0 || j > p - a.window);
-        sc[i][e] = see ? (sc[i][e] + sd[i][e]) * mul : -INFINITY;
+        sc[i][e] = (sc[i][e] + sd[i][e]) * mul;
+        if (!inside) {                                // some row of the block does not see the whole stage
+          const int j = kbase + (e & 1), p = vis[i][e >> 1];
+          if (!(j <= min(p, last) && (a.window <= 0 || j > p - a.window))) sc[i][e] = -INFINITY;
+        }
         mx[e >> 1] = fmaxf(mx[e >> 1], sc[i][e]);
       }
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
-        mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2));
-        if (t == 0) s_part[kg * ROWS + (mg * S::kMTiles + i) * 16 + e * 8 + g] = mx[e];
+        top[i][e] = mx[e];
+        grow = grow || mx[e] > ref[i][e] + kRescaleStep;
       }
     }
-    __syncthreads();                                // the previous stage has been consumed by every warp, too
+    // every warp weighs with one reference per row; it moves only when a row's maximum has grown by 2^8.  Past this barrier
+    // the previous stage has been consumed by every warp, too.
+    const bool move = __syncthreads_or(grow) != 0;
     if (it > 0 && it - 1 + stages < n_stages) load(it - 1 + stages);
-    if (threadIdx.x < ROWS) {
-      const int m = threadIdx.x;
-      const float old = s_max[m];
-      float nm = old;
+    if (move) {
 #pragma unroll
-      for (int w = 0; w < kKGroups; ++w) nm = fmaxf(nm, s_part[w * ROWS + m]);
-      s_max[m] = nm;
-      s_alpha[m] = nm == -INFINITY ? 1.0f : ex2_approx(old - nm);
-    }
-    __syncthreads();
+      for (int i = 0; i < S::kMTiles; ++i)
 #pragma unroll
-    for (int i = 0; i < S::kMTiles; ++i)
+        for (int e = 0; e < 2; ++e) {
+          float mx = fmaxf(top[i][e], __shfl_xor_sync(0xffffffffu, top[i][e], 1));
+          mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+          if (t == 0) s_part[kg * ROWS + (mg * S::kMTiles + i) * 16 + e * 8 + g] = mx;
+        }
+      __syncthreads();
+      if (threadIdx.x < ROWS) {
+        const int m = threadIdx.x;
+        const float old = s_max[m];
+        float nm = old;
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int m = (mg * S::kMTiles + i) * 16 + e * 8 + g;
-        const float nm = s_max[m], mb = nm == -INFINITY ? 0.0f : nm;
-        const float p0 = ex2_approx(sc[i][2 * e] - mb), p1 = ex2_approx(sc[i][2 * e + 1] - mb);   // -inf: 0
-        sum[i][e] = sum[i][e] * s_alpha[m] + p0 + p1;
-        *reinterpret_cast<uint32_t*>(sP + m * kLdP + kg * 8 + t * 2) = bf16_pair(p0, p1);
+        for (int w = 0; w < kKGroups; ++w) nm = fmaxf(nm, s_part[w * ROWS + m]);
+        const bool up = nm > old + kRescaleStep;
+        s_alpha[m] = up ? ex2_approx(old - nm) : 1.0f;
+        if (up) s_max[m] = nm;
       }
+      __syncthreads();
 #pragma unroll
-    for (int i = 0; i < MT; ++i) {
-      const float f0 = s_alpha[i * 16 + g], f1 = s_alpha[i * 16 + 8 + g];
-      if (__any_sync(0xffffffffu, f0 != 1.0f || f1 != 1.0f)) {
+      for (int i = 0; i < S::kMTiles; ++i)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int m = (mg * S::kMTiles + i) * 16 + e * 8 + g;
+          ref[i][e] = s_max[m];
+          sum[i][e] *= s_alpha[m];
+        }
+#pragma unroll
+      for (int i = 0; i < MT; ++i) {
+        const float f0 = s_alpha[i * 16 + g], f1 = s_alpha[i * 16 + 8 + g];
 #pragma unroll
         for (int c = 0; c < CT; ++c)
 #pragma unroll
@@ -225,6 +241,16 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
           }
       }
     }
+#pragma unroll
+    for (int i = 0; i < S::kMTiles; ++i)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int m = (mg * S::kMTiles + i) * 16 + e * 8 + g;
+        const float base_m = ref[i][e] == -INFINITY ? 0.0f : ref[i][e];
+        const float p0 = ex2_approx(sc[i][2 * e] - base_m), p1 = ex2_approx(sc[i][2 * e + 1] - base_m);   // -inf: 0
+        sum[i][e] += p0 + p1;
+        *reinterpret_cast<uint32_t*>(sP + m * kLdP + kg * 8 + t * 2) = bf16_pair(p0, p1);
+      }
     __syncthreads();
     // columns past the latent (a last, partial round of tiles) are multiplied but not stored
     auto weigh = [&](auto tiles, int n) {

@@ -11,6 +11,8 @@
 #include "mixer_common.cuh"
 #include "nx_api_moe.h"
 
+#include <algorithm>
+
 namespace {
 using namespace nx;
 
@@ -185,16 +187,19 @@ __global__ void __launch_bounds__(1024) moe_table_route_kernel(const __grid_cons
   extern __shared__ int s_cnt[];               // [experts] counts, then the next free slot
   __shared__ int s_warp[32], s_total;
   const NxTableRouteLayer& L = a.layer[blockIdx.x];
-  const int total = a.n * L.top, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   for (int e = tid; e < L.experts; e += blockDim.x) s_cnt[e] = 0;
   for (int i = tid; i < L.max_slots; i += blockDim.x) L.rows[i] = -1;
   __syncthreads();
 #pragma unroll 4
-  for (int i = tid; i < total; i += blockDim.x) {
-    const int t = a.tokens[i / L.top];
-    const int e = t >= 0 && t < a.vocab ? L.table[static_cast<int64_t>(t) * L.top + i % L.top] : 0;
-    L.slots[i] = e;                            // the expert for now, read again by this thread
-    atomicAdd(&s_cnt[e], 1);
+  for (int r = tid; r < a.n; r += blockDim.x) {
+    const int t = a.tokens[r];
+    const int32_t* row = L.table + static_cast<int64_t>(t >= 0 && t < a.vocab ? t : 0) * L.top;
+    for (int j = 0; j < L.top; ++j) {
+      const int e = row[j];
+      L.slots[r * L.top + j] = e;              // the expert for now, read again by this thread
+      atomicAdd(&s_cnt[e], 1);
+    }
   }
   __syncthreads();
   int base = 0;
@@ -223,21 +228,26 @@ __global__ void __launch_bounds__(1024) moe_table_route_kernel(const __grid_cons
   }
   for (int g = base / a.align + tid; g < L.max_slots / a.align; g += blockDim.x) L.groups[g] = -1;
 #pragma unroll 4
-  for (int i = tid; i < total; i += blockDim.x) {
-    const int s = atomicAdd(&s_cnt[L.slots[i]], 1);
-    L.slots[i] = s;
-    L.rows[s] = i / L.top;
-  }
+  for (int r = tid; r < a.n; r += blockDim.x)
+    for (int j = 0; j < L.top; ++j) {
+      const int s = atomicAdd(&s_cnt[L.slots[r * L.top + j]], 1);
+      L.slots[r * L.top + j] = s;
+      L.rows[s] = r;
+    }
 }
 
 // ------------------------------------------------------------------------------------------------
-// expert product, few rows: a warp owns 16 rows of one expert's weights and streams them once for up to 8 NT tokens.  A
-// thread's 16-byte load covers eight neighbours along K; the sum over K may take them in any order as long as both
-// operands agree, so each load is two k-steps of the tensor-core tile as it is.
+// product with one weight matrix per group (expert, head), few rows: the weights stream through registers once for up to
+// 8 NT rows.  A thread's 16-byte load covers eight neighbours along K; the sum over K may take them in any order as long as
+// both operands agree, so each load is two k-steps of the tensor-core tile as it is.  A block has four warps: 4 / KS tiles of
+// 16 weight rows, each cut into KS parts along K whose sums meet in shared memory.
 // ------------------------------------------------------------------------------------------------
-template <int NT>
-__device__ __forceinline__ void expert_rows(const NxExpertGemmArgs& a, const __nv_bfloat16* w, int n0, int first, int cnt) {
-  const int lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+template <int NT, int KS>
+__device__ __forceinline__ void group_rows(const NxExpertGemmArgs& a, int group, int tile, int first, int cnt, float* s_acc) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const int part = warp % KS, n0 = (tile * (4 / KS) + warp / KS) * 16;
+  const int k_part = ((a.k + KS - 1) / KS + 63) / 64 * 64, k_end = min(a.k, (part + 1) * k_part);
+  const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(a.w) + group * a.stride_w;
   const __nv_bfloat16 *w0 = w + static_cast<int64_t>(n0 + g) * a.ldw + t * 8, *w1 = w0 + 8 * a.ldw;
   const bool in0 = n0 + g < a.n, in1 = n0 + g + 8 < a.n;
   const __nv_bfloat16* x[NT];
@@ -245,31 +255,48 @@ __device__ __forceinline__ void expert_rows(const NxExpertGemmArgs& a, const __n
 #pragma unroll
   for (int i = 0; i < NT; ++i) {
     const int s = first + min(i * 8 + g, cnt - 1);           // rows past the last repeat it; they are not stored
-    x[i] = static_cast<const __nv_bfloat16*>(a.x) + static_cast<int64_t>(a.rows != nullptr ? a.rows[s] : s) * a.ldx + t * 8;
+    x[i] = static_cast<const __nv_bfloat16*>(a.x) + group * a.group_x +
+           static_cast<int64_t>(a.rows != nullptr ? a.rows[s] : s) * a.ldx + t * 8;
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[i][e] = 0.0f;
   }
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-#pragma unroll(NT == 1 ? 4 : 2)
-  for (int k0 = 0; k0 < a.k; k0 += 64) {
-    uint4 wa[2], wb[2];
+#pragma unroll(NT <= 2 ? 4 : 2)
+  for (int k0 = part * k_part; k0 < k_end; k0 += 64) {
+    uint4 wa[2], wb[2], v[NT][2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
-      const bool ink = k0 + h * 32 + t * 8 < a.k;
-      wa[h] = ink && in0 ? __ldg(reinterpret_cast<const uint4*>(w0 + k0 + h * 32)) : zero;
-      wb[h] = ink && in1 ? __ldg(reinterpret_cast<const uint4*>(w1 + k0 + h * 32)) : zero;
+      const bool ink = k0 + h * 32 + t * 8 < k_end;
+      wa[h] = ink && in0 ? __ldcs(reinterpret_cast<const uint4*>(w0 + k0 + h * 32)) : zero;
+      wb[h] = ink && in1 ? __ldcs(reinterpret_cast<const uint4*>(w1 + k0 + h * 32)) : zero;
+#pragma unroll
+      for (int i = 0; i < NT; ++i) v[i][h] = ink ? __ldg(reinterpret_cast<const uint4*>(x[i] + k0 + h * 32)) : zero;
     }
+#pragma unroll
+    for (int h = 0; h < 2; ++h)
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        const uint32_t f0[4] = {wa[h].x, wb[h].x, wa[h].y, wb[h].y}, f1[4] = {wa[h].z, wb[h].z, wa[h].w, wb[h].w};
+        mma_bf16(acc[i], f0, v[i][h].x, v[i][h].y);
+        mma_bf16(acc[i], f1, v[i][h].z, v[i][h].w);
+      }
+  }
+  if constexpr (KS > 1) {
+    __syncthreads();                                         // a previous round has read s_acc
 #pragma unroll
     for (int i = 0; i < NT; ++i)
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const uint4 v = k0 + h * 32 + t * 8 < a.k ? __ldg(reinterpret_cast<const uint4*>(x[i] + k0 + h * 32)) : zero;
-        const uint32_t f0[4] = {wa[h].x, wb[h].x, wa[h].y, wb[h].y}, f1[4] = {wa[h].z, wb[h].z, wa[h].w, wb[h].w};
-        mma_bf16(acc[i], f0, v.x, v.y);
-        mma_bf16(acc[i], f1, v.z, v.w);
-      }
+      for (int e = 0; e < 4; ++e) s_acc[(warp * NT * 4 + i * 4 + e) * 32 + lane] = acc[i][e];
+    __syncthreads();
+    if (part != 0) return;
+#pragma unroll
+    for (int p = 1; p < KS; ++p)
+#pragma unroll
+      for (int i = 0; i < NT; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[i][e] += s_acc[((warp + p) * NT * 4 + i * 4 + e) * 32 + lane];
   }
-  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out);
+  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + group * a.group_out;
 #pragma unroll
   for (int i = 0; i < NT; ++i)
 #pragma unroll
@@ -281,16 +308,16 @@ __device__ __forceinline__ void expert_rows(const NxExpertGemmArgs& a, const __n
     }
 }
 
+template <int KS>
 __global__ void __launch_bounds__(128) expert_skinny_kernel(const NxExpertGemmArgs a) {
-  const int e = blockIdx.y, n0 = (blockIdx.x * 4 + (threadIdx.x >> 5)) * 16;
-  int cnt = a.count[e];
-  if (cnt <= 0 || n0 >= a.n) return;
-  int first = a.start[e];
-  const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(a.w) + static_cast<int64_t>(e) * a.stride_w;
-  for (; cnt > 0; cnt -= 32, first += 32) {
-    if (cnt <= 8) expert_rows<1>(a, w, n0, first, cnt);
-    else if (cnt <= 16) expert_rows<2>(a, w, n0, first, cnt);
-    else expert_rows<4>(a, w, n0, first, min(cnt, 32));
+  __shared__ float s_acc[KS > 1 ? 4 * 4 * 4 * 32 : 1];
+  const int group = blockIdx.y, step = 32 * gridDim.z;
+  const int all = a.count != nullptr ? a.count[group] : a.m, start = a.start != nullptr ? a.start[group] : 0;
+  for (int c0 = blockIdx.z * 32; c0 < all; c0 += step) {     // the same for the whole block
+    const int cnt = min(32, all - c0);
+    if (cnt <= 8) group_rows<1, KS>(a, group, blockIdx.x, start + c0, cnt, s_acc);
+    else if (cnt <= 16) group_rows<2, KS>(a, group, blockIdx.x, start + c0, cnt, s_acc);
+    else group_rows<4, KS>(a, group, blockIdx.x, start + c0, cnt, s_acc);
   }
 }
 
@@ -335,7 +362,7 @@ __global__ void __launch_bounds__(256) expert_f32_kernel(const NxExpertGemmArgs 
 }
 
 int check_expert(const NxExpertGemmArgs* a) {
-  if (a == nullptr || a->x == nullptr || a->w == nullptr || a->out == nullptr || a->start == nullptr || a->count == nullptr) return -1;
+  if (a == nullptr || a->x == nullptr || a->w == nullptr || a->out == nullptr || (a->start == nullptr) != (a->count == nullptr)) return -1;
   if (a->experts <= 0 || a->n <= 0 || a->k <= 0 || (a->act != NX_ACT_NONE && a->act != NX_ACT_RELU2)) return -1;
   return 0;
 }
@@ -358,14 +385,22 @@ extern "C" int nx_moe_table_route(const NxTableRouteArgs* a, nx_stream_t stream)
 }
 
 extern "C" int nx_expert_skinny(const NxExpertGemmArgs* a, nx_stream_t stream) {
-  if (check_expert(a) || (a->k & 7) || (a->ldx & 7) || (a->ldw & 7) || (a->stride_w & 7) || a->experts > 65535) return -1;
+  if (check_expert(a) || (a->k & 7) || (a->ldx & 7) || (a->ldw & 7) || (a->stride_w & 7) || (a->group_x & 7) || a->experts > 65535)
+    return -1;
   if ((reinterpret_cast<uintptr_t>(a->x) & 15) || (reinterpret_cast<uintptr_t>(a->w) & 15)) return -1;
-  expert_skinny_kernel<<<dim3((a->n + 63) / 64, a->experts), 128, 0, static_cast<cudaStream_t>(stream)>>>(*a);
+  if (a->m <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  // a token uses an expert at most once, so no group has more than m rows
+  const int rounds = std::min((a->m + 31) / 32, 8), ks = a->k >= 1024 ? 4 : a->k >= 256 ? 2 : 1, per = 64 / ks;
+  const dim3 grid((a->n + per - 1) / per, a->experts, rounds);
+  if (ks == 4) expert_skinny_kernel<4><<<grid, 128, 0, st>>>(*a);
+  else if (ks == 2) expert_skinny_kernel<2><<<grid, 128, 0, st>>>(*a);
+  else expert_skinny_kernel<1><<<grid, 128, 0, st>>>(*a);
   return launch_status();
 }
 
 extern "C" int nx_expert_f32(const NxExpertGemmArgs* a, nx_stream_t stream) {
-  if (check_expert(a) || a->groups == nullptr || a->align != 32 || a->tiles < 0 || a->tiles > 65535) return -1;
+  if (check_expert(a) || a->start == nullptr || a->groups == nullptr || a->align != 32 || a->tiles < 0 || a->tiles > 65535) return -1;
   if (a->tiles == 0) return 0;
   expert_f32_kernel<<<dim3((a->n + 63) / 64, a->tiles), 256, 0, static_cast<cudaStream_t>(stream)>>>(*a);
   return launch_status();

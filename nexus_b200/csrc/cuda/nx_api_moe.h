@@ -51,6 +51,7 @@ typedef struct NxTableRouteArgs {
 int nx_moe_table_route(const NxTableRouteArgs* args, nx_stream_t stream);
 
 // out[slot] = act(W[e] x[row of slot]) for every slot of every expert; `rows` null: row = slot.  act: NX_ACT_NONE or RELU2.
+// start and count null: every group has slots 0..m (a matrix per head).
 typedef struct NxExpertGemmArgs {
   const void* x;           // [., ldx]
   const int32_t* rows;
@@ -61,8 +62,10 @@ typedef struct NxExpertGemmArgs {
   const int32_t* groups;   // FP32 form: expert per tile of `align` slots
   int64_t ldx, ldw, stride_w, ldo;
   int32_t experts, n, k, act, tiles, align;
+  int64_t group_x, group_out;  // few rows: what a group adds to the addresses of x and out (elements)
+  int32_t m;                   // few rows: most slots of a group
 } NxExpertGemmArgs;
-// few rows per expert, BF16: the weights stream through registers once per 32 rows; k, ldx, ldw multiples of 8
+// few rows per expert, BF16: the weights stream through registers once per 32 rows; k, ldx, ldw, group_x multiples of 8
 int nx_expert_skinny(const NxExpertGemmArgs* args, nx_stream_t stream);
 // FP32, align 32
 int nx_expert_f32(const NxExpertGemmArgs* args, nx_stream_t stream);

@@ -60,6 +60,9 @@ def load(engine, m: LatentSpec, get) -> dict:
     out["ukv"], _ = engine._pack([ukv])
     w = out["ukv"].w
     out["uk"], out["uv"] = w[: H * s.dim].view(H, s.dim, s.rank), w[H * s.dim:].view(H, s.vdim, s.rank)
+    if engine.fast:                   # the few-rows form wants the summed index last
+        out["uk_t"] = out["uk"].transpose(1, 2).contiguous()
+        engine.weight_nbytes += out["uk_t"].numel() * out["uk_t"].element_size()
     wo = torch.zeros((engine.d, H, s.vdim))
     wo[:, :, : m.vdim] = get("o").float().view(engine.d, H, m.vdim)
     out["out"], _ = engine._pack([wo.view(engine.d, H * s.vdim)])
@@ -68,13 +71,31 @@ def load(engine, m: LatentSpec, get) -> dict:
     return out
 
 
-def _per_head(engine, a, b, out, b_mn: bool) -> None:
-    """out[h] = a[h] b[h]^T (``b_mn``: a[h] b[h]) for strided batches of matrices."""
-    if engine.fast:
+FEW_ROWS = 256       # up to this many rows the per-head products stream their weights, above they are batched GEMMs
+
+
+def _to_latent(engine, lw: dict, q, out) -> None:
+    """out[r, h] = q[r, h] W_uk[h] for [rows, heads, .] views."""
+    if engine.fast and q.shape[0] <= FEW_ROWS:
+        from ..ops import _experts as X
+        X.head_product(q, lw["uk_t"], out)
+    elif engine.fast:
         from ..ops import _cuda as K
-        K.gemm(a, b, b_mn=b_mn, out=out)
+        K.gemm(q.permute(1, 0, 2), lw["uk"], b_mn=True, out=out.permute(1, 0, 2))
     else:
-        out.copy_(a @ (b if b_mn else b.transpose(1, 2)))
+        out.copy_((q.permute(1, 0, 2) @ lw["uk"]).permute(1, 0, 2))
+
+
+def _from_latent(engine, lw: dict, o, out) -> None:
+    """out[r, h] = W_uv[h] o[r, h]."""
+    if engine.fast and o.shape[0] <= FEW_ROWS:
+        from ..ops import _experts as X
+        X.head_product(o, lw["uv"], out)
+    elif engine.fast:
+        from ..ops import _cuda as K
+        K.gemm(o.permute(1, 0, 2), lw["uv"], out=out.permute(1, 0, 2))
+    else:
+        out.copy_((o.permute(1, 0, 2) @ lw["uv"].transpose(1, 2)).permute(1, 0, 2))
 
 
 def absorbed(engine, i: int, m: LatentSpec, lw: dict, q, gate, pos, out, groups) -> None:
@@ -82,7 +103,7 @@ def absorbed(engine, i: int, m: LatentSpec, lw: dict, q, gate, pos, out, groups)
     from ..ops import _mixers as M
     s, H, n = lw["shape"], m.heads, q.shape[0]
     ql = torch.empty((n, H, s.row), dtype=q.dtype, device=q.device)
-    _per_head(engine, q.view(n, H, s.head)[:, :, : s.dim].permute(1, 0, 2), lw["uk"], ql[:, :, : s.rank].permute(1, 0, 2), True)
+    _to_latent(engine, lw, q.view(n, H, s.head)[:, :, : s.dim], ql[:, :, : s.rank])
     ql = ql.view(n, H * s.row)
     M.rope_heads(q, s.head, s.dim, ql, s.row, s.rank, H, m.rope_dims, s.row - s.rank, pos, *lw["rope"])
     ol = torch.empty((n, H * s.rank), dtype=q.dtype, device=q.device)
@@ -94,18 +115,18 @@ def absorbed(engine, i: int, m: LatentSpec, lw: dict, q, gate, pos, out, groups)
             else:
                 M.paged_window_attention(ql, engine.k_cache[i], None, engine.block_table, ol, seg, heads=H,
                                          block_size=engine.cfg.block_size, window=m.window, scale=m.scale, gate=gate, vdim=s.rank)
-    _per_head(engine, ol.view(n, H, s.rank).permute(1, 0, 2), lw["uv"], out.view(n, H, s.vdim).permute(1, 0, 2), False)
+    _from_latent(engine, lw, ol.view(n, H, s.rank), out.view(n, H, s.vdim))
 
 
 def splits(engine, m: LatentSpec, seg) -> int:
     """Spans of the keys: enough blocks for every SM, at least 128 keys each."""
-    if seg.max_len > 1:
-        return 1
-    if engine.cfg.decode_splits > 0:
+    if engine.cfg.decode_splits > 0 and seg.max_len == 1:
         return engine.cfg.decode_splits
     keys = min(m.window, engine.ctx) if m.window > 0 else engine.ctx
-    blocks = seg.count * -(-m.heads // 64)
-    return max(1, min(-(-148 // blocks), -(-keys // 128), 32))
+    pairs = seg.total * m.heads              # (token, head) rows; a block takes up to 64, of one-token segments one token's
+    blocks = seg.count * -(-m.heads // 64) if seg.max_len == 1 else max(seg.count, pairs // 64)
+    sms = 296 if seg.max_len == 1 and m.heads <= 16 else 148
+    return max(1, min(sms // blocks, -(-keys // 128), 16))
 
 
 def expandable(m: LatentSpec) -> bool:

@@ -28,7 +28,7 @@ class ExpertGemmArgs(C.Structure):
     _fields_ = [("x", C.c_void_p), ("rows", C.c_void_p), ("w", C.c_void_p), ("out", C.c_void_p), ("start", C.c_void_p),
                 ("count", C.c_void_p), ("groups", C.c_void_p), ("ldx", C.c_int64), ("ldw", C.c_int64), ("stride_w", C.c_int64),
                 ("ldo", C.c_int64), ("experts", C.c_int32), ("n", C.c_int32), ("k", C.c_int32), ("act", C.c_int32),
-                ("tiles", C.c_int32), ("align", C.c_int32)]
+                ("tiles", C.c_int32), ("align", C.c_int32), ("group_x", C.c_int64), ("group_out", C.c_int64), ("m", C.c_int32)]
 
 
 @dataclass
@@ -88,7 +88,15 @@ def expert_product(x: torch.Tensor, w: torch.Tensor, route: Route, *, gather: bo
         return K.grouped_gemm(x, w, route.groups, route.align, act=act, out=out)
     a = ExpertGemmArgs(x.data_ptr(), route.rows.data_ptr() if gather else None, w.data_ptr(), out.data_ptr(), route.start.data_ptr(),
                        route.count.data_ptr(), route.groups.data_ptr(), x.stride(0), w.stride(1), w.stride(0), out.stride(0), E, n, k,
-                       K.ACT[act], route.groups.shape[0], route.align)
+                       K.ACT[act], route.groups.shape[0], route.align, 0, 0, route.slots.shape[0])
     name = "nx_expert_skinny" if x.dtype == torch.bfloat16 else "nx_expert_f32"
     K._check(getattr(K.lib(), name)(C.byref(a), K._stream()), name)
     return out
+
+
+def head_product(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+    """out[:, h] = x[:, h] w[h]^T for few rows: x [rows, heads, >= k] and out [rows, heads, >= n] views, w BF16 [heads, n, k]."""
+    H, n, k = w.shape
+    a = ExpertGemmArgs(x.data_ptr(), None, w.data_ptr(), out.data_ptr(), None, None, None, x.stride(0), w.stride(1), w.stride(0),
+                       out.stride(0), H, n, k, K.ACT[None], 0, 1, x.stride(1), out.stride(1), x.shape[0])
+    K._check(K.lib().nx_expert_skinny(C.byref(a), K._stream()), "nx_expert_skinny")
