@@ -134,12 +134,36 @@ def expandable(m: LatentSpec) -> bool:
     return s.dim <= 128 and s.rot <= 64 and s.vdim <= 128 and m.scale > 0
 
 
+QUERY_BLOCK = 256    # query rows of one work item of the expanded form
+
+
+def long_segments(segs, window: int):
+    """The work of the expanded form for segments (first row, rows, first position, sequence): (blocks, runs, rows of kv).
+
+    A segment that does not start at position 0 needs latents of earlier steps: if there is one, all keys are gathered from
+    the cache (``runs``: first row, rows, first position, sequence), else they are the rows of the step and ``runs`` is empty.
+    ``blocks``: first query row, rows, position of the first row, kv row of position 0; the most keys first."""
+    back, blocks, runs, d = window - 1 if window > 0 else 1 << 30, [], [], 0
+    gather = any(pos > 0 for _, _, pos, _ in segs)
+    for row0, count, pos, seq in segs:
+        base, kv0 = 0, row0
+        if gather:
+            base = max(0, pos - back)
+            kv0 = d - base
+            runs.append((d, pos + count - base, base, seq))
+            d += pos + count - base
+        for b in range(0, count, QUERY_BLOCK):
+            rows = min(QUERY_BLOCK, count - b)
+            blocks.append((min(pos + b, back) + rows, row0 + b, rows, pos + b, kv0))
+    blocks.sort(key=lambda x: -x[0])
+    return [b[1:] for b in blocks], runs, d
+
+
 class StepPlan:
     """How the segments of a step that has long ones are split between the two forms; built on the host once per step.
 
-    ``rows``: the rows of the one-token and short segments, ``groups`` these segments over the compacted rows.  Per window:
-    ``blocks``, query blocks of the long segments in the order of their cost, and ``runs``, what to gather from the cache
-    when a long segment does not start at position 0 (else the keys are the rows of the step)."""
+    ``rows``: the rows of the one-token and short segments, ``groups`` these segments over the compacted rows; per window the
+    blocks and runs of the long ones (`long_segments`)."""
 
     def __init__(self, engine, windows):
         from ..ops import _mixers as M
@@ -159,30 +183,19 @@ class StepPlan:
             first += count
         put("rows", [r for row0, count, _, _ in segs[:n] for r in range(row0, row0 + count)])
         put("table", [v for t in table for v in t])
-        self.gathered = any(pos > 0 for _, _, pos, _ in segs[n:])
-        self.kv_rows: Dict[int, int] = {}
+        self.kv_rows, self.longest = {}, {}
         for w in windows:
-            back, blocks, runs, d = w - 1 if w > 0 else 1 << 30, [], [], 0
-            for row0, count, pos, seq in segs[n:]:
-                base = max(0, pos - back) if self.gathered else 0
-                kv0 = d - base if self.gathered else row0
-                runs += [d, pos + count - base, base, seq]
-                d += pos + count - base
-                for b in range(0, count, 256):
-                    rows = min(256, count - b)
-                    blocks.append((min(pos + b, back) + rows, row0 + b, rows, pos + b, kv0))
-            blocks.sort(key=lambda x: -x[0])
-            put(("blocks", w), [v for b in blocks for v in b[1:]])
-            put(("runs", w), runs)
-            self.kv_rows[w] = d
+            blocks, runs, self.kv_rows[w] = long_segments(segs[n:], w)
+            self.longest[w] = max((r[1] for r in runs), default=0)
+            put(("blocks", w), [v for b in blocks for v in b])
+            put(("runs", w), [v for r in runs for v in r])
+        self.gathered = any(self.kv_rows.values())
         dev = torch.tensor(data, dtype=torch.int32).pin_memory().to(engine.dev, non_blocking=True)
 
         def get(name):
             return dev[at[name][0]: at[name][0] + at[name][1]]
         self.blocks = {w: get(("blocks", w)).view(-1, 4) for w in windows}
         self.runs = {w: get(("runs", w)).view(-1, 4) for w in windows}
-        self.longest = {w: max(pos + count - max(0, pos - (w - 1 if w > 0 else 1 << 30)) for _, count, pos, _ in segs[n:])
-                        for w in windows}
         self.rows = get("rows").long() if n else None
         if n:
             t = get("table").view(4, n)
