@@ -205,14 +205,18 @@ def run_reference(args) -> int:
     return 0
 
 
-def run_gugedra(args) -> int:
-    """Prefill and decode throughput of Gugedra models (random weights, BF16) at a few sizes, and of GPT-2 models of the same
-    width and depth through the same engine.  One JSON line; `value` is the hybrid model's prefill rate at the middle size."""
+def run_serving(args) -> int:
+    """Prefill and decode throughput of Gugedra or Makuzen models (random weights, BF16) at a few sizes, and of the other
+    models of the same width and depth through the same engine.  One JSON line; `value` is the design's prefill rate at the
+    middle size."""
     if args.impl != "ours" or args.gpus != 1:
-        print(json.dumps({"impl": args.impl, "unavailable": "the gugedra workload is this framework's own, on one GPU"}))
+        print(json.dumps({"impl": args.impl, "unavailable": f"the {args.workload} workload is this framework's own, on one GPU"}))
         return 0
     sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
-    from nexus_b200.bench.hybrid import model_lines
+    if args.workload == "gugedra":
+        from nexus_b200.bench.hybrid import model_lines
+    else:
+        from nexus_b200.bench.latent import model_lines
     from nexus_b200.ops import _cuda as K
     sizes = [int(s) for s in args.sizes.split(",")]
     sampler = ClockSampler(0)
@@ -221,11 +225,12 @@ def run_gugedra(args) -> int:
     clocks = sampler.stop()
     mid = rows[len(rows) // 2]
     print(json.dumps({
-        "metric": "serving tokens/s, prefill of 8 x 1024 tokens, Gugedra", "value": mid["gugedra"]["prefill_tok_s"], "unit": "tokens/s",
+        "metric": f"serving tokens/s, prefill of 8 x 1024 tokens, {args.workload.capitalize()}",
+        "value": mid[args.workload]["prefill_tok_s"], "unit": "tokens/s",
         "n_gpus": 1, "steps": max(3, args.steps), "warmup": 3, "higher_is_better": True, "dtype": "bf16", "impl": "ours",
         "data": "random tokens, random-init weights",
-        "config": {"model": f"gugedra-{mid['width']}", "prefill": "8 x 1024 and 1 x 4096 tokens", "decode": "64 sequences, 1024 behind",
-                   "l2": "weights exceed the 126 MB L2; no explicit flush"},
+        "config": {"model": f"{args.workload}-{mid['width']}", "prefill": "8 x 1024 and 1 x 4096 tokens",
+                   "decode": "64 sequences, 1024 behind", "l2": "weights exceed the 126 MB L2; no explicit flush"},
         "sizes": rows, "clocks": {"sm_mhz": clocks["sm_mhz"], "sm_max_mhz": clocks["sm_max_mhz"], "reasons": clocks["reasons"]},
         "gpu_launches": K.launch_count}))
     return 0
@@ -243,12 +248,12 @@ def main() -> int:
     ap.add_argument("--graph", type=int, default=-1,
                     help="trainer API replays the whole step as one CUDA graph (default: on for 1 GPU, off otherwise)")
     ap.add_argument("--skip-e2e", action="store_true")
-    ap.add_argument("--workload", default="train", choices=["train", "gugedra"],
-                    help="gugedra: serving speed of the hybrid decoder beside a GPT-2 of equal width and depth, one GPU")
-    ap.add_argument("--sizes", default="1024,2048,4096", help="widths of the gugedra workload")
+    ap.add_argument("--workload", default="train", choices=["train", "gugedra", "makuzen"],
+                    help="gugedra, makuzen: serving speed of that design beside the other models of equal width and depth, one GPU")
+    ap.add_argument("--sizes", default="1024,2048,4096", help="widths of the serving workloads")
     args = ap.parse_args()
-    if args.workload == "gugedra":
-        return run_gugedra(args)
+    if args.workload != "train":
+        return run_serving(args)
     if args.impl == "reference":
         return run_reference(args)
     if args.graph < 0:
