@@ -1,8 +1,8 @@
 // Attention over a paged latent cache (see nx_api_mixers.h): all heads share one cache row per token, whose leading columns
 // are the values, so a row is read from memory once for every head and for both products.
 //
-// A block owns 16 MT (token, head) rows of one segment and one span of its keys.  Keys arrive in stages of 32; the pages of a
-// stage come as tiled copies of whole cache rows, split into slabs of 64 columns with the 128-byte swizzle, which the fragment
+// A block owns 16 MT (token, head) rows of one segment and one span of its keys.  Keys arrive in stages of 32 or 64; the pages of
+// a stage come as tiled copies of whole cache rows, split into slabs of 64 columns with the 128-byte swizzle, which the fragment
 // loads undo.  The warps split the keys of a stage for the scores and the latent columns for the weighted sum; row maxima and
 // probabilities cross warps through shared memory.  Scores and softmax are FP32; only the products take BF16 operands.
 #include "flash_common.cuh"
@@ -18,19 +18,20 @@
 namespace {
 using namespace nx;
 
-constexpr int kKeys = 32;           // per stage
-constexpr int kKGroups = 4;         // warps along the keys of a stage, eight keys each
-constexpr int kLdP = kKeys + 8;
+constexpr int kKGroups = 4;         // warps along the keys of a stage
 constexpr int kSmemMax = 226 * 1024;
 
 template <int MT>
 struct Shape {
   static constexpr int kRows = 16 * MT;
+  static constexpr int kKeys = MT == 2 ? 64 : 32;       // per stage: what shared memory holds twice beside the queries
+  static constexpr int kNTiles = kKeys / kKGroups / 8;  // 8-key tiles of a warp
+  static constexpr int kLdP = kKeys + 8;
   static constexpr int kMGroups = MT == 1 ? 1 : 2;      // warps along the rows
   static constexpr int kWarps = kKGroups * kMGroups;
   static constexpr int kMTiles = MT / kMGroups;         // 16-row tiles of a warp
   // behind the stages and Q: P, maxima per key group, running maximum, rescale factor, row sums, barriers
-  static constexpr int kTail = kRows * kLdP * 2 + kKGroups * kRows * 4 + 3 * kRows * 4 + 64;
+  static constexpr int kTail = kRows * kLdP * 2 + kKGroups * kRows * 4 + 3 * kRows * 4 + 128;
 };
 
 // CT: 16-column tiles of the latent per warp.  A box holds `1 << box_shift` keys of one page.
@@ -38,7 +39,7 @@ template <int MT, int CT>
 __global__ void __launch_bounds__(Shape<MT>::kWarps * 32, MT == 1 ? 2 : 1)
 latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArgs a, int rt, int tq, int stages, int box_shift) {
   using S = Shape<MT>;
-  constexpr int ROWS = S::kRows, WARPS = S::kWarps, THREADS = WARPS * 32;
+  constexpr int ROWS = S::kRows, WARPS = S::kWarps, THREADS = WARPS * 32, kKeys = S::kKeys, kLdP = S::kLdP, NTILES = S::kNTiles;
   extern __shared__ __align__(1024) uint8_t smem[];
   const int LD = a.row + 8, slabs = a.row / 64, stage_bytes = kKeys * a.row * 2;
   uint8_t* sKV = smem;                                                // [stages][boxes][slabs][keys of a box][128 B]
@@ -49,6 +50,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
   float* s_alpha = s_max + ROWS;
   float* s_sum = s_alpha + ROWS;
   uint64_t* full = reinterpret_cast<uint64_t*>(s_sum + ROWS);         // [stages]
+  uint64_t* empty = full + stages;                                    // [stages], one arrival per warp
   __shared__ int s_tile[3];
   __shared__ volatile int s_abort;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
@@ -64,7 +66,10 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
       s_tile[1] = seg;
       s_tile[2] = off;
       s_abort = 0;
-      for (int i = 0; i < stages; ++i) mbar_init(&full[i], 1);
+      for (int i = 0; i < stages; ++i) {
+        mbar_init(&full[i], 1);
+        mbar_init(&empty[i], WARPS);
+      }
       fence_mbar_init();
     }
   }
@@ -128,29 +133,43 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
   // byte offset of a key row inside a stage (slab 0), and the swizzle of its 16-byte chunks
   auto key_offset = [&](int key) -> uint32_t { return (key >> box_shift) * (a.row * 2 << box_shift) + (key & (box - 1)) * 128; };
   const int slab_bytes = 128 << box_shift;
-  const uint32_t k_off = key_offset(kg * 8 + (lane & 7)), k_swz = lane & 7;      // boxes hold at least eight keys
+  const uint32_t k_swz = lane & 7;                  // boxes hold at least eight keys
+  uint32_t k_off[NTILES];
+#pragma unroll
+  for (int n = 0; n < NTILES; ++n) k_off[n] = key_offset((kg * NTILES + n) * 8 + (lane & 7));
   const uint32_t kc0 = ((lane >> 3) ^ k_swz) << 4, kc1 = ((4 + (lane >> 3)) ^ k_swz) << 4;
   // value fragments: this warp's first 16 columns, their chunks swizzled by the key; a round of the warps is WARPS / 4 slabs
   const uint32_t v_col = (warp >> 2) * slab_bytes + ((((warp & 3) * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
-  const uint32_t v_off[2] = {key_offset(lane & 15) + v_col, key_offset(16 + (lane & 15)) + v_col};
+  uint32_t v_off[kKeys / 16];
+#pragma unroll
+  for (int kk = 0; kk < kKeys / 16; ++kk) v_off[kk] = key_offset(kk * 16 + (lane & 15)) + v_col;
   const int rounds = (a.rank + WARPS * 16 - 1) / (WARPS * 16);
   const uint32_t q_addr = smem_addr(sQ + (mg * S::kMTiles * 16 + (lane & 15)) * LD + (lane >> 4) * 8);
   __syncthreads();
   bool ok = true;
   for (int it = 0; it < n_stages; ++it) {
     const int s = it % stages, k0 = first + it * kKeys;
+    if (threadIdx.x == 0 && it > 0 && it - 1 + stages < n_stages) {     // the stage of the previous round, once all have used it
+      ok = ok && mbar_wait_bounded(&empty[(it - 1) % stages], ((it - 1) / stages) & 1, &s_abort);
+      if (ok) load(it - 1 + stages);
+    }
     ok = ok && mbar_wait_bounded(&full[s], (it / stages) & 1, &s_abort);
     const uint32_t base = smem_u32(sKV) + s * stage_bytes;
-    float sc[S::kMTiles][4], sd[S::kMTiles][4];     // two chains over the columns
+    float sc[S::kMTiles][NTILES][4], sd[S::kMTiles][NTILES][4];     // two chains over the columns
 #pragma unroll
     for (int i = 0; i < S::kMTiles; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) sc[i][e] = sd[i][e] = 0.0f;
+      for (int n = 0; n < NTILES; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sc[i][n][e] = sd[i][n][e] = 0.0f;
     // the fragments of the next slab are on their way while this one's products run
-    uint32_t kf[2][2][4], qf[2][S::kMTiles][4][4];
+    uint32_t kf[2][NTILES][2][4], qf[2][S::kMTiles][4][4];
     auto fetch = [&](int b, int u) {
-      ldmatrix_x4(kf[u][0], base + k_off + b * slab_bytes + kc0);
-      ldmatrix_x4(kf[u][1], base + k_off + b * slab_bytes + kc1);
+#pragma unroll
+      for (int n = 0; n < NTILES; ++n) {
+        ldmatrix_x4(kf[u][n][0], base + k_off[n] + b * slab_bytes + kc0);
+        ldmatrix_x4(kf[u][n][1], base + k_off[n] + b * slab_bytes + kc1);
+      }
 #pragma unroll
       for (int i = 0; i < S::kMTiles; ++i)
 #pragma unroll
@@ -161,7 +180,9 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
       for (int c = 0; c < 4; ++c)
 #pragma unroll
         for (int i = 0; i < S::kMTiles; ++i)
-          mma_bf16((c & 1) ? sd[i] : sc[i], qf[u][i][c], kf[u][c >> 1][(c & 1) * 2], kf[u][c >> 1][(c & 1) * 2 + 1]);
+#pragma unroll
+          for (int n = 0; n < NTILES; ++n)
+            mma_bf16((c & 1) ? sd[i][n] : sc[i][n], qf[u][i][c], kf[u][n][c >> 1][(c & 1) * 2], kf[u][n][c >> 1][(c & 1) * 2 + 1]);
     };
     fetch(0, 0);
     for (int b = 0; b < slabs; b += 2) {
@@ -172,7 +193,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
         multiply(1);
       }
     }
-    const int kbase = k0 + kg * 8 + t * 2;
+    const int kbase = k0 + kg * NTILES * 8 + t * 2;
     const bool inside = k0 + kKeys - 1 <= min(pos0, last) && (a.window <= 0 || k0 > hi - a.window) && full_tile;
     float top[S::kMTiles][2];
     bool grow = false;
@@ -180,14 +201,16 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
     for (int i = 0; i < S::kMTiles; ++i) {
       float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        sc[i][e] = (sc[i][e] + sd[i][e]) * mul;
-        if (!inside) {                                // some row of the block does not see the whole stage
-          const int j = kbase + (e & 1), p = vis[i][e >> 1];
-          if (!(j <= min(p, last) && (a.window <= 0 || j > p - a.window))) sc[i][e] = -INFINITY;
+      for (int n = 0; n < NTILES; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          sc[i][n][e] = (sc[i][n][e] + sd[i][n][e]) * mul;
+          if (!inside) {                              // some row of the block does not see the whole stage
+            const int j = kbase + n * 8 + (e & 1), p = vis[i][e >> 1];
+            if (!(j <= min(p, last) && (a.window <= 0 || j > p - a.window))) sc[i][n][e] = -INFINITY;
+          }
+          mx[e >> 1] = fmaxf(mx[e >> 1], sc[i][n][e]);
         }
-        mx[e >> 1] = fmaxf(mx[e >> 1], sc[i][e]);
-      }
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         top[i][e] = mx[e];
@@ -195,9 +218,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
       }
     }
     // every warp weighs with one reference per row; it moves only when a row's maximum has grown by 2^8.  Past this barrier
-    // the previous stage has been consumed by every warp, too.
+    // every warp is done with the previous P, too.
     const bool move = __syncthreads_or(grow) != 0;
-    if (it > 0 && it - 1 + stages < n_stages) load(it - 1 + stages);
     if (move) {
 #pragma unroll
       for (int i = 0; i < S::kMTiles; ++i)
@@ -247,9 +269,12 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
       for (int e = 0; e < 2; ++e) {
         const int m = (mg * S::kMTiles + i) * 16 + e * 8 + g;
         const float base_m = ref[i][e] == -INFINITY ? 0.0f : ref[i][e];
-        const float p0 = ex2_approx(sc[i][2 * e] - base_m), p1 = ex2_approx(sc[i][2 * e + 1] - base_m);   // -inf: 0
-        sum[i][e] += p0 + p1;
-        *reinterpret_cast<uint32_t*>(sP + m * kLdP + kg * 8 + t * 2) = bf16_pair(p0, p1);
+#pragma unroll
+        for (int n = 0; n < NTILES; ++n) {
+          const float p0 = ex2_approx(sc[i][n][2 * e] - base_m), p1 = ex2_approx(sc[i][n][2 * e + 1] - base_m);   // -inf: 0
+          sum[i][e] += p0 + p1;
+          *reinterpret_cast<uint32_t*>(sP + m * kLdP + (kg * NTILES + n) * 8 + t * 2) = bf16_pair(p0, p1);
+        }
       }
     __syncthreads();
     // columns past the latent (a last, partial round of tiles) are multiplied but not stored
@@ -277,6 +302,8 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
     };
     if (rounds == CT) weigh(std::integral_constant<int, CT>{}, CT);
     else if constexpr (CT > 1) weigh(std::integral_constant<int, CT - 1>{}, rounds);
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty[s]);
   }
   __syncthreads();
 #pragma unroll
@@ -366,7 +393,7 @@ __global__ void latent_merge_kernel(const NxLatentAttnArgs a) {
 template <int MT, int CT>
 int launch(const CUtensorMap& tm, const NxLatentAttnArgs* a, int box_shift, cudaStream_t st) {
   using S = Shape<MT>;
-  const int stage = kKeys * a->row * 2, fixed = S::kRows * (a->row + 8) * 2 + S::kTail;
+  const int stage = S::kKeys * a->row * 2, fixed = S::kRows * (a->row + 8) * 2 + S::kTail;
   // two blocks per SM where two stages fit twice, else one block with a deeper ring
   const int half = (kSmemMax / 2 - 1024 - fixed) / stage;
   const int stages = std::min(4, half >= 2 ? half : (kSmemMax - 1024 - fixed) / stage);
@@ -419,7 +446,7 @@ extern "C" int nx_latent_attention(const NxLatentAttnArgs* a, nx_stream_t stream
   }
   const int rows = a->seg.max_len > 1 ? 64 : a->heads;      // (token, head) pairs of a block
   const int rc = rows <= 16 ? launch_rank<1>(tm, a, box_shift, st)
-                            : rows <= 32 ? launch_rank<2>(tm, a, box_shift, st) : launch_rank<4>(tm, a, box_shift, st);
+                 : rows <= 32 && a->row <= 640 ? launch_rank<2>(tm, a, box_shift, st) : launch_rank<4>(tm, a, box_shift, st);
   if (rc == 0 && a->splits > 1) {
     latent_merge_kernel<<<dim3(a->seg.max_len, a->heads, a->seg.count), std::min(128, (a->rank / 4 + 31) / 32 * 32), 0, st>>>(*a);
     return launch_status();

@@ -257,7 +257,8 @@ def _absorbed_ref(q, lat, segs, H, rank, window, scale, gate):
     return (out * gate.double()[:, :, None]).view(q.shape[0], -1)
 
 
-ABSORBED = [(6, 96, 32, 16), (16, 512, 64, 16), (5, 48, 16, 24), (20, 256, 48, 8), (70, 112, 16, 32), (1, 16, 16, 64)]
+ABSORBED = [(6, 96, 32, 16), (16, 512, 64, 16), (5, 48, 16, 24), (20, 256, 48, 8), (70, 112, 16, 32), (1, 16, 16, 64), (32, 512, 64, 16),
+            (24, 512, 200, 16)]
 
 
 @pytest.mark.parametrize("window", [0, 1, 33, 130])
