@@ -19,6 +19,8 @@ namespace {
 using namespace nx;
 
 constexpr int kKGroups = 4;         // warps along the keys of a stage
+constexpr int kBox = 8;             // keys of one copy: what every page size is a multiple of, one row group of the swizzle
+constexpr int kSlab = kBox * 128;   // bytes of 64 columns of a box
 constexpr int kSmemMax = 226 * 1024;
 
 template <int MT>
@@ -34,15 +36,15 @@ struct Shape {
   static constexpr int kTail = kRows * kLdP * 2 + kKGroups * kRows * 4 + 3 * kRows * 4 + 128;
 };
 
-// CT: 16-column tiles of the latent per warp.  A box holds `1 << box_shift` keys of one page.
+// CT: 16-column tiles of the latent per warp
 template <int MT, int CT>
 __global__ void __launch_bounds__(Shape<MT>::kWarps * 32, MT == 1 ? 2 : 1)
-latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArgs a, int rt, int tq, int stages, int box_shift) {
+latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArgs a, int rt, int tq, int stages) {
   using S = Shape<MT>;
   constexpr int ROWS = S::kRows, WARPS = S::kWarps, THREADS = WARPS * 32, kKeys = S::kKeys, kLdP = S::kLdP, NTILES = S::kNTiles;
   extern __shared__ __align__(1024) uint8_t smem[];
   const int LD = a.row + 8, slabs = a.row / 64, stage_bytes = kKeys * a.row * 2;
-  uint8_t* sKV = smem;                                                // [stages][boxes][slabs][keys of a box][128 B]
+  uint8_t* sKV = smem;                                                // [stages][boxes][slabs][kBox][128 B]
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem + stages * stage_bytes);   // [ROWS][LD]
   __nv_bfloat16* sP = sQ + ROWS * LD;                                 // [ROWS][kLdP]
   float* s_part = reinterpret_cast<float*>(sP + ROWS * kLdP);         // [key groups][ROWS] stage maxima, then row sums
@@ -78,8 +80,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
   const int sg = s_tile[1], t0 = s_tile[2] * tq, h0 = blockIdx.y * rt;
   const int nh = min(rt, a.heads - h0), nt = min(tq, a.seg.len[sg] - t0), pos0 = a.seg.pos[sg] + t0;
   const int64_t row0 = static_cast<int64_t>(a.seg.row0[sg]) + t0;
-  const int box = 1 << box_shift;
-  const int hi = pos0 + nt - 1, lo = (a.window > 0 ? max(0, pos0 - a.window + 1) : 0) & ~(box - 1);
+  const int hi = pos0 + nt - 1, lo = (a.window > 0 ? max(0, pos0 - a.window + 1) : 0) & ~(kBox - 1);
   const int per = ((hi - lo + kKeys) / kKeys + a.splits - 1) / a.splits * kKeys;
   const int first = lo + static_cast<int>(blockIdx.z) * per, last = min(hi, first + per - 1);
   const int n_stages = last >= first ? (last - first) / kKeys + 1 : 0;
@@ -90,11 +91,13 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
     if (threadIdx.x != 0) return;
     const int s = it % stages;
     mbar_arrive_expect_tx(&full[s], static_cast<uint32_t>(stage_bytes));
-    for (int b = 0; b < kKeys >> box_shift; ++b) {
-      const int j = min(first + it * kKeys + (b << box_shift), hi & ~(box - 1));
-      tma_load_3d(sKV + s * stage_bytes + b * (a.row * 2 << box_shift), &tm, &full[s], 0,
-                  static_cast<int>(page_slot(bt, a.block_size, shift, j)), 0);
-    }
+    int slot[kKeys / kBox];
+#pragma unroll
+    for (int b = 0; b < kKeys / kBox; ++b)
+      slot[b] = static_cast<int>(page_slot(bt, a.block_size, shift, min(first + it * kKeys + b * kBox, hi & ~(kBox - 1))));
+#pragma unroll
+    for (int b = 0; b < kKeys / kBox; ++b)
+      tma_load_3d(sKV + s * stage_bytes + b * slabs * kSlab, &tm, &full[s], 0, slot[b], 0);
   };
   for (int it = 0; it < min(stages, n_stages); ++it) load(it);
   {
@@ -130,16 +133,13 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
     for (int c = 0; c < CT; ++c)
 #pragma unroll
       for (int e = 0; e < 4; ++e) o[i][c][0][e] = o[i][c][1][e] = 0.0f;
-  // byte offset of a key row inside a stage (slab 0), and the swizzle of its 16-byte chunks
-  auto key_offset = [&](int key) -> uint32_t { return (key >> box_shift) * (a.row * 2 << box_shift) + (key & (box - 1)) * 128; };
-  const int slab_bytes = 128 << box_shift;
-  const uint32_t k_swz = lane & 7;                  // boxes hold at least eight keys
+  // byte offset of a key row inside a stage (slab 0); its 16-byte chunks are swizzled by the key
+  auto key_offset = [&](int key) -> uint32_t { return (key / kBox) * slabs * kSlab + (key % kBox) * 128; };
   uint32_t k_off[NTILES];
 #pragma unroll
-  for (int n = 0; n < NTILES; ++n) k_off[n] = key_offset((kg * NTILES + n) * 8 + (lane & 7));
-  const uint32_t kc0 = ((lane >> 3) ^ k_swz) << 4, kc1 = ((4 + (lane >> 3)) ^ k_swz) << 4;
-  // value fragments: this warp's first 16 columns, their chunks swizzled by the key; a round of the warps is WARPS / 4 slabs
-  const uint32_t v_col = (warp >> 2) * slab_bytes + ((((warp & 3) * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
+  for (int n = 0; n < NTILES; ++n) k_off[n] = key_offset((kg * NTILES + n) * 8 + (lane & 7)) + (((lane >> 3) ^ (lane & 7)) << 4);
+  // value fragments: this warp's first 16 columns; a round of the warps is WARPS / 4 slabs
+  const uint32_t v_col = (warp >> 2) * kSlab + ((((warp & 3) * 2 + (lane >> 4)) ^ (lane & 7)) << 4);
   uint32_t v_off[kKeys / 16];
 #pragma unroll
   for (int kk = 0; kk < kKeys / 16; ++kk) v_off[kk] = key_offset(kk * 16 + (lane & 15)) + v_col;
@@ -155,25 +155,29 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
     }
     ok = ok && mbar_wait_bounded(&full[s], (it / stages) & 1, &s_abort);
     const uint32_t base = smem_u32(sKV) + s * stage_bytes;
-    float sc[S::kMTiles][NTILES][4], sd[S::kMTiles][NTILES][4];     // two chains over the columns
+    // partial sums over the columns, so that few products wait for one another
+    constexpr int CHAINS = S::kMTiles * NTILES == 1 ? 4 : 2;
+    float part[CHAINS][S::kMTiles][NTILES][4];
 #pragma unroll
-    for (int i = 0; i < S::kMTiles; ++i)
+    for (int c = 0; c < CHAINS; ++c)
 #pragma unroll
-      for (int n = 0; n < NTILES; ++n)
+      for (int i = 0; i < S::kMTiles; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) sc[i][n][e] = sd[i][n][e] = 0.0f;
+        for (int n = 0; n < NTILES; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) part[c][i][n][e] = 0.0f;
     // the fragments of the next slab are on their way while this one's products run
     uint32_t kf[2][NTILES][2][4], qf[2][S::kMTiles][4][4];
-    auto fetch = [&](int b, int u) {
+    auto fetch = [&](uint32_t slab, uint32_t q, int u) {
 #pragma unroll
       for (int n = 0; n < NTILES; ++n) {
-        ldmatrix_x4(kf[u][n][0], base + k_off[n] + b * slab_bytes + kc0);
-        ldmatrix_x4(kf[u][n][1], base + k_off[n] + b * slab_bytes + kc1);
+        ldmatrix_x4(kf[u][n][0], slab + k_off[n]);
+        ldmatrix_x4(kf[u][n][1], (slab + k_off[n]) ^ 64);          // columns 32..63: the other half of the 128 bytes
       }
 #pragma unroll
       for (int i = 0; i < S::kMTiles; ++i)
 #pragma unroll
-        for (int c = 0; c < 4; ++c) ldmatrix_x4(qf[u][i][c], q_addr + (i * 16 * LD + b * 64 + c * 16) * 2);
+        for (int c = 0; c < 4; ++c) ldmatrix_x4(qf[u][i][c], q + i * 32 * LD + c * 32);
     };
     auto multiply = [&](int u) {
 #pragma unroll
@@ -182,17 +186,31 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
         for (int i = 0; i < S::kMTiles; ++i)
 #pragma unroll
           for (int n = 0; n < NTILES; ++n)
-            mma_bf16((c & 1) ? sd[i][n] : sc[i][n], qf[u][i][c], kf[u][n][c >> 1][(c & 1) * 2], kf[u][n][c >> 1][(c & 1) * 2 + 1]);
+            mma_bf16(part[c % CHAINS][i][n], qf[u][i][c], kf[u][n][c >> 1][(c & 1) * 2], kf[u][n][c >> 1][(c & 1) * 2 + 1]);
     };
-    fetch(0, 0);
-    for (int b = 0; b < slabs; b += 2) {
-      if (b + 1 < slabs) fetch(b + 1, 1);
+    uint32_t slab = base, qs = q_addr;
+    fetch(slab, qs, 0);
+    int b = 0;
+    for (; b + 2 < slabs; b += 2, slab += 2 * kSlab, qs += 256) {
+      fetch(slab + kSlab, qs + 128, 1);
       multiply(0);
-      if (b + 1 < slabs) {
-        if (b + 2 < slabs) fetch(b + 2, 0);
-        multiply(1);
-      }
+      fetch(slab + 2 * kSlab, qs + 256, 0);
+      multiply(1);
     }
+    if (b + 1 < slabs) fetch(slab + kSlab, qs + 128, 1);
+    multiply(0);
+    if (b + 1 < slabs) multiply(1);
+    float sc[S::kMTiles][NTILES][4];
+#pragma unroll
+    for (int i = 0; i < S::kMTiles; ++i)
+#pragma unroll
+      for (int n = 0; n < NTILES; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          sc[i][n][e] = part[0][i][n][e] + part[1][i][n][e];
+          if constexpr (CHAINS == 4) sc[i][n][e] += part[2][i][n][e] + part[3][i][n][e];
+          sc[i][n][e] *= mul;
+        }
     const int kbase = k0 + kg * NTILES * 8 + t * 2;
     const bool inside = k0 + kKeys - 1 <= min(pos0, last) && (a.window <= 0 || k0 > hi - a.window) && full_tile;
     float top[S::kMTiles][2];
@@ -204,7 +222,6 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
       for (int n = 0; n < NTILES; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          sc[i][n][e] = (sc[i][n][e] + sd[i][n][e]) * mul;
           if (!inside) {                              // some row of the block does not see the whole stage
             const int j = kbase + n * 8 + (e & 1), p = vis[i][e >> 1];
             if (!(j <= min(p, last) && (a.window <= 0 || j > p - a.window))) sc[i][n][e] = -INFINITY;
@@ -288,7 +305,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tm, const NxLatentAttnArg
           ldmatrix_x4(pa[i], smem_addr(sP + (i * 16 + (lane & 15)) * kLdP + kk * 16 + (lane >> 4) * 8));
 #pragma unroll
         for (int c = 0; c < N; ++c)
-          if (N == CT || c < n) ldmatrix_x4_trans(vb[c], base + v_off[kk] + c * (WARPS / 4) * slab_bytes);
+          if (N == CT || c < n) ldmatrix_x4_trans(vb[c], base + v_off[kk] + c * (WARPS / 4) * kSlab);
 #pragma unroll
         for (int c = 0; c < N; ++c)
           if (N == CT || c < n) {
@@ -391,7 +408,7 @@ __global__ void latent_merge_kernel(const NxLatentAttnArgs a) {
 }
 
 template <int MT, int CT>
-int launch(const CUtensorMap& tm, const NxLatentAttnArgs* a, int box_shift, cudaStream_t st) {
+int launch(const CUtensorMap& tm, const NxLatentAttnArgs* a, cudaStream_t st) {
   using S = Shape<MT>;
   const int stage = S::kKeys * a->row * 2, fixed = S::kRows * (a->row + 8) * 2 + S::kTail;
   // two blocks per SM where two stages fit twice, else one block with a deeper ring
@@ -406,16 +423,16 @@ int launch(const CUtensorMap& tm, const NxLatentAttnArgs* a, int box_shift, cuda
   }
   const int rt = std::min(a->heads, S::kRows), tq = std::max(1, S::kRows / rt);
   const dim3 grid(a->seg.total_len / tq + a->seg.count, (a->heads + rt - 1) / rt, a->splits);
-  latent_attn_kernel<MT, CT><<<grid, S::kWarps * 32, fixed + stages * stage, st>>>(tm, *a, rt, tq, stages, box_shift);
+  latent_attn_kernel<MT, CT><<<grid, S::kWarps * 32, fixed + stages * stage, st>>>(tm, *a, rt, tq, stages);
   return launch_status();
 }
 
 template <int MT>
-int launch_rank(const CUtensorMap& tm, const NxLatentAttnArgs* a, int box_shift, cudaStream_t st) {
+int launch_rank(const CUtensorMap& tm, const NxLatentAttnArgs* a, cudaStream_t st) {
   constexpr int kW = Shape<MT>::kWarps;
-  if (a->rank <= 128) return launch<MT, 8 / kW>(tm, a, box_shift, st);
-  if (a->rank <= 256) return launch<MT, 16 / kW>(tm, a, box_shift, st);
-  return launch<MT, 32 / kW>(tm, a, box_shift, st);
+  if (a->rank <= 128) return launch<MT, 8 / kW>(tm, a, st);
+  if (a->rank <= 256) return launch<MT, 16 / kW>(tm, a, st);
+  return launch<MT, 32 / kW>(tm, a, st);
 }
 
 }  // namespace
@@ -429,8 +446,6 @@ extern "C" int nx_latent_attention(const NxLatentAttnArgs* a, nx_stream_t stream
   if ((reinterpret_cast<uintptr_t>(a->q) & 15) || (reinterpret_cast<uintptr_t>(a->cache) & 15)) return -1;
   if (a->seg.count <= 0 || a->seg.max_len <= 0) return 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  int box_shift = 3;                                        // keys of one page per copy: a power of two up to a stage
-  while (box_shift < 5 && a->block_size % (2 << box_shift) == 0) ++box_shift;
   CUtensorMap tm;
   {
     // {64 columns, cache slots, slabs}: one copy brings whole rows, slab by slab
@@ -438,15 +453,15 @@ extern "C" int nx_latent_attention(const NxLatentAttnArgs* a, nx_stream_t stream
     if (fn == nullptr) return -3;
     const cuuint32_t slabs = static_cast<cuuint32_t>(a->row / 64);
     cuuint64_t dims[3] = {64, static_cast<cuuint64_t>(a->n_slots), slabs}, strides[2] = {static_cast<cuuint64_t>(a->row) * 2, 128};
-    cuuint32_t box[3] = {64, 1u << box_shift, slabs}, one[3] = {1, 1, 1};
+    cuuint32_t box[3] = {64, kBox, slabs}, one[3] = {1, 1, 1};
     if (fn(&tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(a->cache), dims, strides, box, one,
            CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
            CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
       return -4;
   }
   const int rows = a->seg.max_len > 1 ? 64 : a->heads;      // (token, head) pairs of a block
-  const int rc = rows <= 16 ? launch_rank<1>(tm, a, box_shift, st)
-                 : rows <= 32 && a->row <= 640 ? launch_rank<2>(tm, a, box_shift, st) : launch_rank<4>(tm, a, box_shift, st);
+  const int rc = rows <= 16 ? launch_rank<1>(tm, a, st)
+                 : rows <= 32 && a->row <= 640 ? launch_rank<2>(tm, a, st) : launch_rank<4>(tm, a, st);
   if (rc == 0 && a->splits > 1) {
     latent_merge_kernel<<<dim3(a->seg.max_len, a->heads, a->seg.count), std::min(128, (a->rank / 4 + 31) / 32 * 32), 0, st>>>(*a);
     return launch_status();
