@@ -322,6 +322,21 @@ def test_fp32_latent_attention(H, rank, rot, window):
     assert _err(out, _absorbed_ref(q, lat, segs, H, rank, window, 0.05, gate)) < 5e-6
 
 
+@pytest.mark.parametrize("window", [0, 40])
+def test_paged_window_kernels_on_a_latent_cache(window):
+    """The general BF16 kernels: values as the leading columns of the keys, gated outputs, spans of the keys."""
+    M = _m()
+    H, rank, row = 5, 96, 128
+    cache, table, lat = _paged([150, 60], 16, row, rank, 2, torch.bfloat16)
+    for segs, splits in (([(0, 1, 149, 0), (1, 1, 59, 1)], 1), ([(0, 1, 149, 0), (1, 1, 59, 1)], 3), ([(0, 70, 80, 0), (70, 30, 10, 1)], 1)):
+        n = max(s[0] + s[1] for s in segs)
+        q, gate = _rand((n, H * row), 7, torch.bfloat16), torch.rand((n, H), generator=torch.Generator().manual_seed(3))
+        out = torch.zeros((n, H * rank), dtype=torch.bfloat16, device=DEV)
+        M.paged_window_attention(q.to(DEV), cache.to(DEV), None, table.to(DEV), out, _segs(segs), heads=H, block_size=16, window=window,
+                                 scale=0.08, gate=gate.to(DEV), vdim=rank, splits=splits)
+        assert _err(out, _absorbed_ref(q, lat, segs, H, rank, window, 0.08, gate)) < 6e-3
+
+
 # ---------------------------------------------------------------------------------------------- attention of prompts
 def _prompt_ref(q, kv, lat, segs, H, dim, rot, vdim, rank, window, scale, gate):
     out = torch.zeros((q.shape[0], H, vdim), dtype=torch.float64)
