@@ -1,14 +1,16 @@
-// Attention of prompt segments on tcgen05 where a key is a part of its own head beside a part that all heads share (see
-// nx_api_mixers.h).  Queries, keys and values of all segments lie packed in row buffers; a work item is a block of up to 256
-// query rows of one segment and one head.
+// Attention of prompt segments on tcgen05 (see nx_api_mixers.h).  A key is a part of its own KV head, optionally beside a part
+// that all heads share; a row sees a window of keys and optionally the first keys of its sequence; a sink may count in the
+// denominator.  Queries, keys and values of all segments lie packed in row buffers; a work item is a block of up to 256 query
+// rows of one segment and one head.
 //
 // The pipeline is that of the two-tile flash kernel: one persistent CTA per SM, softmax group A (warps 0-3) on query rows
 // 0-127 of the block, group B (warps 4-7) on rows 128-255, both against the same key tiles; the MMA warp interleaves
 //   PV_A(j-1), QK_A(j), PV_B(j-1), QK_B(j).
 // S and O live in TMEM (S_A 0-127, S_B 128-255, O_A 256.., O_B 384..); the probabilities go back as BF16 into the columns of
 // their score tile and are the A operand of P V from there.  O is rescaled only when a row's maximum has grown by 2^8.
-// Key tiles start at the first key the block can see: with a window no tile is wasted on keys before it.  Keys and values
-// have rings of their own, since a key part of 192 columns leaves room for one stage of values.
+// Key tiles start at the first key the block can see: with a window no tile is wasted on keys before it.  Kept first keys that
+// lie before the window come first, in tiles of their own.  Keys and values have rings of their own, since a key part of 192
+// columns leaves room for one stage of values.
 #include "flash_common.cuh"
 #include "nx_api_mixers.h"
 #include "sm100_ptx.cuh"
@@ -22,11 +24,11 @@ using namespace nx;
 constexpr int kThreads = 320;   // warps 0-3: softmax A, 4-7: softmax B, 8: TMA, 9: MMA
 constexpr int kSlab = 128 * 128;  // bytes of [128 rows][64 columns]
 
-// ND / NV: 64-column slabs of a head's own key part and of its values; the shared part is one slab
-template <int ND, int NV>
+// ND / NV: 64-column slabs of a head's own key part and of its values; NR: of the shared part (0 or 1)
+template <int ND, int NR, int NV>
 struct Cfg {
-  static constexpr int kQBytes = (ND + 1) * kSlab;
-  static constexpr int kKBytes = (ND + 1) * kSlab;
+  static constexpr int kQBytes = (ND + NR) * kSlab;
+  static constexpr int kKBytes = (ND + NR) * kSlab;
   static constexpr int kVBytes = NV * kSlab;
   static constexpr int kKStages = 2;
   static constexpr int kVStages = 2 * kQBytes + 2 * kKBytes + 2 * kVBytes <= 224 * 1024 ? 2 : 1;
@@ -36,19 +38,25 @@ struct Cfg {
 
 struct Dev {
   const int32_t* blocks;     // [n_blocks][4]: first row, rows, position of the first row, buffer row of position 0
+  const int32_t* kept;       // [n_blocks]: buffer row that position 0 has among the kept keys; null: as for the others
   __nv_bfloat16* out;
   const float* gate;
+  const float* sink;
   int* status;
   int64_t ldo;
-  int items, heads, vdim, window, ksteps, rsteps;   // 16-column steps of the own / shared key part
-  float scale;
+  int items, heads, rep, vdim, window, keep_first, ksteps, rsteps;   // rep: query heads per KV head; 16-column steps of the own
+  float scale;                                                       // and the shared key part
 };
 
 struct Work {
   int h, row0, rows, pos0, kv0, k_lo;
-  int jbA, jeA, jbB, jeB, je;      // key tiles of either query tile; tile j holds keys k_lo + 128 j ..
+  int kept0, n_kept;               // buffer row of kept key 0; kept keys before k_lo
+  int shift;                       // key tile j < shift holds kept keys 128 j .., tile j >= shift keys k_lo + 128 (j - shift) ..
+  int jbA, jeA, jbB, jeB, je;      // key tiles of either query tile
+  __device__ __forceinline__ int first_key(int j) const { return j < shift ? j * 128 : k_lo + (j - shift) * 128; }
 };
-// CTA c takes items round * grid + c in even rounds and from the other end in odd ones; blocks are sorted by cost
+// kKeep: rows may keep first keys (the forms without a shared key part).  CTA c takes items round * grid + c in even rounds and from the other end in odd ones; blocks are sorted by cost
+template <bool kKeep>
 __device__ __forceinline__ bool next_work(const Dev& p, int round, Work& w) {
   const int G = static_cast<int>(gridDim.x), c = static_cast<int>(blockIdx.x);
   const int item = round * G + ((round & 1) ? (G - 1 - c) : c);
@@ -61,24 +69,29 @@ __device__ __forceinline__ bool next_work(const Dev& p, int round, Work& w) {
   w.kv0 = b.w;
   const int back = p.window > 0 ? p.window - 1 : 0x3fffffff;
   w.k_lo = max(0, w.pos0 - back);
+  w.n_kept = kKeep ? min(p.keep_first, w.k_lo) : 0;
+  w.shift = (w.n_kept + 127) / 128;
+  w.kept0 = kKeep && p.kept != nullptr ? __ldg(p.kept + item / p.heads) : b.w;
   w.jbA = 0;
-  w.jeA = (w.pos0 + min(128, w.rows) - 1 - w.k_lo) / 128 + 1;
+  w.jeA = w.shift + (w.pos0 + min(128, w.rows) - 1 - w.k_lo) / 128 + 1;
   w.jbB = w.jeB = 0;
   if (w.rows > 128) {
-    w.jbB = (max(0, w.pos0 + 128 - back) - w.k_lo) / 128;
-    w.jeB = (w.pos0 + w.rows - 1 - w.k_lo) / 128 + 1;
+    // rows that keep first keys walk all tiles: those between the kept ones and their window are masked out
+    w.jbB = kKeep && p.keep_first > 0 ? 0 : (max(0, w.pos0 + 128 - back) - w.k_lo) / 128;
+    w.jeB = w.shift + (w.pos0 + w.rows - 1 - w.k_lo) / 128 + 1;
   }
   w.je = max(w.jeA, w.jeB);
   return true;
 }
 
-template <int ND, int NV>
+template <int ND, int NR, int NV>
 __global__ void __launch_bounds__(kThreads, 1)
-latent_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_qr,
-                     const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_kr,
-                     const __grid_constant__ CUtensorMap tm_v, const Dev p) {
-  using C = Cfg<ND, NV>;
+prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_qr,
+              const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_kr,
+              const __grid_constant__ CUtensorMap tm_v, const Dev p) {
+  using C = Cfg<ND, NR, NV>;
   constexpr int KS = C::kKStages, VS = C::kVStages;
+  constexpr bool kKeep = NR == 0;
   extern __shared__ __align__(1024) uint8_t smem[];
   if (smem_u32(smem) & 1023u) {  // the swizzled tiles need a 1 KiB aligned base; uniform early exit
     if (threadIdx.x == 0) atomicCAS(p.status, 0, kStatusBadArgument);
@@ -129,7 +142,7 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         atomicCAS(p.status, 0, kStatusTimeoutProducer);
         return false;
       };
-      for (int round = 0; ok && next_work(p, round, w); ++round) {
+      for (int round = 0; ok && next_work<kKeep>(p, round, w); ++round) {
 #pragma unroll
         for (int x = 0; x < 2; ++x) {
           if (x == 1 && w.jeB <= w.jbB) continue;
@@ -140,23 +153,24 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           uint8_t* d = sQ + x * C::kQBytes;
 #pragma unroll
           for (int s = 0; s < ND; ++s) tma_load_3d(d + s * kSlab, &tm_q, &q_full[x], 64 * s, w.h, w.row0 + x * 128);
-          tma_load_3d(d + ND * kSlab, &tm_qr, &q_full[x], 0, w.h, w.row0 + x * 128);
+          if constexpr (NR > 0) tma_load_3d(d + ND * kSlab, &tm_qr, &q_full[x], 0, w.h, w.row0 + x * 128);
         }
+        const int hk = kKeep ? w.h / p.rep : w.h;
         for (int j = 0; ok && j < w.je; ++j, ++n_kv) {
-          const int row = w.kv0 + w.k_lo + j * 128;
+          const int row = (j < w.shift ? w.kept0 : w.kv0) + w.first_key(j);
           const int s = n_kv % KS, v = n_kv % VS;
           ok = wait(&k_empty[s], ((n_kv / KS) & 1) ^ 1);
           if (!ok) break;
           mbar_arrive_expect_tx(&k_full[s], C::kKBytes);
           uint8_t* d = sK + s * C::kKBytes;
 #pragma unroll
-          for (int c = 0; c < ND; ++c) tma_load_3d(d + c * kSlab, &tm_k, &k_full[s], 64 * c, w.h, row);
-          tma_load_3d(d + ND * kSlab, &tm_kr, &k_full[s], 0, 0, row);
+          for (int c = 0; c < ND; ++c) tma_load_3d(d + c * kSlab, &tm_k, &k_full[s], 64 * c, hk, row);
+          if constexpr (NR > 0) tma_load_3d(d + ND * kSlab, &tm_kr, &k_full[s], 0, 0, row);
           ok = wait(&v_empty[v], ((n_kv / VS) & 1) ^ 1);
           if (!ok) break;
           mbar_arrive_expect_tx(&v_full[v], C::kVBytes);
 #pragma unroll
-          for (int c = 0; c < NV; ++c) tma_load_3d(sV + v * C::kVBytes + c * kSlab, &tm_v, &v_full[v], 64 * c, w.h, row);
+          for (int c = 0; c < NV; ++c) tma_load_3d(sV + v * C::kVBytes + c * kSlab, &tm_v, &v_full[v], 64 * c, hk, row);
         }
       }
     }
@@ -173,7 +187,7 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       if (leader) atomicCAS(p.status, 0, kStatusTimeoutMma);
       return false;
     };
-    for (int round = 0; ok && next_work(p, round, w); ++round) {
+    for (int round = 0; ok && next_work<kKeep>(p, round, w); ++round) {
       ok = wait(&q_full[0], nq[0] & 1);
       ++nq[0];
       if (ok && w.jeB > w.jbB) {
@@ -212,7 +226,7 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
             if (leader) {
               for (int ks = 0; ks < p.ksteps; ++ks)
                 umma_f16_ss(tmem_s, dQ + kstep_kmajor(128, ks), dK + kstep_kmajor(128, ks), idesc_s, ks > 0 ? 1u : 0u);
-              for (int ks = ND * 4; ks < ND * 4 + p.rsteps; ++ks)
+              for (int ks = ND * 4; NR > 0 && ks < ND * 4 + p.rsteps; ++ks)
                 umma_f16_ss(tmem_s, dQ + kstep_kmajor(128, ks), dK + kstep_kmajor(128, ks), idesc_s, 1u);
               umma_commit(&s_full[x]);
               if (j + 1 == je) umma_commit(&q_empty[x]);
@@ -241,14 +255,14 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       if (lane == 0) atomicCAS(p.status, 0, kStatusTimeoutEpilogue);
       return false;
     };
-    for (int round = 0; ok && next_work(p, round, w); ++round) {
+    for (int round = 0; ok && next_work<kKeep>(p, round, w); ++round) {
       const int jb = x == 0 ? w.jbA : w.jbB, je = x == 0 ? w.jeA : w.jeB;
       if (je <= jb) continue;
       const int p0 = w.pos0 + x * 128, pos = p0 + r;
       const int row_lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
       float m_ref = -INFINITY, l_run = 0.0f;
       for (int j = jb; j < je; ++j, ++cnt) {
-        const int k0 = w.k_lo + j * 128;
+        const int k0 = w.first_key(j);
         ok = wait(&s_full[x], cnt & 1);
         if (!ok) break;
         tc_fence_after_sync();
@@ -256,9 +270,23 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
 #pragma unroll
         for (int cc = 0; cc < 4; ++cc) tmem_ld_32x32b_x32(tmem_s + cc * 32, sv[cc]);
         tmem_ld_wait();
-        const bool need_mask = k0 + 127 > p0 || (p.window > 0 && k0 < p0 + 127 - p.window + 1);
+        const bool need_mask = (kKeep && j < w.shift) || k0 + 127 > p0 || (p.window > 0 && k0 < p0 + 127 - p.window + 1);
         if (need_mask) {
-          const int clo = row_lo - k0, chi = pos - k0;   // column c is visible iff clo <= c <= chi
+          // column c is visible iff clo <= c <= chi; kept keys: those before k_lo, and in later tiles a row's window or, for a
+          // tile that still holds kept keys, everything below keep_first
+          int clo = row_lo - k0, chi = pos - k0;
+          if (kKeep && j < w.shift) {
+            clo = 0;
+            chi = min(chi, w.n_kept - 1 - k0);
+          } else if (kKeep && k0 < p.keep_first) {
+            const int keep = p.keep_first - k0;            // columns below it stay visible
+#pragma unroll
+            for (int cc = 0; cc < 4; ++cc)
+#pragma unroll
+              for (int c = 0; c < 32; ++c)
+                if (cc * 32 + c >= keep && cc * 32 + c < clo) sv[cc][c] = 0xff800000u;
+            clo = 0;
+          }
 #pragma unroll
           for (int cc = 0; cc < 4; ++cc)
 #pragma unroll
@@ -332,6 +360,7 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       tc_fence_after_sync();
       const bool row_ok = x * 128 + r < w.rows;
       const int64_t row = w.row0 + x * 128 + r;
+      if (kKeep && p.sink != nullptr) l_run += ex2f(p.sink[w.h] * kLog2e - m_ref);
       const float inv = row_ok ? (p.gate != nullptr ? p.gate[row * p.heads + w.h] : 1.0f) / l_run : 0.0f;
       __nv_bfloat16* orow = p.out + row * p.ldo + static_cast<int64_t>(w.h) * p.vdim;
 #pragma unroll
@@ -368,17 +397,40 @@ latent_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   }
 }
 
-template <int ND, int NV>
-int launch(const NxLatentPromptArgs* a, const CUtensorMap& tq, const CUtensorMap& tqr, const CUtensorMap& tk, const CUtensorMap& tkr,
-           const CUtensorMap& tv, const Dev& p, int grid, cudaStream_t st) {
-  constexpr int kSmem = Cfg<ND, NV>::kSmem;
+// tensor map of [rows][heads][columns], box 128 x 1 x 64: columns past a part's width arrive as zeros
+int part_map(CUtensorMap* m, const void* base, int cols, int heads, int rows, int64_t head_ld, int64_t row_ld) {
+  nx::EncodeTiledFn fn = nx::encode_tiled_fn();
+  if (fn == nullptr) return -3;
+  cuuint64_t dims[3] = {static_cast<cuuint64_t>(cols), static_cast<cuuint64_t>(heads), static_cast<cuuint64_t>(rows)};
+  cuuint64_t strides[2] = {static_cast<cuuint64_t>(head_ld) * 2, static_cast<cuuint64_t>(row_ld) * 2};
+  cuuint32_t box[3] = {64, 1, 128}, one[3] = {1, 1, 1};
+  return fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, one, CU_TENSOR_MAP_INTERLEAVE_NONE,
+            CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS
+             ? 0
+             : -4;
+}
+
+struct Maps {
+  CUtensorMap q, qr, k, kr, v;
+};
+
+template <int ND, int NR, int NV>
+int launch(const Maps& t, const Dev& p, cudaStream_t st) {
+  constexpr int kSmem = Cfg<ND, NR, NV>::kSmem;
   static bool once = false;
   if (!once) {
-    if (cudaFuncSetAttribute(latent_prompt_kernel<ND, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -2;
+    if (cudaFuncSetAttribute(prompt_kernel<ND, NR, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -2;
     once = true;
   }
-  latent_prompt_kernel<ND, NV><<<grid, kThreads, kSmem, st>>>(tq, tqr, tk, tkr, tv, p);
+  int sms = 0, dev = 0;
+  if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) return -2;
+  prompt_kernel<ND, NR, NV><<<std::min(p.items, sms), kThreads, kSmem, st>>>(t.q, t.qr, t.k, t.kr, t.v, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+template <int NR>
+int launch_sizes(int dim, int vdim, const Maps& t, const Dev& p, cudaStream_t st) {
+  if (dim <= 64) return vdim <= 64 ? launch<1, NR, 1>(t, p, st) : launch<1, NR, 2>(t, p, st);
+  return vdim <= 64 ? launch<2, NR, 1>(t, p, st) : launch<2, NR, 2>(t, p, st);
 }
 
 // copies the cache rows of a segment list into one packed buffer: keys `base` .. of every segment, 16 bytes per thread
@@ -418,47 +470,63 @@ extern "C" int nx_latent_prompt(const NxLatentPromptArgs* a, nx_stream_t stream)
   for (const void* ptr : {a->q, a->kv, a->lat, static_cast<const void*>(a->out)})
     if (ptr == nullptr || (reinterpret_cast<uintptr_t>(ptr) & 15)) return -1;
   if (a->n_blocks <= 0) return 0;
-  CUtensorMap tq, tqr, tk, tkr, tv;
-  const auto bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   const auto* q = static_cast<const __nv_bfloat16*>(a->q);
   const auto* kv = static_cast<const __nv_bfloat16*>(a->kv);
   const auto* lat = static_cast<const __nv_bfloat16*>(a->lat);
-  const uint64_t H = static_cast<uint64_t>(a->heads);
-  // {columns, heads, rows}, box {64, 1, 128}: columns past a part's width arrive as zeros
-  const auto map = [&](CUtensorMap* m, const __nv_bfloat16* base, uint64_t cols, uint64_t heads, uint64_t rows, uint64_t head_ld,
-                        uint64_t row_ld) {
-    nx::EncodeTiledFn fn = nx::encode_tiled_fn();
-    if (fn == nullptr) return -3;
-    cuuint64_t dims[3] = {cols, heads, rows}, strides[2] = {head_ld * 2, row_ld * 2};
-    cuuint32_t box[3] = {64, 1, 128}, one[3] = {1, 1, 1};
-    return fn(m, bf, 3, const_cast<__nv_bfloat16*>(base), dims, strides, box, one, CU_TENSOR_MAP_INTERLEAVE_NONE,
-              CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS
-               ? 0
-               : -4;
-  };
+  const int H = a->heads;
+  Maps t;
   int rc;
-  if ((rc = map(&tq, q, a->dim, H, a->q_rows, a->q_head, a->ldq))) return rc;
-  if ((rc = map(&tqr, q + a->dim, a->rot, H, a->q_rows, a->q_head, a->ldq))) return rc;
-  if ((rc = map(&tk, kv, a->dim, H, a->kv_rows, a->dim, a->ldkv))) return rc;
-  if ((rc = map(&tv, kv + static_cast<int64_t>(H) * a->dim, a->vdim, H, a->kv_rows, a->vdim, a->ldkv))) return rc;
-  if ((rc = map(&tkr, lat + a->rank, a->rot, 1, a->kv_rows, a->ld_lat, a->ld_lat))) return rc;
+  if ((rc = part_map(&t.q, q, a->dim, H, a->q_rows, a->q_head, a->ldq))) return rc;
+  if ((rc = part_map(&t.qr, q + a->dim, a->rot, H, a->q_rows, a->q_head, a->ldq))) return rc;
+  if ((rc = part_map(&t.k, kv, a->dim, H, a->kv_rows, a->dim, a->ldkv))) return rc;
+  if ((rc = part_map(&t.v, kv + static_cast<int64_t>(H) * a->dim, a->vdim, H, a->kv_rows, a->vdim, a->ldkv))) return rc;
+  if ((rc = part_map(&t.kr, lat + a->rank, a->rot, 1, a->kv_rows, a->ld_lat, a->ld_lat))) return rc;
   Dev p{};
   p.blocks = a->blocks;
   p.out = static_cast<__nv_bfloat16*>(a->out);
   p.gate = a->gate;
   p.status = a->status;
   p.ldo = a->ldo;
-  p.items = a->n_blocks * a->heads;
-  p.heads = a->heads;
+  p.items = a->n_blocks * H;
+  p.heads = H;
+  p.rep = 1;
   p.vdim = a->vdim;
   p.window = a->window;
   p.ksteps = a->dim / 16;
   p.rsteps = a->rot / 16;
   p.scale = a->scale;
-  int sms = 0, dev = 0;
-  if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) return -2;
-  const int grid = std::min(p.items, sms);
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (a->dim <= 64) return a->vdim <= 64 ? launch<1, 1>(a, tq, tqr, tk, tkr, tv, p, grid, st) : launch<1, 2>(a, tq, tqr, tk, tkr, tv, p, grid, st);
-  return a->vdim <= 64 ? launch<2, 1>(a, tq, tqr, tk, tkr, tv, p, grid, st) : launch<2, 2>(a, tq, tqr, tk, tkr, tv, p, grid, st);
+  return launch_sizes<1>(a->dim, a->vdim, t, p, static_cast<cudaStream_t>(stream));
+}
+
+extern "C" int nx_window_prompt(const NxWindowPromptArgs* a, nx_stream_t stream) {
+  if (a == nullptr || a->status == nullptr || a->blocks == nullptr || a->heads <= 0 || a->kv_heads <= 0 || !(a->scale > 0.0f)) return -1;
+  if (a->heads % a->kv_heads || a->keep_first < 0) return -1;
+  if (a->dim <= 0 || a->dim > 128 || (a->dim & 15) || a->vdim <= 0 || a->vdim > 128 || (a->vdim & 7)) return -1;
+  if ((a->ldq | a->ldk | a->ldv | a->ldo) & 7) return -1;
+  for (const void* ptr : {a->q, a->k, a->v, static_cast<const void*>(a->out), static_cast<const void*>(a->blocks)})
+    if (ptr == nullptr || (reinterpret_cast<uintptr_t>(ptr) & 15)) return -1;
+  if (a->n_blocks <= 0) return 0;
+  Maps t;
+  int rc;
+  if ((rc = part_map(&t.q, a->q, a->dim, a->heads, a->q_rows, a->dim, a->ldq))) return rc;
+  if ((rc = part_map(&t.k, a->k, a->dim, a->kv_heads, a->kv_rows, a->dim, a->ldk))) return rc;
+  if ((rc = part_map(&t.v, a->v, a->vdim, a->kv_heads, a->kv_rows, a->vdim, a->ldv))) return rc;
+  t.qr = t.q;                // not used without a shared key part
+  t.kr = t.k;
+  Dev p{};
+  p.blocks = a->blocks;
+  p.kept = a->kept;
+  p.out = static_cast<__nv_bfloat16*>(a->out);
+  p.sink = a->sink;
+  p.status = a->status;
+  p.ldo = a->ldo;
+  p.items = a->n_blocks * a->heads;
+  p.heads = a->heads;
+  p.rep = a->heads / a->kv_heads;
+  p.vdim = a->vdim;
+  p.window = a->window;
+  p.keep_first = a->window > 0 ? a->keep_first : 0;
+  p.ksteps = a->dim / 16;
+  p.scale = a->scale;
+  return launch_sizes<0>(a->dim, a->vdim, t, p, static_cast<cudaStream_t>(stream));
 }

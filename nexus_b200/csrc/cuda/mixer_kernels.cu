@@ -1,6 +1,7 @@
 // Memory-bound building blocks of decoders with heterogeneous layers (see nx_api_mixers.h): the chain "add the normed
 // sublayer output, norm for the next sublayer", rotary embedding fused with the paged cache append, the short causal
-// convolution with its carried tail, gated norms, the per-layer token input, SwiGLU and logit soft-capping.
+// convolution with its carried tail (alone, or with rotation and append), low-rank decays, gated norms, the per-layer token
+// input, gated activations and logit soft-capping.
 // Everything is computed in FP32; activations are read and written in BF16 or FP32.
 #include "common.cuh"
 #include "mixer_common.cuh"
@@ -47,8 +48,9 @@ __global__ void residual_norm_kernel(const NxResidualNormArgs a) {
         for (int k = 0; k < a.top; ++k) {
           float u[V];
           load_vec<T, V>(static_cast<const T*>(a.experts) + static_cast<int64_t>(a.expert_slots[r * a.top + k]) * a.ld_experts + c, u);
+          const float w = a.expert_weights != nullptr ? a.expert_weights[r * a.top + k] : 1.0f;
 #pragma unroll
-          for (int j = 0; j < V; ++j) v[j] += u[j];
+          for (int j = 0; j < V; ++j) v[j] += w * u[j];
         }
         if (a.y != nullptr) {
           float u[V];
@@ -62,12 +64,24 @@ __global__ void residual_norm_kernel(const NxResidualNormArgs a) {
       } else {
         load_vec<T, V>(yr + c, v);
       }
+      if (a.w_post == nullptr) {            // the output is added as it is
+        float xv[V];
+        load_vec<float, V>(xr + c, xv);
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+          v[j] = xv[j] + a.res_mult * v[j];
+          ss += v[j] * v[j];
+        }
+        store_vec<float, V>(xr + c, v);
+        store_vec<float, V>(s_row + c, v);
+        continue;
+      }
       store_vec<float, V>(s_row + c, v);
 #pragma unroll
       for (int j = 0; j < V; ++j) sy += v[j] * v[j];
     }
-    const float inv = a.res_mult / sqrtf(block_sum(sy, s_red) * inv_cols + a.eps);
-    for (int c = threadIdx.x * V; c < cols; c += blockDim.x * V) {   // each thread re-reads its own columns
+    const float inv = a.w_post != nullptr ? a.res_mult / sqrtf(block_sum(sy, s_red) * inv_cols + a.eps) : 0.0f;
+    for (int c = threadIdx.x * V; c < cols && a.w_post != nullptr; c += blockDim.x * V) {   // each thread re-reads its own columns
       float v[V], xv[V], w[V];
       load_vec<float, V>(s_row + c, v);
       load_vec<float, V>(xr + c, xv);
@@ -195,7 +209,8 @@ __global__ void latent_prep_kernel(const NxLatentPrepArgs a) {
   const T* row = static_cast<const T*>(a.proj) + r * a.ld;
   const int64_t pos = a.positions[r], slot = a.slots[r];
   const T *q = row + a.q_off, *k = row + a.c_off;
-  const float inv_q = 1.0f / sqrtf(block_sum(sum_squares<T, V>(q, a.q_rank), s_red) / static_cast<float>(a.q_rank) + a.eps);
+  const float inv_q =
+      a.q_rank > 0 ? 1.0f / sqrtf(block_sum(sum_squares<T, V>(q, a.q_rank), s_red) / static_cast<float>(a.q_rank) + a.eps) : 0.0f;
   const float inv_k = 1.0f / sqrtf(block_sum(sum_squares<T, V>(k, a.kv_rank), s_red) / static_cast<float>(a.kv_rank) + a.eps);
   T* cq = static_cast<T*>(a.cq) + r * a.ldq;
   for (int c = threadIdx.x * V; c < a.q_rank; c += blockDim.x * V) {
@@ -236,6 +251,7 @@ __global__ void latent_prep_kernel(const NxLatentPrepArgs a) {
     for (int c = a.kv_rank + threadIdx.x; c < a.rot_col; c += blockDim.x) Num<T>::store(lat + c, 0.0f);
     for (int c = a.rot_col + a.rot_dims + threadIdx.x; c < a.ld_cache; c += blockDim.x) Num<T>::store(lat + c, 0.0f);
   }
+  if (a.gate == nullptr) return;
   for (int h = threadIdx.x; h < a.heads; h += blockDim.x)
     a.gate[r * a.heads + h] = sigmoid_exact(Num<T>::load(row + a.g_off + h));
 }
@@ -280,8 +296,9 @@ __global__ void rope_heads_kernel(const T* __restrict__ src, int64_t ld_src, int
 // ------------------------------------------------------------------------------------------------
 constexpr int kConvTile = 32;
 
-template <typename T, int TAPS, int V>
-__global__ void conv_silu_kernel(const NxConvArgs a) {
+// emit(row, token of the segment, sums of V channels) for every token of the tile
+template <typename T, int TAPS, int V, typename Emit>
+__device__ __forceinline__ void conv_tile(const NxConvArgs& a, Emit emit) {
   const int sg = blockIdx.z;
   const int len = a.seg.len[sg];
   const int t0 = blockIdx.y * kConvTile;
@@ -295,7 +312,6 @@ __global__ void conv_silu_kernel(const NxConvArgs a) {
 #pragma unroll
   for (int v = 0; v < V; ++v) bias[v] = a.bias != nullptr ? a.bias[c + v] : 0.0f;
   const T* x = static_cast<const T*>(a.x) + row0 * a.ldx + c;
-  T* y = static_cast<T*>(a.y) + row0 * a.ldy + c;
   T* st = static_cast<T*>(a.state) + static_cast<int64_t>(a.seg.seq[sg]) * (TAPS - 1) * a.channels + c;
   const bool carried = a.seg.pos[sg] > 0;
 #pragma unroll
@@ -338,14 +354,61 @@ __global__ void conv_silu_kernel(const NxConvArgs a) {
     for (int j = 0; j < TAPS - 1; ++j)
 #pragma unroll
       for (int v = 0; v < V; ++v) acc[v] += w[j][v] * hist[j][v];
-#pragma unroll
-    for (int v = 0; v < V; ++v) acc[v] = sizeof(T) == 4 ? silu_exact(acc[v]) : acc[v] * __fdividef(1.0f, 1.0f + __expf(-acc[v]));
-    store_vec<T, V>(y + static_cast<int64_t>(t) * a.ldy, acc);
+    emit(row0 + t, t, acc);
 #pragma unroll
     for (int j = 0; j < TAPS - 1; ++j)
 #pragma unroll
       for (int v = 0; v < V; ++v) hist[j][v] = j + 1 < TAPS - 1 ? hist[j + 1 < HIST ? j + 1 : j][v] : cur[v];
   }
+}
+
+template <typename T, int TAPS, int V>
+__global__ void conv_silu_kernel(const NxConvArgs a) {
+  T* y = static_cast<T*>(a.y) + (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  conv_tile<T, TAPS, V>(a, [&](int64_t row, int, float (&acc)[V]) {
+#pragma unroll
+    for (int v = 0; v < V; ++v) acc[v] = sizeof(T) == 4 ? silu_exact(acc[v]) : acc[v] * __fdividef(1.0f, 1.0f + __expf(-acc[v]));
+    store_vec<T, V>(y + row * a.ldy, acc);
+  });
+}
+
+// convolution + rotation of neighbouring pairs + value mixing + cache append: a thread's V channels lie in one head
+template <typename T, int TAPS, int V>
+__global__ void conv_rope_kernel(const NxConvRopeArgs a) {
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim, half = a.rot_dims / 2;
+  const int part = c < nq ? 0 : c < nq + nk ? 1 : 2;                  // q, k, v
+  const int u = part == 0 ? c : part == 1 ? c - nq : c - nq - nk;     // column inside the part
+  const int d = part < 2 ? u % a.dim : 0;
+  T* y = static_cast<T*>(a.conv.y) + c;
+  T* first = static_cast<T*>(a.first) + u;
+  const float mix = a.mix != nullptr ? *a.mix : 0.0f;
+  const int pos0 = a.conv.seg.pos[blockIdx.z];
+  conv_tile<T, TAPS, V>(a.conv, [&](int64_t row, int t, float (&acc)[V]) {
+    const int64_t slot = part > 0 ? a.slots[row] : -1;
+    if (part < 2) {
+      const int64_t at = static_cast<int64_t>(pos0 + t) * half + d / 2;
+#pragma unroll
+      for (int v = 0; v < V; v += 2)
+        if (d + v < a.rot_dims) {
+          const float cs = a.cos_t[at + v / 2], sn = a.sin_t[at + v / 2], p = acc[v], q = acc[v + 1];
+          acc[v] = p * cs - q * sn;
+          acc[v + 1] = q * cs + p * sn;
+        }
+      if (part == 1 && slot >= 0) store_vec<T, V>(static_cast<T*>(a.k_cache) + slot * nk + u, acc);
+    } else {
+      if (a.mix != nullptr) {
+        float f[V];
+        load_vec<T, V>(first + row * nv, f);
+#pragma unroll
+        for (int v = 0; v < V; ++v) acc[v] = (1.0f - mix) * acc[v] + mix * f[v];
+      } else if (a.first != nullptr) {
+        store_vec<T, V>(first + row * nv, acc);
+      }
+      if (slot >= 0) store_vec<T, V>(static_cast<T*>(a.v_cache) + slot * nv + u, acc);
+    }
+    if (part == 0 || a.store_kv) store_vec<T, V>(y + row * a.conv.ldy, acc);
+  });
 }
 
 // ------------------------------------------------------------------------------------------------
@@ -441,38 +504,95 @@ __global__ void token_side_kernel(const float* __restrict__ a, int64_t lda, cons
   }
 }
 
+// V == 8 or 1; a column's gate and value: halves of a row, or turns of eight columns (interleaved)
 template <typename T, int V>
-__global__ void silu_mul_kernel(const T* __restrict__ h, int64_t ldh, T* __restrict__ out, int64_t ldo, int half) {
+__global__ void glu_kernel(const T* __restrict__ h, int64_t ldh, T* __restrict__ out, int64_t ldo, int half, int interleaved,
+                           const NxGlu f) {
   const int64_t r = blockIdx.y;
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
   if (c >= half) return;
+  const T* p = h + r * ldh + (interleaved ? c / 8 * 16 + c % 8 : c);
   float g[V], u[V];
-  load_vec<T, V>(h + r * ldh + c, g);
-  load_vec<T, V>(h + r * ldh + half + c, u);
+  load_vec<T, V>(p, g);
+  load_vec<T, V>(p + (interleaved ? 8 : half), u);
 #pragma unroll
-  for (int j = 0; j < V; ++j) g[j] = (sizeof(T) == 4 ? silu_exact(g[j]) : g[j] * __fdividef(1.0f, 1.0f + __expf(-g[j]))) * u[j];
+  for (int j = 0; j < V; ++j) g[j] = glu_apply<sizeof(T) == 4>(f, g[j], u[j]);
   store_vec<T, V>(out + r * ldo + c, g);
 }
 
-__global__ void softcap_kernel(float* __restrict__ x, int64_t ld, int cols, float cap) {
+__global__ void softcap_kernel(float* __restrict__ x, int64_t ld, int cols, float cap, float scale) {
   float* xr = x + blockIdx.y * ld;
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
-  if (c < cols) xr[c] = cap * tanhf(xr[c] / cap);
+  if (c < cols) xr[c] = cap > 0.0f ? cap * tanhf(scale * xr[c] / cap) : scale * xr[c];
 }
 
+// log2 of a decay sigmoid(z)^(1 / tau) with z of low rank: 128 columns x 32 rows per block, 16 rows per thread
+constexpr int kDecayCols = 128, kDecayRows = 32, kDecayRank = 16;
+template <typename T>
+__global__ void __launch_bounds__(256)
+decay_gate_kernel(const T* __restrict__ a, int64_t lda, const float* __restrict__ w, const float* __restrict__ bias,
+                  float* __restrict__ out, int64_t ldo, int rows, int cols, int rank, float mul) {
+  __shared__ float s_w[kDecayRank][kDecayCols + 1], s_a[kDecayRows][kDecayRank];
+  const int c0 = blockIdx.x * kDecayCols, tx = threadIdx.x % kDecayCols, ty = threadIdx.x / kDecayCols, c = c0 + tx;
+  const int64_t r0 = static_cast<int64_t>(blockIdx.y) * kDecayRows;
+  float acc[16];
+#pragma unroll
+  for (int i = 0; i < 16; ++i) acc[i] = 0.0f;
+  for (int k0 = 0; k0 < rank; k0 += kDecayRank) {
+    __syncthreads();
+    for (int i = threadIdx.x; i < kDecayCols * kDecayRank; i += 256) {
+      const int col = i / kDecayRank, k = i % kDecayRank;
+      s_w[k][col] = c0 + col < cols && k0 + k < rank ? w[static_cast<int64_t>(c0 + col) * rank + k0 + k] : 0.0f;
+    }
+    for (int i = threadIdx.x; i < kDecayRows * kDecayRank; i += 256) {
+      const int row = i / kDecayRank, k = i % kDecayRank;
+      s_a[row][k] = r0 + row < rows && k0 + k < rank ? Num<T>::load(a + (r0 + row) * lda + k0 + k) : 0.0f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kDecayRank; ++k) {
+      const float wk = s_w[k][tx];
+#pragma unroll
+      for (int i = 0; i < 16; ++i) acc[i] = fmaf(s_a[ty * 16 + i][k], wk, acc[i]);
+    }
+  }
+  if (c >= cols) return;
+  const float b = bias[c];
+#pragma unroll
+  for (int i = 0; i < 16; ++i)
+    if (r0 + ty * 16 + i < rows) out[(r0 + ty * 16 + i) * ldo + c] = -softplus_exact(-(acc[i] + b)) * mul;
+}
+
+bool conv_ok(const NxConvArgs& a) {
+  return a.channels > 0 && a.taps >= 1 && a.taps <= 8 && a.seg.count <= 65535 && (a.seg.max_len + kConvTile - 1) / kConvTile <= 65535;
+}
+template <int V>
+dim3 conv_grid(const NxConvArgs& a, int threads) {
+  return dim3((a.channels / V + threads - 1) / threads, (a.seg.max_len + kConvTile - 1) / kConvTile, a.seg.count);
+}
+constexpr int kConvThreads = 128;
+#define NX_CONV_TAPS(KERNEL_, CONV_)                                                                             \
+  switch ((CONV_).taps) {                                                                                        \
+    case 1: KERNEL_<T, 1, V><<<conv_grid<V>(CONV_, kConvThreads), kConvThreads, 0, st>>>(*a); break;             \
+    case 2: KERNEL_<T, 2, V><<<conv_grid<V>(CONV_, kConvThreads), kConvThreads, 0, st>>>(*a); break;             \
+    case 3: KERNEL_<T, 3, V><<<conv_grid<V>(CONV_, kConvThreads), kConvThreads, 0, st>>>(*a); break;             \
+    case 4: KERNEL_<T, 4, V><<<conv_grid<V>(CONV_, kConvThreads), kConvThreads, 0, st>>>(*a); break;             \
+    case 5: KERNEL_<T, 5, V><<<conv_grid<V>(CONV_, kConvThreads), kConvThreads, 0, st>>>(*a); break;             \
+    case 6: KERNEL_<T, 6, V><<<conv_grid<V>(CONV_, kConvThreads), kConvThreads, 0, st>>>(*a); break;             \
+    case 7: KERNEL_<T, 7, V><<<conv_grid<V>(CONV_, kConvThreads), kConvThreads, 0, st>>>(*a); break;             \
+    case 8: KERNEL_<T, 8, V><<<conv_grid<V>(CONV_, kConvThreads), kConvThreads, 0, st>>>(*a); break;             \
+    default: return -1;                                                                                          \
+  }                                                                                                              \
+  return launch_status()
 template <typename T, int V>
 int launch_conv(const NxConvArgs* a, cudaStream_t st) {
-  const int threads = 128;
-  dim3 grid((a->channels / V + threads - 1) / threads, (a->seg.max_len + kConvTile - 1) / kConvTile, a->seg.count);
-#define NX_CONV(TAPS_) \
-  case TAPS_: conv_silu_kernel<T, TAPS_, V><<<grid, threads, 0, st>>>(*a); break
-  switch (a->taps) {
-    NX_CONV(1); NX_CONV(2); NX_CONV(3); NX_CONV(4); NX_CONV(5); NX_CONV(6); NX_CONV(7); NX_CONV(8);
-    default: return -1;
-  }
-#undef NX_CONV
-  return launch_status();
+  NX_CONV_TAPS(conv_silu_kernel, *a);
 }
+template <typename T, int V>
+int launch_conv_rope(const NxConvRopeArgs* a, cudaStream_t st) {
+  NX_CONV_TAPS(conv_rope_kernel, a->conv);
+}
+#undef NX_CONV_TAPS
 
 template <typename T>
 int launch_residual(const NxResidualNormArgs* a, cudaStream_t st) {
@@ -499,7 +619,6 @@ int launch_residual(const NxResidualNormArgs* a, cudaStream_t st) {
 extern "C" int nx_residual_norm(const NxResidualNormArgs* a, nx_stream_t stream) {
   if (a == nullptr || a->cols <= 0 || a->x == nullptr) return -1;
   if (a->rows <= 0) return 0;
-  if ((a->y != nullptr || a->experts != nullptr) && a->w_post == nullptr) return -1;
   if (a->experts != nullptr && (a->expert_slots == nullptr || a->top < 1)) return -1;
   if (a->scatter != nullptr && (a->scatter_slots == nullptr || a->top < 1 || a->ldh < a->cols)) return -1;
   if (a->w_dot != nullptr && a->dot_out == nullptr) return -1;
@@ -526,7 +645,7 @@ extern "C" int nx_rope_append(const NxRopeAppendArgs* a, nx_stream_t stream) {
 }
 
 extern "C" int nx_latent_prep(const NxLatentPrepArgs* a, nx_stream_t stream) {
-  if (a == nullptr || a->q_rank <= 0 || a->kv_rank <= 0 || a->heads <= 0 || a->rot_dims < 0 || (a->rot_dims & 1)) return -1;
+  if (a == nullptr || a->q_rank < 0 || a->kv_rank <= 0 || a->heads <= 0 || a->rot_dims < 0 || (a->rot_dims & 1)) return -1;
   if (a->ldq < a->q_rank || a->rot_col < a->kv_rank || a->ld_cache < a->rot_col + a->rot_dims) return -1;
   if (a->rows <= 0) return 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
@@ -571,9 +690,8 @@ extern "C" int nx_rope_heads(const void* src, int64_t ld_src, int src_head, int 
 }
 
 extern "C" int nx_conv_silu(const NxConvArgs* a, nx_stream_t stream) {
-  if (a == nullptr || a->channels <= 0 || a->taps < 1 || a->taps > 8) return -1;
+  if (a == nullptr || !conv_ok(*a)) return -1;
   if (a->seg.count <= 0 || a->seg.max_len <= 0) return 0;
-  if (a->seg.count > 65535 || (a->seg.max_len + kConvTile - 1) / kConvTile > 65535) return -1;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const bool v2 = a->channels % 2 == 0 && a->ldx % 2 == 0 && a->ldy % 2 == 0 && (reinterpret_cast<uintptr_t>(a->x) & 7) == 0;
   const bool v4 = a->channels % 4 == 0 && a->ldx % 4 == 0 && a->ldy % 4 == 0 && (reinterpret_cast<uintptr_t>(a->x) & 7) == 0 &&
@@ -582,6 +700,40 @@ extern "C" int nx_conv_silu(const NxConvArgs* a, nx_stream_t stream) {
   if (a->dtype == NX_BF16) return v2 ? launch_conv<__nv_bfloat16, 2>(a, st) : launch_conv<__nv_bfloat16, 1>(a, st);
   if (a->dtype == NX_F32) return v2 ? launch_conv<float, 2>(a, st) : launch_conv<float, 1>(a, st);
   return -1;
+}
+
+extern "C" int nx_conv_rope_append(const NxConvRopeArgs* a, nx_stream_t stream) {
+  if (a == nullptr || !conv_ok(a->conv) || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads) return -1;
+  if (a->dim <= 0 || a->vdim <= 0 || ((a->dim | a->vdim) & 3) || a->rot_dims < 0 || (a->rot_dims & 1) || a->rot_dims > a->dim) return -1;
+  if (a->conv.channels != a->heads * a->dim + a->kv_heads * (a->dim + a->vdim) || ((a->conv.ldx | a->conv.ldy) & 3)) return -1;
+  if (a->mix != nullptr && a->first == nullptr) return -1;
+  for (const void* p : {a->conv.x, static_cast<const void*>(a->conv.y), static_cast<const void*>(a->k_cache),
+                        static_cast<const void*>(a->v_cache), static_cast<const void*>(a->first)})
+    if (reinterpret_cast<uintptr_t>(p) & 15) return -1;
+  if (a->conv.seg.count <= 0 || a->conv.seg.max_len <= 0) return 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (a->conv.dtype == NX_BF16)
+    return a->conv.taps <= 4 ? launch_conv_rope<__nv_bfloat16, 4>(a, st) : launch_conv_rope<__nv_bfloat16, 2>(a, st);
+  if (a->conv.dtype == NX_F32) return launch_conv_rope<float, 2>(a, st);
+  return -1;
+}
+
+extern "C" int nx_decay_gate(const void* a, int64_t lda, const float* w, const float* bias, float* out, int64_t ldo, int rows,
+                             int cols, int rank, float tau, int dtype, nx_stream_t stream) {
+  if (cols <= 0 || rank <= 0 || !(tau > 0.0f) || lda < rank || ldo < cols) return -1;
+  if (rows <= 0) return 0;
+  if ((rows + kDecayRows - 1) / kDecayRows > 65535) return -1;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const dim3 grid((cols + kDecayCols - 1) / kDecayCols, (rows + kDecayRows - 1) / kDecayRows);
+  const float mul = 1.4426950408889634f / tau;
+  if (dtype == NX_BF16)
+    decay_gate_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(static_cast<const __nv_bfloat16*>(a), lda, w, bias, out, ldo, rows, cols,
+                                                           rank, mul);
+  else if (dtype == NX_F32)
+    decay_gate_kernel<float><<<grid, 256, 0, st>>>(static_cast<const float*>(a), lda, w, bias, out, ldo, rows, cols, rank, mul);
+  else
+    return -1;
+  return launch_status();
 }
 
 extern "C" int nx_gated_norm(const NxGatedNormArgs* a, nx_stream_t stream) {
@@ -633,17 +785,18 @@ extern "C" int nx_token_side_gate(const float* a, int64_t lda, const int32_t* to
   return launch_status();
 }
 
-extern "C" int nx_silu_mul(const void* h, int64_t ldh, void* out, int64_t ldo, int rows, int half, int dtype,
-                           nx_stream_t stream) {
-  if (half <= 0) return -1;
+extern "C" int nx_glu(const void* h, int64_t ldh, void* out, int64_t ldo, int rows, int half, int interleaved, NxGlu glu,
+                      int dtype, nx_stream_t stream) {
+  if (half <= 0 || glu.kind < NX_GLU_SILU || glu.kind > NX_GLU_CLAMP || (interleaved && half % 8)) return -1;
   if (rows <= 0) return 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const bool vec = half % 8 == 0 && ldh % 8 == 0 && ldo % 8 == 0;
+  const bool vec = half % 8 == 0 && ldh % 8 == 0 && ldo % 8 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(h) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
   for (int r0 = 0; r0 < rows; r0 += 65535) {
     const int n = std::min(65535, rows - r0);
     dim3 grid((half / (vec ? 8 : 1) + 127) / 128, n);
 #define NX_SM(T_, V_) \
-  silu_mul_kernel<T_, V_><<<grid, 128, 0, st>>>((const T_*)h + r0 * ldh, ldh, (T_*)out + r0 * ldo, ldo, half)
+  glu_kernel<T_, V_><<<grid, 128, 0, st>>>((const T_*)h + r0 * ldh, ldh, (T_*)out + r0 * ldo, ldo, half, interleaved, glu)
     if (dtype == NX_BF16) { if (vec) NX_SM(__nv_bfloat16, 8); else NX_SM(__nv_bfloat16, 1); }
     else if (dtype == NX_F32) { if (vec) NX_SM(float, 8); else NX_SM(float, 1); }
     else return -1;
@@ -652,10 +805,15 @@ extern "C" int nx_silu_mul(const void* h, int64_t ldh, void* out, int64_t ldo, i
   return launch_status();
 }
 
-extern "C" int nx_softcap(float* x, int64_t ld, int rows, int cols, float cap, nx_stream_t stream) {
-  if (cap <= 0.0f || rows > 65535) return -1;
+extern "C" int nx_silu_mul(const void* h, int64_t ldh, void* out, int64_t ldo, int rows, int half, int dtype,
+                           nx_stream_t stream) {
+  return nx_glu(h, ldh, out, ldo, rows, half, 0, NxGlu{NX_GLU_SILU, 0.0f, 0.0f, 0.0f}, dtype, stream);
+}
+
+extern "C" int nx_softcap(float* x, int64_t ld, int rows, int cols, float cap, float scale, nx_stream_t stream) {
+  if (cap < 0.0f || rows > 65535) return -1;
   if (rows <= 0 || cols <= 0) return 0;
   dim3 grid((cols + 255) / 256, rows);
-  softcap_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(x, ld, cols, cap);
+  softcap_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(x, ld, cols, cap, scale);
   return launch_status();
 }

@@ -5,8 +5,9 @@
 // kernels (which also serve expert parallelism over peer memory); the expert FFN itself is a strided
 // batched tcgen05 GEMM over the padded buffers.
 // Parity: src/moe/moe.cpp (router, capacity, permutation) of the reference, which runs on the CPU.
-// Experts that a table picks by token id need no router: one launch sorts a step's assignments for every layer, and the
-// serving forms of the expert products (few rows per expert; FP32) live here too.
+// Serving: experts that a table picks by token id need no router, one launch sorts a step's assignments for every layer; a
+// sigmoid router with a correction and groups of experts picks and sorts per layer.  The serving forms of the expert products
+// (few rows per expert; FP32) live here too.
 #include "common.cuh"
 #include "mixer_common.cuh"
 #include "nx_api_moe.h"
@@ -237,6 +238,196 @@ __global__ void __launch_bounds__(1024) moe_table_route_kernel(const __grid_cons
 }
 
 // ------------------------------------------------------------------------------------------------
+// experts by a sigmoid router
+// ------------------------------------------------------------------------------------------------
+// One warp picks the experts of one row: lane j < top returns the j-th expert and its weight.  s: 2 * experts floats of the warp.
+__device__ __forceinline__ void pick_experts(const NxGateRouteArgs& a, int row, float* s, int& expert, float& weight) {
+  const int lane = threadIdx.x & 31, E = a.experts;
+  const float* z = a.logits + row * a.ld;
+  float* g = s + E;
+  __syncwarp();
+  for (int e = lane; e < E; e += 32) s[e] = sigmoid_exact(z[e]) + a.correction[e];
+  __syncwarp();
+  if (a.n_groups > 1 && a.keep < a.n_groups) {
+    const int size = E / a.n_groups;
+    for (int i = lane; i < a.n_groups; i += 32) {
+      float first = -INFINITY, second = -INFINITY;
+      for (int e = i * size; e < (i + 1) * size; ++e) {
+        second = fmaxf(second, fminf(first, s[e]));
+        first = fmaxf(first, s[e]);
+      }
+      g[i] = size > 1 ? first + second : first;
+    }
+    __syncwarp();
+    for (int i = lane; i < a.n_groups; i += 32) {
+      int better = 0;
+      for (int o = 0; o < a.n_groups; ++o) better += g[o] > g[i] || (g[o] == g[i] && o < i) ? 1 : 0;
+      if (better >= a.keep)
+        for (int e = i * size; e < (i + 1) * size; ++e) s[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  int mine = 0;
+  for (int j = 0; j < a.top; ++j) {
+    float best = -INFINITY;
+    int be = 0x7fffffff;
+    for (int e = lane; e < E; e += 32)
+      if (s[e] > best) {
+        best = s[e];
+        be = e;
+      }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+      if (ob > best || (ob == best && oe < be)) {
+        best = ob;
+        be = oe;
+      }
+    }
+    if (be >= E) be = j;                       // only where scores are not numbers
+    if (lane == j) mine = be;
+    if (lane == (be & 31)) s[be] = -INFINITY;
+    __syncwarp();
+  }
+  const float w = lane < a.top ? sigmoid_exact(z[mine]) : 0.0f;
+  expert = mine;
+  weight = w / (warp_sum(w) + 1e-20f);
+}
+
+// first[e] = slots before expert e, every expert's share rounded up to `align`; returns the total.  All threads of the block.
+__device__ int expert_starts(const int32_t* count, int experts, int align, int* first) {
+  __shared__ int s_warp[32], s_total;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  int base = 0;
+  for (int e0 = 0; e0 < experts; e0 += blockDim.x) {
+    const int e = e0 + tid, padded = e < experts ? (count[e] + align - 1) / align * align : 0;
+    int incl = padded;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, incl, o);
+      if (lane >= o) incl += v;
+    }
+    if (lane == 31) s_warp[warp] = incl;
+    __syncthreads();
+    int before = base;
+    for (int w = 0; w < warp; ++w) before += s_warp[w];
+    if (e < experts) first[e] = before + incl - padded;
+    if (tid == static_cast<int>(blockDim.x) - 1) s_total = before + incl;
+    __syncthreads();
+    base = s_total;
+  }
+  return base;
+}
+// start, groups and the empty slots, by the threads of one block
+__device__ void expert_tables(const NxGateRouteArgs& a, const int32_t* count, const int* first, int total) {
+  for (int e = threadIdx.x; e < a.experts; e += blockDim.x) {
+    const int n = count[e], padded = (n + a.align - 1) / a.align * a.align;
+    a.start[e] = first[e];
+    for (int i = first[e] / a.align; i < (first[e] + padded) / a.align; ++i) a.groups[i] = e;
+    for (int i = first[e] + n; i < first[e] + padded; ++i) a.rows[i] = -1;
+  }
+  for (int i = total / a.align + threadIdx.x; i < a.max_slots / a.align; i += blockDim.x) a.groups[i] = -1;
+  for (int i = total + threadIdx.x; i < a.max_slots; i += blockDim.x) a.rows[i] = -1;
+}
+
+// few rows: everything in one block
+__global__ void __launch_bounds__(1024) gate_route_small_kernel(const NxGateRouteArgs a) {
+  extern __shared__ float s_score[];           // [warps][2 * experts], then int [2 * experts]: counts, starts
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5, E = a.experts;
+  int* s_cnt = reinterpret_cast<int*>(s_score + warps * 2 * E);
+  int* s_first = s_cnt + E;
+  for (int e = threadIdx.x; e < E; e += blockDim.x) s_cnt[e] = 0;
+  __syncthreads();
+  for (int r = warp; r < a.n; r += warps) {
+    int e;
+    float w;
+    pick_experts(a, r, s_score + warp * 2 * E, e, w);
+    if (lane < a.top) {
+      a.expert[r * a.top + lane] = e;
+      a.weight[r * a.top + lane] = w;
+      a.slots[r * a.top + lane] = atomicAdd(&s_cnt[e], 1);     // place inside the expert; read again by this thread
+    }
+  }
+  __syncthreads();
+  const int total = expert_starts(s_cnt, E, a.align, s_first);
+  __syncthreads();
+  expert_tables(a, s_cnt, s_first, total);
+  for (int e = threadIdx.x; e < E; e += blockDim.x) a.count[e] = s_cnt[e];
+  for (int r = warp; r < a.n; r += warps)
+    if (lane < a.top) {
+      const int s = s_first[a.expert[r * a.top + lane]] + a.slots[r * a.top + lane];
+      a.slots[r * a.top + lane] = s;
+      a.rows[s] = r;
+    }
+}
+
+constexpr int kPickRows = 32;                  // rows per block, 8 warps
+__global__ void __launch_bounds__(256) gate_pick_kernel(const NxGateRouteArgs a) {
+  extern __shared__ float s_score[];           // [8][2 * experts], then int [experts]: counts, then the block's first places
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, E = a.experts;
+  int* s_cnt = reinterpret_cast<int*>(s_score + 8 * 2 * E);
+  for (int e = threadIdx.x; e < E; e += 256) s_cnt[e] = 0;
+  __syncthreads();
+  int expert[kPickRows / 8], place[kPickRows / 8];
+#pragma unroll
+  for (int i = 0; i < kPickRows / 8; ++i) {
+    const int r = blockIdx.x * kPickRows + i * 8 + warp;
+    expert[i] = -1;
+    if (r >= a.n) continue;
+    float w;
+    pick_experts(a, r, s_score + warp * 2 * E, expert[i], w);
+    if (lane < a.top) {
+      a.expert[r * a.top + lane] = expert[i];
+      a.weight[r * a.top + lane] = w;
+      place[i] = atomicAdd(&s_cnt[expert[i]], 1);
+    }
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += 256) {
+    const int n = s_cnt[e];
+    s_cnt[e] = n > 0 ? atomicAdd(&a.count[e], n) : 0;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < kPickRows / 8; ++i) {
+    const int r = blockIdx.x * kPickRows + i * 8 + warp;
+    if (expert[i] >= 0 && lane < a.top) a.slots[r * a.top + lane] = s_cnt[expert[i]] + place[i];
+  }
+}
+
+// a warp per row: places inside experts become slots, the row is copied to them; block 0 writes the tables
+__global__ void __launch_bounds__(256) gate_place_kernel(const NxGateRouteArgs a) {
+  extern __shared__ int s_first[];
+  const int total = expert_starts(a.count, a.experts, a.align, s_first);
+  __syncthreads();
+  if (blockIdx.x == 0) expert_tables(a, a.count, s_first, total);
+  const int lane = threadIdx.x & 31, chunks = a.row_bytes / 16;
+  for (int r = blockIdx.x * 8 + (threadIdx.x >> 5); r < a.n; r += gridDim.x * 8) {
+    int slot = 0;
+    if (lane < a.top) {
+      slot = s_first[a.expert[r * a.top + lane]] + a.slots[r * a.top + lane];
+      a.slots[r * a.top + lane] = slot;
+      a.rows[slot] = r;
+    }
+    if (a.by_slot == nullptr) continue;
+    const uint4* src = static_cast<const uint4*>(a.h) + static_cast<int64_t>(r) * chunks;
+    for (int c0 = 0; c0 < chunks; c0 += 128) {
+      uint4 v[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+        if (c0 + u * 32 + lane < chunks) v[u] = __ldg(src + c0 + u * 32 + lane);
+      for (int j = 0; j < a.top; ++j) {
+        uint4* dst = static_cast<uint4*>(a.by_slot) + static_cast<int64_t>(__shfl_sync(0xffffffffu, slot, j)) * chunks;
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+          if (c0 + u * 32 + lane < chunks) dst[c0 + u * 32 + lane] = v[u];
+      }
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
 // product with one weight matrix per group (expert, head), few rows: the weights stream through registers once for up to
 // 8 NT rows.  A thread's 16-byte load covers eight neighbours along K; the sum over K may take them in any order as long as
 // both operands agree, so each load is two k-steps of the tensor-core tile as it is.  A block has four warps: 4 / KS tiles of
@@ -297,6 +488,18 @@ __device__ __forceinline__ void group_rows(const NxExpertGemmArgs& a, int group,
         for (int e = 0; e < 4; ++e) acc[i][e] += s_acc[((warp + p) * NT * 4 + i * 4 + e) * 32 + lane];
   }
   __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + group * a.group_out;
+  if (a.gated) {                       // the tile's rows are eight gates and the eight values that belong to them
+    if (!in1) return;
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int s = i * 8 + t * 2 + e;
+        if (s < cnt)
+          out[static_cast<int64_t>(first + s) * a.ldo + n0 / 2 + g] = __float2bfloat16_rn(glu_apply<false>(a.glu, acc[i][e], acc[i][e + 2]));
+      }
+    return;
+  }
 #pragma unroll
   for (int i = 0; i < NT; ++i)
 #pragma unroll
@@ -364,6 +567,7 @@ __global__ void __launch_bounds__(256) expert_f32_kernel(const NxExpertGemmArgs 
 int check_expert(const NxExpertGemmArgs* a) {
   if (a == nullptr || a->x == nullptr || a->w == nullptr || a->out == nullptr || (a->start == nullptr) != (a->count == nullptr)) return -1;
   if (a->experts <= 0 || a->n <= 0 || a->k <= 0 || (a->act != NX_ACT_NONE && a->act != NX_ACT_RELU2)) return -1;
+  if (a->gated && ((a->n & 15) || a->act != NX_ACT_NONE)) return -1;
   return 0;
 }
 }  // namespace
@@ -384,6 +588,35 @@ extern "C" int nx_moe_table_route(const NxTableRouteArgs* a, nx_stream_t stream)
   return launch_status();
 }
 
+extern "C" int nx_moe_gate_route(const NxGateRouteArgs* a, nx_stream_t stream) {
+  if (a == nullptr || a->align < 1 || a->experts < 1 || a->experts > 1024 || a->top < 1 || a->top > 32 || a->top > a->experts) return -1;
+  if (a->n_groups < 1 || a->experts % a->n_groups || a->keep < 1 || a->keep > a->n_groups || a->max_slots % a->align) return -1;
+  if (a->keep * (a->experts / a->n_groups) < a->top || a->ld < a->experts) return -1;
+  if (a->by_slot != nullptr && (a->h == nullptr || a->row_bytes <= 0 || (a->row_bytes & 15) ||
+                                ((reinterpret_cast<uintptr_t>(a->h) | reinterpret_cast<uintptr_t>(a->by_slot)) & 15)))
+    return -1;
+  if (a->n <= 0) return 0;
+  const int64_t assignments = static_cast<int64_t>(a->n) * a->top, used = assignments < a->experts ? assignments : a->experts;
+  if ((assignments + used * (a->align - 1)) / a->align * a->align > a->max_slots) return -1;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int E = a->experts;
+  if (a->n <= 256 && a->by_slot == nullptr) {
+    const int warps = std::max(4, std::min({32, (a->n + 1) / 2, 64 * 1024 / (E * 8)}));
+    const int smem = (warps + 1) * 2 * E * 4;
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(gate_route_small_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024) != cudaSuccess)
+      return -2;
+    gate_route_small_kernel<<<1, warps * 32, smem, st>>>(*a);
+    return launch_status();
+  }
+  const int smem = 17 * E * 4;
+  if (smem > 48 * 1024 && cudaFuncSetAttribute(gate_pick_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024) != cudaSuccess)
+    return -2;
+  if (cudaMemsetAsync(a->count, 0, sizeof(int32_t) * E, st) != cudaSuccess) return -2;
+  gate_pick_kernel<<<(a->n + kPickRows - 1) / kPickRows, 256, smem, st>>>(*a);
+  gate_place_kernel<<<std::min((a->n + 7) / 8, 1184), 256, E * sizeof(int), st>>>(*a);
+  return launch_status();
+}
+
 extern "C" int nx_expert_skinny(const NxExpertGemmArgs* a, nx_stream_t stream) {
   if (check_expert(a) || (a->k & 7) || (a->ldx & 7) || (a->ldw & 7) || (a->stride_w & 7) || (a->group_x & 7) || a->experts > 65535)
     return -1;
@@ -400,7 +633,7 @@ extern "C" int nx_expert_skinny(const NxExpertGemmArgs* a, nx_stream_t stream) {
 }
 
 extern "C" int nx_expert_f32(const NxExpertGemmArgs* a, nx_stream_t stream) {
-  if (check_expert(a) || a->start == nullptr || a->groups == nullptr || a->align != 32 || a->tiles < 0 || a->tiles > 65535) return -1;
+  if (check_expert(a) || a->start == nullptr || a->groups == nullptr || a->align != 32 || a->tiles < 0 || a->tiles > 65535 || a->gated) return -1;
   if (a->tiles == 0) return 0;
   expert_f32_kernel<<<dim3((a->n + 63) / 64, a->tiles), 256, 0, static_cast<cudaStream_t>(stream)>>>(*a);
   return launch_status();

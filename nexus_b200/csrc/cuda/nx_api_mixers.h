@@ -1,7 +1,7 @@
 // C ABI of the building blocks of decoders with heterogeneous layers: pre / post norms around a sublayer, rotary
 // embedding fused with the cache append, windowed and soft-capped paged attention for any head sizes, the short causal
-// convolution with its carried tail, the Mamba-2 (SSD) and gated-delta-rule recurrences with their carried FP32 state,
-// gated norms, the per-layer token input and soft-capping of logits.
+// convolution with its carried tail, the Mamba-2 (SSD), gated-delta-rule and gated-linear-attention recurrences with their
+// carried FP32 state, gated norms, gated activations, the per-layer token input and soft-capping of logits.
 //
 // Activations are BF16 or FP32 (`dtype`: NX_BF16 / NX_F32); weights of norms, decays and convolutions are FP32.
 //
@@ -31,15 +31,15 @@ typedef struct NxResidualNormArgs {
   const int32_t* tokens;   // with `table`: x = embed_scale * table[tokens[row]]
   const void* table;       // [vocab, cols] dtype, may be null
   const void* y;           // [rows, ldy] sublayer output, may be null: x += res_mult * rms(y) * w_post
-  const float* w_post;
+  const float* w_post;     // may be null: x += res_mult * y
   const float* w_next;     // may be null; else h = rms(x) * w_next
   void* h;                 // [rows, ldh]; columns cols..ldh are zeroed
   void* x_cast;            // [rows, ldh], may be null: x in the activation dtype
   int64_t ldy, ldh;
   int32_t rows, cols, dtype;
   float eps, embed_scale, res_mult;
-  // Sublayer output of a layer of experts, may be null: expert_scale * sum_j experts[expert_slots[row * top + j]], plus
-  // y_gate[row] * y[row] when `y` is given too (y_gate null: plain y).
+  // Sublayer output of a layer of experts, may be null: expert_scale * sum_j w_j experts[expert_slots[row * top + j]] with w_j =
+  // expert_weights[row * top + j] (null: 1), plus y_gate[row] * y[row] when `y` is given too (y_gate null: plain y).
   const void* experts;     // [slots, ld_experts]
   const int32_t* expert_slots;
   const float* y_gate;
@@ -52,6 +52,7 @@ typedef struct NxResidualNormArgs {
   // copies of the x_cast row at scatter[scatter_slots[row * top + j]], may be null (pitch ldh)
   void* scatter;
   const int32_t* scatter_slots;
+  const float* expert_weights;
 } NxResidualNormArgs;
 int nx_residual_norm(const NxResidualNormArgs* args, nx_stream_t stream);
 
@@ -71,7 +72,7 @@ int nx_rope_append(const NxRopeAppendArgs* args, nx_stream_t stream);
 
 // What lies between the down projections of latent attention and its cache: the query latent and the key / value latent
 // are normed, the shared key part is rotated, latent and key part go to the cache (and to `lat`), the output gate's
-// sigmoid is taken.
+// sigmoid is taken.  q_rank 0: queries have no latent; gate null: no output gate.
 typedef struct NxLatentPrepArgs {
   const void* proj;        // [rows, ld]; the parts of a row start at q_off, c_off, r_off, g_off
   int64_t ld;
@@ -111,6 +112,23 @@ typedef struct NxConvArgs {
   NxSegments seg;
 } NxConvArgs;
 int nx_conv_silu(const NxConvArgs* args, nx_stream_t stream);
+
+// The convolution without an activation over the packed projections q (heads * dim) | k (kv_heads * dim) | v (kv_heads *
+// vdim), then what attention needs of them: pairs of neighbouring columns (2 i, 2 i + 1) of q and k rotate for i < rot_dims / 2,
+// v becomes (1 - mix) v + mix first, k and v go to the cache and q (with store_kv also k and v) to y.  dim and vdim are
+// multiples of 4.
+typedef struct NxConvRopeArgs {
+  NxConvArgs conv;         // channels = heads * dim + kv_heads * (dim + vdim)
+  int32_t heads, kv_heads, dim, vdim, rot_dims, store_kv;
+  const int32_t* slots;    // cache slot per row, negative: nothing is appended
+  const float* cos_t;      // [max_pos, rot_dims / 2]
+  const float* sin_t;
+  void* k_cache;           // [slots, kv_heads, dim]
+  void* v_cache;           // [slots, kv_heads, vdim]
+  const float* mix;        // one value, may be null
+  void* first;             // [rows, kv_heads * vdim]: read with `mix`, otherwise written; may be null without `mix`
+} NxConvRopeArgs;
+int nx_conv_rope_append(const NxConvRopeArgs* args, nx_stream_t stream);
 
 // Mamba-2: S = exp(-exp(A_log) dt) S + dt B x^T,  y = S^T C + D x,  dt = softplus(dt_raw + dt_bias).
 typedef struct NxSsdArgs {
@@ -158,6 +176,33 @@ int nx_delta_step(const NxDeltaArgs* args, nx_stream_t stream);
 int64_t nx_delta_scratch_bytes(int heads, int segments, int max_len);
 int nx_delta_chunk(const NxDeltaArgs* args, nx_stream_t stream);
 
+// Gated linear attention: S = diag(2^a) S + k v^T,  o = S^T (q_scale q), a decay per key channel.
+typedef struct NxGlaArgs {
+  const void* q;           // [rows, ld]: heads * dim
+  const void* k;           // [rows, ld]: heads * dim
+  const void* v;           // [rows, ld]: heads * vdim
+  const float* decay;      // [rows, ld_decay]: log2 of the decays (<= 0), heads * dim
+  void* o;                 // [rows, ldo]: heads * vdim
+  float* state;            // [slots, heads, dim, vdim]
+  int64_t ld, ld_decay, ldo;
+  int32_t heads, dim, vdim, dtype;
+  float q_scale;
+  NxSegments seg;
+  // Chunked form only: spans of a segment that run at the same time (as in NxSsdArgs); part_state [seg.count, parts, heads, dim,
+  // vdim], part_decay [seg.count, parts, heads, dim].
+  float* part_state;
+  float* part_decay;
+  int32_t parts, span;
+} NxGlaArgs;
+// token by token, any sizes and both dtypes
+int nx_gla_step(const NxGlaArgs* args, nx_stream_t stream);
+// chunks of 64 tokens on the tensor cores, BF16 activations, dim <= 256
+int nx_gla_chunk(const NxGlaArgs* args, nx_stream_t stream);
+// out[r][c] = log2(sigmoid(z)) / tau (FP32, [rows, ldo]), z = sum_j a[r][j] w[c][j] + bias[c]: a [rows, lda] activations, w FP32
+// [cols, rank]
+int nx_decay_gate(const void* a, int64_t lda, const float* w, const float* bias, float* out, int64_t ldo, int rows, int cols,
+                  int rank, float tau, int dtype, nx_stream_t stream);
+
 // gate_first: out = rms(y * silu(z)) * w * out_scale, else out = rms(y) * w * silu(z) * out_scale; statistics over each
 // of `groups` equal parts of a row.  w has groups * group_size entries, or group_size shared by every part (w_shared).
 typedef struct NxGatedNormArgs {
@@ -177,11 +222,24 @@ int nx_token_side_gate(const float* a, int64_t lda, const int32_t* tokens, const
                        void* out, int64_t ldo, int rows, int dim, int dtype, nx_stream_t stream);
 // out[r][j] = silu(h[r][j]) * h[r][half + j], j < half
 int nx_silu_mul(const void* h, int64_t ldh, void* out, int64_t ldo, int rows, int half, int dtype, nx_stream_t stream);
-// x = cap * tanh(x / cap) in place on FP32 [rows, ld]
-int nx_softcap(float* x, int64_t ld, int rows, int cols, float cap, nx_stream_t stream);
+// Gated activations of a gate g and a value u:  NX_GLU_SILU silu(g) u,  NX_GLU_GELU gelu_tanh(g) u,
+// NX_GLU_CLAMP with g' = min(g, limit), u' = clamp(u, -limit, limit): g' sigmoid(slope g') (u' + offset).
+// half: columns of the output; g and u lie in two halves of h, or (interleaved) in turns of eight columns, gates first.
+#define NX_GLU_SILU 0
+#define NX_GLU_GELU 1
+#define NX_GLU_CLAMP 2
+typedef struct NxGlu {
+  int32_t kind;
+  float limit, slope, offset;
+} NxGlu;
+int nx_glu(const void* h, int64_t ldh, void* out, int64_t ldo, int rows, int half, int interleaved, NxGlu glu, int dtype,
+           nx_stream_t stream);
+// x = cap * tanh(scale * x / cap) in place on FP32 [rows, ld]; cap 0: x = scale * x
+int nx_softcap(float* x, int64_t ld, int rows, int cols, float cap, float scale, nx_stream_t stream);
 
 // Causal attention of packed query rows over a paged cache.  Row at position p sees keys p - window + 1 .. p (window <= 0:
-// 0 .. p); score = scale * q.k, soft-capped when softcap > 0.  The rows' own keys are in the cache already.
+// 0 .. p) and the first keep_first keys; score = scale * q.k, soft-capped when softcap > 0.  sink: a score per head (not scaled)
+// that counts in the denominator only.  The rows' own keys are in the cache already.
 typedef struct NxPagedWindowArgs {
   const void* q;           // [rows, ldq]: heads * dim
   const void* k_cache;     // [blocks * block_size, kv_heads, dim]
@@ -197,6 +255,8 @@ typedef struct NxPagedWindowArgs {
   int64_t k_pitch, v_pitch;  // elements between cache slots: kv_heads * dim and kv_heads * vdim, or the row of a latent cache,
                              // whose values are the leading columns of its keys
   const float* gate;         // [rows, heads] factor of the output, may be null
+  const float* sink;         // [heads], may be null
+  int32_t keep_first;
 } NxPagedWindowArgs;
 // one-row segments, BF16: tensor-core tiles of up to 16 query heads of a KV head against 64 keys, split over the keys
 int nx_paged_window_decode(const NxPagedWindowArgs* args, nx_stream_t stream);
@@ -244,6 +304,25 @@ typedef struct NxLatentPromptArgs {
   float scale;                                                                     // vdim <= 128: multiple of 8; scale > 0
 } NxLatentPromptArgs;
 int nx_latent_prompt(const NxLatentPromptArgs* args, nx_stream_t stream);
+
+// The same kernel on plain grouped keys and values: q [q_rows, ldq]: heads * dim; k [kv_rows, ldk]: kv_heads * dim; v [kv_rows,
+// ldv]: kv_heads * vdim; query head h reads KV head h / (heads / kv_heads).  Windows, kept first keys and sinks as in
+// NxPagedWindowArgs.  blocks as above; kept [n_blocks]: row that position 0 has among the kept keys (null: the fourth entry of
+// the block).  dim <= 128: multiple of 16; vdim <= 128: multiple of 8; scale > 0.
+typedef struct NxWindowPromptArgs {
+  const void* q;
+  const void* k;
+  const void* v;
+  void* out;               // [., ldo]: heads * vdim
+  const float* sink;       // [heads], may be null
+  const int32_t* blocks;
+  const int32_t* kept;
+  int* status;
+  int64_t ldq, ldk, ldv, ldo;
+  int32_t n_blocks, q_rows, kv_rows, heads, kv_heads, dim, vdim, window, keep_first;
+  float scale;
+} NxWindowPromptArgs;
+int nx_window_prompt(const NxWindowPromptArgs* args, nx_stream_t stream);
 // Cache rows of `segments` runs of positions into one packed buffer.  list [segments, 4]: first destination row, rows, first
 // position, sequence; `longest`: most rows of a run.
 int nx_latent_gather(const void* cache, void* dst, const int32_t* block_table, const int32_t* list, int segments, int longest,

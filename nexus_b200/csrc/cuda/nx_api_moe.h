@@ -1,6 +1,7 @@
 // C ABI of the MoE routing kernels.
 #pragma once
 #include "nx_api.h"
+#include "nx_api_mixers.h"
 
 #ifdef __cplusplus
 extern "C" {
@@ -50,7 +51,29 @@ typedef struct NxTableRouteArgs {
 } NxTableRouteArgs;
 int nx_moe_table_route(const NxTableRouteArgs* args, nx_stream_t stream);
 
+// Experts by a learned router.  A row's scores are s = sigmoid(logits), its choice scores s + correction.  With n_groups > 1 the
+// experts form equal groups of neighbours, a group's score is the sum of its two largest choice scores, and only experts of
+// the `keep` best groups can be chosen.  The `top` largest choice scores win (ties: the lower id); weight = s / (sum of the
+// chosen s + 1e-20).  The assignments are sorted as above.  With by_slot, row r of h is copied to by_slot at each of its slots.
+typedef struct NxGateRouteArgs {
+  const float* logits;       // [n, ld]
+  const float* correction;   // [experts]
+  int32_t* expert;           // [n, top]
+  float* weight;             // [n, top]
+  int32_t* slots;            // [n, top]
+  int32_t* rows;             // [max_slots]
+  int32_t* start;            // [experts]
+  int32_t* count;            // [experts]
+  int32_t* groups;           // [max_slots / align]
+  const void* h;             // [n], rows of row_bytes (a multiple of 16)
+  void* by_slot;             // [max_slots], may be null
+  int64_t ld;
+  int32_t n, experts, top, n_groups, keep, align, max_slots, row_bytes;   // experts <= 1024, top <= 32
+} NxGateRouteArgs;
+int nx_moe_gate_route(const NxGateRouteArgs* args, nx_stream_t stream);
+
 // out[slot] = act(W[e] x[row of slot]) for every slot of every expert; `rows` null: row = slot.  act: NX_ACT_NONE or RELU2.
+// gated (few rows only): the rows of W are turns of eight gates and eight values (n counts both), out has n / 2 columns.
 // start and count null: every group has slots 0..m (a matrix per head).
 typedef struct NxExpertGemmArgs {
   const void* x;           // [., ldx]
@@ -64,6 +87,8 @@ typedef struct NxExpertGemmArgs {
   int32_t experts, n, k, act, tiles, align;
   int64_t group_x, group_out;  // few rows: what a group adds to the addresses of x and out (elements)
   int32_t m;                   // few rows: most slots of a group
+  int32_t gated;
+  NxGlu glu;
 } NxExpertGemmArgs;
 // few rows per expert, BF16: the weights stream through registers once per 32 rows; k, ldx, ldw, group_x multiples of 8
 int nx_expert_skinny(const NxExpertGemmArgs* args, nx_stream_t stream);

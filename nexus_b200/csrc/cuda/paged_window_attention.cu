@@ -1,5 +1,5 @@
-// Causal attention over a paged cache for any head sizes: sliding window, score soft-capping, grouped query heads,
-// different key and value widths (see nx_api_mixers.h).  The query heads that share a KV head are packed into the rows of
+// Causal attention over a paged cache for any head sizes: sliding window, kept first keys, a sink in the denominator, score
+// soft-capping, grouped query heads, different key and value widths (see nx_api_mixers.h).  The query heads that share a KV head are packed into the rows of
 // one tensor-core tile, so a KV page is read once for all of them: 64 (token, head) rows per block in prompts, up to 16
 // heads of one token in decoding.  Scores, soft-capping and softmax are FP32; only the products take BF16 operands.
 #include "mixer_common.cuh"
@@ -37,7 +37,21 @@ struct ScoreMap {
   }
 };
 
-// One stage of keys and values into shared memory, each [kKeys][DP + 8]; keys past `last` and columns past the head size
+// The keys a block meets, numbered without the gap between the kept first ones and the window: index i is position i below
+// `kept` and position i + skip from there on.
+struct KeyRange {
+  int kept, skip, count;
+  // rows at positions pos .. last
+  __device__ __forceinline__ KeyRange(const NxPagedWindowArgs& a, int pos, int last) {
+    const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    kept = min(a.keep_first, lo);
+    skip = lo - kept;
+    count = last + 1 - skip;
+  }
+  __device__ __forceinline__ int position(int i) const { return i < kept ? i : i + skip; }
+};
+
+// One stage of keys and values into shared memory, each [kKeys][DP + 8]; keys past index `last` and columns past the head size
 // become zeros.
 struct KvSource {
   const __nv_bfloat16 *k, *v;
@@ -62,13 +76,13 @@ __device__ __forceinline__ void copy8(__nv_bfloat16* d, const __nv_bfloat16* s, 
   }
 }
 template <int DP>
-__device__ __forceinline__ void stage_kv(__nv_bfloat16* dst, const KvSource& src, int k0, int last) {
+__device__ __forceinline__ void stage_kv(__nv_bfloat16* dst, const KvSource& src, const KeyRange& keys, int k0, int last) {
   constexpr int CH = DP / 8, LD = DP + 8;
   for (int i = threadIdx.x; i < kKeys * CH; i += blockDim.x) {
     const int key = i / CH, c = (i % CH) * 8, j = k0 + key;
     __nv_bfloat16 *dk = dst + key * LD + c, *dv = dk + kKeys * LD;
     const bool in = j <= last;
-    const int64_t slot = in ? src.slot(j) : 0;
+    const int64_t slot = in ? src.slot(keys.position(j)) : 0;
     if (in && c < src.dim) copy8(dk, src.k + slot * src.k_pitch, c, src.dim);
     else *reinterpret_cast<uint4*>(dk) = make_uint4(0u, 0u, 0u, 0u);
     if (in && c < src.vdim) copy8(dv, src.v + slot * src.v_pitch, c, src.vdim);
@@ -105,13 +119,14 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
   const int nt = min(tq, a.seg.len[sg] - t0);
   const int pos0 = a.seg.pos[sg] + t0;
   const int64_t row0 = static_cast<int64_t>(a.seg.row0[sg]) + t0;
-  const int first = a.window > 0 ? max(0, pos0 - a.window + 1) : 0, last = pos0 + nt - 1;
+  const KeyRange keys(a, pos0, pos0 + nt - 1);
+  const int last = keys.count - 1;
   const KvSource src(a, a.seg.seq[sg], hk);
   auto stage = [&](int k0, int s) {
-    stage_kv<DP>(sKV + (s * 2) * kKeys * LD, src, k0, last);
+    stage_kv<DP>(sKV + (s * 2) * kKeys * LD, src, keys, k0, last);
     cp_async_commit();
   };
-  stage(first, 0);
+  stage(0, 0);
   {
     const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q);
     const float sign = a.scale < 0.0f ? -1.0f : 1.0f;      // the score map wants a positive factor
@@ -145,7 +160,7 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[i][e] = 0.0f;
   int s = 0;
-  for (int k0 = first; k0 <= last; k0 += kKeys, s ^= 1) {
+  for (int k0 = 0; k0 <= last; k0 += kKeys, s ^= 1) {
     if (k0 + kKeys <= last) {
       stage(k0 + kKeys, s ^ 1);
       cp_async_wait<1>();
@@ -173,15 +188,16 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
       }
     }
     // every row of this warp sees the whole stage, unless it reaches past a row's own position or before its window
-    const bool edge = warp_lo < 0 || k0 + kKeys - 1 > warp_lo || (a.window > 0 && k0 <= warp_hi - a.window);
+    const int p0 = keys.position(k0);
+    const bool edge = warp_lo < 0 || keys.position(k0 + kKeys - 1) > warp_lo || (a.window > 0 && p0 <= warp_hi - a.window);
     float tmax[2] = {-INFINITY, -INFINITY};
     if (edge) {
 #pragma unroll
       for (int n = 0; n < 8; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int j = k0 + n * 8 + (lane & 3) * 2 + (e & 1), qp = qpos[e >> 1];
-          if (!(j <= qp && (a.window <= 0 || j > qp - a.window))) sc[n][e] = -INFINITY;
+          const int j = keys.position(k0 + n * 8 + (lane & 3) * 2 + (e & 1)), qp = qpos[e >> 1];
+          if (!(j <= qp && (a.window <= 0 || j > qp - a.window || j < a.keep_first))) sc[n][e] = -INFINITY;
         }
     }
 #pragma unroll
@@ -233,6 +249,7 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
     if (qpos[i] < 0) continue;
     const int m = warp * 16 + i * 8 + (lane >> 2);
     const float g = a.gate != nullptr ? a.gate[(row0 + m / rt) * a.heads + h0 + m % rt] : 1.0f;
+    if (a.sink != nullptr) sum[i] += exp2f(a.sink[h0 + m % rt] * kLog2e - mx[i]);
     const float inv = a.out_scale * g / sum[i];
     __nv_bfloat16* op = out + (row0 + m / rt) * a.ldo + static_cast<int64_t>(h0 + m % rt) * a.vdim;
 #pragma unroll
@@ -264,11 +281,11 @@ paged_decode_mma_kernel(const NxPagedWindowArgs a, int head_tiles) {
   const int pos = a.seg.pos[sg];
   const int64_t row = a.seg.row0[sg];
   const KvSource src(a, a.seg.seq[sg], hk);
-  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-  const int per = ((pos - lo + kKeys) / kKeys + a.splits - 1) / a.splits * kKeys;
-  const int first = lo + static_cast<int>(blockIdx.z) * per, last = min(pos, first + per - 1);
+  const KeyRange keys(a, pos, pos);
+  const int per = ((keys.count + kKeys - 1) / kKeys + a.splits - 1) / a.splits * kKeys;
+  const int first = static_cast<int>(blockIdx.z) * per, last = min(keys.count, first + per) - 1;
   auto stage = [&](int k0, int s) {
-    stage_kv<DP>(sKV + (s * 2) * kKeys * LD, src, k0, last);
+    stage_kv<DP>(sKV + (s * 2) * kKeys * LD, src, keys, k0, last);
     cp_async_commit();
   };
   if (first <= last) stage(first, 0);
@@ -379,6 +396,7 @@ paged_decode_mma_kernel(const NxPagedWindowArgs a, int head_tiles) {
       go += sO[(w * 16 + m) * DP + d] * f;
     }
     if (a.splits == 1) {
+      if (a.sink != nullptr) gl += exp2f(a.sink[h0 + m] * kLog2e - gm);
       const float g = a.gate != nullptr ? a.gate[row * a.heads + h0 + m] : 1.0f;
       static_cast<__nv_bfloat16*>(a.out)[row * a.ldo + static_cast<int64_t>(h0 + m) * a.vdim + d] =
           __float2bfloat16_rn(go / gl * a.out_scale * g);
@@ -408,6 +426,7 @@ __global__ void paged_decode_merge_kernel(const NxPagedWindowArgs a) {
       gl += a.part_ml[(base + s) * 2 + 1] * w;
       go += a.part_o[(base + s) * a.vdim + d] * w;
     }
+    if (a.sink != nullptr) gl += exp2f(a.sink[h] * kLog2e - gm);
     static_cast<__nv_bfloat16*>(a.out)[row * a.ldo + static_cast<int64_t>(h) * a.vdim + d] =
         __float2bfloat16_rn(go / gl * a.out_scale * g);
   }
@@ -435,12 +454,12 @@ __global__ void __launch_bounds__(128) paged_window_f32_kernel(const NxPagedWind
   float acc[kF32Cols], mx = -INFINITY, sum = 0.0f;
 #pragma unroll
   for (int c = 0; c < kF32Cols; ++c) acc[c] = 0.0f;
-  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-  for (int k0 = lo; k0 <= pos; k0 += 128) {
+  const KeyRange keys(a, pos, pos);
+  for (int k0 = 0; k0 < keys.count; k0 += 128) {
     __syncthreads();
-    const int j = k0 + tid;
     float sc = -INFINITY;
-    if (j <= pos) {
+    if (k0 + tid < keys.count) {
+      const int j = keys.position(k0 + tid);
       const int64_t slot = static_cast<int64_t>(bt[j / a.block_size]) * a.block_size + j % a.block_size;
       s_slot[tid] = slot;
       const float* k = kc + slot * a.k_pitch + hk * a.dim;
@@ -454,7 +473,7 @@ __global__ void __launch_bounds__(128) paged_window_f32_kernel(const NxPagedWind
     mx = nm;
     sP[tid] = p;
     sum = sum * alpha + block_sum(p, s_red);     // the barriers inside publish sP and s_slot
-    const int n = min(128, pos - k0 + 1);
+    const int n = min(128, keys.count - k0);
 #pragma unroll
     for (int c = 0; c < kF32Cols; ++c) {
       const int d = tid + c * 128;
@@ -466,6 +485,7 @@ __global__ void __launch_bounds__(128) paged_window_f32_kernel(const NxPagedWind
     }
   }
   const float g = a.gate != nullptr ? a.gate[row * a.heads + h] : 1.0f;
+  if (a.sink != nullptr) sum += expf(a.sink[h] - mx);
   for (int c = 0; c < kF32Cols; ++c) {
     const int d = tid + c * 128;
     if (d < a.vdim) static_cast<float*>(a.out)[row * a.ldo + static_cast<int64_t>(h) * a.vdim + d] = acc[c] / sum * (a.out_scale * g);
@@ -474,7 +494,7 @@ __global__ void __launch_bounds__(128) paged_window_f32_kernel(const NxPagedWind
 
 int check_paged(const NxPagedWindowArgs* a, int dtype) {
   if (a == nullptr || a->dtype != dtype || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads) return -1;
-  if (a->dim <= 0 || a->vdim <= 0 || a->block_size <= 0 || a->max_blocks <= 0 || a->seg.count > 65535) return -1;
+  if (a->keep_first < 0 || a->dim <= 0 || a->vdim <= 0 || a->block_size <= 0 || a->max_blocks <= 0 || a->seg.count > 65535) return -1;
   if (a->k_pitch < static_cast<int64_t>(a->kv_heads) * a->dim || a->v_pitch < static_cast<int64_t>(a->kv_heads) * a->vdim) return -1;
   return 0;
 }

@@ -1,5 +1,5 @@
-// Token-by-token forms of the two recurrences (see nx_api_mixers.h): Mamba-2 state-space duality and the gated delta
-// rule.  A block owns one tile of value columns of one head of one segment: the columns of the state are independent of
+// Token-by-token forms of the recurrences (see nx_api_mixers.h): Mamba-2 state-space duality, the gated delta rule and gated
+// linear attention.  A block owns one tile of value columns of one head of one segment: the columns of the state are independent of
 // one another, so the tile is staged in shared memory once, every token of the segment is applied to it in FP32, and it
 // is written back.  This is the decode path (one token: the kernel streams the state once each way), the path of short
 // prompt portions, and the FP32 path of any length.
@@ -170,6 +170,61 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const NxDeltaA
   store_state(sS, gS, D, width, Dv, vec);
 }
 
+// grid (heads, column tiles, segments); shared: state [D][tile] | k [D] | q [D] | decay [D] | partial sums [row groups][tile]
+template <typename T>
+__global__ void __launch_bounds__(kStepThreads) gla_step_kernel(const NxGlaArgs a, int tile) {
+  extern __shared__ __align__(16) float smem[];
+  const int h = blockIdx.x, v0 = blockIdx.y * tile, sg = blockIdx.z;
+  const int len = a.seg.len[sg];
+  if (len <= 0) return;
+  const int D = a.dim, Dv = a.vdim, width = min(tile, Dv - v0);
+  float* sS = smem;
+  float* sK = sS + D * tile;
+  float* sQ = sK + D;
+  float* sA = sQ + D;
+  float* sR = sA + D;
+  const int ng = kStepThreads / width;
+  const int tx = threadIdx.x % width, ty = threadIdx.x / width;
+  const bool active = ty < ng;
+  const bool vec = (Dv & 3) == 0 && (width & 3) == 0 && (v0 & 3) == 0;
+  float* gS = a.state + ((static_cast<int64_t>(a.seg.seq[sg]) * a.heads + h) * D) * Dv + v0;
+  const bool zero = a.seg.pos[sg] == 0;
+  load_state(sS, gS, D, width, Dv, vec, zero);
+  const int64_t row0 = a.seg.row0[sg];
+  const T* q = static_cast<const T*>(a.q) + row0 * a.ld + static_cast<int64_t>(h) * D;
+  const T* k = static_cast<const T*>(a.k) + row0 * a.ld + static_cast<int64_t>(h) * D;
+  const T* v = static_cast<const T*>(a.v) + row0 * a.ld + static_cast<int64_t>(h) * Dv + v0;
+  const float* dec = a.decay + row0 * a.ld_decay + static_cast<int64_t>(h) * D;
+  T* o = static_cast<T*>(a.o) + row0 * a.ldo + static_cast<int64_t>(h) * Dv + v0;
+  if (vec && !zero) cp_async_wait<0>();
+  for (int t = 0; t < len; ++t, q += a.ld, k += a.ld, v += a.ld, dec += a.ld_decay, o += a.ldo) {
+    for (int d = threadIdx.x; d < D; d += kStepThreads) {
+      sK[d] = Num<T>::load(k + d);
+      sQ[d] = a.q_scale * Num<T>::load(q + d);
+      sA[d] = exp2f(dec[d]);
+    }
+    const float x = active ? Num<T>::load(v + tx) : 0.0f;
+    __syncthreads();
+    float acc = 0.0f;
+    if (active) {
+#pragma unroll 4
+      for (int d = ty; d < D; d += ng) {
+        const float s = sS[d * width + tx] * sA[d] + sK[d] * x;
+        sS[d * width + tx] = s;
+        acc += s * sQ[d];
+      }
+      sR[ty * width + tx] = acc;
+    }
+    __syncthreads();
+    if (ty == 0) {
+      for (int i = 1; i < ng; ++i) acc += sR[i * width + tx];
+      Num<T>::store(o + tx, acc);
+    }
+  }
+  __syncthreads();
+  store_state(sS, gS, D, width, Dv, vec);
+}
+
 int pick_tile(int cols, int rows, size_t extra_bytes) {
   // a tile of 32 columns keeps many blocks resident; wider only for wide heads of few rows
   int tile = std::min(cols, 32);
@@ -221,6 +276,27 @@ extern "C" int nx_delta_step(const NxDeltaArgs* a, nx_stream_t stream) {
   } else if (a->dtype == NX_F32) {
     if (set_smem(delta_step_kernel<float>, smem)) return -2;
     delta_step_kernel<float><<<grid, kStepThreads, smem, st>>>(*a, tile);
+  } else {
+    return -1;
+  }
+  return launch_status();
+}
+
+extern "C" int nx_gla_step(const NxGlaArgs* a, nx_stream_t stream) {
+  if (a == nullptr || a->heads <= 0 || a->dim <= 0 || a->vdim <= 0) return -1;
+  if (a->seg.count <= 0) return 0;
+  if (a->seg.count > 65535) return -1;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int tile = pick_tile(a->vdim, a->dim, static_cast<size_t>(3 * a->dim + kStepThreads) * 4);
+  const size_t smem = (static_cast<size_t>(a->dim) * tile + 3 * a->dim + kStepThreads) * sizeof(float);
+  if (smem > 220 * 1024) return -1;
+  dim3 grid(a->heads, (a->vdim + tile - 1) / tile, a->seg.count);
+  if (a->dtype == NX_BF16) {
+    if (set_smem(gla_step_kernel<__nv_bfloat16>, smem)) return -2;
+    gla_step_kernel<__nv_bfloat16><<<grid, kStepThreads, smem, st>>>(*a, tile);
+  } else if (a->dtype == NX_F32) {
+    if (set_smem(gla_step_kernel<float>, smem)) return -2;
+    gla_step_kernel<float><<<grid, kStepThreads, smem, st>>>(*a, tile);
   } else {
     return -1;
   }

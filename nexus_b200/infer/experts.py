@@ -1,9 +1,13 @@
-"""Feed-forward of table-routed experts (`lm.hybrid.ExpertsSpec`) on the engine.
+"""Feed-forward of experts (`lm.hybrid.ExpertsSpec`) on the engine.
 
-Which experts a token uses depends on nothing but its id, so one launch at the start of a step sorts the assignments of
-every layer.  Up to 32 rows per expert the weights are streamed once past all of an expert's rows; above, the residual kernel
-writes every row to its slots and the tcgen05 GEMM takes the experts as groups of row tiles.  The kernel that adds the
-sublayer's output to the residual stream sums a token's experts and its gated shared expert on the way."""
+Where a table picks a token's experts by its id, one launch at the start of a step sorts the assignments of every layer; a
+learned router picks and sorts in its layer.  Up to 32 rows per expert the weights are streamed once past all of an expert's
+rows; above, the residual kernel (or the routing kernel) writes every row to its slots and the tcgen05 GEMM takes the experts as
+groups of row tiles.  The kernel that adds the sublayer's output to the residual stream sums a token's experts, with the
+router's weights, and its gated shared expert on the way.
+
+Gated experts keep W_gate and W_up as one matrix in turns of eight rows, so that the few-rows product has a unit's gate and value
+in one thread."""
 from __future__ import annotations
 
 from typing import List, Optional
@@ -28,9 +32,18 @@ def _stack(parts) -> torch.Tensor:
 
 def load(engine, f: ExpertsSpec, get) -> dict:
     """``get(name)``: the feed-forward's tensors."""
-    out = {"table": get("table").to(engine.dev, torch.int32).contiguous()}
+    out = {}
+    if f.router is None:
+        out["table"] = get("table").to(engine.dev, torch.int32).contiguous()
+    else:
+        out["router"], _ = engine._pack([get("router")])
+        out["correction"] = engine._f32(get("correction"))
     for name in ("up", "down"):
-        out[name] = _stack([get(f"e{e}.{name}") for e in range(f.experts)]).to(engine.dev, engine.adt)
+        w = _stack([get(f"e{e}.{name}") for e in range(f.experts)])
+        if f.glu is not None and name == "up":
+            both = torch.stack([_stack([get(f"e{e}.gate") for e in range(f.experts)]), w], 1)       # [experts, 2, rows, columns]
+            w = both.view(f.experts, 2, -1, 8, w.shape[2]).transpose(1, 2).reshape(f.experts, -1, w.shape[2])
+        out[name] = w.to(engine.dev, engine.adt).contiguous()
         engine.weight_nbytes += out[name].numel() * out[name].element_size()
     if f.shared:
         out["shared_up"], _ = engine._pack([get("shared.up")])
@@ -49,12 +62,12 @@ def alignment(engine, f: ExpertsSpec, rows: int) -> int:
 
 
 def route(engine, tok) -> List[Optional[object]]:
-    """A `Route` for every layer that has experts."""
+    """A `Route` for every layer whose experts a table picks."""
     from ..ops import _experts as X
     routes: List[Optional[object]] = [None] * engine.L
     by_align = {}
     for i, layer in enumerate(engine.model.layers):
-        if layer.experts is not None:
+        if layer.experts is not None and layer.experts.router is None:
             by_align.setdefault(alignment(engine, layer.experts, tok.shape[0]), []).append(i)
     for align, which in by_align.items():
         got = X.table_route(tok, [(engine.layers[i]["ff"]["table"], engine.model.layers[i].experts.experts) for i in which], align)
@@ -63,12 +76,23 @@ def route(engine, tok) -> List[Optional[object]]:
     return routes
 
 
+def gate(engine, f: ExpertsSpec, lw: dict, h):
+    """The `Route` of the router's choices for the rows ``h``, and the rows in slot order where the GEMM wants them."""
+    from ..ops import _experts as X
+    align = alignment(engine, f, h.shape[0])
+    logits = engine._linear(h, lw["router"], out_dtype=torch.float32)
+    return X.gate_route(logits, lw["correction"], f.top, align, n_groups=f.router.groups, keep=f.router.keep,
+                        h=h if align >= 128 else None)
+
+
 def forward(engine, f: ExpertsSpec, lw: dict, r, h, sorted_h):
     """``h``: the rows of the batch; ``sorted_h``: the same in slot order (GEMM form) or None.  Returns the experts' rows in
     slot order and the shared expert's output (or None)."""
     from ..ops import _experts as X
+    from ..ops import _mixers as M
     gather = sorted_h is None
-    a = X.expert_product(h if gather else sorted_h, lw["up"], r, gather=gather, act="relu2")
+    act = {"act": "relu2"} if f.glu is None else {"gate": M.Glu(2, f.glu.limit, f.glu.slope, f.glu.offset)}
+    a = X.expert_product(h if gather else sorted_h, lw["up"], r, gather=gather, **act)
     y = X.expert_product(a, lw["down"], r, gather=False)
     if not f.shared:
         return y, None

@@ -2,7 +2,7 @@
 
 What differs from the GPT-2 family is below `Engine.forward`: the layer loop, and what a sequence owns beside its cache
 pages.  Pages exist for the layers with attention only (keys and values may have different widths); the layers with a
-recurrence keep one slot per sequence: the FP32 state and the last inputs of the short convolution.  A sequence that
+recurrence or a short convolution keep one slot per sequence: the FP32 state and the last inputs of the convolution.  A sequence that
 starts over starts from zeros because its first segment starts at position 0, so a slot needs no clearing when it is used
 again.
 
@@ -11,9 +11,10 @@ per sequence) in up to three groups, one-token segments, short ones and long one
 
 * attention: split-key decode kernel | paged prompt kernel | tcgen05 flash kernel (fresh prompts, head sizes 64 / 128)
 * recurrences: token-by-token kernel with the state tile in shared memory | chunked tensor-core kernel
-* latent attention: `latent`; feed-forwards of experts: `experts`
+* latent attention: `latent`; attention over convolved projections: `conv_attention`; gated linear attention: `gla`;
+  feed-forwards of experts: `experts`; the long segments of a step on the prompt kernels: `prompt`
 
-The residual stream is FP32; one kernel adds a normed sublayer output to it and prepares it for the next sublayer.  In FP32
+The residual stream is FP32; one kernel adds a sublayer output (normed or not) to it and prepares it for the next sublayer.  In FP32
 precision the same layer loop runs the kernels' FP32 forms and plain FP32 matrix products.
 """
 from __future__ import annotations
@@ -24,9 +25,9 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from ..lm.config import RopeScaling
-from ..lm.hybrid import DeltaSpec, HybridConfig, HybridWeights, LatentSpec, ParallelSpec
+from ..lm.hybrid import ConvAttentionSpec, DeltaSpec, GlaSpec, HybridConfig, HybridWeights, LatentSpec, ParallelSpec
 from ..lm.rope import rope_inv_freq
-from . import experts, latent
+from . import conv_attention, experts, gla, latent, prompt
 from .engine import Chunk, Engine, _Linear
 
 __all__ = ["HybridEngine"]
@@ -62,6 +63,8 @@ class HybridEngine(Engine):
                 raise ValueError(f"layer {i}: the BF16 attention kernels take head sizes up to 256")
             if isinstance(m, LatentSpec):
                 latent.check(self, i, m)
+            if isinstance(m, ConvAttentionSpec):
+                conv_attention.check(self, i, m)
             if layer.experts and layer.experts.shared and self.model.pre_norm:
                 raise ValueError(f"layer {i}: the gate of the shared expert reads the residual stream, which this design norms first")
         self.adt = torch.bfloat16 if self.fast else torch.float32
@@ -72,6 +75,9 @@ class HybridEngine(Engine):
         self.ctx = cfg.context if cfg.context > 0 else self.n_blocks * cfg.block_size
         self._rope: Dict[tuple, tuple] = {}
         self._short_len = 16 if self.fast else 1 << 30
+        mixers = [layer.mixer for layer in self.model.layers]
+        self._prompt_windows = {prompt.Window(m.window) for m in mixers if isinstance(m, LatentSpec) and latent.expandable(m)} | {
+            conv_attention.window(m) for m in mixers if isinstance(m, ConvAttentionSpec) and conv_attention.promptable(m)}
 
     def _rope_tables(self, dims: int, base: float, scaling: Optional[RopeScaling] = None):
         """cos / sin [ctx, dims / 2]: angles in double, kept in FP32."""
@@ -84,9 +90,9 @@ class HybridEngine(Engine):
         return self._rope[key]
 
     # ----------------------------------------------------------------------------- weights
-    def _pack(self, parts: Sequence[torch.Tensor]):
+    def _pack(self, parts: Sequence[torch.Tensor], bias: Optional[torch.Tensor] = None):
         """Stacks projections of one input: rows of each part padded to a multiple of 8, columns padded to a multiple of
-        8.  Returns the linear layer and the first output column of every part."""
+        8 (``bias``: that of a single part).  Returns the linear layer and the first output column of every part."""
         k = _pad8(parts[0].shape[1])
         offsets, n = [], 0
         for p in parts:
@@ -95,7 +101,9 @@ class HybridEngine(Engine):
         w = torch.zeros((n, k))
         for p, o in zip(parts, offsets):
             w[o: o + p.shape[0], : p.shape[1]] = p.float()
-        lin = _Linear(w, None, self.dev, self.fast)
+        if bias is not None:
+            bias = torch.nn.functional.pad(bias.float(), (0, n - bias.shape[0]))
+        lin = _Linear(w, bias, self.dev, self.fast)
         self.weight_nbytes += lin.nbytes
         return lin, offsets
 
@@ -111,7 +119,7 @@ class HybridEngine(Engine):
         self.embed = t["embed"].to(self.dev, self.adt).contiguous()
         self.side_embed = t["side.embed"].to(self.dev, self.adt).contiguous() if model.token_side else None
         self.weight_nbytes += sum(e.numel() * e.element_size() for e in (self.embed, self.side_embed) if e is not None)
-        self.final_norm = self._f32(t["final.norm"])
+        self.final_norm = self._f32(t["final.norm"]) + model.norm_offset
         self.layers: List[dict] = []
         for i, layer in enumerate(model.layers):
             p, m = f"l{i}.", layer.mixer
@@ -119,10 +127,12 @@ class HybridEngine(Engine):
             out = {}
             for k, needed in (("1", True), ("2", bool(layer.ff or layer.experts))):
                 if needed:
-                    out["pre" + k] = self._f32(t[p + "norm" + k]) if model.pre_norm else None
-                    out["post" + k] = self._f32(t[p + "norm" + k + ("b" if model.pre_norm else "")])
-            if isinstance(m, LatentSpec):
-                out["mix"] = latent.load(self, m, lambda n: t[p + "mix." + n])
+                    out["pre" + k] = self._f32(t[p + "norm" + k]) + model.norm_offset if model.pre_norm else None
+                    name = p + "norm" + k + ("b" if model.pre_norm else "")
+                    out["post" + k] = self._f32(t[name]) + model.norm_offset if model.post_norm else None
+            module = {LatentSpec: latent, ConvAttentionSpec: conv_attention, GlaSpec: gla}.get(type(m))
+            if module is not None:
+                out["mix"] = module.load(self, m, lambda n: t[p + "mix." + n])
             elif isinstance(m, ParallelSpec):
                 a, r = m.left, m.right
                 w_in = t[p + "mix.right.in"]
@@ -171,6 +181,12 @@ class HybridEngine(Engine):
         self.conv_tail: list = [None] * self.L    # [slots, taps - 1, channels]
         for i, layer in enumerate(self.model.layers):
             m = layer.mixer
+            if isinstance(m, ConvAttentionSpec):
+                conv_attention.alloc(self, i, m)
+                continue
+            if isinstance(m, GlaSpec):
+                self.state[i] = torch.zeros((cfg.max_seqs, m.heads, m.dim, m.vdim), dtype=torch.float32, device=self.dev)
+                continue
             if isinstance(m, LatentSpec):     # one row per token, whose leading columns are the values; the padding stays zero
                 row = latent.LatentShape(m).row
                 self.k_cache[i] = torch.zeros((self.n_blocks, cfg.block_size, 1, row), dtype=self.adt, device=self.dev)
@@ -226,7 +242,7 @@ class HybridEngine(Engine):
         self._stepped = M.Segments(table, 0, single.count + short.count, max(single.max_len, short.max_len),
                                    single.total + short.total)
         self._every = M.Segments(table, 0, first, max(g.max_len for g in groups), sum(g.total for g in groups))
-        latent.plan(self)
+        prompt.plan(self, self._prompt_windows)
         return self._body(dv[0], dv[1], dv[2], dv[3], dv[4], dv[5][:logit_rows], runs, nl)
 
     def _buffer(self, rows: int, cols: int) -> torch.Tensor:
@@ -237,7 +253,7 @@ class HybridEngine(Engine):
     def _decode_splits(self, a, rows: int) -> int:
         if self.cfg.decode_splits > 0:
             return self.cfg.decode_splits
-        keys = min(a.window, self.ctx) if a.window > 0 else self.ctx
+        keys = min(a.window + getattr(a, "keep_first", 0), self.ctx) if a.window > 0 else self.ctx
         ctas = rows * a.kv_heads * (-(-(a.heads // a.kv_heads) // 16))
         return max(1, min(592 // max(ctas, 1), -(-keys // 256), 32))
 
@@ -339,6 +355,10 @@ class HybridEngine(Engine):
     def _mixer(self, i: int, m, lw: dict, h, pos, slot) -> torch.Tensor:
         if isinstance(m, LatentSpec):
             return latent.mixer(self, i, m, lw["mix"], h, pos, slot)
+        if isinstance(m, ConvAttentionSpec):
+            return conv_attention.mixer(self, i, m, lw["mix"], h, slot)
+        if isinstance(m, GlaSpec):
+            return gla.mixer(self, i, m, lw["mix"], h)
         if isinstance(m, ParallelSpec):
             return self._parallel_mixer(i, m, lw, h, pos, slot)
         return self._delta_mixer(i, m, lw, h)
@@ -360,23 +380,27 @@ class HybridEngine(Engine):
             y, add = self._mixer(i, layer.mixer, lw, h, pos, slot), {"w_post": lw["post1"]}
             if layer.experts:
                 f, ff, r = layer.experts, lw["ff"], routes[i]
-                extra = {}
+                extra, by_slot = {}, None
                 if f.shared:
                     gate = torch.empty(n, dtype=torch.float32, device=self.dev)
                     extra.update(w_dot=ff["sg"], dot_out=gate)
-                by_slot = None
-                if r.align >= 128:
+                if r is not None and r.align >= 128:
                     by_slot = torch.empty((r.max_slots, h.shape[1]), dtype=self.adt, device=self.dev)
                     extra.update(scatter=by_slot, slots=r.slots, top=r.top)
                 M.residual_norm(x, y=y, eps=eps, res_mult=mult, **add, **feed(lw["pre2"]), **extra)
+                if f.router:
+                    r, by_slot = experts.gate(self, f, ff, h)
                 rows, y = experts.forward(self, f, ff, r, h, by_slot)
                 add = {"w_post": lw["post2"], "experts": rows, "slots": r.slots, "top": r.top,
-                       "y_gate": gate if f.shared else None}
+                       "weights": r.weight, "y_gate": gate if f.shared else None}
             elif layer.ff:
                 M.residual_norm(x, y=y, eps=eps, res_mult=mult, **add, **feed(lw["pre2"]))
                 gu = self._linear(h, lw["up"])
                 act = torch.empty((n, gu.shape[1] // 2), dtype=self.adt, device=self.dev)
-                M.silu_mul(gu, act)
+                if layer.act == "silu":
+                    M.silu_mul(gu, act)
+                else:
+                    M.glu(gu, act, M.Glu(1))
                 y, add = self._linear(act, lw["down"]), {"w_post": lw["post2"]}
             M.residual_norm(x, y=y, eps=eps, res_mult=mult, **add, **after)
             if model.token_side:
@@ -393,6 +417,6 @@ class HybridEngine(Engine):
         hr = torch.empty((xr.shape[0], _pad8(self.d)), dtype=self.adt, device=self.dev)
         M.residual_norm(xr, w_next=self.final_norm, h=hr, eps=eps)
         logits = self._linear(hr, self.head, out_dtype=torch.float32)
-        if model.logit_softcap > 0:
-            M.softcap_(logits, self.V, model.logit_softcap)
+        if model.logit_softcap > 0 or model.logit_scale != 1.0:
+            M.softcap_(logits, self.V, model.logit_softcap, model.logit_scale)
         return logits

@@ -15,6 +15,7 @@ from typing import Dict
 import torch
 
 from ..lm.hybrid import LatentSpec
+from .prompt import StepPlan, Window
 
 
 def _pad(n: int, to: int) -> int:
@@ -48,11 +49,21 @@ def load(engine, m: LatentSpec, get) -> dict:
     s, H = LatentShape(m), m.heads
     dkv = get("dkv")
     out: Dict[str, object] = {"shape": s}
-    out["in"], out["off"] = engine._pack([get("dq"), dkv[: m.kv_rank], dkv[m.kv_rank:], get("g")])
-    uq = torch.zeros((H, s.head, m.q_rank))
-    src = get("uq").float().view(H, m.dim + m.rope_dims, m.q_rank)
-    uq[:, : m.dim], uq[:, s.dim: s.dim + m.rope_dims] = src[:, : m.dim], src[:, m.dim:]
-    out["uq"], _ = engine._pack([uq.view(H * s.head, m.q_rank)])
+    # queries from the input or from their latent; neighbouring pairs become halves: q and the shared key part, whose products
+    # alone matter, are permuted alike
+    src = get("uq" if m.q_rank else "q").float()
+    src = src.view(H, m.dim + m.rope_dims, src.shape[1])
+    order = torch.arange(m.rope_dims)
+    if m.interleaved:
+        order = order.view(-1, 2).t().reshape(-1)
+    wq = torch.zeros((H, s.head, src.shape[2]))
+    wq[:, : m.dim], wq[:, s.dim: s.dim + m.rope_dims] = src[:, : m.dim], src[:, m.dim:][:, order]
+    wq = wq.view(H * s.head, -1)
+    gate = [get("g")] if m.gate else []
+    out["in"], off = engine._pack([get("dq") if m.q_rank else wq, dkv[: m.kv_rank], dkv[m.kv_rank:][order], *gate])
+    out["off"] = (*off, 0) if not m.gate else tuple(off)
+    if m.q_rank:
+        out["uq"], _ = engine._pack([wq])
     # [W_uk | W_uv], rows head by head: one product expands a latent; W_uk also serves as [heads, dim, rank]
     ukv = torch.zeros((H * (s.dim + s.vdim), s.rank))
     ukv[: H * s.dim].view(H, s.dim, s.rank)[:, : m.dim, : m.kv_rank] = get("uk").float().view(H, m.dim, m.kv_rank)
@@ -66,7 +77,7 @@ def load(engine, m: LatentSpec, get) -> dict:
     wo = torch.zeros((engine.d, H, s.vdim))
     wo[:, :, : m.vdim] = get("o").float().view(engine.d, H, m.vdim)
     out["out"], _ = engine._pack([wo.view(engine.d, H * s.vdim)])
-    out["w_q"], out["w_kv"] = engine._f32(get("dq.norm")), engine._f32(get("dkv.norm"))
+    out["w_q"], out["w_kv"] = engine._f32(get("dq.norm")) if m.q_rank else None, engine._f32(get("dkv.norm"))
     out["rope"] = engine._rope_tables(m.rope_dims, m.rope_base, m.rope_scaling)
     return out
 
@@ -134,109 +145,30 @@ def expandable(m: LatentSpec) -> bool:
     return s.dim <= 128 and s.rot <= 64 and s.vdim <= 128 and m.scale > 0
 
 
-QUERY_BLOCK = 256    # query rows of one work item of the expanded form
-
-
-def long_segments(segs, window: int):
-    """The work of the expanded form for segments (first row, rows, first position, sequence): (blocks, runs, rows of kv).
-
-    A segment that does not start at position 0 needs latents of earlier steps: if there is one, all keys are gathered from
-    the cache (``runs``: first row, rows, first position, sequence), else they are the rows of the step and ``runs`` is empty.
-    ``blocks``: first query row, rows, position of the first row, kv row of position 0; the most keys first."""
-    back, blocks, runs, d = window - 1 if window > 0 else 1 << 30, [], [], 0
-    gather = any(pos > 0 for _, _, pos, _ in segs)
-    for row0, count, pos, seq in segs:
-        base, kv0 = 0, row0
-        if gather:
-            base = max(0, pos - back)
-            kv0 = d - base
-            runs.append((d, pos + count - base, base, seq))
-            d += pos + count - base
-        for b in range(0, count, QUERY_BLOCK):
-            rows = min(QUERY_BLOCK, count - b)
-            blocks.append((min(pos + b, back) + rows, row0 + b, rows, pos + b, kv0))
-    blocks.sort(key=lambda x: -x[0])
-    return [b[1:] for b in blocks], runs, d
-
-
-class StepPlan:
-    """How the segments of a step that has long ones are split between the two forms; built on the host once per step.
-
-    ``rows``: the rows of the one-token and short segments, ``groups`` these segments over the compacted rows; per window the
-    blocks and runs of the long ones (`long_segments`)."""
-
-    def __init__(self, engine, windows):
-        from ..ops import _mixers as M
-        single, short, long_ = engine._groups
-        host, n = engine._host_rows[engine.INDEX_ROWS:], single.count + short.count
-        segs = [tuple(int(v) for v in host[:, j]) for j in range(n + long_.count)]
-        data, at = [], {}
-
-        def put(name, values):
-            at[name] = (len(data), len(values))
-            data.extend(values)
-            data.extend([0] * (-len(data) % 4))        # tables start on 16 bytes
-        first, table = 0, [[], [], [], []]
-        for row0, count, pos, seq in segs[:n]:
-            for t, v in zip(table, (first, count, pos, seq)):
-                t.append(v)
-            first += count
-        put("rows", [r for row0, count, _, _ in segs[:n] for r in range(row0, row0 + count)])
-        put("table", [v for t in table for v in t])
-        self.kv_rows, self.longest = {}, {}
-        for w in windows:
-            blocks, runs, self.kv_rows[w] = long_segments(segs[n:], w)
-            self.longest[w] = max((r[1] for r in runs), default=0)
-            put(("blocks", w), [v for b in blocks for v in b])
-            put(("runs", w), [v for r in runs for v in r])
-        self.gathered = any(self.kv_rows.values())
-        dev = torch.tensor(data, dtype=torch.int32).pin_memory().to(engine.dev, non_blocking=True)
-
-        def get(name):
-            return dev[at[name][0]: at[name][0] + at[name][1]]
-        self.blocks = {w: get(("blocks", w)).view(-1, 4) for w in windows}
-        self.runs = {w: get(("runs", w)).view(-1, 4) for w in windows}
-        self.rows = get("rows").long() if n else None
-        if n:
-            t = get("table").view(4, n)
-            self.groups = [M.Segments(t, 0, single.count, single.max_len, single.total),
-                           M.Segments(t, single.count, short.count, short.max_len, short.total)]
-
-
-def plan(engine) -> None:
-    """Called once per step, before the layers."""
-    engine._latent_plan = None
-    if not engine.fast or engine._groups[2].count == 0:
-        return
-    windows = sorted({x.mixer.window for x in engine.model.layers if isinstance(x.mixer, LatentSpec) and expandable(x.mixer)})
-    if windows:
-        engine._latent_plan = StepPlan(engine, windows)
-
-
 def expanded(engine, i: int, m: LatentSpec, lw: dict, q, lat, gate, pos, out, step: StepPlan) -> None:
     """The long segments of a step.  ``lat``: latent rows of the step; ``q`` is rotated in place."""
     from ..ops import _mixers as M
-    s, w = lw["shape"], m.window
+    s, w = lw["shape"], Window(m.window)
     if step.gathered:
         lat = torch.empty((step.kv_rows[w], s.row), dtype=engine.adt, device=engine.dev)
         M.latent_gather(engine.k_cache[i], engine.block_table, step.runs[w], step.longest[w], lat)
     kv = engine._linear(lat[:, : s.rank], lw["ukv"])
     M.rope_heads(q, s.head, s.dim, q, s.head, s.dim, m.heads, m.rope_dims, s.rot, pos, *lw["rope"])
-    M.latent_prompt(q, kv, lat, out, step.blocks[w], heads=m.heads, dim=s.dim, rot=s.rot, vdim=s.vdim, rank=s.rank, window=w,
+    M.latent_prompt(q, kv, lat, out, step.blocks[w], heads=m.heads, dim=s.dim, rot=s.rot, vdim=s.vdim, rank=s.rank, window=w.size,
                     scale=m.scale, gate=gate)
 
 
 def mixer(engine, i: int, m: LatentSpec, lw: dict, h, pos, slot):
     from ..ops import _mixers as M
     s, n = lw["shape"], h.shape[0]
-    step = engine._latent_plan if expandable(m) else None
+    step = engine._prompt_plan if expandable(m) else None
     proj = engine._linear(h, lw["in"])
-    cq = torch.empty((n, _pad(m.q_rank, 8)), dtype=engine.adt, device=engine.dev)
-    gate = torch.empty((n, m.heads), dtype=torch.float32, device=engine.dev)
+    cq = torch.empty((n, _pad(m.q_rank, 8)), dtype=engine.adt, device=engine.dev) if m.q_rank else None
+    gate = torch.empty((n, m.heads), dtype=torch.float32, device=engine.dev) if m.gate else None
     lat = torch.empty((n, s.row), dtype=engine.adt, device=engine.dev) if step is not None and not step.gathered else None
     M.latent_prep(proj, lw["off"], m.q_rank, m.kv_rank, m.rope_dims, m.heads, lw["w_q"], lw["w_kv"], pos, slot, *lw["rope"], cq,
                   engine.k_cache[i], s.rank, gate, eps=engine.model.norm_eps, lat=lat)
-    q = engine._linear(cq, lw["uq"])
+    q = engine._linear(cq, lw["uq"]) if m.q_rank else proj[:, : m.heads * s.head]
     out = torch.empty((n, m.heads * s.vdim), dtype=engine.adt, device=engine.dev)
     if step is None:
         groups = [engine._groups[0], engine._many] if engine.fast else [engine._every]
@@ -244,8 +176,8 @@ def mixer(engine, i: int, m: LatentSpec, lw: dict, h, pos, slot):
     else:
         if step.rows is not None:       # before the rotation in place
             part = torch.empty((step.rows.shape[0], out.shape[1]), dtype=engine.adt, device=engine.dev)
-            absorbed(engine, i, m, lw, q.index_select(0, step.rows), gate.index_select(0, step.rows), pos.index_select(0, step.rows),
-                     part, step.groups)
+            absorbed(engine, i, m, lw, q.index_select(0, step.rows), gate.index_select(0, step.rows) if m.gate else None,
+                     pos.index_select(0, step.rows), part, step.groups)
         expanded(engine, i, m, lw, q, lat, gate, pos, out, step)
         if step.rows is not None:
             out.index_copy_(0, step.rows, part)

@@ -1,0 +1,95 @@
+"""How the long segments of a step reach the tcgen05 prompt kernels: blocks of query rows, and the keys that earlier steps left in
+the cache pages gathered beside those of the step.  Built on the host once per step, one table per window."""
+from __future__ import annotations
+
+from typing import NamedTuple
+
+import torch
+
+QUERY_BLOCK = 256    # query rows of one work item
+
+
+class Window(NamedTuple):
+    """What a layer's rows see: the last ``size`` keys (0: all of them) and the first ``keep_first`` ones."""
+    size: int
+    keep_first: int = 0
+
+
+def long_segments(segs, window: int, keep_first: int = 0):
+    """The work for segments (first row, rows, first position, sequence): (blocks, runs, rows of kv).
+
+    A segment that does not start at position 0 needs keys of earlier steps: if there is one, all keys are gathered from the
+    cache (``runs``: first row, rows, first position, sequence), else they are the rows of the step and ``runs`` is empty.
+    ``blocks``: first query row, rows, position of the first row, kv row of position 0 and, last, the row that position 0 has
+    among the kept first keys; the most keys first."""
+    back, blocks, runs, d = window - 1 if window > 0 else 1 << 30, [], [], 0
+    gather = any(pos > 0 for _, _, pos, _ in segs)
+    for row0, count, pos, seq in segs:
+        kv0 = kept0 = row0
+        if gather:
+            base = max(0, pos - back)
+            kept, kept0 = min(keep_first, base), d
+            if kept:                          # in front of the keys from `base` on
+                runs.append((d, kept, 0, seq))
+                d += kept
+            kv0 = d - base
+            if not kept:
+                kept0 = kv0
+            runs.append((d, pos + count - base, base, seq))
+            d += pos + count - base
+        for b in range(0, count, QUERY_BLOCK):
+            rows = min(QUERY_BLOCK, count - b)
+            blocks.append((min(pos + b, back) + rows, row0 + b, rows, pos + b, kv0, kept0))
+    blocks.sort(key=lambda x: -x[0])
+    return [b[1:] for b in blocks], runs, d
+
+
+class StepPlan:
+    """How the segments of a step that has long ones are split; ``rows``: the rows of the one-token and short segments,
+    ``groups`` these segments over the compacted rows; per window the blocks and runs of the long ones (`long_segments`)."""
+
+    def __init__(self, engine, windows):
+        from ..ops import _mixers as M
+        single, short, long_ = engine._groups
+        host, n = engine._host_rows[engine.INDEX_ROWS:], single.count + short.count
+        segs = [tuple(int(v) for v in host[:, j]) for j in range(n + long_.count)]
+        data, at = [], {}
+
+        def put(name, values):
+            at[name] = (len(data), len(values))
+            data.extend(values)
+            data.extend([0] * (-len(data) % 4))        # tables start on 16 bytes
+        first, table = 0, [[], [], [], []]
+        for row0, count, pos, seq in segs[:n]:
+            for t, v in zip(table, (first, count, pos, seq)):
+                t.append(v)
+            first += count
+        put("rows", [r for row0, count, _, _ in segs[:n] for r in range(row0, row0 + count)])
+        put("table", [v for t in table for v in t])
+        self.kv_rows, self.longest = {}, {}
+        for w in windows:
+            blocks, runs, self.kv_rows[w] = long_segments(segs[n:], *w)
+            self.longest[w] = max((r[1] for r in runs), default=0)
+            put(("blocks", w), [v for b in blocks for v in b[:4]])
+            put(("kept", w), [b[4] for b in blocks])
+            put(("runs", w), [v for r in runs for v in r])
+        self.gathered = any(self.kv_rows.values())
+        dev = torch.tensor(data, dtype=torch.int32).pin_memory().to(engine.dev, non_blocking=True)
+
+        def get(name):
+            return dev[at[name][0]: at[name][0] + at[name][1]]
+        self.blocks = {w: get(("blocks", w)).view(-1, 4) for w in windows}
+        self.kept = {w: get(("kept", w)) for w in windows}
+        self.runs = {w: get(("runs", w)).view(-1, 4) for w in windows}
+        self.rows = get("rows").long() if n else None
+        if n:
+            t = get("table").view(4, n)
+            self.groups = [M.Segments(t, 0, single.count, single.max_len, single.total),
+                           M.Segments(t, single.count, short.count, short.max_len, short.total)]
+
+
+def plan(engine, windows) -> None:
+    """Called once per step, before the layers; ``windows``: those of the layers that a prompt kernel can take."""
+    engine._prompt_plan = None
+    if engine.fast and engine._groups[2].count > 0 and windows:
+        engine._prompt_plan = StepPlan(engine, sorted(windows))

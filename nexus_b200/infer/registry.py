@@ -10,6 +10,7 @@ import os
 from dataclasses import dataclass
 from typing import Callable, Dict, Optional
 
+from ..lm.gutivik import load_gutivik
 from ..lm.hybrid import HybridWeights, load_gugedra
 from ..lm.makuzen import load_makuzen
 from .engine import Engine, EngineConfig, Gpt2Weights, load_gpt2
@@ -68,3 +69,4 @@ def _load_gpt2_folder(path: str) -> Gpt2Weights:
 register_family(ModelFamily("GPT2", _load_gpt2_folder, Gpt2Weights, Engine))
 register_family(ModelFamily("Gugedra", load_gugedra, HybridWeights, HybridEngine))
 register_family(ModelFamily("Makuzen", load_makuzen, HybridWeights, HybridEngine))
+register_family(ModelFamily("Gutivik", load_gutivik, HybridWeights, HybridEngine))

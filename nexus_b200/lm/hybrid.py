@@ -1,15 +1,16 @@
 """Decoders whose layers differ from one another: the layer list, the mixers' sizes and constants, and the weights.
 
 A model is an ordered list of :class:`HybridLayer`; each has one mixer - :class:`AttentionSpec` and :class:`SsdSpec` side
-by side (:class:`ParallelSpec`), :class:`DeltaSpec` or :class:`LatentSpec` - and optionally a feed-forward, gated or of
-experts (:class:`ExpertsSpec`).  The engine (`infer.hybrid.HybridEngine`) builds its cache, its state slots and its
+by side (:class:`ParallelSpec`), :class:`ConvAttentionSpec`, :class:`DeltaSpec`, :class:`GlaSpec` or :class:`LatentSpec` - and
+optionally a feed-forward, gated or of experts (:class:`ExpertsSpec`).  The engine (`infer.hybrid.HybridEngine`) builds its cache, its state slots and its
 kernels' arguments from these specs and reads no size from anywhere else, so another order of layers or another
 combination of constants is another configuration, not another class.
 
 `Gugedra` is one design that uses them: RMS norms before and after every sublayer, a sliding-window soft-capped
 attention branch beside a Mamba-2 branch in some layers, the gated delta rule in the others, a per-layer token input at
 the end of every layer and soft-capped logits.  :func:`gugedra_config` reads its ``config.json``, and
-:func:`load_gugedra` its ``model.safetensors``.  `Makuzen` (`lm.makuzen`) is another.
+:func:`load_gugedra` its ``model.safetensors``.  `Makuzen` (`lm.makuzen`) and
+`Gutivik` (`lm.gutivik`) are others.
 """
 from __future__ import annotations
 
@@ -23,8 +24,8 @@ import torch
 
 from .config import ConfigError, RopeScaling
 
-__all__ = ["AttentionSpec", "SsdSpec", "ParallelSpec", "DeltaSpec", "LatentSpec", "ExpertsSpec", "HybridLayer", "HybridConfig",
-           "HybridWeights", "gugedra_config", "gugedra_tensors", "load_gugedra", "random_gugedra"]
+__all__ = ["AttentionSpec", "ConvAttentionSpec", "SsdSpec", "ParallelSpec", "DeltaSpec", "GlaSpec", "LatentSpec", "RouterSpec",
+           "ClampedGlu", "ExpertsSpec", "HybridLayer", "HybridConfig", "HybridWeights", "gugedra_config", "gugedra_tensors", "load_gugedra", "random_gugedra"]
 
 
 def _positive(obj, *names) -> None:
@@ -55,6 +56,25 @@ class AttentionSpec:
             raise ConfigError("attention: the rotary dimensions must be even and at most the head size")
         if self.window < 0 or self.softcap < 0:
             raise ConfigError("attention: window and softcap cannot be negative")
+
+
+@dataclass(frozen=True)
+class ConvAttentionSpec(AttentionSpec):
+    """Attention whose projections go through a short causal convolution before the rotation (of neighbouring pairs).  The first
+    ``keep_first`` keys stay visible behind a window."""
+    conv: int = 1            # taps of the short convolution
+    keep_first: int = 0
+    bias: bool = True        # on the projections of q, k and v
+    sink: bool = True        # a learned score per head that counts in the softmax denominator only
+    mix_values: bool = False     # values are mixed with those of the first layer that has this set
+
+    def __post_init__(self):
+        super().__post_init__()
+        _positive(self, "conv")
+        if self.conv > 8:
+            raise ConfigError("attention: the convolution kernel has at most 8 taps")
+        if self.keep_first < 0:
+            raise ConfigError("attention: keep_first cannot be negative")
 
 
 @dataclass(frozen=True)
@@ -117,37 +137,81 @@ class DeltaSpec:
 
 
 @dataclass(frozen=True)
+class GlaSpec:
+    """Gated linear attention: a decay sigmoid(z)^(1 / tau) per key channel, z through ``rank`` columns."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    rank: int
+
+    def __post_init__(self):
+        _positive(self, "heads", "dim", "vdim", "rank")
+        if not self.tau > 0:
+            raise ConfigError("gated linear attention: tau must be positive")
+
+
+@dataclass(frozen=True)
 class LatentSpec:
     """Causal softmax attention whose keys and values are linear in one normed latent per token; a token's cache row is the
     latent and one rotated key part, both shared by the heads."""
     heads: int
     dim: int                 # unrotated query / key size of a head
-    rope_dims: int           # rotated query / key size of a head (rotate-half pairing)
+    rope_dims: int           # rotated query / key size of a head
     vdim: int                # value size of a head
-    q_rank: int              # size of the latent the queries go through
+    q_rank: int              # size of the latent the queries go through, 0: none
     kv_rank: int             # size of the cached latent
     scale: float
     window: int = 0          # > 0: a token sees itself and the window - 1 tokens before it
     rope_base: float = 10000.0
     rope_scaling: Optional[RopeScaling] = None
+    interleaved: bool = False    # neighbouring dimensions rotate together, else dimensions i and i + rope_dims / 2
+    gate: bool = True            # a sigmoid per head on the output
 
     def __post_init__(self):
-        _positive(self, "heads", "dim", "rope_dims", "vdim", "q_rank", "kv_rank")
+        _positive(self, "heads", "dim", "rope_dims", "vdim", "kv_rank")
         if self.rope_dims % 2:
             raise ConfigError("latent attention: the rotary dimensions must be even")
-        if self.window < 0:
-            raise ConfigError("latent attention: window cannot be negative")
+        if self.window < 0 or self.q_rank < 0:
+            raise ConfigError("latent attention: window and q_rank cannot be negative")
+
+
+@dataclass(frozen=True)
+class RouterSpec:
+    """Experts chosen by sigmoid scores plus a correction, weighted by the scores alone; with ``groups`` > 1 only experts of the
+    ``keep`` groups whose two best corrected scores sum highest can be chosen."""
+    groups: int = 1
+    keep: int = 1
+
+    def __post_init__(self):
+        _positive(self, "groups", "keep")
+        if self.keep > self.groups:
+            raise ConfigError("router: more groups are kept than there are")
+
+
+@dataclass(frozen=True)
+class ClampedGlu:
+    """g sigmoid(slope g) (u + offset) with the gate g = min(., limit) and the value u = clamp(., -limit, limit)."""
+    limit: float
+    slope: float = 1.702
+    offset: float = 1.0
+
+    def __post_init__(self):
+        if not self.limit > 0:
+            raise ConfigError("clamped gated unit: the limit must be positive")
 
 
 @dataclass(frozen=True)
 class ExpertsSpec:
-    """Feed-forward of small experts, W_down act(W_up h) with act = relu squared, of which a token uses ``top`` with equal
-    weights; a table gives every token id its experts.  ``shared``: width of an expert that runs for every token, times
-    one sigmoid per token (0: none)."""
+    """Feed-forward of small experts of which a token uses ``top``.  Without a router a table gives every token id its experts,
+    all with equal weights.  An expert is W_down act(W_up h) with act = relu squared, or with ``glu`` W_down glu(W_gate h, W_up h).
+    ``shared``: width of an expert that runs for every token, times one sigmoid per token (0: none)."""
     experts: int
     top: int
     ff: int
     shared: int = 0
+    router: Optional[RouterSpec] = None
+    glu: Optional[ClampedGlu] = None
 
     def __post_init__(self):
         _positive(self, "experts", "top", "ff")
@@ -155,13 +219,26 @@ class ExpertsSpec:
             raise ConfigError("experts: a token cannot use more experts than there are")
         if self.shared < 0:
             raise ConfigError("experts: the width of the shared expert cannot be negative")
+        if self.router is not None:
+            if self.experts % self.router.groups:
+                raise ConfigError("experts: groups must divide the experts")
+            if self.experts // self.router.groups * self.router.keep < self.top:
+                raise ConfigError("experts: the groups that are kept have fewer experts than a token uses")
+
+
+GLU_ACTS = ("silu", "gelu_tanh")
 
 
 @dataclass(frozen=True)
 class HybridLayer:
-    mixer: Union[ParallelSpec, DeltaSpec, LatentSpec]
-    ff: int = 0              # width of the SwiGLU feed-forward, 0: none
+    mixer: Union[ParallelSpec, ConvAttentionSpec, DeltaSpec, GlaSpec, LatentSpec]
+    ff: int = 0              # width of the gated feed-forward, 0: none
     experts: Optional[ExpertsSpec] = None
+    act: str = "silu"        # activation of the gate of the feed-forward
+
+    def __post_init__(self):
+        if self.act not in GLU_ACTS:
+            raise ConfigError(f"unknown activation {self.act!r}")
 
 
 @dataclass
@@ -173,9 +250,12 @@ class HybridConfig:
     token_side: int = 0      # width of the per-layer token input, 0: none
     logit_softcap: float = 0.0
     name: str = "hybrid"
-    pre_norm: bool = True    # sublayers read the normed residual stream, else the stream itself; their outputs are normed always
+    pre_norm: bool = True    # sublayers read the normed residual stream, else the stream itself
+    post_norm: bool = True   # the outputs of sublayers are normed
+    norm_offset: float = 0.0     # added to the stored weights of the layers' norms and the final one
     embed_scale: float = 1.0
-    residual_mult: float = 1.0   # factor of every normed sublayer output
+    residual_mult: float = 1.0   # factor of every sublayer output
+    logit_scale: float = 1.0     # before the soft cap
 
     def __post_init__(self):
         _positive(self, "vocab", "width")
@@ -183,17 +263,28 @@ class HybridConfig:
             raise ConfigError("token_side cannot be negative")
         if not self.layers:
             raise ConfigError("a model needs at least one layer")
+        if len({m.kv_heads * m.vdim for m in self._mixing()}) > 1:
+            raise ConfigError("layers that mix values must have equal sizes of them")
+
+    def _mixing(self) -> list:
+        return [x.mixer for x in self.layers if isinstance(x.mixer, ConvAttentionSpec) and x.mixer.mix_values]
+
+    @property
+    def first_mixing(self) -> int:
+        """The layer whose values later layers mix with theirs, -1: none."""
+        return next((i for i, x in enumerate(self.layers) if isinstance(x.mixer, ConvAttentionSpec) and x.mixer.mix_values), -1)
 
     @property
     def recurrent(self) -> bool:
         """Whether a sequence owns state beside its cache pages."""
-        return any(isinstance(layer.mixer, (ParallelSpec, DeltaSpec)) for layer in self.layers)
+        return any(isinstance(layer.mixer, (ParallelSpec, ConvAttentionSpec, DeltaSpec, GlaSpec)) for layer in self.layers)
 
     def kv_bytes_per_token(self, element: int) -> int:
         n = 0
         for m in (layer.mixer for layer in self.layers):
-            if isinstance(m, ParallelSpec):
-                n += m.left.kv_heads * (m.left.dim + m.left.vdim) * element
+            if isinstance(m, (ParallelSpec, ConvAttentionSpec)):
+                a = m.left if isinstance(m, ParallelSpec) else m
+                n += a.kv_heads * (a.dim + a.vdim) * element
             elif isinstance(m, LatentSpec):
                 n += (m.kv_rank + m.rope_dims) * element
         return n

@@ -1,6 +1,6 @@
 """ctypes bindings of the mixer kernels (``nx_api_mixers.h``): the residual / norm chain, rotary embedding with cache
-append, windowed soft-capped paged attention, the short causal convolution, the SSD and gated-delta recurrences, gated
-norms and the per-layer token input.  BF16 or FP32 activations; every wrapper launches on the current torch stream."""
+append, windowed soft-capped paged attention, the short causal convolution, the SSD, gated-delta and gated-linear
+recurrences, gated norms, gated activations and the per-layer token input.  BF16 or FP32 activations; every wrapper launches on the current torch stream."""
 from __future__ import annotations
 
 import ctypes as C
@@ -26,7 +26,7 @@ class ResidualNormArgs(C.Structure):
                 ("rows", C.c_int32), ("cols", C.c_int32), ("dtype", C.c_int32), ("eps", C.c_float), ("embed_scale", C.c_float),
                 ("res_mult", C.c_float), ("experts", C.c_void_p), ("expert_slots", C.c_void_p), ("y_gate", C.c_void_p),
                 ("ld_experts", C.c_int64), ("top", C.c_int32), ("expert_scale", C.c_float), ("w_dot", C.c_void_p),
-                ("dot_out", C.c_void_p), ("scatter", C.c_void_p), ("scatter_slots", C.c_void_p)]
+                ("dot_out", C.c_void_p), ("scatter", C.c_void_p), ("scatter_slots", C.c_void_p), ("expert_weights", C.c_void_p)]
 
 
 class LatentPrepArgs(C.Structure):
@@ -49,6 +49,24 @@ class ConvArgs(C.Structure):
     _fields_ = [("x", C.c_void_p), ("y", C.c_void_p), ("w", C.c_void_p), ("bias", C.c_void_p), ("state", C.c_void_p),
                 ("ldx", C.c_int64), ("ldy", C.c_int64), ("channels", C.c_int32), ("taps", C.c_int32), ("dtype", C.c_int32),
                 ("seg", SegmentArgs)]
+
+
+class ConvRopeArgs(C.Structure):
+    _fields_ = [("conv", ConvArgs), ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32),
+                ("rot_dims", C.c_int32), ("store_kv", C.c_int32), ("slots", C.c_void_p), ("cos_t", C.c_void_p), ("sin_t", C.c_void_p),
+                ("k_cache", C.c_void_p), ("v_cache", C.c_void_p), ("mix", C.c_void_p), ("first", C.c_void_p)]
+
+
+class GlaArgs(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("decay", C.c_void_p), ("o", C.c_void_p),
+                ("state", C.c_void_p), ("ld", C.c_int64), ("ld_decay", C.c_int64), ("ldo", C.c_int64), ("heads", C.c_int32),
+                ("dim", C.c_int32), ("vdim", C.c_int32), ("dtype", C.c_int32), ("q_scale", C.c_float), ("seg", SegmentArgs),
+                ("part_state", C.c_void_p), ("part_decay", C.c_void_p), ("parts", C.c_int32), ("span", C.c_int32)]
+
+
+class Glu(C.Structure):
+    """A gated activation: ``kind`` 0 silu(g) u, 1 gelu_tanh(g) u, 2 clamped (limit, slope, offset)."""
+    _fields_ = [("kind", C.c_int32), ("limit", C.c_float), ("slope", C.c_float), ("offset", C.c_float)]
 
 
 class SsdArgs(C.Structure):
@@ -79,7 +97,8 @@ class PagedWindowArgs(C.Structure):
                 ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32),
                 ("block_size", C.c_int32), ("max_blocks", C.c_int32), ("window", C.c_int32), ("splits", C.c_int32),
                 ("dtype", C.c_int32), ("scale", C.c_float), ("softcap", C.c_float), ("out_scale", C.c_float),
-                ("seg", SegmentArgs), ("k_pitch", C.c_int64), ("v_pitch", C.c_int64), ("gate", C.c_void_p)]
+                ("seg", SegmentArgs), ("k_pitch", C.c_int64), ("v_pitch", C.c_int64), ("gate", C.c_void_p), ("sink", C.c_void_p),
+                ("keep_first", C.c_int32)]
 
 
 class LatentPromptArgs(C.Structure):
@@ -88,6 +107,14 @@ class LatentPromptArgs(C.Structure):
                 ("ldo", C.c_int64), ("n_blocks", C.c_int32), ("q_rows", C.c_int32), ("kv_rows", C.c_int32), ("q_head", C.c_int32),
                 ("rank", C.c_int32), ("heads", C.c_int32), ("dim", C.c_int32), ("rot", C.c_int32), ("vdim", C.c_int32),
                 ("window", C.c_int32), ("scale", C.c_float)]
+
+
+class WindowPromptArgs(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("out", C.c_void_p), ("sink", C.c_void_p),
+                ("blocks", C.c_void_p), ("kept", C.c_void_p), ("status", C.c_void_p), ("ldq", C.c_int64), ("ldk", C.c_int64),
+                ("ldv", C.c_int64), ("ldo", C.c_int64), ("n_blocks", C.c_int32), ("q_rows", C.c_int32), ("kv_rows", C.c_int32),
+                ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("window", C.c_int32),
+                ("keep_first", C.c_int32), ("scale", C.c_float)]
 
 
 class LatentAttnArgs(C.Structure):
@@ -124,10 +151,12 @@ def _ptr(t: Optional[torch.Tensor]):
 
 
 def residual_norm(x, *, y=None, w_post=None, w_next=None, h=None, x_cast=None, tokens=None, table=None, eps, embed_scale=1.0,
-                  res_mult=1.0, experts=None, slots=None, top=0, y_gate=None, w_dot=None, dot_out=None, scatter=None) -> None:
-    """x (FP32) = embed_scale * table[tokens], or x + res_mult * rms(y) * w_post;  h = rms(x) * w_next;  x_cast = x in the
-    activation dtype.  With ``experts`` the sublayer output is the mean of the rows ``experts[slots[r, :]]`` (+ y_gate[r] *
-    y[r]).  ``dot_out`` = sigmoid(x . w_dot); ``scatter[slots[r, :]]`` = the row of x_cast."""
+                  res_mult=1.0, experts=None, slots=None, top=0, weights=None, y_gate=None, w_dot=None, dot_out=None,
+                  scatter=None) -> None:
+    """x (FP32) = embed_scale * table[tokens], or x + res_mult * rms(y) * w_post (without w_post: x + res_mult * y);  h = rms(x) *
+    w_next;  x_cast = x in the activation dtype.  With ``experts`` the sublayer output is the mean of the rows
+    ``experts[slots[r, :]]``, or their sum with ``weights`` [rows, top] (FP32), + y_gate[r] * y[r].  ``dot_out`` = sigmoid(x .
+    w_dot); ``scatter[slots[r, :]]`` = the row of x_cast."""
     lead = next((t for t in (h, x_cast, scatter) if t is not None), None)
     act = next(t for t in (lead, y, experts, table) if t is not None)
     if any(t is not None and t.stride(0) != lead.stride(0) for t in (h, x_cast, scatter)):
@@ -135,17 +164,18 @@ def residual_norm(x, *, y=None, w_post=None, w_next=None, h=None, x_cast=None, t
     a = ResidualNormArgs(_ptr(x), _ptr(tokens), _ptr(table), _ptr(y), _ptr(w_post), _ptr(w_next), _ptr(h), _ptr(x_cast),
                          y.stride(0) if y is not None else 0, lead.stride(0) if lead is not None else x.shape[1], x.shape[0],
                          x.shape[1], _dt(act), eps, embed_scale, res_mult, _ptr(experts), _ptr(slots), _ptr(y_gate),
-                         experts.stride(0) if experts is not None else 0, top, 1.0 / top if top else 1.0, _ptr(w_dot),
-                         _ptr(dot_out), _ptr(scatter), _ptr(slots))
+                         experts.stride(0) if experts is not None else 0, top, 1.0 / top if top and weights is None else 1.0,
+                         _ptr(w_dot), _ptr(dot_out), _ptr(scatter), _ptr(slots), _ptr(weights))
     K._check(K.lib().nx_residual_norm(C.byref(a), K._stream()), "nx_residual_norm")
 
 
 def latent_prep(proj, offsets, q_rank, kv_rank, rot_dims, heads, w_q, w_kv, positions, slots, cos_t, sin_t, cq, cache, rot_col,
                 gate, *, eps, lat=None) -> None:
     """``offsets``: first columns of the query latent, the key / value latent, the shared key part and the gate in ``proj``;
-    cache [blocks, block_size, row], lat [rows, row] or None, gate FP32 [rows, heads]."""
+    cache [blocks, block_size, row], lat [rows, row] or None, gate FP32 [rows, heads] or None; q_rank 0: no query latent."""
     a = LatentPrepArgs(_ptr(proj), proj.stride(0), *offsets, proj.shape[0], q_rank, kv_rank, rot_dims, heads, _dt(proj), eps,
-                       _ptr(w_q), _ptr(w_kv), _ptr(positions), _ptr(slots), _ptr(cos_t), _ptr(sin_t), _ptr(cq), cq.stride(0),
+                       _ptr(w_q), _ptr(w_kv), _ptr(positions), _ptr(slots), _ptr(cos_t), _ptr(sin_t), _ptr(cq),
+                       cq.stride(0) if cq is not None else 0,
                        _ptr(cache), cache.shape[-1], rot_col, _ptr(lat), _ptr(gate))
     K._check(K.lib().nx_latent_prep(C.byref(a), K._stream()), "nx_latent_prep")
 
@@ -172,6 +202,48 @@ def conv_silu(x, y, w, bias, state, seg: Segments) -> None:
     K._check(K.lib().nx_conv_silu(C.byref(a), K._stream()), "nx_conv_silu")
 
 
+def conv_rope_append(x, y, w, bias, state, seg: Segments, *, heads, kv_heads, dim, vdim, rot_dims, cos_t, sin_t, slots, k_cache,
+                     v_cache, store_kv=False, mix=None, first=None) -> None:
+    """Convolution over the packed q | k | v columns of ``x``, rotation of neighbouring pairs, value mixing (``mix``: FP32 [1] with
+    the values ``first`` [rows, kv_heads * vdim]; without it ``first`` is written) and cache append; ``y`` receives q (and k, v)."""
+    a = ConvRopeArgs(ConvArgs(_ptr(x), _ptr(y), _ptr(w), _ptr(bias), _ptr(state), x.stride(0), y.stride(0), w.shape[1], w.shape[0],
+                              _dt(x), seg.args()), heads, kv_heads, dim, vdim, rot_dims, int(store_kv), _ptr(slots), _ptr(cos_t),
+                     _ptr(sin_t), _ptr(k_cache), _ptr(v_cache), _ptr(mix), _ptr(first))
+    K._check(K.lib().nx_conv_rope_append(C.byref(a), K._stream()), "nx_conv_rope_append")
+
+
+def decay_gate(a, w, bias, tau) -> torch.Tensor:
+    """log2(sigmoid(a w^T + bias)) / tau in FP32; w FP32 [cols, rank], a [rows, >= rank]."""
+    out = torch.empty((a.shape[0], w.shape[0]), dtype=torch.float32, device=a.device)
+    K._check(K.lib().nx_decay_gate(K._p(a), C.c_int64(a.stride(0)), K._p(w), K._p(bias), K._p(out), C.c_int64(out.stride(0)),
+                                   C.c_int(a.shape[0]), C.c_int(w.shape[0]), C.c_int(w.shape[1]), C.c_float(tau), C.c_int(_dt(a)),
+                                   K._stream()), "nx_decay_gate")
+    return out
+
+
+def _spans(a, seg: Segments, parts: int) -> None:
+    chunks = -(-seg.max_len // CHUNK)
+    per = -(-chunks // max(1, parts))
+    a.span, a.parts = per * CHUNK, -(-chunks // per)
+
+
+def gla(q, k, v, decay, o, state, seg: Segments, *, q_scale, chunked=False, parts=1) -> None:
+    """q, k, v: views of one row pitch; decay: FP32 log2 decays [rows, heads * dim]; state: FP32 [slots, heads, dim, vdim]."""
+    _, H, D, Dv = state.shape
+    if not q.stride(0) == k.stride(0) == v.stride(0):
+        raise ValueError("gla: q, k and v must share one row pitch")
+    a = GlaArgs(_ptr(q), _ptr(k), _ptr(v), _ptr(decay), _ptr(o), _ptr(state), q.stride(0), decay.stride(0), o.stride(0), H, D, Dv,
+                _dt(q), q_scale, seg.args(), None, None, 1, 0)
+    if not chunked:
+        K._check(K.lib().nx_gla_step(C.byref(a), K._stream()), "nx_gla_step")
+        return
+    _spans(a, seg, parts)
+    if a.parts > 1:
+        a.part_state = K.scratch(seg.count * a.parts * H * D * Dv * 4, "gla_state", q.device).data_ptr()
+        a.part_decay = K.scratch(seg.count * a.parts * H * D * 4, "gla_decay", q.device).data_ptr()
+    K._check(K.lib().nx_gla_chunk(C.byref(a), K._stream()), "nx_gla_chunk")
+
+
 def ssd(xbc, dt, y, dt_bias, a_log, d_skip, state, groups, seg: Segments, *, chunked=False, parts=1) -> None:
     """state: FP32 [slots, heads, N, P].  ``chunked``: the tensor-core form; its segments are cut into ``parts`` spans
     that run at the same time."""
@@ -181,9 +253,7 @@ def ssd(xbc, dt, y, dt_bias, a_log, d_skip, state, groups, seg: Segments, *, chu
     if not chunked:
         K._check(K.lib().nx_ssd_step(C.byref(a), K._stream()), "nx_ssd_step")
         return
-    chunks = -(-seg.max_len // CHUNK)
-    per = -(-chunks // max(1, parts))
-    a.span, a.parts = per * CHUNK, -(-chunks // per)
+    _spans(a, seg, parts)
     if a.parts > 1:
         a.part_state = K.scratch(seg.count * a.parts * H * N * P * 4, "ssd_state", xbc.device).data_ptr()
         a.part_decay = K.scratch(seg.count * a.parts * H * 4, "ssd_decay", xbc.device).data_ptr()
@@ -228,19 +298,27 @@ def silu_mul(h, out) -> None:
                                  C.c_int(h.shape[1] // 2), C.c_int(_dt(h)), K._stream()), "nx_silu_mul")
 
 
-def softcap_(x, cols, cap) -> None:
+def glu(h, out, kind: Glu, *, interleaved=False) -> None:
+    """h: [rows, 2 F], gates and values in two halves or in turns of eight columns; out: [rows, F]."""
+    K._check(K.lib().nx_glu(K._p(h), C.c_int64(h.stride(0)), K._p(out), C.c_int64(out.stride(0)), C.c_int(h.shape[0]),
+                            C.c_int(h.shape[1] // 2), C.c_int(int(interleaved)), kind, C.c_int(_dt(h)), K._stream()), "nx_glu")
+
+
+def softcap_(x, cols, cap, scale=1.0) -> None:
+    """x = cap * tanh(scale * x / cap) in place (cap 0: x = scale * x)."""
     for r0 in range(0, x.shape[0], 32768):
         part = x[r0: r0 + 32768]
         K._check(K.lib().nx_softcap(K._p(part), C.c_int64(part.stride(0)), C.c_int(part.shape[0]), C.c_int(cols), C.c_float(cap),
-                                    K._stream()), "nx_softcap")
+                                    C.c_float(scale), K._stream()), "nx_softcap")
 
 
 def paged_window_attention(q, k_cache, v_cache, block_table, out, seg: Segments, *, heads, block_size, window, scale,
-                           softcap=0.0, out_scale=1.0, splits=1, gate=None, vdim=0) -> None:
+                           softcap=0.0, out_scale=1.0, splits=1, gate=None, vdim=0, keep_first=0, sink=None) -> None:
     """q: [rows, heads * dim] view; caches [blocks, block_size, kv_heads, dim | vdim]; out [rows, heads * vdim] view.
     One-row segments run the decode kernel, longer ones the prompt kernel (BF16); FP32 has one kernel for both.
     ``vdim`` > 0: a latent cache, the values are the leading ``vdim`` columns of the keys (``v_cache`` is not used).
-    ``gate``: FP32 [rows, heads] factor of the output."""
+    ``gate``: FP32 [rows, heads] factor of the output.  ``keep_first``: the first keys stay visible; ``sink``: FP32 [heads], a
+    score that counts in the denominator only."""
     G, D = k_cache.shape[2], k_cache.shape[3]
     if vdim:
         v_cache = k_cache
@@ -249,7 +327,7 @@ def paged_window_attention(q, k_cache, v_cache, block_table, out, seg: Segments,
     Dv = vdim or v_cache.shape[3]
     a = PagedWindowArgs(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(out), q.stride(0), out.stride(0), None,
                         None, heads, G, D, Dv, block_size, block_table.shape[1], window, 1, _dt(q), scale, softcap, out_scale,
-                        seg.args(), k_cache.stride(1), v_cache.stride(1), _ptr(gate))
+                        seg.args(), k_cache.stride(1), v_cache.stride(1), _ptr(gate), _ptr(sink), keep_first)
     if q.dtype == torch.float32:
         K._check(K.lib().nx_paged_window_f32(C.byref(a), K._stream()), "nx_paged_window_f32")
     elif seg.max_len == 1:
@@ -285,8 +363,18 @@ def latent_prompt(q, kv, lat, out, blocks, *, heads, dim, rot, vdim, rank, windo
     K._check(K.lib().nx_latent_prompt(C.byref(a), K._stream()), "nx_latent_prompt")
 
 
+def window_prompt(q, k, v, out, blocks, *, heads, kv_heads, dim, vdim, window, scale, keep_first=0, kept=None, sink=None) -> None:
+    """The tcgen05 form on plain grouped keys and values.  q [rows, heads * dim], k [kv rows, kv_heads * dim], v [kv rows, kv_heads *
+    vdim]; blocks as in `latent_prompt`; kept int32 [n]: the row that position 0 has among the kept first keys (None: the block's)."""
+    a = WindowPromptArgs(_ptr(q), _ptr(k), _ptr(v), _ptr(out), _ptr(sink), _ptr(blocks), _ptr(kept),
+                         K.status_word(q.device).data_ptr(), q.stride(0), k.stride(0), v.stride(0), out.stride(0), blocks.shape[0],
+                         q.shape[0], k.shape[0], heads, kv_heads, dim, vdim, window, keep_first, scale)
+    K._check(K.lib().nx_window_prompt(C.byref(a), K._stream()), "nx_window_prompt")
+
+
 def latent_gather(cache, block_table, runs, longest, dst) -> None:
-    """Cache rows of ``runs`` (int32 [n, 4]: first row of ``dst``, rows, first position, sequence) into ``dst`` [., row]."""
+    """Cache rows of ``runs`` (int32 [n, 4]: first row of ``dst``, rows, first position, sequence) into ``dst`` [., row]; cache
+    [blocks, block_size, 1, row], or keys or values [blocks, block_size, heads, size] whose rows are heads * size wide."""
     K._check(K.lib().nx_latent_gather(K._p(cache), K._p(dst), K._p(block_table), K._p(runs), C.c_int(runs.shape[0]), C.c_int(longest),
-                                      C.c_int(block_table.shape[1]), C.c_int(cache.shape[1]), C.c_int(cache.shape[-1]), K._stream()),
-             "nx_latent_gather")
+                                      C.c_int(block_table.shape[1]), C.c_int(cache.shape[1]), C.c_int(cache.shape[2] * cache.shape[3]),
+                                      K._stream()), "nx_latent_gather")

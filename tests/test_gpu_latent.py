@@ -352,7 +352,7 @@ def _prompt_ref(q, kv, lat, segs, H, dim, rot, vdim, rank, window, scale, gate):
 
 
 def _blocks(segs, window):
-    from nexus_b200.infer.latent import long_segments
+    from nexus_b200.infer.prompt import long_segments
     out = []
     for r0, n, p0, kv0 in segs:
         for b in long_segments([(r0, n, 0, 0)], window)[0]:

@@ -106,7 +106,7 @@ def test_yarn_frequencies():
 @pytest.mark.parametrize("window", [0, 1, 40, 300, 5000])
 def test_blocks_and_runs_of_long_segments(window):
     """Every query row is in one block; the kv row of every key a row can see is the one the runs put it in."""
-    from nexus_b200.infer.latent import QUERY_BLOCK, long_segments
+    from nexus_b200.infer.prompt import QUERY_BLOCK, long_segments
     back = window - 1 if window else 10 ** 6
     for segs in ([(0, 17, 0, 3), (17, 600, 0, 1)], [(5, 17, 900, 2), (22, 256, 0, 0), (300, 257, 31, 1)]):
         blocks, runs, kv_rows = long_segments(segs, window)
@@ -121,9 +121,9 @@ def test_blocks_and_runs_of_long_segments(window):
                 assert first + k not in held
                 held[first + k] = (seq, base + k)
         assert len(held) == kv_rows and (kv_rows > 0) == any(s[2] > 0 for s in segs)
-        for row0, count, pos0, kv0 in blocks:
+        for row0, count, pos0, kv0, kept0 in blocks:
             s = next(s for s in segs if s[0] <= row0 < s[0] + s[1])
-            assert pos0 == s[2] + row0 - s[0]
+            assert pos0 == s[2] + row0 - s[0] and kept0 == kv0
             for pos in (pos0, pos0 + count - 1):
                 for key in {max(0, pos - back), pos}:
                     if runs:
