@@ -184,3 +184,100 @@ def forward(cfg, weights, tokens, dtype=torch.float64, capture=None):
             capture.append(x.clone())
     z = offset_norm(x, w["final.norm"], eps) @ w["head"].T * cfg["logit_scale"]
     return cfg["logit_softcap"] * torch.tanh(z / cfg["logit_softcap"])
+
+
+# ---------------------------------------------------------------------------------------------- random models
+def dense_ff(ff=44):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe_ff(experts=6, top=2, ff=28, limit=0.8, groups=(3, 2)):
+    router = {"experts": experts, "top": top}
+    if groups is not None:
+        router["groups"] = {"count": groups[0], "keep": groups[1]}
+    return {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": router}
+
+
+def attention_layer(mlp, heads=6, kv_heads=2, dim=24, vdim=20, conv=4, scale=0.22, window=21, keep=5, rot=16, base=4000.0, v_mix=True):
+    return {"type": "attention", "mlp": mlp,
+            "mixer": {"conv": conv, "dim": dim, "heads": heads, "kv_heads": kv_heads, "mask": {"keep_first": keep, "size": window},
+                      "rot": {"base": base, "dims": rot}, "scale": scale, "v_mix": v_mix, "vdim": vdim}}
+
+
+def latent_layer(mlp, heads=5, dim=24, rot_dim=16, vdim=20, kv_rank=56, scale=0.19, window=17, base=7000.0):
+    return {"type": "latent_attention", "mlp": mlp,
+            "mixer": {"dim": dim, "heads": heads, "kv_rank": kv_rank, "mask": {"size": window}, "rot": {"base": base, "dims": rot_dim},
+                      "rot_dim": rot_dim, "scale": scale, "vdim": vdim}}
+
+
+def gla_layer(mlp, heads=3, dim=24, vdim=20, tau=8.0):
+    return {"type": "gla", "mlp": mlp, "mixer": {"dim": dim, "heads": heads, "tau": tau, "vdim": vdim}}
+
+
+def random_config(layers=None, vocab=181, width=88, eps=1e-4, scale=1.7, softcap=9.0):
+    layers = layers or [attention_layer(moe_ff()), gla_layer(dense_ff()), latent_layer(None), attention_layer(moe_ff(groups=None)),
+                        gla_layer(moe_ff())]
+    return {"architecture": "Gutivik", "layers": layers, "logit_scale": scale, "logit_softcap": softcap, "norm": {"eps": eps},
+            "vocab": vocab, "width": width}
+
+
+ROUTED = 6      # columns of the residual stream that only the embedding writes and only routers read
+
+
+def random_weights(cfg, seed=0, rank=5):
+    """Routers read a sign pattern that every token carries in the first columns, where no layer writes: their choices rest on no
+    close call that rounding could turn."""
+    g = torch.Generator().manual_seed(seed)
+    W, V = cfg["width"], cfg["vocab"]
+
+    def n(*shape, s=1.0):
+        return torch.randn(*shape, generator=g) * s / math.sqrt(shape[-1])
+
+    def reads(*shape, s=1.0):
+        w = n(*shape, s=s)
+        w[:, :ROUTED] = 0
+        return w
+
+    def writes(*shape):
+        w = n(*shape)
+        w[:ROUTED] = 0
+        return w
+
+    def norm(size, mean):
+        return mean + 0.3 * torch.randn(size, generator=g)
+    embed = torch.randn(V, W, generator=g)
+    embed[:, :ROUTED] = torch.randint(0, 2, (V, ROUTED), generator=g) * 4.0 - 2.0
+    out = {"embed": embed, "final.norm": norm(W, 0.0), "head": n(V, W)}
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", layer["mixer"], layer["mlp"]
+        H, D, Dv = m["heads"], m["dim"], m["vdim"]
+        out[p + "norm1"] = norm(W, 0.0)
+        if layer["type"] == "latent_attention":
+            R, C = m["rot_dim"], m["kv_rank"]
+            out.update({p + "mix.q": reads(H * (D + R), W, s=1.6), p + "mix.dkv": reads(C + R, W), p + "mix.dkv.norm": norm(C, 1.0),
+                        p + "mix.uk": n(H * D, C, s=1.6), p + "mix.uv": n(H * Dv, C), p + "mix.o": writes(W, H * Dv)})
+        elif layer["type"] == "attention":
+            G = m["kv_heads"]
+            for name, size in (("q", H * D), ("k", G * D), ("v", G * Dv)):
+                out[p + "mix." + name], out[p + f"mix.{name}.b"] = reads(size, W, s=1.5), 0.4 * torch.randn(size, generator=g)
+                out[p + f"mix.{name}.conv"] = n(size, m["conv"], s=1.5)
+            out[p + "mix.sink"], out[p + "mix.o"] = torch.randn(H, generator=g), writes(W, H * Dv)
+            if m["v_mix"]:
+                out[p + "mix.vmix"] = torch.tensor(0.3 + 0.1 * i)
+        else:
+            out.update({p + "mix.q": reads(H * D, W), p + "mix.k": reads(H * D, W), p + "mix.v": reads(H * Dv, W), p + "mix.g": reads(H * Dv, W),
+                        p + "mix.o": writes(W, H * Dv), p + "mix.norm": norm(Dv, 1.0), p + "mix.a1": reads(rank, W),
+                        p + "mix.a2": n(H * D, rank, s=1.5), p + "mix.a2.b": torch.linspace(-4.0, 5.0, H * D)})
+        if f is None:
+            continue
+        out[p + "norm2"] = norm(W, 0.0)
+        if f["kind"] == "dense":
+            out[p + "mlp.gate"], out[p + "mlp.up"], out[p + "mlp.down"] = reads(f["ff"], W), reads(f["ff"], W), writes(W, f["ff"])
+            continue
+        E, F = f["router"]["experts"], f["expert"]["ff"]
+        for e in range(E):
+            out[p + f"mlp.e{e}.gate"], out[p + f"mlp.e{e}.up"], out[p + f"mlp.e{e}.down"] = reads(F, W), reads(F, W), writes(W, F)
+        router = torch.zeros(E, W)
+        router[:, :ROUTED] = torch.randn(E, ROUTED, generator=g) * 0.6
+        out[p + "mlp.router"], out[p + "mlp.correction"] = router, torch.randn(E, generator=g) * 0.4 - 0.5
+    return {k: v.to(torch.bfloat16) for k, v in out.items()}
