@@ -15,6 +15,7 @@
 //
 // Replaces the reference's cuBLASLt layer and its epilogues Bias / BiasGelu(+aux) / DGelu /
 // beta=1 accumulate (include/nexus/cuda/gemm.hpp:38-121, src/cuda/gemm_lt.cpp:260-360).
+#include "glu.cuh"
 #include "nx_api_comm.h"
 #include "sm100_ptx.cuh"
 #include "tensor_map.h"
@@ -76,6 +77,8 @@ struct DevParams {
   unsigned int* amax_out;  // max |out| as float bits (may be null)
   int tma_store;           // BF16 out (and aux_out) leave through shared memory and tiled TMA stores
   int n_fastest;           // consecutive work units walk along N (A tile reused from L2) instead of along M
+  int gated;               // the lean epilogue of the pair kernel only: n / 2 output columns
+  NxGlu glu;
   const int32_t* row_groups;  // grouped form: which B each block of `group_rows` rows meets (negative: none)
   int group_rows;
   // All-gather fused into the GEMM (nx_gemm_ag): A is this rank's [M][lda] gather buffer; the last `ag_copiers`
@@ -231,6 +234,19 @@ __device__ __forceinline__ void stage_row32_bf16(uint8_t* buf, int r, const floa
     q.z = pack_bf16x2(v[8 * i + 4], v[8 * i + 5]);
     q.w = pack_bf16x2(v[8 * i + 6], v[8 * i + 7]);
     *reinterpret_cast<uint4*>(buf + r * 64 + ((i ^ ((r >> 1) & 3)) << 4)) = q;
+  }
+}
+
+// 16 columns of a staging row: its first or its second half
+__device__ __forceinline__ void stage_row16_bf16(uint8_t* buf, int r, int half, const float (&v)[16]) {
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    uint4 q;
+    q.x = pack_bf16x2(v[8 * i + 0], v[8 * i + 1]);
+    q.y = pack_bf16x2(v[8 * i + 2], v[8 * i + 3]);
+    q.z = pack_bf16x2(v[8 * i + 4], v[8 * i + 5]);
+    q.w = pack_bf16x2(v[8 * i + 6], v[8 * i + 7]);
+    *reinterpret_cast<uint4*>(buf + r * 64 + (((half * 2 + i) ^ ((r >> 1) & 3)) << 4)) = q;
   }
 }
 
@@ -783,6 +799,32 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
             __syncwarp();
             if (lane == 0) mbar_arrive_cluster(mapa_shared(smem_u32(&tempty_bar[acc]), 0));
             released = true;
+          }
+          if (p.gated) {
+            // two chunks of eight gates and eight values in turn make the 32 columns of one staging tile
+            const int second = (c - c_begin) & 1;
+            if (gpos == 0 && !second) {
+              if (lane == 0) tma_store_wait_read<0>();
+              __syncwarp();
+              gcol0 = col0 / 2;
+            }
+            float o[16];
+#pragma unroll
+            for (int j = 0; j < 16; ++j) o[j] = glu_apply<false>(p.glu, v[(j / 8) * 16 + j % 8], v[(j / 8) * 16 + 8 + j % 8]);
+            stage_row16_bf16(st_base + gpos * 2048, lane, second, o);
+            if (second || last_chunk) ++gpos;       // columns past the matrix are clipped by the store
+            if (gpos > 0 && (gpos == group || last_chunk)) {
+              fence_proxy_async_smem();
+              __syncwarp();
+              if (lane == 0 && row0 < p.m) {
+                for (int g = 0; g < gpos; ++g)
+                  if (NX_INDEX_OK(gcol0 + 32 * g >= 0 && 2 * (gcol0 + 32 * g) < p.n && ((gcol0 + 32 * g) & 7) == 0 && row0 >= 0, p.status))
+                    tma_store_3d(&tmap_out, st_base + g * 2048, gcol0 + 32 * g, row0, w.batch);
+                tma_store_commit();
+              }
+              gpos = 0;
+            }
+            continue;
           }
           if (gpos == 0) {
             // the staging tiles are free once the previous group's stores have read them (long ago, as a rule)
@@ -1337,6 +1379,12 @@ int gemm_impl(const NxGemmArgs* a, const NxGemmAg* ag, nx_stream_t stream_, cons
   static bool pair_ok = true;  // cleared when the device cannot place clusters of two
   const bool pair = bn == 256 && !fp8 && a->m >= 2 * kBM && pair_ok && (!single_only || ag != nullptr || rs != nullptr) &&
                     (a->max_ctas <= 0 || a->max_ctas >= 2) && !(grouped && a->group_rows < 2 * kBM);
+  const bool gated = a->glu != nullptr;
+  if (gated && (!pair || ag != nullptr || rs != nullptr || a->in_dtype != NX_BF16 || a->out_dtype != NX_BF16 || (a->n & 15) || split > 1 ||
+                batch != 1 || a->bias != nullptr || a->residual != nullptr || a->aux_in != nullptr || a->aux_out != nullptr ||
+                a->accumulate || a->act != NX_ACT_NONE || a->alpha != 1.0f || a->scale_a != nullptr || a->scale_b != nullptr ||
+                a->amax_out != nullptr))
+    return -1;
   if ((ag != nullptr || rs != nullptr) && !pair) return -3;  // the fused forms run on the CTA-pair kernel only
   const int tile_m = pair ? 2 * kBM : kBM;
 
@@ -1362,6 +1410,8 @@ int gemm_impl(const NxGemmArgs* a, const NxGemmAg* ag, nx_stream_t stream_, cons
   p.n = a->n;
   p.k = a->k;
   p.batch = batch;
+  p.gated = gated ? 1 : 0;
+  if (gated) p.glu = *a->glu;
   p.row_groups = a->row_groups;
   p.group_rows = grouped ? a->group_rows : 1;
   p.out_dtype = a->out_dtype;
@@ -1430,8 +1480,8 @@ int gemm_impl(const NxGemmArgs* a, const NxGemmAg* ag, nx_stream_t stream_, cons
   static const bool direct_only = std::getenv("NX_GEMM_DIRECT_STORE") != nullptr;  // measurement switch
   if (can_tma_out && !direct_only) {
     const uint64_t so = batch > 1 ? static_cast<uint64_t>(a->stride_o) : 0;
-    rc = nx::make_tensor_map_3d(&to, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a->out, a->n, a->m, batch, a->ldo, so, 32, 32,
-                                CU_TENSOR_MAP_SWIZZLE_64B);
+    rc = nx::make_tensor_map_3d(&to, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a->out, gated ? a->n / 2 : a->n, a->m, batch, a->ldo, so, 32,
+                                32, CU_TENSOR_MAP_SWIZZLE_64B);
     if (rc == 0 && a->aux_out != nullptr)
       rc = nx::make_tensor_map_3d(&tx, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a->aux_out, a->n, a->m, 1, a->ld_aux, 0, 32, 32,
                                   CU_TENSOR_MAP_SWIZZLE_64B);
@@ -1463,6 +1513,7 @@ int gemm_impl(const NxGemmArgs* a, const NxGemmAg* ag, nx_stream_t stream_, cons
       p.rs_done = rs->done;
       for (int q = 0; q < rs->n_ranks; ++q) p.rs_slots[q] = rs->slots[q];
     }
+    if (gated && (generic_only || !p.tma_store)) return -1;
     const bool fast = (rs != nullptr || !generic_only) && p.tma_store && a->residual == nullptr && a->scale_a == nullptr &&
                       a->scale_b == nullptr && a->amax_out == nullptr && (reinterpret_cast<uintptr_t>(a->bias) & 15) == 0 &&
                       (a->aux_in == nullptr || (reinterpret_cast<uintptr_t>(a->aux_in) & 15) == 0) &&

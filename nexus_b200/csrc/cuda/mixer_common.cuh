@@ -2,6 +2,7 @@
 // warp-level BF16 tensor-core tile (m16n8k16) with its shared-memory fragment loads.
 #pragma once
 #include "common.cuh"
+#include "glu.cuh"
 #include "nx_api_mixers.h"
 
 namespace nx {
@@ -46,25 +47,7 @@ __device__ __forceinline__ void store_vec(T* p, const float (&v)[V]) {
 }
 
 __device__ __forceinline__ float silu_exact(float x) { return x / (1.0f + expf(-x)); }
-__device__ __forceinline__ float sigmoid_exact(float x) { return 1.0f / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus_exact(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
-__device__ __forceinline__ float gelu_tanh_exact(float x) {
-  return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
-}
-
-// gated activations; kExact: full FP32 accuracy, else the fast exponential and division (results are rounded to BF16)
-template <bool kExact>
-__device__ __forceinline__ float sigmoid_as(float x) {
-  return kExact ? sigmoid_exact(x) : __fdividef(1.0f, 1.0f + __expf(-x));
-}
-template <bool kExact>
-__device__ __forceinline__ float glu_apply(const NxGlu& f, float g, float u) {
-  if (f.kind == NX_GLU_SILU) return g * sigmoid_as<kExact>(g) * u;
-  if (f.kind == NX_GLU_GELU) return gelu_tanh_exact(g) * u;
-  g = fminf(g, f.limit);
-  u = fminf(fmaxf(u, -f.limit), f.limit);
-  return g * sigmoid_as<kExact>(f.slope * g) * (u + f.offset);
-}
 
 // the hardware exponential and reciprocal (results below the normal range flush to zero)
 __device__ __forceinline__ float ex2_approx(float x) {

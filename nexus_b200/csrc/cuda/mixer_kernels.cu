@@ -532,7 +532,8 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 decay_gate_kernel(const T* __restrict__ a, int64_t lda, const float* __restrict__ w, const float* __restrict__ bias,
                   float* __restrict__ out, int64_t ldo, int rows, int cols, int rank, float mul) {
-  __shared__ float s_w[kDecayRank][kDecayCols + 1], s_a[kDecayRows][kDecayRank];
+  __shared__ float s_w[kDecayRank][kDecayCols + 1];
+  __shared__ __align__(16) float s_a[kDecayRows][kDecayRank];
   const int c0 = blockIdx.x * kDecayCols, tx = threadIdx.x % kDecayCols, ty = threadIdx.x / kDecayCols, c = c0 + tx;
   const int64_t r0 = static_cast<int64_t>(blockIdx.y) * kDecayRows;
   float acc[16];
@@ -549,12 +550,16 @@ decay_gate_kernel(const T* __restrict__ a, int64_t lda, const float* __restrict_
       s_a[row][k] = r0 + row < rows && k0 + k < rank ? Num<T>::load(a + (r0 + row) * lda + k0 + k) : 0.0f;
     }
     __syncthreads();
+    float wk[kDecayRank];
 #pragma unroll
-    for (int k = 0; k < kDecayRank; ++k) {
-      const float wk = s_w[k][tx];
+    for (int k = 0; k < kDecayRank; ++k) wk[k] = s_w[k][tx];
 #pragma unroll
-      for (int i = 0; i < 16; ++i) acc[i] = fmaf(s_a[ty * 16 + i][k], wk, acc[i]);
-    }
+    for (int i = 0; i < 16; ++i)
+#pragma unroll
+      for (int k = 0; k < kDecayRank; k += 4) {
+        const float4 v = *reinterpret_cast<const float4*>(&s_a[ty * 16 + i][k]);     // the same for the whole warp
+        acc[i] = fmaf(v.x, wk[k], fmaf(v.y, wk[k + 1], fmaf(v.z, wk[k + 2], fmaf(v.w, wk[k + 3], acc[i]))));
+      }
   }
   if (c >= cols) return;
   const float b = bias[c];

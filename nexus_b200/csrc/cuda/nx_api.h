@@ -18,6 +18,16 @@ enum NxDType { NX_BF16 = 0, NX_F32 = 1, NX_F16 = 2, NX_E4M3 = 3, NX_E5M2 = 4 };
 enum NxAct { NX_ACT_NONE = 0, NX_ACT_GELU = 1, NX_ACT_RELU = 2, NX_ACT_DGELU = 3, NX_ACT_SILU = 4,
              NX_ACT_RELU2 = 5 /* square of relu */ };
 
+// Gated activations of a gate g and a value u:  NX_GLU_SILU silu(g) u,  NX_GLU_GELU gelu_tanh(g) u,
+// NX_GLU_CLAMP with g' = min(g, limit), u' = clamp(u, -limit, limit): g' sigmoid(slope g') (u' + offset).
+#define NX_GLU_SILU 0
+#define NX_GLU_GELU 1
+#define NX_GLU_CLAMP 2
+typedef struct NxGlu {
+  int32_t kind;
+  float limit, slope, offset;
+} NxGlu;
+
 // out[b][m][n] = epilogue( alpha * sum_k A[b][m][k] * B[b][n][k] )
 // Operand memory: a_mn_major == 0 -> A is [M][lda] (K contiguous); 1 -> A is [K][lda] (M contiguous).
 //                 b_mn_major == 0 -> B is [N][ldb] (K contiguous); 1 -> B is [K][ldb] (N contiguous).
@@ -56,6 +66,9 @@ typedef struct NxGemmArgs {
   // captured graph.  No split-K, no FP8.
   const int32_t* row_groups;
   int32_t group_rows;
+  // Gated output, may be null: the N columns are turns of eight gates and eight values, out has N / 2 columns.  BF16 operands
+  // and output, M and N of at least 256, M-tiles of 256 rows, no bias, residual, aux, act or accumulation.
+  const NxGlu* glu;
 } NxGemmArgs;
 
 int nx_gemm(const NxGemmArgs* args, nx_stream_t stream);

@@ -222,16 +222,8 @@ int nx_token_side_gate(const float* a, int64_t lda, const int32_t* tokens, const
                        void* out, int64_t ldo, int rows, int dim, int dtype, nx_stream_t stream);
 // out[r][j] = silu(h[r][j]) * h[r][half + j], j < half
 int nx_silu_mul(const void* h, int64_t ldh, void* out, int64_t ldo, int rows, int half, int dtype, nx_stream_t stream);
-// Gated activations of a gate g and a value u:  NX_GLU_SILU silu(g) u,  NX_GLU_GELU gelu_tanh(g) u,
-// NX_GLU_CLAMP with g' = min(g, limit), u' = clamp(u, -limit, limit): g' sigmoid(slope g') (u' + offset).
-// half: columns of the output; g and u lie in two halves of h, or (interleaved) in turns of eight columns, gates first.
-#define NX_GLU_SILU 0
-#define NX_GLU_GELU 1
-#define NX_GLU_CLAMP 2
-typedef struct NxGlu {
-  int32_t kind;
-  float limit, slope, offset;
-} NxGlu;
+// Gated activation; half: columns of the output; gates and values lie in two halves of h, or (interleaved) in turns of eight
+// columns, gates first.
 int nx_glu(const void* h, int64_t ldh, void* out, int64_t ldo, int rows, int half, int interleaved, NxGlu glu, int dtype,
            nx_stream_t stream);
 // x = cap * tanh(scale * x / cap) in place on FP32 [rows, ld]; cap 0: x = scale * x

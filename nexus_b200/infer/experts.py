@@ -6,8 +6,8 @@ rows; above, the residual kernel (or the routing kernel) writes every row to its
 groups of row tiles.  The kernel that adds the sublayer's output to the residual stream sums a token's experts, with the
 router's weights, and its gated shared expert on the way.
 
-Gated experts keep W_gate and W_up as one matrix in turns of eight rows, so that the few-rows product has a unit's gate and value
-in one thread."""
+Gated experts keep W_gate and W_up as one matrix in turns of eight rows, so that a unit's gate and value meet in one thread of the
+few-rows product and of the GEMM's epilogue."""
 from __future__ import annotations
 
 from typing import List, Optional
@@ -30,6 +30,13 @@ def _stack(parts) -> torch.Tensor:
     return w
 
 
+def in_turns(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+    """[..., n, k] gates and values as [..., 2 n, k] in turns of eight rows, gates first; n is padded to a multiple of 8."""
+    pad = (0, 0, 0, -gate.shape[-2] % 8)
+    both = torch.stack([torch.nn.functional.pad(t.float(), pad).unflatten(-2, (-1, 8)) for t in (gate, up)], -3)
+    return both.flatten(-4, -2)
+
+
 def load(engine, f: ExpertsSpec, get) -> dict:
     """``get(name)``: the feed-forward's tensors."""
     out = {}
@@ -41,8 +48,7 @@ def load(engine, f: ExpertsSpec, get) -> dict:
     for name in ("up", "down"):
         w = _stack([get(f"e{e}.{name}") for e in range(f.experts)])
         if f.glu is not None and name == "up":
-            both = torch.stack([_stack([get(f"e{e}.gate") for e in range(f.experts)]), w], 1)       # [experts, 2, rows, columns]
-            w = both.view(f.experts, 2, -1, 8, w.shape[2]).transpose(1, 2).reshape(f.experts, -1, w.shape[2])
+            w = in_turns(_stack([get(f"e{e}.gate") for e in range(f.experts)]), w)
         out[name] = w.to(engine.dev, engine.adt).contiguous()
         engine.weight_nbytes += out[name].numel() * out[name].element_size()
     if f.shared:

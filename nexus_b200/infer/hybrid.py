@@ -25,7 +25,7 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from ..lm.config import RopeScaling
-from ..lm.hybrid import ConvAttentionSpec, DeltaSpec, GlaSpec, HybridConfig, HybridWeights, LatentSpec, ParallelSpec
+from ..lm.hybrid import GLU_ACTS, ConvAttentionSpec, DeltaSpec, GlaSpec, HybridConfig, HybridWeights, LatentSpec, ParallelSpec
 from ..lm.rope import rope_inv_freq
 from . import conv_attention, experts, gla, latent, prompt
 from .engine import Chunk, Engine, _Linear
@@ -163,7 +163,7 @@ class HybridEngine(Engine):
             if layer.experts:
                 out["ff"] = experts.load(self, layer.experts, lambda n: t[p + "mlp." + n])
             if layer.ff:
-                out["up"], _ = self._pack([t[p + "mlp.gate"], t[p + "mlp.up"]])
+                out["up"], _ = self._pack([experts.in_turns(t[p + "mlp.gate"], t[p + "mlp.up"])])
                 out["down"], _ = self._pack([t[p + "mlp.down"]])
             if model.token_side:
                 out["side_gate"], _ = self._pack([t[p + "side.gate"]])
@@ -352,6 +352,17 @@ class HybridEngine(Engine):
                      gate_first=False, eps=self.model.norm_eps)
         return self._linear(out, lw["out"])
 
+    def _gated(self, h, lin: _Linear, glu) -> torch.Tensor:
+        """Gated activation of a product whose columns are turns of eight gates and eight values."""
+        from ..ops import _cuda as K
+        from ..ops import _mixers as M
+        if self.fast and K.gated_gemm_ok(h.shape[0], lin.n):
+            return K.gated_gemm(h, lin.w, glu)
+        both = self._linear(h, lin)
+        act = torch.empty((h.shape[0], lin.n // 2), dtype=self.adt, device=self.dev)
+        M.glu(both, act, glu, interleaved=True)
+        return act
+
     def _mixer(self, i: int, m, lw: dict, h, pos, slot) -> torch.Tensor:
         if isinstance(m, LatentSpec):
             return latent.mixer(self, i, m, lw["mix"], h, pos, slot)
@@ -395,12 +406,7 @@ class HybridEngine(Engine):
                        "weights": r.weight, "y_gate": gate if f.shared else None}
             elif layer.ff:
                 M.residual_norm(x, y=y, eps=eps, res_mult=mult, **add, **feed(lw["pre2"]))
-                gu = self._linear(h, lw["up"])
-                act = torch.empty((n, gu.shape[1] // 2), dtype=self.adt, device=self.dev)
-                if layer.act == "silu":
-                    M.silu_mul(gu, act)
-                else:
-                    M.glu(gu, act, M.Glu(1))
+                act = self._gated(h, lw["up"], M.Glu(GLU_ACTS.index(layer.act)))
                 y, add = self._linear(act, lw["down"]), {"w_post": lw["post2"]}
             M.residual_norm(x, y=y, eps=eps, res_mult=mult, **add, **after)
             if model.token_side:

@@ -43,7 +43,7 @@ class GemmArgs(C.Structure):
         ("act", C.c_int32), ("accumulate", C.c_int32), ("split_k", C.c_int32), ("block_n", C.c_int32),
         ("alpha", C.c_float), ("max_ctas", C.c_int32), ("b_dtype_plus1", C.c_int32),
         ("scale_a", C.c_void_p), ("scale_b", C.c_void_p), ("amax_out", C.c_void_p),
-        ("row_groups", C.c_void_p), ("group_rows", C.c_int32),
+        ("row_groups", C.c_void_p), ("group_rows", C.c_int32), ("glu", C.c_void_p),
     ]
 
 
@@ -295,10 +295,36 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn: bool = False, b_mn: bool = F
 
 
 # -------------------------------------------------------------------------------------------- norms
+class Glu(C.Structure):
+    """A gated activation: ``kind`` 0 silu(g) u, 1 gelu_tanh(g) u, 2 clamped (limit, slope, offset)."""
+    _fields_ = [("kind", C.c_int32), ("limit", C.c_float), ("slope", C.c_float), ("offset", C.c_float)]
+
+
+def gated_gemm_ok(rows: int, n: int) -> bool:
+    """Whether a product of these sizes can apply a gated activation in its epilogue."""
+    return rows >= 256 and n >= 256 and n % 16 == 0
+
+
+def gated_gemm(a: torch.Tensor, b: torch.Tensor, glu: Glu) -> torch.Tensor:
+    """glu(a b^T) for BF16 a [M, K] and b [N, K] whose rows are turns of eight gates and eight values: [M, N / 2]."""
+    (m, k), n = a.shape, b.shape[0]
+    out = torch.empty((m, n // 2), dtype=a.dtype, device=a.device)
+    g = GemmArgs()
+    g.a, g.b, g.out = a.data_ptr(), b.data_ptr(), out.data_ptr()
+    g.lda, g.ldb, g.ldo = a.stride(0), b.stride(0), out.stride(0)
+    g.m, g.n, g.k, g.batch = m, n, k, 1
+    g.in_dtype, g.out_dtype = _DT[a.dtype], _DT[out.dtype]
+    g.alpha, g.split_k, g.glu = 1.0, 1, C.addressof(glu)
+    g.status = status_word(a.device).data_ptr()
+    _check(lib().nx_gemm(C.byref(g), _stream()), "nx_gemm")
+    return out
+
+
 def grouped_gemm(a: torch.Tensor, b: torch.Tensor, groups: torch.Tensor, group_rows: int, *, act: Optional[str] = None,
-                 out: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+                 out: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None, glu: Optional[Glu] = None) -> torch.Tensor:
     """Rows ``i * group_rows ..`` of ``a`` [M, K] times ``b[groups[i]]`` ([groups, N, K]); a negative entry skips the rows.
-    ``groups``: int32 on the device, one entry per ``group_rows`` (128 or 256) rows."""
+    ``groups``: int32 on the device, one entry per ``group_rows`` (128 or 256) rows.  ``glu`` (256 rows, `gated_gemm_ok`): the N
+    columns are turns of eight gates and eight values, ``out`` has N / 2."""
     m, k = a.shape
     batch, n, kb = b.shape
     if k != kb or a.stride(1) != 1 or b.stride(2) != 1 or a.dtype != b.dtype or a.dtype != torch.bfloat16:
@@ -314,6 +340,8 @@ def grouped_gemm(a: torch.Tensor, b: torch.Tensor, groups: torch.Tensor, group_r
     g.in_dtype, g.out_dtype = _DT[a.dtype], _DT[out.dtype]
     g.act, g.alpha, g.split_k = ACT[act], 1.0, 1
     g.row_groups, g.group_rows = groups.data_ptr(), group_rows
+    if glu is not None:
+        g.glu = C.addressof(glu)
     g.status = status_word(a.device).data_ptr()
     _check(lib().nx_gemm(C.byref(g), _stream()), "nx_gemm")
     return out

@@ -118,6 +118,9 @@ def expert_product(x: torch.Tensor, w: torch.Tensor, route: Route, *, gather: bo
     (whose x is in slot order)."""
     E, n, k = w.shape
     few = x.dtype == torch.bfloat16 and route.align < 128
+    if gate is not None and not few and route.align == 256 and K.gated_gemm_ok(route.max_slots, n):
+        out = torch.empty((route.max_slots, n // 2), dtype=x.dtype, device=x.device)
+        return K.grouped_gemm(x, w, route.groups, route.align, out=out, glu=gate)
     if gate is not None and not few:
         both = expert_product(x, w, route, gather=gather)
         out = torch.empty((route.max_slots, n // 2), dtype=x.dtype, device=x.device)

@@ -10,6 +10,7 @@ from typing import Optional
 import torch
 
 from . import _cuda as K
+from ._cuda import Glu
 
 CHUNK = 64            # tokens per chunk of the tensor-core recurrences
 CHUNK_MAX_KEY = 256   # their largest state size along the key dimension
@@ -62,11 +63,6 @@ class GlaArgs(C.Structure):
                 ("state", C.c_void_p), ("ld", C.c_int64), ("ld_decay", C.c_int64), ("ldo", C.c_int64), ("heads", C.c_int32),
                 ("dim", C.c_int32), ("vdim", C.c_int32), ("dtype", C.c_int32), ("q_scale", C.c_float), ("seg", SegmentArgs),
                 ("part_state", C.c_void_p), ("part_decay", C.c_void_p), ("parts", C.c_int32), ("span", C.c_int32)]
-
-
-class Glu(C.Structure):
-    """A gated activation: ``kind`` 0 silu(g) u, 1 gelu_tanh(g) u, 2 clamped (limit, slope, offset)."""
-    _fields_ = [("kind", C.c_int32), ("limit", C.c_float), ("slope", C.c_float), ("offset", C.c_float)]
 
 
 class SsdArgs(C.Structure):
