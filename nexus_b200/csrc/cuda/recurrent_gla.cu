@@ -10,8 +10,9 @@
 //   y_t  = sum_d q^_t 2^{R_0 + .. + R_{i-1}} S  +  sum_{s <= t} (sum_d q^_t F_ij k^_s) v_s,   t in sub-block i, s in j
 //          F_ij = 2^{R_{j+1} + .. + R_{i-1}} for j < i,   F_ii = 2^{-R_i}
 //   S'   : S = 2^{R_j} S + k^_j^T v_j for j = 0 .. 3
-// Only F_ii grows with the decay.  Where a sub-block decays by more than 2^60 its own 16 x 16 products are formed pair by pair
-// from the exponents' differences instead, so any decay is exact.
+// The ten 16 x 16 blocks of the inner sums are shared out among the warps and pass through shared memory.  Only F_ii grows with the
+// decay.  Where a sub-block decays by more than 2^60 its own products are formed pair by pair from the exponents' differences
+// instead, so any decay is exact.
 //
 // Precision: v is BF16 and enters as it is; q^, k^, S and the token-by-token products are FP32 values split into BF16 pairs
 // (value and rounding remainder), which keeps 16 bits of mantissa.
@@ -25,13 +26,16 @@ using namespace nx;
 constexpr int kCols = 64;              // value columns per block
 constexpr int kSub = 16;               // tokens per sub-block
 constexpr float kSafe = -60.0f;        // smallest R whose inverse is used
+constexpr int kBlocks = 10;            // (sub-block, earlier or same sub-block): block i (i + 1) / 2 + j
 
 template <int NP>
 struct Smem {
   static constexpr int LN = NP + 8, LP = kCols + 8;
   static constexpr int kQh = 0, kQl = kQh + kQ * LN, kKh = kQl + kQ * LN, kKl = kKh + kQ * LN, kV = kKl + kQ * LN,
                        kSh = kV + kQ * LP, kSl = kSh + NP * LP, kEnd = kSl + NP * LP;
-  static constexpr int kBytes = kEnd * 2 + 4 * NP * 4;
+  // the blocks of token products lie over q, whose last use is before theirs, where the rest leaves no room
+  static constexpr bool kOverQ = kEnd * 2 + 8 * NP * 4 + kBlocks * 1024 > 226 * 1024;
+  static constexpr int kBytes = kEnd * 2 + 8 * NP * 4 + (kOverQ ? 0 : kBlocks * 1024);
 };
 
 // a fragment pair (value, remainder) times one factor per column: f = columns qc, qc + 1, qc + 8, qc + 9
@@ -41,6 +45,32 @@ __device__ __forceinline__ void scale_pair(uint32_t (&h)[4], uint32_t (&l)[4], c
     const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(&h[r]), y = *reinterpret_cast<const __nv_bfloat162*>(&l[r]);
     const int i = (r >> 1) * 2;
     bf16_split((__low2float(x) + __low2float(y)) * f[i], (__high2float(x) + __high2float(y)) * f[i + 1], h[r], l[r]);
+  }
+}
+
+// G = (q of sub-block i, times `f` per channel where `scaled`) k^T of sub-block j, pairs of BF16
+template <int NP, typename Factor>
+__device__ __forceinline__ void block_product(float (&g)[2][4], const __nv_bfloat16* sQh, const __nv_bfloat16* sQl,
+                                              const __nv_bfloat16* sKh, const __nv_bfloat16* sKl, int i, int j, bool scaled, Factor factor) {
+  constexpr int LN = Smem<NP>::LN;
+#pragma unroll
+  for (int kk = 0; kk < NP / 16; ++kk) {
+    uint32_t qh[4], ql[4], bh[4], bl[4];
+    ldmatrix_x4(qh, addr_a<LN>(sQh, i * kSub, kk * 16));
+    ldmatrix_x4(ql, addr_a<LN>(sQl, i * kSub, kk * 16));
+    ldmatrix_x4(bh, addr_b<LN>(sKh, j * kSub, kk * 16));
+    ldmatrix_x4(bl, addr_b<LN>(sKl, j * kSub, kk * 16));
+    if (scaled) {
+      float f[4];
+      factor(kk, f);
+      scale_pair(qh, ql, f);
+    }
+    mma_bf16(g[0], qh, bh[0], bh[1]);
+    mma_bf16(g[1], qh, bh[2], bh[3]);
+    mma_bf16(g[0], qh, bl[0], bl[1]);
+    mma_bf16(g[1], qh, bl[2], bl[3]);
+    mma_bf16(g[0], ql, bh[0], bh[1]);
+    mma_bf16(g[1], ql, bh[2], bh[3]);
   }
 }
 
@@ -54,13 +84,15 @@ __global__ void __launch_bounds__(256, NP <= 64 ? 2 : 1) gla_chunk_kernel(const 
   extern __shared__ __align__(16) __nv_bfloat16 sm[];
   __nv_bfloat16 *sQh = sm + L::kQh, *sQl = sm + L::kQl, *sKh = sm + L::kKh, *sKl = sm + L::kKl, *sV = sm + L::kV, *sSh = sm + L::kSh,
                 *sSl = sm + L::kSl;
-  float* sR = reinterpret_cast<float*>(sm + L::kEnd);    // [4][NP]: log2 decay of every sub-block
+  float* sD = reinterpret_cast<float*>(sm + L::kEnd);    // [4][NP]: 2^R of every sub-block
+  float* sI = sD + 4 * NP;                               // [4][NP]: 2^-R
+  uint4* sG = L::kOverQ ? reinterpret_cast<uint4*>(sQh) : reinterpret_cast<uint4*>(sI + 4 * NP);   // [kBlocks][hi, lo][lane]
   __shared__ int s_far[2][4];                            // sub-blocks whose decay is not inverted, by chunk parity
   const int h = blockIdx.x / col_tiles, p0 = (blockIdx.x % col_tiles) * kCols, part = blockIdx.y, sg = blockIdx.z;
   const int len = a.seg.len[sg], t_begin = part * a.span, t_end = min(len, t_begin + a.span);
   if (t_begin >= len || (kLocal && t_end == len)) return;   // the last span's contribution is never needed
   const int D = a.dim, P = a.vdim, cols = min(kCols, P - p0);
-  const int warp = (threadIdx.x >> 5) & 3, cb = (threadIdx.x >> 7) * 32, lane = threadIdx.x & 31, qr = lane >> 2, qc = (lane & 3) * 2;
+  const int wid = threadIdx.x >> 5, warp = wid & 3, cb = (wid >> 2) * 32, lane = threadIdx.x & 31, qr = lane >> 2, qc = (lane & 3) * 2;
   const int64_t row0 = a.seg.row0[sg];
   const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q) + row0 * a.ld + static_cast<int64_t>(h) * D;
   const __nv_bfloat16* k = static_cast<const __nv_bfloat16*>(a.k) + row0 * a.ld + static_cast<int64_t>(h) * D;
@@ -68,16 +100,17 @@ __global__ void __launch_bounds__(256, NP <= 64 ? 2 : 1) gla_chunk_kernel(const 
   const float* dec = a.decay + row0 * a.ld_decay + static_cast<int64_t>(h) * D;
   const auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   const bool vec_d = (a.ld & 7) == 0 && (D & 7) == 0 && al(a.q) && al(a.k), vec_p = (a.ld & 7) == 0 && (P & 7) == 0 && al(a.v);
+  const bool vec_a = (a.ld_decay & 1) == 0 && (D & 1) == 0 && al(a.decay);
   const int64_t plane = static_cast<int64_t>(D) * P;
   float* pool = a.state + (static_cast<int64_t>(a.seg.seq[sg]) * a.heads + h) * plane;
   const int64_t unit = (static_cast<int64_t>(sg) * a.parts + part) * a.heads + h;
   float* part_state = a.parts > 1 ? a.part_state + unit * plane : nullptr;
-  float S[MT][4][4], total[MT][2];
+  float S[MT][4][4], total[MT][2];                       // total: decay of the span
   {
     const float* src = kLocal ? nullptr : a.parts > 1 ? part_state : (a.seg.pos[sg] == 0 ? nullptr : pool);
 #pragma unroll
     for (int m = 0; m < MT; ++m) {
-      total[m][0] = total[m][1] = 0.0f;
+      total[m][0] = total[m][1] = 1.0f;
 #pragma unroll
       for (int n = 0; n < 4; ++n)
 #pragma unroll
@@ -92,14 +125,37 @@ __global__ void __launch_bounds__(256, NP <= 64 ? 2 : 1) gla_chunk_kernel(const 
     load_tile<NP>(sKh, k + t0 * a.ld, a.ld, min(kQ, t_end - t0), D, vec_d);
     load_tile<kCols>(sV, v + t0 * a.ld, a.ld, min(kQ, t_end - t0), cols, vec_p);
   };
-  float raw[ITEMS][kSub];                                // log2 decays of the chunk to convert next: one channel, one sub-block
+  // Log2 decays of the chunk to convert next.  A warp takes one sub-block and 16 pairs of channels; lanes 16-31 hold the
+  // sub-block's last eight tokens.
+  const int half = lane >> 4;
+  float raw[ITEMS][8][2];
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int i = 0; i < ITEMS; ++i) {
-      const int item = threadIdx.x + i * 256, d = item % NP, t = t0 + item / NP * kSub;
+      const int item = wid + i * 8, d = (item % (NP / 32)) * 32 + (lane & 15) * 2, t = t0 + item / (NP / 32) * kSub + half * 8;
 #pragma unroll
-      for (int u = 0; u < kSub; ++u) raw[i][u] = d < D && t + u < t_end ? dec[static_cast<int64_t>(t + u) * a.ld_decay + d] : 0.0f;
+      for (int u = 0; u < 8; ++u) {
+        const float* p = dec + static_cast<int64_t>(t + u) * a.ld_decay + d;
+        float2 x = make_float2(0.0f, 0.0f);
+        if (t + u < t_end) {
+          if (vec_a) {
+            if (d < D) x = *reinterpret_cast<const float2*>(p);
+          } else {
+            if (d < D) x.x = p[0];
+            if (d + 1 < D) x.y = p[1];
+          }
+        }
+        raw[i][u][0] = x.x;
+        raw[i][u][1] = x.y;
+      }
     }
+  };
+  auto scale_store = [&](__nv_bfloat16* hi, __nv_bfloat16* lo, int o, float f0, float f1) {
+    const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(hi + o);
+    uint32_t xh, xl;
+    bf16_split(__low2float(x) * f0, __high2float(x) * f1, xh, xl);
+    *reinterpret_cast<uint32_t*>(hi + o) = xh;
+    *reinterpret_cast<uint32_t*>(lo + o) = xl;
   };
   if (!kLocal) load_q(t_begin);
   load_kv(t_begin);
@@ -118,79 +174,55 @@ __global__ void __launch_bounds__(256, NP <= 64 ? 2 : 1) gla_chunk_kernel(const 
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < ITEMS; ++i) {
-      const int item = threadIdx.x + i * 256, d = item % NP, j = item / NP;
+      const int item = wid + i * 8, d = (item % (NP / 32)) * 32 + (lane & 15) * 2, j = item / (NP / 32);
+      float before[2], end[2];
 #pragma unroll
-      for (int u = 1; u < kSub; ++u) raw[i][u] += raw[i][u - 1];
-      const float end = raw[i][kSub - 1];
-      sR[j * NP + d] = end;
-      if (end < kSafe) s_far[par][j] = 1;
+      for (int e = 0; e < 2; ++e) {
 #pragma unroll
-      for (int u = 0; u < kSub; ++u) {
-        const int o = (j * kSub + u) * LN + d;
-        if (!kLocal) {
-          const float x = __bfloat162float(sQh[o]) * (a.q_scale * ex2_approx(raw[i][u]));
-          const __nv_bfloat16 hi = __float2bfloat16_rn(x);
-          sQh[o] = hi;
-          sQl[o] = __float2bfloat16_rn(x - __bfloat162float(hi));
-        }
-        const float x = __bfloat162float(sKh[o]) * ex2_approx(end - raw[i][u]);
-        const __nv_bfloat16 hi = __float2bfloat16_rn(x);
-        sKh[o] = hi;
-        sKl[o] = __float2bfloat16_rn(x - __bfloat162float(hi));
+        for (int u = 1; u < 8; ++u) raw[i][u][e] += raw[i][u - 1][e];
+        const float other = __shfl_xor_sync(0xffffffffu, raw[i][7][e], 16);
+        before[e] = half ? other : 0.0f;
+        end[e] = raw[i][7][e] + other;
+      }
+      if (half == 0) {
+        *reinterpret_cast<float2*>(sD + j * NP + d) = make_float2(ex2_approx(end[0]), ex2_approx(end[1]));
+        *reinterpret_cast<float2*>(sI + j * NP + d) = make_float2(ex2_approx(-end[0]), ex2_approx(-end[1]));
+        if (fminf(end[0], end[1]) < kSafe) s_far[par][j] = 1;
+      }
+#pragma unroll
+      for (int u = 0; u < 8; ++u) {
+        // the halves of a warp are four rows apart in the walk, which keeps their banks apart
+        const float c0 = (half ? raw[i][u ^ 4][0] : raw[i][u][0]) + before[0], c1 = (half ? raw[i][u ^ 4][1] : raw[i][u][1]) + before[1];
+        const int o = (j * kSub + half * 8 + (half ? u ^ 4 : u)) * LN + d;
+        if (!kLocal) scale_store(sQh, sQl, o, a.q_scale * ex2_approx(c0), a.q_scale * ex2_approx(c1));
+        scale_store(sKh, sKl, o, ex2_approx(end[0] - c0), ex2_approx(end[1] - c1));
       }
     }
     if (more) fetch(t0 + kQ);
     __syncthreads();
     if (threadIdx.x < 4) s_far[par ^ 1][threadIdx.x] = 0;
     if (!kLocal) {
-      // 2^(sum of R over sub-blocks j0 .. j1 - 1), times -1 in the exponent where `inverse`, for the lane's four channels
-      auto factors = [&](int kk, int j0, int j1, bool inverse, float (&f)[4]) {
-        float2 s0 = make_float2(0.0f, 0.0f), s1 = s0;
+      // the lane's four channels of the product of the decays of sub-blocks j0 .. j1 - 1
+      auto decays = [&](int kk, int j0, int j1, float (&f)[4]) {
+        f[0] = f[1] = f[2] = f[3] = 1.0f;
         for (int j = j0; j < j1; ++j) {
-          const float2 r0 = *reinterpret_cast<const float2*>(sR + j * NP + kk * 16 + qc);
-          const float2 r1 = *reinterpret_cast<const float2*>(sR + j * NP + kk * 16 + 8 + qc);
-          s0.x += r0.x;
-          s0.y += r0.y;
-          s1.x += r1.x;
-          s1.y += r1.y;
+          const float2 x = *reinterpret_cast<const float2*>(sD + j * NP + kk * 16 + qc);
+          const float2 y = *reinterpret_cast<const float2*>(sD + j * NP + kk * 16 + 8 + qc);
+          f[0] *= x.x;
+          f[1] *= x.y;
+          f[2] *= y.x;
+          f[3] *= y.y;
         }
-        const float sign = inverse ? -1.0f : 1.0f;
-        f[0] = ex2_approx(sign * s0.x);
-        f[1] = ex2_approx(sign * s0.y);
-        f[2] = ex2_approx(sign * s1.x);
-        f[3] = ex2_approx(sign * s1.y);
       };
-      float y[4][4];
-      zero(y);
-#pragma unroll
-      for (int kk = 0; kk < NP / 16; ++kk) {             // q S
-        uint32_t qh[4], ql[4];
-        ldmatrix_x4(qh, addr_a<LN>(sQh, warp * 16, kk * 16));
-        ldmatrix_x4(ql, addr_a<LN>(sQl, warp * 16, kk * 16));
-        if (warp > 0) {
-          float f[4];
-          factors(kk, 0, warp, false, f);
-          scale_pair(qh, ql, f);
-        }
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          uint32_t bh[4], bl[4];
-          ldmatrix_x4_trans(bh, addr_b_t<LP>(sSh, kk * 16, cb + n * 16));
-          ldmatrix_x4_trans(bl, addr_b_t<LP>(sSl, kk * 16, cb + n * 16));
-          mma_bf16(y[2 * n], qh, bh[0], bh[1]);
-          mma_bf16(y[2 * n + 1], qh, bh[2], bh[3]);
-          mma_bf16(y[2 * n], qh, bl[0], bl[1]);
-          mma_bf16(y[2 * n + 1], qh, bl[2], bl[3]);
-          mma_bf16(y[2 * n], ql, bh[0], bh[1]);
-          mma_bf16(y[2 * n + 1], ql, bh[2], bh[3]);
-        }
-      }
-      for (int j = 0; j <= warp; ++j) {                  // 16 keys at a time, up to the diagonal
-        float g[2][4];
+      auto inner = [&](int i, int j, float (&g)[2][4]) {
         zero(g);
-        if (j == warp && s_far[par][warp]) {
+        if (j < i) {
+          block_product<NP>(g, sQh, sQl, sKh, sKl, i, j, j + 1 < i, [&](int kk, float (&f)[4]) { decays(kk, j + 1, i, f); });
+          return;
+        }
+        if (s_far[par][i]) {
           // the decay between two tokens directly: lane t < 16 holds token t of the sub-block
-          const int t = t0 + warp * kSub + (lane & 15);
+          const int t = t0 + i * kSub + (lane & 15);
           const bool in = t < t_end;
           for (int d = 0; d < D; ++d) {
             float c = in ? dec[static_cast<int64_t>(t) * a.ld_decay + d] : 0.0f;
@@ -210,43 +242,78 @@ __global__ void __launch_bounds__(256, NP <= 64 ? 2 : 1) gla_chunk_kernel(const 
             }
           }
         } else {
-#pragma unroll
-          for (int kk = 0; kk < NP / 16; ++kk) {
-            uint32_t qh[4], ql[4], bh[4], bl[4];
-            ldmatrix_x4(qh, addr_a<LN>(sQh, warp * 16, kk * 16));
-            ldmatrix_x4(ql, addr_a<LN>(sQl, warp * 16, kk * 16));
-            ldmatrix_x4(bh, addr_b<LN>(sKh, j * 16, kk * 16));
-            ldmatrix_x4(bl, addr_b<LN>(sKl, j * 16, kk * 16));
-            if (j != warp - 1) {
-              float f[4];
-              if (j == warp) factors(kk, warp, warp + 1, true, f);
-              else factors(kk, j + 1, warp, false, f);
-              scale_pair(qh, ql, f);
-            }
-            mma_bf16(g[0], qh, bh[0], bh[1]);
-            mma_bf16(g[1], qh, bh[2], bh[3]);
-            mma_bf16(g[0], qh, bl[0], bl[1]);
-            mma_bf16(g[1], qh, bl[2], bl[3]);
-            mma_bf16(g[0], ql, bh[0], bh[1]);
-            mma_bf16(g[1], ql, bh[2], bh[3]);
-          }
+          block_product<NP>(g, sQh, sQl, sKh, sKl, i, i, true, [&](int kk, float (&f)[4]) {
+            const float2 x = *reinterpret_cast<const float2*>(sI + i * NP + kk * 16 + qc);
+            const float2 y = *reinterpret_cast<const float2*>(sI + i * NP + kk * 16 + 8 + qc);
+            f[0] = x.x;
+            f[1] = x.y;
+            f[2] = y.x;
+            f[3] = y.y;
+          });
         }
-        if (j == warp) {
 #pragma unroll
-          for (int n = 0; n < 2; ++n)
+        for (int n = 0; n < 2; ++n)
 #pragma unroll
-            for (int e = 0; e < 4; ++e)
-              if (n * 8 + qc + (e & 1) > (e >> 1) * 8 + qr) g[n][e] = 0.0f;
+          for (int e = 0; e < 4; ++e)
+            if (n * 8 + qc + (e & 1) > (e >> 1) * 8 + qr) g[n][e] = 0.0f;
+      };
+      auto put = [&](int i, int j, const float (&g)[2][4]) {
+        uint4 hi, lo;
+        bf16_split(g[0][0], g[0][1], hi.x, lo.x);
+        bf16_split(g[0][2], g[0][3], hi.y, lo.y);
+        bf16_split(g[1][0], g[1][1], hi.z, lo.z);
+        bf16_split(g[1][2], g[1][3], hi.w, lo.w);
+        uint4* dst = sG + (i * (i + 1) / 2 + j) * 64 + lane;
+        dst[0] = hi;
+        dst[32] = lo;
+      };
+      // Ten blocks on eight warps: the three next to the diagonal need no factors, so two warps take two blocks.
+      //   warp   0      1      2             3      4      5             6      7
+      //   block  (3,0)  (3,1)  (3,2), (0,0)  (3,3)  (2,0)  (2,1), (1,0)  (2,2)  (1,1)
+      const int bi = wid < 4 ? 3 : wid < 7 ? 2 : 1, bj = wid < 4 ? wid : wid < 7 ? wid - 4 : 1;
+      float g0[2][4], g1[2][4];
+      inner(bi, bj, g0);
+      if (wid == 2) inner(0, 0, g1);
+      if (wid == 5) inner(1, 0, g1);
+      float y[4][4];
+      zero(y);
+#pragma unroll
+      for (int kk = 0; kk < NP / 16; ++kk) {             // q S
+        uint32_t qh[4], ql[4];
+        ldmatrix_x4(qh, addr_a<LN>(sQh, warp * kSub, kk * 16));
+        ldmatrix_x4(ql, addr_a<LN>(sQl, warp * kSub, kk * 16));
+        if (warp > 0) {
+          float f[4];
+          decays(kk, 0, warp, f);
+          scale_pair(qh, ql, f);
         }
-        uint32_t mh[4], ml[4];
-        bf16_split(g[0][0], g[0][1], mh[0], ml[0]);
-        bf16_split(g[0][2], g[0][3], mh[1], ml[1]);
-        bf16_split(g[1][0], g[1][1], mh[2], ml[2]);
-        bf16_split(g[1][2], g[1][3], mh[3], ml[3]);
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          uint32_t bh[4], bl[4];
+          ldmatrix_x4_trans(bh, addr_b_t<LP>(sSh, kk * 16, cb + n * 16));
+          ldmatrix_x4_trans(bl, addr_b_t<LP>(sSl, kk * 16, cb + n * 16));
+          mma_bf16(y[2 * n], qh, bh[0], bh[1]);
+          mma_bf16(y[2 * n + 1], qh, bh[2], bh[3]);
+          mma_bf16(y[2 * n], qh, bl[0], bl[1]);
+          mma_bf16(y[2 * n + 1], qh, bl[2], bl[3]);
+          mma_bf16(y[2 * n], ql, bh[0], bh[1]);
+          mma_bf16(y[2 * n + 1], ql, bh[2], bh[3]);
+        }
+      }
+      if constexpr (L::kOverQ) __syncthreads();          // q has been read
+      put(bi, bj, g0);
+      if (wid == 2) put(0, 0, g1);
+      if (wid == 5) put(1, 0, g1);
+      __syncthreads();                                   // the blocks are complete; q is free
+      if (!L::kOverQ && more) load_q(t0 + kQ);
+      for (int j = 0; j <= warp; ++j) {
+        const uint4* src = sG + (warp * (warp + 1) / 2 + j) * 64 + lane;
+        const uint4 hi = src[0], lo = src[32];
+        const uint32_t mh[4] = {hi.x, hi.y, hi.z, hi.w}, ml[4] = {lo.x, lo.y, lo.z, lo.w};
 #pragma unroll
         for (int n = 0; n < 2; ++n) {
           uint32_t b[4];
-          ldmatrix_x4_trans(b, addr_b_t<LP>(sV, j * 16, cb + n * 16));
+          ldmatrix_x4_trans(b, addr_b_t<LP>(sV, j * kSub, cb + n * 16));
           mma_bf16(y[2 * n], mh, b[0], b[1]);
           mma_bf16(y[2 * n + 1], mh, b[2], b[3]);
           mma_bf16(y[2 * n], ml, b[0], b[1]);
@@ -270,8 +337,6 @@ __global__ void __launch_bounds__(256, NP <= 64 ? 2 : 1) gla_chunk_kernel(const 
           }
         }
       }
-      __syncthreads();                                   // q is free
-      if (more) load_q(t0 + kQ);
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
@@ -279,12 +344,11 @@ __global__ void __launch_bounds__(256, NP <= 64 ? 2 : 1) gla_chunk_kernel(const 
 #pragma unroll
       for (int m = 0; m < MT; ++m) {
         const int r = (warp * MT + m) * 16;
-        ldmatrix_x4_trans(kh[m], addr_a_t<LN>(sKh, j * 16, r));
-        ldmatrix_x4_trans(kl[m], addr_a_t<LN>(sKl, j * 16, r));
-        const float r0 = sR[j * NP + r + qr], r1 = sR[j * NP + r + 8 + qr];
-        const float d0 = ex2_approx(r0), d1 = ex2_approx(r1);
-        total[m][0] += r0;
-        total[m][1] += r1;
+        ldmatrix_x4_trans(kh[m], addr_a_t<LN>(sKh, j * kSub, r));
+        ldmatrix_x4_trans(kl[m], addr_a_t<LN>(sKl, j * kSub, r));
+        const float d0 = sD[j * NP + r + qr], d1 = sD[j * NP + r + 8 + qr];
+        total[m][0] *= d0;
+        total[m][1] *= d1;
 #pragma unroll
         for (int n = 0; n < 4; ++n) {
           S[m][n][0] *= d0;
@@ -296,7 +360,7 @@ __global__ void __launch_bounds__(256, NP <= 64 ? 2 : 1) gla_chunk_kernel(const 
 #pragma unroll
       for (int n = 0; n < 2; ++n) {
         uint32_t b[4];
-        ldmatrix_x4_trans(b, addr_b_t<LP>(sV, j * 16, cb + n * 16));
+        ldmatrix_x4_trans(b, addr_b_t<LP>(sV, j * kSub, cb + n * 16));
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           mma_bf16(S[m][2 * n], kh[m], b[0], b[1]);
@@ -308,6 +372,7 @@ __global__ void __launch_bounds__(256, NP <= 64 ? 2 : 1) gla_chunk_kernel(const 
     }
     __syncthreads();                                     // k, v and the decays are free
     if (more) {
+      if (L::kOverQ && !kLocal) load_q(t0 + kQ);
       load_kv(t0 + kQ);
       cp_async_commit();
     }
@@ -329,7 +394,7 @@ __global__ void __launch_bounds__(256, NP <= 64 ? 2 : 1) gla_chunk_kernel(const 
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
         const int r = (warp * MT + m) * 16 + i * 8 + qr;
-        if (r < D) a.part_decay[unit * D + r] = ex2_approx(total[m][i]);
+        if (r < D) a.part_decay[unit * D + r] = total[m][i];
       }
   }
 }
@@ -355,7 +420,7 @@ __global__ void gla_span_scan_kernel(const NxGlaArgs a) {
 template <int NP>
 int launch(const NxGlaArgs* a, cudaStream_t st) {
   constexpr int kBytes = Smem<NP>::kBytes;
-  static_assert(kBytes <= 226 * 1024, "shared memory");
+  static_assert(kBytes <= 227 * 1024 - 64, "shared memory");
   static bool once = false;
   if (!once) {
     if (cudaFuncSetAttribute(gla_chunk_kernel<NP, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kBytes) != cudaSuccess ||
