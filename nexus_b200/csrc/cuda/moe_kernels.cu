@@ -276,15 +276,9 @@ __device__ __forceinline__ void pick_experts(const NxGateRouteArgs& a, int row, 
         best = s[e];
         be = e;
       }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oe = __shfl_xor_sync(0xffffffffu, be, o);
-      if (ob > best || (ob == best && oe < be)) {
-        best = ob;
-        be = oe;
-      }
-    }
+    const int bits = __float_as_int(best), key = bits < 0 ? bits ^ 0x7fffffff : bits;     // ordered like the floats
+    const int top_key = __reduce_max_sync(0xffffffffu, key);
+    be = __reduce_min_sync(0xffffffffu, key == top_key ? be : 0x7fffffff);
     if (be >= E) be = j;                       // only where scores are not numbers
     if (lane == j) mine = be;
     if (lane == (be & 31)) s[be] = -INFINITY;

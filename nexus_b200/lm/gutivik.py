@@ -20,7 +20,7 @@ __all__ = ["gutivik_config", "gutivik_tensors", "load_gutivik", "random_gutivik"
 
 
 def _window(mask: dict, where: str) -> int:
-    size = mask["size"]
+    size = mask.get("size")
     if not isinstance(size, int) or isinstance(size, bool) or size < 1:
         raise ConfigError(f"{where}.mask: the size must be a positive integer")
     return size
@@ -138,6 +138,9 @@ def load_gutivik(folder: str) -> HybridWeights:
         obj = json.load(f)
     tensors = load_file(os.path.join(folder, "model.safetensors"))
     cfg = gutivik_config(obj, decay_ranks(len(obj.get("layers", ())), tensors))
+    for i, layer in enumerate(cfg.layers):      # a layer that does not mix values has no use for the factor
+        if isinstance(layer.mixer, ConvAttentionSpec) and not layer.mixer.mix_values:
+            tensors.pop(f"l{i}.mix.vmix", None)
     check_gutivik(cfg, tensors)
     return HybridWeights(cfg, tensors)
 

@@ -263,7 +263,7 @@ class HybridConfig:
             raise ConfigError("token_side cannot be negative")
         if not self.layers:
             raise ConfigError("a model needs at least one layer")
-        if len({m.kv_heads * m.vdim for m in self._mixing()}) > 1:
+        if len({(m.kv_heads, m.vdim) for m in self._mixing()}) > 1:
             raise ConfigError("layers that mix values must have equal sizes of them")
 
     def _mixing(self) -> list:
