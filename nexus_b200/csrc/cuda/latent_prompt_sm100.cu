@@ -1,7 +1,8 @@
 // Attention of prompt segments on tcgen05 (see nx_api_mixers.h).  A key is a part of its own KV head, optionally beside a part
 // that all heads share; a row sees a window of keys and optionally the first keys of its sequence; a sink may count in the
 // denominator.  Queries, keys and values of all segments lie packed in row buffers; a work item is a block of up to 256 query
-// rows of one segment and one head.
+// rows of one segment and one head.  Without a shared key part a row may also see only the keys of its own chunk of positions, scores
+// may have a bias by distance, and an item may be a query head with the values of another KV head than its keys'.
 //
 // The pipeline is that of the two-tile flash kernel: one persistent CTA per SM, softmax group A (warps 0-3) on query rows
 // 0-127 of the block, group B (warps 4-7) on rows 128-255, both against the same key tiles; the MMA warp interleaves
@@ -24,15 +25,20 @@ using namespace nx;
 constexpr int kThreads = 320;   // warps 0-3: softmax A, 4-7: softmax B, 8: TMA, 9: MMA
 constexpr int kSlab = 128 * 128;  // bytes of [128 rows][64 columns]
 
+// distances of a bias table in shared memory, and how far it goes on to the masked ones (a row and a key of one tile pair are up to 254
+// apart in the wrong direction) and beyond the last one
+constexpr int kBiasMax = 3584, kBiasNear = 256, kBiasFar = 256, kBiasTable = kBiasNear + kBiasMax + kBiasFar;
+
 // ND / NV: 64-column slabs of a head's own key part and of its values; NR: of the shared part (0 or 1)
-template <int ND, int NR, int NV>
+// kBias: a table of biases per softmax group behind the barriers
+template <int ND, int NR, int NV, bool kBias>
 struct Cfg {
   static constexpr int kQBytes = (ND + NR) * kSlab;
   static constexpr int kKBytes = (ND + NR) * kSlab;
   static constexpr int kVBytes = NV * kSlab;
   static constexpr int kKStages = 2;
   static constexpr int kVStages = 2 * kQBytes + 2 * kKBytes + 2 * kVBytes <= 224 * 1024 ? 2 : 1;
-  static constexpr int kSmem = 2 * kQBytes + kKStages * kKBytes + kVStages * kVBytes + 256;
+  static constexpr int kSmem = 2 * kQBytes + kKStages * kKBytes + kVStages * kVBytes + 256 + (kBias ? 2 * kBiasTable * 4 : 0);
   static_assert(kSmem <= 227 * 1024, "shared memory");
 };
 
@@ -44,12 +50,18 @@ struct Dev {
   const float* sink;
   int* status;
   int64_t ldo;
+  const float* bias;         // [heads][bias_len]
   int items, heads, rep, vdim, window, keep_first, ksteps, rsteps;   // rep: query heads per KV head; 16-column steps of the own
-  float scale;                                                       // and the shared key part
+  int chunk, bias_len, values;                                       // and the shared key part; values: KV heads whose values a
+  float scale;                                                       // query head meets, 1: its own
+  __device__ __forceinline__ int first_key(int pos) const {          // apart from the kept ones
+    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    return chunk > 0 ? max(lo, pos / chunk * chunk) : lo;
+  }
 };
 
 struct Work {
-  int h, row0, rows, pos0, kv0, k_lo;
+  int h, hv, row0, rows, pos0, kv0, k_lo;   // hv: KV head of the values
   int kept0, n_kept;               // buffer row of kept key 0; kept keys before k_lo
   int shift;                       // key tile j < shift holds kept keys 128 j .., tile j >= shift keys k_lo + 128 (j - shift) ..
   int jbA, jeA, jbB, jeB, je;      // key tiles of either query tile
@@ -61,35 +73,36 @@ __device__ __forceinline__ bool next_work(const Dev& p, int round, Work& w) {
   const int G = static_cast<int>(gridDim.x), c = static_cast<int>(blockIdx.x);
   const int item = round * G + ((round & 1) ? (G - 1 - c) : c);
   if (item >= p.items) return false;
-  const int4 b = __ldg(reinterpret_cast<const int4*>(p.blocks) + item / p.heads);
-  w.h = item % p.heads;
+  const int per = kKeep ? p.heads * p.values : p.heads, block = item / per, sub = item % per;
+  const int4 b = __ldg(reinterpret_cast<const int4*>(p.blocks) + block);
+  w.h = kKeep ? sub / p.values : sub;
+  w.hv = kKeep ? (p.values > 1 ? sub % p.values : w.h / p.rep) : w.h;
   w.row0 = b.x;
   w.rows = b.y;
   w.pos0 = b.z;
   w.kv0 = b.w;
-  const int back = p.window > 0 ? p.window - 1 : 0x3fffffff;
-  w.k_lo = max(0, w.pos0 - back);
+  w.k_lo = p.first_key(w.pos0);
   w.n_kept = kKeep ? min(p.keep_first, w.k_lo) : 0;
   w.shift = (w.n_kept + 127) / 128;
-  w.kept0 = kKeep && p.kept != nullptr ? __ldg(p.kept + item / p.heads) : b.w;
+  w.kept0 = kKeep && p.kept != nullptr ? __ldg(p.kept + block) : b.w;
   w.jbA = 0;
   w.jeA = w.shift + (w.pos0 + min(128, w.rows) - 1 - w.k_lo) / 128 + 1;
   w.jbB = w.jeB = 0;
   if (w.rows > 128) {
     // rows that keep first keys walk all tiles: those between the kept ones and their window are masked out
-    w.jbB = kKeep && p.keep_first > 0 ? 0 : (max(0, w.pos0 + 128 - back) - w.k_lo) / 128;
+    w.jbB = kKeep && p.keep_first > 0 ? 0 : (p.first_key(w.pos0 + 128) - w.k_lo) / 128;
     w.jeB = w.shift + (w.pos0 + w.rows - 1 - w.k_lo) / 128 + 1;
   }
   w.je = max(w.jeA, w.jeB);
   return true;
 }
 
-template <int ND, int NR, int NV>
+template <int ND, int NR, int NV, bool kBias>
 __global__ void __launch_bounds__(kThreads, 1)
 prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_qr,
               const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_kr,
               const __grid_constant__ CUtensorMap tm_v, const Dev p) {
-  using C = Cfg<ND, NR, NV>;
+  using C = Cfg<ND, NR, NV, kBias>;
   constexpr int KS = C::kKStages, VS = C::kVStages;
   constexpr bool kKeep = NR == 0;
   extern __shared__ __align__(1024) uint8_t smem[];
@@ -102,9 +115,10 @@ prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
   uint8_t* sV = sK + KS * C::kKBytes;              // [VS]
   uint64_t* bars = reinterpret_cast<uint64_t*>(sV + VS * C::kVBytes);
   uint64_t *q_full = bars, *q_empty = bars + 2, *k_full = bars + 4, *k_empty = bars + 6, *v_full = bars + 8, *v_empty = bars + 10,
-           *s_full = bars + 12, *p_full = bars + 14, *o_done = bars + 16;      // two each
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 18);
+           *s_full = bars + 12, *p_full = bars + 14, *o_done = bars + 16, *group = bars + 18;      // two each
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 20);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  float* s_bias = reinterpret_cast<float*>(bars + 32);   // [2][kBiasTable], entry kBiasNear + distance, in units of log2
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
@@ -118,6 +132,7 @@ prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
       mbar_init(&s_full[x], 1);
       mbar_init(&p_full[x], 4);  // one arrival per softmax warp of the group
       mbar_init(&o_done[x], 1);
+      mbar_init(&group[x], 4);   // the warps of one softmax group among themselves
     }
     *abort_flag = 0;
     fence_mbar_init();
@@ -170,7 +185,7 @@ prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
           if (!ok) break;
           mbar_arrive_expect_tx(&v_full[v], C::kVBytes);
 #pragma unroll
-          for (int c = 0; c < NV; ++c) tma_load_3d(sV + v * C::kVBytes + c * kSlab, &tm_v, &v_full[v], 64 * c, hk, row);
+          for (int c = 0; c < NV; ++c) tma_load_3d(sV + v * C::kVBytes + c * kSlab, &tm_v, &v_full[v], 64 * c, w.hv, row);
         }
       }
     }
@@ -247,6 +262,7 @@ prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
     const uint32_t lane_addr = static_cast<uint32_t>((warp & 3) * 32) << 16;
     const uint32_t tmem_s = tmem_base + x * 128 + lane_addr, tmem_o = tmem_base + 256 + x * 128 + lane_addr;
     const float sc = p.scale * kLog2e;
+    int meets = 0;
     int cnt = 0;   // key tiles this group has processed: phase counter of s_full / o_done
     bool ok = true;
     Work w;
@@ -255,11 +271,31 @@ prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
       if (lane == 0) atomicCAS(p.status, 0, kStatusTimeoutEpilogue);
       return false;
     };
+    auto meet = [&]() {      // barrier of the group's four warps
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&group[x]);
+      return wait(&group[x], meets++ & 1);
+    };
     for (int round = 0; ok && next_work<kKeep>(p, round, w); ++round) {
       const int jb = x == 0 ? w.jbA : w.jbB, je = x == 0 ? w.jeA : w.jeB;
       if (je <= jb) continue;
       const int p0 = w.pos0 + x * 128, pos = p0 + r;
-      const int row_lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+      const int row_lo = p.first_key(pos), last_lo = p.first_key(p0 + 127);
+      const float* bias = nullptr;
+      float b_far = 0.0f;
+      if constexpr (kBias) {
+        // this head's biases for distances -kBiasNear .. bias_len + kBiasFar - 1, the last one from bias_len on
+        float* table = s_bias + x * kBiasTable;
+        const float* src = p.bias + static_cast<int64_t>(w.h) * p.bias_len;
+        ok = meet();                               // the group has left the previous item's table
+        if (!ok) break;
+        for (int i = r; i < kBiasNear + p.bias_len + kBiasFar; i += 128)
+          table[i] = __ldg(src + min(max(i - kBiasNear, 0), p.bias_len - 1)) * kLog2e;
+        b_far = __ldg(src + p.bias_len - 1) * kLog2e;
+        ok = meet();
+        if (!ok) break;
+        bias = table + kBiasNear + pos;
+      }
       float m_ref = -INFINITY, l_run = 0.0f;
       for (int j = jb; j < je; ++j, ++cnt) {
         const int k0 = w.first_key(j);
@@ -270,7 +306,21 @@ prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
 #pragma unroll
         for (int cc = 0; cc < 4; ++cc) tmem_ld_32x32b_x32(tmem_s + cc * 32, sv[cc]);
         tmem_ld_wait();
-        const bool need_mask = (kKeep && j < w.shift) || k0 + 127 > p0 || (p.window > 0 && k0 < p0 + 127 - p.window + 1);
+        // scores in units of log2: sc * product + add; a tile that no row is far from gets its biases one by one
+        float mul = sc, add = 0.0f;
+        if constexpr (kBias) {
+          add = b_far;
+          if (p0 - k0 - 127 < p.bias_len - 1) {
+            mul = 1.0f;
+            add = 0.0f;
+            const float* b = bias - k0;
+#pragma unroll
+            for (int cc = 0; cc < 4; ++cc)
+#pragma unroll
+              for (int c = 0; c < 32; ++c) sv[cc][c] = __float_as_uint(fmaf(__uint_as_float(sv[cc][c]), sc, b[-(cc * 32 + c)]));
+          }
+        }
+        const bool need_mask = (kKeep && j < w.shift) || k0 + 127 > p0 || k0 < last_lo;
         if (need_mask) {
           // column c is visible iff clo <= c <= chi; kept keys: those before k_lo, and in later tiles a row's window or, for a
           // tile that still holds kept keys, everything below keep_first
@@ -303,7 +353,7 @@ prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
             m2 = fmaxf(m2, __uint_as_float(sv[cc][c + 2]));
             m3 = fmaxf(m3, __uint_as_float(sv[cc][c + 3]));
           }
-        const float m_new = fmaxf(m_ref, fmaxf(fmaxf(m0, m1), fmaxf(m2, m3)) * sc);
+        const float m_new = fmaxf(m_ref, fmaf(fmaxf(fmaxf(m0, m1), fmaxf(m2, m3)), mul, add));
         const bool grow = m_new - kRescaleStep > m_ref;
         if (__any_sync(0xffffffffu, grow)) {
           const float alpha = grow ? ex2f(m_ref - m_new) : 1.0f;  // m_ref == -inf -> 0
@@ -327,7 +377,7 @@ prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
             tmem_st_wait();
           }
         }
-        const float m_use = m_ref == -INFINITY ? 0.0f : m_ref;
+        const float m_use = (m_ref == -INFINITY ? 0.0f : m_ref) - add;
         float r0 = 0.0f, r1 = 0.0f, r2 = 0.0f, r3 = 0.0f;
 #pragma unroll
         for (int cc = 0; cc < 4; ++cc) {
@@ -336,7 +386,7 @@ prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
           for (int g = 0; g < 4; ++g) {
             float e[8];
 #pragma unroll
-            for (int i = 0; i < 8; ++i) e[i] = ex2f(fmaf(__uint_as_float(sv[cc][8 * g + i]), sc, -m_use));  // -inf -> 0
+            for (int i = 0; i < 8; ++i) e[i] = ex2f(fmaf(__uint_as_float(sv[cc][8 * g + i]), mul, -m_use));  // -inf -> 0
             r0 += e[0] + e[4];
             r1 += e[1] + e[5];
             r2 += e[2] + e[6];
@@ -362,7 +412,8 @@ prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
       const int64_t row = w.row0 + x * 128 + r;
       if (kKeep && p.sink != nullptr) l_run += ex2f(p.sink[w.h] * kLog2e - m_ref);
       const float inv = row_ok ? (p.gate != nullptr ? p.gate[row * p.heads + w.h] : 1.0f) / l_run : 0.0f;
-      __nv_bfloat16* orow = p.out + row * p.ldo + static_cast<int64_t>(w.h) * p.vdim;
+      const int64_t slice = kKeep && p.values > 1 ? static_cast<int64_t>(w.h) * p.values + w.hv : w.h;
+      __nv_bfloat16* orow = p.out + row * p.ldo + slice * p.vdim;
 #pragma unroll
       for (int cc = 0; cc < NV * 2; ++cc) {
         uint32_t ov[32];
@@ -414,23 +465,23 @@ struct Maps {
   CUtensorMap q, qr, k, kr, v;
 };
 
-template <int ND, int NR, int NV>
+template <int ND, int NR, int NV, bool kBias>
 int launch(const Maps& t, const Dev& p, cudaStream_t st) {
-  constexpr int kSmem = Cfg<ND, NR, NV>::kSmem;
+  constexpr int kSmem = Cfg<ND, NR, NV, kBias>::kSmem;
   static bool once = false;
   if (!once) {
-    if (cudaFuncSetAttribute(prompt_kernel<ND, NR, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -2;
+    if (cudaFuncSetAttribute(prompt_kernel<ND, NR, NV, kBias>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -2;
     once = true;
   }
   int sms = 0, dev = 0;
   if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) return -2;
-  prompt_kernel<ND, NR, NV><<<std::min(p.items, sms), kThreads, kSmem, st>>>(t.q, t.qr, t.k, t.kr, t.v, p);
+  prompt_kernel<ND, NR, NV, kBias><<<std::min(p.items, sms), kThreads, kSmem, st>>>(t.q, t.qr, t.k, t.kr, t.v, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -2;
 }
-template <int NR>
+template <int NR, bool kBias>
 int launch_sizes(int dim, int vdim, const Maps& t, const Dev& p, cudaStream_t st) {
-  if (dim <= 64) return vdim <= 64 ? launch<1, NR, 1>(t, p, st) : launch<1, NR, 2>(t, p, st);
-  return vdim <= 64 ? launch<2, NR, 1>(t, p, st) : launch<2, NR, 2>(t, p, st);
+  if (dim <= 64) return vdim <= 64 ? launch<1, NR, 1, kBias>(t, p, st) : launch<1, NR, 2, kBias>(t, p, st);
+  return vdim <= 64 ? launch<2, NR, 1, kBias>(t, p, st) : launch<2, NR, 2, kBias>(t, p, st);
 }
 
 // copies the cache rows of a segment list into one packed buffer: keys `base` .. of every segment, 16 bytes per thread
@@ -495,12 +546,14 @@ extern "C" int nx_latent_prompt(const NxLatentPromptArgs* a, nx_stream_t stream)
   p.ksteps = a->dim / 16;
   p.rsteps = a->rot / 16;
   p.scale = a->scale;
-  return launch_sizes<1>(a->dim, a->vdim, t, p, static_cast<cudaStream_t>(stream));
+  return launch_sizes<1, false>(a->dim, a->vdim, t, p, static_cast<cudaStream_t>(stream));
 }
 
 extern "C" int nx_window_prompt(const NxWindowPromptArgs* a, nx_stream_t stream) {
   if (a == nullptr || a->status == nullptr || a->blocks == nullptr || a->heads <= 0 || a->kv_heads <= 0 || !(a->scale > 0.0f)) return -1;
-  if (a->heads % a->kv_heads || a->keep_first < 0) return -1;
+  if (a->heads % a->kv_heads || a->keep_first < 0 || a->chunk < 0) return -1;
+  if (a->bias != nullptr && (a->bias_len <= 0 || a->bias_len > kBiasMax)) return -1;
+  if (a->all_values && static_cast<int64_t>(a->n_blocks) * a->heads * a->kv_heads > 0x3fffffff) return -1;
   if (a->dim <= 0 || a->dim > 128 || (a->dim & 15) || a->vdim <= 0 || a->vdim > 128 || (a->vdim & 7)) return -1;
   if ((a->ldq | a->ldk | a->ldv | a->ldo) & 7) return -1;
   for (const void* ptr : {a->q, a->k, a->v, static_cast<const void*>(a->out), static_cast<const void*>(a->blocks)})
@@ -518,15 +571,21 @@ extern "C" int nx_window_prompt(const NxWindowPromptArgs* a, nx_stream_t stream)
   p.kept = a->kept;
   p.out = static_cast<__nv_bfloat16*>(a->out);
   p.sink = a->sink;
+  p.gate = a->gate;
+  p.bias = a->bias;
+  p.bias_len = a->bias_len;
+  p.chunk = a->chunk;
+  p.values = a->all_values ? a->kv_heads : 1;
   p.status = a->status;
   p.ldo = a->ldo;
-  p.items = a->n_blocks * a->heads;
+  p.items = a->n_blocks * a->heads * p.values;
   p.heads = a->heads;
   p.rep = a->heads / a->kv_heads;
   p.vdim = a->vdim;
   p.window = a->window;
-  p.keep_first = a->window > 0 ? a->keep_first : 0;
+  p.keep_first = a->window > 0 || a->chunk > 0 ? a->keep_first : 0;
   p.ksteps = a->dim / 16;
   p.scale = a->scale;
-  return launch_sizes<0>(a->dim, a->vdim, t, p, static_cast<cudaStream_t>(stream));
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return p.bias != nullptr ? launch_sizes<0, true>(a->dim, a->vdim, t, p, st) : launch_sizes<0, false>(a->dim, a->vdim, t, p, st);
 }

@@ -31,6 +31,12 @@ __global__ void residual_norm_kernel(const NxResidualNormArgs a) {
       load_vec<T, V>(e + c, v);
 #pragma unroll
       for (int j = 0; j < V; ++j) v[j] *= a.embed_scale;
+      if (a.pos_table != nullptr) {
+        float p[V];
+        load_vec<T, V>(static_cast<const T*>(a.pos_table) + static_cast<int64_t>(a.positions[r]) * cols + c, p);
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[j] += p[j];
+      }
       store_vec<float, V>(xr + c, v);
       store_vec<float, V>(s_row + c, v);
 #pragma unroll

@@ -1,4 +1,5 @@
-// C ABI of the building blocks of decoders with heterogeneous layers: pre / post norms around a sublayer, rotary
+// C ABI of the building blocks of decoders with heterogeneous layers: pre / post norms around a sublayer, residuals of several
+// streams, norms of queries and keys, heads that mix, rotary
 // embedding fused with the cache append, windowed and soft-capped paged attention for any head sizes, the short causal
 // convolution with its carried tail, the Mamba-2 (SSD), gated-delta-rule and gated-linear-attention recurrences with their
 // carried FP32 state, gated norms, gated activations, the per-layer token input and soft-capping of logits.
@@ -53,8 +54,58 @@ typedef struct NxResidualNormArgs {
   void* scatter;
   const int32_t* scatter_slots;
   const float* expert_weights;
+  // with `table`: x += pos_table[positions[row]], may be null
+  const int32_t* positions;
+  const void* pos_table;   // [positions, cols] dtype
 } NxResidualNormArgs;
 int nx_residual_norm(const NxResidualNormArgs* args, nx_stream_t stream);
+
+// Residual of several streams x_s.  table: every stream becomes embed_scale * table[token] + pos_table[position]; else with y the
+// streams become x_t <- sum_s mix[s][t] x_s + out[t] y.  Then h = rms(sum_s in[s] x_s) * w_next of the new streams.
+typedef struct NxStreamResidualArgs {
+  float* x;                // [rows, streams, cols], updated in place
+  const int32_t* tokens;
+  const void* table;       // [vocab, cols] dtype, may be null
+  const int32_t* positions;
+  const void* pos_table;   // [positions, cols] dtype, may be null
+  const void* y;           // [rows, ldy], may be null
+  const float* mix;        // [streams, streams]: from, to
+  const float* out;        // [streams]
+  const float* in;         // [streams]; null: ones
+  const float* w_next;     // [cols]
+  void* h;                 // [rows, ldh], may be null; columns cols..ldh are zeroed
+  int64_t ldy, ldh;
+  int32_t rows, cols, streams, dtype;   // up to 8 streams of up to 12288 columns
+  float eps, embed_scale;
+} NxStreamResidualArgs;
+int nx_stream_residual(const NxStreamResidualArgs* args, nx_stream_t stream);
+
+// What lies between the projections and the scores of attention on normed queries and keys, in place in `proj`: RMS norms of q and
+// k (over each head with one shared weight, or norm_all: over all heads at once), q also times q_scale * head_scale[head] * (1 + coef
+// ln(floor((p + 1) / every) + 1)), unit_values: v divided by its root mean square per head; k and v go to the cache (with store_kv
+// back to proj too), gate = sigmoid.  Heads are dim / vdim columns wide, of which the leading norm_dim / norm_vdim count (the rest
+// are zeros).
+typedef struct NxHeadPrepArgs {
+  void* proj;              // [rows, ld]; the parts of a row start at q_off, k_off, v_off, g_off
+  int64_t ld;
+  int32_t q_off, k_off, v_off, g_off;
+  int32_t rows, heads, kv_heads, dim, vdim, norm_dim, norm_vdim, norm_all, unit_values, store_kv, every, dtype;   // every 0: none
+  float eps, q_scale, coef;
+  const float* w_q;        // [dim], or [heads * dim] with norm_all
+  const float* w_k;        // [dim], or [kv_heads * dim]
+  const float* head_scale; // [heads], may be null
+  const int32_t* positions;
+  const int32_t* slots;    // cache slot per row, negative: nothing is appended
+  void* k_cache;           // [slots, kv_heads, dim]
+  void* v_cache;           // [slots, kv_heads, vdim]
+  float* gate;             // [rows, heads], may be null
+} NxHeadPrepArgs;
+int nx_head_prep(const NxHeadPrepArgs* args, nx_stream_t stream);
+
+// Heads that mix their weights after the softmax, on the outputs: wide [rows, heads, kv_heads, vdim] holds what every head's weights
+// give with the values of every KV head; out [rows, heads, vdim]: out_h = gate_h sum_g talk[h][g] wide[g][KV head of h].
+int nx_head_mix(const void* wide, int64_t ldw, const float* talk, const float* gate, void* out, int64_t ldo, int rows, int heads,
+                int kv_heads, int vdim, int dtype, nx_stream_t stream);
 
 typedef struct NxRopeAppendArgs {
   void* proj;              // [rows, ld]; q, k, v of a row start at q_off, k_off, v_off; q and k are rotated in place
@@ -230,8 +281,10 @@ int nx_glu(const void* h, int64_t ldh, void* out, int64_t ldo, int rows, int hal
 int nx_softcap(float* x, int64_t ld, int rows, int cols, float cap, float scale, nx_stream_t stream);
 
 // Causal attention of packed query rows over a paged cache.  Row at position p sees keys p - window + 1 .. p (window <= 0:
-// 0 .. p) and the first keep_first keys; score = scale * q.k, soft-capped when softcap > 0.  sink: a score per head (not scaled)
-// that counts in the denominator only.  The rows' own keys are in the cache already.
+// 0 .. p), with chunk > 0 only those of its own chunk (p / chunk), and the first keep_first keys; score = scale * q.k, soft-capped
+// when softcap > 0, plus bias[head][min(distance, bias_len - 1)].  sink: a score per head (not scaled) that counts in the denominator
+// only.  The rows' own keys are in the cache already.  all_values: every query head meets the values of every KV head, out is
+// [rows, heads, kv_heads, vdim] (prompt and FP32 kernels).
 typedef struct NxPagedWindowArgs {
   const void* q;           // [rows, ldq]: heads * dim
   const void* k_cache;     // [blocks * block_size, kv_heads, dim]
@@ -249,6 +302,8 @@ typedef struct NxPagedWindowArgs {
   const float* gate;         // [rows, heads] factor of the output, may be null
   const float* sink;         // [heads], may be null
   int32_t keep_first;
+  int32_t chunk, bias_len, all_values;
+  const float* bias;         // [heads, bias_len], may be null
 } NxPagedWindowArgs;
 // one-row segments, BF16: tensor-core tiles of up to 16 query heads of a KV head against 64 keys, split over the keys
 int nx_paged_window_decode(const NxPagedWindowArgs* args, nx_stream_t stream);
@@ -256,6 +311,16 @@ int nx_paged_window_decode(const NxPagedWindowArgs* args, nx_stream_t stream);
 int nx_paged_window_prefill(const NxPagedWindowArgs* args, nx_stream_t stream);
 // any segments, FP32
 int nx_paged_window_f32(const NxPagedWindowArgs* args, nx_stream_t stream);
+// One-row segments, BF16, of heads that mix their weights: weight_h <- sum_g talk[h][g] weight_g, FP32, before the values of the KV
+// head of h.  Scores of all heads first (scores [count, heads, score_pitch], log2; part_ml [count, heads, splits, 2] always), then
+// mixture and values; part_o as above.  No sink, no all_values; up to 96 heads, vdim <= 256.
+typedef struct NxTalkDecodeArgs {
+  NxPagedWindowArgs base;
+  const float* talk;         // [heads, heads]
+  float* scores;
+  int64_t score_pitch;       // a multiple of 64, at least the keys a row can see
+} NxTalkDecodeArgs;
+int nx_talk_decode(const NxTalkDecodeArgs* args, nx_stream_t stream);
 
 
 // Attention of packed query rows over a latent cache, BF16: every head meets the same cache row [latent (rank) | rotated key
@@ -299,8 +364,8 @@ int nx_latent_prompt(const NxLatentPromptArgs* args, nx_stream_t stream);
 
 // The same kernel on plain grouped keys and values: q [q_rows, ldq]: heads * dim; k [kv_rows, ldk]: kv_heads * dim; v [kv_rows,
 // ldv]: kv_heads * vdim; query head h reads KV head h / (heads / kv_heads).  Windows, kept first keys and sinks as in
-// NxPagedWindowArgs.  blocks as above; kept [n_blocks]: row that position 0 has among the kept keys (null: the fourth entry of
-// the block).  dim <= 128: multiple of 16; vdim <= 128: multiple of 8; scale > 0.
+// NxPagedWindowArgs, chunks, biases (up to 3584 distances) and all_values too.  blocks as above; kept [n_blocks]: row that position 0
+// has among the kept keys (null: the fourth entry of the block).  dim <= 128: multiple of 16; vdim <= 128: multiple of 8; scale > 0.
 typedef struct NxWindowPromptArgs {
   const void* q;
   const void* k;
@@ -313,6 +378,9 @@ typedef struct NxWindowPromptArgs {
   int64_t ldq, ldk, ldv, ldo;
   int32_t n_blocks, q_rows, kv_rows, heads, kv_heads, dim, vdim, window, keep_first;
   float scale;
+  const float* gate;       // [rows, heads], may be null
+  const float* bias;       // [heads, bias_len], may be null
+  int32_t bias_len, chunk, all_values;
 } NxWindowPromptArgs;
 int nx_window_prompt(const NxWindowPromptArgs* args, nx_stream_t stream);
 // Cache rows of `segments` runs of positions into one packed buffer.  list [segments, 4]: first destination row, rows, first

@@ -1,10 +1,10 @@
-// Causal attention over a paged cache for any head sizes: sliding window, kept first keys, a sink in the denominator, score
-// soft-capping, grouped query heads, different key and value widths (see nx_api_mixers.h).  The query heads that share a KV head are packed into the rows of
-// one tensor-core tile, so a KV page is read once for all of them: 64 (token, head) rows per block in prompts, up to 16
-// heads of one token in decoding.  Scores, soft-capping and softmax are FP32; only the products take BF16 operands.
+// Causal attention over a paged cache for any head sizes: sliding window, chunks, kept first keys, a sink in the denominator, score
+// soft-capping, biases by distance, grouped query heads, different key and value widths (see nx_api_mixers.h).  The query heads that
+// share a KV head are packed into the rows of one tensor-core tile, so a KV page is read once for all of them: 128 (token, head) rows
+// per block in prompts, up to 16 heads of one token in decoding.  Scores, soft-capping and softmax are FP32; only the products take BF16 operands.
 #include "mixer_common.cuh"
 #include "nx_api_mixers.h"
-#include "paged_common.cuh"
+#include "paged_keys.cuh"
 
 #include <algorithm>
 
@@ -13,68 +13,9 @@ using namespace nx;
 
 constexpr int kKeys = 64;              // keys per shared-memory stage
 constexpr int kRows = 128;             // (token, head) rows per block in prompts
-constexpr float kLog2e = 1.4426950408889634f;
-
-// Scores in units of log2.  Soft-capping goes through one exponential: cap tanh(z) = cap - 2 cap / (1 + e^{2z}).  It is
-// monotone, so row maxima are taken over the raw products and only the maximum is mapped.
-struct ScoreMap {
-  bool capped;
-  float mul, cap2, cap;      // capped: x -> cap - cap2 / (1 + 2^(mul x)); else x -> mul x
-  __device__ __forceinline__ ScoreMap(float scale, float softcap) {
-    capped = softcap > 0.0f;
-    mul = capped ? 2.0f * kLog2e * scale / softcap : scale * kLog2e;
-    cap = softcap * kLog2e;
-    cap2 = 2.0f * cap;
-  }
-  __device__ __forceinline__ float operator()(float x) const {       // -inf (nothing visible) stays -inf
-    if (!capped || x == -INFINITY) return mul * x;
-    return cap - cap2 * rcp_approx(1.0f + ex2_approx(mul * x));
-  }
-  // 2^(mapped x - base)
-  __device__ __forceinline__ float prob(float x, float base) const {
-    if (!capped) return ex2_approx(fmaf(mul, x, -base));
-    return ex2_approx(fmaf(-cap2, rcp_approx(1.0f + ex2_approx(mul * x)), cap - base));
-  }
-};
-
-// The keys a block meets, numbered without the gap between the kept first ones and the window: index i is position i below
-// `kept` and position i + skip from there on.
-struct KeyRange {
-  int kept, skip, count;
-  // rows at positions pos .. last
-  __device__ __forceinline__ KeyRange(const NxPagedWindowArgs& a, int pos, int last) {
-    const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-    kept = min(a.keep_first, lo);
-    skip = lo - kept;
-    count = last + 1 - skip;
-  }
-  __device__ __forceinline__ int position(int i) const { return i < kept ? i : i + skip; }
-};
 
 // One stage of keys and values into shared memory, each [kKeys][DP + 8]; keys past index `last` and columns past the head size
 // become zeros.
-struct KvSource {
-  const __nv_bfloat16 *k, *v;
-  const int32_t* bt;
-  int64_t k_pitch, v_pitch;                            // elements between cache slots
-  int block_size, shift, dim, vdim;                    // shift: log2 of a power-of-two block size, else -1
-  __device__ __forceinline__ KvSource(const NxPagedWindowArgs& a, int seq, int head)
-      : k(static_cast<const __nv_bfloat16*>(a.k_cache) + static_cast<int64_t>(head) * a.dim),
-        v(static_cast<const __nv_bfloat16*>(a.v_cache) + static_cast<int64_t>(head) * a.vdim),
-        bt(a.block_table + static_cast<int64_t>(seq) * a.max_blocks), k_pitch(a.k_pitch), v_pitch(a.v_pitch),
-        block_size(a.block_size), shift(log2_of(a.block_size)), dim(a.dim), vdim(a.vdim) {}
-  __device__ __forceinline__ int64_t slot(int j) const {
-    return page_slot(bt, block_size, shift, j);
-  }
-};
-__device__ __forceinline__ void copy8(__nv_bfloat16* d, const __nv_bfloat16* s, int c, int cols) {   // columns c .. c + 7 of a row
-  if ((cols & 7) == 0) {
-    cp_async16(d, s + c);
-  } else {
-#pragma unroll
-    for (int e = 0; e < 8; ++e) d[e] = c + e < cols ? s[c + e] : __float2bfloat16_rn(0.0f);
-  }
-}
 template <int DP>
 __device__ __forceinline__ void stage_kv(__nv_bfloat16* dst, const KvSource& src, const KeyRange& keys, int k0, int last) {
   constexpr int CH = DP / 8, LD = DP + 8;
@@ -91,9 +32,9 @@ __device__ __forceinline__ void stage_kv(__nv_bfloat16* dst, const KvSource& src
 }
 
 // ------------------------------------------------------------------------------------------------
-// prompts: grid (tiles, kv_heads * head tiles), 8 warps of 16 rows
+// prompts: grid (tiles, kv_heads * head tiles, value heads), 8 warps of 16 rows
 // ------------------------------------------------------------------------------------------------
-template <int DP>
+template <int DP, bool kBias>
 __global__ void __launch_bounds__(kRows * 2)
 paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) {
   constexpr int LD = DP + 8;
@@ -121,7 +62,7 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
   const int64_t row0 = static_cast<int64_t>(a.seg.row0[sg]) + t0;
   const KeyRange keys(a, pos0, pos0 + nt - 1);
   const int last = keys.count - 1;
-  const KvSource src(a, a.seg.seq[sg], hk);
+  const KvSource src(a, a.seg.seq[sg], hk, a.all_values ? blockIdx.z : hk);
   auto stage = [&](int k0, int s) {
     stage_kv<DP>(sKV + (s * 2) * kKeys * LD, src, keys, k0, last);
     cp_async_commit();
@@ -144,15 +85,19 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
       }
     }
   }
-  int qpos[2];                                  // position of this thread's two rows, -1: padding row
+  int qpos[2], qlo[2];                          // position of this thread's two rows, -1: padding row; its first key
+  const float* brow[2];                         // its head's biases
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int m = warp * 16 + i * 8 + (lane >> 2);
-    qpos[i] = (m / rt < nt && m % rt < nh) ? pos0 + m / rt : -1;
+    const bool in = m / rt < nt && m % rt < nh;
+    qpos[i] = in ? pos0 + m / rt : -1;
+    qlo[i] = in ? first_key(a, qpos[i]) : 0;
+    brow[i] = kBias ? a.bias + static_cast<int64_t>(h0 + (in ? m % rt : 0)) * a.bias_len : nullptr;
   }
-  // lowest and highest position among the warp's 16 rows; -1 with a padding row among them
+  // lowest position among the warp's 16 rows; -1 with a padding row among them
   const int warp_lo = __reduce_min_sync(0xffffffffu, min(qpos[0], qpos[1]));
-  const int warp_hi = __reduce_max_sync(0xffffffffu, max(qpos[0], qpos[1]));
+  const int warp_qlo = __reduce_max_sync(0xffffffffu, max(qlo[0], qlo[1]));     // the last first key of a row
   const ScoreMap map(fabsf(a.scale), a.softcap);
   float o[DP / 8][4], mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.0f, 0.0f};
 #pragma unroll
@@ -189,15 +134,34 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
     }
     // every row of this warp sees the whole stage, unless it reaches past a row's own position or before its window
     const int p0 = keys.position(k0);
-    const bool edge = warp_lo < 0 || keys.position(k0 + kKeys - 1) > warp_lo || (a.window > 0 && p0 <= warp_hi - a.window);
+    const bool edge = warp_lo < 0 || keys.position(k0 + kKeys - 1) > warp_lo || p0 < warp_qlo;
     float tmax[2] = {-INFINITY, -INFINITY};
+    if constexpr (kBias) {
+      const bool far = warp_lo >= 0 && warp_lo - keys.position(k0 + kKeys - 1) >= a.bias_len - 1;
+      float b[2] = {0.0f, 0.0f};
+      if (far) {
+        b[0] = __ldg(brow[0] + a.bias_len - 1);
+        b[1] = __ldg(brow[1] + a.bias_len - 1);
+      }
+#pragma unroll
+      for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          float bias = b[e >> 1];
+          if (!far) {
+            const int dist = qpos[e >> 1] - keys.position(k0 + n * 8 + (lane & 3) * 2 + (e & 1));
+            bias = __ldg(brow[e >> 1] + min(max(dist, 0), a.bias_len - 1));
+          }
+          sc[n][e] = fmaf(bias, kLog2e, map(sc[n][e]));
+        }
+    }
     if (edge) {
 #pragma unroll
       for (int n = 0; n < 8; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int j = keys.position(k0 + n * 8 + (lane & 3) * 2 + (e & 1)), qp = qpos[e >> 1];
-          if (!(j <= qp && (a.window <= 0 || j > qp - a.window || j < a.keep_first))) sc[n][e] = -INFINITY;
+          const int j = keys.position(k0 + n * 8 + (lane & 3) * 2 + (e & 1));
+          if (!(j <= qpos[e >> 1] && (j >= qlo[e >> 1] || j < a.keep_first))) sc[n][e] = -INFINITY;
         }
     }
 #pragma unroll
@@ -209,7 +173,7 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
     for (int i = 0; i < 2; ++i) {
       tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 1));
       tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 2));
-      const float nm = fmaxf(mx[i], map(tmax[i]));
+      const float nm = fmaxf(mx[i], kBias ? tmax[i] : map(tmax[i]));
       base[i] = nm == -INFINITY ? 0.0f : nm;
       const float alpha = ex2_approx(mx[i] - base[i]);     // first stage: 2^-inf = 0
       mx[i] = nm;
@@ -224,7 +188,9 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
     for (int n = 0; n < 8; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        sc[n][e] = edge && sc[n][e] == -INFINITY ? 0.0f : map.prob(sc[n][e], base[e >> 1]);
+        sc[n][e] = edge && sc[n][e] == -INFINITY ? 0.0f
+                   : kBias                       ? ex2_approx(sc[n][e] - base[e >> 1])
+                                                 : map.prob(sc[n][e], base[e >> 1]);
         sum[e >> 1] += sc[n][e];
       }
 #pragma unroll
@@ -251,7 +217,8 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
     const float g = a.gate != nullptr ? a.gate[(row0 + m / rt) * a.heads + h0 + m % rt] : 1.0f;
     if (a.sink != nullptr) sum[i] += exp2f(a.sink[h0 + m % rt] * kLog2e - mx[i]);
     const float inv = a.out_scale * g / sum[i];
-    __nv_bfloat16* op = out + (row0 + m / rt) * a.ldo + static_cast<int64_t>(h0 + m % rt) * a.vdim;
+    const int64_t slice = a.all_values ? static_cast<int64_t>(h0 + m % rt) * a.kv_heads + blockIdx.z : h0 + m % rt;
+    __nv_bfloat16* op = out + (row0 + m / rt) * a.ldo + slice * a.vdim;
 #pragma unroll
     for (int n = 0; n < DP / 8; ++n) {
       const int d = n * 8 + (lane & 3) * 2;
@@ -265,7 +232,7 @@ paged_prefill_kernel(const NxPagedWindowArgs a, int rt, int tq, int head_tiles) 
 // decoding: grid (segments, kv_heads * head tiles, splits); the 4 warps take 16 keys each of every
 // 64-key stage, with their own running softmax, and merge at the end
 // ------------------------------------------------------------------------------------------------
-template <int DP>
+template <int DP, bool kBias>
 __global__ void __launch_bounds__(128)
 paged_decode_mma_kernel(const NxPagedWindowArgs a, int head_tiles) {
   constexpr int LD = DP + 8;
@@ -280,7 +247,7 @@ paged_decode_mma_kernel(const NxPagedWindowArgs a, int head_tiles) {
   const int rep = a.heads / a.kv_heads, h0 = hk * rep + ht * 16, nh = min(16, rep - ht * 16);
   const int pos = a.seg.pos[sg];
   const int64_t row = a.seg.row0[sg];
-  const KvSource src(a, a.seg.seq[sg], hk);
+  const KvSource src(a, a.seg.seq[sg], hk, hk);
   const KeyRange keys(a, pos, pos);
   const int per = ((keys.count + kKeys - 1) / kKeys + a.splits - 1) / a.splits * kKeys;
   const int first = static_cast<int>(blockIdx.z) * per, last = min(keys.count, first + per) - 1;
@@ -330,6 +297,11 @@ paged_decode_mma_kernel(const NxPagedWindowArgs a, int head_tiles) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int j = k0 + warp * 16 + n * 8 + (lane & 3) * 2 + (e & 1);
+          if constexpr (kBias) {
+            const int m = min((e >> 1) * 8 + (lane >> 2), nh - 1);
+            const int dist = min(max(pos - keys.position(j), 0), a.bias_len - 1);
+            sc[n][e] = fmaf(__ldg(a.bias + static_cast<int64_t>(h0 + m) * a.bias_len + dist), kLog2e, map(sc[n][e]));
+          }
           sc[n][e] = j <= last ? sc[n][e] : -INFINITY;
           tmax[e >> 1] = fmaxf(tmax[e >> 1], sc[n][e]);
         }
@@ -337,7 +309,7 @@ paged_decode_mma_kernel(const NxPagedWindowArgs a, int head_tiles) {
       for (int i = 0; i < 2; ++i) {
         tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 1));
         tmax[i] = fmaxf(tmax[i], __shfl_xor_sync(0xffffffffu, tmax[i], 2));
-        const float nm = fmaxf(mx[i], map(tmax[i]));  // at least one key of this warp is in range
+        const float nm = fmaxf(mx[i], kBias ? tmax[i] : map(tmax[i]));  // at least one key of this warp is in range
         const float alpha = ex2_approx(mx[i] - nm);
         mx[i] = nm;
         sum[i] *= alpha;
@@ -351,7 +323,7 @@ paged_decode_mma_kernel(const NxPagedWindowArgs a, int head_tiles) {
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          sc[n][e] = sc[n][e] == -INFINITY ? 0.0f : map.prob(sc[n][e], mx[e >> 1]);
+          sc[n][e] = sc[n][e] == -INFINITY ? 0.0f : kBias ? ex2_approx(sc[n][e] - mx[e >> 1]) : map.prob(sc[n][e], mx[e >> 1]);
           sum[e >> 1] += sc[n][e];
         }
       const uint32_t pa[4] = {bf16_pair(sc[0][0], sc[0][1]), bf16_pair(sc[0][2], sc[0][3]), bf16_pair(sc[1][0], sc[1][1]),
@@ -443,13 +415,14 @@ __global__ void __launch_bounds__(128) paged_window_f32_kernel(const NxPagedWind
   __shared__ int64_t s_slot[128];
   float* sQ = sf;               // [dim]
   float* sP = sf + a.dim;       // [128]
-  const int t = blockIdx.x, h = blockIdx.y, sg = blockIdx.z;
+  const int nv = a.all_values ? a.kv_heads : 1;
+  const int t = blockIdx.x, h = blockIdx.y / nv, sg = blockIdx.z;
   if (t >= a.seg.len[sg]) return;
   const int hk = h / (a.heads / a.kv_heads), pos = a.seg.pos[sg] + t, tid = threadIdx.x;
   const int64_t row = static_cast<int64_t>(a.seg.row0[sg]) + t;
   const int32_t* bt = a.block_table + static_cast<int64_t>(a.seg.seq[sg]) * a.max_blocks;
   const float* kc = static_cast<const float*>(a.k_cache);
-  const float* vc = static_cast<const float*>(a.v_cache);
+  const float* vc = static_cast<const float*>(a.v_cache) + (a.all_values ? blockIdx.y % nv : hk) * a.vdim;
   for (int d = tid; d < a.dim; d += 128) sQ[d] = static_cast<const float*>(a.q)[row * a.ldq + static_cast<int64_t>(h) * a.dim + d];
   float acc[kF32Cols], mx = -INFINITY, sum = 0.0f;
 #pragma unroll
@@ -467,6 +440,7 @@ __global__ void __launch_bounds__(128) paged_window_f32_kernel(const NxPagedWind
       for (int d = 0; d < a.dim; ++d) s += sQ[d] * k[d];
       sc = s * a.scale;
       if (a.softcap > 0.0f) sc = a.softcap * tanhf(sc / a.softcap);
+      if (a.bias != nullptr) sc += a.bias[static_cast<int64_t>(h) * a.bias_len + min(pos - j, a.bias_len - 1)];
     }
     const float nm = fmaxf(mx, block_max(sc, s_red));
     const float p = expf(sc - nm), alpha = expf(mx - nm);
@@ -479,7 +453,7 @@ __global__ void __launch_bounds__(128) paged_window_f32_kernel(const NxPagedWind
       const int d = tid + c * 128;
       if (d < a.vdim) {
         float v = acc[c] * alpha;
-        for (int i = 0; i < n; ++i) v += sP[i] * vc[s_slot[i] * a.v_pitch + hk * a.vdim + d];
+        for (int i = 0; i < n; ++i) v += sP[i] * vc[s_slot[i] * a.v_pitch + d];
         acc[c] = v;
       }
     }
@@ -488,13 +462,14 @@ __global__ void __launch_bounds__(128) paged_window_f32_kernel(const NxPagedWind
   if (a.sink != nullptr) sum += expf(a.sink[h] - mx);
   for (int c = 0; c < kF32Cols; ++c) {
     const int d = tid + c * 128;
-    if (d < a.vdim) static_cast<float*>(a.out)[row * a.ldo + static_cast<int64_t>(h) * a.vdim + d] = acc[c] / sum * (a.out_scale * g);
+    if (d < a.vdim) static_cast<float*>(a.out)[row * a.ldo + static_cast<int64_t>(blockIdx.y) * a.vdim + d] = acc[c] / sum * (a.out_scale * g);
   }
 }
 
 int check_paged(const NxPagedWindowArgs* a, int dtype) {
   if (a == nullptr || a->dtype != dtype || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads) return -1;
   if (a->keep_first < 0 || a->dim <= 0 || a->vdim <= 0 || a->block_size <= 0 || a->max_blocks <= 0 || a->seg.count > 65535) return -1;
+  if (a->chunk < 0 || (a->bias != nullptr && a->bias_len <= 0)) return -1;
   if (a->k_pitch < static_cast<int64_t>(a->kv_heads) * a->dim || a->v_pitch < static_cast<int64_t>(a->kv_heads) * a->vdim) return -1;
   return 0;
 }
@@ -503,29 +478,38 @@ int padded_dim(const NxPagedWindowArgs* a) {
   return d <= 32 ? 32 : d <= 64 ? 64 : d <= 128 ? 128 : d <= 256 ? 256 : 0;
 }
 
-template <int DP>
-int launch_prefill(const NxPagedWindowArgs* a, dim3 grid, int rt, int tq, int head_tiles, cudaStream_t st) {
+template <int DP, bool kBias>
+int launch_prefill_as(const NxPagedWindowArgs* a, dim3 grid, int rt, int tq, int head_tiles, cudaStream_t st) {
   constexpr int kSmem = (kRows + 4 * kKeys) * (DP + 8) * 2;
   static bool once = false;
   if (!once) {
-    if (cudaFuncSetAttribute(paged_prefill_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -2;
+    if (cudaFuncSetAttribute(paged_prefill_kernel<DP, kBias>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -2;
     once = true;
   }
-  paged_prefill_kernel<DP><<<grid, kRows * 2, kSmem, st>>>(*a, rt, tq, head_tiles);
+  paged_prefill_kernel<DP, kBias><<<grid, kRows * 2, kSmem, st>>>(*a, rt, tq, head_tiles);
   return launch_status();
 }
-
 template <int DP>
-int launch_decode(const NxPagedWindowArgs* a, dim3 grid, int head_tiles, cudaStream_t st) {
+int launch_prefill(const NxPagedWindowArgs* a, dim3 grid, int rt, int tq, int head_tiles, cudaStream_t st) {
+  return a->bias != nullptr ? launch_prefill_as<DP, true>(a, grid, rt, tq, head_tiles, st)
+                            : launch_prefill_as<DP, false>(a, grid, rt, tq, head_tiles, st);
+}
+
+template <int DP, bool kBias>
+int launch_decode_as(const NxPagedWindowArgs* a, dim3 grid, int head_tiles, cudaStream_t st) {
   constexpr int kSmem = (16 + 4 * kKeys) * (DP + 8) * 2;
   static_assert(4 * kKeys * (DP + 8) * 2 >= 4 * 16 * DP * 4, "partial outputs reuse the stages");
   static bool once = false;
   if (!once) {
-    if (cudaFuncSetAttribute(paged_decode_mma_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -2;
+    if (cudaFuncSetAttribute(paged_decode_mma_kernel<DP, kBias>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem) != cudaSuccess) return -2;
     once = true;
   }
-  paged_decode_mma_kernel<DP><<<grid, 128, kSmem, st>>>(*a, head_tiles);
+  paged_decode_mma_kernel<DP, kBias><<<grid, 128, kSmem, st>>>(*a, head_tiles);
   return launch_status();
+}
+template <int DP>
+int launch_decode(const NxPagedWindowArgs* a, dim3 grid, int head_tiles, cudaStream_t st) {
+  return a->bias != nullptr ? launch_decode_as<DP, true>(a, grid, head_tiles, st) : launch_decode_as<DP, false>(a, grid, head_tiles, st);
 }
 
 }  // namespace
@@ -536,7 +520,7 @@ extern "C" int nx_paged_window_prefill(const NxPagedWindowArgs* a, nx_stream_t s
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int rep = a->heads / a->kv_heads;
   const int rt = std::min(rep, 16), head_tiles = (rep + rt - 1) / rt, tq = kRows / rt;
-  dim3 grid(a->seg.total_len / tq + a->seg.count, a->kv_heads * head_tiles);
+  dim3 grid(a->seg.total_len / tq + a->seg.count, a->kv_heads * head_tiles, a->all_values ? a->kv_heads : 1);
   switch (padded_dim(a)) {
     case 32: return launch_prefill<32>(a, grid, rt, tq, head_tiles, st);
     case 64: return launch_prefill<64>(a, grid, rt, tq, head_tiles, st);
@@ -547,7 +531,7 @@ extern "C" int nx_paged_window_prefill(const NxPagedWindowArgs* a, nx_stream_t s
 }
 
 extern "C" int nx_paged_window_decode(const NxPagedWindowArgs* a, nx_stream_t stream) {
-  if (check_paged(a, NX_BF16) || a->splits < 1 || a->splits > 65535) return -1;
+  if (check_paged(a, NX_BF16) || a->splits < 1 || a->splits > 65535 || a->all_values) return -1;
   if (a->splits > 1 && (a->part_o == nullptr || a->part_ml == nullptr)) return -1;
   if (a->seg.count <= 0) return 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
@@ -571,7 +555,7 @@ extern "C" int nx_paged_window_decode(const NxPagedWindowArgs* a, nx_stream_t st
 extern "C" int nx_paged_window_f32(const NxPagedWindowArgs* a, nx_stream_t stream) {
   if (check_paged(a, NX_F32) || a->vdim > 128 * kF32Cols || a->dim > 4096) return -1;
   if (a->seg.count <= 0 || a->seg.max_len <= 0) return 0;
-  dim3 grid(a->seg.max_len, a->heads, a->seg.count);
+  dim3 grid(a->seg.max_len, a->heads * (a->all_values ? a->kv_heads : 1), a->seg.count);
   paged_window_f32_kernel<<<grid, 128, (a->dim + 128) * sizeof(float), static_cast<cudaStream_t>(stream)>>>(*a);
   return launch_status();
 }

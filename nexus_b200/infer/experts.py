@@ -72,11 +72,11 @@ def route(engine, tok) -> List[Optional[object]]:
     from ..ops import _experts as X
     routes: List[Optional[object]] = [None] * engine.L
     by_align = {}
-    for i, layer in enumerate(engine.model.layers):
+    for i, layer in enumerate(engine.runs):
         if layer.experts is not None and layer.experts.router is None:
             by_align.setdefault(alignment(engine, layer.experts, tok.shape[0]), []).append(i)
     for align, which in by_align.items():
-        got = X.table_route(tok, [(engine.layers[i]["ff"]["table"], engine.model.layers[i].experts.experts) for i in which], align)
+        got = X.table_route(tok, [(engine.layers[i]["ff"]["table"], engine.runs[i].experts.experts) for i in which], align)
         for i, r in zip(which, got):
             routes[i] = r
     return routes

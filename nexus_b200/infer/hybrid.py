@@ -11,11 +11,11 @@ per sequence) in up to three groups, one-token segments, short ones and long one
 
 * attention: split-key decode kernel | paged prompt kernel | tcgen05 flash kernel (fresh prompts, head sizes 64 / 128)
 * recurrences: token-by-token kernel with the state tile in shared memory | chunked tensor-core kernel
-* latent attention: `latent`; attention over convolved projections: `conv_attention`; gated linear attention: `gla`;
-  feed-forwards of experts: `experts`; the long segments of a step on the prompt kernels: `prompt`
+* latent attention: `latent`; attention over convolved projections: `conv_attention`; attention on normed queries and keys:
+  `normed_attention`; gated linear attention: `gla`; feed-forwards of experts: `experts`; the long segments of a step on the prompt kernels: `prompt`
 
-The residual stream is FP32; one kernel adds a sublayer output (normed or not) to it and prepares it for the next sublayer.  In FP32
-precision the same layer loop runs the kernels' FP32 forms and plain FP32 matrix products.
+The residual stream is FP32; one kernel adds a sublayer output (normed or not) to it and prepares it for the next sublayer, also where
+the residual is several streams.  A layer that runs several times has a cache of its own for every run.  In FP32 precision the same layer loop runs the kernels' FP32 forms and plain FP32 matrix products.
 """
 from __future__ import annotations
 
@@ -25,9 +25,10 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from ..lm.config import RopeScaling
-from ..lm.hybrid import GLU_ACTS, ConvAttentionSpec, DeltaSpec, GlaSpec, HybridConfig, HybridWeights, LatentSpec, ParallelSpec
+from ..lm.hybrid import (GLU_ACTS, PLAIN_ACTS, ConvAttentionSpec, DeltaSpec, GlaSpec, HybridConfig, HybridWeights, LatentSpec,
+                         NormedAttentionSpec, ParallelSpec)
 from ..lm.rope import rope_inv_freq
-from . import conv_attention, experts, gla, latent, prompt
+from . import conv_attention, experts, gla, latent, normed_attention, prompt
 from .engine import Chunk, Engine, _Linear
 
 __all__ = ["HybridEngine"]
@@ -56,7 +57,8 @@ class HybridEngine(Engine):
         if not self.fast:
             torch.backends.cuda.matmul.allow_tf32 = False
         self.model: HybridConfig = weights.config
-        self.L, self.d, self.V = len(self.model.layers), self.model.width, self.model.vocab
+        self.runs = self.model.runs               # the layers in the order they run, some of them several times
+        self.L, self.d, self.V = len(self.runs), self.model.width, self.model.vocab
         for i, layer in enumerate(self.model.layers):
             m = layer.mixer
             if self.fast and isinstance(m, ParallelSpec) and max(m.left.dim, m.left.vdim) > 256:
@@ -65,6 +67,8 @@ class HybridEngine(Engine):
                 latent.check(self, i, m)
             if isinstance(m, ConvAttentionSpec):
                 conv_attention.check(self, i, m)
+            if isinstance(m, NormedAttentionSpec):
+                normed_attention.check(self, i, m)
             if layer.experts and layer.experts.shared and self.model.pre_norm:
                 raise ValueError(f"layer {i}: the gate of the shared expert reads the residual stream, which this design norms first")
         self.adt = torch.bfloat16 if self.fast else torch.float32
@@ -73,11 +77,14 @@ class HybridEngine(Engine):
         self._kv_tok_bytes = max(1, self.model.kv_bytes_per_token(elem))
         self.n_blocks = self._pool_blocks(self._kv_tok_bytes)
         self.ctx = cfg.context if cfg.context > 0 else self.n_blocks * cfg.block_size
+        if self.model.positions:
+            self.ctx = min(self.ctx, self.model.positions)
         self._rope: Dict[tuple, tuple] = {}
         self._short_len = 16 if self.fast else 1 << 30
         mixers = [layer.mixer for layer in self.model.layers]
         self._prompt_windows = {prompt.Window(m.window) for m in mixers if isinstance(m, LatentSpec) and latent.expandable(m)} | {
-            conv_attention.window(m) for m in mixers if isinstance(m, ConvAttentionSpec) and conv_attention.promptable(m)}
+            conv_attention.window(m) for m in mixers if isinstance(m, ConvAttentionSpec) and conv_attention.promptable(m)} | {
+            normed_attention.window(m) for m in mixers if isinstance(m, NormedAttentionSpec) and normed_attention.promptable(m)}
 
     def _rope_tables(self, dims: int, base: float, scaling: Optional[RopeScaling] = None):
         """cos / sin [ctx, dims / 2]: angles in double, kept in FP32."""
@@ -118,7 +125,8 @@ class HybridEngine(Engine):
         self.head, _ = self._pack([head])
         self.embed = t["embed"].to(self.dev, self.adt).contiguous()
         self.side_embed = t["side.embed"].to(self.dev, self.adt).contiguous() if model.token_side else None
-        self.weight_nbytes += sum(e.numel() * e.element_size() for e in (self.embed, self.side_embed) if e is not None)
+        self.pos_embed = t["pos"].to(self.dev, self.adt).contiguous() if model.positions else None
+        self.weight_nbytes += sum(e.numel() * e.element_size() for e in (self.embed, self.side_embed, self.pos_embed) if e is not None)
         self.final_norm = self._f32(t["final.norm"]) + model.norm_offset
         self.layers: List[dict] = []
         for i, layer in enumerate(model.layers):
@@ -130,7 +138,10 @@ class HybridEngine(Engine):
                     out["pre" + k] = self._f32(t[p + "norm" + k]) + model.norm_offset if model.pre_norm else None
                     name = p + "norm" + k + ("b" if model.pre_norm else "")
                     out["post" + k] = self._f32(t[name]) + model.norm_offset if model.post_norm else None
-            module = {LatentSpec: latent, ConvAttentionSpec: conv_attention, GlaSpec: gla}.get(type(m))
+                    if model.streams:
+                        out["hc" + k] = {n: self._f32(t[p + f"hc{k}.{n}"]) for n in ("in", "out", "mix")}
+            module = {LatentSpec: latent, ConvAttentionSpec: conv_attention, NormedAttentionSpec: normed_attention,
+                      GlaSpec: gla}.get(type(m))
             if module is not None:
                 out["mix"] = module.load(self, m, lambda n: t[p + "mix." + n])
             elif isinstance(m, ParallelSpec):
@@ -162,7 +173,10 @@ class HybridEngine(Engine):
                     out[key] = self._f32(t[p + "mix." + n])
             if layer.experts:
                 out["ff"] = experts.load(self, layer.experts, lambda n: t[p + "mlp." + n])
-            if layer.ff:
+            if layer.ff and layer.act in PLAIN_ACTS:
+                for n in ("up", "down"):
+                    out[n], _ = self._pack([t[p + "mlp." + n]], bias=t[p + f"mlp.{n}.b"] if layer.ff_bias else None)
+            elif layer.ff:
                 out["up"], _ = self._pack([experts.in_turns(t[p + "mlp.gate"], t[p + "mlp.up"])])
                 out["down"], _ = self._pack([t[p + "mlp.down"]])
             if model.token_side:
@@ -170,6 +184,7 @@ class HybridEngine(Engine):
                 out["side_proj"], _ = self._pack([t[p + "side.proj"]])
                 out["side_norm"] = self._f32(t[p + "side.norm"])
             self.layers.append(out)
+        self.layers = [self.layers[i] for i in model.order]
 
     # ----------------------------------------------------------------------------- cache pages and state slots
     def _alloc_kv(self) -> None:
@@ -179,10 +194,13 @@ class HybridEngine(Engine):
         self.v_cache: list = [None] * self.L
         self.state: list = [None] * self.L        # FP32 [slots, heads, key size, value size]
         self.conv_tail: list = [None] * self.L    # [slots, taps - 1, channels]
-        for i, layer in enumerate(self.model.layers):
+        for i, layer in enumerate(self.runs):
             m = layer.mixer
             if isinstance(m, ConvAttentionSpec):
                 conv_attention.alloc(self, i, m)
+                continue
+            if isinstance(m, NormedAttentionSpec):
+                normed_attention.alloc(self, i, m)
                 continue
             if isinstance(m, GlaSpec):
                 self.state[i] = torch.zeros((cfg.max_seqs, m.heads, m.dim, m.vdim), dtype=torch.float32, device=self.dev)
@@ -250,10 +268,15 @@ class HybridEngine(Engine):
         ld = _pad8(cols)
         return (torch.zeros if ld != cols else torch.empty)((rows, ld), dtype=self.adt, device=self.dev)
 
+    def _most_keys(self, a) -> int:
+        """The most keys a row can see."""
+        sizes = [n for n in (a.window, getattr(a, "chunk", 0)) if n > 0]
+        return min(min(sizes) + getattr(a, "keep_first", 0), self.ctx) if sizes else self.ctx
+
     def _decode_splits(self, a, rows: int) -> int:
         if self.cfg.decode_splits > 0:
             return self.cfg.decode_splits
-        keys = min(a.window + getattr(a, "keep_first", 0), self.ctx) if a.window > 0 else self.ctx
+        keys = self._most_keys(a)
         ctas = rows * a.kv_heads * (-(-(a.heads // a.kv_heads) // 16))
         return max(1, min(592 // max(ctas, 1), -(-keys // 256), 32))
 
@@ -363,11 +386,19 @@ class HybridEngine(Engine):
         M.glu(both, act, glu, interleaved=True)
         return act
 
+    def _plain(self, h, lw: dict, act: str) -> torch.Tensor:
+        """A feed-forward without a gate."""
+        if self.fast:
+            return self._linear(self._linear(h, lw["up"], act=act), lw["down"])
+        return self._linear(torch.relu(self._linear(h, lw["up"])).square_(), lw["down"])
+
     def _mixer(self, i: int, m, lw: dict, h, pos, slot) -> torch.Tensor:
         if isinstance(m, LatentSpec):
             return latent.mixer(self, i, m, lw["mix"], h, pos, slot)
         if isinstance(m, ConvAttentionSpec):
             return conv_attention.mixer(self, i, m, lw["mix"], h, slot)
+        if isinstance(m, NormedAttentionSpec):
+            return normed_attention.mixer(self, i, m, lw["mix"], h, pos, slot)
         if isinstance(m, GlaSpec):
             return gla.mixer(self, i, m, lw["mix"], h)
         if isinstance(m, ParallelSpec):
@@ -378,17 +409,31 @@ class HybridEngine(Engine):
         from ..ops import _mixers as M
         n, eps, model, cap = tok.shape[0], self.model.norm_eps, self.model, self._capture
         mult = model.residual_mult
-        x = torch.empty((n, self.d), dtype=torch.float32, device=self.dev)
+        streams = model.streams
+        x = torch.empty((n, streams, self.d) if streams else (n, self.d), dtype=torch.float32, device=self.dev)
         h = torch.empty((n, _pad8(self.d)), dtype=self.adt, device=self.dev)
         routes = experts.route(self, tok)
 
-        def feed(norm) -> dict:      # what the next sublayer reads
+        # one kernel between two sublayers: `took(lw, k)` says how the output of sublayer k of a layer joins the residual, `feed(lw, k)`
+        # what sublayer k reads of it
+        residual = M.stream_residual if streams else M.residual_norm
+
+        def feed(lw, k: str) -> dict:
+            norm = lw["pre" + k]
+            if streams:
+                return {"w_next": norm, "h": h, "read": lw["hc" + k]["in"]}
             return {"w_next": norm, "h": h} if norm is not None else {"x_cast": h}
-        M.residual_norm(x, tokens=tok, table=self.embed, eps=eps, embed_scale=model.embed_scale, **feed(self.layers[0]["pre1"]))
-        for i, (layer, lw) in enumerate(zip(model.layers[:nl], self.layers)):
-            more = feed(self.layers[i + 1]["pre1"]) if i + 1 < nl else {}
+
+        def took(lw, k: str) -> dict:
+            if streams:
+                return {"mix": lw["hc" + k]["mix"], "out": lw["hc" + k]["out"]}
+            return {"w_post": lw["post" + k], "res_mult": mult}
+        residual(x, tokens=tok, table=self.embed, eps=eps, embed_scale=model.embed_scale, positions=pos, pos_table=self.pos_embed,
+                 **feed(self.layers[0], "1"))
+        for i, (layer, lw) in enumerate(zip(self.runs[:nl], self.layers)):
+            more = feed(self.layers[i + 1], "1") if i + 1 < nl else {}
             after = more if not model.token_side else {"x_cast": h}
-            y, add = self._mixer(i, layer.mixer, lw, h, pos, slot), {"w_post": lw["post1"]}
+            y, add = self._mixer(i, layer.mixer, lw, h, pos, slot), took(lw, "1")
             if layer.experts:
                 f, ff, r = layer.experts, lw["ff"], routes[i]
                 extra, by_slot = {}, None
@@ -398,17 +443,20 @@ class HybridEngine(Engine):
                 if r is not None and r.align >= 128:
                     by_slot = torch.empty((r.max_slots, h.shape[1]), dtype=self.adt, device=self.dev)
                     extra.update(scatter=by_slot, slots=r.slots, top=r.top)
-                M.residual_norm(x, y=y, eps=eps, res_mult=mult, **add, **feed(lw["pre2"]), **extra)
+                residual(x, y=y, eps=eps, **add, **feed(lw, "2"), **extra)
                 if f.router:
                     r, by_slot = experts.gate(self, f, ff, h)
                 rows, y = experts.forward(self, f, ff, r, h, by_slot)
-                add = {"w_post": lw["post2"], "experts": rows, "slots": r.slots, "top": r.top,
+                add = {**took(lw, "2"), "experts": rows, "slots": r.slots, "top": r.top,
                        "weights": r.weight, "y_gate": gate if f.shared else None}
             elif layer.ff:
-                M.residual_norm(x, y=y, eps=eps, res_mult=mult, **add, **feed(lw["pre2"]))
-                act = self._gated(h, lw["up"], M.Glu(GLU_ACTS.index(layer.act)))
-                y, add = self._linear(act, lw["down"]), {"w_post": lw["post2"]}
-            M.residual_norm(x, y=y, eps=eps, res_mult=mult, **add, **after)
+                residual(x, y=y, eps=eps, **add, **feed(lw, "2"))
+                if layer.act in PLAIN_ACTS:
+                    y = self._plain(h, lw, layer.act)
+                else:
+                    y = self._linear(self._gated(h, lw["up"], M.Glu(GLU_ACTS.index(layer.act))), lw["down"])
+                add = took(lw, "2")
+            residual(x, y=y, eps=eps, **add, **after)
             if model.token_side:
                 gate = self._linear(h, lw["side_gate"], out_dtype=torch.float32)
                 side = torch.empty(gate.shape, dtype=self.adt, device=self.dev)
@@ -416,12 +464,12 @@ class HybridEngine(Engine):
                 y = self._linear(side, lw["side_proj"])
                 M.residual_norm(x, y=y, w_post=lw["side_norm"], eps=eps, res_mult=mult, **more)
             if cap is not None:
-                cap.append(x.detach().float().cpu())
+                cap.append((x.sum(1) if streams else x.detach()).float().cpu())
         if logit_rows.shape[0] == 0:
             return torch.zeros((0, self.Vp), dtype=torch.float32, device=self.dev)
         xr = x.index_select(0, logit_rows.long())
         hr = torch.empty((xr.shape[0], _pad8(self.d)), dtype=self.adt, device=self.dev)
-        M.residual_norm(xr, w_next=self.final_norm, h=hr, eps=eps)
+        residual(xr, w_next=self.final_norm, h=hr, eps=eps)
         logits = self._linear(hr, self.head, out_dtype=torch.float32)
         if model.logit_softcap > 0 or model.logit_scale != 1.0:
             M.softcap_(logits, self.V, model.logit_softcap, model.logit_scale)

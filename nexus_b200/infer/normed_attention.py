@@ -1,0 +1,134 @@
+"""Attention on normed queries and keys (`lm.hybrid.NormedAttentionSpec`) on the engine.
+
+One projection gives q, k, v and the output gate; one kernel norms q and k (and v), applies every factor of the scores to q (scale,
+the head's factor, the position's temperature), appends k and v to the cache pages and takes the gate's sigmoid.  Heads are
+zero-padded to sizes the kernels load in whole vectors; norms count the real columns.
+
+Heads that mix their weights after the softmax.  out_h = sum_g T[h, g] (P_g V of the KV head of h), so:
+
+* decoding: scores of all heads, then per KV head the mixture of the normalised weights and one product with its values;
+* prompts: every head's weights meet the values of every KV head inside the attention kernel, and the mixture is taken over those
+  outputs."""
+from __future__ import annotations
+
+import torch
+
+from ..lm.hybrid import NormedAttentionSpec
+from .conv_attention import _pad, _pad_heads
+from .prompt import Window
+
+
+class NormedAttentionShape:
+    """Padded sizes of one layer."""
+
+    def __init__(self, m: NormedAttentionSpec):
+        self.dim, self.vdim = _pad(m.dim, 16), _pad(m.vdim, 8)
+        self.q, self.k, self.v = m.heads * self.dim, m.kv_heads * self.dim, m.kv_heads * self.vdim
+        self.offsets = (0, self.q, self.q + self.k, self.q + self.k + self.v)      # q, k, v, gate
+        self.values = m.kv_heads if m.talk else 1        # KV heads whose values a query head meets
+
+
+def check(engine, i: int, m: NormedAttentionSpec) -> None:
+    from ..ops import _mixers as M
+    s = NormedAttentionShape(m)
+    if engine.fast and max(s.dim, s.vdim) > 256:
+        raise ValueError(f"layer {i}: the BF16 attention kernels take head sizes up to 256")
+    if not engine.fast and s.vdim > 1024:
+        raise ValueError(f"layer {i}: the FP32 kernel takes value sizes up to 1024")
+    if m.talk and m.heads > M.TALK_MAX_HEADS:
+        raise ValueError(f"layer {i}: up to {M.TALK_MAX_HEADS} heads mix their weights")
+
+
+def load(engine, m: NormedAttentionSpec, get) -> dict:
+    """``get(name)``: the mixer's tensors."""
+    s = NormedAttentionShape(m)
+    parts = (("q", m.heads, s.dim), ("k", m.kv_heads, s.dim), ("v", m.kv_heads, s.vdim))
+
+    def stack(suffix):
+        return torch.cat([_pad_heads(get(n + suffix), heads, size) for n, heads, size in parts], 0)
+    out = {"shape": s}
+    w = torch.cat([stack("")] + ([get("g").float()] if m.gate else []), 0)
+    out["in"], _ = engine._pack([w], bias=stack(".b") if m.bias else None)
+    wo = torch.zeros((engine.d, m.heads, s.vdim))
+    wo[:, :, : m.vdim] = get("o").float().view(engine.d, m.heads, m.vdim)
+    out["out"], _ = engine._pack([wo.view(engine.d, m.heads * s.vdim)], bias=get("o.b") if m.bias else None)
+    for n, heads in (("q", m.heads), ("k", m.kv_heads)):
+        out[n + "_norm"] = engine._f32(_pad_heads(get(n + ".norm"), heads if m.norm == "all" else 1, s.dim))
+    out["head_scale"] = engine._f32(get("temp")) if m.head_scale else None
+    out["talk"] = engine._f32(get("talk")) if m.talk else None
+    out["bias"] = None
+    if m.distance is not None:      # one entry per distance; the last one counts for all beyond
+        rows = [m.distance.bucket(n) for n in range(m.distance.far + 1)]
+        while len(rows) > 1 and rows[-1] == rows[-2]:
+            rows.pop()
+        out["bias"] = engine._f32(get("rel").float()[rows].t())
+    return out
+
+
+def alloc(engine, i: int, m: NormedAttentionSpec) -> None:
+    s, cfg = NormedAttentionShape(m), engine.cfg
+    for cache, size in ((engine.k_cache, s.dim), (engine.v_cache, s.vdim)):
+        cache[i] = torch.zeros((engine.n_blocks, cfg.block_size, m.kv_heads, size), dtype=engine.adt, device=engine.dev)
+
+
+def window(m: NormedAttentionSpec) -> Window:
+    return Window(m.window, 0, m.chunk)
+
+
+def promptable(m: NormedAttentionSpec) -> bool:
+    """Whether the tcgen05 prompt kernel has this layer's sizes."""
+    from ..ops import _mixers as M
+    s = NormedAttentionShape(m)
+    return s.dim <= 128 and s.vdim <= 128 and m.softcap == 0 and (m.distance is None or m.distance.far < M.PROMPT_MAX_BIAS)
+
+
+def mixer(engine, i: int, m: NormedAttentionSpec, lw: dict, h, pos, slot):
+    from ..ops import _mixers as M
+    s, n = lw["shape"], h.shape[0]
+    single, short, long_ = engine._groups
+    step = engine._prompt_plan if promptable(m) else None
+    proj = engine._linear(h, lw["in"])
+    gate = torch.empty((n, m.heads), dtype=torch.float32, device=engine.dev) if m.gate else None
+    temp = m.temperature
+    M.head_prep(proj, s.offsets, heads=m.heads, kv_heads=m.kv_heads, dim=s.dim, vdim=s.vdim, norm_dim=m.dim, norm_vdim=m.vdim,
+                norm_all=m.norm == "all", unit_values=m.unit_values, store_kv=step is not None and not step.gathered,
+                eps=engine.model.norm_eps, q_scale=m.scale, head_scale=lw["head_scale"], coef=temp.coef if temp else 0.0,
+                every=temp.every if temp else 0, w_q=lw["q_norm"], w_k=lw["k_norm"], positions=pos, slots=slot,
+                k_cache=engine.k_cache[i], v_cache=engine.v_cache[i], gate=gate)
+    q = proj[:, : s.q]
+    out = torch.empty((n, m.heads * s.vdim), dtype=engine.adt, device=engine.dev)
+    # heads that mix: `wide` takes what the attention kernels give; decoding in BF16 writes `out` itself
+    mixed = m.talk and (not engine.fast or engine._many.count > 0)
+    wide = torch.empty((n, m.heads * s.values * s.vdim), dtype=engine.adt, device=engine.dev) if mixed else out
+    kw = dict(heads=m.heads, block_size=engine.cfg.block_size, window=m.window, chunk=m.chunk, scale=1.0, softcap=m.softcap,
+              bias=lw["bias"])
+    paged = (engine.k_cache[i], engine.v_cache[i], engine.block_table)
+    late = dict(gate=None if m.talk else gate, all_values=s.values > 1)
+
+    def attend(seg, **more):
+        if seg.count:
+            M.paged_window_attention(q, *paged, wide, seg, **kw, **late, **more)
+    if not engine.fast:
+        attend(engine._every)
+    elif step is None:
+        attend(engine._many)
+    else:
+        attend(short)
+        w = window(m)
+        if step.gathered:
+            k, v = (torch.empty((step.kv_rows[w], cols), dtype=engine.adt, device=engine.dev) for cols in (s.k, s.v))
+            for c, dst in ((engine.k_cache[i], k), (engine.v_cache[i], v)):
+                M.latent_gather(c, engine.block_table, step.runs[w], step.longest[w], dst)
+        else:
+            k, v = (proj[:, o: o + cols] for o, cols in zip(s.offsets[1:3], (s.k, s.v)))
+        M.window_prompt(q, k, v, wide, step.blocks[w], heads=m.heads, kv_heads=m.kv_heads, dim=s.dim, vdim=s.vdim, window=m.window,
+                        chunk=m.chunk, scale=1.0, bias=lw["bias"], **late)
+    if mixed:
+        M.head_mix(wide, lw["talk"], gate, out, heads=m.heads, kv_heads=m.kv_heads, vdim=s.vdim)
+    if engine.fast and single.count:
+        splits = engine._decode_splits(m, single.count)
+        if m.talk:
+            M.talk_decode(q, *paged, out, lw["talk"], single, keys=engine._most_keys(m), splits=splits, gate=gate, **kw)
+        else:
+            M.paged_window_attention(q, *paged, out, single, splits=splits, gate=gate, **kw)
+    return engine._linear(out, lw["out"])

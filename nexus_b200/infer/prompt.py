@@ -10,12 +10,25 @@ QUERY_BLOCK = 256    # query rows of one work item
 
 
 class Window(NamedTuple):
-    """What a layer's rows see: the last ``size`` keys (0: all of them) and the first ``keep_first`` ones."""
+    """What a layer's rows see: the last ``size`` keys (0: all of them), with ``chunk`` > 0 only those of the row's own chunk of
+    positions, and the first ``keep_first`` ones."""
     size: int
     keep_first: int = 0
+    chunk: int = 0
 
 
-def long_segments(segs, window: int, keep_first: int = 0):
+def _cuts(pos: int, count: int, chunk: int):
+    """(offset, rows) of the query blocks; chunks that fill a block end one."""
+    at = 0
+    while at < count:
+        rows = min(QUERY_BLOCK, count - at)
+        if chunk >= QUERY_BLOCK:
+            rows = min(rows, chunk - (pos + at) % chunk)
+        yield at, rows
+        at += rows
+
+
+def long_segments(segs, window: int, keep_first: int = 0, chunk: int = 0):
     """The work for segments (first row, rows, first position, sequence): (blocks, runs, rows of kv).
 
     A segment that does not start at position 0 needs keys of earlier steps: if there is one, all keys are gathered from the
@@ -23,11 +36,14 @@ def long_segments(segs, window: int, keep_first: int = 0):
     ``blocks``: first query row, rows, position of the first row, kv row of position 0 and, last, the row that position 0 has
     among the kept first keys; the most keys first."""
     back, blocks, runs, d = window - 1 if window > 0 else 1 << 30, [], [], 0
+
+    def first_key(p):
+        return max(0, p - back, p // chunk * chunk if chunk > 0 else 0)
     gather = any(pos > 0 for _, _, pos, _ in segs)
     for row0, count, pos, seq in segs:
         kv0 = kept0 = row0
         if gather:
-            base = max(0, pos - back)
+            base = first_key(pos)
             kept, kept0 = min(keep_first, base), d
             if kept:                          # in front of the keys from `base` on
                 runs.append((d, kept, 0, seq))
@@ -37,9 +53,8 @@ def long_segments(segs, window: int, keep_first: int = 0):
                 kept0 = kv0
             runs.append((d, pos + count - base, base, seq))
             d += pos + count - base
-        for b in range(0, count, QUERY_BLOCK):
-            rows = min(QUERY_BLOCK, count - b)
-            blocks.append((min(pos + b, back) + rows, row0 + b, rows, pos + b, kv0, kept0))
+        for b, rows in _cuts(pos, count, chunk):
+            blocks.append((pos + b - first_key(pos + b) + rows, row0 + b, rows, pos + b, kv0, kept0))
     blocks.sort(key=lambda x: -x[0])
     return [b[1:] for b in blocks], runs, d
 

@@ -12,6 +12,7 @@ from typing import Callable, Dict, Optional
 
 from ..lm.gutivik import load_gutivik
 from ..lm.hybrid import HybridWeights, load_gugedra
+from ..lm.lukopel import load_lukopel
 from ..lm.makuzen import load_makuzen
 from .engine import Engine, EngineConfig, Gpt2Weights, load_gpt2
 from .hybrid import HybridEngine
@@ -70,3 +71,4 @@ register_family(ModelFamily("GPT2", _load_gpt2_folder, Gpt2Weights, Engine))
 register_family(ModelFamily("Gugedra", load_gugedra, HybridWeights, HybridEngine))
 register_family(ModelFamily("Makuzen", load_makuzen, HybridWeights, HybridEngine))
 register_family(ModelFamily("Gutivik", load_gutivik, HybridWeights, HybridEngine))
+register_family(ModelFamily("Lukopel", load_lukopel, HybridWeights, HybridEngine))

@@ -1,8 +1,9 @@
 """Decoders whose layers differ from one another: the layer list, the mixers' sizes and constants, and the weights.
 
 A model is an ordered list of :class:`HybridLayer`; each has one mixer - :class:`AttentionSpec` and :class:`SsdSpec` side
-by side (:class:`ParallelSpec`), :class:`ConvAttentionSpec`, :class:`DeltaSpec`, :class:`GlaSpec` or :class:`LatentSpec` - and
-optionally a feed-forward, gated or of experts (:class:`ExpertsSpec`).  The engine (`infer.hybrid.HybridEngine`) builds its cache, its state slots and its
+by side (:class:`ParallelSpec`), :class:`ConvAttentionSpec`, :class:`NormedAttentionSpec`, :class:`DeltaSpec`, :class:`GlaSpec` or
+:class:`LatentSpec` - and optionally a feed-forward, gated, plain or of experts (:class:`ExpertsSpec`).  A range of layers may run
+several times (:class:`Loop`), and the residual may be several streams that every sublayer mixes.  The engine (`infer.hybrid.HybridEngine`) builds its cache, its state slots and its
 kernels' arguments from these specs and reads no size from anywhere else, so another order of layers or another
 combination of constants is another configuration, not another class.
 
@@ -10,7 +11,7 @@ combination of constants is another configuration, not another class.
 attention branch beside a Mamba-2 branch in some layers, the gated delta rule in the others, a per-layer token input at
 the end of every layer and soft-capped logits.  :func:`gugedra_config` reads its ``config.json``, and
 :func:`load_gugedra` its ``model.safetensors``.  `Makuzen` (`lm.makuzen`) and
-`Gutivik` (`lm.gutivik`) are others.
+`Gutivik` (`lm.gutivik`) and `Lukopel` (`lm.lukopel`) are others.
 """
 from __future__ import annotations
 
@@ -24,7 +25,7 @@ import torch
 
 from .config import ConfigError, RopeScaling
 
-__all__ = ["AttentionSpec", "ConvAttentionSpec", "SsdSpec", "ParallelSpec", "DeltaSpec", "GlaSpec", "LatentSpec", "RouterSpec",
+__all__ = ["AttentionSpec", "ConvAttentionSpec", "DistanceBias", "QueryTemperature", "NormedAttentionSpec", "Loop", "SsdSpec", "ParallelSpec", "DeltaSpec", "GlaSpec", "LatentSpec", "RouterSpec",
            "ClampedGlu", "ExpertsSpec", "HybridLayer", "HybridConfig", "HybridWeights", "gugedra_config", "gugedra_tensors", "load_gugedra", "random_gugedra"]
 
 
@@ -75,6 +76,58 @@ class ConvAttentionSpec(AttentionSpec):
             raise ConfigError("attention: the convolution kernel has at most 8 taps")
         if self.keep_first < 0:
             raise ConfigError("attention: keep_first cannot be negative")
+
+
+@dataclass(frozen=True)
+class DistanceBias:
+    """A learned score per head and bucket of the distance between query and key: ``rows`` buckets, one for each distance in the
+    first half, logarithmic from there to distance ``far``, the last one for everything beyond."""
+    rows: int
+    far: int
+
+    def __post_init__(self):
+        _positive(self, "rows", "far")
+        if self.far <= self.rows // 2 or self.rows < 2:
+            raise ConfigError("distance bias: at least two rows, and a largest distance beyond the first half of them")
+
+    def bucket(self, n: int) -> int:
+        half = self.rows // 2
+        if n < half:
+            return n
+        return min(self.rows - 1, half + math.floor(math.log(n / half) / math.log(self.far / half) * (self.rows - half)))
+
+
+@dataclass(frozen=True)
+class QueryTemperature:
+    """Queries at position p are multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
+    coef: float
+    every: int
+
+    def __post_init__(self):
+        _positive(self, "every")
+
+
+@dataclass(frozen=True)
+class NormedAttentionSpec(AttentionSpec):
+    """Attention on normed queries and keys, without a rotation."""
+    norm: str = "head"       # "head": every head by itself with one shared weight; "all": the whole projection at once
+    bias: bool = False       # on the projections, the output's too
+    unit_values: bool = False    # every head's value is divided by its root mean square
+    head_scale: bool = False     # a learned factor of the scores per head
+    temperature: Optional[QueryTemperature] = None
+    distance: Optional[DistanceBias] = None
+    talk: bool = False       # after the softmax the heads' weights are mixed by a learned [heads, heads] matrix
+    gate: bool = False       # a sigmoid per head on the output
+    chunk: int = 0           # > 0: a token sees the tokens of its own chunk only (chunks count from position 0)
+
+    def __post_init__(self):
+        super().__post_init__()
+        if self.norm not in ("head", "all"):
+            raise ConfigError(f"attention: unknown extent {self.norm!r} of the query and key norm")
+        if self.rope_dims:
+            raise ConfigError("attention on normed queries and keys has no rotation")
+        if self.chunk < 0:
+            raise ConfigError("attention: chunk cannot be negative")
 
 
 @dataclass(frozen=True)
@@ -227,18 +280,35 @@ class ExpertsSpec:
 
 
 GLU_ACTS = ("silu", "gelu_tanh")
+PLAIN_ACTS = ("relu2",)      # W_down act(W_up h): no gate
 
 
 @dataclass(frozen=True)
 class HybridLayer:
-    mixer: Union[ParallelSpec, ConvAttentionSpec, DeltaSpec, GlaSpec, LatentSpec]
-    ff: int = 0              # width of the gated feed-forward, 0: none
+    mixer: Union[ParallelSpec, ConvAttentionSpec, NormedAttentionSpec, DeltaSpec, GlaSpec, LatentSpec]
+    ff: int = 0              # width of the feed-forward, 0: none
     experts: Optional[ExpertsSpec] = None
-    act: str = "silu"        # activation of the gate of the feed-forward
+    act: str = "silu"        # activation of the gate of the feed-forward, or of one without a gate
+    ff_bias: bool = False    # on the projections of a feed-forward without a gate
 
     def __post_init__(self):
-        if self.act not in GLU_ACTS:
+        if self.act not in GLU_ACTS + PLAIN_ACTS:
             raise ConfigError(f"unknown activation {self.act!r}")
+        if self.ff_bias and self.act in GLU_ACTS:
+            raise ConfigError("gated feed-forwards have no biases")
+
+
+@dataclass(frozen=True)
+class Loop:
+    """Layers start .. stop - 1 run ``times`` times in a row, each pass with a cache of its own."""
+    start: int
+    stop: int
+    times: int
+
+    def __post_init__(self):
+        _positive(self, "times")
+        if not all(isinstance(v, int) and not isinstance(v, bool) for v in (self.start, self.stop)) or not 0 <= self.start <= self.stop:
+            raise ConfigError("loop: 0 <= start <= stop is expected")
 
 
 @dataclass
@@ -256,9 +326,19 @@ class HybridConfig:
     embed_scale: float = 1.0
     residual_mult: float = 1.0   # factor of every sublayer output
     logit_scale: float = 1.0     # before the soft cap
+    streams: int = 0             # copies of the residual that every sublayer reads, mixes and writes (0: one plain residual)
+    loop: Optional[Loop] = None
+    positions: int = 0           # learned position vectors, which are the longest sequence too (0: none)
 
     def __post_init__(self):
         _positive(self, "vocab", "width")
+        if not 0 <= self.streams <= 8 or self.positions < 0:
+            raise ConfigError("streams must be 0 to 8, positions cannot be negative")
+        if self.streams and (self.token_side or self.post_norm or not self.pre_norm or self.residual_mult != 1.0 or any(
+                x.experts for x in self.layers)):
+            raise ConfigError("residual streams: sublayers with a norm on their input only, no token side and no experts")
+        if self.loop is not None and self.loop.stop > len(self.layers):
+            raise ConfigError("loop: there are not as many layers")
         if self.token_side < 0:
             raise ConfigError("token_side cannot be negative")
         if not self.layers:
@@ -266,13 +346,24 @@ class HybridConfig:
         if len({(m.kv_heads, m.vdim) for m in self._mixing()}) > 1:
             raise ConfigError("layers that mix values must have equal sizes of them")
 
+    @property
+    def order(self) -> List[int]:
+        """The layer of every run, in order."""
+        n = list(range(len(self.layers)))
+        p = self.loop
+        return n if p is None else n[: p.start] + n[p.start: p.stop] * p.times + n[p.stop:]
+
+    @property
+    def runs(self) -> List[HybridLayer]:
+        return [self.layers[i] for i in self.order]
+
     def _mixing(self) -> list:
         return [x.mixer for x in self.layers if isinstance(x.mixer, ConvAttentionSpec) and x.mixer.mix_values]
 
     @property
     def first_mixing(self) -> int:
-        """The layer whose values later layers mix with theirs, -1: none."""
-        return next((i for i, x in enumerate(self.layers) if isinstance(x.mixer, ConvAttentionSpec) and x.mixer.mix_values), -1)
+        """The layer run whose values later ones mix with theirs, -1: none."""
+        return next((i for i, x in enumerate(self.runs) if isinstance(x.mixer, ConvAttentionSpec) and x.mixer.mix_values), -1)
 
     @property
     def recurrent(self) -> bool:
@@ -281,8 +372,8 @@ class HybridConfig:
 
     def kv_bytes_per_token(self, element: int) -> int:
         n = 0
-        for m in (layer.mixer for layer in self.layers):
-            if isinstance(m, (ParallelSpec, ConvAttentionSpec)):
+        for m in (layer.mixer for layer in self.runs):
+            if isinstance(m, (ParallelSpec, ConvAttentionSpec, NormedAttentionSpec)):
                 a = m.left if isinstance(m, ParallelSpec) else m
                 n += a.kv_heads * (a.dim + a.vdim) * element
             elif isinstance(m, LatentSpec):

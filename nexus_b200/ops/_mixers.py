@@ -27,7 +27,25 @@ class ResidualNormArgs(C.Structure):
                 ("rows", C.c_int32), ("cols", C.c_int32), ("dtype", C.c_int32), ("eps", C.c_float), ("embed_scale", C.c_float),
                 ("res_mult", C.c_float), ("experts", C.c_void_p), ("expert_slots", C.c_void_p), ("y_gate", C.c_void_p),
                 ("ld_experts", C.c_int64), ("top", C.c_int32), ("expert_scale", C.c_float), ("w_dot", C.c_void_p),
-                ("dot_out", C.c_void_p), ("scatter", C.c_void_p), ("scatter_slots", C.c_void_p), ("expert_weights", C.c_void_p)]
+                ("dot_out", C.c_void_p), ("scatter", C.c_void_p), ("scatter_slots", C.c_void_p), ("expert_weights", C.c_void_p),
+                ("positions", C.c_void_p), ("pos_table", C.c_void_p)]
+
+
+class StreamResidualArgs(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("tokens", C.c_void_p), ("table", C.c_void_p), ("positions", C.c_void_p), ("pos_table", C.c_void_p),
+                ("y", C.c_void_p), ("mix", C.c_void_p), ("out", C.c_void_p), ("in_", C.c_void_p), ("w_next", C.c_void_p),
+                ("h", C.c_void_p), ("ldy", C.c_int64), ("ldh", C.c_int64), ("rows", C.c_int32), ("cols", C.c_int32),
+                ("streams", C.c_int32), ("dtype", C.c_int32), ("eps", C.c_float), ("embed_scale", C.c_float)]
+
+
+class HeadPrepArgs(C.Structure):
+    _fields_ = [("proj", C.c_void_p), ("ld", C.c_int64), ("q_off", C.c_int32), ("k_off", C.c_int32), ("v_off", C.c_int32),
+                ("g_off", C.c_int32), ("rows", C.c_int32), ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32),
+                ("vdim", C.c_int32), ("norm_dim", C.c_int32), ("norm_vdim", C.c_int32), ("norm_all", C.c_int32),
+                ("unit_values", C.c_int32), ("store_kv", C.c_int32), ("every", C.c_int32), ("dtype", C.c_int32), ("eps", C.c_float),
+                ("q_scale", C.c_float), ("coef", C.c_float), ("w_q", C.c_void_p), ("w_k", C.c_void_p), ("head_scale", C.c_void_p),
+                ("positions", C.c_void_p), ("slots", C.c_void_p), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p),
+                ("gate", C.c_void_p)]
 
 
 class LatentPrepArgs(C.Structure):
@@ -94,7 +112,12 @@ class PagedWindowArgs(C.Structure):
                 ("block_size", C.c_int32), ("max_blocks", C.c_int32), ("window", C.c_int32), ("splits", C.c_int32),
                 ("dtype", C.c_int32), ("scale", C.c_float), ("softcap", C.c_float), ("out_scale", C.c_float),
                 ("seg", SegmentArgs), ("k_pitch", C.c_int64), ("v_pitch", C.c_int64), ("gate", C.c_void_p), ("sink", C.c_void_p),
-                ("keep_first", C.c_int32)]
+                ("keep_first", C.c_int32), ("chunk", C.c_int32), ("bias_len", C.c_int32), ("all_values", C.c_int32),
+                ("bias", C.c_void_p)]
+
+
+class TalkDecodeArgs(C.Structure):
+    _fields_ = [("base", PagedWindowArgs), ("talk", C.c_void_p), ("scores", C.c_void_p), ("score_pitch", C.c_int64)]
 
 
 class LatentPromptArgs(C.Structure):
@@ -110,7 +133,8 @@ class WindowPromptArgs(C.Structure):
                 ("blocks", C.c_void_p), ("kept", C.c_void_p), ("status", C.c_void_p), ("ldq", C.c_int64), ("ldk", C.c_int64),
                 ("ldv", C.c_int64), ("ldo", C.c_int64), ("n_blocks", C.c_int32), ("q_rows", C.c_int32), ("kv_rows", C.c_int32),
                 ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("window", C.c_int32),
-                ("keep_first", C.c_int32), ("scale", C.c_float)]
+                ("keep_first", C.c_int32), ("scale", C.c_float), ("gate", C.c_void_p), ("bias", C.c_void_p), ("bias_len", C.c_int32),
+                ("chunk", C.c_int32), ("all_values", C.c_int32)]
 
 
 class LatentAttnArgs(C.Structure):
@@ -121,6 +145,8 @@ class LatentAttnArgs(C.Structure):
 
 
 LATENT_MAX_RANK, LATENT_MAX_ROW = 512, 768
+PROMPT_MAX_BIAS = 3584       # distances of a bias table of the tcgen05 prompt kernel
+TALK_MAX_HEADS = 96          # heads that mix their weights
 
 
 @dataclass
@@ -148,8 +174,8 @@ def _ptr(t: Optional[torch.Tensor]):
 
 def residual_norm(x, *, y=None, w_post=None, w_next=None, h=None, x_cast=None, tokens=None, table=None, eps, embed_scale=1.0,
                   res_mult=1.0, experts=None, slots=None, top=0, weights=None, y_gate=None, w_dot=None, dot_out=None,
-                  scatter=None) -> None:
-    """x (FP32) = embed_scale * table[tokens], or x + res_mult * rms(y) * w_post (without w_post: x + res_mult * y);  h = rms(x) *
+                  scatter=None, positions=None, pos_table=None) -> None:
+    """x (FP32) = embed_scale * table[tokens] (+ pos_table[positions]), or x + res_mult * rms(y) * w_post (without w_post: x + res_mult * y);  h = rms(x) *
     w_next;  x_cast = x in the activation dtype.  With ``experts`` the sublayer output is the mean of the rows
     ``experts[slots[r, :]]``, or their sum with ``weights`` [rows, top] (FP32), + y_gate[r] * y[r].  ``dot_out`` = sigmoid(x .
     w_dot); ``scatter[slots[r, :]]`` = the row of x_cast."""
@@ -161,8 +187,36 @@ def residual_norm(x, *, y=None, w_post=None, w_next=None, h=None, x_cast=None, t
                          y.stride(0) if y is not None else 0, lead.stride(0) if lead is not None else x.shape[1], x.shape[0],
                          x.shape[1], _dt(act), eps, embed_scale, res_mult, _ptr(experts), _ptr(slots), _ptr(y_gate),
                          experts.stride(0) if experts is not None else 0, top, 1.0 / top if top and weights is None else 1.0,
-                         _ptr(w_dot), _ptr(dot_out), _ptr(scatter), _ptr(slots), _ptr(weights))
+                         _ptr(w_dot), _ptr(dot_out), _ptr(scatter), _ptr(slots), _ptr(weights), _ptr(positions), _ptr(pos_table))
     K._check(K.lib().nx_residual_norm(C.byref(a), K._stream()), "nx_residual_norm")
+
+
+def stream_residual(x, *, eps, y=None, mix=None, out=None, tokens=None, table=None, embed_scale=1.0, positions=None, pos_table=None,
+                    w_next=None, h=None, read=None) -> None:
+    """x (FP32 [rows, streams, cols]): every stream = embed_scale * table[tokens] + pos_table[positions], or x_t = sum_s mix[s, t] x_s +
+    out[t] y;  h = rms(sum_s read[s] x_s) * w_next (``read`` None: ones)."""
+    act = next(t for t in (h, y, table) if t is not None)
+    a = StreamResidualArgs(_ptr(x), _ptr(tokens), _ptr(table), _ptr(positions), _ptr(pos_table), _ptr(y), _ptr(mix), _ptr(out),
+                           _ptr(read), _ptr(w_next), _ptr(h), y.stride(0) if y is not None else 0, h.stride(0) if h is not None else 0,
+                           x.shape[0], x.shape[2], x.shape[1], _dt(act), eps, embed_scale)
+    K._check(K.lib().nx_stream_residual(C.byref(a), K._stream()), "nx_stream_residual")
+
+
+def head_prep(proj, offsets, *, heads, kv_heads, dim, vdim, norm_dim, norm_vdim, eps, w_q, w_k, positions, slots, k_cache, v_cache,
+              norm_all=False, unit_values=False, store_kv=False, q_scale=1.0, head_scale=None, coef=0.0, every=0, gate=None) -> None:
+    """Norms of q and k, the query's factors, cache append and the output gate, in place in ``proj``; ``offsets``: first columns of q,
+    k, v and the gate."""
+    a = HeadPrepArgs(_ptr(proj), proj.stride(0), *offsets, proj.shape[0], heads, kv_heads, dim, vdim, norm_dim, norm_vdim,
+                     int(norm_all), int(unit_values), int(store_kv), every, _dt(proj), eps, q_scale, coef, _ptr(w_q), _ptr(w_k),
+                     _ptr(head_scale), _ptr(positions), _ptr(slots), _ptr(k_cache), _ptr(v_cache), _ptr(gate))
+    K._check(K.lib().nx_head_prep(C.byref(a), K._stream()), "nx_head_prep")
+
+
+def head_mix(wide, talk, gate, out, *, heads, kv_heads, vdim) -> None:
+    """out [rows, heads * vdim]: out_h = gate_h sum_g talk[h, g] wide[g, KV head of h]; wide [rows, heads * kv_heads * vdim]."""
+    K._check(K.lib().nx_head_mix(K._p(wide), C.c_int64(wide.stride(0)), K._p(talk), K._p(gate), K._p(out), C.c_int64(out.stride(0)),
+                                 C.c_int(wide.shape[0]), C.c_int(heads), C.c_int(kv_heads), C.c_int(vdim), C.c_int(_dt(wide)),
+                                 K._stream()), "nx_head_mix")
 
 
 def latent_prep(proj, offsets, q_rank, kv_rank, rot_dims, heads, w_q, w_kv, positions, slots, cos_t, sin_t, cq, cache, rot_col,
@@ -308,32 +362,55 @@ def softcap_(x, cols, cap, scale=1.0) -> None:
                                     C.c_float(scale), K._stream()), "nx_softcap")
 
 
-def paged_window_attention(q, k_cache, v_cache, block_table, out, seg: Segments, *, heads, block_size, window, scale,
-                           softcap=0.0, out_scale=1.0, splits=1, gate=None, vdim=0, keep_first=0, sink=None) -> None:
-    """q: [rows, heads * dim] view; caches [blocks, block_size, kv_heads, dim | vdim]; out [rows, heads * vdim] view.
-    One-row segments run the decode kernel, longer ones the prompt kernel (BF16); FP32 has one kernel for both.
-    ``vdim`` > 0: a latent cache, the values are the leading ``vdim`` columns of the keys (``v_cache`` is not used).
-    ``gate``: FP32 [rows, heads] factor of the output.  ``keep_first``: the first keys stay visible; ``sink``: FP32 [heads], a
-    score that counts in the denominator only."""
+def _paged_args(q, k_cache, v_cache, block_table, out, seg, heads, block_size, window, scale, softcap, out_scale, gate, vdim, keep_first,
+                sink, chunk, bias, all_values) -> PagedWindowArgs:
     G, D = k_cache.shape[2], k_cache.shape[3]
     if vdim:
         v_cache = k_cache
         if G != 1:
             raise ValueError("paged_window_attention: a latent cache has one KV head")
     Dv = vdim or v_cache.shape[3]
-    a = PagedWindowArgs(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(out), q.stride(0), out.stride(0), None,
-                        None, heads, G, D, Dv, block_size, block_table.shape[1], window, 1, _dt(q), scale, softcap, out_scale,
-                        seg.args(), k_cache.stride(1), v_cache.stride(1), _ptr(gate), _ptr(sink), keep_first)
+    return PagedWindowArgs(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), _ptr(out), q.stride(0), out.stride(0),
+                           None, None, heads, G, D, Dv, block_size, block_table.shape[1], window, 1, _dt(q), scale, softcap, out_scale,
+                           seg.args(), k_cache.stride(1), v_cache.stride(1), _ptr(gate), _ptr(sink), keep_first, chunk,
+                           bias.shape[1] if bias is not None else 0, int(all_values), _ptr(bias))
+
+
+def paged_window_attention(q, k_cache, v_cache, block_table, out, seg: Segments, *, heads, block_size, window, scale,
+                           softcap=0.0, out_scale=1.0, splits=1, gate=None, vdim=0, keep_first=0, sink=None, chunk=0, bias=None,
+                           all_values=False) -> None:
+    """q: [rows, heads * dim] view; caches [blocks, block_size, kv_heads, dim | vdim]; out [rows, heads * vdim] view.
+    One-row segments run the decode kernel, longer ones the prompt kernel (BF16); FP32 has one kernel for both.
+    ``vdim`` > 0: a latent cache, the values are the leading ``vdim`` columns of the keys (``v_cache`` is not used).
+    ``gate``: FP32 [rows, heads] factor of the output.  ``keep_first``: the first keys stay visible; ``sink``: FP32 [heads], a
+    score that counts in the denominator only.  ``chunk``: only keys of the row's chunk of positions; ``bias``: FP32 [heads, distances],
+    the last one for all beyond; ``all_values``: out is [rows, heads * kv_heads * vdim], every head's weights with the values of every
+    KV head (not for one-row segments in BF16)."""
+    a = _paged_args(q, k_cache, v_cache, block_table, out, seg, heads, block_size, window, scale, softcap, out_scale, gate, vdim,
+                    keep_first, sink, chunk, bias, all_values)
     if q.dtype == torch.float32:
         K._check(K.lib().nx_paged_window_f32(C.byref(a), K._stream()), "nx_paged_window_f32")
-    elif seg.max_len == 1:
+    elif seg.max_len == 1 and not all_values:
         a.splits = splits
         if splits > 1:
-            a.part_o = K.scratch(seg.count * heads * splits * Dv * 4, "window_o", q.device).data_ptr()
+            a.part_o = K.scratch(seg.count * heads * splits * a.vdim * 4, "window_o", q.device).data_ptr()
             a.part_ml = K.scratch(seg.count * heads * splits * 8, "window_ml", q.device).data_ptr()
         K._check(K.lib().nx_paged_window_decode(C.byref(a), K._stream()), "nx_paged_window_decode")
     else:
         K._check(K.lib().nx_paged_window_prefill(C.byref(a), K._stream()), "nx_paged_window_prefill")
+
+
+def talk_decode(q, k_cache, v_cache, block_table, out, talk, seg: Segments, *, heads, block_size, window, scale, keys, softcap=0.0,
+                splits=1, gate=None, keep_first=0, chunk=0, bias=None) -> None:
+    """Decoding with heads that mix their weights (``talk``: FP32 [heads, heads]); ``keys``: the most keys a row can see."""
+    a = TalkDecodeArgs(_paged_args(q, k_cache, v_cache, block_table, out, seg, heads, block_size, window, scale, softcap, 1.0, gate, 0,
+                                   keep_first, None, chunk, bias, False), _ptr(talk), None, (keys + 63) // 64 * 64)
+    a.base.splits = splits
+    a.base.part_ml = K.scratch(seg.count * heads * splits * 8, "window_ml", q.device).data_ptr()
+    if splits > 1:
+        a.base.part_o = K.scratch(seg.count * heads * splits * a.base.vdim * 4, "window_o", q.device).data_ptr()
+    a.scores = K.scratch(seg.count * heads * a.score_pitch * 4, "talk_scores", q.device).data_ptr()
+    K._check(K.lib().nx_talk_decode(C.byref(a), K._stream()), "nx_talk_decode")
 
 
 def latent_attention(q, cache, block_table, out, seg: Segments, *, heads, rank, window, scale, gate=None, splits=1) -> None:
@@ -359,12 +436,15 @@ def latent_prompt(q, kv, lat, out, blocks, *, heads, dim, rot, vdim, rank, windo
     K._check(K.lib().nx_latent_prompt(C.byref(a), K._stream()), "nx_latent_prompt")
 
 
-def window_prompt(q, k, v, out, blocks, *, heads, kv_heads, dim, vdim, window, scale, keep_first=0, kept=None, sink=None) -> None:
+def window_prompt(q, k, v, out, blocks, *, heads, kv_heads, dim, vdim, window, scale, keep_first=0, kept=None, sink=None, gate=None,
+                  chunk=0, bias=None, all_values=False) -> None:
     """The tcgen05 form on plain grouped keys and values.  q [rows, heads * dim], k [kv rows, kv_heads * dim], v [kv rows, kv_heads *
-    vdim]; blocks as in `latent_prompt`; kept int32 [n]: the row that position 0 has among the kept first keys (None: the block's)."""
+    vdim]; blocks as in `latent_prompt`; kept int32 [n]: the row that position 0 has among the kept first keys (None: the block's);
+    chunk, bias and all_values as in `paged_window_attention`."""
     a = WindowPromptArgs(_ptr(q), _ptr(k), _ptr(v), _ptr(out), _ptr(sink), _ptr(blocks), _ptr(kept),
                          K.status_word(q.device).data_ptr(), q.stride(0), k.stride(0), v.stride(0), out.stride(0), blocks.shape[0],
-                         q.shape[0], k.shape[0], heads, kv_heads, dim, vdim, window, keep_first, scale)
+                         q.shape[0], k.shape[0], heads, kv_heads, dim, vdim, window, keep_first, scale, _ptr(gate), _ptr(bias),
+                         bias.shape[1] if bias is not None else 0, chunk, int(all_values))
     K._check(K.lib().nx_window_prompt(C.byref(a), K._stream()), "nx_window_prompt")
 
 
