@@ -206,7 +206,7 @@ def run_reference(args) -> int:
 
 
 def run_serving(args) -> int:
-    """Prefill and decode throughput of Gugedra, Makuzen or Gutivik models (random weights, BF16) at a few sizes, and of the other
+    """Prefill and decode throughput of Gugedra, Makuzen, Gutivik or Lukopel models (random weights, BF16) at a few sizes, and of the other
     models of the same width and depth through the same engine.  One JSON line; `value` is the design's prefill rate at the
     middle size."""
     if args.impl != "ours" or args.gpus != 1:
@@ -217,6 +217,8 @@ def run_serving(args) -> int:
         from nexus_b200.bench.hybrid import model_lines
     elif args.workload == "makuzen":
         from nexus_b200.bench.latent import model_lines
+    elif args.workload == "lukopel":
+        from nexus_b200.bench.talking import model_lines
     else:
         from nexus_b200.bench.routed import model_lines
     from nexus_b200.ops import _cuda as K
@@ -250,8 +252,8 @@ def main() -> int:
     ap.add_argument("--graph", type=int, default=-1,
                     help="trainer API replays the whole step as one CUDA graph (default: on for 1 GPU, off otherwise)")
     ap.add_argument("--skip-e2e", action="store_true")
-    ap.add_argument("--workload", default="train", choices=["train", "gugedra", "makuzen", "gutivik"],
-                    help="gugedra, makuzen, gutivik: serving speed of that design beside the other models of equal width and depth, one GPU")
+    ap.add_argument("--workload", default="train", choices=["train", "gugedra", "makuzen", "gutivik", "lukopel"],
+                    help="gugedra, makuzen, gutivik, lukopel: serving speed of that design beside the other models of equal width and depth, one GPU")
     ap.add_argument("--sizes", default="1024,2048,4096", help="widths of the serving workloads")
     args = ap.parse_args()
     if args.workload != "train":

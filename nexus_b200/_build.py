@@ -153,7 +153,7 @@ def build_host(force: bool = False, verbose: bool = False) -> Path:
 # what `ensure_serving` compiles where nothing has been built: the kernels and host code of the layered decoders
 SERVING_CUDA = ("attention_sm100", "gemm_sm100", "infer_kernels", "latent_attention", "latent_prompt_sm100", "mixer_kernels", "moe_kernels",
                 "normed_heads", "paged_talk_attention", "paged_window_attention", "recurrent_chunk", "recurrent_gla", "recurrent_step",
-                "residual_streams")
+                "residual_streams", "talk_prompt_sm100")
 SERVING_HOST = ("cpu_kernels", "kv_sched", "module")
 
 

@@ -2,7 +2,7 @@
 // that all heads share; a row sees a window of keys and optionally the first keys of its sequence; a sink may count in the
 // denominator.  Queries, keys and values of all segments lie packed in row buffers; a work item is a block of up to 256 query
 // rows of one segment and one head.  Without a shared key part a row may also see only the keys of its own chunk of positions, scores
-// may have a bias by distance, and an item may be a query head with the values of another KV head than its keys'.
+// may have a bias by distance.
 //
 // The pipeline is that of the two-tile flash kernel: one persistent CTA per SM, softmax group A (warps 0-3) on query rows
 // 0-127 of the block, group B (warps 4-7) on rows 128-255, both against the same key tiles; the MMA warp interleaves
@@ -27,7 +27,7 @@ constexpr int kSlab = 128 * 128;  // bytes of [128 rows][64 columns]
 
 // distances of a bias table in shared memory, and how far it goes on to the masked ones (a row and a key of one tile pair are up to 254
 // apart in the wrong direction) and beyond the last one
-constexpr int kBiasMax = 3584, kBiasNear = 256, kBiasFar = 256, kBiasTable = kBiasNear + kBiasMax + kBiasFar;
+constexpr int kBiasMax = 3072, kBiasNear = 256, kBiasFar = 256, kBiasTable = kBiasNear + kBiasMax + kBiasFar;
 
 // ND / NV: 64-column slabs of a head's own key part and of its values; NR: of the shared part (0 or 1)
 // kBias: a table of biases per softmax group behind the barriers
@@ -52,8 +52,8 @@ struct Dev {
   int64_t ldo;
   const float* bias;         // [heads][bias_len]
   int items, heads, rep, vdim, window, keep_first, ksteps, rsteps;   // rep: query heads per KV head; 16-column steps of the own
-  int chunk, bias_len, values;                                       // and the shared key part; values: KV heads whose values a
-  float scale;                                                       // query head meets, 1: its own
+  int chunk, bias_len;                                               // and the shared key part
+  float scale;
   __device__ __forceinline__ int first_key(int pos) const {          // apart from the kept ones
     const int lo = window > 0 ? max(0, pos - window + 1) : 0;
     return chunk > 0 ? max(lo, pos / chunk * chunk) : lo;
@@ -61,7 +61,7 @@ struct Dev {
 };
 
 struct Work {
-  int h, hv, row0, rows, pos0, kv0, k_lo;   // hv: KV head of the values
+  int h, row0, rows, pos0, kv0, k_lo;
   int kept0, n_kept;               // buffer row of kept key 0; kept keys before k_lo
   int shift;                       // key tile j < shift holds kept keys 128 j .., tile j >= shift keys k_lo + 128 (j - shift) ..
   int jbA, jeA, jbB, jeB, je;      // key tiles of either query tile
@@ -73,10 +73,8 @@ __device__ __forceinline__ bool next_work(const Dev& p, int round, Work& w) {
   const int G = static_cast<int>(gridDim.x), c = static_cast<int>(blockIdx.x);
   const int item = round * G + ((round & 1) ? (G - 1 - c) : c);
   if (item >= p.items) return false;
-  const int per = kKeep ? p.heads * p.values : p.heads, block = item / per, sub = item % per;
-  const int4 b = __ldg(reinterpret_cast<const int4*>(p.blocks) + block);
-  w.h = kKeep ? sub / p.values : sub;
-  w.hv = kKeep ? (p.values > 1 ? sub % p.values : w.h / p.rep) : w.h;
+  const int4 b = __ldg(reinterpret_cast<const int4*>(p.blocks) + item / p.heads);
+  w.h = item % p.heads;
   w.row0 = b.x;
   w.rows = b.y;
   w.pos0 = b.z;
@@ -84,7 +82,7 @@ __device__ __forceinline__ bool next_work(const Dev& p, int round, Work& w) {
   w.k_lo = p.first_key(w.pos0);
   w.n_kept = kKeep ? min(p.keep_first, w.k_lo) : 0;
   w.shift = (w.n_kept + 127) / 128;
-  w.kept0 = kKeep && p.kept != nullptr ? __ldg(p.kept + block) : b.w;
+  w.kept0 = kKeep && p.kept != nullptr ? __ldg(p.kept + item / p.heads) : b.w;
   w.jbA = 0;
   w.jeA = w.shift + (w.pos0 + min(128, w.rows) - 1 - w.k_lo) / 128 + 1;
   w.jbB = w.jeB = 0;
@@ -185,7 +183,7 @@ prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
           if (!ok) break;
           mbar_arrive_expect_tx(&v_full[v], C::kVBytes);
 #pragma unroll
-          for (int c = 0; c < NV; ++c) tma_load_3d(sV + v * C::kVBytes + c * kSlab, &tm_v, &v_full[v], 64 * c, w.hv, row);
+          for (int c = 0; c < NV; ++c) tma_load_3d(sV + v * C::kVBytes + c * kSlab, &tm_v, &v_full[v], 64 * c, hk, row);
         }
       }
     }
@@ -412,8 +410,7 @@ prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ 
       const int64_t row = w.row0 + x * 128 + r;
       if (kKeep && p.sink != nullptr) l_run += ex2f(p.sink[w.h] * kLog2e - m_ref);
       const float inv = row_ok ? (p.gate != nullptr ? p.gate[row * p.heads + w.h] : 1.0f) / l_run : 0.0f;
-      const int64_t slice = kKeep && p.values > 1 ? static_cast<int64_t>(w.h) * p.values + w.hv : w.h;
-      __nv_bfloat16* orow = p.out + row * p.ldo + slice * p.vdim;
+      __nv_bfloat16* orow = p.out + row * p.ldo + static_cast<int64_t>(w.h) * p.vdim;
 #pragma unroll
       for (int cc = 0; cc < NV * 2; ++cc) {
         uint32_t ov[32];
@@ -553,7 +550,6 @@ extern "C" int nx_window_prompt(const NxWindowPromptArgs* a, nx_stream_t stream)
   if (a == nullptr || a->status == nullptr || a->blocks == nullptr || a->heads <= 0 || a->kv_heads <= 0 || !(a->scale > 0.0f)) return -1;
   if (a->heads % a->kv_heads || a->keep_first < 0 || a->chunk < 0) return -1;
   if (a->bias != nullptr && (a->bias_len <= 0 || a->bias_len > kBiasMax)) return -1;
-  if (a->all_values && static_cast<int64_t>(a->n_blocks) * a->heads * a->kv_heads > 0x3fffffff) return -1;
   if (a->dim <= 0 || a->dim > 128 || (a->dim & 15) || a->vdim <= 0 || a->vdim > 128 || (a->vdim & 7)) return -1;
   if ((a->ldq | a->ldk | a->ldv | a->ldo) & 7) return -1;
   for (const void* ptr : {a->q, a->k, a->v, static_cast<const void*>(a->out), static_cast<const void*>(a->blocks)})
@@ -575,10 +571,9 @@ extern "C" int nx_window_prompt(const NxWindowPromptArgs* a, nx_stream_t stream)
   p.bias = a->bias;
   p.bias_len = a->bias_len;
   p.chunk = a->chunk;
-  p.values = a->all_values ? a->kv_heads : 1;
   p.status = a->status;
   p.ldo = a->ldo;
-  p.items = a->n_blocks * a->heads * p.values;
+  p.items = a->n_blocks * a->heads;
   p.heads = a->heads;
   p.rep = a->heads / a->kv_heads;
   p.vdim = a->vdim;

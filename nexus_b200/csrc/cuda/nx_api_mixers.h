@@ -311,16 +311,20 @@ int nx_paged_window_decode(const NxPagedWindowArgs* args, nx_stream_t stream);
 int nx_paged_window_prefill(const NxPagedWindowArgs* args, nx_stream_t stream);
 // any segments, FP32
 int nx_paged_window_f32(const NxPagedWindowArgs* args, nx_stream_t stream);
-// One-row segments, BF16, of heads that mix their weights: weight_h <- sum_g talk[h][g] weight_g, FP32, before the values of the KV
-// head of h.  Scores of all heads first (scores [count, heads, score_pitch], log2; part_ml [count, heads, splits, 2] always), then
-// mixture and values; part_o as above.  No sink, no all_values; up to 96 heads, vdim <= 256.
-typedef struct NxTalkDecodeArgs {
+// One-row and short segments, BF16, of heads that mix their weights: weight_h <- sum_g talk[h][g] weight_g, FP32, before the values of
+// the KV head of h.  Scratch has `rows` = nx_talk_rows(..) rows: scores [rows, heads, pitch] and weights of the same shape, part_ml
+// [rows, heads, splits, 2], with splits > 1 part_o [rows, heads, splits, vdim].  No sink, no all_values; up to 96 heads of up to 256
+// columns.
+typedef struct NxTalkPagedArgs {
   NxPagedWindowArgs base;
   const float* talk;         // [heads, heads]
   float* scores;
-  int64_t score_pitch;       // a multiple of 64, at least the keys a row can see
-} NxTalkDecodeArgs;
-int nx_talk_decode(const NxTalkDecodeArgs* args, nx_stream_t stream);
+  void* weights;             // BF16
+  int64_t pitch;             // a multiple of 64, at least the keys that rows of one tile (64 / query heads per KV head) can see
+  int32_t rows;
+} NxTalkPagedArgs;
+int nx_talk_rows(int heads, int kv_heads, int count, int max_len, int total_len);
+int nx_talk_paged(const NxTalkPagedArgs* args, nx_stream_t stream);
 
 
 // Attention of packed query rows over a latent cache, BF16: every head meets the same cache row [latent (rank) | rotated key
@@ -364,7 +368,7 @@ int nx_latent_prompt(const NxLatentPromptArgs* args, nx_stream_t stream);
 
 // The same kernel on plain grouped keys and values: q [q_rows, ldq]: heads * dim; k [kv_rows, ldk]: kv_heads * dim; v [kv_rows,
 // ldv]: kv_heads * vdim; query head h reads KV head h / (heads / kv_heads).  Windows, kept first keys and sinks as in
-// NxPagedWindowArgs, chunks, biases (up to 3584 distances) and all_values too.  blocks as above; kept [n_blocks]: row that position 0
+// NxPagedWindowArgs, chunks and biases (up to 3072 distances) too.  blocks as above; kept [n_blocks]: row that position 0
 // has among the kept keys (null: the fourth entry of the block).  dim <= 128: multiple of 16; vdim <= 128: multiple of 8; scale > 0.
 typedef struct NxWindowPromptArgs {
   const void* q;
@@ -380,9 +384,28 @@ typedef struct NxWindowPromptArgs {
   float scale;
   const float* gate;       // [rows, heads], may be null
   const float* bias;       // [heads, bias_len], may be null
-  int32_t bias_len, chunk, all_values;
+  int32_t bias_len, chunk;
 } NxWindowPromptArgs;
 int nx_window_prompt(const NxWindowPromptArgs* args, nx_stream_t stream);
+
+// The same for heads that mix: every query head with the values of every KV head, out [., ldo]: heads * kv_heads * vdim.  Layouts,
+// sizes and blocks as above, without kept keys and sinks.  bias [heads, bias_pitch], may be null: entry NX_TALK_BIAS_NEAR + distance in
+// units of log2, for the distances -NX_TALK_BIAS_NEAR .. bias_len + NX_TALK_BIAS_FAR - 1 (any finite value below 0, the last one from
+// bias_len on); bias_pitch a multiple of 4.
+enum { NX_TALK_BIAS_NEAR = 256, NX_TALK_BIAS_FAR = 256, NX_TALK_BIAS_MAX = 3072 };
+typedef struct NxTalkPromptArgs {
+  const void* q;
+  const void* k;
+  const void* v;
+  void* out;
+  const float* bias;
+  const int32_t* blocks;
+  int* status;
+  int64_t ldq, ldk, ldv, ldo;
+  int32_t n_blocks, q_rows, kv_rows, heads, kv_heads, dim, vdim, window, chunk, bias_len, bias_pitch;
+  float scale;
+} NxTalkPromptArgs;
+int nx_talk_prompt(const NxTalkPromptArgs* args, nx_stream_t stream);
 // Cache rows of `segments` runs of positions into one packed buffer.  list [segments, 4]: first destination row, rows, first
 // position, sequence; `longest`: most rows of a run.
 int nx_latent_gather(const void* cache, void* dst, const int32_t* block_table, const int32_t* list, int segments, int longest,

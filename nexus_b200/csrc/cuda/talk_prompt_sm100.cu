@@ -1,0 +1,515 @@
+// Attention of prompt segments on tcgen05 where every query head's weights meet the values of every KV head: heads that mix their
+// weights (see nx_api_mixers.h).  out_h = sum_g talk[h][g] (P_g V of the KV head of h), so the kernel forms P_g V_c for all g and c and
+// nx_head_mix takes the mixture.
+//
+// A work item is a tile of 128 query rows, one query head and up to 256 columns of values (several KV heads side by side): the scores and
+// the softmax are formed once for all of them.  S lives twice in TMEM (columns 0-127, 128-255), O behind it (256-511).  One persistent
+// CTA per SM: softmax group A (warps 0-3) takes the even key tiles of the CTA's running count, group B (warps 4-7) the odd ones, so
+// that one group exponentiates while the other's scores are on their way.  The MMA warp issues
+//   S(0), S(1), P(0) V, S(2), P(1) V, S(3), ..
+// Both groups add to one O, so they share the row maxima O is scaled by: tile j passes them on to tile j + 1, between the two warps
+// that own the same 32 rows.  O is rescaled only when a row's maximum has grown by 2^8.  A head's table of biases (in units of log2,
+// extended to both sides) arrives by bulk copy beside its queries.
+#include "flash_common.cuh"
+#include "nx_api_mixers.h"
+#include "sm100_ptx.cuh"
+#include "tensor_map.h"
+
+#include <algorithm>
+
+namespace {
+using namespace nx;
+
+constexpr int kThreads = 384;        // warps 0-3: softmax A, 4-7: softmax B, 8: TMA, 9: MMA, 10-11 idle
+constexpr int kSoftmaxRegs = 216, kOtherRegs = 72;     // 256 * 216 + 128 * 72 = 384 * 168: what the block was launched with
+constexpr int kSlab = 128 * 128;     // bytes of [128 rows][64 columns]
+constexpr int kHalfSlab = 64 * 128;  // of [64 keys][64 columns] of values
+constexpr int kSlabs = 4;            // 64-column slabs of values in one item
+constexpr int kBiasNear = NX_TALK_BIAS_NEAR, kBiasTable = NX_TALK_BIAS_NEAR + NX_TALK_BIAS_MAX + NX_TALK_BIAS_FAR;
+
+// ND: 64-column slabs of a key
+template <int ND>
+struct Cfg {
+  static constexpr int kQStages = ND == 1 ? 2 : 1, kKStages = 2, kVStages = ND == 1 ? 4 : 3;
+  static constexpr int kQBytes = ND * kSlab, kKBytes = ND * kSlab, kVBytes = kSlabs * kHalfSlab;
+  static constexpr int kTiles = kQStages * kQBytes + kKStages * kKBytes + kVStages * kVBytes;
+  static constexpr int kBarriers = 512, kStats = 128 * 4 + 2 * 2 * 128 * 8;
+  static constexpr int kSmem = kTiles + kBarriers + kStats + 2 * kBiasTable * 4;
+  static_assert(kSmem <= 227 * 1024, "shared memory");
+};
+
+struct Dev {
+  const int32_t* blocks;     // [n_blocks][4]: first row, rows, position of the first row, buffer row of position 0
+  const float* bias;         // [heads][bias_pitch], null: none
+  __nv_bfloat16* out;
+  int* status;
+  int64_t ldo;
+  int items, heads, kv_heads, rep, vdim, window, chunk, ksteps, bias_len, bias_pitch;
+  int slabs, at_once, passes;   // slabs of one KV head's values, KV heads of one item, items per (tile, head)
+  float scale;
+  __device__ __forceinline__ int first_key(int pos) const {
+    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    return chunk > 0 ? max(lo, pos / chunk * chunk) : lo;
+  }
+};
+
+struct Work {
+  int h, c0, slabs;                // query head, first KV head of the values, their slabs
+  int row0, rows, pos0, kv0, k_lo, n;   // n: key tiles
+};
+// the CTA's items in order; an item whose half block holds no rows is left out by every role
+__device__ __forceinline__ bool next_work(const Dev& p, int& round, Work& w) {
+  const int G = static_cast<int>(gridDim.x), c = static_cast<int>(blockIdx.x);
+  for (;; ++round) {
+    const int item = round * G + ((round & 1) ? (G - 1 - c) : c);
+    if (round * G >= p.items) return false;
+    if (item >= p.items) continue;
+    const int per = 2 * p.heads * p.passes, block = item / per, sub = item % per;
+    const int4 b = __ldg(reinterpret_cast<const int4*>(p.blocks) + block);
+    const int half = 1 - sub / (p.heads * p.passes);       // the half with more keys first
+    w.rows = min(128, b.y - half * 128);
+    if (w.rows <= 0) continue;
+    w.h = sub % p.heads;
+    w.c0 = sub / p.heads % p.passes * p.at_once;
+    w.slabs = min(p.at_once, p.kv_heads - w.c0) * p.slabs;
+    w.row0 = b.x + half * 128;
+    w.pos0 = b.z + half * 128;
+    w.kv0 = b.w;
+    w.k_lo = p.first_key(w.pos0);
+    w.n = (w.pos0 + w.rows - 1 - w.k_lo) / 128 + 1;
+    ++round;
+    return true;
+  }
+}
+
+template <int ND>
+__global__ void __launch_bounds__(kThreads, 1)
+talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
+                   const __grid_constant__ CUtensorMap tm_v, const Dev p) {
+  using C = Cfg<ND>;
+  constexpr int QS = C::kQStages, KS = C::kKStages, VS = C::kVStages;
+  extern __shared__ __align__(1024) uint8_t smem[];
+  if (smem_u32(smem) & 1023u) {  // the swizzled tiles need a 1 KiB aligned base; uniform early exit
+    if (threadIdx.x == 0) atomicCAS(p.status, 0, kStatusBadArgument);
+    return;
+  }
+  uint8_t* sQ = smem;
+  uint8_t* sK = sQ + QS * C::kQBytes;
+  uint8_t* sV = sK + KS * C::kKBytes;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + C::kTiles);
+  uint64_t *q_full = bars, *q_empty = bars + 2, *k_full = bars + 4, *k_empty = bars + 6, *v_full = bars + 8, *v_empty = bars + 12,
+           *s_full = bars + 16, *p_full = bars + 18, *b_full = bars + 20, *b_empty = bars + 22, *o_done = bars + 24, *o_free = bars + 26,
+           *chain = bars + 27 /* [2][4] */, *fin = bars + 35 /* [2][4] */;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 44);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  float* s_m = reinterpret_cast<float*>(smem + C::kTiles + C::kBarriers);      // [128] row maximum that O is scaled by
+  float2* s_l = reinterpret_cast<float2*>(s_m + 128);                          // [2 items][2 groups][128] sum and its maximum
+  float* s_bias = reinterpret_cast<float*>(s_l + 2 * 2 * 128);                 // [2][kBiasTable]
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x == 0) {
+    for (int x = 0; x < 2; ++x) {
+      mbar_init(&q_full[x], 1);
+      mbar_init(&q_empty[x], 1);
+      mbar_init(&k_full[x], 1);
+      mbar_init(&k_empty[x], 1);
+      mbar_init(&s_full[x], 1);
+      mbar_init(&p_full[x], 4);   // one arrival per softmax warp of the group
+      mbar_init(&b_full[x], 1);
+      mbar_init(&b_empty[x], 8);  // one arrival per softmax warp
+      mbar_init(&o_done[x], 1);   // of even and odd tiles: a wait must know that the phase before the one it waits for is over
+    }
+    for (int x = 0; x < 4; ++x) {
+      mbar_init(&v_full[x], 1);
+      mbar_init(&v_empty[x], 1);
+    }
+    for (int x = 0; x < 8; ++x) {
+      mbar_init(&chain[x], 1);
+      mbar_init(&fin[x], 1);
+    }
+    mbar_init(o_free, 8);
+    *abort_flag = 0;
+    fence_mbar_init();
+  }
+  if (warp == 9) {
+    tmem_alloc(tmem_slot, 512);
+    tmem_relinquish();
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem_base = *tmem_slot;
+
+  if (warp >= 8) {
+    asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(kOtherRegs));
+    if (warp == 8 && lane == 0) {
+      // ---------------------------------------------------------------- TMA producer
+      int items = 0, nk = 0, nv = 0, round = 0;
+      bool ok = true;
+      Work w;
+      auto wait = [&](uint64_t* bar, int parity) {
+        if (mbar_wait_bounded(bar, parity, abort_flag)) return true;
+        atomicCAS(p.status, 0, kStatusTimeoutProducer);
+        return false;
+      };
+      auto keys = [&](int j) {
+        const int s = nk % KS;
+        if (!wait(&k_empty[s], ((nk / KS) & 1) ^ 1)) return false;
+        ++nk;
+        mbar_arrive_expect_tx(&k_full[s], C::kKBytes);
+#pragma unroll
+        for (int c = 0; c < ND; ++c)
+          tma_load_3d(sK + s * C::kKBytes + c * kSlab, &tm_k, &k_full[s], 64 * c, w.h / p.rep, w.kv0 + w.k_lo + j * 128);
+        return true;
+      };
+      for (; ok && next_work(p, round, w); ++items) {
+        const int qs = items % QS;
+        ok = wait(&q_empty[qs], ((items / QS) & 1) ^ 1);   // the Q K^T of the item that used it are done
+        if (!ok) break;
+        mbar_arrive_expect_tx(&q_full[qs], C::kQBytes);
+#pragma unroll
+        for (int c = 0; c < ND; ++c) tma_load_3d(sQ + qs * C::kQBytes + c * kSlab, &tm_q, &q_full[qs], 64 * c, w.h, w.row0);
+        if (p.bias != nullptr) {
+          const int b = items & 1;
+          ok = wait(&b_empty[b], ((items >> 1) & 1) ^ 1);
+          if (!ok) break;
+          mbar_arrive_expect_tx(&b_full[b], p.bias_pitch * 4);
+          bulk_load(s_bias + b * kBiasTable, p.bias + static_cast<int64_t>(w.h) * p.bias_pitch, p.bias_pitch * 4, &b_full[b]);
+        }
+        ok = keys(0);
+        if (ok && w.n > 1) ok = keys(1);
+        for (int j = 0; ok && j < w.n; ++j) {
+          for (int half = 0; ok && half < 2; ++half, ++nv) {
+            const int s = nv % VS;
+            ok = wait(&v_empty[s], ((nv / VS) & 1) ^ 1);
+            if (!ok) break;
+            mbar_arrive_expect_tx(&v_full[s], w.slabs * kHalfSlab);
+            for (int c = 0; c < w.slabs; ++c)
+              tma_load_3d(sV + s * C::kVBytes + c * kHalfSlab, &tm_v, &v_full[s], 64 * (c % p.slabs), w.c0 + c / p.slabs,
+                          w.kv0 + w.k_lo + j * 128 + half * 64);
+          }
+          if (ok && j + 2 < w.n) ok = keys(j + 2);
+        }
+      }
+    } else if (warp == 9) {
+      // ---------------------------------------------------------------- MMA issuer: the warp walks, one elected lane issues
+      const bool leader = elect_one();
+      const uint32_t idesc_s = make_idesc(kFmtBF16, kFmtBF16, false, false, 128, 128);
+      const uint32_t tmem_o = tmem_base + 256;
+      int items = 0, t0 = 0, nv = 0, round = 0;
+      bool ok = true;
+      Work w{};
+      auto wait = [&](uint64_t* bar, int parity) {
+        if (__all_sync(0xffffffffu, mbar_wait_bounded(bar, parity, abort_flag))) return true;
+        if (leader) atomicCAS(p.status, 0, kStatusTimeoutMma);
+        return false;
+      };
+      auto scores = [&](int j) {             // S(j) = Q K(j)^T; the P of tile j - 2, in the same columns, has been issued to P V
+        const int t = t0 + j;
+        if (!wait(&k_full[t % KS], (t / KS) & 1)) return false;
+        tc_fence_after_sync();
+        if (leader) {
+          const uint64_t dQ = desc_kmajor(smem_u32(sQ + (items % QS) * C::kQBytes), 128, 0);
+          const uint64_t dK = desc_kmajor(smem_u32(sK + (t % KS) * C::kKBytes), 128, 0);
+          for (int ks = 0; ks < p.ksteps; ++ks)
+            umma_f16_ss(tmem_base + (t & 1) * 128, dQ + kstep_kmajor(128, ks), dK + kstep_kmajor(128, ks), idesc_s, ks > 0 ? 1u : 0u);
+          umma_commit(&s_full[t & 1]);
+          umma_commit(&k_empty[t % KS]);
+          if (j + 1 == w.n) umma_commit(&q_empty[items % QS]);
+        }
+        __syncwarp();
+        return true;
+      };
+      for (; ok && next_work(p, round, w); ++items) {
+        const uint32_t idesc_o = make_idesc(kFmtBF16, kFmtBF16, false, true, 128, w.slabs * 64);
+        ok = wait(&q_full[items % QS], (items / QS) & 1);
+        if (ok) ok = scores(0);
+        if (ok && w.n > 1) ok = scores(1);
+        for (int j = 0; ok && j < w.n; ++j) {
+          const int t = t0 + j;
+          ok = wait(&p_full[t & 1], (t >> 1) & 1);
+          if (ok && j == 0 && items > 0) ok = wait(o_free, (items - 1) & 1);     // the rows of the previous item have been read
+          for (int half = 0; ok && half < 2; ++half, ++nv) {
+            const int s = nv % VS;
+            ok = wait(&v_full[s], (nv / VS) & 1);
+            if (!ok) break;
+            tc_fence_after_sync();
+            if (leader) {
+              const uint64_t dV = desc_mnmajor(smem_u32(sV + s * C::kVBytes), 64, 0);
+              const uint32_t pa = tmem_base + (t & 1) * 128 + half * 32;
+#pragma unroll
+              for (int ks = 0; ks < 4; ++ks)
+                umma_f16_ts(tmem_o, pa + ks * 8, dV + kstep_mnmajor(ks), idesc_o, j > 0 || half > 0 || ks > 0 ? 1u : 0u);
+              umma_commit(&v_empty[s]);
+              if (half == 1) umma_commit(&o_done[t & 1]);
+            }
+            __syncwarp();
+          }
+          if (ok && j + 2 < w.n) ok = scores(j + 2);
+        }
+        t0 += w.n;
+      }
+    }
+  } else {
+    // ------------------------------------------------------------------ softmax + output rows
+    asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(kSoftmaxRegs));
+    const int x = warp >> 2, quad = warp & 3, r = quad * 32 + lane;    // group; row inside the tile == TMEM lane
+    const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
+    const uint32_t tmem_s = tmem_base + x * 128 + lane_addr, tmem_o = tmem_base + 256 + lane_addr;
+    uint64_t *mine = chain + x * 4 + quad, *theirs = chain + (x ^ 1) * 4 + quad;
+    const float sc = p.scale * kLog2e;
+    int items = 0, t0 = 0, round = 0;
+    bool ok = true;
+    Work w;
+    auto wait = [&](uint64_t* bar, int parity) {
+      if (__all_sync(0xffffffffu, mbar_wait_bounded(bar, parity, abort_flag))) return true;
+      if (lane == 0) atomicCAS(p.status, 0, kStatusTimeoutEpilogue);
+      return false;
+    };
+    for (; ok && next_work(p, round, w); ++items) {
+      const int pos = w.pos0 + r, row_lo = p.first_key(pos), last_lo = p.first_key(w.pos0 + 127);
+      const float* bias = nullptr;
+      float b_far = 0.0f;
+      if (p.bias != nullptr) {
+        ok = wait(&b_full[items & 1], (items >> 1) & 1);
+        if (!ok) break;
+        bias = s_bias + (items & 1) * kBiasTable + kBiasNear;
+        b_far = bias[p.bias_len - 1];
+        bias += pos;
+      }
+      float m_own = -INFINITY, l_run = 0.0f;
+      for (int j = (t0 ^ x) & 1; j < w.n; j += 2) {
+        const int t = t0 + j, k0 = w.k_lo + j * 128;
+        ok = wait(&s_full[x], (t >> 1) & 1);
+        if (!ok) break;
+        tc_fence_after_sync();
+        uint32_t sv[4][32];
+#pragma unroll
+        for (int cc = 0; cc < 4; ++cc) tmem_ld_32x32b_x32(tmem_s + cc * 32, sv[cc]);
+        tmem_ld_wait();
+        // scores in units of log2: mul * product + add; a tile that no row is far from gets its biases one by one
+        float mul = sc, add = b_far;
+        if (bias != nullptr && w.pos0 - k0 - 127 < p.bias_len - 1) {
+          mul = 1.0f;
+          add = 0.0f;
+          const float* b = bias - k0;
+#pragma unroll
+          for (int cc = 0; cc < 4; ++cc)
+#pragma unroll
+            for (int c = 0; c < 32; ++c) sv[cc][c] = __float_as_uint(fmaf(__uint_as_float(sv[cc][c]), sc, b[-(cc * 32 + c)]));
+        }
+        if (k0 + 127 > w.pos0 || k0 < last_lo) {
+          const int clo = row_lo - k0, chi = pos - k0;       // column c is visible iff clo <= c <= chi
+#pragma unroll
+          for (int cc = 0; cc < 4; ++cc)
+#pragma unroll
+            for (int c = 0; c < 32; ++c)
+              if (cc * 32 + c < clo || cc * 32 + c > chi) sv[cc][c] = 0xff800000u;  // -inf
+        }
+        float m0 = -INFINITY, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;
+#pragma unroll
+        for (int cc = 0; cc < 4; ++cc)
+#pragma unroll
+          for (int c = 0; c < 32; c += 4) {
+            m0 = fmaxf(m0, __uint_as_float(sv[cc][c]));
+            m1 = fmaxf(m1, __uint_as_float(sv[cc][c + 1]));
+            m2 = fmaxf(m2, __uint_as_float(sv[cc][c + 2]));
+            m3 = fmaxf(m3, __uint_as_float(sv[cc][c + 3]));
+          }
+        const float m_tile = fmaf(fmaxf(fmaxf(m0, m1), fmaxf(m2, m3)), mul, add);
+        // the maxima after tile j - 1, from the warp that has the same rows there
+        if (t > 0) {
+          ok = wait(theirs, ((t - 1) >> 1) & 1);
+          if (!ok) break;
+        }
+        const float m_prev = j > 0 ? s_m[r] : -INFINITY;
+        const float m_new = fmaxf(m_prev, m_tile);
+        const bool grow = m_new - kRescaleStep > m_prev;
+        const float m_ref = grow ? m_new : m_prev;
+        s_m[r] = m_ref;
+        __syncwarp();
+        if (lane == 0) mbar_arrive(mine);
+        if (j > 0 && __any_sync(0xffffffffu, grow)) {   // the output tile holds the sums of the earlier key tiles
+          const float alpha = grow ? ex2f(m_prev - m_new) : 1.0f;
+          ok = wait(&o_done[x ^ 1], ((t - 1) >> 1) & 1);   // S(t) came after P(t - 2) V
+          if (!ok) break;
+          tc_fence_after_sync();
+          for (int cc = 0; cc < w.slabs * 2; ++cc) {
+            uint32_t ov[32];
+            tmem_ld_32x32b_x32(tmem_o + cc * 32, ov);
+            tmem_ld_wait();
+#pragma unroll
+            for (int c = 0; c < 32; ++c) ov[c] = __float_as_uint(__uint_as_float(ov[c]) * alpha);
+            tmem_st_32x32b_x32(tmem_o + cc * 32, ov);
+          }
+          tmem_st_wait();
+        }
+        if (m_ref != m_own) {
+          l_run *= ex2f(m_own - m_ref);               // m_own == -inf -> 0
+          m_own = m_ref;
+        }
+        const float m_use = (m_ref == -INFINITY ? 0.0f : m_ref) - add;
+        float r0 = 0.0f, r1 = 0.0f, r2 = 0.0f, r3 = 0.0f;
+#pragma unroll
+        for (int cc = 0; cc < 4; ++cc) {
+          uint32_t pk[16];
+#pragma unroll
+          for (int g = 0; g < 4; ++g) {
+            float e[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) e[i] = ex2f(fmaf(__uint_as_float(sv[cc][8 * g + i]), mul, -m_use));  // -inf -> 0
+            r0 += e[0] + e[4];
+            r1 += e[1] + e[5];
+            r2 += e[2] + e[6];
+            r3 += e[3] + e[7];
+            pk[4 * g + 0] = pack_bf16x2(e[0], e[1]);
+            pk[4 * g + 1] = pack_bf16x2(e[2], e[3]);
+            pk[4 * g + 2] = pack_bf16x2(e[4], e[5]);
+            pk[4 * g + 3] = pack_bf16x2(e[6], e[7]);
+          }
+          tmem_st_32x32b_x16(tmem_s + cc * 16, pk);  // two probabilities per column
+        }
+        l_run += (r0 + r1) + (r2 + r3);
+        tmem_st_wait();
+        tc_fence_before_sync();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&p_full[x]);
+      }
+      if (!ok) break;
+      // both groups' sums, each relative to the maximum it last saw; not before all warps are done with the previous item's
+      if (items > 0) {
+        ok = wait(o_free, (items - 1) & 1);
+        if (!ok) break;
+      }
+      float2* stats = s_l + (items & 1) * 256;
+      stats[x * 128 + r] = make_float2(l_run, m_own);
+      __syncwarp();
+      if (lane == 0) {
+        if (p.bias != nullptr) mbar_arrive(&b_empty[items & 1]);
+        mbar_arrive(fin + x * 4 + quad);
+      }
+      ok = wait(fin + (x ^ 1) * 4 + quad, items & 1);
+      if (!ok) break;
+      const float2 other = stats[(x ^ 1) * 128 + r];
+      const float m_end = fmaxf(m_own, other.y);
+      const float total = (m_own == -INFINITY ? 0.0f : l_run * ex2f(m_own - m_end)) +
+                          (other.y == -INFINITY ? 0.0f : other.x * ex2f(other.y - m_end));
+      const int t_last = t0 + w.n - 1;
+      ok = wait(&o_done[t_last & 1], (t_last >> 1) & 1);   // the last P V has retired; S(t_last), seen by now, came after P(t_last - 2) V
+      if (!ok) break;
+      tc_fence_after_sync();
+      const bool row_ok = r < w.rows;
+      const float inv = row_ok ? 1.0f / total : 0.0f;
+      __nv_bfloat16* orow = p.out + static_cast<int64_t>(w.row0 + r) * p.ldo + (static_cast<int64_t>(w.h) * p.kv_heads + w.c0) * p.vdim;
+      for (int s = x * 2; s < min(x * 2 + 2, w.slabs); ++s) {      // group A: the first two slabs, B: the others
+        __nv_bfloat16* o = orow + static_cast<int64_t>(s / p.slabs) * p.vdim;
+        const int d0 = 64 * (s % p.slabs);
+#pragma unroll
+        for (int cc = 0; cc < 2; ++cc) {
+          uint32_t ov[32];
+          tmem_ld_32x32b_x32(tmem_o + s * 64 + cc * 32, ov);
+          tmem_ld_wait();
+          if (!row_ok) continue;
+#pragma unroll
+          for (int g = 0; g < 4; ++g) {
+            const int d = d0 + cc * 32 + g * 8;
+            if (d >= p.vdim) continue;
+            uint4 wv;
+            wv.x = pack_bf16x2(__uint_as_float(ov[8 * g + 0]) * inv, __uint_as_float(ov[8 * g + 1]) * inv);
+            wv.y = pack_bf16x2(__uint_as_float(ov[8 * g + 2]) * inv, __uint_as_float(ov[8 * g + 3]) * inv);
+            wv.z = pack_bf16x2(__uint_as_float(ov[8 * g + 4]) * inv, __uint_as_float(ov[8 * g + 5]) * inv);
+            wv.w = pack_bf16x2(__uint_as_float(ov[8 * g + 6]) * inv, __uint_as_float(ov[8 * g + 7]) * inv);
+            *reinterpret_cast<uint4*>(o + d) = wv;
+          }
+        }
+      }
+      tc_fence_before_sync();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(o_free);
+      t0 += w.n;
+    }
+  }
+
+  tc_fence_before_sync();
+  __syncthreads();
+  if (*abort_flag != 0) {       // copies in flight still write to this CTA's shared memory
+    const uint64_t t_end = globaltimer_ns();
+    while (globaltimer_ns() - t_end < 2000000ull) __nanosleep(2000);
+    __syncthreads();
+  }
+  if (warp == 9) {
+    tc_fence_after_sync();
+    tmem_dealloc(tmem_base, 512);
+  }
+}
+
+// tensor map of [rows][heads][columns], box `box_rows` x 1 x 64: columns past a head's width arrive as zeros
+int head_map(CUtensorMap* m, const void* base, int cols, int heads, int rows, int64_t row_ld, int box_rows) {
+  nx::EncodeTiledFn fn = nx::encode_tiled_fn();
+  if (fn == nullptr) return -3;
+  cuuint64_t dims[3] = {static_cast<cuuint64_t>(cols), static_cast<cuuint64_t>(heads), static_cast<cuuint64_t>(rows)};
+  cuuint64_t strides[2] = {static_cast<cuuint64_t>(cols) * 2, static_cast<cuuint64_t>(row_ld) * 2};
+  cuuint32_t box[3] = {64, 1, static_cast<cuuint32_t>(box_rows)}, one[3] = {1, 1, 1};
+  return fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, one, CU_TENSOR_MAP_INTERLEAVE_NONE,
+            CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS
+             ? 0
+             : -4;
+}
+
+template <int ND>
+int launch(const CUtensorMap& q, const CUtensorMap& k, const CUtensorMap& v, const Dev& p, cudaStream_t st) {
+  static bool once = false;
+  if (!once) {
+    cudaFuncAttributes at;     // the register split above counts on what the block is launched with
+    if (cudaFuncGetAttributes(&at, talk_prompt_kernel<ND>) != cudaSuccess || at.numRegs != 168) return -5;
+    if (cudaFuncSetAttribute(talk_prompt_kernel<ND>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<ND>::kSmem) != cudaSuccess) return -2;
+    once = true;
+  }
+  int sms = 0, dev = 0;
+  if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) return -2;
+  talk_prompt_kernel<ND><<<std::min(p.items, sms), kThreads, Cfg<ND>::kSmem, st>>>(q, k, v, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -2;
+}
+
+}  // namespace
+
+extern "C" int nx_talk_prompt(const NxTalkPromptArgs* a, nx_stream_t stream) {
+  if (a == nullptr || a->status == nullptr || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || !(a->scale > 0.0f)) return -1;
+  if (a->dim <= 0 || a->dim > 128 || (a->dim & 15) || a->vdim <= 0 || a->vdim > 128 || (a->vdim & 7) || a->chunk < 0) return -1;
+  if ((a->ldq | a->ldk | a->ldv | a->ldo) & 7) return -1;
+  for (const void* ptr : {a->q, a->k, a->v, static_cast<const void*>(a->out), static_cast<const void*>(a->blocks)})
+    if (ptr == nullptr || (reinterpret_cast<uintptr_t>(ptr) & 15)) return -1;
+  if (a->bias != nullptr && (a->bias_len <= 0 || a->bias_pitch < NX_TALK_BIAS_NEAR + a->bias_len + NX_TALK_BIAS_FAR || (a->bias_pitch & 3) ||
+                             a->bias_pitch > kBiasTable || (reinterpret_cast<uintptr_t>(a->bias) & 15)))
+    return -1;
+  if (a->n_blocks <= 0) return 0;
+  CUtensorMap q, k, v;
+  int rc;
+  if ((rc = head_map(&q, a->q, a->dim, a->heads, a->q_rows, a->ldq, 128))) return rc;
+  if ((rc = head_map(&k, a->k, a->dim, a->kv_heads, a->kv_rows, a->ldk, 128))) return rc;
+  if ((rc = head_map(&v, a->v, a->vdim, a->kv_heads, a->kv_rows, a->ldv, 64))) return rc;
+  Dev p{};
+  p.blocks = a->blocks;
+  p.bias = a->bias;
+  p.out = static_cast<__nv_bfloat16*>(a->out);
+  p.status = a->status;
+  p.ldo = a->ldo;
+  p.heads = a->heads;
+  p.kv_heads = a->kv_heads;
+  p.rep = a->heads / a->kv_heads;
+  p.vdim = a->vdim;
+  p.window = a->window;
+  p.chunk = a->chunk;
+  p.ksteps = a->dim / 16;
+  p.bias_len = a->bias_len;
+  p.bias_pitch = a->bias_pitch;
+  p.slabs = a->vdim <= 64 ? 1 : 2;
+  p.at_once = kSlabs / p.slabs;
+  p.passes = (a->kv_heads + p.at_once - 1) / p.at_once;
+  const int64_t items = static_cast<int64_t>(a->n_blocks) * 2 * a->heads * p.passes;
+  if (items > 0x3fffffff) return -1;
+  p.items = static_cast<int>(items);
+  p.scale = a->scale;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return a->dim <= 64 ? launch<1>(q, k, v, p, st) : launch<2>(q, k, v, p, st);
+}

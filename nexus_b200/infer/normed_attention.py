@@ -6,9 +6,10 @@ zero-padded to sizes the kernels load in whole vectors; norms count the real col
 
 Heads that mix their weights after the softmax.  out_h = sum_g T[h, g] (P_g V of the KV head of h), so:
 
-* decoding: scores of all heads, then per KV head the mixture of the normalised weights and one product with its values;
-* prompts: every head's weights meet the values of every KV head inside the attention kernel, and the mixture is taken over those
-  outputs."""
+* decoding and short segments: scores of all heads, then the mixture of the normalised weights, then one product per KV head with its
+  values;
+* longer segments and FP32: every head's weights meet the values of every KV head inside the attention kernel, and the mixture is taken
+  over those outputs."""
 from __future__ import annotations
 
 import torch
@@ -25,7 +26,6 @@ class NormedAttentionShape:
         self.dim, self.vdim = _pad(m.dim, 16), _pad(m.vdim, 8)
         self.q, self.k, self.v = m.heads * self.dim, m.kv_heads * self.dim, m.kv_heads * self.vdim
         self.offsets = (0, self.q, self.q + self.k, self.q + self.k + self.v)      # q, k, v, gate
-        self.values = m.kv_heads if m.talk else 1        # KV heads whose values a query head meets
 
 
 def check(engine, i: int, m: NormedAttentionSpec) -> None:
@@ -41,6 +41,7 @@ def check(engine, i: int, m: NormedAttentionSpec) -> None:
 
 def load(engine, m: NormedAttentionSpec, get) -> dict:
     """``get(name)``: the mixer's tensors."""
+    from ..ops import _mixers as M
     s = NormedAttentionShape(m)
     parts = (("q", m.heads, s.dim), ("k", m.kv_heads, s.dim), ("v", m.kv_heads, s.vdim))
 
@@ -56,12 +57,14 @@ def load(engine, m: NormedAttentionSpec, get) -> dict:
         out[n + "_norm"] = engine._f32(_pad_heads(get(n + ".norm"), heads if m.norm == "all" else 1, s.dim))
     out["head_scale"] = engine._f32(get("temp")) if m.head_scale else None
     out["talk"] = engine._f32(get("talk")) if m.talk else None
-    out["bias"] = None
+    out["bias"] = out["bias_wide"] = None
     if m.distance is not None:      # one entry per distance; the last one counts for all beyond
         rows = [m.distance.bucket(n) for n in range(m.distance.far + 1)]
         while len(rows) > 1 and rows[-1] == rows[-2]:
             rows.pop()
         out["bias"] = engine._f32(get("rel").float()[rows].t())
+        if promptable(m):
+            out["bias_wide"] = M.extended_bias(out["bias"])
     return out
 
 
@@ -97,38 +100,45 @@ def mixer(engine, i: int, m: NormedAttentionSpec, lw: dict, h, pos, slot):
                 k_cache=engine.k_cache[i], v_cache=engine.v_cache[i], gate=gate)
     q = proj[:, : s.q]
     out = torch.empty((n, m.heads * s.vdim), dtype=engine.adt, device=engine.dev)
-    # heads that mix: `wide` takes what the attention kernels give; decoding in BF16 writes `out` itself
-    mixed = m.talk and (not engine.fast or engine._many.count > 0)
-    wide = torch.empty((n, m.heads * s.values * s.vdim), dtype=engine.adt, device=engine.dev) if mixed else out
     kw = dict(heads=m.heads, block_size=engine.cfg.block_size, window=m.window, chunk=m.chunk, scale=1.0, softcap=m.softcap,
               bias=lw["bias"])
     paged = (engine.k_cache[i], engine.v_cache[i], engine.block_table)
-    late = dict(gate=None if m.talk else gate, all_values=s.values > 1)
+    sizes = dict(heads=m.heads, kv_heads=m.kv_heads, vdim=s.vdim)
+
+    def keys_of_step():
+        w = window(m)
+        if not step.gathered:
+            return (proj[:, o: o + cols] for o, cols in zip(s.offsets[1:3], (s.k, s.v)))
+        k, v = (torch.empty((step.kv_rows[w], cols), dtype=engine.adt, device=engine.dev) for cols in (s.k, s.v))
+        for c, dst in ((engine.k_cache[i], k), (engine.v_cache[i], v)):
+            M.latent_gather(c, engine.block_table, step.runs[w], step.longest[w], dst)
+        return k, v
+    if m.talk:
+        if not engine.fast or long_.count:
+            wide = torch.empty((n, m.heads * m.kv_heads * s.vdim), dtype=engine.adt, device=engine.dev)
+            if step is not None:
+                M.talk_prompt(q, *keys_of_step(), wide, step.blocks[window(m)], dim=s.dim, window=m.window, chunk=m.chunk, scale=1.0,
+                              bias=lw["bias_wide"], distances=lw["bias"].shape[1] if lw["bias"] is not None else 0, **sizes)
+            else:
+                M.paged_window_attention(q, *paged, wide, long_ if engine.fast else engine._every, all_values=True, **kw)
+            M.head_mix(wide, lw["talk"], gate, out, **sizes)
+        for seg in (single, short) if engine.fast else ():       # after the mixture, which ran over all rows
+            if seg.count:
+                M.talk_paged(q, *paged, out, lw["talk"], seg, keys=engine._most_keys(m), splits=engine._decode_splits(m, seg.count),
+                             gate=gate, **kw)
+        return engine._linear(out, lw["out"])
 
     def attend(seg, **more):
         if seg.count:
-            M.paged_window_attention(q, *paged, wide, seg, **kw, **late, **more)
+            M.paged_window_attention(q, *paged, out, seg, gate=gate, **kw, **more)
     if not engine.fast:
         attend(engine._every)
-    elif step is None:
+        return engine._linear(out, lw["out"])
+    attend(single, splits=engine._decode_splits(m, single.count))
+    if step is None:
         attend(engine._many)
     else:
         attend(short)
-        w = window(m)
-        if step.gathered:
-            k, v = (torch.empty((step.kv_rows[w], cols), dtype=engine.adt, device=engine.dev) for cols in (s.k, s.v))
-            for c, dst in ((engine.k_cache[i], k), (engine.v_cache[i], v)):
-                M.latent_gather(c, engine.block_table, step.runs[w], step.longest[w], dst)
-        else:
-            k, v = (proj[:, o: o + cols] for o, cols in zip(s.offsets[1:3], (s.k, s.v)))
-        M.window_prompt(q, k, v, wide, step.blocks[w], heads=m.heads, kv_heads=m.kv_heads, dim=s.dim, vdim=s.vdim, window=m.window,
-                        chunk=m.chunk, scale=1.0, bias=lw["bias"], **late)
-    if mixed:
-        M.head_mix(wide, lw["talk"], gate, out, heads=m.heads, kv_heads=m.kv_heads, vdim=s.vdim)
-    if engine.fast and single.count:
-        splits = engine._decode_splits(m, single.count)
-        if m.talk:
-            M.talk_decode(q, *paged, out, lw["talk"], single, keys=engine._most_keys(m), splits=splits, gate=gate, **kw)
-        else:
-            M.paged_window_attention(q, *paged, out, single, splits=splits, gate=gate, **kw)
+        M.window_prompt(q, *keys_of_step(), out, step.blocks[window(m)], dim=s.dim, window=m.window, chunk=m.chunk, scale=1.0,
+                        bias=lw["bias"], gate=gate, **sizes)
     return engine._linear(out, lw["out"])

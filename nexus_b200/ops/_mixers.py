@@ -4,6 +4,7 @@ recurrences, gated norms, gated activations and the per-layer token input.  BF16
 from __future__ import annotations
 
 import ctypes as C
+import math
 from dataclasses import dataclass
 from typing import Optional
 
@@ -116,8 +117,17 @@ class PagedWindowArgs(C.Structure):
                 ("bias", C.c_void_p)]
 
 
-class TalkDecodeArgs(C.Structure):
-    _fields_ = [("base", PagedWindowArgs), ("talk", C.c_void_p), ("scores", C.c_void_p), ("score_pitch", C.c_int64)]
+class TalkPagedArgs(C.Structure):
+    _fields_ = [("base", PagedWindowArgs), ("talk", C.c_void_p), ("scores", C.c_void_p), ("weights", C.c_void_p), ("pitch", C.c_int64),
+                ("rows", C.c_int32)]
+
+
+class TalkPromptArgs(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("out", C.c_void_p), ("bias", C.c_void_p),
+                ("blocks", C.c_void_p), ("status", C.c_void_p), ("ldq", C.c_int64), ("ldk", C.c_int64), ("ldv", C.c_int64),
+                ("ldo", C.c_int64), ("n_blocks", C.c_int32), ("q_rows", C.c_int32), ("kv_rows", C.c_int32), ("heads", C.c_int32),
+                ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("window", C.c_int32), ("chunk", C.c_int32),
+                ("bias_len", C.c_int32), ("bias_pitch", C.c_int32), ("scale", C.c_float)]
 
 
 class LatentPromptArgs(C.Structure):
@@ -134,7 +144,7 @@ class WindowPromptArgs(C.Structure):
                 ("ldv", C.c_int64), ("ldo", C.c_int64), ("n_blocks", C.c_int32), ("q_rows", C.c_int32), ("kv_rows", C.c_int32),
                 ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("window", C.c_int32),
                 ("keep_first", C.c_int32), ("scale", C.c_float), ("gate", C.c_void_p), ("bias", C.c_void_p), ("bias_len", C.c_int32),
-                ("chunk", C.c_int32), ("all_values", C.c_int32)]
+                ("chunk", C.c_int32)]
 
 
 class LatentAttnArgs(C.Structure):
@@ -145,8 +155,10 @@ class LatentAttnArgs(C.Structure):
 
 
 LATENT_MAX_RANK, LATENT_MAX_ROW = 512, 768
-PROMPT_MAX_BIAS = 3584       # distances of a bias table of the tcgen05 prompt kernel
+PROMPT_MAX_BIAS = 3072       # distances of a bias table of the tcgen05 prompt kernels
 TALK_MAX_HEADS = 96          # heads that mix their weights
+TALK_SCRATCH = 1 << 29       # bytes of scores and weights of one launch of such heads
+BIAS_MARGIN = 256            # entries of an extended bias table on either side of its distances
 
 
 @dataclass
@@ -400,17 +412,28 @@ def paged_window_attention(q, k_cache, v_cache, block_table, out, seg: Segments,
         K._check(K.lib().nx_paged_window_prefill(C.byref(a), K._stream()), "nx_paged_window_prefill")
 
 
-def talk_decode(q, k_cache, v_cache, block_table, out, talk, seg: Segments, *, heads, block_size, window, scale, keys, softcap=0.0,
-                splits=1, gate=None, keep_first=0, chunk=0, bias=None) -> None:
-    """Decoding with heads that mix their weights (``talk``: FP32 [heads, heads]); ``keys``: the most keys a row can see."""
-    a = TalkDecodeArgs(_paged_args(q, k_cache, v_cache, block_table, out, seg, heads, block_size, window, scale, softcap, 1.0, gate, 0,
-                                   keep_first, None, chunk, bias, False), _ptr(talk), None, (keys + 63) // 64 * 64)
-    a.base.splits = splits
-    a.base.part_ml = K.scratch(seg.count * heads * splits * 8, "window_ml", q.device).data_ptr()
-    if splits > 1:
-        a.base.part_o = K.scratch(seg.count * heads * splits * a.base.vdim * 4, "window_o", q.device).data_ptr()
-    a.scores = K.scratch(seg.count * heads * a.score_pitch * 4, "talk_scores", q.device).data_ptr()
-    K._check(K.lib().nx_talk_decode(C.byref(a), K._stream()), "nx_talk_decode")
+def talk_paged(q, k_cache, v_cache, block_table, out, talk, seg: Segments, *, heads, block_size, window, scale, keys, softcap=0.0,
+               splits=1, gate=None, keep_first=0, chunk=0, bias=None) -> None:
+    """One-row and short segments of heads that mix their weights (``talk``: FP32 [heads, heads], to, from); ``keys``: the most keys a
+    row can see.  The segments run in portions whose scratch stays below `TALK_SCRATCH`."""
+    G, Dv, lib = k_cache.shape[2], v_cache.shape[3], K.lib()
+    pitch = (keys + min(seg.max_len, 64) + 63) // 64 * 64       # the rows of one tile, up to 64 tokens, see this many together
+    each = heads * (pitch * 6 + splits * (8 + (Dv * 4 if splits > 1 else 0)))
+    rows = lib.nx_talk_rows(C.c_int(heads), C.c_int(G), C.c_int(seg.count), C.c_int(seg.max_len), C.c_int(seg.total))
+    at = max(1, seg.count * TALK_SCRATCH // max(1, rows * each)) if rows * each > TALK_SCRATCH else seg.count
+    for i in range(0, seg.count, at):
+        part = seg if at >= seg.count else Segments(seg.table, seg.first + i, min(at, seg.count - i), seg.max_len,
+                                                    min(seg.total, min(at, seg.count - i) * seg.max_len))
+        n = lib.nx_talk_rows(C.c_int(heads), C.c_int(G), C.c_int(part.count), C.c_int(part.max_len), C.c_int(part.total))
+        a = TalkPagedArgs(_paged_args(q, k_cache, v_cache, block_table, out, part, heads, block_size, window, scale, softcap, 1.0, gate, 0,
+                                      keep_first, None, chunk, bias, False), _ptr(talk), None, None, pitch, n)
+        a.base.splits = splits
+        a.base.part_ml = K.scratch(n * heads * splits * 8, "window_ml", q.device).data_ptr()
+        if splits > 1:
+            a.base.part_o = K.scratch(n * heads * splits * Dv * 4, "window_o", q.device).data_ptr()
+        a.scores = K.scratch(n * heads * pitch * 4, "talk_scores", q.device).data_ptr()
+        a.weights = K.scratch(n * heads * pitch * 2, "talk_weights", q.device).data_ptr()
+        K._check(lib.nx_talk_paged(C.byref(a), K._stream()), "nx_talk_paged")
 
 
 def latent_attention(q, cache, block_table, out, seg: Segments, *, heads, rank, window, scale, gate=None, splits=1) -> None:
@@ -437,15 +460,32 @@ def latent_prompt(q, kv, lat, out, blocks, *, heads, dim, rot, vdim, rank, windo
 
 
 def window_prompt(q, k, v, out, blocks, *, heads, kv_heads, dim, vdim, window, scale, keep_first=0, kept=None, sink=None, gate=None,
-                  chunk=0, bias=None, all_values=False) -> None:
+                  chunk=0, bias=None) -> None:
     """The tcgen05 form on plain grouped keys and values.  q [rows, heads * dim], k [kv rows, kv_heads * dim], v [kv rows, kv_heads *
     vdim]; blocks as in `latent_prompt`; kept int32 [n]: the row that position 0 has among the kept first keys (None: the block's);
-    chunk, bias and all_values as in `paged_window_attention`."""
+    chunk and bias as in `paged_window_attention`."""
     a = WindowPromptArgs(_ptr(q), _ptr(k), _ptr(v), _ptr(out), _ptr(sink), _ptr(blocks), _ptr(kept),
                          K.status_word(q.device).data_ptr(), q.stride(0), k.stride(0), v.stride(0), out.stride(0), blocks.shape[0],
                          q.shape[0], k.shape[0], heads, kv_heads, dim, vdim, window, keep_first, scale, _ptr(gate), _ptr(bias),
-                         bias.shape[1] if bias is not None else 0, chunk, int(all_values))
+                         bias.shape[1] if bias is not None else 0, chunk)
     K._check(K.lib().nx_window_prompt(C.byref(a), K._stream()), "nx_window_prompt")
+
+
+def extended_bias(bias: torch.Tensor) -> torch.Tensor:
+    """The biases [heads, distances] in the layout of `talk_prompt`: units of log2, the first and last one repeated on either side, rows
+    of whole 16 bytes."""
+    n = bias.shape[1]
+    at = torch.arange(-BIAS_MARGIN, (n + BIAS_MARGIN + 3) // 4 * 4, device=bias.device).clamp(0, n - 1)
+    return (bias.double() * math.log2(math.e)).float()[:, at].contiguous()
+
+
+def talk_prompt(q, k, v, out, blocks, *, heads, kv_heads, dim, vdim, window, scale, chunk=0, bias=None, distances=0) -> None:
+    """`window_prompt` for heads that mix: every head's weights with the values of every KV head, out [rows, heads * kv_heads * vdim].
+    ``bias``: `extended_bias` of ``distances`` distances."""
+    a = TalkPromptArgs(_ptr(q), _ptr(k), _ptr(v), _ptr(out), _ptr(bias), _ptr(blocks), K.status_word(q.device).data_ptr(), q.stride(0),
+                       k.stride(0), v.stride(0), out.stride(0), blocks.shape[0], q.shape[0], k.shape[0], heads, kv_heads, dim, vdim,
+                       window, chunk, distances, bias.shape[1] if bias is not None else 0, scale)
+    K._check(K.lib().nx_talk_prompt(C.byref(a), K._stream()), "nx_talk_prompt")
 
 
 def latent_gather(cache, block_table, runs, longest, dst) -> None:
