@@ -145,7 +145,7 @@ def kernel_cases():
             lambda qd=qd, od=od, kc=kc, vc=vc, table=table, pk=pk: M.paged_window_attention(qd, kc, vc, table, od, one, **pk), 0, kv)
         cases[f"talk_paged, 32 portions of 8 behind 1016, {sizes}"] = (
             lambda qd=qd, od=od, kc=kc, vc=vc, table=table, rel=rel, talk=talk, gate=gate, pk=pk: M.talk_paged(
-                qd, kc, vc, table, od, talk, short, keys=1024, gate=gate, bias=rel, **pk), 4.0 * B * H * D * 1024, 32 * 1024 * G * D * 4)
+                qd, kc, vc, table, od, talk, short, keys=1024, gate=gate, bias=rel, splits=2, **pk), 4.0 * B * H * D * 1024, 32 * 1024 * G * D * 4)
         cases[f"like: paged_window_prefill, 32 portions of 8 behind 1016, {sizes}"] = (
             lambda qd=qd, od=od, kc=kc, vc=vc, table=table, pk=pk: M.paged_window_attention(qd, kc, vc, table, od, short, **pk),
             4.0 * B * H * D * 1024, 32 * 1024 * G * D * 4)

@@ -87,49 +87,64 @@ __global__ void head_prep_kernel(const NxHeadPrepArgs a) {
 
 // ------------------------------------------------------------------------------------------------
 // out_h = gate_h sum_g talk[h][g] wide[g][KV head of h]: a thread owns V adjacent columns of one KV head's values and forms all
-// query heads of that KV head, kHeadsAtOnce at a time
+// query heads of that KV head, N at a time; a group of N mixture factors is one or two vector loads
 // ------------------------------------------------------------------------------------------------
-constexpr int kHeadsAtOnce = 8;
+constexpr int kMixAhead = 8;       // rows of `wide` in flight per thread
 
-template <typename T, int V>
-__global__ void head_mix_kernel(const T* __restrict__ wide, int64_t ldw, const float* __restrict__ talk,
-                                const float* __restrict__ gate, T* __restrict__ out, int64_t ldo, int rows, int heads, int kv_heads,
-                                int vdim) {
-  extern __shared__ __align__(16) float s_talk[];       // [heads][heads]
-  for (int i = threadIdx.x + threadIdx.y * blockDim.x; i < heads * heads; i += blockDim.x * blockDim.y) s_talk[i] = talk[i];
+template <typename T, int V, int N>
+__global__ void __launch_bounds__(256)
+head_mix_kernel(const T* __restrict__ wide, int64_t ldw, const float* __restrict__ talk, const float* __restrict__ gate,
+                T* __restrict__ out, int64_t ldo, int rows, int heads, int kv_heads, int vdim) {
+  extern __shared__ __align__(16) float s_talk[];       // [KV head][group of N heads][from head][N]
+  const int rep = heads / kv_heads, groups = (rep + N - 1) / N, cols = kv_heads * vdim;
+  for (int i = threadIdx.x + threadIdx.y * blockDim.x; i < kv_heads * groups * heads * N; i += blockDim.x * blockDim.y) {
+    const int k = i % N, g = i / N % heads, grp = i / (N * heads) % groups, c = i / (N * heads * groups), h = grp * N + k;
+    s_talk[i] = h < rep ? talk[(c * rep + h) * heads + g] : 0.0f;
+  }
   __syncthreads();
-  const int rep = heads / kv_heads, cols = kv_heads * vdim;
   for (int64_t r = blockIdx.x * static_cast<int64_t>(blockDim.y) + threadIdx.y; r < rows;
        r += static_cast<int64_t>(gridDim.x) * blockDim.y) {
     for (int i = threadIdx.x * V; i < cols; i += blockDim.x * V) {
       const int c = i / vdim, d = i % vdim;
       const T* src = wide + r * ldw + i;
-      for (int h0 = c * rep; h0 < (c + 1) * rep; h0 += kHeadsAtOnce) {
-        const int nh = min(kHeadsAtOnce, (c + 1) * rep - h0);
-        float acc[kHeadsAtOnce][V];
+      for (int grp = 0; grp < groups; ++grp) {
+        const float* t = s_talk + static_cast<int64_t>(c * groups + grp) * heads * N;
+        float acc[N][V];
 #pragma unroll
-        for (int k = 0; k < kHeadsAtOnce; ++k)
+        for (int k = 0; k < N; ++k)
 #pragma unroll
           for (int j = 0; j < V; ++j) acc[k][j] = 0.0f;
-#pragma unroll 4
-        for (int g = 0; g < heads; ++g) {
-          float v[V];
-          load_vec<T, V>(src + static_cast<int64_t>(g) * cols, v);
+        for (int g0 = 0; g0 < heads; g0 += kMixAhead) {
+          uint4 raw[kMixAhead];                           // V elements of T each
 #pragma unroll
-          for (int k = 0; k < kHeadsAtOnce; ++k) {
-            if (k >= nh) break;
-            const float t = s_talk[(h0 + k) * heads + g];
+          for (int u = 0; u < kMixAhead; ++u) {
+            const T* p = src + static_cast<int64_t>(min(g0 + u, heads - 1)) * cols;
+            if constexpr (V * sizeof(T) == 16) raw[u] = __ldcs(reinterpret_cast<const uint4*>(p));
+            else *reinterpret_cast<T*>(&raw[u]) = *p;
+          }
 #pragma unroll
-            for (int j = 0; j < V; ++j) acc[k][j] += t * v[j];
+          for (int u = 0; u < kMixAhead; ++u) {
+            if (g0 + u >= heads) break;
+            const T* e = reinterpret_cast<const T*>(&raw[u]);
+            float f[N];
+#pragma unroll
+            for (int k = 0; k < N; k += 4) *reinterpret_cast<float4*>(f + k) = *reinterpret_cast<const float4*>(t + (g0 + u) * N + k);
+#pragma unroll
+            for (int j = 0; j < V; ++j) {
+              const float v = Num<T>::load(e + j);
+#pragma unroll
+              for (int k = 0; k < N; ++k) acc[k][j] = fmaf(f[k], v, acc[k][j]);
+            }
           }
         }
 #pragma unroll
-        for (int k = 0; k < kHeadsAtOnce; ++k) {
-          if (k >= nh) break;
-          const float f = gate != nullptr ? gate[r * heads + h0 + k] : 1.0f;
+        for (int k = 0; k < N; ++k) {
+          const int h = c * rep + grp * N + k;
+          if (grp * N + k >= rep) break;
+          const float w = gate != nullptr ? gate[r * heads + h] : 1.0f;
 #pragma unroll
-          for (int j = 0; j < V; ++j) acc[k][j] *= f;
-          store_vec<T, V>(out + r * ldo + static_cast<int64_t>(h0 + k) * vdim + d, acc[k]);
+          for (int j = 0; j < V; ++j) acc[k][j] *= w;
+          store_vec<T, V>(out + r * ldo + static_cast<int64_t>(h) * vdim + d, acc[k]);
         }
       }
     }
@@ -170,17 +185,33 @@ extern "C" int nx_head_mix(const void* wide, int64_t ldw, const float* talk, con
   if (ldw < static_cast<int64_t>(heads) * kv_heads * vdim || ldo < static_cast<int64_t>(heads) * vdim) return -1;
   if (rows <= 0) return 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const bool vec = vdim % 4 == 0 && ldw % 4 == 0 && ldo % 4 == 0 &&
+  const int v16 = dtype == NX_BF16 ? 8 : 4, n = heads / kv_heads <= 4 ? 4 : 8, groups = (heads / kv_heads + n - 1) / n;
+  const bool vec = vdim % v16 == 0 && ldw % v16 == 0 && ldo % v16 == 0 &&
                    ((reinterpret_cast<uintptr_t>(wide) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
-  const int work = kv_heads * vdim / (vec ? 4 : 1);
+  const int work = kv_heads * vdim / (vec ? v16 : 1);
   const int tx = std::max(32, std::min(256, (work + 31) / 32 * 32)), ty = std::max(1, 256 / tx);
   const dim3 threads(tx, ty);
-  const int blocks = std::min((rows + ty - 1) / ty, kNumSmsB200 * 16);
-  const size_t smem = static_cast<size_t>(heads) * heads * sizeof(float);
-#define NX_HM(T_, V_) head_mix_kernel<T_, V_><<<blocks, threads, smem, st>>>((const T_*)wide, ldw, talk, gate, (T_*)out, ldo, rows, heads, kv_heads, vdim)
-  if (dtype == NX_BF16) { if (vec) NX_HM(__nv_bfloat16, 4); else NX_HM(__nv_bfloat16, 1); }
-  else if (dtype == NX_F32) { if (vec) NX_HM(float, 4); else NX_HM(float, 1); }
-  else return -1;
+  const int blocks = std::min((rows + ty - 1) / ty, kNumSmsB200 * 8);
+  const int smem = kv_heads * groups * n * heads * static_cast<int>(sizeof(float));
+#define NX_HM(T_, V_, N_)                                                                                                       \
+  do {                                                                                                                          \
+    if (smem > 48 * 1024 &&                                                                                                     \
+        cudaFuncSetAttribute(head_mix_kernel<T_, V_, N_>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)    \
+      return -2;                                                                                                                \
+    head_mix_kernel<T_, V_, N_><<<blocks, threads, smem, st>>>((const T_*)wide, ldw, talk, gate, (T_*)out, ldo, rows, heads,    \
+                                                               kv_heads, vdim);                                                 \
+  } while (0)
+  if (dtype == NX_BF16) {
+    if (vec) { if (n == 4) NX_HM(__nv_bfloat16, 8, 4); else NX_HM(__nv_bfloat16, 8, 8); }
+    else if (n == 4) NX_HM(__nv_bfloat16, 1, 4);
+    else NX_HM(__nv_bfloat16, 1, 8);
+  } else if (dtype == NX_F32) {
+    if (vec) { if (n == 4) NX_HM(float, 4, 4); else NX_HM(float, 4, 8); }
+    else if (n == 4) NX_HM(float, 1, 4);
+    else NX_HM(float, 1, 8);
+  } else {
+    return -1;
+  }
 #undef NX_HM
   return launch_status();
 }

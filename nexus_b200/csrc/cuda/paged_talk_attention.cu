@@ -4,7 +4,7 @@
 //   scores   rows of one KV head against its keys, FP32 scores with the maximum and sum of each span of keys
 //   mixture  per row and 64 keys: the normalised weights of all heads, mixed (FP32), as the BF16 operand of the products
 //   values   rows of one KV head: weights times values; spans of keys are added up by a fourth kernel
-// A tile is 16 or 64 (token, head) rows of one KV head; keys and values are read once per tile.
+// A tile is 16, 32 or 64 (token, head) rows of one KV head; keys and values are read once per tile.
 #include "mixer_common.cuh"
 #include "nx_api_mixers.h"
 #include "paged_keys.cuh"
@@ -417,7 +417,7 @@ int launch_all(const NxTalkPagedArgs* t, int rt, int tq, cudaStream_t st) {
   if (smem > 48 * 1024 &&
       cudaFuncSetAttribute(talk_mix_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
     return -2;
-  const int strides = static_cast<int>(std::max<int64_t>(1, std::min<int64_t>(t->pitch / kKeys, 1184 / std::max(1, t->rows))));
+  const int strides = static_cast<int>(std::max<int64_t>(1, std::min<int64_t>(t->pitch / kKeys, 4736 / std::max(1, t->rows))));
   talk_mix_kernel<<<dim3(t->rows, strides), kMixThreads, smem, st>>>(*t, tq);
   if ((rc = launch_status())) return rc;
   rc = a.vdim <= 64    ? launch_values<64, MT>(t, grid, rt, tq, head_tiles, st)
@@ -430,8 +430,14 @@ int launch_all(const NxTalkPagedArgs* t, int rt, int tq, cudaStream_t st) {
   return rc;
 }
 
-// tokens of a tile
-int tile_tokens(int heads, int kv_heads, int max_len) { return max_len == 1 ? 1 : 64 / std::min(heads / kv_heads, 16); }
+// rows (a multiple of 16) and tokens of a tile
+int tile_rows(int heads, int kv_heads, int max_len) {
+  const int rt = std::min(heads / kv_heads, 16);
+  return max_len == 1 ? 16 : max_len * rt <= 32 ? 32 : 64;
+}
+int tile_tokens(int heads, int kv_heads, int max_len) {
+  return max_len == 1 ? 1 : tile_rows(heads, kv_heads, max_len) / std::min(heads / kv_heads, 16);
+}
 
 }  // namespace
 
@@ -454,5 +460,9 @@ extern "C" int nx_talk_paged(const NxTalkPagedArgs* t, nx_stream_t stream) {
   if (t->rows != nx_talk_rows(a->heads, a->kv_heads, a->seg.count, a->seg.max_len, a->seg.total_len)) return -1;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int rt = std::min(a->heads / a->kv_heads, 16), tq = tile_tokens(a->heads, a->kv_heads, a->seg.max_len);
-  return a->seg.max_len == 1 ? launch_all<1>(t, rt, tq, st) : launch_all<4>(t, rt, tq, st);
+  switch (tile_rows(a->heads, a->kv_heads, a->seg.max_len)) {
+    case 16: return launch_all<1>(t, rt, tq, st);
+    case 32: return launch_all<2>(t, rt, tq, st);
+    default: return launch_all<4>(t, rt, tq, st);
+  }
 }

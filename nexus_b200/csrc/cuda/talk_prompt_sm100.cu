@@ -20,8 +20,7 @@
 namespace {
 using namespace nx;
 
-constexpr int kThreads = 384;        // warps 0-3: softmax A, 4-7: softmax B, 8: TMA, 9: MMA, 10-11 idle
-constexpr int kSoftmaxRegs = 216, kOtherRegs = 72;     // 256 * 216 + 128 * 72 = 384 * 168: what the block was launched with
+constexpr int kThreads = 320;        // warps 0-3: softmax A, 4-7: softmax B, 8: TMA, 9: MMA
 constexpr int kSlab = 128 * 128;     // bytes of [128 rows][64 columns]
 constexpr int kHalfSlab = 64 * 128;  // of [64 keys][64 columns] of values
 constexpr int kSlabs = 4;            // 64-column slabs of values in one item
@@ -45,7 +44,8 @@ struct Dev {
   int* status;
   int64_t ldo;
   int items, heads, kv_heads, rep, vdim, window, chunk, ksteps, bias_len, bias_pitch;
-  int slabs, at_once, passes;   // slabs of one KV head's values, KV heads of one item, items per (tile, head)
+  int slabs, at_once, passes;   // slabs of one KV head's values (1, 2), KV heads of one item, items per (tile, head)
+  int wide_store;               // output rows and heads start on 32 bytes
   float scale;
   __device__ __forceinline__ int first_key(int pos) const {
     const int lo = window > 0 ? max(0, pos - window + 1) : 0;
@@ -53,8 +53,15 @@ struct Dev {
   }
 };
 
+// 32 bytes, 32-byte aligned
+__device__ __forceinline__ void store32(void* p, const uint32_t* v) {
+  asm volatile("st.global.v8.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(p), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]),
+               "r"(v[5]), "r"(v[6]), "r"(v[7])
+               : "memory");
+}
+
 struct Work {
-  int h, c0, slabs;                // query head, first KV head of the values, their slabs
+  int h, hk, c0;                   // query head, its KV head, first KV head of the values
   int row0, rows, pos0, kv0, k_lo, n;   // n: key tiles
 };
 // the CTA's items in order; an item whose half block holds no rows is left out by every role
@@ -70,8 +77,8 @@ __device__ __forceinline__ bool next_work(const Dev& p, int& round, Work& w) {
     w.rows = min(128, b.y - half * 128);
     if (w.rows <= 0) continue;
     w.h = sub % p.heads;
+    w.hk = w.h / p.rep;
     w.c0 = sub / p.heads % p.passes * p.at_once;
-    w.slabs = min(p.at_once, p.kv_heads - w.c0) * p.slabs;
     w.row0 = b.x + half * 128;
     w.pos0 = b.z + half * 128;
     w.kv0 = b.w;
@@ -141,10 +148,10 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
   const uint32_t tmem_base = *tmem_slot;
 
   if (warp >= 8) {
-    asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(kOtherRegs));
     if (warp == 8 && lane == 0) {
       // ---------------------------------------------------------------- TMA producer
       int items = 0, nk = 0, nv = 0, round = 0;
+      const int v_bytes = p.at_once * p.slabs * kHalfSlab;
       bool ok = true;
       Work w;
       auto wait = [&](uint64_t* bar, int parity) {
@@ -159,7 +166,7 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
         mbar_arrive_expect_tx(&k_full[s], C::kKBytes);
 #pragma unroll
         for (int c = 0; c < ND; ++c)
-          tma_load_3d(sK + s * C::kKBytes + c * kSlab, &tm_k, &k_full[s], 64 * c, w.h / p.rep, w.kv0 + w.k_lo + j * 128);
+          tma_load_3d(sK + s * C::kKBytes + c * kSlab, &tm_k, &k_full[s], 64 * c, w.hk, w.kv0 + w.k_lo + j * 128);
         return true;
       };
       for (; ok && next_work(p, round, w); ++items) {
@@ -183,10 +190,11 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
             const int s = nv % VS;
             ok = wait(&v_empty[s], ((nv / VS) & 1) ^ 1);
             if (!ok) break;
-            mbar_arrive_expect_tx(&v_full[s], w.slabs * kHalfSlab);
-            for (int c = 0; c < w.slabs; ++c)
-              tma_load_3d(sV + s * C::kVBytes + c * kHalfSlab, &tm_v, &v_full[s], 64 * (c % p.slabs), w.c0 + c / p.slabs,
-                          w.kv0 + w.k_lo + j * 128 + half * 64);
+            mbar_arrive_expect_tx(&v_full[s], v_bytes);
+            uint8_t* d = sV + s * C::kVBytes;                // one slab of every KV head, then their second slabs
+            const int row = w.kv0 + w.k_lo + j * 128 + half * 64;
+            tma_load_3d(d, &tm_v, &v_full[s], 0, row, w.c0);
+            if (p.slabs > 1) tma_load_3d(d + p.at_once * kHalfSlab, &tm_v, &v_full[s], 64, row, w.c0);
           }
           if (ok && j + 2 < w.n) ok = keys(j + 2);
         }
@@ -195,6 +203,7 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
       // ---------------------------------------------------------------- MMA issuer: the warp walks, one elected lane issues
       const bool leader = elect_one();
       const uint32_t idesc_s = make_idesc(kFmtBF16, kFmtBF16, false, false, 128, 128);
+      const uint32_t idesc_o = make_idesc(kFmtBF16, kFmtBF16, false, true, 128, p.at_once * p.slabs * 64);
       const uint32_t tmem_o = tmem_base + 256;
       int items = 0, t0 = 0, nv = 0, round = 0;
       bool ok = true;
@@ -221,7 +230,6 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
         return true;
       };
       for (; ok && next_work(p, round, w); ++items) {
-        const uint32_t idesc_o = make_idesc(kFmtBF16, kFmtBF16, false, true, 128, w.slabs * 64);
         ok = wait(&q_full[items % QS], (items / QS) & 1);
         if (ok) ok = scores(0);
         if (ok && w.n > 1) ok = scores(1);
@@ -252,7 +260,6 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
     }
   } else {
     // ------------------------------------------------------------------ softmax + output rows
-    asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(kSoftmaxRegs));
     const int x = warp >> 2, quad = warp & 3, r = quad * 32 + lane;    // group; row inside the tile == TMEM lane
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
     const uint32_t tmem_s = tmem_base + x * 128 + lane_addr, tmem_o = tmem_base + 256 + lane_addr;
@@ -283,40 +290,46 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
         ok = wait(&s_full[x], (t >> 1) & 1);
         if (!ok) break;
         tc_fence_after_sync();
-        uint32_t sv[4][32];
+        // Two passes over the 128 columns, 64 at a time, each in a loop that is not unrolled: the code of a tile stays small enough not
+        // to push that of the other warps out of the instruction cache.  Scores in units of log2: mul * product + add; a tile that has
+        // masked columns, or biases of its own for every distance, is rewritten with both applied.
+        const bool near = bias != nullptr && w.pos0 - k0 - 127 < p.bias_len - 1;
+        const bool rewrite = near || k0 + 127 > w.pos0 || k0 < last_lo;
+        const float mul = rewrite ? 1.0f : sc, add = rewrite ? 0.0f : b_far;
+        const int clo = row_lo - k0, chi = pos - k0;       // column c is visible iff clo <= c <= chi
+        float m_tile = -INFINITY;
+#pragma unroll 1
+        for (int c0 = 0; c0 < 128; c0 += 64) {
+          uint32_t sv[2][32];
+          tmem_ld_32x32b_x32(tmem_s + c0, sv[0]);
+          tmem_ld_32x32b_x32(tmem_s + c0 + 32, sv[1]);
+          tmem_ld_wait();
+          if (rewrite) {
+            const float* b = bias - k0 - c0;
 #pragma unroll
-        for (int cc = 0; cc < 4; ++cc) tmem_ld_32x32b_x32(tmem_s + cc * 32, sv[cc]);
-        tmem_ld_wait();
-        // scores in units of log2: mul * product + add; a tile that no row is far from gets its biases one by one
-        float mul = sc, add = b_far;
-        if (bias != nullptr && w.pos0 - k0 - 127 < p.bias_len - 1) {
-          mul = 1.0f;
-          add = 0.0f;
-          const float* b = bias - k0;
+            for (int cc = 0; cc < 2; ++cc) {
 #pragma unroll
-          for (int cc = 0; cc < 4; ++cc)
-#pragma unroll
-            for (int c = 0; c < 32; ++c) sv[cc][c] = __float_as_uint(fmaf(__uint_as_float(sv[cc][c]), sc, b[-(cc * 32 + c)]));
-        }
-        if (k0 + 127 > w.pos0 || k0 < last_lo) {
-          const int clo = row_lo - k0, chi = pos - k0;       // column c is visible iff clo <= c <= chi
-#pragma unroll
-          for (int cc = 0; cc < 4; ++cc)
-#pragma unroll
-            for (int c = 0; c < 32; ++c)
-              if (cc * 32 + c < clo || cc * 32 + c > chi) sv[cc][c] = 0xff800000u;  // -inf
-        }
-        float m0 = -INFINITY, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;
-#pragma unroll
-        for (int cc = 0; cc < 4; ++cc)
-#pragma unroll
-          for (int c = 0; c < 32; c += 4) {
-            m0 = fmaxf(m0, __uint_as_float(sv[cc][c]));
-            m1 = fmaxf(m1, __uint_as_float(sv[cc][c + 1]));
-            m2 = fmaxf(m2, __uint_as_float(sv[cc][c + 2]));
-            m3 = fmaxf(m3, __uint_as_float(sv[cc][c + 3]));
+              for (int c = 0; c < 32; ++c) {
+                const float v = fmaf(__uint_as_float(sv[cc][c]), sc, near ? b[-(cc * 32 + c)] : b_far);
+                sv[cc][c] = cc * 32 + c < clo - c0 || cc * 32 + c > chi - c0 ? 0xff800000u : __float_as_uint(v);  // -inf
+              }
+              tmem_st_32x32b_x32(tmem_s + c0 + cc * 32, sv[cc]);
+            }
           }
-        const float m_tile = fmaf(fmaxf(fmaxf(m0, m1), fmaxf(m2, m3)), mul, add);
+          float m0 = m_tile, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;
+#pragma unroll
+          for (int cc = 0; cc < 2; ++cc)
+#pragma unroll
+            for (int c = 0; c < 32; c += 4) {
+              m0 = fmaxf(m0, __uint_as_float(sv[cc][c]));
+              m1 = fmaxf(m1, __uint_as_float(sv[cc][c + 1]));
+              m2 = fmaxf(m2, __uint_as_float(sv[cc][c + 2]));
+              m3 = fmaxf(m3, __uint_as_float(sv[cc][c + 3]));
+            }
+          m_tile = fmaxf(fmaxf(m0, m1), fmaxf(m2, m3));
+        }
+        if (rewrite) tmem_st_wait();
+        m_tile = fmaf(m_tile, mul, add);
         // the maxima after tile j - 1, from the warp that has the same rows there
         if (t > 0) {
           ok = wait(theirs, ((t - 1) >> 1) & 1);
@@ -334,7 +347,8 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
           ok = wait(&o_done[x ^ 1], ((t - 1) >> 1) & 1);   // S(t) came after P(t - 2) V
           if (!ok) break;
           tc_fence_after_sync();
-          for (int cc = 0; cc < w.slabs * 2; ++cc) {
+#pragma unroll 1
+          for (int cc = 0; cc < p.at_once * p.slabs * 2; ++cc) {
             uint32_t ov[32];
             tmem_ld_32x32b_x32(tmem_o + cc * 32, ov);
             tmem_ld_wait();
@@ -350,24 +364,29 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
         }
         const float m_use = (m_ref == -INFINITY ? 0.0f : m_ref) - add;
         float r0 = 0.0f, r1 = 0.0f, r2 = 0.0f, r3 = 0.0f;
+#pragma unroll 1
+        for (int c0 = 0; c0 < 128; c0 += 64) {
+          uint32_t sv[2][32], pk[32];
+          tmem_ld_32x32b_x32(tmem_s + c0, sv[0]);
+          tmem_ld_32x32b_x32(tmem_s + c0 + 32, sv[1]);
+          tmem_ld_wait();
 #pragma unroll
-        for (int cc = 0; cc < 4; ++cc) {
-          uint32_t pk[16];
+          for (int cc = 0; cc < 2; ++cc)
 #pragma unroll
-          for (int g = 0; g < 4; ++g) {
-            float e[8];
+            for (int g = 0; g < 4; ++g) {
+              float e[8];
 #pragma unroll
-            for (int i = 0; i < 8; ++i) e[i] = ex2f(fmaf(__uint_as_float(sv[cc][8 * g + i]), mul, -m_use));  // -inf -> 0
-            r0 += e[0] + e[4];
-            r1 += e[1] + e[5];
-            r2 += e[2] + e[6];
-            r3 += e[3] + e[7];
-            pk[4 * g + 0] = pack_bf16x2(e[0], e[1]);
-            pk[4 * g + 1] = pack_bf16x2(e[2], e[3]);
-            pk[4 * g + 2] = pack_bf16x2(e[4], e[5]);
-            pk[4 * g + 3] = pack_bf16x2(e[6], e[7]);
-          }
-          tmem_st_32x32b_x16(tmem_s + cc * 16, pk);  // two probabilities per column
+              for (int i = 0; i < 8; ++i) e[i] = ex2f(fmaf(__uint_as_float(sv[cc][8 * g + i]), mul, -m_use));  // -inf -> 0
+              r0 += e[0] + e[4];
+              r1 += e[1] + e[5];
+              r2 += e[2] + e[6];
+              r3 += e[3] + e[7];
+              pk[16 * cc + 4 * g + 0] = pack_bf16x2(e[0], e[1]);
+              pk[16 * cc + 4 * g + 1] = pack_bf16x2(e[2], e[3]);
+              pk[16 * cc + 4 * g + 2] = pack_bf16x2(e[4], e[5]);
+              pk[16 * cc + 4 * g + 3] = pack_bf16x2(e[6], e[7]);
+            }
+          tmem_st_32x32b_x32(tmem_s + c0 / 2, pk);  // two probabilities per column, over scores that have been read
         }
         l_run += (r0 + r1) + (r2 + r3);
         tmem_st_wait();
@@ -401,26 +420,25 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
       const bool row_ok = r < w.rows;
       const float inv = row_ok ? 1.0f / total : 0.0f;
       __nv_bfloat16* orow = p.out + static_cast<int64_t>(w.row0 + r) * p.ldo + (static_cast<int64_t>(w.h) * p.kv_heads + w.c0) * p.vdim;
-      for (int s = x * 2; s < min(x * 2 + 2, w.slabs); ++s) {      // group A: the first two slabs, B: the others
-        __nv_bfloat16* o = orow + static_cast<int64_t>(s / p.slabs) * p.vdim;
-        const int d0 = 64 * (s % p.slabs);
+      const int heads_here = min(p.at_once, p.kv_heads - w.c0);
+#pragma unroll 1
+      for (int cc = x; cc < p.at_once * p.slabs * 2; cc += 2) {      // 32 columns each, the groups in turn
+        const int s = cc >> 1, second = s >= p.at_once ? 1 : 0, c = s - second * p.at_once, d0 = second * 64 + (cc & 1) * 32;
+        uint32_t ov[32];
+        tmem_ld_32x32b_x32(tmem_o + cc * 32, ov);
+        tmem_ld_wait();
+        if (!row_ok || c >= heads_here || d0 >= p.vdim) continue;
+        uint32_t pk[16];
 #pragma unroll
-        for (int cc = 0; cc < 2; ++cc) {
-          uint32_t ov[32];
-          tmem_ld_32x32b_x32(tmem_o + s * 64 + cc * 32, ov);
-          tmem_ld_wait();
-          if (!row_ok) continue;
+        for (int i = 0; i < 16; ++i) pk[i] = pack_bf16x2(__uint_as_float(ov[2 * i]) * inv, __uint_as_float(ov[2 * i + 1]) * inv);
+        __nv_bfloat16* o = orow + static_cast<int64_t>(c) * p.vdim + d0;
+        if (p.wide_store && d0 + 32 <= p.vdim) {       // whole sectors
+          store32(o, pk);
+          store32(o + 16, pk + 8);
+        } else {
 #pragma unroll
-          for (int g = 0; g < 4; ++g) {
-            const int d = d0 + cc * 32 + g * 8;
-            if (d >= p.vdim) continue;
-            uint4 wv;
-            wv.x = pack_bf16x2(__uint_as_float(ov[8 * g + 0]) * inv, __uint_as_float(ov[8 * g + 1]) * inv);
-            wv.y = pack_bf16x2(__uint_as_float(ov[8 * g + 2]) * inv, __uint_as_float(ov[8 * g + 3]) * inv);
-            wv.z = pack_bf16x2(__uint_as_float(ov[8 * g + 4]) * inv, __uint_as_float(ov[8 * g + 5]) * inv);
-            wv.w = pack_bf16x2(__uint_as_float(ov[8 * g + 6]) * inv, __uint_as_float(ov[8 * g + 7]) * inv);
-            *reinterpret_cast<uint4*>(o + d) = wv;
-          }
+          for (int g = 0; g < 4; ++g)
+            if (d0 + g * 8 < p.vdim) *reinterpret_cast<uint4*>(o + g * 8) = make_uint4(pk[4 * g], pk[4 * g + 1], pk[4 * g + 2], pk[4 * g + 3]);
         }
       }
       tc_fence_before_sync();
@@ -443,13 +461,20 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
   }
 }
 
-// tensor map of [rows][heads][columns], box `box_rows` x 1 x 64: columns past a head's width arrive as zeros
-int head_map(CUtensorMap* m, const void* base, int cols, int heads, int rows, int64_t row_ld, int box_rows) {
+// Tensor map of [rows][heads][columns]: columns past a head's width and heads past the last arrive as zeros.  box_heads 0: box of 128
+// rows of one head, coordinates (column, head, row); else of box_heads slabs of 64 rows, coordinates (column, row, head).
+int head_map(CUtensorMap* m, const void* base, int cols, int heads, int rows, int64_t row_ld, int box_heads) {
   nx::EncodeTiledFn fn = nx::encode_tiled_fn();
   if (fn == nullptr) return -3;
-  cuuint64_t dims[3] = {static_cast<cuuint64_t>(cols), static_cast<cuuint64_t>(heads), static_cast<cuuint64_t>(rows)};
-  cuuint64_t strides[2] = {static_cast<cuuint64_t>(cols) * 2, static_cast<cuuint64_t>(row_ld) * 2};
-  cuuint32_t box[3] = {64, 1, static_cast<cuuint32_t>(box_rows)}, one[3] = {1, 1, 1};
+  const int head = box_heads > 0 ? 2 : 1, row = 3 - head;
+  cuuint64_t dims[3] = {static_cast<cuuint64_t>(cols), 0, 0}, strides[2];
+  cuuint32_t box[3] = {64, 1, 1}, one[3] = {1, 1, 1};
+  dims[head] = static_cast<cuuint64_t>(heads);
+  dims[row] = static_cast<cuuint64_t>(rows);
+  strides[head - 1] = static_cast<cuuint64_t>(cols) * 2;
+  strides[row - 1] = static_cast<cuuint64_t>(row_ld) * 2;
+  box[head] = static_cast<cuuint32_t>(std::max(1, box_heads));
+  box[row] = box_heads > 0 ? 64 : 128;
   return fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, one, CU_TENSOR_MAP_INTERLEAVE_NONE,
             CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS
              ? 0
@@ -460,8 +485,6 @@ template <int ND>
 int launch(const CUtensorMap& q, const CUtensorMap& k, const CUtensorMap& v, const Dev& p, cudaStream_t st) {
   static bool once = false;
   if (!once) {
-    cudaFuncAttributes at;     // the register split above counts on what the block is launched with
-    if (cudaFuncGetAttributes(&at, talk_prompt_kernel<ND>) != cudaSuccess || at.numRegs != 168) return -5;
     if (cudaFuncSetAttribute(talk_prompt_kernel<ND>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<ND>::kSmem) != cudaSuccess) return -2;
     once = true;
   }
@@ -485,10 +508,13 @@ extern "C" int nx_talk_prompt(const NxTalkPromptArgs* a, nx_stream_t stream) {
   if (a->n_blocks <= 0) return 0;
   CUtensorMap q, k, v;
   int rc;
-  if ((rc = head_map(&q, a->q, a->dim, a->heads, a->q_rows, a->ldq, 128))) return rc;
-  if ((rc = head_map(&k, a->k, a->dim, a->kv_heads, a->kv_rows, a->ldk, 128))) return rc;
-  if ((rc = head_map(&v, a->v, a->vdim, a->kv_heads, a->kv_rows, a->ldv, 64))) return rc;
   Dev p{};
+  p.slabs = a->vdim <= 64 ? 1 : 2;
+  p.at_once = std::min(kSlabs / p.slabs, a->kv_heads);
+  p.passes = (a->kv_heads + p.at_once - 1) / p.at_once;
+  if ((rc = head_map(&q, a->q, a->dim, a->heads, a->q_rows, a->ldq, 0))) return rc;
+  if ((rc = head_map(&k, a->k, a->dim, a->kv_heads, a->kv_rows, a->ldk, 0))) return rc;
+  if ((rc = head_map(&v, a->v, a->vdim, a->kv_heads, a->kv_rows, a->ldv, p.at_once))) return rc;
   p.blocks = a->blocks;
   p.bias = a->bias;
   p.out = static_cast<__nv_bfloat16*>(a->out);
@@ -503,9 +529,7 @@ extern "C" int nx_talk_prompt(const NxTalkPromptArgs* a, nx_stream_t stream) {
   p.ksteps = a->dim / 16;
   p.bias_len = a->bias_len;
   p.bias_pitch = a->bias_pitch;
-  p.slabs = a->vdim <= 64 ? 1 : 2;
-  p.at_once = kSlabs / p.slabs;
-  p.passes = (a->kv_heads + p.at_once - 1) / p.at_once;
+  p.wide_store = (a->ldo % 16 == 0 && a->vdim % 16 == 0 && (reinterpret_cast<uintptr_t>(a->out) & 31) == 0) ? 1 : 0;
   const int64_t items = static_cast<int64_t>(a->n_blocks) * 2 * a->heads * p.passes;
   if (items > 0x3fffffff) return -1;
   p.items = static_cast<int>(items);
