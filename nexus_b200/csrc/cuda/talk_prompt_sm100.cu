@@ -3,13 +3,11 @@
 // nx_head_mix takes the mixture.
 //
 // A work item is a tile of 128 query rows, one query head and up to 256 columns of values (several KV heads side by side): the scores and
-// the softmax are formed once for all of them.  S lives twice in TMEM (columns 0-127, 128-255), O behind it (256-511).  One persistent
-// CTA per SM: softmax group A (warps 0-3) takes the even key tiles of the CTA's running count, group B (warps 4-7) the odd ones, so
-// that one group exponentiates while the other's scores are on their way.  The MMA warp issues
-//   S(0), S(1), P(0) V, S(2), P(1) V, S(3), ..
-// Both groups add to one O, so they share the row maxima O is scaled by: tile j passes them on to tile j + 1, between the two warps
-// that own the same 32 rows.  O is rescaled only when a row's maximum has grown by 2^8.  A head's table of biases (in units of log2,
-// extended to both sides) arrives by bulk copy beside its queries.
+// the softmax are formed once for all of them.  Key tiles have 64 keys; S lives four times in TMEM (columns 0-255), O behind it
+// (256-511).  One persistent CTA per SM: two softmax groups of four warps take the key tiles of the CTA's running count in turn; one warp
+// issues the products Q K^T up to four tiles ahead, another P V.  Both groups add to one O, so they share the row maxima that O is scaled
+// by: tile j passes them on to tile j + 1, between the two warps that own the same 32 rows.  O is rescaled only when a row's maximum has
+// grown by 2^8.  A head's table of biases (in units of log2, extended to both sides) arrives by bulk copy beside its queries.
 #include "flash_common.cuh"
 #include "nx_api_mixers.h"
 #include "sm100_ptx.cuh"
@@ -20,19 +18,22 @@
 namespace {
 using namespace nx;
 
-constexpr int kThreads = 320;        // warps 0-3: softmax A, 4-7: softmax B, 8: TMA, 9: MMA
+constexpr int kGroups = 2;           // softmax groups
+constexpr int kThreads = (kGroups * 4 + 3) * 32;   // after the softmax warps: TMA, Q K^T, P V
+constexpr int kKeys = 64;            // keys of a tile
+constexpr int kTilesAhead = 4;       // score tiles in TMEM
 constexpr int kSlab = 128 * 128;     // bytes of [128 rows][64 columns]
-constexpr int kHalfSlab = 64 * 128;  // of [64 keys][64 columns] of values
+constexpr int kKeySlab = kKeys * 128;  // of [64 keys][64 columns]
 constexpr int kSlabs = 4;            // 64-column slabs of values in one item
 constexpr int kBiasNear = NX_TALK_BIAS_NEAR, kBiasTable = NX_TALK_BIAS_NEAR + NX_TALK_BIAS_MAX + NX_TALK_BIAS_FAR;
 
 // ND: 64-column slabs of a key
 template <int ND>
 struct Cfg {
-  static constexpr int kQStages = ND == 1 ? 2 : 1, kKStages = 2, kVStages = ND == 1 ? 4 : 3;
-  static constexpr int kQBytes = ND * kSlab, kKBytes = ND * kSlab, kVBytes = kSlabs * kHalfSlab;
+  static constexpr int kQStages = ND == 1 ? 2 : 1, kKStages = 4, kVStages = ND == 1 ? 4 : 3;
+  static constexpr int kQBytes = ND * kSlab, kKBytes = ND * kKeySlab, kVBytes = kSlabs * kKeySlab;
   static constexpr int kTiles = kQStages * kQBytes + kKStages * kKBytes + kVStages * kVBytes;
-  static constexpr int kBarriers = 512, kStats = 128 * 4 + 2 * 2 * 128 * 8;
+  static constexpr int kBarriers = 512, kStats = 128 * 4 + kGroups * 128 * 8;
   static constexpr int kSmem = kTiles + kBarriers + kStats + 2 * kBiasTable * 4;
   static_assert(kSmem <= 227 * 1024, "shared memory");
 };
@@ -43,7 +44,7 @@ struct Dev {
   __nv_bfloat16* out;
   int* status;
   int64_t ldo;
-  int items, heads, kv_heads, rep, vdim, window, chunk, ksteps, bias_len, bias_pitch;
+  int items, heads, kv_heads, rep, vdim, window, chunk, bias_len, bias_pitch;
   int slabs, at_once, passes;   // slabs of one KV head's values (1, 2), KV heads of one item, items per (tile, head)
   int wide_store;               // output rows and heads start on 32 bytes
   float scale;
@@ -83,7 +84,7 @@ __device__ __forceinline__ bool next_work(const Dev& p, int& round, Work& w) {
     w.pos0 = b.z + half * 128;
     w.kv0 = b.w;
     w.k_lo = p.first_key(w.pos0);
-    w.n = (w.pos0 + w.rows - 1 - w.k_lo) / 128 + 1;
+    w.n = (w.pos0 + w.rows - 1 - w.k_lo) / kKeys + 1;
     ++round;
     return true;
   }
@@ -104,41 +105,39 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
   uint8_t* sK = sQ + QS * C::kQBytes;
   uint8_t* sV = sK + KS * C::kKBytes;
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + C::kTiles);
-  uint64_t *q_full = bars, *q_empty = bars + 2, *k_full = bars + 4, *k_empty = bars + 6, *v_full = bars + 8, *v_empty = bars + 12,
-           *s_full = bars + 16, *p_full = bars + 18, *b_full = bars + 20, *b_empty = bars + 22, *o_done = bars + 24, *o_free = bars + 26,
-           *chain = bars + 27 /* [2][4] */, *fin = bars + 35 /* [2][4] */;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 44);
+  uint64_t *q_full = bars, *q_empty = bars + 2, *b_full = bars + 4, *b_empty = bars + 6, *k_full = bars + 8, *k_empty = bars + 12,
+           *v_full = bars + 16, *v_empty = bars + 20, *s_full = bars + 24, *p_full = bars + 28, *o_done = bars + 32 /* one per score tile */,
+           *chain = bars + 36 /* [groups][4] */, *fin = bars + 52 /* [4] */, *o_free = bars + 56;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 57);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   float* s_m = reinterpret_cast<float*>(smem + C::kTiles + C::kBarriers);      // [128] row maximum that O is scaled by
-  float2* s_l = reinterpret_cast<float2*>(s_m + 128);                          // [2 items][2 groups][128] sum and its maximum
-  float* s_bias = reinterpret_cast<float*>(s_l + 2 * 2 * 128);                 // [2][kBiasTable]
+  float2* s_l = reinterpret_cast<float2*>(s_m + 128);                          // [groups][128] sum and its maximum
+  float* s_bias = reinterpret_cast<float*>(s_l + kGroups * 128);               // [2][kBiasTable]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
     for (int x = 0; x < 2; ++x) {
       mbar_init(&q_full[x], 1);
       mbar_init(&q_empty[x], 1);
+      mbar_init(&b_full[x], 1);
+      mbar_init(&b_empty[x], kGroups * 4);   // one arrival per softmax warp
+    }
+    for (int x = 0; x < 4; ++x) {
       mbar_init(&k_full[x], 1);
       mbar_init(&k_empty[x], 1);
       mbar_init(&s_full[x], 1);
       mbar_init(&p_full[x], 4);   // one arrival per softmax warp of the group
-      mbar_init(&b_full[x], 1);
-      mbar_init(&b_empty[x], 8);  // one arrival per softmax warp
-      mbar_init(&o_done[x], 1);   // of even and odd tiles: a wait must know that the phase before the one it waits for is over
-    }
-    for (int x = 0; x < 4; ++x) {
+      mbar_init(&o_done[x], 1);
       mbar_init(&v_full[x], 1);
       mbar_init(&v_empty[x], 1);
     }
-    for (int x = 0; x < 8; ++x) {
-      mbar_init(&chain[x], 1);
-      mbar_init(&fin[x], 1);
-    }
-    mbar_init(o_free, 8);
+    for (int x = 0; x < kGroups * 4; ++x) mbar_init(&chain[x], 1);
+    for (int x = 0; x < 4; ++x) mbar_init(&fin[x], kGroups);
+    mbar_init(o_free, kGroups * 4);
     *abort_flag = 0;
     fence_mbar_init();
   }
-  if (warp == 9) {
+  if (warp == kGroups * 4 + 1) {
     tmem_alloc(tmem_slot, 512);
     tmem_relinquish();
   }
@@ -147,123 +146,127 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
   tc_fence_after_sync();
   const uint32_t tmem_base = *tmem_slot;
 
-  if (warp >= 8) {
-    if (warp == 8 && lane == 0) {
+  if (warp >= kGroups * 4) {
+    if (warp == kGroups * 4) {
       // ---------------------------------------------------------------- TMA producer
-      int items = 0, nk = 0, nv = 0, round = 0;
-      const int v_bytes = p.at_once * p.slabs * kHalfSlab;
-      bool ok = true;
-      Work w;
-      auto wait = [&](uint64_t* bar, int parity) {
-        if (mbar_wait_bounded(bar, parity, abort_flag)) return true;
-        atomicCAS(p.status, 0, kStatusTimeoutProducer);
-        return false;
-      };
-      auto keys = [&](int j) {
-        const int s = nk % KS;
-        if (!wait(&k_empty[s], ((nk / KS) & 1) ^ 1)) return false;
-        ++nk;
-        mbar_arrive_expect_tx(&k_full[s], C::kKBytes);
+      if (lane == 0) {
+        int items = 0, nk = 0, nv = 0, round = 0;
+        const int v_bytes = p.at_once * p.slabs * kKeySlab;
+        bool ok = true;
+        Work w;
+        auto wait = [&](uint64_t* bar, int parity) {
+          if (mbar_wait_bounded(bar, parity, abort_flag)) return true;
+          atomicCAS(p.status, 0, kStatusTimeoutProducer);
+          return false;
+        };
+        auto keys = [&](int j) {
+          const int s = nk % KS;
+          if (!wait(&k_empty[s], ((nk / KS) & 1) ^ 1)) return false;
+          ++nk;
+          mbar_arrive_expect_tx(&k_full[s], C::kKBytes);
 #pragma unroll
-        for (int c = 0; c < ND; ++c)
-          tma_load_3d(sK + s * C::kKBytes + c * kSlab, &tm_k, &k_full[s], 64 * c, w.hk, w.kv0 + w.k_lo + j * 128);
-        return true;
-      };
-      for (; ok && next_work(p, round, w); ++items) {
-        const int qs = items % QS;
-        ok = wait(&q_empty[qs], ((items / QS) & 1) ^ 1);   // the Q K^T of the item that used it are done
-        if (!ok) break;
-        mbar_arrive_expect_tx(&q_full[qs], C::kQBytes);
-#pragma unroll
-        for (int c = 0; c < ND; ++c) tma_load_3d(sQ + qs * C::kQBytes + c * kSlab, &tm_q, &q_full[qs], 64 * c, w.h, w.row0);
-        if (p.bias != nullptr) {
-          const int b = items & 1;
-          ok = wait(&b_empty[b], ((items >> 1) & 1) ^ 1);
+          for (int c = 0; c < ND; ++c)
+            tma_load_3d(sK + s * C::kKBytes + c * kKeySlab, &tm_k, &k_full[s], 64 * c, w.hk, w.kv0 + w.k_lo + j * kKeys);
+          return true;
+        };
+        for (; ok && next_work(p, round, w); ++items) {
+          const int qs = items % QS;
+          ok = wait(&q_empty[qs], ((items / QS) & 1) ^ 1);   // the Q K^T of the item that used it are done
           if (!ok) break;
-          mbar_arrive_expect_tx(&b_full[b], p.bias_pitch * 4);
-          bulk_load(s_bias + b * kBiasTable, p.bias + static_cast<int64_t>(w.h) * p.bias_pitch, p.bias_pitch * 4, &b_full[b]);
-        }
-        ok = keys(0);
-        if (ok && w.n > 1) ok = keys(1);
-        for (int j = 0; ok && j < w.n; ++j) {
-          for (int half = 0; ok && half < 2; ++half, ++nv) {
+          mbar_arrive_expect_tx(&q_full[qs], C::kQBytes);
+#pragma unroll
+          for (int c = 0; c < ND; ++c) tma_load_3d(sQ + qs * C::kQBytes + c * kSlab, &tm_q, &q_full[qs], 64 * c, w.h, w.row0);
+          if (p.bias != nullptr) {
+            const int b = items & 1;
+            ok = wait(&b_empty[b], ((items >> 1) & 1) ^ 1);
+            if (!ok) break;
+            mbar_arrive_expect_tx(&b_full[b], p.bias_pitch * 4);
+            bulk_load(s_bias + b * kBiasTable, p.bias + static_cast<int64_t>(w.h) * p.bias_pitch, p.bias_pitch * 4, &b_full[b]);
+          }
+          for (int j = 0; ok && j < min(KS, w.n); ++j) ok = keys(j);
+          for (int j = 0; ok && j < w.n; ++j, ++nv) {
             const int s = nv % VS;
             ok = wait(&v_empty[s], ((nv / VS) & 1) ^ 1);
             if (!ok) break;
             mbar_arrive_expect_tx(&v_full[s], v_bytes);
             uint8_t* d = sV + s * C::kVBytes;                // one slab of every KV head, then their second slabs
-            const int row = w.kv0 + w.k_lo + j * 128 + half * 64;
+            const int row = w.kv0 + w.k_lo + j * kKeys;
             tma_load_3d(d, &tm_v, &v_full[s], 0, row, w.c0);
-            if (p.slabs > 1) tma_load_3d(d + p.at_once * kHalfSlab, &tm_v, &v_full[s], 64, row, w.c0);
+            if (p.slabs > 1) tma_load_3d(d + p.at_once * kKeySlab, &tm_v, &v_full[s], 64, row, w.c0);
+            if (j + KS < w.n) ok = keys(j + KS);
           }
-          if (ok && j + 2 < w.n) ok = keys(j + 2);
         }
       }
-    } else if (warp == 9) {
-      // ---------------------------------------------------------------- MMA issuer: the warp walks, one elected lane issues
-      const bool leader = elect_one();
-      const uint32_t idesc_s = make_idesc(kFmtBF16, kFmtBF16, false, false, 128, 128);
-      const uint32_t idesc_o = make_idesc(kFmtBF16, kFmtBF16, false, true, 128, p.at_once * p.slabs * 64);
-      const uint32_t tmem_o = tmem_base + 256;
-      int items = 0, t0 = 0, nv = 0, round = 0;
-      bool ok = true;
-      Work w{};
-      auto wait = [&](uint64_t* bar, int parity) {
-        if (__all_sync(0xffffffffu, mbar_wait_bounded(bar, parity, abort_flag))) return true;
-        if (leader) atomicCAS(p.status, 0, kStatusTimeoutMma);
-        return false;
-      };
-      auto scores = [&](int j) {             // S(j) = Q K(j)^T; the P of tile j - 2, in the same columns, has been issued to P V
-        const int t = t0 + j;
-        if (!wait(&k_full[t % KS], (t / KS) & 1)) return false;
-        tc_fence_after_sync();
-        if (leader) {
-          const uint64_t dQ = desc_kmajor(smem_u32(sQ + (items % QS) * C::kQBytes), 128, 0);
-          const uint64_t dK = desc_kmajor(smem_u32(sK + (t % KS) * C::kKBytes), 128, 0);
-          for (int ks = 0; ks < p.ksteps; ++ks)
-            umma_f16_ss(tmem_base + (t & 1) * 128, dQ + kstep_kmajor(128, ks), dK + kstep_kmajor(128, ks), idesc_s, ks > 0 ? 1u : 0u);
-          umma_commit(&s_full[t & 1]);
-          umma_commit(&k_empty[t % KS]);
-          if (j + 1 == w.n) umma_commit(&q_empty[items % QS]);
-        }
-        __syncwarp();
-        return true;
-      };
-      for (; ok && next_work(p, round, w); ++items) {
-        ok = wait(&q_full[items % QS], (items / QS) & 1);
-        if (ok) ok = scores(0);
-        if (ok && w.n > 1) ok = scores(1);
-        for (int j = 0; ok && j < w.n; ++j) {
-          const int t = t0 + j;
-          ok = wait(&p_full[t & 1], (t >> 1) & 1);
-          if (ok && j == 0 && items > 0) ok = wait(o_free, (items - 1) & 1);     // the rows of the previous item have been read
-          for (int half = 0; ok && half < 2; ++half, ++nv) {
-            const int s = nv % VS;
-            ok = wait(&v_full[s], (nv / VS) & 1);
-            if (!ok) break;
-            tc_fence_after_sync();
-            if (leader) {
-              const uint64_t dV = desc_mnmajor(smem_u32(sV + s * C::kVBytes), 64, 0);
-              const uint32_t pa = tmem_base + (t & 1) * 128 + half * 32;
+    } else {
+      // ---------------------------------------------------------------- MMA issuers: one lane each
+      if (elect_one()) {
+        int items = 0, round = 0;
+        uint32_t t = 0, ring = 0, ring_phase = 0;      // running number of the key tile; its stage of keys or values
+        bool ok = true;
+        Work w;
+        auto wait = [&](uint64_t* bar, uint32_t parity) {
+          if (mbar_try_wait(bar, parity) || mbar_wait_bounded(bar, parity, abort_flag)) return true;
+          atomicCAS(p.status, 0, kStatusTimeoutMma);
+          return false;
+        };
+        if (warp == kGroups * 4 + 1) {                 // S(t) = Q K(t)^T
+          constexpr uint32_t idesc = make_idesc(kFmtBF16, kFmtBF16, false, false, 128, kKeys);
+          const uint64_t dK0 = desc_kmajor(smem_u32(sK), kKeys, 0);
+          for (; ok && next_work(p, round, w); ++items) {
+            const uint64_t dQ = desc_kmajor(smem_u32(sQ + (items % QS) * C::kQBytes), 128, 0);
+            ok = wait(&q_full[items % QS], (items / QS) & 1);
+            for (int j = 0; ok && j < w.n; ++j, ++t) {
+              const uint32_t b = t % kTilesAhead;
+              ok = wait(&o_done[b], ((t / kTilesAhead) & 1) ^ 1) &&    // the weights in these columns have been used
+                   wait(&k_full[ring], ring_phase);
+              if (!ok) break;
+              tc_fence_after_sync();
+              const uint64_t dK = dK0 + ring * (C::kKBytes >> 4);
 #pragma unroll
-              for (int ks = 0; ks < 4; ++ks)
-                umma_f16_ts(tmem_o, pa + ks * 8, dV + kstep_mnmajor(ks), idesc_o, j > 0 || half > 0 || ks > 0 ? 1u : 0u);
-              umma_commit(&v_empty[s]);
-              if (half == 1) umma_commit(&o_done[t & 1]);
+              for (int ks = 0; ks < ND * 4; ++ks)      // columns past the head size are zeros
+                umma_f16_ss(tmem_base + b * kKeys, dQ + kstep_kmajor(128, ks), dK + kstep_kmajor(kKeys, ks), idesc, ks > 0 ? 1u : 0u);
+              umma_commit(&s_full[b]);
+              umma_commit(&k_empty[ring]);
+              if (j + 1 == w.n) umma_commit(&q_empty[items % QS]);
+              if (++ring == KS) {
+                ring = 0;
+                ring_phase ^= 1;
+              }
             }
-            __syncwarp();
           }
-          if (ok && j + 2 < w.n) ok = scores(j + 2);
+        } else {                                       // O (+)= P(t) V(t)
+          const uint32_t idesc = make_idesc(kFmtBF16, kFmtBF16, false, true, 128, p.at_once * p.slabs * 64);
+          const uint64_t dV0 = desc_mnmajor(smem_u32(sV), kKeys, 0);
+          for (; ok && next_work(p, round, w); ++items) {
+            for (int j = 0; ok && j < w.n; ++j, ++t) {
+              const uint32_t b = t % kTilesAhead;
+              ok = wait(&v_full[ring], ring_phase) &&
+                   (j > 0 || items == 0 || wait(o_free, (items - 1) & 1)) &&      // the rows of the previous item have been read
+                   wait(&p_full[b], (t / kTilesAhead) & 1);
+              if (!ok) break;
+              tc_fence_after_sync();
+              const uint64_t dV = dV0 + ring * (C::kVBytes >> 4);
+#pragma unroll
+              for (int ks = 0; ks < kKeys / 16; ++ks)
+                umma_f16_ts(tmem_base + 256, tmem_base + b * kKeys + ks * 8, dV + kstep_mnmajor(ks), idesc, j > 0 || ks > 0 ? 1u : 0u);
+              umma_commit(&o_done[b]);
+              umma_commit(&v_empty[ring]);
+              if (++ring == VS) {
+                ring = 0;
+                ring_phase ^= 1;
+              }
+            }
+          }
         }
-        t0 += w.n;
       }
+      __syncwarp();
     }
   } else {
     // ------------------------------------------------------------------ softmax + output rows
     const int x = warp >> 2, quad = warp & 3, r = quad * 32 + lane;    // group; row inside the tile == TMEM lane
     const uint32_t lane_addr = static_cast<uint32_t>(quad * 32) << 16;
-    const uint32_t tmem_s = tmem_base + x * 128 + lane_addr, tmem_o = tmem_base + 256 + lane_addr;
-    uint64_t *mine = chain + x * 4 + quad, *theirs = chain + (x ^ 1) * 4 + quad;
+    const uint32_t tmem_o = tmem_base + 256 + lane_addr;
+    uint64_t *mine = chain + x * 4 + quad, *theirs = chain + ((x + kGroups - 1) % kGroups) * 4 + quad;
     const float sc = p.scale * kLog2e;
     int items = 0, t0 = 0, round = 0;
     bool ok = true;
@@ -285,54 +288,42 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
         bias += pos;
       }
       float m_own = -INFINITY, l_run = 0.0f;
-      for (int j = (t0 ^ x) & 1; j < w.n; j += 2) {
-        const int t = t0 + j, k0 = w.k_lo + j * 128;
-        ok = wait(&s_full[x], (t >> 1) & 1);
+      for (int j = (x + kGroups - t0 % kGroups) % kGroups; j < w.n; j += kGroups) {
+        const int t = t0 + j, b = t % kTilesAhead, k0 = w.k_lo + j * kKeys;
+        const uint32_t tmem_s = tmem_base + b * kKeys + lane_addr;
+        ok = wait(&s_full[b], (t / kTilesAhead) & 1);
         if (!ok) break;
         tc_fence_after_sync();
-        // Two passes over the 128 columns, 64 at a time, each in a loop that is not unrolled: the code of a tile stays small enough not
-        // to push that of the other warps out of the instruction cache.  Scores in units of log2: mul * product + add; a tile that has
-        // masked columns, or biases of its own for every distance, is rewritten with both applied.
-        const bool near = bias != nullptr && w.pos0 - k0 - 127 < p.bias_len - 1;
-        const bool rewrite = near || k0 + 127 > w.pos0 || k0 < last_lo;
-        const float mul = rewrite ? 1.0f : sc, add = rewrite ? 0.0f : b_far;
-        const int clo = row_lo - k0, chi = pos - k0;       // column c is visible iff clo <= c <= chi
-        float m_tile = -INFINITY;
-#pragma unroll 1
-        for (int c0 = 0; c0 < 128; c0 += 64) {
-          uint32_t sv[2][32];
-          tmem_ld_32x32b_x32(tmem_s + c0, sv[0]);
-          tmem_ld_32x32b_x32(tmem_s + c0 + 32, sv[1]);
-          tmem_ld_wait();
-          if (rewrite) {
-            const float* b = bias - k0 - c0;
+        uint32_t sv[2][32];
+        tmem_ld_32x32b_x32(tmem_s, sv[0]);
+        tmem_ld_32x32b_x32(tmem_s + 32, sv[1]);
+        tmem_ld_wait();
+        // Scores in units of log2: mul * product + add; in a tile that has masked columns, or biases of its own for every distance, both
+        // are applied at once.
+        const bool near = bias != nullptr && w.pos0 - k0 - (kKeys - 1) < p.bias_len - 1;
+        const bool special = near || k0 + kKeys - 1 > w.pos0 || k0 < last_lo;
+        const float mul = special ? 1.0f : sc, add = special ? 0.0f : b_far;
+        if (special) {
+          const int clo = row_lo - k0, chi = pos - k0;       // column c is visible iff clo <= c <= chi
+          const float* at = bias - k0;
 #pragma unroll
-            for (int cc = 0; cc < 2; ++cc) {
-#pragma unroll
-              for (int c = 0; c < 32; ++c) {
-                const float v = fmaf(__uint_as_float(sv[cc][c]), sc, near ? b[-(cc * 32 + c)] : b_far);
-                sv[cc][c] = cc * 32 + c < clo - c0 || cc * 32 + c > chi - c0 ? 0xff800000u : __float_as_uint(v);  // -inf
-              }
-              tmem_st_32x32b_x32(tmem_s + c0 + cc * 32, sv[cc]);
-            }
+          for (int c = 0; c < kKeys; ++c) {
+            const float v = fmaf(__uint_as_float(sv[c >> 5][c & 31]), sc, near ? at[-c] : b_far);
+            sv[c >> 5][c & 31] = c < clo || c > chi ? 0xff800000u : __float_as_uint(v);  // -inf
           }
-          float m0 = m_tile, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;
-#pragma unroll
-          for (int cc = 0; cc < 2; ++cc)
-#pragma unroll
-            for (int c = 0; c < 32; c += 4) {
-              m0 = fmaxf(m0, __uint_as_float(sv[cc][c]));
-              m1 = fmaxf(m1, __uint_as_float(sv[cc][c + 1]));
-              m2 = fmaxf(m2, __uint_as_float(sv[cc][c + 2]));
-              m3 = fmaxf(m3, __uint_as_float(sv[cc][c + 3]));
-            }
-          m_tile = fmaxf(fmaxf(m0, m1), fmaxf(m2, m3));
         }
-        if (rewrite) tmem_st_wait();
-        m_tile = fmaf(m_tile, mul, add);
+        float m0 = -INFINITY, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;
+#pragma unroll
+        for (int c = 0; c < kKeys; c += 4) {
+          m0 = fmaxf(m0, __uint_as_float(sv[c >> 5][c & 31]));
+          m1 = fmaxf(m1, __uint_as_float(sv[c >> 5][(c & 31) + 1]));
+          m2 = fmaxf(m2, __uint_as_float(sv[c >> 5][(c & 31) + 2]));
+          m3 = fmaxf(m3, __uint_as_float(sv[c >> 5][(c & 31) + 3]));
+        }
+        const float m_tile = fmaf(fmaxf(fmaxf(m0, m1), fmaxf(m2, m3)), mul, add);
         // the maxima after tile j - 1, from the warp that has the same rows there
         if (t > 0) {
-          ok = wait(theirs, ((t - 1) >> 1) & 1);
+          ok = wait(theirs, ((t - 1) / kGroups) & 1);
           if (!ok) break;
         }
         const float m_prev = j > 0 ? s_m[r] : -INFINITY;
@@ -344,7 +335,7 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
         if (lane == 0) mbar_arrive(mine);
         if (j > 0 && __any_sync(0xffffffffu, grow)) {   // the output tile holds the sums of the earlier key tiles
           const float alpha = grow ? ex2f(m_prev - m_new) : 1.0f;
-          ok = wait(&o_done[x ^ 1], ((t - 1) >> 1) & 1);   // S(t) came after P(t - 2) V
+          ok = wait(&o_done[(t - 1) % kTilesAhead], ((t - 1) / kTilesAhead) & 1);   // S(t) came after P(t - 4) V, so this phase is next
           if (!ok) break;
           tc_fence_after_sync();
 #pragma unroll 1
@@ -364,57 +355,56 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
         }
         const float m_use = (m_ref == -INFINITY ? 0.0f : m_ref) - add;
         float r0 = 0.0f, r1 = 0.0f, r2 = 0.0f, r3 = 0.0f;
-#pragma unroll 1
-        for (int c0 = 0; c0 < 128; c0 += 64) {
-          uint32_t sv[2][32], pk[32];
-          tmem_ld_32x32b_x32(tmem_s + c0, sv[0]);
-          tmem_ld_32x32b_x32(tmem_s + c0 + 32, sv[1]);
-          tmem_ld_wait();
 #pragma unroll
-          for (int cc = 0; cc < 2; ++cc)
+        for (int cc = 0; cc < 2; ++cc) {
+          uint32_t pk[16];
 #pragma unroll
-            for (int g = 0; g < 4; ++g) {
-              float e[8];
+          for (int g = 0; g < 4; ++g) {
+            float e[8];
 #pragma unroll
-              for (int i = 0; i < 8; ++i) e[i] = ex2f(fmaf(__uint_as_float(sv[cc][8 * g + i]), mul, -m_use));  // -inf -> 0
-              r0 += e[0] + e[4];
-              r1 += e[1] + e[5];
-              r2 += e[2] + e[6];
-              r3 += e[3] + e[7];
-              pk[16 * cc + 4 * g + 0] = pack_bf16x2(e[0], e[1]);
-              pk[16 * cc + 4 * g + 1] = pack_bf16x2(e[2], e[3]);
-              pk[16 * cc + 4 * g + 2] = pack_bf16x2(e[4], e[5]);
-              pk[16 * cc + 4 * g + 3] = pack_bf16x2(e[6], e[7]);
-            }
-          tmem_st_32x32b_x32(tmem_s + c0 / 2, pk);  // two probabilities per column, over scores that have been read
+            for (int i = 0; i < 8; ++i) e[i] = ex2f(fmaf(__uint_as_float(sv[cc][8 * g + i]), mul, -m_use));  // -inf -> 0
+            r0 += e[0] + e[4];
+            r1 += e[1] + e[5];
+            r2 += e[2] + e[6];
+            r3 += e[3] + e[7];
+            pk[4 * g + 0] = pack_bf16x2(e[0], e[1]);
+            pk[4 * g + 1] = pack_bf16x2(e[2], e[3]);
+            pk[4 * g + 2] = pack_bf16x2(e[4], e[5]);
+            pk[4 * g + 3] = pack_bf16x2(e[6], e[7]);
+          }
+          tmem_st_32x32b_x16(tmem_s + cc * 16, pk);  // two probabilities per column
         }
         l_run += (r0 + r1) + (r2 + r3);
         tmem_st_wait();
         tc_fence_before_sync();
         __syncwarp();
-        if (lane == 0) mbar_arrive(&p_full[x]);
+        if (lane == 0) mbar_arrive(&p_full[b]);
       }
       if (!ok) break;
-      // both groups' sums, each relative to the maximum it last saw; not before all warps are done with the previous item's
+      // the groups' sums, each relative to the maximum it last saw; not before all warps are done with the previous item's
       if (items > 0) {
         ok = wait(o_free, (items - 1) & 1);
         if (!ok) break;
       }
-      float2* stats = s_l + (items & 1) * 256;
-      stats[x * 128 + r] = make_float2(l_run, m_own);
+      s_l[x * 128 + r] = make_float2(l_run, m_own);
       __syncwarp();
       if (lane == 0) {
         if (p.bias != nullptr) mbar_arrive(&b_empty[items & 1]);
-        mbar_arrive(fin + x * 4 + quad);
+        mbar_arrive(&fin[quad]);
       }
-      ok = wait(fin + (x ^ 1) * 4 + quad, items & 1);
+      ok = wait(&fin[quad], items & 1);
       if (!ok) break;
-      const float2 other = stats[(x ^ 1) * 128 + r];
-      const float m_end = fmaxf(m_own, other.y);
-      const float total = (m_own == -INFINITY ? 0.0f : l_run * ex2f(m_own - m_end)) +
-                          (other.y == -INFINITY ? 0.0f : other.x * ex2f(other.y - m_end));
+      float m_end = -INFINITY, total = 0.0f;
+#pragma unroll
+      for (int g = 0; g < kGroups; ++g) m_end = fmaxf(m_end, s_l[g * 128 + r].y);
+#pragma unroll
+      for (int g = 0; g < kGroups; ++g) {
+        const float2 part = s_l[g * 128 + r];
+        total += part.y == -INFINITY ? 0.0f : part.x * ex2f(part.y - m_end);
+      }
       const int t_last = t0 + w.n - 1;
-      ok = wait(&o_done[t_last & 1], (t_last >> 1) & 1);   // the last P V has retired; S(t_last), seen by now, came after P(t_last - 2) V
+      // the last P V has retired; S(t_last), which a group has seen, came after P(t_last - 4) V
+      ok = wait(&o_done[t_last % kTilesAhead], (t_last / kTilesAhead) & 1);
       if (!ok) break;
       tc_fence_after_sync();
       const bool row_ok = r < w.rows;
@@ -422,7 +412,7 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
       __nv_bfloat16* orow = p.out + static_cast<int64_t>(w.row0 + r) * p.ldo + (static_cast<int64_t>(w.h) * p.kv_heads + w.c0) * p.vdim;
       const int heads_here = min(p.at_once, p.kv_heads - w.c0);
 #pragma unroll 1
-      for (int cc = x; cc < p.at_once * p.slabs * 2; cc += 2) {      // 32 columns each, the groups in turn
+      for (int cc = x; cc < p.at_once * p.slabs * 2; cc += kGroups) {      // 32 columns each, the groups in turn
         const int s = cc >> 1, second = s >= p.at_once ? 1 : 0, c = s - second * p.at_once, d0 = second * 64 + (cc & 1) * 32;
         uint32_t ov[32];
         tmem_ld_32x32b_x32(tmem_o + cc * 32, ov);
@@ -455,15 +445,15 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
     while (globaltimer_ns() - t_end < 2000000ull) __nanosleep(2000);
     __syncthreads();
   }
-  if (warp == 9) {
+  if (warp == kGroups * 4 + 1) {
     tc_fence_after_sync();
     tmem_dealloc(tmem_base, 512);
   }
 }
 
-// Tensor map of [rows][heads][columns]: columns past a head's width and heads past the last arrive as zeros.  box_heads 0: box of 128
-// rows of one head, coordinates (column, head, row); else of box_heads slabs of 64 rows, coordinates (column, row, head).
-int head_map(CUtensorMap* m, const void* base, int cols, int heads, int rows, int64_t row_ld, int box_heads) {
+// Tensor map of [rows][heads][columns]: columns past a head's width and heads past the last arrive as zeros.  box_heads 0: box of
+// box_rows rows of one head, coordinates (column, head, row); else of box_heads slabs of box_rows rows, coordinates (column, row, head).
+int head_map(CUtensorMap* m, const void* base, int cols, int heads, int rows, int64_t row_ld, int box_rows, int box_heads) {
   nx::EncodeTiledFn fn = nx::encode_tiled_fn();
   if (fn == nullptr) return -3;
   const int head = box_heads > 0 ? 2 : 1, row = 3 - head;
@@ -474,7 +464,7 @@ int head_map(CUtensorMap* m, const void* base, int cols, int heads, int rows, in
   strides[head - 1] = static_cast<cuuint64_t>(cols) * 2;
   strides[row - 1] = static_cast<cuuint64_t>(row_ld) * 2;
   box[head] = static_cast<cuuint32_t>(std::max(1, box_heads));
-  box[row] = box_heads > 0 ? 64 : 128;
+  box[row] = static_cast<cuuint32_t>(box_rows);
   return fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, one, CU_TENSOR_MAP_INTERLEAVE_NONE,
             CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS
              ? 0
@@ -512,9 +502,9 @@ extern "C" int nx_talk_prompt(const NxTalkPromptArgs* a, nx_stream_t stream) {
   p.slabs = a->vdim <= 64 ? 1 : 2;
   p.at_once = std::min(kSlabs / p.slabs, a->kv_heads);
   p.passes = (a->kv_heads + p.at_once - 1) / p.at_once;
-  if ((rc = head_map(&q, a->q, a->dim, a->heads, a->q_rows, a->ldq, 0))) return rc;
-  if ((rc = head_map(&k, a->k, a->dim, a->kv_heads, a->kv_rows, a->ldk, 0))) return rc;
-  if ((rc = head_map(&v, a->v, a->vdim, a->kv_heads, a->kv_rows, a->ldv, p.at_once))) return rc;
+  if ((rc = head_map(&q, a->q, a->dim, a->heads, a->q_rows, a->ldq, 128, 0))) return rc;
+  if ((rc = head_map(&k, a->k, a->dim, a->kv_heads, a->kv_rows, a->ldk, kKeys, 0))) return rc;
+  if ((rc = head_map(&v, a->v, a->vdim, a->kv_heads, a->kv_rows, a->ldv, kKeys, p.at_once))) return rc;
   p.blocks = a->blocks;
   p.bias = a->bias;
   p.out = static_cast<__nv_bfloat16*>(a->out);
@@ -526,7 +516,6 @@ extern "C" int nx_talk_prompt(const NxTalkPromptArgs* a, nx_stream_t stream) {
   p.vdim = a->vdim;
   p.window = a->window;
   p.chunk = a->chunk;
-  p.ksteps = a->dim / 16;
   p.bias_len = a->bias_len;
   p.bias_pitch = a->bias_pitch;
   p.wide_store = (a->ldo % 16 == 0 && a->vdim % 16 == 0 && (reinterpret_cast<uintptr_t>(a->out) & 31) == 0) ? 1 : 0;
