@@ -49,6 +49,7 @@ def model_lines(sizes, iters=10):
 # ------------------------------------------------------------------------------------------ kernels
 def kernel_cases():
     """name -> (launch, flops, bytes)."""
+    from ..infer.prompt import row_slices
     from ..ops import _cuda as K
     from ..ops import _mixers as M
     dev, bf, f32 = "cuda", torch.bfloat16, torch.float32
@@ -90,7 +91,7 @@ def kernel_cases():
         kc, vc = rn(B * 1024 // bs, bs, G, D), rn(B * 1024 // bs, bs, G, D)
         table = torch.randperm(B * 1024 // bs, generator=torch.Generator().manual_seed(1)).view(B, -1).to(torch.int32).to(dev)
         q0, k0, v0, g0 = 0, H * D, (H + G) * D, (H + 2 * G) * D
-        proj, gate = rn(N, g0 + H), torch.rand((N, H), device=dev)
+        proj, gate = rn(N, g0 + 64), torch.rand((N, H), device=dev)
         wq, wk = torch.ones(H * D, device=dev), torch.ones(G * D, device=dev)
         prep = dict(heads=H, kv_heads=G, dim=D, vdim=D, norm_dim=D, norm_vdim=D, eps=1e-5, w_q=wq, w_k=wk, positions=pos, slots=slot,
                     k_cache=kc, v_cache=vc, q_scale=D ** -0.5, store_kv=True)
@@ -108,16 +109,18 @@ def kernel_cases():
                 n * (H * D // 2 * 4 + G * D * 2 * 4 + G * D // 2 * 2))
         rel, talk = rn(H, 129, dtype=f32), torch.eye(H, device=dev) * 0.8 + rn(H, H, dtype=f32, s=0.1)
         ext = M.extended_bias(rel)
-        q, k, v = proj[:, : H * D], proj[:, k0: v0], proj[:, v0: g0]
+        qkv = rn(N, g0 + 64)
+        qkv[:, : H * D] *= D ** -0.5            # as normed queries that carry the scale of the scores
+        q, k, v = qkv[:, : H * D], qkv[:, k0: v0], qkv[:, v0: g0]
         out, wide = rn(N, H * D), rn(N, H * G * D)
         kw = dict(heads=H, kv_heads=G, dim=D, vdim=D, scale=1.0)
         for count, length in ((8, 1024), (2, 4096)):
             bl, p = blocks(count, length, 0), pairs(count, length)
             mixing = 2.0 * H * H * p
+            slices = [(torch.tensor(g, dtype=torch.int32, device=dev), r, n) for g, r, n in row_slices(bl.tolist(), M.talk_rows(H, G, D))]
             cases[f"prompt attention, heads that mix, {count} x {length}, {sizes}"] = (
-                lambda bl=bl, q=q, k=k, v=v, wide=wide, out=out, ext=ext, talk=talk, gate=gate, kw=kw, H=H, G=G, D=D: (
-                    M.talk_prompt(q, k, v, wide, bl, window=0, bias=ext, distances=129, **kw),
-                    M.head_mix(wide, talk, gate, out, heads=H, kv_heads=G, vdim=D)), 4.0 * D * H * p + mixing, 0)
+                lambda slices=slices, q=q, k=k, v=v, out=out, ext=ext, talk=talk, gate=gate, kw=kw: M.talk_prompt_mixed(
+                    q, k, v, out, slices, talk, gate, window=0, bias=ext, distances=129, **kw), 4.0 * D * H * p + mixing, 0)
             cases[f"prompt attention with distance biases, {count} x {length}, {sizes}"] = (
                 lambda bl=bl, q=q, k=k, v=v, out=out, rel=rel, kw=kw: M.window_prompt(q, k, v, out, bl, window=0, bias=rel, **kw),
                 4.0 * D * H * p, 0)

@@ -85,6 +85,7 @@ class HybridEngine(Engine):
         self._prompt_windows = {prompt.Window(m.window) for m in mixers if isinstance(m, LatentSpec) and latent.expandable(m)} | {
             conv_attention.window(m) for m in mixers if isinstance(m, ConvAttentionSpec) and conv_attention.promptable(m)} | {
             normed_attention.window(m) for m in mixers if isinstance(m, NormedAttentionSpec) and normed_attention.promptable(m)}
+        self._prompt_slices = normed_attention.slices(mixers)
 
     def _rope_tables(self, dims: int, base: float, scaling: Optional[RopeScaling] = None):
         """cos / sin [ctx, dims / 2]: angles in double, kept in FP32."""
@@ -260,7 +261,7 @@ class HybridEngine(Engine):
         self._stepped = M.Segments(table, 0, single.count + short.count, max(single.max_len, short.max_len),
                                    single.total + short.total)
         self._every = M.Segments(table, 0, first, max(g.max_len for g in groups), sum(g.total for g in groups))
-        prompt.plan(self, self._prompt_windows)
+        prompt.plan(self, self._prompt_windows, self._prompt_slices)
         return self._body(dv[0], dv[1], dv[2], dv[3], dv[4], dv[5][:logit_rows], runs, nl)
 
     def _buffer(self, rows: int, cols: int) -> torch.Tensor:

@@ -49,6 +49,7 @@ def load(engine, m: NormedAttentionSpec, get) -> dict:
         return torch.cat([_pad_heads(get(n + suffix), heads, size) for n, heads, size in parts], 0)
     out = {"shape": s}
     w = torch.cat([stack("")] + ([get("g").float()] if m.gate else []), 0)
+    w = torch.nn.functional.pad(w, (0, 0, 0, -w.shape[0] % 64))      # rows of the projection start on 128 bytes, as the tiles read from them
     out["in"], _ = engine._pack([w], bias=stack(".b") if m.bias else None)
     wo = torch.zeros((engine.d, m.heads, s.vdim))
     wo[:, :, : m.vdim] = get("o").float().view(engine.d, m.heads, m.vdim)
@@ -85,6 +86,17 @@ def promptable(m: NormedAttentionSpec) -> bool:
     return s.dim <= 128 and s.vdim <= 128 and m.softcap == 0 and (m.distance is None or m.distance.far < M.PROMPT_MAX_BIAS)
 
 
+def slices(mixers) -> dict:
+    """The most rows that layers of heads that mix take at once, by window."""
+    from ..ops import _mixers as M
+    out: dict = {}
+    for m in mixers:
+        if isinstance(m, NormedAttentionSpec) and m.talk and promptable(m):
+            rows = M.talk_rows(m.heads, m.kv_heads, NormedAttentionShape(m).vdim)
+            out[window(m)] = min(rows, out.get(window(m), rows))
+    return out
+
+
 def mixer(engine, i: int, m: NormedAttentionSpec, lw: dict, h, pos, slot):
     from ..ops import _mixers as M
     s, n = lw["shape"], h.shape[0]
@@ -114,15 +126,14 @@ def mixer(engine, i: int, m: NormedAttentionSpec, lw: dict, h, pos, slot):
             M.latent_gather(c, engine.block_table, step.runs[w], step.longest[w], dst)
         return k, v
     if m.talk:
-        if not engine.fast or long_.count:
+        if step is not None:
+            M.talk_prompt_mixed(q, *keys_of_step(), out, step.slices[window(m)], lw["talk"], gate, dim=s.dim, window=m.window, chunk=m.chunk,
+                                scale=1.0, bias=lw["bias_wide"], distances=lw["bias"].shape[1] if lw["bias"] is not None else 0, **sizes)
+        elif not engine.fast or long_.count:
             wide = torch.empty((n, m.heads * m.kv_heads * s.vdim), dtype=engine.adt, device=engine.dev)
-            if step is not None:
-                M.talk_prompt(q, *keys_of_step(), wide, step.blocks[window(m)], dim=s.dim, window=m.window, chunk=m.chunk, scale=1.0,
-                              bias=lw["bias_wide"], distances=lw["bias"].shape[1] if lw["bias"] is not None else 0, **sizes)
-            else:
-                M.paged_window_attention(q, *paged, wide, long_ if engine.fast else engine._every, all_values=True, **kw)
+            M.paged_window_attention(q, *paged, wide, long_ if engine.fast else engine._every, all_values=True, **kw)
             M.head_mix(wide, lw["talk"], gate, out, **sizes)
-        for seg in (single, short) if engine.fast else ():       # after the mixture, which ran over all rows
+        for seg in (single, short) if engine.fast else ():       # after the mixture, which wrote rows between the long segments
             if seg.count:
                 M.talk_paged(q, *paged, out, lw["talk"], seg, keys=engine._most_keys(m), splits=engine._decode_splits(m, seg.count),
                              gate=gate, **kw)

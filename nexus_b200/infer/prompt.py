@@ -59,11 +59,30 @@ def long_segments(segs, window: int, keep_first: int = 0, chunk: int = 0):
     return [b[1:] for b in blocks], runs, d
 
 
+def row_slices(blocks, most: int):
+    """Blocks (first row, rows, ..; the most keys first) in groups of up to ``most`` consecutive rows, each in the order given: (blocks, first row,
+    rows of the group).  A block is never cut."""
+    out, group, first, end = [], [], 0, 0
+    for i in sorted(range(len(blocks)), key=lambda i: blocks[i][0]):
+        row, rows = blocks[i][:2]
+        if group and row + rows - first > most:
+            out.append((group, first, end - first))
+            group = []
+        if not group:
+            first = row
+        group.append(i)
+        end = row + rows
+    if group:
+        out.append((group, first, end - first))
+    return [([blocks[i] for i in sorted(g)], row, rows) for g, row, rows in out]
+
+
 class StepPlan:
     """How the segments of a step that has long ones are split; ``rows``: the rows of the one-token and short segments,
-    ``groups`` these segments over the compacted rows; per window the blocks and runs of the long ones (`long_segments`)."""
+    ``groups`` these segments over the compacted rows; per window the blocks and runs of the long ones (`long_segments`).  ``sliced``:
+    windows whose blocks are wanted in groups of consecutive rows too, and the most rows of a group (`row_slices`)."""
 
-    def __init__(self, engine, windows):
+    def __init__(self, engine, windows, sliced):
         from ..ops import _mixers as M
         single, short, long_ = engine._groups
         host, n = engine._host_rows[engine.INDEX_ROWS:], single.count + short.count
@@ -81,13 +100,17 @@ class StepPlan:
             first += count
         put("rows", [r for row0, count, _, _ in segs[:n] for r in range(row0, row0 + count)])
         put("table", [v for t in table for v in t])
-        self.kv_rows, self.longest = {}, {}
+        self.kv_rows, self.longest, self.slices = {}, {}, {}
         for w in windows:
             blocks, runs, self.kv_rows[w] = long_segments(segs[n:], *w)
             self.longest[w] = max((r[1] for r in runs), default=0)
             put(("blocks", w), [v for b in blocks for v in b[:4]])
             put(("kept", w), [b[4] for b in blocks])
             put(("runs", w), [v for r in runs for v in r])
+            groups = row_slices(blocks, sliced[w]) if w in sliced else []
+            self.slices[w] = [(("slice", w, i), row, rows) for i, (_, row, rows) in enumerate(groups)]
+            for i, (part, _, _) in enumerate(groups):
+                put(("slice", w, i), [v for b in part for v in b[:4]])
         self.gathered = any(self.kv_rows.values())
         dev = torch.tensor(data, dtype=torch.int32).pin_memory().to(engine.dev, non_blocking=True)
 
@@ -96,6 +119,7 @@ class StepPlan:
         self.blocks = {w: get(("blocks", w)).view(-1, 4) for w in windows}
         self.kept = {w: get(("kept", w)) for w in windows}
         self.runs = {w: get(("runs", w)).view(-1, 4) for w in windows}
+        self.slices = {w: [(get(name).view(-1, 4), row, rows) for name, row, rows in s] for w, s in self.slices.items()}
         self.rows = get("rows").long() if n else None
         if n:
             t = get("table").view(4, n)
@@ -103,8 +127,8 @@ class StepPlan:
                            M.Segments(t, single.count, short.count, short.max_len, short.total)]
 
 
-def plan(engine, windows) -> None:
+def plan(engine, windows, sliced=None) -> None:
     """Called once per step, before the layers; ``windows``: those of the layers that a prompt kernel can take."""
     engine._prompt_plan = None
     if engine.fast and engine._groups[2].count > 0 and windows:
-        engine._prompt_plan = StepPlan(engine, sorted(windows))
+        engine._prompt_plan = StepPlan(engine, sorted(windows), sliced or {})

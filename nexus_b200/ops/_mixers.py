@@ -158,6 +158,7 @@ LATENT_MAX_RANK, LATENT_MAX_ROW = 512, 768
 PROMPT_MAX_BIAS = 3072       # distances of a bias table of the tcgen05 prompt kernels
 TALK_MAX_HEADS = 96          # heads that mix their weights
 TALK_SCRATCH = 1 << 29       # bytes of scores and weights of one launch of such heads
+TALK_WIDE = 1 << 29          # bytes of every head's outputs with the values of every KV head that wait for their mixture at a time
 BIAS_MARGIN = 256            # entries of an extended bias table on either side of its distances
 
 
@@ -479,13 +480,30 @@ def extended_bias(bias: torch.Tensor) -> torch.Tensor:
     return (bias.double() * math.log2(math.e)).float()[:, at].contiguous()
 
 
-def talk_prompt(q, k, v, out, blocks, *, heads, kv_heads, dim, vdim, window, scale, chunk=0, bias=None, distances=0) -> None:
+def talk_prompt(q, k, v, out, blocks, *, heads, kv_heads, dim, vdim, window, scale, chunk=0, bias=None, distances=0, row0=0) -> None:
     """`window_prompt` for heads that mix: every head's weights with the values of every KV head, out [rows, heads * kv_heads * vdim].
-    ``bias``: `extended_bias` of ``distances`` distances."""
-    a = TalkPromptArgs(_ptr(q), _ptr(k), _ptr(v), _ptr(out), _ptr(bias), _ptr(blocks), K.status_word(q.device).data_ptr(), q.stride(0),
+    ``bias``: `extended_bias` of ``distances`` distances; ``row0``: the query row that the first row of ``out`` belongs to."""
+    first = out.data_ptr() - row0 * out.stride(0) * out.element_size()
+    a = TalkPromptArgs(_ptr(q), _ptr(k), _ptr(v), first, _ptr(bias), _ptr(blocks), K.status_word(q.device).data_ptr(), q.stride(0),
                        k.stride(0), v.stride(0), out.stride(0), blocks.shape[0], q.shape[0], k.shape[0], heads, kv_heads, dim, vdim,
                        window, chunk, distances, bias.shape[1] if bias is not None else 0, scale)
     K._check(K.lib().nx_talk_prompt(C.byref(a), K._stream()), "nx_talk_prompt")
+
+
+def talk_prompt_mixed(q, k, v, out, slices, talk, gate, *, heads, kv_heads, dim, vdim, **kw) -> None:
+    """`talk_prompt` and the mixture of its outputs (`head_mix`), slice by slice; slices: (blocks, first row, rows), the rows of one slice
+    at most ``talk_rows``.  Rows of ``out`` that lie in a slice and in none of its blocks get no defined values."""
+    cols = heads * kv_heads * vdim
+    wide = K.scratch(max((n for _, _, n in slices), default=0) * cols * q.element_size(), "talk_wide", q.device).view(q.dtype)
+    for blocks, row0, n in slices:
+        part = wide[: n * cols].view(n, cols)
+        talk_prompt(q, k, v, part, blocks, heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, row0=row0, **kw)
+        head_mix(part, talk, None if gate is None else gate[row0: row0 + n], out[row0: row0 + n], heads=heads, kv_heads=kv_heads, vdim=vdim)
+
+
+def talk_rows(heads: int, kv_heads: int, vdim: int) -> int:
+    """Rows of a slice of `talk_prompt_mixed`."""
+    return max(256, TALK_WIDE // (heads * kv_heads * vdim * 2))
 
 
 def latent_gather(cache, block_table, runs, longest, dst) -> None:

@@ -344,6 +344,13 @@ def test_prompts(heads, kv, dim, vdim, window, chunk, bias_len):
         M.talk_prompt(c.qd, k, v, wide, blocks, bias=ext, distances=bias_len, **kw)
         K.check_status()
         assert _rows_err(wide, c.want_all(window, chunk)) < 1.5e-2
+        # the mixture, in slices of two or three blocks
+        from nexus_b200.infer.prompt import row_slices
+        talk = 0.5 * torch.eye(heads) + _rand((heads, heads), 4, s=0.5)
+        slices = [(torch.tensor(b, dtype=torch.int32, device=DEV), r, n) for b, r, n in row_slices(blocks.tolist(), 300)]
+        assert len(slices) > 1
+        M.talk_prompt_mixed(c.qd, k, v, out, slices, talk.to(DEV), gate.to(DEV), bias=ext, distances=bias_len, **kw)
+        assert _rows_err(out, c.want(window, chunk, talk, gate)) < 4e-2
         again = torch.empty_like(wide)
         for _ in range(5):
             M.talk_prompt(c.qd, k, v, again, blocks, bias=ext, distances=bias_len, **kw)

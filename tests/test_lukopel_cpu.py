@@ -129,6 +129,20 @@ def test_long_segments_in_chunks(chunk):
         assert rows == {r for r0, n, _, _ in segs for r in range(r0, r0 + n)}
 
 
+@pytest.mark.parametrize("most", [256, 300, 1000, 10 ** 6])
+def test_slices_of_rows(most):
+    from nexus_b200.infer.prompt import long_segments, row_slices
+    blocks, _, _ = long_segments([(5, 17, 900, 2), (22, 256, 0, 0), (300, 700, 31, 1), (1000, 20, 4000, 3)], 0, 0, 0)
+    got = row_slices(blocks, most)
+    assert sorted(b for part, _, _ in got for b in part) == sorted(blocks)
+    last = 0
+    for part, row, rows in got:
+        assert row >= last and rows <= max(most, 256)
+        assert min(b[0] for b in part) == row and max(b[0] + b[1] for b in part) == row + rows
+        assert [blocks.index(b) for b in part] == sorted(blocks.index(b) for b in part)
+        last = row + rows
+
+
 def _moved(cfg, w, length, j):
     """Whether the last position's logits depend on token j."""
     toks = torch.randint(0, cfg["vocab"], (length,), generator=torch.Generator().manual_seed(0)).tolist()
