@@ -12,25 +12,30 @@ using namespace nx;
 // ------------------------------------------------------------------------------------------------
 // norms of queries, keys and values, the query's factors, cache append, gate: one block per row
 // ------------------------------------------------------------------------------------------------
+// `group`: lanes that share a head in the sums
 template <typename T, int V>
-__global__ void head_prep_kernel(const NxHeadPrepArgs a) {
+__global__ void __launch_bounds__(256) head_prep_kernel(const NxHeadPrepArgs a, int group) {
   extern __shared__ __align__(16) float s_inv[];       // [heads + 2 kv_heads]: factor of every head of q, k and v
   const int64_t r = blockIdx.x;
   T* row = static_cast<T*>(a.proj) + r * a.ld;
   const int H = a.heads, G = a.kv_heads, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
   const int normed = H + G, all = normed + (a.unit_values ? G : 0);
-  for (int u = warp; u < all; u += warps) {             // sums of squares, a warp per head; padding columns are zeros
-    const T* p = row + (u < H ? a.q_off + u * a.dim : u < normed ? a.k_off + (u - H) * a.dim : a.v_off + (u - normed) * a.vdim);
-    const int size = u < normed ? a.dim : a.vdim;
+  const int per_warp = 32 / group, in_group = lane % group;
+  for (int u0 = warp * per_warp; u0 < all; u0 += warps * per_warp) {   // sums of squares; padding columns are zeros
+    const int u = u0 + lane / group;
     float ss = 0.0f;
-    for (int c = lane * V; c < size; c += 32 * V) {
-      float v[V];
-      load_vec<T, V>(p + c, v);
+    if (u < all) {
+      const T* p = row + (u < H ? a.q_off + u * a.dim : u < normed ? a.k_off + (u - H) * a.dim : a.v_off + (u - normed) * a.vdim);
+      const int size = u < normed ? a.dim : a.vdim;
+      for (int c = in_group * V; c < size; c += group * V) {
+        float v[V];
+        load_vec<T, V>(p + c, v);
 #pragma unroll
-      for (int j = 0; j < V; ++j) ss += v[j] * v[j];
+        for (int j = 0; j < V; ++j) ss += v[j] * v[j];
+      }
     }
-    ss = warp_sum(ss);
-    if (lane == 0) s_inv[u] = ss;
+    for (int o = group / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (in_group == 0 && u < all) s_inv[u] = ss;
   }
   __syncthreads();
   float temp = 1.0f;
@@ -161,17 +166,20 @@ extern "C" int nx_head_prep(const NxHeadPrepArgs* a, nx_stream_t stream) {
   if (a->rows <= 0) return 0;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-  const bool vec = ((a->dim | a->vdim | a->q_off | a->k_off | a->v_off | static_cast<int>(a->ld)) & 3) == 0 && al(a->proj) &&
+  const int v16 = a->dtype == NX_BF16 ? 8 : 4;
+  const bool vec = ((a->dim | a->vdim | a->q_off | a->k_off | a->v_off | static_cast<int>(a->ld)) & (v16 - 1)) == 0 && al(a->proj) &&
                    al(a->w_q) && al(a->w_k) && al(a->k_cache) && al(a->v_cache);
-  const int chunks = (a->heads * a->dim + a->kv_heads * (a->dim + a->vdim)) / 4;
+  const int chunks = (a->heads * a->dim + a->kv_heads * (a->dim + a->vdim)) / (vec ? v16 : 1);
   const int threads = std::max(64, std::min(256, (chunks / 2 + 31) / 32 * 32));
   const size_t smem = static_cast<size_t>(a->heads + 2 * a->kv_heads) * sizeof(float);
+  int group = 32;
+  while (group > 1 && group / 2 * (vec ? v16 : 1) >= std::max(a->dim, a->vdim)) group /= 2;
   if (a->dtype == NX_BF16) {
-    if (vec) head_prep_kernel<__nv_bfloat16, 4><<<a->rows, threads, smem, st>>>(*a);
-    else head_prep_kernel<__nv_bfloat16, 1><<<a->rows, threads, smem, st>>>(*a);
+    if (vec) head_prep_kernel<__nv_bfloat16, 8><<<a->rows, threads, smem, st>>>(*a, group);
+    else head_prep_kernel<__nv_bfloat16, 1><<<a->rows, threads, smem, st>>>(*a, group);
   } else if (a->dtype == NX_F32) {
-    if (vec) head_prep_kernel<float, 4><<<a->rows, threads, smem, st>>>(*a);
-    else head_prep_kernel<float, 1><<<a->rows, threads, smem, st>>>(*a);
+    if (vec) head_prep_kernel<float, 4><<<a->rows, threads, smem, st>>>(*a, group);
+    else head_prep_kernel<float, 1><<<a->rows, threads, smem, st>>>(*a, group);
   } else {
     return -1;
   }
@@ -195,7 +203,7 @@ extern "C" int nx_head_mix(const void* wide, int64_t ldw, const float* talk, con
   const int smem = kv_heads * groups * n * heads * static_cast<int>(sizeof(float));
 #define NX_HM(T_, V_, N_)                                                                                                       \
   do {                                                                                                                          \
-    if (smem > 48 * 1024 &&                                                                                                     \
+    if (smem > 40 * 1024 &&                                                                                                     \
         cudaFuncSetAttribute(head_mix_kernel<T_, V_, N_>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)    \
       return -2;                                                                                                                \
     head_mix_kernel<T_, V_, N_><<<blocks, threads, smem, st>>>((const T_*)wide, ldw, talk, gate, (T_*)out, ldo, rows, heads,    \

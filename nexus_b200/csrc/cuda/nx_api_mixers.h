@@ -75,7 +75,7 @@ typedef struct NxStreamResidualArgs {
   const float* w_next;     // [cols]
   void* h;                 // [rows, ldh], may be null; columns cols..ldh are zeroed
   int64_t ldy, ldh;
-  int32_t rows, cols, streams, dtype;   // up to 8 streams of up to 12288 columns
+  int32_t rows, cols, streams, dtype;   // up to 8 streams of up to 49152 columns
   float eps, embed_scale;
 } NxStreamResidualArgs;
 int nx_stream_residual(const NxStreamResidualArgs* args, nx_stream_t stream);

@@ -392,7 +392,7 @@ __global__ void talk_sum_kernel(const NxPagedWindowArgs a, int tq) {
 
 template <typename Kernel>
 int launch(Kernel kernel, const NxTalkPagedArgs* t, dim3 grid, int smem, int rt, int tq, int head_tiles, cudaStream_t st) {
-  if (smem > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -2;
+  if (smem > 40 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -2;
   kernel<<<grid, kThreads, smem, st>>>(*t, rt, tq, head_tiles);
   return launch_status();
 }
@@ -414,7 +414,7 @@ int launch_all(const NxTalkPagedArgs* t, int rt, int tq, cudaStream_t st) {
                           : launch_scores<256, MT>(t, grid, rt, tq, head_tiles, st);
   if (rc) return rc;
   const int smem = a.heads * (((a.heads + 3) & ~3) + kKeys + 1) * static_cast<int>(sizeof(float));
-  if (smem > 48 * 1024 &&
+  if (smem > 40 * 1024 &&
       cudaFuncSetAttribute(talk_mix_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
     return -2;
   const int strides = static_cast<int>(std::max<int64_t>(1, std::min<int64_t>(t->pitch / kKeys, 4736 / std::max(1, t->rows))));

@@ -10,9 +10,11 @@
 namespace {
 using namespace nx;
 
+constexpr int kMaxThreads = 256;
+
 // S: streams the registers hold (a.streams <= S)
 template <typename T, int V, int S>
-__global__ void stream_residual_kernel(const NxStreamResidualArgs a) {
+__global__ void __launch_bounds__(kMaxThreads) stream_residual_kernel(const NxStreamResidualArgs a) {
   extern __shared__ __align__(16) float s_u[];          // [cols]: the weighted sum of the streams
   __shared__ float s_red[32], s_mix[S * S], s_out[S], s_in[S];
   const int64_t r = blockIdx.x;
@@ -113,19 +115,24 @@ __global__ void stream_residual_kernel(const NxStreamResidualArgs a) {
 
 template <typename T, int V>
 int launch(const NxStreamResidualArgs* a, cudaStream_t st) {
-  const int threads = std::max(64, std::min(512, (a->cols / V + 31) / 32 * 32));
+  const int threads = std::max(64, std::min(kMaxThreads, (a->cols / V + 31) / 32 * 32));
   const size_t smem = static_cast<size_t>(a->cols) * sizeof(float);
-  if (a->streams <= 2) stream_residual_kernel<T, V, 2><<<a->rows, threads, smem, st>>>(*a);
-  else if (a->streams <= 3) stream_residual_kernel<T, V, 3><<<a->rows, threads, smem, st>>>(*a);
-  else if (a->streams <= 4) stream_residual_kernel<T, V, 4><<<a->rows, threads, smem, st>>>(*a);
-  else stream_residual_kernel<T, V, 8><<<a->rows, threads, smem, st>>>(*a);
-  return launch_status();
+  const auto run = [&](auto kernel) {
+    if (smem > 40 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess)
+      return -2;
+    kernel<<<a->rows, threads, smem, st>>>(*a);
+    return launch_status();
+  };
+  if (a->streams <= 2) return run(stream_residual_kernel<T, V, 2>);
+  if (a->streams <= 3) return run(stream_residual_kernel<T, V, 3>);
+  if (a->streams <= 4) return run(stream_residual_kernel<T, V, 4>);
+  return run(stream_residual_kernel<T, V, 8>);
 }
 
 }  // namespace
 
 extern "C" int nx_stream_residual(const NxStreamResidualArgs* a, nx_stream_t stream) {
-  if (a == nullptr || a->x == nullptr || a->cols <= 0 || a->cols > 12288 || a->streams < 1 || a->streams > 8) return -1;
+  if (a == nullptr || a->x == nullptr || a->cols <= 0 || a->cols > 49152 || a->streams < 1 || a->streams > 8) return -1;
   if (a->table != nullptr && (a->tokens == nullptr || (a->pos_table != nullptr && a->positions == nullptr))) return -1;
   if (a->table == nullptr && a->y != nullptr && (a->mix == nullptr || a->out == nullptr || a->ldy < a->cols)) return -1;
   if (a->h != nullptr && (a->w_next == nullptr || a->ldh < a->cols)) return -1;

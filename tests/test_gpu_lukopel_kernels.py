@@ -39,7 +39,7 @@ def _segs(parts, max_len=0):
 
 # ---------------------------------------------------------------------------------------------- residual
 @pytest.mark.parametrize("dt,tol", DTYPES)
-@pytest.mark.parametrize("streams,cols", [(1, 96), (2, 50), (3, 2048), (4, 88), (5, 40), (8, 24)])
+@pytest.mark.parametrize("streams,cols", [(1, 96), (2, 50), (3, 2048), (4, 88), (5, 40), (8, 24), (7, 4096), (2, 12288), (1, 20480), (4, 3001)])
 def test_residual_streams(dt, tol, streams, cols):
     M = _m()
     n, V, P, ld, eps = 7, 30, 40, (cols + 7) // 8 * 8, 1e-3
