@@ -301,16 +301,21 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
         // Scores in units of log2: mul * product + add; in a tile that has masked columns, or biases of its own for every distance, both
         // are applied at once.
         const bool near = bias != nullptr && w.pos0 - k0 - (kKeys - 1) < p.bias_len - 1;
-        const bool special = near || k0 + kKeys - 1 > w.pos0 || k0 < last_lo;
+        const bool masked = k0 + kKeys - 1 > w.pos0 || k0 < last_lo, special = near || masked;
         const float mul = special ? 1.0f : sc, add = special ? 0.0f : b_far;
-        if (special) {
-          const int clo = row_lo - k0, chi = pos - k0;       // column c is visible iff clo <= c <= chi
+        if (near) {
           const float* at = bias - k0;
 #pragma unroll
-          for (int c = 0; c < kKeys; ++c) {
-            const float v = fmaf(__uint_as_float(sv[c >> 5][c & 31]), sc, near ? at[-c] : b_far);
-            sv[c >> 5][c & 31] = c < clo || c > chi ? 0xff800000u : __float_as_uint(v);  // -inf
-          }
+          for (int c = 0; c < kKeys; ++c) sv[c >> 5][c & 31] = __float_as_uint(fmaf(__uint_as_float(sv[c >> 5][c & 31]), sc, at[-c]));
+        } else if (special) {
+#pragma unroll
+          for (int c = 0; c < kKeys; ++c) sv[c >> 5][c & 31] = __float_as_uint(fmaf(__uint_as_float(sv[c >> 5][c & 31]), sc, b_far));
+        }
+        if (masked) {
+          const int clo = row_lo - k0, chi = pos - k0;       // column c is visible iff clo <= c <= chi
+#pragma unroll
+          for (int c = 0; c < kKeys; ++c)
+            if (c < clo || c > chi) sv[c >> 5][c & 31] = 0xff800000u;  // -inf
         }
         float m0 = -INFINITY, m1 = -INFINITY, m2 = -INFINITY, m3 = -INFINITY;
 #pragma unroll
@@ -417,19 +422,21 @@ talk_prompt_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
         uint32_t ov[32];
         tmem_ld_32x32b_x32(tmem_o + cc * 32, ov);
         tmem_ld_wait();
-        if (!row_ok || c >= heads_here || d0 >= p.vdim) continue;
-        uint32_t pk[16];
+        if (row_ok && c < heads_here && d0 < p.vdim) {
+          uint32_t pk[16];
 #pragma unroll
-        for (int i = 0; i < 16; ++i) pk[i] = pack_bf16x2(__uint_as_float(ov[2 * i]) * inv, __uint_as_float(ov[2 * i + 1]) * inv);
-        __nv_bfloat16* o = orow + static_cast<int64_t>(c) * p.vdim + d0;
-        if (p.wide_store && d0 + 32 <= p.vdim) {       // whole sectors
-          store32(o, pk);
-          store32(o + 16, pk + 8);
-        } else {
+          for (int i = 0; i < 16; ++i) pk[i] = pack_bf16x2(__uint_as_float(ov[2 * i]) * inv, __uint_as_float(ov[2 * i + 1]) * inv);
+          __nv_bfloat16* o = orow + static_cast<int64_t>(c) * p.vdim + d0;
+          if (p.wide_store && d0 + 32 <= p.vdim) {       // whole sectors
+            store32(o, pk);
+            store32(o + 16, pk + 8);
+          } else {
 #pragma unroll
-          for (int g = 0; g < 4; ++g)
-            if (d0 + g * 8 < p.vdim) *reinterpret_cast<uint4*>(o + g * 8) = make_uint4(pk[4 * g], pk[4 * g + 1], pk[4 * g + 2], pk[4 * g + 3]);
+            for (int g = 0; g < 4; ++g)
+              if (d0 + g * 8 < p.vdim) *reinterpret_cast<uint4*>(o + g * 8) = make_uint4(pk[4 * g], pk[4 * g + 1], pk[4 * g + 2], pk[4 * g + 3]);
+          }
         }
+        __syncwarp();
       }
       tc_fence_before_sync();
       __syncwarp();
